@@ -616,8 +616,54 @@ __global__ void swiglu_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat1
 // Tick logit post-processing.  Per row r:
 //   cum[r] = depth[r] > 0 ? cum[r] + logits[r] : logits[r]      (bf16 add, like the model's
 //   additive logit update), and argmax over cum[r] -> best[r] (lowest index wins ties).
-// One CTA of 1024 threads per row.
+// One CTA of 1024 threads per row.  logits_post_f32_kernel is the fp32 form without the vector loads.
 // ---------------------------------------------------------------------------------------------
+// block-wide arg-max of (value desc, index asc); thread 0 stores it
+__device__ __forceinline__ void store_block_argmax(float bv, int bi, int r, int* best, float* best_val) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+  }
+  __shared__ float sv[32];
+  __shared__ int si[32];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (lane == 0) { sv[warp] = bv; si[warp] = bi; }
+  __syncthreads();
+  if (warp == 0) {
+    bv = sv[lane];
+    bi = si[lane];
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+    }
+    if (lane == 0) {
+      best[r] = bi;
+      if (best_val != nullptr) best_val[r] = bv;   // lets a vocabulary-parallel caller merge shards
+    }
+  }
+}
+
+__global__ void __launch_bounds__(1024) logits_post_f32_kernel(const float* __restrict__ logits, float* __restrict__ cum,
+                                                               const int* __restrict__ depth, int* __restrict__ best,
+                                                               float* __restrict__ best_val, int V, long long ld_logits,
+                                                               long long ld_cum) {
+  const int r = blockIdx.x;
+  const bool add = depth != nullptr && depth[r] > 0;
+  float bv = -INFINITY;
+  int bi = 0x7fffffff;
+  for (int i = threadIdx.x; i < V; i += blockDim.x) {
+    float v = logits[(size_t)r * ld_logits + i];
+    if (add) v += cum[(size_t)r * ld_cum + i];
+    cum[(size_t)r * ld_cum + i] = v;
+    if (v > bv || (v == bv && i < bi)) { bv = v; bi = i; }
+  }
+  store_block_argmax(bv, bi, r, best, best_val);
+}
+
 __global__ void __launch_bounds__(1024) logits_post_kernel(const __nv_bfloat16* __restrict__ logits,
                                                            __nv_bfloat16* __restrict__ cum,
                                                            const int* __restrict__ depth, int* __restrict__ best,
@@ -652,32 +698,7 @@ __global__ void __launch_bounds__(1024) logits_post_kernel(const __nv_bfloat16* 
     cr[i] = __float2bfloat16_rn(v);
     if (v > bv || (v == bv && i < bi)) { bv = v; bi = i; }
   }
-  // block argmax (value desc, index asc)
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-    if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
-  }
-  __shared__ float sv[32];
-  __shared__ int si[32];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (lane == 0) { sv[warp] = bv; si[warp] = bi; }
-  __syncthreads();
-  if (warp == 0) {
-    bv = sv[lane];
-    bi = si[lane];
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
-    }
-    if (lane == 0) {
-      best[r] = bi;
-      if (best_val != nullptr) best_val[r] = bv;   // lets a vocabulary-parallel caller merge shards
-    }
-  }
+  store_block_argmax(bv, bi, r, best, best_val);
 }
 
 static unsigned long long g_peer_wait_limit_ns = WAIT_TIMEOUT_NS;
@@ -842,6 +863,13 @@ extern "C" int tahb_swiglu(const void* gu, void* out, int M, int I, long long ld
   else
     swiglu_kernel<<<blocks, 256, 0, stream>>>(reinterpret_cast<const __nv_bfloat16*>(gu),
                                               reinterpret_cast<__nv_bfloat16*>(out), M, I, ld_in, ld_out);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+extern "C" int tahb_logits_post_f32(const float* logits, float* cum, const int* depth, int* best, float* best_val, int M,
+                                    int V, long long ld_logits, long long ld_cum, cudaStream_t stream) {
+  if (M <= 0) return 0;
+  logits_post_f32_kernel<<<M, 1024, 0, stream>>>(logits, cum, depth, best, best_val, V, ld_logits, ld_cum);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 

@@ -1,0 +1,326 @@
+// Kernels of decoders that keep the residual stream in fp32 (independent of the activation type T, bf16 or fp32):
+//
+//   embed_norm      x = scale * E[token];                     h = T(rms(x) * w)
+//   residual_norm   x += rms(y) * w_out;                      h = T(rms(x) * w_next)
+//
+// with rms(v) = v / sqrt(mean(v^2) + eps).  residual_norm is the whole seam between two sublayers of a layer with a norm
+// before and after each sublayer: y is the sublayer's output projection, w_out the product of the output norm's weight
+// and the layer scale, w_next the weight of the norm that feeds the next projection.
+//
+// Rows are padded: `ld` columns (a multiple of 64) of which the first `width` are real; padding columns of every operand
+// are zero, so only the mean knows the difference.
+//
+//   few_linear      z[t, f] = x[t, :] . w[f, :] + b[f] in fp32 for a handful of features (gate pre-activations that
+//                   enter a recurrence), where a GEMM with a 16-bit output would round them
+//   gemm_f32        plain fp32 matrix product for the 32-bit mode
+#include "common.cuh"
+
+namespace tahb {
+
+template <typename T> struct Vec4;
+template <> struct Vec4<float> {
+  static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
+  static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+};
+template <> struct Vec4<__nv_bfloat16> {
+  static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
+    uint2 u;
+    *reinterpret_cast<__nv_bfloat162*>(&u.x) = __floats2bfloat162_rn(v.x, v.y);
+    *reinterpret_cast<__nv_bfloat162*>(&u.y) = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = u;
+  }
+};
+
+constexpr int RN_THREADS = 128;
+
+__device__ __forceinline__ float block_sum_128(float v, float* red) {
+  v = warp_sum(v);
+  __syncthreads();                       // red may still be read from the previous use
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  return red[0] + red[1] + red[2] + red[3];
+}
+
+__device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+template <typename T, int VPT>
+__global__ void __launch_bounds__(RN_THREADS) embed_norm_kernel(const T* __restrict__ E, const int* __restrict__ tok,
+                                                                float scale, float* __restrict__ x,
+                                                                const float* __restrict__ w, T* __restrict__ h, int vocab,
+                                                                int width, int ld, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[4];
+  const size_t row = blockIdx.x;
+  const int id = min(max(tok[row], 0), vocab - 1);
+  const int nvec = ld / 4;
+  float4 v[VPT];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) {
+      v[i] = Vec4<T>::load(E + (size_t)id * ld + c * 4);
+      v[i].x *= scale; v[i].y *= scale; v[i].z *= scale; v[i].w *= scale;
+      ss += sq4(v[i]);
+      Vec4<float>::store(x + row * ld + c * 4, v[i]);
+    }
+  }
+  const float r = 1.0f / sqrtf(block_sum_128(ss, red) / (float)width + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) {
+      const float4 g = Vec4<float>::load(w + c * 4);
+      Vec4<T>::store(h + row * ld + c * 4, make_float4(v[i].x * r * g.x, v[i].y * r * g.y, v[i].z * r * g.z, v[i].w * r * g.w));
+    }
+  }
+}
+
+template <typename T, int VPT>
+__global__ void __launch_bounds__(RN_THREADS) residual_norm_kernel(const T* __restrict__ y, long long ldy,
+                                                                   float* __restrict__ x, const float* __restrict__ w_out,
+                                                                   const float* __restrict__ w_next, T* __restrict__ h,
+                                                                   int width, int ld, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[4];
+  const size_t row = blockIdx.x;
+  const int nvec = ld / 4;
+  float4 u[VPT], v[VPT];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) {
+      u[i] = Vec4<T>::load(y + row * ldy + c * 4);
+      v[i] = Vec4<float>::load(x + row * ld + c * 4);
+      ss += sq4(u[i]);
+    }
+  }
+  const float ry = 1.0f / sqrtf(block_sum_128(ss, red) / (float)width + eps);
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) {
+      const float4 g = Vec4<float>::load(w_out + c * 4);
+      v[i].x += u[i].x * ry * g.x; v[i].y += u[i].y * ry * g.y; v[i].z += u[i].z * ry * g.z; v[i].w += u[i].w * ry * g.w;
+      ss += sq4(v[i]);
+      Vec4<float>::store(x + row * ld + c * 4, v[i]);
+    }
+  }
+  const float rx = 1.0f / sqrtf(block_sum_128(ss, red) / (float)width + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) {
+      const float4 g = Vec4<float>::load(w_next + c * 4);
+      Vec4<T>::store(h + row * ld + c * 4, make_float4(v[i].x * rx * g.x, v[i].y * rx * g.y, v[i].z * rx * g.z, v[i].w * rx * g.w));
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
+// few_linear: grid (ceil(M / FL_TOK)); the rows of FL_TOK tokens sit in shared memory as fp32, one warp per feature and
+// step.  A weight row is read once per FL_TOK tokens.
+// ---------------------------------------------------------------------------------------------
+constexpr int FL_THREADS = 256;
+
+template <typename T, int TOK>
+__global__ void __launch_bounds__(FL_THREADS) few_linear_kernel(const T* __restrict__ x, long long ldx,
+                                                                const T* __restrict__ w, const float* __restrict__ b,
+                                                                float* __restrict__ out, int M, int K, int F) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float xs[];              // [TOK][K]
+  const int t0 = blockIdx.x * TOK, n = min(TOK, M - t0);
+  const int nvec = K / 4;
+  for (int i = threadIdx.x; i < TOK * nvec; i += FL_THREADS) {
+    const int r = i / nvec, c = i % nvec;
+    Vec4<float>::store(xs + r * K + c * 4,
+                       r < n ? Vec4<T>::load(x + (size_t)(t0 + r) * ldx + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f));
+  }
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int f = blockIdx.y * (FL_THREADS / 32) + warp; f < F; f += gridDim.y * (FL_THREADS / 32)) {
+    float acc[TOK];
+#pragma unroll
+    for (int r = 0; r < TOK; ++r) acc[r] = 0.f;
+    for (int c = lane; c < nvec; c += 32) {
+      const float4 wv = Vec4<T>::load(w + (size_t)f * K + c * 4);
+#pragma unroll
+      for (int r = 0; r < TOK; ++r) {
+        const float4 xv = Vec4<float>::load(xs + r * K + c * 4);
+        acc[r] += xv.x * wv.x + xv.y * wv.y + xv.z * wv.z + xv.w * wv.w;
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < TOK; ++r) {
+      const float s = warp_sum(acc[r]);
+      if (lane == 0 && r < n) out[(size_t)(t0 + r) * F + f] = s + (b != nullptr ? b[f] : 0.f);
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
+// out[M, F] = x[M, K] w[F, K]^T in fp32 (FMA units, no reduced-precision matrix mode): 64 x 64 tiles, 4 x 4 per thread.
+// ---------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ x, long long ldx,
+                                                       const float* __restrict__ w, long long ldw, float* __restrict__ out,
+                                                       long long ldo, int M, int F, int K) {
+  constexpr int BK = 16;
+  __shared__ float xs[BK][64 + 4], ws[BK][64 + 4];
+  const int t0 = blockIdx.y * 64, f0 = blockIdx.x * 64;
+  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  const int lr = tid >> 2, lc = (tid & 3) * 4;              // tile row, first of 4 columns this thread loads
+  float acc[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  for (int k0 = 0; k0 < K; k0 += BK) {
+    const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 xv = t0 + lr < M ? Vec4<float>::load(x + (size_t)(t0 + lr) * ldx + k0 + lc) : z;
+    const float4 wv = f0 + lr < F ? Vec4<float>::load(w + (size_t)(f0 + lr) * ldw + k0 + lc) : z;
+    __syncthreads();
+    xs[lc][lr] = xv.x; xs[lc + 1][lr] = xv.y; xs[lc + 2][lr] = xv.z; xs[lc + 3][lr] = xv.w;
+    ws[lc][lr] = wv.x; ws[lc + 1][lr] = wv.y; ws[lc + 2][lr] = wv.z; ws[lc + 3][lr] = wv.w;
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < BK; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&xs[k][ty * 4]);
+      const float4 b = *reinterpret_cast<const float4*>(&ws[k][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = t0 + ty * 4 + i, f = f0 + tx * 4 + j;
+      if (t < M && f < F) out[(size_t)t * ldo + f] = acc[i][j];
+    }
+}
+
+__global__ void swiglu_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, int M, int I, long long ld_in,
+                                  long long ld_out) {
+  const long long n = (long long)M * I;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / I, c = i % I;
+    const float g = gu[r * ld_in + c], u = gu[r * ld_in + I + c];
+    out[r * ld_out + c] = g / (1.0f + expf(-g)) * u;
+  }
+}
+
+template <typename T>
+static int embed_norm_launch(const void* E, const int* tok, float scale, float* x, const float* w, void* h, int M,
+                             int vocab, int width, int ld, float eps, cudaStream_t stream) {
+  const int need = (ld / 4 + RN_THREADS - 1) / RN_THREADS;
+  auto e = reinterpret_cast<const T*>(E);
+  auto o = reinterpret_cast<T*>(h);
+  cudaError_t rc;
+#define TAHB_EN(V_) rc = launch_chain(embed_norm_kernel<T, V_>, dim3(M), dim3(RN_THREADS), 0, stream, e, tok, scale, x, w, o, vocab, width, ld, eps)
+  if (need <= 1) TAHB_EN(1);
+  else if (need <= 2) TAHB_EN(2);
+  else if (need <= 4) TAHB_EN(4);
+  else if (need <= 8) TAHB_EN(8);
+  else if (need <= 16) TAHB_EN(16);
+  else return -2;
+#undef TAHB_EN
+  return rc == cudaSuccess ? 0 : -3;
+}
+
+template <typename T>
+static int residual_norm_launch(const void* y, long long ldy, float* x, const float* w_out, const float* w_next, void* h,
+                                int M, int width, int ld, float eps, cudaStream_t stream) {
+  const int need = (ld / 4 + RN_THREADS - 1) / RN_THREADS;
+  auto yy = reinterpret_cast<const T*>(y);
+  auto o = reinterpret_cast<T*>(h);
+  cudaError_t rc;
+#define TAHB_RN(V_) rc = launch_chain(residual_norm_kernel<T, V_>, dim3(M), dim3(RN_THREADS), 0, stream, yy, ldy, x, w_out, w_next, o, width, ld, eps)
+  if (need <= 1) TAHB_RN(1);
+  else if (need <= 2) TAHB_RN(2);
+  else if (need <= 4) TAHB_RN(4);
+  else if (need <= 8) TAHB_RN(8);
+  else if (need <= 16) TAHB_RN(16);
+  else return -2;
+#undef TAHB_RN
+  return rc == cudaSuccess ? 0 : -3;
+}
+
+template <typename T, int TOK>
+static int few_linear_launch(const void* x, long long ldx, const void* w, const float* b, float* out, int M, int K, int F,
+                             cudaStream_t stream) {
+  const size_t smem = (size_t)TOK * K * 4;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(few_linear_kernel<T, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+      return -10;
+    configured = true;
+  }
+  if (smem > 200 * 1024) return -2;
+  const dim3 grid((M + TOK - 1) / TOK, TOK == 1 ? (F + 7) / 8 : 1);
+  cudaError_t rc = launch_chain(few_linear_kernel<T, TOK>, grid, dim3(FL_THREADS), smem, stream,
+                                reinterpret_cast<const T*>(x), ldx, reinterpret_cast<const T*>(w), b, out, M, K, F);
+  return rc == cudaSuccess ? 0 : -3;
+}
+
+}  // namespace tahb
+
+using namespace tahb;
+
+extern "C" int tahb_embed_norm(const void* E, const int* tok, float scale, float* x, const float* w, void* h, int M,
+                               int vocab, int width, int ld, float eps, int f32, cudaStream_t stream) {
+  if (M <= 0) return 0;
+  if (ld % 4 || width > ld) return -1;
+  return f32 ? embed_norm_launch<float>(E, tok, scale, x, w, h, M, vocab, width, ld, eps, stream)
+             : embed_norm_launch<__nv_bfloat16>(E, tok, scale, x, w, h, M, vocab, width, ld, eps, stream);
+}
+
+extern "C" int tahb_residual_norm(const void* y, long long ldy, float* x, const float* w_out, const float* w_next, void* h,
+                                  int M, int width, int ld, float eps, int f32, cudaStream_t stream) {
+  if (M <= 0) return 0;
+  if (ld % 4 || ldy % 4 || width > ld) return -1;
+  return f32 ? residual_norm_launch<float>(y, ldy, x, w_out, w_next, h, M, width, ld, eps, stream)
+             : residual_norm_launch<__nv_bfloat16>(y, ldy, x, w_out, w_next, h, M, width, ld, eps, stream);
+}
+
+extern "C" int tahb_few_linear(const void* x, long long ldx, const void* w, const float* b, float* out, int M, int K, int F,
+                               int f32, cudaStream_t stream) {
+  if (M <= 0 || F <= 0) return 0;
+  if (K % 4 || ldx % 4) return -1;
+  const bool one = M <= 148 || (size_t)4 * K * 4 > 200 * 1024;
+  if (f32)
+    return one ? few_linear_launch<float, 1>(x, ldx, w, b, out, M, K, F, stream)
+               : few_linear_launch<float, 4>(x, ldx, w, b, out, M, K, F, stream);
+  return one ? few_linear_launch<__nv_bfloat16, 1>(x, ldx, w, b, out, M, K, F, stream)
+             : few_linear_launch<__nv_bfloat16, 4>(x, ldx, w, b, out, M, K, F, stream);
+}
+
+extern "C" int tahb_gemm_f32(const float* x, long long ldx, const float* w, long long ldw, float* out, long long ldo, int M,
+                             int F, int K, cudaStream_t stream) {
+  if (M <= 0 || F <= 0) return 0;
+  if (K % 16 || ldx % 4 || ldw % 4) return -1;
+  gemm_f32_kernel<<<dim3((F + 63) / 64, (M + 63) / 64), 256, 0, stream>>>(x, ldx, w, ldw, out, ldo, M, F, K);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+extern "C" int tahb_swiglu_f32(const float* gu, float* out, int M, int I, long long ld_in, long long ld_out,
+                               cudaStream_t stream) {
+  if (M <= 0) return 0;
+  long long blocks = ((long long)M * I + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  swiglu_f32_kernel<<<(int)blocks, 256, 0, stream>>>(gu, out, M, I, ld_in, ld_out);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}

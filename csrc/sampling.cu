@@ -596,6 +596,7 @@ __global__ void __launch_bounds__(128) tick_begin_kernel(const TickState s, cons
     }
     s.gate[r] = d > 0;
   }
+  if (x_in == nullptr) return;               // the caller gathers the embeddings itself
   const uint4* src = (d == 0) ? reinterpret_cast<const uint4*>(E + (size_t)s.tok[r] * H)
                               : reinterpret_cast<const uint4*>(soft + (size_t)r * H);
   uint4* dst = reinterpret_cast<uint4*>(x_in + (size_t)r * H);

@@ -1,0 +1,575 @@
+"""HybridEngine: decoders whose layers differ - windowed attention over the paged cache beside recurrent layers with a
+state per row - on an fp32 residual stream.
+
+One function, :meth:`HybridEngine._layers`, runs the layers for a packed set of tokens.  It serves
+
+* :meth:`step` - any mixture of prompt portions and single decoded tokens of different rows in one batch: the step
+  function of prefill, of request admission and of trace replay.  New keys and values go to the paged cache first and
+  attention reads the cache only, so where a prompt was cut, which pages a row holds and what else is in the batch do not
+  enter the arithmetic;
+* the decode tick - one token of every row, captured in a CUDA graph (:class:`tah_b200.engine.base.DecodeEngine`).
+
+Rows are cache rows: a row owns pages of the KV pool and one slot of the recurrent state.  ``admit`` / ``release`` hand
+them out.  Sizes are padded once, when the weights are laid out: matrix rows and columns to multiples of 64, head sizes
+to multiples of 8, with zeros that drop out of every result.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import List, Optional, Sequence
+
+import torch
+
+from tah_b200.engine.base import DecodeEngine
+from tah_b200.engine.kv_cache import CacheGeometry, LayerKV, PagedKVCache, RecurrentState
+from tah_b200.models.gunuvik import AttentionSpec, GunuvikForCausalLM, MLSTMSpec
+from tah_b200.ops import cuda as K
+from tah_b200.utils.observe import nvtx_range
+
+NO_WINDOW = 2 ** 31 - 1
+
+
+def _pad(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+def distance_table(rel: torch.Tensor, far: int) -> torch.Tensor:
+    """``[heads, far + 1]`` fp32 bias by distance from a bucket table ``rel [rows, heads]``: distance ``n`` below
+    ``half = rows // 2`` has a row of its own; larger ones share rows logarithmically up to ``far``, from where the last
+    row serves.  The bucket's floor is evaluated in integers (``(far / half) ** k <= (n / half) ** (rows - half)``)."""
+    rows = rel.shape[0]
+    half = rows // 2
+    if far <= half:
+        raise ValueError(f"distance bias: the far end {far} lies inside the {half} exact distances")
+    m, k, idx = rows - half, 0, []
+    for n in range(far + 1):
+        if n < half:
+            idx.append(n)
+            continue
+        while k < m and far ** (k + 1) * half ** (m - k - 1) <= n ** m:
+            k += 1
+        idx.append(min(rows - 1, half + k))
+    return rel.float()[torch.tensor(idx, device=rel.device)].t().contiguous()
+
+
+@dataclass
+class AttentionLayer:
+    spec: AttentionSpec
+    dk: int
+    dv: int
+    nkv: int                      # heads this layer writes (0: it reads another layer's cache)
+    w_in: torch.Tensor            # rows: queries, own keys, own values, gate numbers
+    b_in: torch.Tensor
+    gate_col: int
+    q_norm: torch.Tensor
+    k_norm: Optional[torch.Tensor]
+    bias: torch.Tensor            # [heads, far + 1]
+    sink: torch.Tensor
+    w_o: torch.Tensor
+
+
+@dataclass
+class MemoryLayer:
+    spec: MLSTMSpec
+    dk: int
+    dv: int
+    w_in: torch.Tensor            # rows: q, k, v, output gate
+    w_if: torch.Tensor            # input and forget gate rows
+    b_if: torch.Tensor
+    norm: torch.Tensor
+    w_o: torch.Tensor
+
+
+@dataclass
+class BlockWeights:
+    mixer: object
+    norm1: torch.Tensor
+    out1: torch.Tensor            # output norm weight x layer scale
+    norm2: Optional[torch.Tensor] = None
+    out2: Optional[torch.Tensor] = None
+    w_gu: Optional[torch.Tensor] = None
+    w_down: Optional[torch.Tensor] = None
+
+
+class HybridWeights:
+    """Kernel-ready layout of a Gunuvik model's weights in the activation type ``dtype``."""
+
+    def __init__(self, model: GunuvikForCausalLM, dtype: torch.dtype):
+        cfg = model.config
+        dev = model.device
+        self.W, self.Wp = cfg.hidden_size, _pad(cfg.hidden_size, 64)
+        self.vocab = cfg.vocab_size
+        self.vocab_shard = (0, self.vocab, _pad(self.vocab, 64))
+        T = model.tensor
+
+        def vec(t, n):                                       # fp32 vector padded to n
+            o = torch.zeros(n, dtype=torch.float32, device=dev)
+            o[:t.numel()] = t.float()
+            return o
+
+        def heads_rows(w, h, d, dp):                         # [h * d, W] -> [h * dp, Wp]
+            o = torch.zeros(h, dp, self.Wp, dtype=dtype, device=dev)
+            o[:, :d, :w.shape[1]] = w.view(h, d, -1)
+            return o.view(h * dp, self.Wp)
+
+        def heads_vec(b, h, d, dp):
+            o = torch.zeros(h, dp, dtype=torch.float32, device=dev)
+            o[:, :d] = b.float().view(h, d)
+            return o.view(-1)
+
+        def heads_cols(w, h, d, dp):                         # [W, h * d] -> [Wp, pad64(h * dp)]
+            o = torch.zeros(self.Wp, _pad(h * dp, 64), dtype=dtype, device=dev)
+            o[:w.shape[0], :h * dp].view(w.shape[0], h, dp)[:, :, :d] = w.view(w.shape[0], h, d)
+            return o
+
+        def mat(w, rows, cols):
+            o = torch.zeros(rows, cols, dtype=dtype, device=dev)
+            o[:w.shape[0], :w.shape[1]] = w
+            return o
+
+        def stack(parts):                                    # row blocks, padded to a multiple of 64 rows
+            n = sum(p.shape[0] for p in parts)
+            return mat(torch.cat(parts), _pad(n, 64), self.Wp)
+
+        self.embed = mat(T("embed"), self.vocab, self.Wp)
+        self.head = mat(T("head"), self.vocab_shard[2], self.Wp)
+        self.final_norm = vec(T("final.norm"), self.Wp)
+        self.layers: List[BlockWeights] = []
+        for i, l in enumerate(cfg.layers):
+            p, m = f"l{i}.", l.mixer
+            x = p + "mix."
+            dk, dv = _pad(m.dim, 8), _pad(m.vdim, 8)
+            w_o = heads_cols(T(x + "o"), m.heads, m.vdim, dv)
+            if isinstance(m, AttentionSpec):
+                if max(dk, dv) > 256:
+                    raise NotImplementedError("attention head sizes above 256")
+                H, G = m.heads, m.kv_heads
+                rows = [heads_rows(T(x + "q"), H, m.dim, dk)]
+                bias = [heads_vec(T(x + "q.b"), H, m.dim, dk)]
+                own = m.kv_from is None
+                if own:
+                    rows += [heads_rows(T(x + "k"), G, m.dim, dk), heads_rows(T(x + "v"), G, m.vdim, dv)]
+                    bias += [heads_vec(T(x + "k.b"), G, m.dim, dk), heads_vec(T(x + "v.b"), G, m.vdim, dv)]
+                gate_col = sum(r.shape[0] for r in rows)
+                w_in = stack(rows + [heads_rows(T(x + "g"), H, 1, 1)])
+                mixer = AttentionLayer(m, dk, dv, G if own else 0, w_in, vec(torch.cat(bias), w_in.shape[0]), gate_col,
+                                       vec(T(x + "q.norm"), dk), vec(T(x + "k.norm"), dk) if own else None,
+                                       distance_table(T(x + "rel"), m.bias_max), vec(T(x + "sink"), H), w_o)
+            else:
+                if max(dk, dv) > 1024:
+                    raise NotImplementedError("mLSTM head sizes above 1024")
+                H = m.heads
+                w_in = stack([heads_rows(T(x + "q"), H, m.dim, dk), heads_rows(T(x + "k"), H, m.dim, dk),
+                              heads_rows(T(x + "v"), H, m.vdim, dv), heads_rows(T(x + "g"), H, m.vdim, dv)])
+                w_if = mat(torch.cat([T(x + "i"), T(x + "f")]), 2 * H, self.Wp)
+                mixer = MemoryLayer(m, dk, dv, w_in, w_if, torch.cat([T(x + "i.b"), T(x + "f.b")]).float(),
+                                    heads_vec(T(x + "norm"), H, m.vdim, dv), w_o)
+            b = BlockWeights(mixer, vec(T(p + "norm1"), self.Wp), vec(T(p + "norm1b").float() * T(p + "ls1").float(), self.Wp))
+            if l.ff is not None:
+                Ip = _pad(l.ff, 64)
+                gu = torch.cat([mat(T(p + "mlp.gate"), Ip, self.Wp), mat(T(p + "mlp.up"), Ip, self.Wp)])
+                b.w_gu = K.interleave_gate_up(gu) if dtype == torch.bfloat16 else gu
+                b.w_down = mat(T(p + "mlp.down"), self.Wp, Ip)
+                b.norm2 = vec(T(p + "norm2"), self.Wp)
+                b.out2 = vec(T(p + "norm2b").float() * T(p + "ls2").float(), self.Wp)
+            self.layers.append(b)
+
+
+class _Plan:
+    """Which tokens a pass runs: packed token ids, positions, cache rows and KV slots.  The first ``n_dec`` tokens are
+    single tokens of a row each; behind them lie the prompt portions, portion ``e`` at ``seq_start[e]``,
+    ``seq_len[e]`` tokens long, cut into query tiles of up to 128 tokens."""
+    tok = pos = row = slot = None
+    n_dec = 0
+    seq_start = seq_len = None
+    tile_q0 = tile_qn = None
+    n_split = 1
+    ws = None
+
+
+class _Buffers:
+    """Activations of a pass over ``n`` tokens."""
+
+    def __init__(self, w: HybridWeights, n: int, dtype, dev):
+        e = lambda *s: torch.empty(*s, dtype=dtype, device=dev)
+        mix = [b.mixer for b in w.layers]
+        self.x = torch.empty(n, w.Wp, dtype=torch.float32, device=dev)
+        self.h, self.y = e(n, w.Wp), e(n, w.Wp)
+        self.proj = e(n, max(m.w_in.shape[0] for m in mix))
+        self.q = e(n, max([m.spec.heads * m.dk for m in mix if isinstance(m, AttentionLayer)] or [0]))
+        # columns between heads * dv and the padded width meet zero weight columns; they only have to be finite
+        self.o = torch.zeros(n, max(m.w_o.shape[1] for m in mix), dtype=dtype, device=dev)
+        self.gates = torch.empty(n * max([m.w_if.shape[0] for m in mix if isinstance(m, MemoryLayer)] or [0]),
+                                 dtype=torch.float32, device=dev)
+        self.act = e(n, max([b.w_down.shape[1] for b in w.layers if b.w_down is not None] or [0]))
+
+
+@dataclass
+class StepEntry:
+    """One row's part of a step: its next tokens and the places among them whose logits are wanted."""
+    row: int
+    tokens: Sequence[int]
+    want: Sequence[int] = ()
+
+
+class HybridEngine(DecodeEngine):
+    def __init__(self, model: GunuvikForCausalLM, max_rows: int = 64, max_seq_len: int = 2048, page_size: int = 16,
+                 use_cuda_graph: bool = True, prefill_tokens: int = 16384):
+        """``prefill_tokens``: the most prompt tokens one step runs (longer prompts are cut into portions)."""
+        self.model, self.cfg = model, model.config
+        self.device = model.device
+        if self.device.type != "cuda":
+            raise RuntimeError("HybridEngine needs the model on a CUDA device")
+        self.dtype = model.dtype
+        if self.dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError(f"HybridEngine runs in bfloat16 or float32, not {self.dtype}")
+        self.max_iter, self.topk, self.tp = 1, 1, None
+        self.w = HybridWeights(model, self.dtype)
+        self.prefill_tokens = prefill_tokens
+        self.state: Optional[RecurrentState] = None
+        self._free_rows: List[int] = []
+        self.layer_hook = None                     # optional callable(layer index, residual stream) after every layer
+        self._init_scheduler(max_rows, max_seq_len, page_size, use_cuda_graph)
+
+    # ------------------------------------------------------------------------------------------
+    # cache, state, rows
+    # ------------------------------------------------------------------------------------------
+    def _new_cache(self, rows: int, max_tokens: int, pool_tokens: Optional[int] = None) -> None:
+        kv, st = [], []
+        for b in self.w.layers:
+            m = b.mixer
+            if isinstance(m, AttentionLayer):
+                kv.append(LayerKV(shared_with=m.spec.kv_from) if m.nkv == 0 else LayerKV(m.nkv, m.dk, m.dv))
+                st.append(None)
+            else:
+                kv.append(None)
+                st.append([(m.spec.heads, m.dk, m.dv), (m.spec.heads, m.dk), (m.spec.heads,)])
+        self.kv = self.state = None
+        self._states.clear()                       # captured ticks point into the old pools
+        torch.cuda.empty_cache()
+        self.kv = PagedKVCache(CacheGeometry.per_layer(kv, self.page_size), rows, max_tokens, 1, device=self.device,
+                               dtype=self.dtype, pool_tokens=pool_tokens)
+        self.state = RecurrentState(st, rows, self.device)
+        self._free_rows = list(range(rows - 1, -1, -1))
+
+    def open(self, rows: int, pool_tokens: int, max_tokens_per_row: Optional[int] = None) -> None:
+        """Make the cache for ``rows`` live requests that together hold at most ``pool_tokens`` tokens (each request's
+        count rounded up to whole pages), for use with :meth:`admit` / :meth:`step` / :meth:`release`."""
+        self._new_cache(rows, max_tokens_per_row or pool_tokens, pool_tokens)
+
+    def admit(self) -> int:
+        """A free row for a new request."""
+        if not self._free_rows:
+            raise RuntimeError("no free row: every row holds a request")
+        return self._free_rows.pop()
+
+    def release(self, row: int) -> None:
+        """The request of ``row`` is finished: its pages and its state slot may be used again."""
+        self.kv.free_rows(torch.tensor([row], device=self.device))
+        self._free_rows.append(row)
+
+    # ------------------------------------------------------------------------------------------
+    # the layers
+    # ------------------------------------------------------------------------------------------
+    def _attention(self, li: int, m: AttentionLayer, b: _Buffers, plan: _Plan) -> torch.Tensor:
+        s = m.spec
+        n = b.h.shape[0]
+        proj = K.linear(b.h, m.w_in, out=b.proj[:, :m.w_in.shape[0]])
+        q = b.q.view(-1)[:n * s.heads * m.dk].view(n, s.heads * m.dk)
+        pool = self.kv.layer_pool(0, li)
+        K.qkv_post(proj, m.b_in, m.q_norm, m.k_norm, q, pool, plan.slot, s.heads, m.nkv, m.dk, m.dv, s.dim, self.page_size,
+                   self.cfg.rms_norm_eps)
+        o = b.o[:, :m.w_o.shape[1]]
+        kw = dict(nq=s.heads, nkv=s.kv_heads, dk=m.dk, dv=m.dv, page_size=self.page_size, scale=s.scale,
+                  window=NO_WINDOW if s.window is None else s.window, keep_first=s.keep_first, bias=m.bias, sink=m.sink)
+        gate = proj[:, m.gate_col:m.gate_col + s.heads]
+        K.window_attn_plain(q, o, pool, self.kv.page_table[0], plan.pos, plan.row, gate=gate, **kw)
+        return o
+
+    def _memory(self, li: int, m: MemoryLayer, b: _Buffers, plan: _Plan) -> torch.Tensor:
+        s = m.spec
+        n, nd = b.h.shape[0], plan.n_dec
+        proj = K.linear(b.h, m.w_in, out=b.proj[:, :m.w_in.shape[0]])
+        gates = K.few_linear(b.h, m.w_if, m.b_if, out=b.gates[:n * m.w_if.shape[0]].view(n, -1))
+        o = b.o[:, :m.w_o.shape[1]]
+        kw = dict(heads=s.heads, dk=m.dk, dv=m.dv, dim=s.dim, vdim=s.vdim, cap=s.gate_cap, eps=self.cfg.rms_norm_eps)
+        state = self.state.layers[li]
+        if nd:
+            K.mlstm_recurrent(proj[:nd], gates[:nd], m.norm, o[:nd], state, plan.pos, plan.row, slot=plan.slot, **kw)
+        if nd < n:
+            K.mlstm_recurrent(proj, gates, m.norm, o, state, plan.pos, plan.row, seq_start=plan.seq_start,
+                              seq_len=plan.seq_len, **kw)
+        return o
+
+    def _layers(self, b: _Buffers, plan: _Plan) -> torch.Tensor:
+        """Run every layer on the packed tokens of ``plan`` (``b.x`` / ``b.h`` hold their embeddings and first normed
+        input); returns the final-norm output."""
+        w, eps = self.w, self.cfg.rms_norm_eps
+        n_layers = len(w.layers)
+        for li, L in enumerate(w.layers):
+            run = self._attention if isinstance(L.mixer, AttentionLayer) else self._memory
+            K.linear(run(li, L.mixer, b, plan), L.mixer.w_o, out=b.y)
+            after = w.layers[li + 1].norm1 if li + 1 < n_layers else w.final_norm
+            K.residual_norm(b.y, b.x, L.out1, L.norm2 if L.w_gu is not None else after, w.W, eps, b.h)
+            if L.w_gu is not None:
+                act = K.swiglu_linear(b.h, L.w_gu, out=b.act[:, :L.w_down.shape[1]])
+                K.linear(act, L.w_down, out=b.y)
+                K.residual_norm(b.y, b.x, L.out2, after, w.W, eps, b.h)
+            if self.layer_hook is not None:
+                self.layer_hook(li, b.x[:, :w.W])
+        return b.h
+
+    # ------------------------------------------------------------------------------------------
+    # one step of portions and single tokens
+    # ------------------------------------------------------------------------------------------
+    @torch.no_grad()
+    def _run(self, rows: Sequence[int], counts: Sequence[int], tok: torch.Tensor, want: Sequence[int]) -> torch.Tensor:
+        """Append ``counts[e]`` tokens to row ``rows[e]`` for every entry and run them as one batch.  ``tok``: int32 token
+        ids of all entries back to back (device); ``want``: indices into ``tok`` whose logits are returned, in order."""
+        dev, n = self.device, int(tok.numel())
+        if len(set(rows)) != len(rows) or min(counts) < 1:
+            raise ValueError("a step needs distinct rows with at least one token each")
+        start, first = [], 0
+        for c in counts:
+            start.append(first)
+            first += c
+        order = [e for e, c in enumerate(counts) if c == 1] + [e for e, c in enumerate(counts) if c > 1]
+        n_dec = sum(1 for c in counts if c == 1)
+        if order != list(range(len(counts))):                    # single tokens first: move the packed tokens along
+            perm, place, new_start, at = [], [0] * n, [0] * len(counts), 0
+            for e in order:
+                new_start[e] = at
+                for t in range(counts[e]):
+                    place[start[e] + t] = at + t
+                    perm.append(start[e] + t)
+                at += counts[e]
+            tok = tok[torch.tensor(perm, device=dev)]
+            want = [place[i] for i in want]
+            start = new_start
+        rows, counts, start = [rows[e] for e in order], [counts[e] for e in order], [start[e] for e in order]
+        q0, qn = [], []
+        for s0, c in zip(start[n_dec:], counts[n_dec:]):
+            for a in range(0, c, 128):
+                q0.append(s0 + a)
+                qn.append(min(128, c - a))
+        ne, nt, nw = len(rows), len(q0), len(want)
+        meta = torch.tensor(rows + counts + start + q0 + qn + list(want), dtype=torch.int32).pin_memory().to(dev, non_blocking=True)
+        d_rows, d_counts, d_start, d_q0, d_qn, d_want = meta.split([ne, ne, ne, nt, nt, nw])
+        plan = _Plan()
+        plan.tok = tok
+        plan.pos, plan.row, plan.slot = (torch.empty(n, dtype=torch.int32, device=dev) for _ in range(3))
+        plan.n_dec = n_dec
+        plan.seq_start, plan.seq_len = d_start[n_dec:], d_counts[n_dec:]
+        plan.tile_q0, plan.tile_qn = d_q0, d_qn
+        K.kv_append(d_rows, d_counts, d_start, self.kv, 0, plan.pos, plan.row, plan.slot)
+        b = _Buffers(self.w, n, self.dtype, dev)
+        K.embed_norm(self.w.embed, plan.tok, self.cfg.embedding_scale, self.w.layers[0].norm1, self.w.W,
+                     self.cfg.rms_norm_eps, b.x, b.h)
+        h = self._layers(b, plan)
+        if nw == 0:
+            return torch.empty(0, self.w.vocab, dtype=self.dtype, device=dev)
+        return K.linear(h[d_want.long()], self.w.head)[:, :self.w.vocab]
+
+    def step(self, entries: Sequence[StepEntry]) -> torch.Tensor:
+        """Run the entries as one batch, from the cache and state that earlier steps left; returns the logits
+        ``[wanted, vocab]`` in the order of the entries and of their ``want``."""
+        toks, want, at = [], [], 0
+        for e in entries:
+            if any(not 0 <= w < len(e.tokens) for w in e.want):
+                raise ValueError("a wanted place lies outside the entry's tokens")
+            toks += list(e.tokens)
+            want += [at + w for w in e.want]
+            at += len(e.tokens)
+        if any(not 0 <= t < self.w.vocab for t in toks):
+            raise ValueError("token id outside the vocabulary")
+        tok = torch.tensor(toks, dtype=torch.int32).to(self.device)
+        with nvtx_range("engine/step"):
+            return self._run([e.row for e in entries], [len(e.tokens) for e in entries], tok, want)
+
+    # ------------------------------------------------------------------------------------------
+    # prefill / decode tick for generate() and serve()
+    # ------------------------------------------------------------------------------------------
+    @torch.no_grad()
+    def prefill(self, input_ids: torch.Tensor, attention_mask: Optional[torch.Tensor], max_new_tokens: int,
+                row_ids: Optional[torch.Tensor] = None):
+        """Run a batch of prompts (left- or right-padded) in steps of at most ``prefill_tokens`` tokens.  Without
+        ``row_ids`` the cache is (re)built for exactly this batch; with it the prompts go into those empty rows."""
+        dev = self.device
+        B, T = input_ids.shape
+        valid = attention_mask[:, -T:].bool() if attention_mask is not None else torch.ones(B, T, dtype=torch.bool, device=dev)
+        lens = valid.sum(1)
+        host_lens = lens.tolist()
+        max_total = max(host_lens) + max_new_tokens + 1
+        fits = self.kv is not None and self.kv.max_pages[0] * self.page_size >= max_total
+        if row_ids is not None:
+            if not fits:
+                raise RuntimeError("admission needs an existing KV cache whose rows can hold prompt + new tokens")
+        else:
+            if not fits or self.kv.rows != B or self.kv.n_pages[0] < B * self.kv.max_pages[0]:
+                self._new_cache(B, max_total)
+            self.kv.reset()
+        rows = list(range(B)) if row_ids is None else [int(r) for r in row_ids.tolist()]
+        packed = input_ids[valid].to(torch.int32).contiguous()
+        last: List[Optional[torch.Tensor]] = [None] * B
+        portion_rows, portion_counts, ends, used, at = [], [], [], 0, 0
+
+        def flush():
+            nonlocal at
+            if not portion_rows:
+                return
+            want, first = [], 0
+            for r, c, e in zip(portion_rows, portion_counts, ends):
+                first += c
+                if e:
+                    want.append(first - 1)
+            lg = self._run([rows[r] for r in portion_rows], list(portion_counts), packed[at:at + first], want)
+            for j, r in enumerate(r for r, e in zip(portion_rows, ends) if e):
+                last[r] = lg[j]
+            at += first
+            portion_rows.clear(), portion_counts.clear(), ends.clear()
+
+        for r, n in enumerate(host_lens):
+            done = 0
+            while done < n:
+                c = min(n - done, self.prefill_tokens - used)
+                portion_rows.append(r)
+                portion_counts.append(c)
+                done += c
+                ends.append(done == n)
+                used += c
+                if used == self.prefill_tokens or len(portion_rows) == K.APPEND_MAX_ENTRIES:
+                    flush()
+                    used = 0
+        flush()
+        out = torch.empty(B, self.w.vocab_shard[2], dtype=self.dtype, device=dev)[:, :self.w.vocab]
+        out.copy_(torch.stack(last))
+        return out, lens, None
+
+    def _alloc_tick_buffers(self, B: int, max_new: int):
+        s = self._alloc_scheduler_state(B, max_new)
+        dev = self.device
+        s.buf = _Buffers(self.w, B, self.dtype, dev)
+        s.plan = _Plan()
+        s.plan.tok, s.plan.pos, s.plan.slot = s.tok, s.pos, s.slot
+        s.plan.row = torch.arange(B, dtype=torch.int32, device=dev)
+        s.plan.n_dec = B
+        z = lambda dt: torch.zeros(B, self.w.vocab_shard[2], dtype=dt, device=dev)
+        s.logits, s.cum = z(self.dtype), z(self.dtype)
+        s.cum16 = s.cum if self.dtype == torch.bfloat16 else z(torch.bfloat16)
+        return s
+
+    def _tick(self, s, sampling):
+        """Enqueue one decode tick on the current stream (graph-capturable)."""
+        w = self.w
+        s.binding.tick_begin(None, None, None)
+        K.embed_norm(w.embed, s.tok, self.cfg.embedding_scale, w.layers[0].norm1, w.W, self.cfg.rms_norm_eps, s.buf.x, s.buf.h)
+        K.linear(self._layers(s.buf, s.plan), w.head, out=s.logits)
+        V = w.vocab
+        K.logits_post(s.logits[:, :V], s.cum[:, :V], None, s.best, s.best_val)
+        if sampling is not None and self.dtype != torch.bfloat16:
+            s.cum16.copy_(s.cum)                      # the samplers take bf16 logits
+        s.binding.tick_end(s.need_soft, self._pick_next(s, s.cum16[:, :V], sampling))
+
+    # ------------------------------------------------------------------------------------------
+    # serving: prompt portions ride along with the decoding rows
+    # ------------------------------------------------------------------------------------------
+    @torch.no_grad()
+    def serve(self, prompts: Sequence[torch.Tensor], *, max_new_tokens: int = 128, rows: Optional[int] = None,
+              eos_token_id: Optional[int] = None, do_sample: bool = False, temperature: float = 1.0, top_p: float = 1.0,
+              top_k: int = 0, min_p: float = 0.0, seed: Optional[int] = None, check_every: int = 16, portion: int = 2048):
+        """Continuous batching over a queue of requests (1-D token id tensors of any lengths).
+
+        While a prompt is being read its portions (at most ``portion`` prompt tokens a step) share mixed steps with the
+        decoding rows, one token each, so admission never stalls them; when no prompt is pending the rows advance by
+        captured decode ticks, ``check_every`` at a time.  A finished row hands back its tokens, its pages and its state
+        slot.  Returns the generated token lists in request order and a statistics dict."""
+        dev = self.device
+        n_req = len(prompts)
+        B = min(rows or self.max_rows, n_req, self.max_rows)
+        lens = [int(p.numel()) for p in prompts]
+        if min(lens) < 1:
+            raise ValueError("serve: an empty prompt")
+        need = max(lens) + max_new_tokens + 1
+        sampling = None
+        if do_sample:
+            sampling = dict(temperature=float(temperature), top_p=float(top_p), min_p=float(min_p), top_k=int(top_k))
+            seed = int(torch.randint(0, 2 ** 62, (1,)).item()) if seed is None else int(seed)
+        if self.kv is None or self.kv.rows != B or self.kv.max_pages[0] * self.page_size < need or \
+                self.kv.n_pages[0] < B * self.kv.max_pages[0]:
+            self._new_cache(B, need)
+        self.kv.reset()
+        self._calls += 1
+        s = self._tick_state(B, max_new_tokens, sampling, eos_token_id)
+        if sampling is not None:
+            s.seed_dev.fill_(seed & (2 ** 62 - 1))
+        s.finished.fill_(1)                                  # idle rows are frozen for the tick kernels
+        if self.use_cuda_graph and s.graph is None:
+            self._tick(s, sampling)                          # lazy one-time kernel setup outside capture; no row is live
+        run = self._tick_runner(s, sampling)
+        owner, read, queue = [-1] * B, [0] * B, 0            # request of a row, prompt tokens read
+        ids = [p.to(device=dev, dtype=torch.int32).flatten() for p in prompts]
+        results: List[Optional[List[int]]] = [None] * n_req
+        stats = {"ticks": 0, "mixed_steps": 0, "admitted": 0, "rows": B, "peak_pages": [0], "pages_released": 0}
+        while True:
+            done = ((s.finished != 0) | (s.n_out >= max_new_tokens)).tolist()
+            decoding = [r for r in range(B) if owner[r] >= 0 and read[r] == lens[owner[r]]]
+            fin = [r for r in decoding if done[r]]
+            if fin:
+                n_out = s.n_out.tolist()
+                for r, row_toks in zip(fin, s.out_tokens[fin].tolist()):
+                    results[owner[r]] = row_toks[:n_out[r]]
+                    owner[r] = -1
+                fin_t = torch.tensor(fin, device=dev)
+                s.finished[fin_t] = 1
+                stats["pages_released"] += self.kv.free_rows(fin_t)
+                decoding = [r for r in decoding if not done[r]]
+            for r in range(B):
+                if owner[r] < 0 and queue < n_req:
+                    owner[r], read[r] = queue, 0
+                    queue += 1
+                    stats["admitted"] += 1
+            reading = [r for r in range(B) if owner[r] >= 0 and read[r] < lens[owner[r]]]
+            if not reading and not decoding:
+                break
+            if not reading:
+                for _ in range(check_every):
+                    run()
+                stats["ticks"] += check_every
+            else:
+                step_rows, counts, toks, finish = list(decoding), [1] * len(decoding), [], []
+                if decoding:
+                    toks.append(s.tok[torch.tensor(decoding, device=dev)])
+                left, at, want = portion, len(decoding), list(range(len(decoding)))
+                for r in reading:
+                    c = min(left, lens[owner[r]] - read[r])
+                    if c == 0 or len(step_rows) == K.APPEND_MAX_ENTRIES:
+                        break
+                    step_rows.append(r)
+                    counts.append(c)
+                    toks.append(ids[owner[r]][read[r]:read[r] + c])
+                    read[r] += c
+                    at += c
+                    left -= c
+                    if read[r] == lens[owner[r]]:
+                        finish.append(r)
+                        want.append(at - 1)
+                logits = self._run(step_rows, counts, torch.cat(toks), want)
+                stats["mixed_steps"] += 1
+                if want:
+                    where = torch.tensor(decoding + finish, device=dev)
+                    last = torch.cat([s.pos[where[:len(decoding)]],
+                                      torch.tensor([lens[owner[r]] - 1 for r in finish], dtype=torch.int32, device=dev)])
+                    nxt = self._choose(logits, last, sampling, seed or 0, None)
+                    if finish:                               # they emit their first token below, as a decoding row does
+                        f = where[len(decoding):]
+                        s.n_out[f], s.finished[f], s.depth[f], s.cur_iters[f], s.iter_sum[f] = 0, 0, 0, 0, 0
+                        s.out_tokens[f] = 0
+                        s.pos[f] = last[len(decoding):]
+                    s.best[where] = nxt
+                    s.need_soft.zero_()
+                    s.binding.tick_end(s.need_soft, s.best)
+            stats["peak_pages"][0] = max(stats["peak_pages"][0], self.kv.pages_in_use(0))
+        torch.cuda.synchronize()
+        K.check_status(dev)
+        stats["tokens"] = sum(len(r) for r in results)
+        return results, stats

@@ -9,15 +9,29 @@ depth->=1 slots over the whole batch.  Here each depth has a pool of fixed-size 
 and a row owns only the pages its real entries need; the depth->=1 pools hold hard-token
 entries only.  Free pages are handed out on the device (``free_stack``/``free_count``,
 popped by the tick kernel), so decode never returns to the host for memory.
+
+A model whose layers differ gives ``CacheGeometry.layers``: one :class:`LayerKV` per layer with its own K and V sizes, or
+``None`` for a layer without keys (a recurrent layer), or ``LayerKV(shared_with=j)`` for a layer that reads the cache of
+layer ``j``.  All layers share one page table; the pool of a layer is then a tensor of its own with the same page layout
+``[K: kv_heads, page_size, k_dim][V: kv_heads, page_size, v_dim]``.  What recurrent layers carry from token to token
+lives beside the pages in :class:`RecurrentState`, one slot per cache row.
 """
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import List
+from typing import List, Optional, Sequence, Tuple
 
 import os
 
 import torch
+
+
+@dataclass
+class LayerKV:
+    kv_heads: int = 0
+    k_dim: int = 0
+    v_dim: int = 0
+    shared_with: Optional[int] = None     # the layer whose pool this layer reads
 
 
 @dataclass
@@ -26,6 +40,16 @@ class CacheGeometry:
     n_kv_heads: int
     head_dim: int
     page_size: int = 16
+    layers: Optional[List[Optional[LayerKV]]] = None
+
+    @classmethod
+    def per_layer(cls, layers: Sequence[Optional[LayerKV]], page_size: int = 16) -> "CacheGeometry":
+        for i, l in enumerate(layers):
+            if l is not None and l.shared_with is not None:
+                j = l.shared_with
+                if not 0 <= j < len(layers) or layers[j] is None or layers[j].shared_with is not None:
+                    raise ValueError(f"layer {i} shares the cache of layer {j}, which has none of its own")
+        return cls(len(layers), 0, 0, page_size, list(layers))
 
 
 GUARD_PATTERN = 0x5A5A          # int16 view of the bf16 guard pages
@@ -33,13 +57,15 @@ GUARD_PATTERN = 0x5A5A          # int16 view of the bf16 guard pages
 
 class PagedKVCache:
     def __init__(self, geo: CacheGeometry, rows: int, max_tokens_per_row: int, n_depths: int,
-                 deep_fraction: float = 0.25, device="cuda", dtype=torch.bfloat16):
+                 deep_fraction: float = 0.25, device="cuda", dtype=torch.bfloat16, pool_tokens: Optional[int] = None):
+        """``pool_tokens``: capacity of the depth-0 pool in tokens, when it is not ``rows * max_tokens_per_row`` (rows
+        then compete for pages)."""
         self.geo, self.rows, self.n_depths = geo, rows, n_depths
         self.page_size = geo.page_size
         ppr = (max_tokens_per_row + geo.page_size - 1) // geo.page_size + 1
         self.max_pages = [ppr] * n_depths
         self.n_pages: List[int] = []
-        self.pool: List[torch.Tensor] = []
+        self.pool: List = []              # per depth: one tensor, or with geo.layers a list with one tensor (or None) per layer
         self.page_table: List[torch.Tensor] = []
         self.len: List[torch.Tensor] = []
         self.free_stack: List[torch.Tensor] = []
@@ -49,12 +75,20 @@ class PagedKVCache:
         self.guard_pages = int(os.environ.get("TAH_B200_CANARY", "0") or 0)
         for d in range(n_depths):
             pages = rows * ppr if d == 0 else max(rows * 2, int(rows * ppr * deep_fraction))
+            if d == 0 and pool_tokens is not None:
+                pages = max(1, (pool_tokens + geo.page_size - 1) // geo.page_size)
             self.n_pages.append(pages)
-            pool = torch.zeros(geo.n_layers, pages + self.guard_pages, 2, geo.n_kv_heads, geo.page_size, geo.head_dim,
-                               dtype=dtype, device=device)
-            if self.guard_pages:
-                pool[:, pages:].view(torch.int16).fill_(GUARD_PATTERN)
+            if geo.layers is None:
+                pool = torch.zeros(geo.n_layers, pages + self.guard_pages, 2, geo.n_kv_heads, geo.page_size, geo.head_dim,
+                                   dtype=dtype, device=device)
+            else:
+                pool = [None if l is None or l.shared_with is not None else
+                        torch.zeros(pages + self.guard_pages, l.kv_heads * geo.page_size * (l.k_dim + l.v_dim), dtype=dtype,
+                                    device=device) for l in geo.layers]
             self.pool.append(pool)
+            if self.guard_pages:
+                for t in self._pools(d):
+                    t[..., pages:, :].view(torch.int16).fill_(GUARD_PATTERN)
             self.page_table.append(torch.zeros(rows, ppr, dtype=torch.int32, device=device))
             self.len.append(torch.zeros(rows, dtype=torch.int32, device=device))
             self.free_stack.append(torch.arange(pages, dtype=torch.int32, device=device))
@@ -64,10 +98,16 @@ class PagedKVCache:
         """True when every guard page still holds the pattern (always true without ``TAH_B200_CANARY``)."""
         if not self.guard_pages:
             return True
-        return all(bool((p[:, n:].view(torch.int16) == GUARD_PATTERN).all()) for p, n in zip(self.pool, self.n_pages))
+        return all(bool((t[..., n:, :].view(torch.int16) == GUARD_PATTERN).all())
+                   for d, n in enumerate(self.n_pages) for t in self._pools(d))
+
+    def _pools(self, depth: int) -> List[torch.Tensor]:
+        """The pool tensors of a depth as ``[..., pages, elements of a page]`` views."""
+        p = self.pool[depth]
+        return [p.flatten(2)] if self.geo.layers is None else [t for t in p if t is not None]
 
     def bytes(self) -> int:
-        return sum(p.numel() * p.element_size() for p in self.pool)
+        return sum(t.numel() * t.element_size() for d in range(self.n_depths) for t in self._pools(d))
 
     def reset(self) -> None:
         for d in range(self.n_depths):
@@ -77,6 +117,8 @@ class PagedKVCache:
             self.free_count[d].fill_(self.n_pages[d])
 
     def layer_pool(self, depth: int, layer: int) -> torch.Tensor:
+        if self.geo.layers is not None and self.geo.layers[layer].shared_with is not None:
+            layer = self.geo.layers[layer].shared_with
         return self.pool[depth][layer]
 
     def assign_prefill(self, depth: int, counts: torch.Tensor) -> torch.Tensor:
@@ -158,3 +200,17 @@ class PagedKVCache:
 
     def pages_in_use(self, depth: int) -> int:
         return self.n_pages[depth] - int(self.free_count[depth])
+
+
+class RecurrentState:
+    """fp32 state that recurrent layers carry from token to token: for each layer a tuple of tensors whose first
+    dimension is the cache row (a row's slot is its row number).  Kernels start a sequence from zeros at position 0, so a
+    row that changes hands needs no clearing."""
+
+    def __init__(self, shapes: Sequence[Optional[Sequence[Tuple[int, ...]]]], rows: int, device="cuda"):
+        self.rows = rows
+        self.layers = [None if sh is None else tuple(torch.zeros(rows, *s, dtype=torch.float32, device=device) for s in sh)
+                       for sh in shapes]
+
+    def bytes(self) -> int:
+        return sum(t.numel() * 4 for l in self.layers if l is not None for t in l)

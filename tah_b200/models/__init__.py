@@ -1,6 +1,9 @@
-"""Backbone model families (Qwen3 0.6B / 1.7B / 4B shapes and the tiny test model)."""
+"""Model families: the Qwen3 backbone of TaH (0.6B / 1.7B / 4B shapes and the tiny test model) and Gunuvik."""
+from tah_b200.models.gunuvik import GunuvikConfig, GunuvikForCausalLM, gunuvik_preset
 from tah_b200.models.qwen3 import (PRESETS, LoRASpec, Qwen3Config, Qwen3ForCausalLM, attach_lora,
                                    export_hf_state_dict, from_hf_model, import_hf_state_dict, preset)
+from tah_b200.models.registry import load_model, make_engine, register_family
 
-__all__ = ["PRESETS", "LoRASpec", "Qwen3Config", "Qwen3ForCausalLM", "attach_lora", "export_hf_state_dict",
-           "from_hf_model", "import_hf_state_dict", "preset"]
+__all__ = ["PRESETS", "LoRASpec", "Qwen3Config", "Qwen3ForCausalLM", "attach_lora",
+           "export_hf_state_dict", "from_hf_model", "import_hf_state_dict", "preset",
+           "GunuvikConfig", "GunuvikForCausalLM", "gunuvik_preset", "load_model", "make_engine", "register_family"]

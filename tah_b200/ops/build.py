@@ -25,8 +25,13 @@ FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std
 FLAGS.remove("--use_fast_math")
 
 
-def _sources():
-    return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cu"))
+# sources of the smaller libraries that a process may build instead of the whole one
+GROUPS = {"decoder": ("gemm_tcgen05", "elementwise", "sampling", "residual_norm", "attn_window", "mlstm")}
+
+
+def _sources(group=None):
+    return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC)
+                  if f.endswith(".cu") and (group is None or f[:-3] in GROUPS[group]))
 
 
 def _hash(path: str) -> str:
@@ -38,12 +43,14 @@ def _hash(path: str) -> str:
     return h.hexdigest()[:16]
 
 
-def build(verbose: bool = False, force: bool = False) -> str:
+def build(verbose: bool = False, force: bool = False, group=None) -> str:
+    """Compile what changed and link; ``group`` names a subset of the sources with a library of its own."""
+    lib_path = LIB_PATH if group is None else LIB_PATH[:-3] + f"_{group}.so"
     os.makedirs(LIB_DIR, exist_ok=True)
     obj_dir = os.path.join(LIB_DIR, "obj")
     os.makedirs(obj_dir, exist_ok=True)
     jobs = []
-    for src in _sources():
+    for src in _sources(group):
         obj = os.path.join(obj_dir, f"{os.path.basename(src)[:-3]}.{_hash(src)}.o")
         jobs.append((src, obj))
 
@@ -54,10 +61,12 @@ def build(verbose: bool = False, force: bool = False) -> str:
         for old in os.listdir(obj_dir):
             if old.startswith(os.path.basename(src)[:-3] + ".") and old.endswith(".o"):
                 os.remove(os.path.join(obj_dir, old))
-        cmd = [NVCC, *FLAGS, "-I", CSRC, "-c", src, "-o", obj]
+        part = f"{obj}.{os.getpid()}"
+        cmd = [NVCC, *FLAGS, "-I", CSRC, "-c", src, "-o", part]
         res = subprocess.run(cmd, capture_output=True, text=True)
         if res.returncode != 0:
             raise RuntimeError(f"nvcc failed for {src}:\n{res.stdout}\n{res.stderr}")
+        os.replace(part, obj)
         return obj, res.stderr
 
     with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as pool:
@@ -68,14 +77,16 @@ def build(verbose: bool = False, force: bool = False) -> str:
         with open(os.path.join(LIB_DIR, "ptxas.log"), "a") as fh:
             fh.write(logs)
     newest = max(os.path.getmtime(o) for o in objs)
-    if force or not os.path.exists(LIB_PATH) or os.path.getmtime(LIB_PATH) < newest:
-        cmd = [NVCC, "-shared", "-o", LIB_PATH, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
+    if force or not os.path.exists(lib_path) or os.path.getmtime(lib_path) < newest:
+        part = f"{lib_path}.{os.getpid()}"
+        cmd = [NVCC, "-shared", "-o", part, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
         res = subprocess.run(cmd, capture_output=True, text=True)
         if res.returncode != 0:
             raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
+        os.replace(part, lib_path)
     if verbose and logs:
         print(logs)
-    return LIB_PATH
+    return lib_path
 
 
 if __name__ == "__main__":

@@ -39,8 +39,18 @@ def lib():
             from tah_b200.ops.build import build
             build()
         _LIB = ctypes.CDLL(_LIB_PATH)
-        _LIB.tahb_decode_attn_ws_floats.restype = c_ll
+        if hasattr(_LIB, "tahb_decode_attn_ws_floats"):      # absent from the decoder-only build
+            _LIB.tahb_decode_attn_ws_floats.restype = c_ll
     return _LIB
+
+
+def use_decoder_build() -> None:
+    """Load the library from the sources that serving a :class:`HybridEngine` needs, compiling only those when the full
+    library is not there (a process that replays a trace or serves such a model; nothing may have been loaded yet)."""
+    global _LIB_PATH
+    if _LIB is None and not os.path.exists(_LIB_PATH):
+        from tah_b200.ops.build import build
+        _LIB_PATH = build(group="decoder")
 
 
 def available() -> bool:
@@ -538,10 +548,155 @@ def swiglu(gate_up, out=None):
 
 
 def logits_post(logits, cum, depth, best, best_val=None):
-    _rc(lib().tahb_logits_post(_p(logits), _p(cum), _p(depth), _p(best), _p(best_val), c_int(logits.shape[0]),
-                               c_int(logits.shape[1]), c_ll(logits.stride(0)), c_ll(cum.stride(0)), _stream()),
-        "tahb_logits_post")
+    fn = lib().tahb_logits_post_f32 if logits.dtype == torch.float32 else lib().tahb_logits_post
+    _rc(fn(_p(logits), _p(cum), _p(depth), _p(best), _p(best_val), c_int(logits.shape[0]), c_int(logits.shape[1]),
+           c_ll(logits.stride(0)), c_ll(cum.stride(0)), _stream()), "tahb_logits_post")
     return best
+
+
+# -------------------------------------------------------------------------------------------
+# decoders with an fp32 residual stream (activations bf16, or fp32 in the 32-bit mode)
+# -------------------------------------------------------------------------------------------
+def _act_f32(*ts: torch.Tensor) -> int:
+    """1 when the activation operands are fp32, 0 when they are bf16 (they must agree)."""
+    dt = ts[0].dtype
+    if dt not in (torch.float32, torch.bfloat16) or any(t.dtype != dt for t in ts):
+        raise ValueError(f"activations must be all bf16 or all fp32, got {[t.dtype for t in ts]}")
+    return 1 if dt == torch.float32 else 0
+
+
+def linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[M, F] = x[M, K] @ w[F, K]^T``: the tensor-core GEMM for bf16, the fp32 FMA kernel for fp32 operands."""
+    if not _act_f32(x, w):
+        return gemm(x, w, out=out)
+    if x.dim() != 2 or w.dim() != 2 or x.shape[1] != w.shape[1] or x.stride(1) != 1 or w.stride(1) != 1:
+        raise ValueError(f"linear: x {tuple(x.shape)} w {tuple(w.shape)}")
+    M, Kd = x.shape
+    if out is None:
+        out = torch.empty(M, w.shape[0], dtype=torch.float32, device=x.device)
+    _rc(lib().tahb_gemm_f32(_p(x), c_ll(x.stride(0)), _p(w), c_ll(w.stride(0)), _p(out), c_ll(out.stride(0)), c_int(M),
+                            c_int(w.shape[0]), c_int(Kd), _stream()), "tahb_gemm_f32")
+    return out
+
+
+def swiglu_linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``silu(gate) * up`` of ``x @ w^T``: bf16 weights have interleaved gate / up rows (:func:`interleave_gate_up`, the
+    fused GEMM epilogue), fp32 weights the stacked ``[gate; up]`` rows (product, then an activation kernel)."""
+    if not _act_f32(x, w):
+        return gemm(x, w, out=out, swiglu_interleaved=True)
+    gu = linear(x, w)
+    M, inter = gu.shape[0], gu.shape[1] // 2
+    if out is None:
+        out = torch.empty(M, inter, dtype=torch.float32, device=x.device)
+    _rc(lib().tahb_swiglu_f32(_p(gu), _p(out), c_int(M), c_int(inter), c_ll(gu.stride(0)), c_ll(out.stride(0)),
+                              _stream()), "tahb_swiglu_f32")
+    return out
+
+
+def embed_norm(E, tok, scale: float, w, width: int, eps: float, x, h):
+    """``x = scale * E[tok]`` (fp32 residual stream) and ``h = rms(x) * w`` in the activation type of ``E``.  Rows are
+    padded to ``E.shape[1]`` columns, ``width`` of them real."""
+    f32 = _act_f32(E, h)
+    _rc(lib().tahb_embed_norm(_p(E), _p(tok), c_float(scale), _p(x), _p(w), _p(h), c_int(tok.shape[0]), c_int(E.shape[0]),
+                              c_int(width), c_int(E.shape[1]), c_float(eps), c_int(f32), _stream()), "tahb_embed_norm")
+
+
+def residual_norm(y, x, w_out, w_next, width: int, eps: float, h):
+    """``x += rms(y) * w_out`` (fp32, in place) and ``h = rms(x) * w_next``: output norm, layer scale, residual sum and
+    the next sublayer's input norm in one launch.  ``w_out`` / ``w_next``: fp32 rows padded with zeros."""
+    f32 = _act_f32(y, h)
+    _rc(lib().tahb_residual_norm(_p(y), c_ll(y.stride(0)), _p(x), _p(w_out), _p(w_next), _p(h), c_int(y.shape[0]),
+                                 c_int(width), c_int(x.shape[1]), c_float(eps), c_int(f32), _stream()), "tahb_residual_norm")
+
+
+def few_linear(x, w, b, out=None):
+    """``x @ w^T + b`` with an fp32 result for a handful of output features (gates of a recurrence)."""
+    M, F = x.shape[0], w.shape[0]
+    if out is None:
+        out = torch.empty(M, F, dtype=torch.float32, device=x.device)
+    _rc(lib().tahb_few_linear(_p(x), c_ll(x.stride(0)), _p(w), _p(b), _p(out), c_int(M), c_int(w.shape[1]), c_int(F),
+                              c_int(_act_f32(x, w)), _stream()), "tahb_few_linear")
+    return out
+
+
+APPEND_MAX_ENTRIES = 1024
+
+
+def kv_append(rows, counts, starts, cache, depth: int, pos, row_of, slot):
+    """Append ``counts[e]`` tokens to row ``rows[e]`` of the paged cache for every entry of a step (pages from the device
+    free stack); fills position, row and slot of every packed token (entry ``e`` starts at ``starts[e]``)."""
+    pt = cache.page_table[depth]
+    _rc(lib().tahb_kv_append(_p(rows), _p(counts), _p(starts), c_int(rows.numel()), _p(cache.len[depth]), _p(pt),
+                             _p(cache.free_stack[depth]), _p(cache.free_count[depth]), c_int(cache.rows), c_int(pt.shape[1]),
+                             c_int(cache.page_size), _p(pos), _p(row_of), _p(slot), _p(status_word(pt.device)), _stream()),
+        "tahb_kv_append")
+
+
+def qkv_post(qkv, bias, q_w, k_w, q_out, cache, slot, nq: int, nkv: int, dk: int, dv: int, dim: int, page_size: int,
+             eps: float):
+    """Projection bias, per-head RMS norm of q / k, q to ``q_out``, k / v into the paged cache.  ``nkv = 0``: queries
+    only (a layer that reads another layer's keys)."""
+    _rc(lib().tahb_qkv_post(_p(qkv), c_ll(qkv.stride(0)), _p(bias), _p(q_w), _p(k_w), _p(q_out), _p(cache), _p(slot),
+                            c_int(qkv.shape[0]), c_int(nq), c_int(nkv), c_int(dk), c_int(dv), c_int(dim), c_int(page_size),
+                            c_float(eps), c_int(_act_f32(qkv, q_out)), _stream()), "tahb_qkv_post")
+
+
+class _WindowAttn(ctypes.Structure):
+    _fields_ = [("q", c_void_p), ("out", c_void_p), ("cache", c_void_p), ("page_table", c_void_p), ("pos", c_void_p),
+                ("row", c_void_p), ("bias", c_void_p), ("sink", c_void_p), ("gate", c_void_p)] + \
+               [(n, c_int) for n in ("n", "nq", "nkv", "dk", "dv", "page_size", "max_pages", "window", "keep_first", "far")] + \
+               [("ld_out", c_ll), ("ld_gate", c_ll), ("scale", c_float), ("ws", c_void_p), ("n_split", c_int),
+                ("status", c_void_p)]
+
+
+def window_attn_args(q, out, pool, page_table, pos, row, *, nq: int, nkv: int, dk: int, dv: int, page_size: int,
+                     scale: float, window: int, keep_first: int, bias=None, sink=None, gate=None, n_split: int = 1, ws=None):
+    """Arguments of one windowed attention launch: queries ``q [n, nq * dk]`` at positions ``pos`` of cache rows ``row``
+    over the paged ``pool`` of the layer that owns the keys; see ``csrc/attn_window.cu`` for the rule."""
+    a = _WindowAttn()
+    ptr = lambda t: 0 if t is None else t.data_ptr()
+    a.q, a.out, a.cache, a.page_table, a.pos, a.row = (ptr(t) for t in (q, out, pool, page_table, pos, row))
+    a.bias, a.sink, a.gate = ptr(bias), ptr(sink), ptr(gate)
+    a.n, a.nq, a.nkv, a.dk, a.dv, a.page_size, a.max_pages = q.shape[0], nq, nkv, dk, dv, page_size, page_table.shape[1]
+    a.window, a.keep_first, a.far = window, keep_first, 0 if bias is None else bias.shape[1] - 1
+    a.ld_out, a.ld_gate = out.stride(0), 0 if gate is None else gate.stride(0)
+    a.scale, a.ws, a.n_split, a.status = scale, ptr(ws), n_split, status_word(q.device).data_ptr()
+    return a
+
+
+def window_attn_plain(q, out, pool, page_table, pos, row, **kw):
+    """Windowed attention, one warp per (query, head): any head size up to 256, bf16 or fp32."""
+    a = window_attn_args(q, out, pool, page_table, pos, row, **kw)
+    _rc(lib().tahb_window_attn_plain(ctypes.byref(a), c_int(_act_f32(q, out)), _stream()), "tahb_window_attn_plain")
+    return out
+
+
+class _Mlstm(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("qkvg", "gates", "norm_w", "out", "S", "nvec", "mval", "seq_start", "seq_len", "pos",
+                                        "row", "slot")] + \
+               [(n, c_int) for n in ("n_seq", "heads", "dk", "dv", "dim", "vdim")] + [("ld", c_ll), ("ld_out", c_ll)] + \
+               [(n, c_float) for n in ("cap", "eps", "q_scale")]
+
+
+def mlstm_args(qkvg, gates, norm_w, out, state, pos, row, *, heads: int, dk: int, dv: int, dim: int, vdim: int, cap: float,
+               eps: float, seq_start=None, seq_len=None, slot=None):
+    a = _Mlstm()
+    ptr = lambda t: 0 if t is None else t.data_ptr()
+    S, nvec, mval = state
+    a.qkvg, a.gates, a.norm_w, a.out = ptr(qkvg), ptr(gates), ptr(norm_w), ptr(out)
+    a.S, a.nvec, a.mval = ptr(S), ptr(nvec), ptr(mval)
+    a.seq_start, a.seq_len, a.pos, a.row, a.slot = ptr(seq_start), ptr(seq_len), ptr(pos), ptr(row), ptr(slot)
+    a.n_seq = qkvg.shape[0] if seq_start is None else seq_start.shape[0]
+    a.heads, a.dk, a.dv, a.dim, a.vdim = heads, dk, dv, dim, vdim
+    a.ld, a.ld_out, a.cap, a.eps, a.q_scale = qkvg.stride(0), out.stride(0), cap, eps, dim ** -0.5
+    return a
+
+
+def mlstm_recurrent(qkvg, gates, norm_w, out, state, pos, row, **kw):
+    """mLSTM token by token (the decode step; also any portion): updates ``state = (S, n, m)`` in place."""
+    a = mlstm_args(qkvg, gates, norm_w, out, state, pos, row, **kw)
+    _rc(lib().tahb_mlstm_recurrent(ctypes.byref(a), c_int(_act_f32(qkvg, out)), _stream()), "tahb_mlstm_recurrent")
+    return out
 
 
 # -------------------------------------------------------------------------------------------
@@ -856,8 +1011,9 @@ class TickStateBinding:
         self.ints = (c_int * len(ints))(*ints)
 
     def tick_begin(self, E, soft, x_in, rope_cs=None, hd: int = 0, theta: float = 0.0):
-        """``rope_cs`` (optional ``[rows, hd]`` bf16): also write the RoPE cos | sin row of every row's position."""
-        _rc(lib().tahb_tick_begin(self.ptrs, self.ints, _p(E), _p(soft), _p(x_in), c_int(E.shape[1]), _p(rope_cs),
+        """``rope_cs`` (optional ``[rows, hd]`` bf16): also write the RoPE cos | sin row of every row's position.
+        ``E = None``: only the scheduler part (KV slots); the caller gathers the embeddings itself."""
+        _rc(lib().tahb_tick_begin(self.ptrs, self.ints, _p(E), _p(soft), _p(x_in), c_int(0 if E is None else E.shape[1]), _p(rope_cs),
                                   c_int(hd), c_float(theta), _stream()), "tahb_tick_begin")
 
     def tick_end(self, need_soft, next_tok):

@@ -25,7 +25,7 @@ from tah_b200.models.qwen3 import (LoRASpec, Qwen3Config, Qwen3ForCausalLM, expo
                                    import_hf_state_dict)
 
 
-def _save_sharded(tensors: Dict[str, torch.Tensor], directory: str, max_shard_bytes: int) -> None:
+def save_tensors(tensors: Dict[str, torch.Tensor], directory: str, max_shard_bytes: int) -> None:
     tensors = {k: v.detach().to("cpu").contiguous() for k, v in tensors.items()}
     total = sum(t.numel() * t.element_size() for t in tensors.values())
     if total <= max_shard_bytes:
@@ -50,7 +50,7 @@ def _save_sharded(tensors: Dict[str, torch.Tensor], directory: str, max_shard_by
         json.dump(index, fh, indent=2)
 
 
-def _load_all(directory: str) -> Dict[str, torch.Tensor]:
+def load_tensors(directory: str) -> Dict[str, torch.Tensor]:
     out: Dict[str, torch.Tensor] = {}
     index = os.path.join(directory, "model.safetensors.index.json")
     if os.path.exists(index):
@@ -90,7 +90,7 @@ def save_hf_checkpoint(model: Qwen3ForCausalLM, directory: str, adapter_kwargs: 
            if getattr(model.config, k) is not None}
     with open(os.path.join(directory, "generation_config.json"), "w", encoding="utf-8") as fh:
         json.dump(gen, fh, indent=2)
-    _save_sharded(base, directory, max_shard_bytes)
+    save_tensors(base, directory, max_shard_bytes)
     lora_dir = os.path.join(directory, "lora")
     os.makedirs(lora_dir, exist_ok=True)
     with open(os.path.join(lora_dir, "adapter_config.json"), "w", encoding="utf-8") as fh:
@@ -111,5 +111,5 @@ def load_hf_checkpoint(directory: str, lora: Optional[LoRASpec] = None, dtype=No
         with safe_open(lora_file, framework="pt", device="cpu") as fh:
             for k in fh.keys():
                 lora_sd[k] = fh.get_tensor(k)
-    import_hf_state_dict(model, base=_load_all(directory), lora=lora_sd, strict=True)
+    import_hf_state_dict(model, base=load_tensors(directory), lora=lora_sd, strict=True)
     return model
