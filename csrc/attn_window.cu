@@ -9,6 +9,9 @@
 // portions of a prompt, single decoded tokens and layers that read another layer's cache are the same case:
 //   page of one layer:  [K: kv_heads][page_size][dk]  then  [V: kv_heads][page_size][dv]
 // dk and dv are padded to multiples of 8; padding dims hold zeros.
+#include <cuda.h>
+
+#include "attn_common.cuh"
 #include "common.cuh"
 
 namespace tahb {
@@ -299,6 +302,610 @@ __global__ void __launch_bounds__(128) window_attn_plain_kernel(const WindowAttn
   }
 }
 
+// ---------------------------------------------------------------------------------------------
+// Decode kernel (bf16, pages of 16): one query per CTA row, all GB query heads of a group share the K / V reads.
+// Grid (nkv * groups, n, n_split); warp 4 streams whole K / V page blocks of one KV head with bulk copies through a
+// three-stage ring, warps 0..3 are 16 groups of 8 lanes, one token of a page per group.  Only pages that hold a visible
+// key are visited: the pages of the kept first tokens, then those of the window.  bias and sink are in log2 units.
+// ---------------------------------------------------------------------------------------------
+constexpr int WD_PAGE = 16;
+constexpr int WD_STAGE_PAGES = 2;
+constexpr int WD_NSTAGE = 3;
+constexpr float LOG2E = 1.4426950408889634f;
+
+// pages of a query at position i: `kp` pages of the kept part, then pages w0 .. i / 16; returns their number
+__device__ __forceinline__ int visible_pages(int i, int window, int keep_first, int& kp, int& w0) {
+  int keep_end, lo;
+  visible_range(i, window, keep_first, keep_end, lo);
+  kp = (keep_end + WD_PAGE - 1) / WD_PAGE;
+  w0 = max(lo / WD_PAGE, kp);
+  return kp + max(0, i / WD_PAGE - w0 + 1);
+}
+
+// o = sum / (mass + exp2(sink - m)), times the head's gate; m, mass, sink in log2 units
+__device__ __forceinline__ float finish_scale(const WindowAttnParams& p, int t, int h, float m, float mass) {
+  float f = 1.0f;
+  if (p.sink != nullptr) {
+    const float top = fmaxf(m, p.sink[h]);
+    f = exp2f(m - top);
+    mass = mass * f + exp2f(p.sink[h] - top);
+  }
+  f = mass > 0.f ? f / mass : 0.f;
+  if (p.gate != nullptr)
+    f *= sigmoid_f(__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(size_t)t * p.ld_gate + h]));
+  return f;
+}
+
+template <int VEC, int GB>
+__global__ void __launch_bounds__(160, (VEC * GB <= 4) ? 4 : 2) window_decode_kernel(const WindowAttnParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int DPL = VEC * 8;
+  extern __shared__ __align__(128) uint8_t wd_smem[];
+  const int kblk = WD_PAGE * p.dk, vblk = WD_PAGE * p.dv;              // elements of one K / V block of a page
+  const int stage_elems = WD_STAGE_PAGES * (kblk + vblk);
+  __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(wd_smem);
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(wd_smem + (size_t)WD_NSTAGE * stage_elems * 2);
+  uint64_t* empty_bar = full_bar + WD_NSTAGE;
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(empty_bar + WD_NSTAGE);
+
+  const int G = p.nq / p.nkv, groups = (G + GB - 1) / GB;
+  const int kvh = blockIdx.x / groups, grp0 = (blockIdx.x % groups) * GB;   // first query head of the group inside kvh
+  const int t = blockIdx.y, split = blockIdx.z;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int i = p.pos[t];
+  const int* pt = p.page_table + (size_t)p.row[t] * p.max_pages;
+  int kp, w0;
+  const int total = visible_pages(i, p.window, p.keep_first, kp, w0);
+  const int lo = p.window > i ? 0 : i - p.window + 1;
+  const int ppc = (total + p.n_split - 1) / p.n_split;
+  const int pb = split * ppc, pe = min(total, pb + ppc);
+  const int n_iter = pe > pb ? (pe - pb + WD_STAGE_PAGES - 1) / WD_STAGE_PAGES : 0;
+
+  if (tid == 0) {
+    for (int s = 0; s < WD_NSTAGE; ++s) {
+      mbar_init(&full_bar[s], 1);
+      mbar_init(&empty_bar[s], 4);
+    }
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  __syncthreads();
+
+  float m[GB], l[GB], acc[GB][DPL];
+#pragma unroll
+  for (int g = 0; g < GB; ++g) {
+    m[g] = -INFINITY;
+    l[g] = 0.f;
+#pragma unroll
+    for (int c = 0; c < DPL; ++c) acc[g][c] = 0.f;
+  }
+  const int grp = (warp & 3) * 4 + (lane >> 3);
+  const int gl = lane & 7;
+
+  if (warp == 4) {
+    if (lane == 0) {
+      const size_t page_elems = (size_t)p.nkv * (kblk + vblk);
+      for (int it = 0; it < n_iter; ++it) {
+        const int s = it % WD_NSTAGE;
+        mbar_wait(&empty_bar[s], ((it / WD_NSTAGE) & 1) ^ 1, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
+        const int first = pb + it * WD_STAGE_PAGES;
+        const int n_here = min(WD_STAGE_PAGES, pe - first);
+        mbar_expect_tx(&full_bar[s], n_here * (kblk + vblk) * 2);
+        for (int u = 0; u < n_here; ++u) {
+          const int idx = first + u;
+          const int page = pt[idx < kp ? idx : w0 + idx - kp];
+          const __nv_bfloat16* base = reinterpret_cast<const __nv_bfloat16*>(p.cache) + (size_t)page * page_elems;
+          __nv_bfloat16* dst = stages + (size_t)s * stage_elems + (size_t)u * (kblk + vblk);
+          bulk_load(dst, base + (size_t)kvh * kblk, kblk * 2, &full_bar[s]);
+          bulk_load(dst + kblk, base + (size_t)p.nkv * kblk + (size_t)kvh * vblk, vblk * 2, &full_bar[s]);
+        }
+      }
+    }
+    __syncwarp();
+  } else {
+    float qv[GB][DPL];
+    const float* bias[GB];
+#pragma unroll
+    for (int g = 0; g < GB; ++g) {
+      const bool live = grp0 + g < G;
+      const int h = kvh * G + (live ? grp0 + g : 0);
+      const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(p.q) + ((size_t)t * p.nq + h) * p.dk;
+      bias[g] = p.bias == nullptr ? nullptr : p.bias + (size_t)h * (p.far + 1);
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) {
+        const int c = (v * 8 + gl) * 8;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) qv[g][v * 8 + e] = live && c < p.dk ? __bfloat162float(qp[c + e]) * (p.scale * LOG2E) : 0.f;
+      }
+    }
+    for (int it = 0; it < n_iter; ++it) {
+      const int s = it % WD_NSTAGE;
+      mbar_wait(&full_bar[s], (it / WD_NSTAGE) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
+      const __nv_bfloat16* st = stages + (size_t)s * stage_elems;
+      float sc[WD_STAGE_PAGES][GB];
+      bool ok[WD_STAGE_PAGES];
+#pragma unroll
+      for (int u = 0; u < WD_STAGE_PAGES; ++u) {
+        const int idx = pb + it * WD_STAGE_PAGES + u;
+        const int j = (idx < kp ? idx : w0 + idx - kp) * WD_PAGE + grp;
+        ok[u] = idx < pe && j <= i && (j >= lo || j < p.keep_first);
+        float b[GB];
+#pragma unroll
+        for (int g = 0; g < GB; ++g) b[g] = ok[u] && bias[g] != nullptr ? bias[g][min(i - j, p.far)] : 0.f;
+        const __nv_bfloat16* kq = st + (size_t)u * (kblk + vblk) + grp * p.dk;
+        float se[GB], so[GB];
+#pragma unroll
+        for (int g = 0; g < GB; ++g) { se[g] = 0.f; so[g] = 0.f; }
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) {
+          const int c = (v * 8 + gl) * 8;
+          if (c < p.dk) {
+            const uint4 kr = *reinterpret_cast<const uint4*>(kq + c);
+            const __nv_bfloat162* kh = reinterpret_cast<const __nv_bfloat162*>(&kr);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 kf = __bfloat1622float2(kh[e]);
+#pragma unroll
+              for (int g = 0; g < GB; ++g) {
+                se[g] = fmaf(qv[g][v * 8 + 2 * e], kf.x, se[g]);
+                so[g] = fmaf(qv[g][v * 8 + 2 * e + 1], kf.y, so[g]);
+              }
+            }
+          }
+        }
+#pragma unroll
+        for (int g = 0; g < GB; ++g) {
+          float d = se[g] + so[g];
+          d += __shfl_xor_sync(0xffffffffu, d, 1);
+          d += __shfl_xor_sync(0xffffffffu, d, 2);
+          d += __shfl_xor_sync(0xffffffffu, d, 4);
+          sc[u][g] = ok[u] ? d + b[g] : -INFINITY;
+        }
+      }
+#pragma unroll
+      for (int g = 0; g < GB; ++g) {
+        float mx = m[g];
+#pragma unroll
+        for (int u = 0; u < WD_STAGE_PAGES; ++u) mx = fmaxf(mx, sc[u][g]);
+        const float corr = (m[g] == -INFINITY) ? 0.f : exp2f(m[g] - mx);
+        m[g] = mx;
+        l[g] *= corr;
+#pragma unroll
+        for (int c = 0; c < DPL; ++c) acc[g][c] *= corr;
+      }
+#pragma unroll
+      for (int u = 0; u < WD_STAGE_PAGES; ++u) {
+        if (!ok[u]) continue;            // never touch stage memory that holds no visible key
+        const __nv_bfloat16* vq = st + (size_t)u * (kblk + vblk) + kblk + grp * p.dv;
+        float pw[GB];
+#pragma unroll
+        for (int g = 0; g < GB; ++g) {
+          pw[g] = exp2f(sc[u][g] - m[g]);
+          l[g] += pw[g];
+        }
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) {
+          const int c = (v * 8 + gl) * 8;
+          if (c < p.dv) {
+            const uint4 vr = *reinterpret_cast<const uint4*>(vq + c);
+            const __nv_bfloat162* vh = reinterpret_cast<const __nv_bfloat162*>(&vr);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 vf = __bfloat1622float2(vh[e]);
+#pragma unroll
+              for (int g = 0; g < GB; ++g) {
+                acc[g][v * 8 + 2 * e] += pw[g] * vf.x;
+                acc[g][v * 8 + 2 * e + 1] += pw[g] * vf.y;
+              }
+            }
+          }
+        }
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&empty_bar[s]);
+    }
+  }
+
+  // merge the 16 token groups through shared memory (the ring is free now)
+  __syncthreads();
+  float* sm_m = reinterpret_cast<float*>(wd_smem);           // [16][GB]
+  float* sm_l = sm_m + 16 * GB;                              // [16][GB]
+  float* sm_acc = sm_l + 16 * GB;                            // [16][GB][dv]
+  if (warp < 4) {
+    if (gl == 0) {
+#pragma unroll
+      for (int g = 0; g < GB; ++g) { sm_m[grp * GB + g] = m[g]; sm_l[grp * GB + g] = l[g]; }
+    }
+#pragma unroll
+    for (int g = 0; g < GB; ++g)
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) {
+        const int c = (v * 8 + gl) * 8;
+        if (c < p.dv) {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) sm_acc[(grp * GB + g) * p.dv + c + e] = acc[g][v * 8 + e];
+        }
+      }
+  }
+  __syncthreads();
+  for (int idx = tid; idx < GB * p.dv; idx += 160) {
+    const int g = idx / p.dv, d = idx % p.dv;
+    if (grp0 + g >= G) continue;
+    float mx = -INFINITY;
+#pragma unroll
+    for (int k = 0; k < 16; ++k) mx = fmaxf(mx, sm_m[k * GB + g]);
+    float num = 0.f, den = 0.f;
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      const float mk = sm_m[k * GB + g];
+      const float w = (mk == -INFINITY) ? 0.f : exp2f(mk - mx);
+      num += w * sm_acc[(k * GB + g) * p.dv + d];
+      den += w * sm_l[k * GB + g];
+    }
+    const int h = kvh * G + grp0 + g;
+    if (p.n_split == 1) {
+      reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ld_out + (size_t)h * p.dv + d] =
+          __float2bfloat16_rn(num * finish_scale(p, t, h, mx, den));
+    } else {
+      float* w = p.ws + (((size_t)t * p.nq + h) * p.n_split + split) * (p.dv + 2);
+      w[d] = num;
+      if (d == 0) { w[p.dv] = mx; w[p.dv + 1] = den; }
+    }
+  }
+}
+
+__global__ void __launch_bounds__(128) window_decode_merge_kernel(const WindowAttnParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x / p.nq, h = blockIdx.x % p.nq, stride = p.dv + 2;
+  const float* w = p.ws + (size_t)blockIdx.x * p.n_split * stride;
+  float mx = -INFINITY, den = 0.f;
+  for (int s = 0; s < p.n_split; ++s) mx = fmaxf(mx, w[s * stride + p.dv]);
+  for (int s = 0; s < p.n_split; ++s) {
+    const float ms = w[s * stride + p.dv];
+    if (ms != -INFINITY) den += exp2f(ms - mx) * w[s * stride + p.dv + 1];
+  }
+  const float f = finish_scale(p, t, h, mx, den);
+  for (int d = threadIdx.x; d < p.dv; d += blockDim.x) {
+    float num = 0.f;
+    for (int s = 0; s < p.n_split; ++s) {
+      const float ms = w[s * stride + p.dv];
+      if (ms != -INFINITY) num += exp2f(ms - mx) * w[s * stride + d];
+    }
+    reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ld_out + (size_t)h * p.dv + d] = __float2bfloat16_rn(num * f);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
+// Portion kernel on the tensor cores (bf16, pages of 16): one CTA = a tile of up to 128 consecutive queries of one row
+// and one query head, walking the blocks of 64 keys that any of its queries sees (kept part, then window).  Same
+// structure as prefill_attn_kernel - S = Q K^T and O += P V by tcgen05 with S and O in tensor memory, two softmax
+// threads per query, lazily refreshed maximum, two-stage TMA ring - with K / V fetched page by page from the cache
+// (four 16-row boxes per 64-key block form one swizzled tile; dims past dk / dv and pages past the last key read as
+// zeros) and with the distance bias added to the scores in registers.
+// Warp roles (320 threads): warp 0 TMA, warp 1 tensor memory + MMA, warps 2..9 softmax / epilogue.
+// ---------------------------------------------------------------------------------------------
+struct WindowTiles {
+  const int* q0;              // [n_tiles] first packed query
+  const int* qn;              // [n_tiles] queries (<= 128)
+  int n_pages;                // pages of the pool (an index past it reads zeros)
+};
+
+template <int HK, int HV>
+struct WpCfg {
+  static constexpr int BK = 64;
+  static constexpr int QTILE = 128 * 64 * 2, KTILE = BK * 64 * 2;
+  static constexpr int Q_BYTES = HK * QTILE, K_BYTES = HK * KTILE, V_BYTES = HV * KTILE;
+  static constexpr int P_BYTES = 128 * BK * 2;
+  static constexpr int STAGE_BYTES = K_BYTES + V_BYTES;
+  static constexpr int NSTAGE = 2;
+  static constexpr int SMEM_BYTES = Q_BYTES + P_BYTES + NSTAGE * STAGE_BYTES + 128;
+  static constexpr int XCOL = 64;                            // exchange columns between the two halves of a query
+  static constexpr int TMEM_COLS = HV <= 2 ? 256 : 512;      // S at 0, O at 128
+  static constexpr int MIN_CTAS = HK + HV <= 4 ? 2 : 1;
+};
+constexpr int WP_THREADS = 320;
+
+__device__ __forceinline__ void tma_load_4d(void* smem_dst, const void* tmap, int c0, int c1, int c2, int c3, uint64_t* bar) {
+  asm volatile(
+      "cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];"
+      ::"r"(smem_u32(smem_dst)), "l"(reinterpret_cast<uint64_t>(tmap)), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2), "r"(c3)
+      : "memory");
+}
+
+template <int HK, int HV>
+__global__ void __launch_bounds__(WP_THREADS, WpCfg<HK, HV>::MIN_CTAS)
+window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
+                      const __grid_constant__ CUtensorMap tm_v, const WindowAttnParams p, const WindowTiles tl) {
+  using C = WpCfg<HK, HV>;
+  constexpr int BK = C::BK;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  uint8_t* q_s = smem;
+  uint8_t* p_s = q_s + C::Q_BYTES;
+  uint8_t* kv_s = p_s + C::P_BYTES;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(kv_s + C::NSTAGE * C::STAGE_BYTES);
+  uint64_t* q_full = bars;
+  uint64_t* kv_full = bars + 1;
+  uint64_t* kv_empty = kv_full + C::NSTAGE;
+  uint64_t* s_full = kv_empty + C::NSTAGE;
+  uint64_t* p_ready = s_full + 1;
+  uint64_t* pv_done = p_ready + 1;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 1);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int tile = blockIdx.x, head = blockIdx.y;
+  const int kvh = head / (p.nq / p.nkv);
+  if ((smem_u32(smem) & 1023u) != 0) {          // the swizzled tiles need a 1024-byte aligned base
+    if (threadIdx.x == 0) atomicCAS(p.status, 0, STATUS_BAD_INDEX);
+    return;
+  }
+  if (threadIdx.x == 0) {
+    mbar_init(q_full, 1);
+    for (int s = 0; s < C::NSTAGE; ++s) { mbar_init(&kv_full[s], 1); mbar_init(&kv_empty[s], 1); }
+    mbar_init(s_full, 1);
+    mbar_init(p_ready, 256);
+    mbar_init(pv_done, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, C::TMEM_COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+  const uint32_t tmem_s = tmem_base, tmem_o = tmem_base + 128;
+
+  const int q0 = tl.q0[tile], qn = tl.qn[tile];
+  const int i0 = p.pos[q0], i_last = i0 + qn - 1;             // the tile's positions are consecutive
+  int keep_end, lo0;
+  visible_range(i0, p.window, p.keep_first, keep_end, lo0);
+  const int kb = (keep_end + BK - 1) / BK;                    // blocks of the kept part
+  const int w0 = max(lo0 / BK, kb);                           // first block of the window part
+  const int total_blocks = kb + max(0, i_last / BK - w0 + 1);
+
+  if (warp == 0) {
+    // ---------------- TMA producer ----------------
+    if (lane == 0) {
+      mbar_expect_tx(q_full, C::Q_BYTES);
+#pragma unroll
+      for (int h = 0; h < HK; ++h) tma_load_2d(q_s + h * C::QTILE, &tm_q, head * p.dk + h * 64, q0, q_full);
+      const int* pt = p.page_table + (size_t)p.row[q0] * p.max_pages;
+      const int last_page = i_last / WD_PAGE;
+      for (int n = 0; n < total_blocks; ++n) {
+        const int st = n % C::NSTAGE;
+        const int b = n < kb ? n : w0 + n - kb;
+        int page[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) page[u] = b * 4 + u <= last_page ? pt[b * 4 + u] : tl.n_pages;
+        mbar_wait(&kv_empty[st], ((n / C::NSTAGE) & 1) ^ 1, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
+        if (*abort_flag) break;
+        mbar_expect_tx(&kv_full[st], C::STAGE_BYTES);
+        uint8_t* ks = kv_s + st * C::STAGE_BYTES;
+        uint8_t* vs = ks + C::K_BYTES;
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+#pragma unroll
+          for (int h = 0; h < HK; ++h) tma_load_4d(ks + h * C::KTILE + u * 2048, &tm_k, h * 64, 0, kvh, page[u], &kv_full[st]);
+#pragma unroll
+          for (int h = 0; h < HV; ++h) tma_load_4d(vs + h * C::KTILE + u * 2048, &tm_v, h * 64, 0, kvh, page[u], &kv_full[st]);
+        }
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    // ---------------- MMA issuer ----------------
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = umma_idesc_bf16(128, BK);
+      constexpr uint32_t idesc_o = umma_idesc_bf16_bmn(128, HV * 64);
+      mbar_wait(q_full, 0, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
+      const uint32_t q_addr = smem_u32(q_s), p_addr = smem_u32(p_s);
+      for (int n = 0; n < total_blocks; ++n) {
+        const int st = n % C::NSTAGE;
+        mbar_wait(&kv_full[st], (n / C::NSTAGE) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
+        tc_fence_after();
+        const uint32_t k_addr = smem_u32(kv_s + st * C::STAGE_BYTES);
+        const uint32_t v_addr = k_addr + C::K_BYTES;
+#pragma unroll
+        for (int ks = 0; ks < HK * 4; ++ks) {
+          const uint32_t qo = (ks / 4) * C::QTILE + (ks % 4) * 32;
+          const uint32_t ko = (ks / 4) * C::KTILE + (ks % 4) * 32;
+          umma_bf16(tmem_s, umma_desc_sw128(q_addr + qo), umma_desc_sw128(k_addr + ko), idesc_s, ks > 0 ? 1u : 0u);
+        }
+        umma_commit(s_full);
+        mbar_wait(p_ready, n & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+        tc_fence_after();
+#pragma unroll
+        for (int ks = 0; ks < BK / 16; ++ks)
+          umma_bf16(tmem_o, umma_desc_sw128(p_addr + ks * 32), umma_desc_mn_sw128(v_addr + ks * 2048, C::KTILE), idesc_o,
+                    (n > 0 || ks > 0) ? 1u : 0u);
+        umma_commit(&kv_empty[st]);
+        umma_commit(pv_done);
+      }
+    }
+    __syncwarp();
+  } else {
+    // ---------------- softmax / epilogue: two threads per query, 32 key columns each ----------------
+    const int qd = warp & 3, half = (warp - 2) >> 2;
+    const int row = qd * 32 + lane;
+    const bool row_ok = row < qn;
+    const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
+    const float sc = p.scale * LOG2E;
+    const int i = i0 + row;
+    const int iw0 = i0 + qd * 32, iw1 = iw0 + 31;             // positions of the warp's first and last query
+    const int lo = p.window > i ? 0 : i - p.window + 1;
+    const int lo_w1 = p.window > iw1 ? 0 : iw1 - p.window + 1;
+    const float* bias = p.bias == nullptr ? nullptr : p.bias + (size_t)head * (p.far + 1);
+    const float far_bias = bias == nullptr ? 0.f : bias[p.far];
+    float m_ref = -INFINITY, l = 0.f;
+    for (int n = 0; n < total_blocks; ++n) {
+      const int j0 = (n < kb ? n : w0 + n - kb) * BK + half * 32;        // first key column of this thread
+      mbar_wait(s_full, n & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+      tc_fence_after();
+      float sv[32];
+      tmem_ld32(tmem_s + lane_off + half * 32, sv);
+      tmem_ld_wait();
+      const int dmin = iw0 - (j0 + 31), dmax = iw1 - j0;                 // distances inside the warp's 32 x 32 patch
+      if (bias == nullptr || dmin >= p.far) {
+#pragma unroll
+        for (int c = 0; c < 32; ++c) sv[c] = fmaf(sv[c], sc, far_bias);
+      } else if (dmin >= 0 && dmax <= p.far) {
+        const float* b = bias + (i - j0);
+#pragma unroll
+        for (int c = 0; c < 32; ++c) sv[c] = fmaf(sv[c], sc, __ldg(b - c));
+      } else {
+#pragma unroll
+        for (int c = 0; c < 32; ++c) sv[c] = fmaf(sv[c], sc, __ldg(bias + min(max(i - j0 - c, 0), p.far)));
+      }
+      if (!(dmin >= 0 && (j0 >= lo_w1 || j0 + 31 < p.keep_first))) {
+#pragma unroll
+        for (int c = 0; c < 32; ++c) {
+          const int j = j0 + c;
+          if (j > i || (j < lo && j >= p.keep_first)) sv[c] = -INFINITY;
+        }
+      }
+      float mx = sv[0];
+#pragma unroll
+      for (int c = 1; c < 32; ++c) mx = fmaxf(mx, sv[c]);
+      const uint32_t xcol = tmem_base + lane_off + C::XCOL + (n & 1) * 2;
+      tmem_st1(xcol + half, mx);
+      tmem_st_wait();
+      tc_fence_before();
+      named_bar_sync(1, 256);
+      tc_fence_after();
+      mx = fmaxf(mx, tmem_ld1(xcol + (half ^ 1)));
+      const bool grow = mx > m_ref + 8.0f;
+      const float m_new = grow ? mx : m_ref;
+      const float f = (grow && m_ref != -INFINITY) ? exp2f(m_ref - m_new) : 1.0f;
+      if (n > 0) mbar_wait(pv_done, (n - 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+      tc_fence_after();
+      if (n > 0 && __any_sync(0xffffffffu, f != 1.0f)) {
+#pragma unroll 1
+        for (int c = 0; c < HV * 32; c += 32) {
+          float o[32];
+          tmem_ld32(tmem_o + lane_off + half * (HV * 32) + c, o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int e = 0; e < 32; ++e) o[e] *= f;
+          tmem_st32(tmem_o + lane_off + half * (HV * 32) + c, o);
+        }
+        tmem_st_wait();
+      }
+      l *= f;
+      m_ref = m_new;
+      const float neg_m = (m_ref == -INFINITY) ? 0.f : -m_ref;
+      float ps0 = 0.f, ps1 = 0.f;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        uint4 pk;
+        __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&pk);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float a = ex2_approx(sv[c * 8 + 2 * e] + neg_m);
+          const float b = ex2_approx(sv[c * 8 + 2 * e + 1] + neg_m);
+          p2[e] = __floats2bfloat162_rn(a, b);
+          ps0 += a;
+          ps1 += b;
+        }
+        *reinterpret_cast<uint4*>(p_s + row * 128 + (((half * 4 + c) ^ (row & 7)) << 4)) = pk;
+      }
+      l += ps0 + ps1;
+      fence_proxy_async_smem();
+      tc_fence_before();
+      mbar_arrive(p_ready);
+    }
+    if (total_blocks > 0) mbar_wait(pv_done, (total_blocks - 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+    tc_fence_after();
+    {
+      const uint32_t xcol = tmem_base + lane_off + C::XCOL;
+      named_bar_sync(1, 256);
+      tmem_st1(xcol + half, l);
+      tmem_st_wait();
+      tc_fence_before();
+      named_bar_sync(1, 256);
+      tc_fence_after();
+      l += tmem_ld1(xcol + (half ^ 1));
+    }
+    const float inv = row_ok ? finish_scale(p, q0 + row, head, m_ref, l) : 0.f;
+    __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(q0 + row) * p.ld_out + (size_t)head * p.dv;
+#pragma unroll 1
+    for (int c = half * (HV * 32); c < (half + 1) * (HV * 32); c += 32) {
+      float o[32];
+      tmem_ld32(tmem_o + lane_off + c, o);
+      tmem_ld_wait();
+      if (row_ok) {
+#pragma unroll
+        for (int v = 0; v < 4; ++v) {
+          if (c + v * 8 < p.dv) {
+            uint4 pk;
+            __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&pk);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) p2[e] = __floats2bfloat162_rn(o[v * 8 + 2 * e] * inv, o[v * 8 + 2 * e + 1] * inv);
+            *reinterpret_cast<uint4*>(dst + c + v * 8) = pk;
+          }
+        }
+      }
+    }
+    tc_fence_before();
+  }
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, C::TMEM_COLS);
+  }
+}
+
+template <int VEC, int GB>
+static int launch_window_decode(const WindowAttnParams& p, cudaStream_t stream) {
+  const int groups = (p.nq / p.nkv + GB - 1) / GB;
+  const size_t ring = (size_t)WD_NSTAGE * WD_STAGE_PAGES * WD_PAGE * (p.dk + p.dv) * 2 + 128;
+  const size_t merge = (size_t)16 * GB * (p.dv + 2) * 4;
+  const size_t smem = ring > merge ? ring : merge;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(window_decode_kernel<VEC, GB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
+      return -10;
+    configured = true;
+  }
+  if (smem > 160 * 1024) return -11;
+  cudaError_t e = launch_chain(window_decode_kernel<VEC, GB>, dim3(p.nkv * groups, p.n, p.n_split), dim3(160), smem, stream, p);
+  if (e == cudaSuccess && p.n_split > 1)
+    e = launch_chain(window_decode_merge_kernel, dim3(p.n * p.nq), dim3(128), 0, stream, p);
+  return e == cudaSuccess ? 0 : -3;
+}
+
+// K (or V) of a paged cache as a 4-D tensor [pages][kv heads][16 tokens][dims], read in boxes of one page's 16 tokens x 64 dims
+static int make_page_map(CUtensorMap* m, const void* base, int d, int nkv, int n_pages, size_t page_elems) {
+  PfEncodeFn fn = pf_encode_fn();
+  if (fn == nullptr) return -1;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || d % 8 || page_elems % 8) return -2;
+  cuuint64_t dims[4] = {(cuuint64_t)d, WD_PAGE, (cuuint64_t)nkv, (cuuint64_t)n_pages};
+  cuuint64_t strides[3] = {(cuuint64_t)d * 2, (cuuint64_t)d * WD_PAGE * 2, (cuuint64_t)page_elems * 2};
+  cuuint32_t box[4] = {64u, WD_PAGE, 1u, 1u}, estr[4] = {1u, 1u, 1u, 1u};
+  CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -3;
+}
+
+template <int HK, int HV>
+static int launch_window_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
+                                 const WindowAttnParams& p, const WindowTiles& tl, int n_tiles, cudaStream_t stream) {
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(window_prefill_kernel<HK, HV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             WpCfg<HK, HV>::SMEM_BYTES) != cudaSuccess)
+      return -10;
+    configured = true;
+  }
+  window_prefill_kernel<HK, HV><<<dim3(n_tiles, p.nq), WP_THREADS, WpCfg<HK, HV>::SMEM_BYTES, stream>>>(mq, mk, mv, p, tl);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
 }  // namespace tahb
 
 using namespace tahb;
@@ -338,4 +945,47 @@ extern "C" int tahb_window_attn_plain(const WindowAttnParams* p, int f32, cudaSt
   cudaError_t e = f32 ? launch_chain(window_attn_plain_kernel<float>, grid, dim3(128), 0, stream, *p)
                       : launch_chain(window_attn_plain_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, *p);
   return e == cudaSuccess ? 0 : -3;
+}
+
+static int check_window_attn(const WindowAttnParams* p) {
+  return p->nkv <= 0 || p->nq % p->nkv || p->dk > 256 || p->dv > 256 || p->dk % 8 || p->dv % 8 || p->window < 1 || p->far < 0 ||
+         p->keep_first < 0 ? -2 : 0;
+}
+
+// One query per entry (decode).  bias and sink in log2 units; ws: n * nq * n_split * (dv + 2) floats when n_split > 1.
+extern "C" int tahb_window_attn_decode(const WindowAttnParams* p, cudaStream_t stream) {
+  if (p->n <= 0) return 0;
+  if (check_window_attn(p) || p->n > 65535 || p->n_split < 1 || p->n_split > 64) return -2;
+  if (p->page_size != WD_PAGE) return -5;
+  if (p->n_split > 1 && p->ws == nullptr) return -4;
+  const int d = p->dk > p->dv ? p->dk : p->dv, vec = d <= 64 ? 1 : d <= 128 ? 2 : 4;
+  const int G = p->nq / p->nkv, gb = G == 1 ? 1 : (G == 2 || vec == 4) ? 2 : 4;
+#define TAHB_WD(V_, G_) if (vec == V_ && gb == G_) return launch_window_decode<V_, G_>(*p, stream);
+  TAHB_WD(1, 1) TAHB_WD(1, 2) TAHB_WD(1, 4)
+  TAHB_WD(2, 1) TAHB_WD(2, 2) TAHB_WD(2, 4)
+  TAHB_WD(4, 1) TAHB_WD(4, 2)
+#undef TAHB_WD
+  return -2;
+}
+
+// Query tiles of portions; n_pages = pages of the layer's pool.  bias and sink in log2 units.
+extern "C" int tahb_window_attn_tiles(const WindowAttnParams* p, const int* q0, const int* qn, int n_tiles, int n_pages,
+                                      cudaStream_t stream) {
+  if (p->n <= 0 || n_tiles <= 0) return 0;
+  if (check_window_attn(p) || p->ld_out % 8) return -2;
+  if (p->page_size != WD_PAGE) return -5;
+  const size_t page_elems = (size_t)p->nkv * WD_PAGE * (p->dk + p->dv);
+  CUtensorMap mq, mk, mv;
+  int rc;
+  if ((rc = pf_make_map(&mq, p->q, p->n, (long long)p->nq * p->dk, 128u))) return rc;
+  if ((rc = make_page_map(&mk, p->cache, p->dk, p->nkv, n_pages, page_elems))) return rc;
+  if ((rc = make_page_map(&mv, reinterpret_cast<const __nv_bfloat16*>(p->cache) + (size_t)p->nkv * WD_PAGE * p->dk, p->dv,
+                          p->nkv, n_pages, page_elems))) return rc;
+  WindowTiles tl{q0, qn, n_pages};
+  const int hk = p->dk <= 64 ? 1 : p->dk <= 128 ? 2 : 4, hv = p->dv <= 64 ? 1 : p->dv <= 128 ? 2 : 4;
+  if (hk == 4 || hv == 4) return launch_window_prefill<4, 4>(mq, mk, mv, *p, tl, n_tiles, stream);
+  if (hk == 2) return hv == 2 ? launch_window_prefill<2, 2>(mq, mk, mv, *p, tl, n_tiles, stream)
+                              : launch_window_prefill<2, 1>(mq, mk, mv, *p, tl, n_tiles, stream);
+  return hv == 2 ? launch_window_prefill<1, 2>(mq, mk, mv, *p, tl, n_tiles, stream)
+                 : launch_window_prefill<1, 1>(mq, mk, mv, *p, tl, n_tiles, stream);
 }

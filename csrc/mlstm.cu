@@ -8,6 +8,9 @@
 //
 // S, n and m live in fp32, one slot per cache row: state[slot][head] = S [dk][dv], n [dk], m.  A token at position 0
 // starts from zero, so a slot needs no clearing when it changes hands.  dk and dv are padded to multiples of 8 with zeros.
+#include <cuda.h>
+
+#include "attn_common.cuh"
 #include "common.cuh"
 
 namespace tahb {
@@ -154,6 +157,589 @@ __global__ void __launch_bounds__(MR_THREADS) mlstm_recurrent_kernel(const Mlstm
   if (tid == 0) p.mval[sh] = m;
 }
 
+// ---------------------------------------------------------------------------------------------
+// Chunkwise form for prompt portions (bf16 activations) on the tensor cores.  A portion is cut into chunks of up to 128
+// tokens.  Inside a chunk with incoming state (S0, n0, m0), F_t the running sum of the log forget gates and
+// B_s = i_s - F_s:
+//
+//   m_t = F_t + max(m0, max_{s <= t} B_s)                                    the same running maximum as token by token
+//   P_ts = (q_t . k_s) exp(F_t - m_t + B_s)        for s <= t
+//   o_t  = (sum_s P_ts v_s + a_t S0^T q_t) / (max(|sum_s P_ts + a_t n0 . q_t|, exp(-m_t)) + 1e-6),  a_t = exp(F_t + m0 - m_t)
+//
+// Three launches, every chunk of every portion in parallel except for the element-wise scan:
+//   mlstm_chunk_state_kernel   dS = sum_s exp(F_L + B_s - M) k_s v_s^T,  M = F_L + max_s B_s         [K^T V by tcgen05]
+//   mlstm_chunk_scan_kernel    the incoming state of every chunk and the state the portion leaves behind (fp32)
+//   mlstm_chunk_out_kernel     P by tcgen05 (Q K^T) and registers, O by tcgen05, head norm and output gate in the epilogue
+//
+// fp32 operands of a matrix product (P, the weighted keys, the incoming state) enter as a bf16 pair hi + lo, two
+// accumulating products (relative error 2^-17 or less); queries, keys and values are bf16 to begin with.
+// ---------------------------------------------------------------------------------------------
+struct MlstmChunkParams {
+  const int* c_start;         // [n_chunks] first packed token
+  const int* c_len;           // [n_chunks] tokens (<= 128)
+  const int* seq_chunk0;      // [n_seq] first chunk of each portion
+  const int* seq_chunks;      // [n_seq] chunks of each portion
+  float* dS;                  // [n_chunks, heads, dk, dv]
+  float* dn;                  // [n_chunks, heads, dk]
+  float* cg;                  // [n_chunks, heads, 2]: F_L, max_s B_s
+  __nv_bfloat16* s0;          // [n_chunks, heads, 2 (hi, lo), dk, dv] incoming state
+  float* n0;                  // [n_chunks, heads, dk]
+  float* m0;                  // [n_chunks, heads]
+  int n_chunks;
+  int* status;
+};
+
+constexpr int MC_TOK = 128;
+constexpr int MC_KCH = MC_TOK * 128;          // bytes of one 64-column chunk of a 128-token tile
+
+__device__ __forceinline__ void tma_load_3d(void* smem_dst, const void* tmap, int c0, int c1, int c2, uint64_t* bar) {
+  asm volatile(
+      "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+      ::"r"(smem_u32(smem_dst)), "l"(reinterpret_cast<uint64_t>(tmap)), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2)
+      : "memory");
+}
+// A MN-major (transposed), B MN-major
+__host__ __device__ constexpr uint32_t umma_idesc_bf16_amn_bmn(int m, int n) { return umma_idesc_bf16(m, n) | (1u << 15) | (1u << 16); }
+
+// Gate scan of a chunk by the first 128 threads of the block (every thread calls it): token t = tid < 128.
+// F = inclusive sum of the log forget gates, B = log_i - F, Bmax = inclusive prefix maximum of B.  xw: 8 floats.
+__device__ __forceinline__ void chunk_gates(const float* gates, int heads, int h, int start, int len, float cap, float* xw,
+                                            float& F, float& B, float& Bmax) {
+  const int t = threadIdx.x, lane = t & 31, w = t >> 5;
+  F = 0.f;
+  B = -INFINITY;
+  float li = -INFINITY;
+  if (t < len) {
+    li = mlstm_log_i(gates[(size_t)(start + t) * 2 * heads + h], cap);
+    F = mlstm_log_f(gates[(size_t)(start + t) * 2 * heads + heads + h], cap);
+  }
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float v = __shfl_up_sync(0xffffffffu, F, o);
+    if (lane >= o) F += v;
+  }
+  if (w < 4 && lane == 31) xw[w] = F;
+  __syncthreads();
+  for (int k = 0; k < min(w, 4); ++k) F += xw[k];
+  if (t < len) B = li - F;
+  Bmax = B;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float v = __shfl_up_sync(0xffffffffu, Bmax, o);
+    if (lane >= o) Bmax = fmaxf(Bmax, v);
+  }
+  if (w < 4 && lane == 31) xw[4 + w] = Bmax;
+  __syncthreads();
+  for (int k = 0; k < min(w, 4); ++k) Bmax = fmaxf(Bmax, xw[4 + k]);
+}
+
+__device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const float2 f = __bfloat1622float2(h);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+
+// dS of one (chunk, head): grid (n_chunks, heads), 256 threads.  Shared: K hi and lo (2 chunks of 16 KiB each), V (nv
+// chunks of 16 KiB).
+struct McStateSmem {
+  static constexpr int K_HI = 0, K_LO = 2 * MC_KCH, V = 4 * MC_KCH;
+  static int bytes(int nv) { return (4 + nv) * MC_KCH + 1024; }
+};
+
+__global__ void __launch_bounds__(256, 1)
+mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
+                         const MlstmParams p, const MlstmChunkParams c, const int nv) {
+  extern __shared__ __align__(1024) uint8_t mc_smem[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int ch = blockIdx.x, h = blockIdx.y;
+  if ((smem_u32(mc_smem) & 1023u) != 0) {
+    if (tid == 0) atomicCAS(c.status, 0, STATUS_BAD_INDEX);
+    return;
+  }
+  uint8_t* tail = mc_smem + McStateSmem::V + nv * MC_KCH;
+  float* s_w = reinterpret_cast<float*>(tail);                 // [128] weight of each token
+  float* s_x = s_w + MC_TOK;                                   // [8]
+  uint64_t* full = reinterpret_cast<uint64_t*>(s_x + 8);
+  uint64_t* done = full + 1;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(done + 1);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  if (tid == 0) {
+    mbar_init(full, 1);
+    mbar_init(done, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, 256);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
+  const int start = c.c_start[ch], len = c.c_len[ch];
+  if (tid == 0) {
+    mbar_expect_tx(full, (2 + nv) * MC_KCH);
+    for (int k = 0; k < 2; ++k) tma_load_3d(mc_smem + McStateSmem::K_HI + k * MC_KCH, &tm_k, k * 64, p.heads + h, start, full);
+    for (int k = 0; k < nv; ++k) tma_load_3d(mc_smem + McStateSmem::V + k * MC_KCH, &tm_v, k * 64, h, start, full);
+  }
+  float F, B, Bmax;
+  chunk_gates(p.gates, p.heads, h, start, len, p.cap, s_x, F, B, Bmax);
+  float* s_last = reinterpret_cast<float*>(tmem_slot + 2);     // [2] F and prefix maximum of the chunk's last token
+  if (tid == len - 1) { s_last[0] = F; s_last[1] = Bmax; }
+  __syncthreads();
+  const size_t chh = (size_t)ch * p.heads + h;
+  if (tid < MC_TOK) s_w[tid] = tid < len ? expf(B - s_last[1]) : 0.f;
+  if (tid == 0) { c.cg[chh * 2] = s_last[0]; c.cg[chh * 2 + 1] = s_last[1]; }
+  __syncthreads();
+  mbar_wait(full, 0, abort_flag, c.status, STATUS_TIMEOUT_TMA_FULL);
+  // weighted keys: hi in place, lo beside them (16 bytes = 8 dims of one token per step; the swizzle only permutes
+  // 16-byte pieces inside a token's 128 bytes)
+  for (int i = tid; i < 2 * MC_TOK * 8; i += 256) {
+    const int tok = (i >> 3) & (MC_TOK - 1);
+    const float w = s_w[tok];
+    uint4* kp = reinterpret_cast<uint4*>(mc_smem + McStateSmem::K_HI) + i;
+    const uint4 kv = *kp;
+    const __nv_bfloat162* k2 = reinterpret_cast<const __nv_bfloat162*>(&kv);
+    uint32_t hi[4], lo[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(k2[e]);
+      split_bf16(tok < len ? f.x * w : 0.f, tok < len ? f.y * w : 0.f, hi[e], lo[e]);
+    }
+    *kp = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    reinterpret_cast<uint4*>(mc_smem + McStateSmem::K_LO)[i] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+  }
+  fence_proxy_async_smem();
+  __syncthreads();
+  if (tid == 32) {
+    tc_fence_after();
+    const uint32_t v_addr = smem_u32(mc_smem + McStateSmem::V);
+    for (int v0 = 0; v0 < nv; v0 += 2) {
+      const int n = v0 + 1 < nv ? 128 : 64;
+      const uint32_t idesc = umma_idesc_bf16_amn_bmn(128, n);
+      for (int part = 0; part < 2; ++part) {
+        const uint32_t a_addr = smem_u32(mc_smem + (part == 0 ? McStateSmem::K_HI : McStateSmem::K_LO));
+#pragma unroll
+        for (int ks = 0; ks < MC_TOK / 16; ++ks)
+          umma_bf16(tmem + v0 * 64, umma_desc_mn_sw128(a_addr + ks * 2048, MC_KCH),
+                    umma_desc_mn_sw128(v_addr + v0 * MC_KCH + ks * 2048, MC_KCH), idesc, (part > 0 || ks > 0) ? 1u : 0u);
+      }
+    }
+    umma_commit(done);
+  }
+  // dn[d] = sum of the weighted keys of dim d
+  if (tid < p.dk) {
+    float s = 0.f;
+    const uint8_t* base = mc_smem + (tid >> 6) * MC_KCH;
+    const int piece = (tid & 63) >> 3, within = (tid & 7) * 2;
+    for (int t = 0; t < len; ++t) {
+      const int off = t * 128 + ((piece ^ (t & 7)) << 4) + within;
+      s += __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(base + McStateSmem::K_HI + off)) +
+           __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(base + McStateSmem::K_LO + off));
+    }
+    c.dn[chh * p.dk + tid] = s;
+  }
+  mbar_wait(done, 0, abort_flag, c.status, STATUS_TIMEOUT_ACCUM);
+  __syncwarp();                       // the issuing lane of warp 1 rejoins before the warp-wide tensor-memory loads
+  tc_fence_after();
+  {
+    const int d = (warp & 3) * 32 + lane;                      // row of S (key dim)
+    const uint32_t trow = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
+    float* dst = c.dS + (chh * p.dk + d) * p.dv;
+#pragma unroll 1
+    for (int col = (warp >> 2) * 32; col < nv * 64; col += 64) {
+      float o[32];
+      tmem_ld32(trow + col, o);
+      tmem_ld_wait();
+      if (d < p.dk) {
+#pragma unroll
+        for (int e = 0; e < 32; e += 4)
+          if (col + e < p.dv) *reinterpret_cast<float4*>(dst + col + e) = make_float4(o[e], o[e + 1], o[e + 2], o[e + 3]);
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, 256);
+  }
+}
+
+// Scan over the chunks of a portion, element by element: grid (ceil(dk * dv / 4 / 256) + 1, heads, n_seq).  The last
+// block of x handles n and m.
+__global__ void __launch_bounds__(256) mlstm_chunk_scan_kernel(const MlstmParams p, const MlstmChunkParams c) {
+  const int h = blockIdx.y, s = blockIdx.z;
+  const int c0 = c.seq_chunk0[s], nc = c.seq_chunks[s];
+  if (nc <= 0) return;
+  const int t0 = c.c_start[c0];
+  const size_t sh = (size_t)p.row[t0] * p.heads + h;
+  const bool fresh = p.pos[t0] == 0;
+  float m = fresh ? 0.f : p.mval[sh];
+  const size_t per = (size_t)p.dk * p.dv;
+  if (blockIdx.x + 1 < gridDim.x) {
+    const int e = blockIdx.x * 256 + threadIdx.x;
+    if ((size_t)e * 4 >= per) return;
+    float4* Sp = reinterpret_cast<float4*>(p.S + sh * per) + e;
+    float4 S = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *Sp;
+#pragma unroll 4
+    for (int k = 0; k < nc; ++k) {
+      const size_t chh = (size_t)(c0 + k) * p.heads + h;
+      const float4 d = reinterpret_cast<const float4*>(c.dS + chh * per)[e];
+      uint32_t hi0, lo0, hi1, lo1;
+      split_bf16(S.x, S.y, hi0, lo0);
+      split_bf16(S.z, S.w, hi1, lo1);
+      reinterpret_cast<uint2*>(c.s0 + chh * 2 * per)[e] = make_uint2(hi0, hi1);
+      reinterpret_cast<uint2*>(c.s0 + (chh * 2 + 1) * per)[e] = make_uint2(lo0, lo1);
+      const float FL = c.cg[chh * 2], Bm = c.cg[chh * 2 + 1];
+      const float m_new = FL + fmaxf(m, Bm);
+      const float keep = expf(FL + m - m_new), add = expf(FL + Bm - m_new);
+      S.x = keep * S.x + add * d.x; S.y = keep * S.y + add * d.y;
+      S.z = keep * S.z + add * d.z; S.w = keep * S.w + add * d.w;
+      m = m_new;
+    }
+    *Sp = S;
+    return;
+  }
+  // n and the chunks' m (the slot's m itself is read by every block of this grid; the output kernel rewrites it)
+  float n[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int d = threadIdx.x + j * 256;
+    n[j] = d < p.dk && !fresh ? p.nvec[sh * p.dk + d] : 0.f;
+  }
+  for (int k = 0; k < nc; ++k) {
+    const size_t chh = (size_t)(c0 + k) * p.heads + h;
+    const float FL = c.cg[chh * 2], Bm = c.cg[chh * 2 + 1];
+    const float m_new = FL + fmaxf(m, Bm);
+    const float keep = expf(FL + m - m_new), add = expf(FL + Bm - m_new);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int d = threadIdx.x + j * 256;
+      if (d < p.dk) {
+        c.n0[chh * p.dk + d] = n[j];
+        n[j] = keep * n[j] + add * c.dn[chh * p.dk + d];
+      }
+    }
+    if (threadIdx.x == 0) c.m0[chh] = m;
+    m = m_new;
+  }
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int d = threadIdx.x + j * 256;
+    if (d < p.dk) p.nvec[sh * p.dk + d] = n[j];
+  }
+}
+
+// Outputs of one (chunk, head): grid (n_chunks, heads), 320 threads: warp 0 TMA, warp 1 tensor memory + MMA, warps 2..9
+// two threads per token.  Shared: Q (2 x 16 KiB), K then P hi (2 x 16 KiB), P lo (2 x 16 KiB), ring of 3 tiles of
+// 32 KiB: the slices (128 columns) of the incoming state, hi and lo, then the slices of V.
+struct McOutSmem {
+  static constexpr int Q = 0, K = 2 * MC_KCH, PLO = 4 * MC_KCH, RING = 6 * MC_KCH, TILE = 2 * MC_KCH, NRING = 3;
+  static constexpr int TAIL = RING + NRING * TILE;
+  static constexpr int BYTES = TAIL + 2304;
+};
+constexpr int MC_OUT_THREADS = 320;
+
+__global__ void __launch_bounds__(MC_OUT_THREADS, 1)
+mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_v,
+                       const __grid_constant__ CUtensorMap tm_s0, const MlstmParams p, const MlstmChunkParams c, const int nk,
+                       const int nv) {
+  extern __shared__ __align__(1024) uint8_t mc_smem[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int ch = blockIdx.x, h = blockIdx.y;
+  if ((smem_u32(mc_smem) & 1023u) != 0) {
+    if (tid == 0) atomicCAS(c.status, 0, STATUS_BAD_INDEX);
+    return;
+  }
+  float* s_B = reinterpret_cast<float*>(mc_smem + McOutSmem::TAIL);   // [128] B_s
+  float* s_A = s_B + MC_TOK;                                          // [128] F_t - m_t
+  float* s_n0 = s_A + MC_TOK;                                         // [128]
+  float* s_x = s_n0 + MC_TOK;                                         // [128] exchange (low half -> high half and back)
+  float* s_g = s_x + MC_TOK;                                          // [8]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_g + 8);
+  uint64_t* qk_full = bars;
+  uint64_t* full = bars + 1;                     // [NRING]
+  uint64_t* empty = full + McOutSmem::NRING;     // [NRING]
+  uint64_t* s_done = empty + McOutSmem::NRING;   // Q K^T complete
+  uint64_t* o2_done = s_done + 1;                // Q S0 complete
+  uint64_t* p_ready = o2_done + 1;               // P written, O scaled (256 arrivals)
+  uint64_t* o_done = p_ready + 1;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_done + 1);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  if (tid == 0) {
+    mbar_init(qk_full, 1);
+    for (int s = 0; s < McOutSmem::NRING; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
+    mbar_init(s_done, 1);
+    mbar_init(o2_done, 1);
+    mbar_init(p_ready, 256);
+    mbar_init(o_done, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 128;
+  const int start = c.c_start[ch], len = c.c_len[ch];
+  const size_t chh = (size_t)ch * p.heads + h;
+  const float m0 = c.m0[chh];
+  {
+    float F, B, Bmax;
+    chunk_gates(p.gates, p.heads, h, start, len, p.cap, s_g, F, B, Bmax);
+    if (tid < MC_TOK) {
+      s_B[tid] = B;
+      s_A[tid] = -fmaxf(m0, Bmax);               // F_t - m_t
+      s_n0[tid] = tid < p.dk ? c.n0[chh * p.dk + tid] : 0.f;
+      s_x[tid] = F;
+    }
+  }
+  __syncthreads();
+  const int slices = (nv + 1) / 2;
+  if (warp == 0) {
+    // ---------------- TMA producer ----------------
+    if (lane == 0) {
+      mbar_expect_tx(qk_full, 2 * nk * MC_KCH);
+      for (int k = 0; k < nk; ++k) {
+        tma_load_3d(mc_smem + McOutSmem::Q + k * MC_KCH, &tm_q, k * 64, h, start, qk_full);
+        tma_load_3d(mc_smem + McOutSmem::K + k * MC_KCH, &tm_q, k * 64, p.heads + h, start, qk_full);
+      }
+      for (int i = 0; i < 3 * slices; ++i) {
+        const int st = i % McOutSmem::NRING;
+        mbar_wait(&empty[st], ((i / McOutSmem::NRING) & 1) ^ 1, abort_flag, c.status, STATUS_TIMEOUT_STAGE_EMPTY);
+        if (*abort_flag) break;
+        uint8_t* dst = mc_smem + McOutSmem::RING + st * McOutSmem::TILE;
+        const bool state = i < 2 * slices;
+        const int sl = state ? i / 2 : i - 2 * slices;
+        const int cols = min(2, nv - 2 * sl);
+        const int bytes = state ? nk * 8192 : MC_KCH;         // one 64-column chunk: nk * 64 state rows, or 128 tokens
+        mbar_expect_tx(&full[st], cols * bytes);
+        for (int k = 0; k < cols; ++k) {
+          const int x = (2 * sl + k) * 64;
+          if (state) {
+            for (int r = 0; r < nk; ++r)
+              tma_load_3d(dst + k * bytes + r * 8192, &tm_s0, x, r * 64, (int)(chh * 2 + (i & 1)), &full[st]);
+          } else {
+            tma_load_3d(dst + k * bytes, &tm_v, x, h, start, &full[st]);
+          }
+        }
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    // ---------------- MMA issuer ----------------
+    if (lane == 0) {
+      const uint32_t q_addr = smem_u32(mc_smem + McOutSmem::Q), k_addr = smem_u32(mc_smem + McOutSmem::K);
+      const uint32_t plo_addr = smem_u32(mc_smem + McOutSmem::PLO);
+      mbar_wait(qk_full, 0, abort_flag, c.status, STATUS_TIMEOUT_TMA_FULL);
+      tc_fence_after();
+      for (int ks = 0; ks < nk * 4; ++ks) {
+        const uint32_t off = (ks / 4) * MC_KCH + (ks % 4) * 32;
+        umma_bf16(tmem_s, umma_desc_sw128(q_addr + off), umma_desc_sw128(k_addr + off), umma_idesc_bf16(128, 128), ks > 0 ? 1u : 0u);
+      }
+      umma_commit(s_done);
+      for (int i = 0; i < 3 * slices; ++i) {
+        const int st = i % McOutSmem::NRING;
+        if (i == 2 * slices) {
+          umma_commit(o2_done);
+          mbar_wait(p_ready, 0, abort_flag, c.status, STATUS_TIMEOUT_ACCUM);
+          tc_fence_after();
+        }
+        mbar_wait(&full[st], (i / McOutSmem::NRING) & 1, abort_flag, c.status, STATUS_TIMEOUT_TMA_FULL);
+        tc_fence_after();
+        const uint32_t b_addr = smem_u32(mc_smem + McOutSmem::RING + st * McOutSmem::TILE);
+        const bool state = i < 2 * slices;
+        const int sl = state ? i / 2 : i - 2 * slices;
+        const uint32_t idesc = umma_idesc_bf16_bmn(128, min(2, nv - 2 * sl) * 64);
+        const uint32_t d = tmem_o + sl * 128;
+        if (state) {
+          const uint32_t lbo = nk * 8192;
+          for (int ks = 0; ks < nk * 4; ++ks)
+            umma_bf16(d, umma_desc_sw128(q_addr + (ks / 4) * MC_KCH + (ks % 4) * 32), umma_desc_mn_sw128(b_addr + ks * 2048, lbo),
+                      idesc, (ks > 0 || (i & 1)) ? 1u : 0u);
+        } else {
+          for (int part = 0; part < 2; ++part) {
+            const uint32_t a_addr = part == 0 ? k_addr : plo_addr;
+            for (int ks = 0; ks < 8; ++ks)
+              umma_bf16(d, umma_desc_sw128(a_addr + (ks / 4) * MC_KCH + (ks % 4) * 32),
+                        umma_desc_mn_sw128(b_addr + ks * 2048, MC_KCH), idesc, 1u);
+          }
+        }
+        umma_commit(&empty[st]);
+      }
+      umma_commit(o_done);
+    }
+    __syncwarp();
+  } else {
+    // ---------------- two threads per token ----------------
+    const int qd = warp & 3, half = (warp - 2) >> 2;
+    const int t = qd * 32 + lane;
+    const bool ok = t < len;
+    const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
+    const float At = s_A[t];
+    const float m_t = s_x[t] - At;
+    const float a_t = ok ? expf(At + m0) * p.q_scale : 0.f;       // weight of the incoming state, q scaling included
+    named_bar_sync(1, 256);                                       // s_x is read; it becomes the exchange buffer
+    // n0 . q_t: this thread's 64 dims
+    mbar_wait(qk_full, 0, abort_flag, c.status, STATUS_TIMEOUT_TMA_FULL);
+    float nq = 0.f;
+    if (half < nk) {
+      const uint8_t* qr = mc_smem + McOutSmem::Q + half * MC_KCH + t * 128;
+#pragma unroll
+      for (int piece = 0; piece < 8; ++piece) {
+        const uint4 u = *reinterpret_cast<const uint4*>(qr + ((piece ^ (t & 7)) << 4));
+        const __nv_bfloat162* q2 = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 f = __bfloat1622float2(q2[e]);
+          nq = fmaf(f.x, s_n0[half * 64 + piece * 8 + 2 * e], nq);
+          nq = fmaf(f.y, s_n0[half * 64 + piece * 8 + 2 * e + 1], nq);
+        }
+      }
+    }
+    nq *= a_t;
+    // P = (q . k) * q_scale * exp(F_t - m_t + B_s) for s <= t: this thread's 64 columns, written over K and beside it
+    mbar_wait(s_done, 0, abort_flag, c.status, STATUS_TIMEOUT_ACCUM);
+    tc_fence_after();
+#pragma unroll 1
+    for (int c0 = 0; c0 < 64; c0 += 32) {
+      const int s0 = half * 64 + c0;
+      float sv[32];
+      tmem_ld32(tmem_s + lane_off + s0, sv);
+      tmem_ld_wait();
+#pragma unroll
+      for (int e = 0; e < 32; ++e) {
+        const int s = s0 + e;
+        sv[e] = ok && s <= t ? sv[e] * p.q_scale * expf(At + s_B[s]) : 0.f;
+        nq += sv[e];
+      }
+#pragma unroll
+      for (int v = 0; v < 4; ++v) {
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) split_bf16(sv[v * 8 + 2 * e], sv[v * 8 + 2 * e + 1], hi[e], lo[e]);
+        const int off = half * MC_KCH + t * 128 + (((c0 / 8 + v) ^ (t & 7)) << 4);
+        *reinterpret_cast<uint4*>(mc_smem + McOutSmem::K + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(mc_smem + McOutSmem::PLO + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      }
+    }
+    fence_proxy_async_smem();
+    // O = a_t * (Q S0): this thread's columns are half, half + 2, ... of the 32-column pieces
+    mbar_wait(o2_done, 0, abort_flag, c.status, STATUS_TIMEOUT_ACCUM);
+    tc_fence_after();
+#pragma unroll 1
+    for (int col = half * 32; col < nv * 64; col += 64) {
+      float o[32];
+      tmem_ld32(tmem_o + lane_off + col, o);
+      tmem_ld_wait();
+#pragma unroll
+      for (int e = 0; e < 32; ++e) o[e] *= a_t;
+      tmem_st32(tmem_o + lane_off + col, o);
+    }
+    tmem_st_wait();
+    tc_fence_before();
+    mbar_arrive(p_ready);
+    // n . q of the token: both halves
+    if (half == 1) s_x[t] = nq;
+    named_bar_sync(1, 256);
+    if (half == 0) { nq += s_x[t]; s_x[t] = nq; }
+    named_bar_sync(1, 256);
+    nq = s_x[t];
+    const float inv = 1.0f / (fmaxf(fabsf(nq), expf(-m_t)) + 1e-6f);
+    named_bar_sync(1, 256);
+    mbar_wait(o_done, 0, abort_flag, c.status, STATUS_TIMEOUT_ACCUM);
+    tc_fence_after();
+    float ss = 0.f;
+#pragma unroll 1
+    for (int col = half * 32; col < nv * 64; col += 64) {
+      float o[32];
+      tmem_ld32(tmem_o + lane_off + col, o);
+      tmem_ld_wait();
+#pragma unroll
+      for (int e = 0; e < 32; ++e) ss = fmaf(o[e], o[e], ss);
+    }
+    if (half == 1) s_x[t] = ss;
+    named_bar_sync(1, 256);
+    if (half == 0) { ss += s_x[t]; s_x[t] = ss; }
+    named_bar_sync(1, 256);
+    ss = s_x[t] * inv * inv;
+    const float r = inv / sqrtf(ss / (float)p.vdim + p.eps);
+    const __nv_bfloat16* g = reinterpret_cast<const __nv_bfloat16*>(p.qkvg) + (size_t)(start + (ok ? t : 0)) * p.ld +
+                             (size_t)2 * p.heads * p.dk + (size_t)(p.heads + h) * p.dv;
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(start + t) * p.ld_out + (size_t)h * p.dv;
+    const float* nw = p.norm_w + (size_t)h * p.dv;
+#pragma unroll 1
+    for (int col = half * 32; col < nv * 64; col += 64) {
+      float o[32];
+      tmem_ld32(tmem_o + lane_off + col, o);
+      tmem_ld_wait();
+      if (ok) {
+#pragma unroll
+        for (int v = 0; v < 32; v += 8) {
+          if (col + v < p.dv) {
+            const uint4 gu = *reinterpret_cast<const uint4*>(g + col + v);
+            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gu);
+            uint4 pk;
+            __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&pk);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 z = __bfloat1622float2(g2[e]);
+              const float2 w = *reinterpret_cast<const float2*>(nw + col + v + 2 * e);
+              p2[e] = __floats2bfloat162_rn(o[v + 2 * e] * r * w.x / (1.0f + __expf(-z.x)),
+                                            o[v + 2 * e + 1] * r * w.y / (1.0f + __expf(-z.y)));
+            }
+            *reinterpret_cast<uint4*>(out + col + v) = pk;
+          }
+        }
+      }
+    }
+    // the state's running maximum after the portion (the scan reads the old one): its last chunk writes it
+    if (half == 0 && t == len - 1) {
+      const bool last = ch + 1 == c.n_chunks || p.row[c.c_start[ch + 1]] != p.row[start];
+      if (last) p.mval[(size_t)p.row[start] * p.heads + h] = m_t;
+    }
+    tc_fence_before();
+  }
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_s, 512);
+  }
+}
+
+// [n tokens][heads of d dims] inside a row-major matrix of pitch ld: boxes of 128 tokens x 64 dims of one head
+static int make_head_map(CUtensorMap* m, const __nv_bfloat16* base, int d, int heads, long long n, long long ld) {
+  PfEncodeFn fn = pf_encode_fn();
+  if (fn == nullptr) return -1;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || d % 8 || ld % 8) return -2;
+  cuuint64_t dims[3] = {(cuuint64_t)d, (cuuint64_t)heads, (cuuint64_t)n};
+  cuuint64_t strides[2] = {(cuuint64_t)d * 2, (cuuint64_t)ld * 2};
+  cuuint32_t box[3] = {64u, 1u, (cuuint32_t)MC_TOK}, estr[3] = {1u, 1u, 1u};
+  CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<__nv_bfloat16*>(base), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -3;
+}
+static int make_state_map(CUtensorMap* m, const __nv_bfloat16* base, int dk, int dv, long long n) {
+  PfEncodeFn fn = pf_encode_fn();
+  if (fn == nullptr) return -1;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || dv % 8) return -2;
+  cuuint64_t dims[3] = {(cuuint64_t)dv, (cuuint64_t)dk, (cuuint64_t)n};
+  cuuint64_t strides[2] = {(cuuint64_t)dv * 2, (cuuint64_t)dk * dv * 2};
+  cuuint32_t box[3] = {64u, 64u, 1u}, estr[3] = {1u, 1u, 1u};
+  CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<__nv_bfloat16*>(base), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -3;
+}
+
 }  // namespace tahb
 
 using namespace tahb;
@@ -167,4 +753,30 @@ extern "C" int tahb_mlstm_recurrent(const MlstmParams* p, int f32, cudaStream_t 
   cudaError_t e = f32 ? launch_chain(mlstm_recurrent_kernel<float>, grid, dim3(MR_THREADS), smem, stream, *p)
                       : launch_chain(mlstm_recurrent_kernel<__nv_bfloat16>, grid, dim3(MR_THREADS), smem, stream, *p);
   return e == cudaSuccess ? 0 : -3;
+}
+
+// Chunkwise form: bf16 activations, dk <= 128, dv <= 256.  `n_tokens` = rows of qkvg.
+extern "C" int tahb_mlstm_chunks(const MlstmParams* p, const MlstmChunkParams* c, int n_tokens, cudaStream_t stream) {
+  if (p->n_seq <= 0 || c->n_chunks <= 0) return 0;
+  if (p->dk % 8 || p->dv % 8 || p->dk > 128 || p->dv > 256 || p->n_seq > 65535 || p->heads > 65535 || p->ld_out % 8) return -2;
+  const int nk = (p->dk + 63) / 64, nv = (p->dv + 63) / 64;
+  auto base = reinterpret_cast<const __nv_bfloat16*>(p->qkvg);
+  CUtensorMap mq, mv, ms;
+  int rc;
+  if ((rc = make_head_map(&mq, base, p->dk, 2 * p->heads, n_tokens, p->ld))) return rc;
+  if ((rc = make_head_map(&mv, base + (size_t)2 * p->heads * p->dk, p->dv, 2 * p->heads, n_tokens, p->ld))) return rc;
+  if ((rc = make_state_map(&ms, c->s0, p->dk, p->dv, (long long)c->n_chunks * p->heads * 2))) return rc;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(mlstm_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, McStateSmem::bytes(4)) != cudaSuccess ||
+        cudaFuncSetAttribute(mlstm_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, McOutSmem::BYTES) != cudaSuccess)
+      return -10;
+    configured = true;
+  }
+  const dim3 grid(c->n_chunks, p->heads);
+  mlstm_chunk_state_kernel<<<grid, 256, McStateSmem::bytes(nv), stream>>>(mq, mv, *p, *c, nv);
+  const int blocks = (int)(((long long)p->dk * p->dv / 4 + 255) / 256) + 1;
+  mlstm_chunk_scan_kernel<<<dim3(blocks, p->heads, p->n_seq), 256, 0, stream>>>(*p, *c);
+  mlstm_chunk_out_kernel<<<grid, MC_OUT_THREADS, McOutSmem::BYTES, stream>>>(mq, mv, ms, *p, *c, nk, nv);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

@@ -15,6 +15,7 @@ to multiples of 8, with zeros that drop out of every result.
 """
 from __future__ import annotations
 
+import os
 from dataclasses import dataclass
 from typing import List, Optional, Sequence
 
@@ -27,6 +28,9 @@ from tah_b200.ops import cuda as K
 from tah_b200.utils.observe import nvtx_range
 
 NO_WINDOW = 2 ** 31 - 1
+LOG2E = 1.4426950408889634
+TILE = 128                        # tokens of an attention query tile and of an mLSTM chunk
+MEMORY_CHUNKS = 192               # chunks per mLSTM launch (bounds the workspace)
 
 
 def _pad(n: int, m: int) -> int:
@@ -63,7 +67,7 @@ class AttentionLayer:
     gate_col: int
     q_norm: torch.Tensor
     k_norm: Optional[torch.Tensor]
-    bias: torch.Tensor            # [heads, far + 1]
+    bias: torch.Tensor            # [heads, far + 1], natural units for the plain kernel, log2 units for the others
     sink: torch.Tensor
     w_o: torch.Tensor
 
@@ -94,8 +98,9 @@ class BlockWeights:
 class HybridWeights:
     """Kernel-ready layout of a Gunuvik model's weights in the activation type ``dtype``."""
 
-    def __init__(self, model: GunuvikForCausalLM, dtype: torch.dtype):
+    def __init__(self, model: GunuvikForCausalLM, dtype: torch.dtype, plain: bool):
         cfg = model.config
+        unit = 1.0 if plain else LOG2E
         dev = model.device
         self.W, self.Wp = cfg.hidden_size, _pad(cfg.hidden_size, 64)
         self.vocab = cfg.vocab_size
@@ -154,7 +159,7 @@ class HybridWeights:
                 w_in = stack(rows + [heads_rows(T(x + "g"), H, 1, 1)])
                 mixer = AttentionLayer(m, dk, dv, G if own else 0, w_in, vec(torch.cat(bias), w_in.shape[0]), gate_col,
                                        vec(T(x + "q.norm"), dk), vec(T(x + "k.norm"), dk) if own else None,
-                                       distance_table(T(x + "rel"), m.bias_max), vec(T(x + "sink"), H), w_o)
+                                       distance_table(T(x + "rel"), m.bias_max) * unit, vec(T(x + "sink"), H) * unit, w_o)
             else:
                 if max(dk, dv) > 1024:
                     raise NotImplementedError("mLSTM head sizes above 1024")
@@ -178,19 +183,29 @@ class HybridWeights:
 class _Plan:
     """Which tokens a pass runs: packed token ids, positions, cache rows and KV slots.  The first ``n_dec`` tokens are
     single tokens of a row each; behind them lie the prompt portions, portion ``e`` at ``seq_start[e]``,
-    ``seq_len[e]`` tokens long, cut into query tiles of up to 128 tokens."""
+    ``seq_len[e]`` tokens long, cut into tiles of up to 128 tokens (attention query tiles and mLSTM chunks)."""
     tok = pos = row = slot = None
     n_dec = 0
     seq_start = seq_len = None
     tile_q0 = tile_qn = None
-    n_split = 1
-    ws = None
+    groups = ()                   # mLSTM launches: (tiles a..b, first tile and tile count of each of their portions)
+
+
+def decode_splits(m: AttentionLayer, n: int) -> int:
+    """Key splits of the decode attention: enough CTAs to fill the SMs at small batches, at least four pages each."""
+    if n == 0:
+        return 1
+    g = m.spec.heads // m.spec.kv_heads
+    ctas = n * m.spec.kv_heads * ((g + 3) // 4)
+    pages = 64 if m.spec.window is None else (m.spec.window + m.spec.keep_first) // 16 + 1
+    return max(1, min(K.SM_COUNT * 4 // ctas, pages // 4, 16))
 
 
 class _Buffers:
-    """Activations of a pass over ``n`` tokens."""
+    """Activations of a pass over ``n`` tokens, the first ``n_dec`` of them single tokens; ``chunks``: mLSTM chunks of a
+    launch."""
 
-    def __init__(self, w: HybridWeights, n: int, dtype, dev):
+    def __init__(self, w: HybridWeights, n: int, dtype, dev, n_dec: int, chunks: int = 0):
         e = lambda *s: torch.empty(*s, dtype=dtype, device=dev)
         mix = [b.mixer for b in w.layers]
         self.x = torch.empty(n, w.Wp, dtype=torch.float32, device=dev)
@@ -201,6 +216,11 @@ class _Buffers:
         self.o = torch.zeros(n, max(m.w_o.shape[1] for m in mix), dtype=dtype, device=dev)
         self.gates = torch.empty(n * max([m.w_if.shape[0] for m in mix if isinstance(m, MemoryLayer)] or [0]),
                                  dtype=torch.float32, device=dev)
+        f32 = lambda k: torch.empty(k, dtype=torch.float32, device=dev)
+        self.attn_ws = f32(max([n_dec * m.spec.heads * decode_splits(m, n_dec) * (m.dv + 2) for m in mix
+                                if isinstance(m, AttentionLayer)] or [0]))
+        self.mem_ws = f32(max([K.mlstm_chunk_ws_floats(chunks, m.spec.heads, m.dk, m.dv) for m in mix
+                               if isinstance(m, MemoryLayer)] or [0]))
         self.act = e(n, max([b.w_down.shape[1] for b in w.layers if b.w_down is not None] or [0]))
 
 
@@ -224,7 +244,10 @@ class HybridEngine(DecodeEngine):
         if self.dtype not in (torch.bfloat16, torch.float32):
             raise ValueError(f"HybridEngine runs in bfloat16 or float32, not {self.dtype}")
         self.max_iter, self.topk, self.tp = 1, 1, None
-        self.w = HybridWeights(model, self.dtype)
+        # the plain kernels (any page size, fp32; bring-up and comparison in bf16) instead of the tensor-core / pipelined ones
+        self.plain = (self.dtype != torch.bfloat16 or page_size != 16
+                      or os.environ.get("TAH_B200_NAIVE_PREFILL", "0") == "1")
+        self.w = HybridWeights(model, self.dtype, self.plain)
         self.prefill_tokens = prefill_tokens
         self.state: Optional[RecurrentState] = None
         self._free_rows: List[int] = []
@@ -282,8 +305,15 @@ class HybridEngine(DecodeEngine):
         o = b.o[:, :m.w_o.shape[1]]
         kw = dict(nq=s.heads, nkv=s.kv_heads, dk=m.dk, dv=m.dv, page_size=self.page_size, scale=s.scale,
                   window=NO_WINDOW if s.window is None else s.window, keep_first=s.keep_first, bias=m.bias, sink=m.sink)
-        gate = proj[:, m.gate_col:m.gate_col + s.heads]
-        K.window_attn_plain(q, o, pool, self.kv.page_table[0], plan.pos, plan.row, gate=gate, **kw)
+        gate, pt, nd = proj[:, m.gate_col:m.gate_col + s.heads], self.kv.page_table[0], plan.n_dec
+        if self.plain:
+            K.window_attn_plain(q, o, pool, pt, plan.pos, plan.row, gate=gate, **kw)
+            return o
+        if nd:
+            K.window_attn_decode(q[:nd], o[:nd], pool, pt, plan.pos, plan.row, gate=gate, n_split=decode_splits(m, nd),
+                                 ws=b.attn_ws, **kw)
+        if nd < n:
+            K.window_attn_tiles(q, o, pool, pt, plan.pos, plan.row, plan.tile_q0, plan.tile_qn, self.kv.n_pages[0], gate=gate, **kw)
         return o
 
     def _memory(self, li: int, m: MemoryLayer, b: _Buffers, plan: _Plan) -> torch.Tensor:
@@ -296,9 +326,13 @@ class HybridEngine(DecodeEngine):
         state = self.state.layers[li]
         if nd:
             K.mlstm_recurrent(proj[:nd], gates[:nd], m.norm, o[:nd], state, plan.pos, plan.row, slot=plan.slot, **kw)
-        if nd < n:
+        if nd < n and (self.plain or m.dk > 128 or m.dv > 256):
             K.mlstm_recurrent(proj, gates, m.norm, o, state, plan.pos, plan.row, seq_start=plan.seq_start,
                               seq_len=plan.seq_len, **kw)
+        elif nd < n:
+            for ta, tb, chunk0, chunks in plan.groups:
+                K.mlstm_chunks(proj, gates, m.norm, o, state, plan.pos, plan.row, chunk_start=plan.tile_q0[ta:tb],
+                               chunk_len=plan.tile_qn[ta:tb], seq_chunk0=chunk0, seq_chunks=chunks, ws=b.mem_ws, **kw)
         return o
 
     def _layers(self, b: _Buffers, plan: _Plan) -> torch.Tensor:
@@ -347,26 +381,33 @@ class HybridEngine(DecodeEngine):
             want = [place[i] for i in want]
             start = new_start
         rows, counts, start = [rows[e] for e in order], [counts[e] for e in order], [start[e] for e in order]
-        q0, qn = [], []
+        q0, qn, first_tile, tiles, groups = [], [], [], [], []
         for s0, c in zip(start[n_dec:], counts[n_dec:]):
-            for a in range(0, c, 128):
-                q0.append(s0 + a)
-                qn.append(min(128, c - a))
-        ne, nt, nw = len(rows), len(q0), len(want)
-        meta = torch.tensor(rows + counts + start + q0 + qn + list(want), dtype=torch.int32).pin_memory().to(dev, non_blocking=True)
-        d_rows, d_counts, d_start, d_q0, d_qn, d_want = meta.split([ne, ne, ne, nt, nt, nw])
+            k = (c + TILE - 1) // TILE
+            if not groups or groups[-1][3] + k > MEMORY_CHUNKS:
+                groups.append([len(first_tile), len(first_tile), len(q0), 0])       # portions a..b, first tile, tiles
+            groups[-1][1] += 1
+            first_tile.append(groups[-1][3])
+            tiles.append(k)
+            groups[-1][3] += k
+            q0 += [s0 + a for a in range(0, c, TILE)]
+            qn += [min(TILE, c - a) for a in range(0, c, TILE)]
+        parts = [rows, counts, start, q0, qn, first_tile, tiles, list(want)]
+        meta = torch.tensor(sum(parts, []), dtype=torch.int32).pin_memory().to(dev, non_blocking=True)
+        d_rows, d_counts, d_start, d_q0, d_qn, d_first, d_tiles, d_want = meta.split([len(p) for p in parts])
         plan = _Plan()
         plan.tok = tok
         plan.pos, plan.row, plan.slot = (torch.empty(n, dtype=torch.int32, device=dev) for _ in range(3))
         plan.n_dec = n_dec
         plan.seq_start, plan.seq_len = d_start[n_dec:], d_counts[n_dec:]
         plan.tile_q0, plan.tile_qn = d_q0, d_qn
+        plan.groups = [(t, t + k, d_first[a:z], d_tiles[a:z]) for a, z, t, k in groups]
         K.kv_append(d_rows, d_counts, d_start, self.kv, 0, plan.pos, plan.row, plan.slot)
-        b = _Buffers(self.w, n, self.dtype, dev)
+        b = _Buffers(self.w, n, self.dtype, dev, n_dec, 0 if self.plain else max([g[3] for g in groups] or [0]))
         K.embed_norm(self.w.embed, plan.tok, self.cfg.embedding_scale, self.w.layers[0].norm1, self.w.W,
                      self.cfg.rms_norm_eps, b.x, b.h)
         h = self._layers(b, plan)
-        if nw == 0:
+        if not want:
             return torch.empty(0, self.w.vocab, dtype=self.dtype, device=dev)
         return K.linear(h[d_want.long()], self.w.head)[:, :self.w.vocab]
 
@@ -448,7 +489,7 @@ class HybridEngine(DecodeEngine):
     def _alloc_tick_buffers(self, B: int, max_new: int):
         s = self._alloc_scheduler_state(B, max_new)
         dev = self.device
-        s.buf = _Buffers(self.w, B, self.dtype, dev)
+        s.buf = _Buffers(self.w, B, self.dtype, dev, B)
         s.plan = _Plan()
         s.plan.tok, s.plan.pos, s.plan.slot = s.tok, s.pos, s.slot
         s.plan.row = torch.arange(B, dtype=torch.int32, device=dev)

@@ -671,6 +671,23 @@ def window_attn_plain(q, out, pool, page_table, pos, row, **kw):
     return out
 
 
+def window_attn_decode(q, out, pool, page_table, pos, row, **kw):
+    """Windowed attention of single tokens (bf16, pages of 16): pipelined page copies, optional key splits (``n_split``,
+    ``ws`` of ``n * nq * n_split * (dv + 2)`` floats).  ``bias`` and ``sink`` in log2 units."""
+    a = window_attn_args(q, out, pool, page_table, pos, row, **kw)
+    _rc(lib().tahb_window_attn_decode(ctypes.byref(a), _stream()), "tahb_window_attn_decode")
+    return out
+
+
+def window_attn_tiles(q, out, pool, page_table, pos, row, tile_q0, tile_qn, n_pages: int, **kw):
+    """Windowed attention of prompt portions on the tensor cores (bf16, pages of 16): tiles of up to 128 consecutive
+    tokens of one row.  ``bias`` and ``sink`` in log2 units."""
+    a = window_attn_args(q, out, pool, page_table, pos, row, **kw)
+    _rc(lib().tahb_window_attn_tiles(ctypes.byref(a), _p(tile_q0), _p(tile_qn), c_int(tile_q0.numel()), c_int(n_pages),
+                                     _stream()), "tahb_window_attn_tiles")
+    return out
+
+
 class _Mlstm(ctypes.Structure):
     _fields_ = [(n, c_void_p) for n in ("qkvg", "gates", "norm_w", "out", "S", "nvec", "mval", "seq_start", "seq_len", "pos",
                                         "row", "slot")] + \
@@ -690,6 +707,36 @@ def mlstm_args(qkvg, gates, norm_w, out, state, pos, row, *, heads: int, dk: int
     a.heads, a.dk, a.dv, a.dim, a.vdim = heads, dk, dv, dim, vdim
     a.ld, a.ld_out, a.cap, a.eps, a.q_scale = qkvg.stride(0), out.stride(0), cap, eps, dim ** -0.5
     return a
+
+
+class _MlstmChunks(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("c_start", "c_len", "seq_chunk0", "seq_chunks", "dS", "dn", "cg", "s0", "n0", "m0")] + \
+               [("n_chunks", c_int), ("status", c_void_p)]
+
+
+def mlstm_chunk_ws_floats(n_chunks: int, heads: int, dk: int, dv: int) -> int:
+    """fp32 workspace of :func:`mlstm_chunks`: dS, the incoming state as a bf16 pair, dn, n0, chunk scalars."""
+    return n_chunks * heads * (2 * dk * dv + 2 * dk + 4)
+
+
+def mlstm_chunks(qkvg, gates, norm_w, out, state, pos, row, *, chunk_start, chunk_len, seq_chunk0, seq_chunks, ws, **kw):
+    """mLSTM of prompt portions in chunks of up to 128 tokens on the tensor cores (bf16, dk <= 128, dv <= 256); updates
+    ``state`` in place.  Chunk ``c`` = tokens ``chunk_start[c] .. + chunk_len[c]``; portion ``s`` = chunks ``seq_chunk0[s]
+    .. + seq_chunks[s]``."""
+    a = mlstm_args(qkvg, gates, norm_w, out, state, pos, row, **kw)
+    a.n_seq = seq_chunk0.shape[0]
+    heads, dk, dv, n = kw["heads"], kw["dk"], kw["dv"], chunk_start.shape[0]
+    c = _MlstmChunks()
+    c.c_start, c.c_len, c.seq_chunk0, c.seq_chunks = (t.data_ptr() for t in (chunk_start, chunk_len, seq_chunk0, seq_chunks))
+    at = ws.data_ptr()
+    if ws.numel() < mlstm_chunk_ws_floats(n, heads, dk, dv):
+        raise ValueError("mlstm_chunks: workspace too small")
+    for name, floats in (("dS", dk * dv), ("s0", dk * dv), ("dn", dk), ("n0", dk), ("cg", 2), ("m0", 1)):
+        setattr(c, name, at)
+        at += 4 * n * heads * floats
+    c.n_chunks, c.status = n, status_word(qkvg.device).data_ptr()
+    _rc(lib().tahb_mlstm_chunks(ctypes.byref(a), ctypes.byref(c), c_int(qkvg.shape[0]), _stream()), "tahb_mlstm_chunks")
+    return out
 
 
 def mlstm_recurrent(qkvg, gates, norm_w, out, state, pos, row, **kw):
