@@ -60,7 +60,7 @@ constexpr int MR_THREADS = 256;
 constexpr int MR_MAX_D = 1024;
 
 template <typename T>
-__global__ void __launch_bounds__(MR_THREADS) mlstm_recurrent_kernel(const MlstmParams p) {
+__global__ void __launch_bounds__(MR_THREADS, 3) mlstm_recurrent_kernel(const MlstmParams p) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float sm[];
@@ -113,7 +113,7 @@ __global__ void __launch_bounds__(MR_THREADS) mlstm_recurrent_kernel(const Mlstm
     if (rg < nrg) {
       const float4 vv = ldf4(v + c * 4);
       float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
+#pragma unroll 8
       for (int r = rg; r < dk; r += nrg) {
         float4* sp = reinterpret_cast<float4*>(S + (size_t)r * dv) + c;
         float4 a = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *sp;
@@ -198,14 +198,20 @@ __device__ __forceinline__ void tma_load_3d(void* smem_dst, const void* tmap, in
       ::"r"(smem_u32(smem_dst)), "l"(reinterpret_cast<uint64_t>(tmap)), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2)
       : "memory");
 }
+__device__ __forceinline__ void tma_store_3d(const void* tmap, const void* smem_src, int c0, int c1, int c2) {
+  asm volatile("cp.async.bulk.tensor.3d.global.shared::cta.bulk_group [%0, {%2, %3, %4}], [%1];"
+               ::"l"(reinterpret_cast<uint64_t>(tmap)), "r"(smem_u32(smem_src)), "r"(c0), "r"(c1), "r"(c2)
+               : "memory");
+}
+constexpr float MC_LOG2E = 1.4426950408889634f;
 // A MN-major (transposed), B MN-major
 __host__ __device__ constexpr uint32_t umma_idesc_bf16_amn_bmn(int m, int n) { return umma_idesc_bf16(m, n) | (1u << 15) | (1u << 16); }
 
-// Gate scan of a chunk by the first 128 threads of the block (every thread calls it): token t = tid < 128.
+// Gate scan of a chunk by 256 threads (named barrier 1), t = their index; tokens are t < 128.
 // F = inclusive sum of the log forget gates, B = log_i - F, Bmax = inclusive prefix maximum of B.  xw: 8 floats.
 __device__ __forceinline__ void chunk_gates(const float* gates, int heads, int h, int start, int len, float cap, float* xw,
-                                            float& F, float& B, float& Bmax) {
-  const int t = threadIdx.x, lane = t & 31, w = t >> 5;
+                                            int t, float& F, float& B, float& Bmax) {
+  const int lane = t & 31, w = t >> 5;
   F = 0.f;
   B = -INFINITY;
   float li = -INFINITY;
@@ -219,7 +225,7 @@ __device__ __forceinline__ void chunk_gates(const float* gates, int heads, int h
     if (lane >= o) F += v;
   }
   if (w < 4 && lane == 31) xw[w] = F;
-  __syncthreads();
+  named_bar_sync(1, 256);
   for (int k = 0; k < min(w, 4); ++k) F += xw[k];
   if (t < len) B = li - F;
   Bmax = B;
@@ -229,7 +235,7 @@ __device__ __forceinline__ void chunk_gates(const float* gates, int heads, int h
     if (lane >= o) Bmax = fmaxf(Bmax, v);
   }
   if (w < 4 && lane == 31) xw[4 + w] = Bmax;
-  __syncthreads();
+  named_bar_sync(1, 256);
   for (int k = 0; k < min(w, 4); ++k) Bmax = fmaxf(Bmax, xw[4 + k]);
 }
 
@@ -241,26 +247,26 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint3
   lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
-// dS of one (chunk, head): grid (n_chunks, heads), 256 threads.  Shared: K hi and lo (2 chunks of 16 KiB each), V (nv
-// chunks of 16 KiB).
+// 128 columns of dS of one (chunk, head): grid (n_chunks, heads, ceil(nv / 2)), 256 threads, two CTAs per SM.  Shared: K hi
+// and lo (2 chunks of 16 KiB each), V (2 chunks of 16 KiB).
 struct McStateSmem {
-  static constexpr int K_HI = 0, K_LO = 2 * MC_KCH, V = 4 * MC_KCH;
-  static int bytes(int nv) { return (4 + nv) * MC_KCH + 1024; }
+  static constexpr int K_HI = 0, K_LO = 2 * MC_KCH, V = 4 * MC_KCH, TAIL = 6 * MC_KCH;
+  static constexpr int BYTES = TAIL + 2048;
 };
 
-__global__ void __launch_bounds__(256, 1)
+__global__ void __launch_bounds__(256, 2)
 mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
-                         const MlstmParams p, const MlstmChunkParams c, const int nv) {
+                         const MlstmParams p, const MlstmChunkParams c, const int nv_all) {
   extern __shared__ __align__(1024) uint8_t mc_smem[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int ch = blockIdx.x, h = blockIdx.y;
+  const int ch = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * 2, nv = min(2, nv_all - v0);
   if ((smem_u32(mc_smem) & 1023u) != 0) {
     if (tid == 0) atomicCAS(c.status, 0, STATUS_BAD_INDEX);
     return;
   }
-  uint8_t* tail = mc_smem + McStateSmem::V + nv * MC_KCH;
-  float* s_w = reinterpret_cast<float*>(tail);                 // [128] weight of each token
-  float* s_x = s_w + MC_TOK;                                   // [8]
+  float* s_w = reinterpret_cast<float*>(mc_smem + McStateSmem::TAIL);   // [128] weight of each token
+  float* s_dn = s_w + MC_TOK;                                  // [128] half sums of dn
+  float* s_x = s_dn + MC_TOK;                                  // [8]
   uint64_t* full = reinterpret_cast<uint64_t*>(s_x + 8);
   uint64_t* done = full + 1;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(done + 1);
@@ -272,7 +278,7 @@ mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
     mbar_fence_init();
   }
   if (warp == 1) {
-    tmem_alloc(tmem_slot, 256);
+    tmem_alloc(tmem_slot, 128);
     tmem_relinquish();
   }
   tc_fence_before();
@@ -283,16 +289,16 @@ mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   if (tid == 0) {
     mbar_expect_tx(full, (2 + nv) * MC_KCH);
     for (int k = 0; k < 2; ++k) tma_load_3d(mc_smem + McStateSmem::K_HI + k * MC_KCH, &tm_k, k * 64, p.heads + h, start, full);
-    for (int k = 0; k < nv; ++k) tma_load_3d(mc_smem + McStateSmem::V + k * MC_KCH, &tm_v, k * 64, h, start, full);
+    for (int k = 0; k < nv; ++k) tma_load_3d(mc_smem + McStateSmem::V + k * MC_KCH, &tm_v, (v0 + k) * 64, h, start, full);
   }
   float F, B, Bmax;
-  chunk_gates(p.gates, p.heads, h, start, len, p.cap, s_x, F, B, Bmax);
+  chunk_gates(p.gates, p.heads, h, start, len, p.cap, s_x, tid, F, B, Bmax);
   float* s_last = reinterpret_cast<float*>(tmem_slot + 2);     // [2] F and prefix maximum of the chunk's last token
   if (tid == len - 1) { s_last[0] = F; s_last[1] = Bmax; }
   __syncthreads();
   const size_t chh = (size_t)ch * p.heads + h;
   if (tid < MC_TOK) s_w[tid] = tid < len ? expf(B - s_last[1]) : 0.f;
-  if (tid == 0) { c.cg[chh * 2] = s_last[0]; c.cg[chh * 2 + 1] = s_last[1]; }
+  if (tid == 0 && v0 == 0) { c.cg[chh * 2] = s_last[0]; c.cg[chh * 2 + 1] = s_last[1]; }
   __syncthreads();
   mbar_wait(full, 0, abort_flag, c.status, STATUS_TIMEOUT_TMA_FULL);
   // weighted keys: hi in place, lo beside them (16 bytes = 8 dims of one token per step; the swizzle only permutes
@@ -317,38 +323,40 @@ mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   if (tid == 32) {
     tc_fence_after();
     const uint32_t v_addr = smem_u32(mc_smem + McStateSmem::V);
-    for (int v0 = 0; v0 < nv; v0 += 2) {
-      const int n = v0 + 1 < nv ? 128 : 64;
-      const uint32_t idesc = umma_idesc_bf16_amn_bmn(128, n);
-      for (int part = 0; part < 2; ++part) {
-        const uint32_t a_addr = smem_u32(mc_smem + (part == 0 ? McStateSmem::K_HI : McStateSmem::K_LO));
+    const uint32_t idesc = umma_idesc_bf16_amn_bmn(128, nv * 64);
+    for (int part = 0; part < 2; ++part) {
+      const uint32_t a_addr = smem_u32(mc_smem + (part == 0 ? McStateSmem::K_HI : McStateSmem::K_LO));
 #pragma unroll
-        for (int ks = 0; ks < MC_TOK / 16; ++ks)
-          umma_bf16(tmem + v0 * 64, umma_desc_mn_sw128(a_addr + ks * 2048, MC_KCH),
-                    umma_desc_mn_sw128(v_addr + v0 * MC_KCH + ks * 2048, MC_KCH), idesc, (part > 0 || ks > 0) ? 1u : 0u);
-      }
+      for (int ks = 0; ks < MC_TOK / 16; ++ks)
+        umma_bf16(tmem, umma_desc_mn_sw128(a_addr + ks * 2048, MC_KCH), umma_desc_mn_sw128(v_addr + ks * 2048, MC_KCH), idesc,
+                  (part > 0 || ks > 0) ? 1u : 0u);
     }
     umma_commit(done);
   }
-  // dn[d] = sum of the weighted keys of dim d
-  if (tid < p.dk) {
-    float s = 0.f;
-    const uint8_t* base = mc_smem + (tid >> 6) * MC_KCH;
-    const int piece = (tid & 63) >> 3, within = (tid & 7) * 2;
-    for (int t = 0; t < len; ++t) {
+  __syncwarp();                       // the issuing lane of warp 1 rejoins
+  // dn[d] = sum of the weighted keys of dim d: two threads per dim, 64 tokens each
+  if (v0 == 0) {
+    const int d = tid & (MC_TOK - 1), th = tid >> 7;
+    float s0 = 0.f, s1 = 0.f;
+    const uint8_t* base = mc_smem + (d >> 6) * MC_KCH;
+    const int piece = (d & 63) >> 3, within = (d & 7) * 2;
+#pragma unroll 8
+    for (int t = th * 64; t < th * 64 + 64; ++t) {             // tokens past the end weigh zero
       const int off = t * 128 + ((piece ^ (t & 7)) << 4) + within;
-      s += __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(base + McStateSmem::K_HI + off)) +
-           __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(base + McStateSmem::K_LO + off));
+      s0 += __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(base + McStateSmem::K_HI + off));
+      s1 += __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(base + McStateSmem::K_LO + off));
     }
-    c.dn[chh * p.dk + tid] = s;
+    if (th == 1) s_dn[d] = s0 + s1;
+    __syncthreads();
+    if (th == 0 && d < p.dk) c.dn[chh * p.dk + d] = s0 + s1 + s_dn[d];
   }
   mbar_wait(done, 0, abort_flag, c.status, STATUS_TIMEOUT_ACCUM);
-  __syncwarp();                       // the issuing lane of warp 1 rejoins before the warp-wide tensor-memory loads
+  __syncwarp();
   tc_fence_after();
   {
     const int d = (warp & 3) * 32 + lane;                      // row of S (key dim)
     const uint32_t trow = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
-    float* dst = c.dS + (chh * p.dk + d) * p.dv;
+    float* dst = c.dS + (chh * p.dk + d) * p.dv + v0 * 64;
 #pragma unroll 1
     for (int col = (warp >> 2) * 32; col < nv * 64; col += 64) {
       float o[32];
@@ -357,7 +365,7 @@ mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
       if (d < p.dk) {
 #pragma unroll
         for (int e = 0; e < 32; e += 4)
-          if (col + e < p.dv) *reinterpret_cast<float4*>(dst + col + e) = make_float4(o[e], o[e + 1], o[e + 2], o[e + 3]);
+          if (v0 * 64 + col + e < p.dv) *reinterpret_cast<float4*>(dst + col + e) = make_float4(o[e], o[e + 1], o[e + 2], o[e + 3]);
       }
     }
   }
@@ -365,7 +373,7 @@ mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tmem, 256);
+    tmem_dealloc(tmem, 128);
   }
 }
 
@@ -436,7 +444,8 @@ __global__ void __launch_bounds__(256) mlstm_chunk_scan_kernel(const MlstmParams
 
 // Outputs of one (chunk, head): grid (n_chunks, heads), 320 threads: warp 0 TMA, warp 1 tensor memory + MMA, warps 2..9
 // two threads per token.  Shared: Q (2 x 16 KiB), K then P hi (2 x 16 KiB), P lo (2 x 16 KiB), ring of 3 tiles of
-// 32 KiB: the slices (128 columns) of the incoming state, hi and lo, then the slices of V.
+// 32 KiB: the slices (128 columns) of the incoming state, hi and lo, then the slices of V, then those of the output gate,
+// which the outputs replace in place on their way to a TMA store (a chunk of fewer than 128 tokens stores row by row).
 struct McOutSmem {
   static constexpr int Q = 0, K = 2 * MC_KCH, PLO = 4 * MC_KCH, RING = 6 * MC_KCH, TILE = 2 * MC_KCH, NRING = 3;
   static constexpr int TAIL = RING + NRING * TILE;
@@ -446,8 +455,8 @@ constexpr int MC_OUT_THREADS = 320;
 
 __global__ void __launch_bounds__(MC_OUT_THREADS, 1)
 mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_v,
-                       const __grid_constant__ CUtensorMap tm_s0, const MlstmParams p, const MlstmChunkParams c, const int nk,
-                       const int nv) {
+                       const __grid_constant__ CUtensorMap tm_s0, const __grid_constant__ CUtensorMap tm_out,
+                       const MlstmParams p, const MlstmChunkParams c, const int nk, const int nv) {
   extern __shared__ __align__(1024) uint8_t mc_smem[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int ch = blockIdx.x, h = blockIdx.y;
@@ -490,18 +499,6 @@ mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
   const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 128;
   const int start = c.c_start[ch], len = c.c_len[ch];
   const size_t chh = (size_t)ch * p.heads + h;
-  const float m0 = c.m0[chh];
-  {
-    float F, B, Bmax;
-    chunk_gates(p.gates, p.heads, h, start, len, p.cap, s_g, F, B, Bmax);
-    if (tid < MC_TOK) {
-      s_B[tid] = B;
-      s_A[tid] = -fmaxf(m0, Bmax);               // F_t - m_t
-      s_n0[tid] = tid < p.dk ? c.n0[chh * p.dk + tid] : 0.f;
-      s_x[tid] = F;
-    }
-  }
-  __syncthreads();
   const int slices = (nv + 1) / 2;
   if (warp == 0) {
     // ---------------- TMA producer ----------------
@@ -511,13 +508,13 @@ mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         tma_load_3d(mc_smem + McOutSmem::Q + k * MC_KCH, &tm_q, k * 64, h, start, qk_full);
         tma_load_3d(mc_smem + McOutSmem::K + k * MC_KCH, &tm_q, k * 64, p.heads + h, start, qk_full);
       }
-      for (int i = 0; i < 3 * slices; ++i) {
+      for (int i = 0; i < 4 * slices; ++i) {
         const int st = i % McOutSmem::NRING;
         mbar_wait(&empty[st], ((i / McOutSmem::NRING) & 1) ^ 1, abort_flag, c.status, STATUS_TIMEOUT_STAGE_EMPTY);
         if (*abort_flag) break;
         uint8_t* dst = mc_smem + McOutSmem::RING + st * McOutSmem::TILE;
         const bool state = i < 2 * slices;
-        const int sl = state ? i / 2 : i - 2 * slices;
+        const int sl = state ? i / 2 : i % slices;              // 2 * slices and 3 * slices are multiples of slices
         const int cols = min(2, nv - 2 * sl);
         const int bytes = state ? nk * 8192 : MC_KCH;         // one 64-column chunk: nk * 64 state rows, or 128 tokens
         mbar_expect_tx(&full[st], cols * bytes);
@@ -527,7 +524,7 @@ mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
             for (int r = 0; r < nk; ++r)
               tma_load_3d(dst + k * bytes + r * 8192, &tm_s0, x, r * 64, (int)(chh * 2 + (i & 1)), &full[st]);
           } else {
-            tma_load_3d(dst + k * bytes, &tm_v, x, h, start, &full[st]);
+            tma_load_3d(dst + k * bytes, &tm_v, x, i < 3 * slices ? h : p.heads + h, start, &full[st]);
           }
         }
       }
@@ -583,7 +580,20 @@ mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     const int t = qd * 32 + lane;
     const bool ok = t < len;
     const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
-    const float At = s_A[t];
+    const float m0 = c.m0[chh];
+    {
+      const int ct = half * 128 + t;               // index among the 256 threads; tokens are the first 128
+      float F, B, Bmax;
+      chunk_gates(p.gates, p.heads, h, start, len, p.cap, s_g, ct, F, B, Bmax);
+      if (half == 0) {
+        s_B[t] = B * MC_LOG2E;
+        s_A[t] = -fmaxf(m0, Bmax);                 // F_t - m_t
+        s_n0[t] = t < p.dk ? c.n0[chh * p.dk + t] : 0.f;
+        s_x[t] = F;
+      }
+      named_bar_sync(1, 256);
+    }
+    const float At = s_A[t], At2 = At * MC_LOG2E;
     const float m_t = s_x[t] - At;
     const float a_t = ok ? expf(At + m0) * p.q_scale : 0.f;       // weight of the incoming state, q scaling included
     named_bar_sync(1, 256);                                       // s_x is read; it becomes the exchange buffer
@@ -612,13 +622,27 @@ mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     for (int c0 = 0; c0 < 64; c0 += 32) {
       const int s0 = half * 64 + c0;
       float sv[32];
+      if (s0 > qd * 32 + 31) {                     // right of the diagonal for every token of the warp
+        const uint4 z = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+        for (int v = 0; v < 4; ++v) {
+          const int off = half * MC_KCH + t * 128 + (((c0 / 8 + v) ^ (t & 7)) << 4);
+          *reinterpret_cast<uint4*>(mc_smem + McOutSmem::K + off) = z;
+          *reinterpret_cast<uint4*>(mc_smem + McOutSmem::PLO + off) = z;
+        }
+        continue;
+      }
       tmem_ld32(tmem_s + lane_off + s0, sv);
       tmem_ld_wait();
 #pragma unroll
-      for (int e = 0; e < 32; ++e) {
-        const int s = s0 + e;
-        sv[e] = ok && s <= t ? sv[e] * p.q_scale * expf(At + s_B[s]) : 0.f;
-        nq += sv[e];
+      for (int e = 0; e < 32; e += 4) {
+        const float4 b4 = *reinterpret_cast<const float4*>(s_B + s0 + e);
+        const float bb[4] = {b4.x, b4.y, b4.z, b4.w};
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          sv[e + u] = ok && s0 + e + u <= t ? sv[e + u] * p.q_scale * ex2_approx(At2 + bb[u]) : 0.f;
+          nq += sv[e + u];
+        }
       }
 #pragma unroll
       for (int v = 0; v < 4; ++v) {
@@ -671,35 +695,48 @@ mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     named_bar_sync(1, 256);
     ss = s_x[t] * inv * inv;
     const float r = inv / sqrtf(ss / (float)p.vdim + p.eps);
-    const __nv_bfloat16* g = reinterpret_cast<const __nv_bfloat16*>(p.qkvg) + (size_t)(start + (ok ? t : 0)) * p.ld +
-                             (size_t)2 * p.heads * p.dk + (size_t)(p.heads + h) * p.dv;
     __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(start + t) * p.ld_out + (size_t)h * p.dv;
     const float* nw = p.norm_w + (size_t)h * p.dv;
+    const bool whole = len == MC_TOK;
+    for (int sl = 0; sl < slices; ++sl) {
+      const int i = 3 * slices + sl, st = i % McOutSmem::NRING;
+      uint8_t* tile = mc_smem + McOutSmem::RING + st * McOutSmem::TILE;
+      mbar_wait(&full[st], (i / McOutSmem::NRING) & 1, abort_flag, c.status, STATUS_TIMEOUT_TMA_FULL);
 #pragma unroll 1
-    for (int col = half * 32; col < nv * 64; col += 64) {
-      float o[32];
-      tmem_ld32(tmem_o + lane_off + col, o);
-      tmem_ld_wait();
-      if (ok) {
+      for (int c0 = half * 32; c0 < min(2, nv - 2 * sl) * 64; c0 += 64) {
+        const int col = sl * 128 + c0;
+        float o[32];
+        tmem_ld32(tmem_o + lane_off + col, o);
+        tmem_ld_wait();
 #pragma unroll
         for (int v = 0; v < 32; v += 8) {
-          if (col + v < p.dv) {
-            const uint4 gu = *reinterpret_cast<const uint4*>(g + col + v);
-            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gu);
-            uint4 pk;
-            __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&pk);
+          uint4* slot = reinterpret_cast<uint4*>(tile + (c0 / 64) * MC_KCH + t * 128 + ((((c0 & 63) + v) / 8 ^ (t & 7)) << 4));
+          const uint4 gu = *slot;
+          const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gu);
+          uint4 pk;
+          __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&pk);
+          const bool in = col + v < p.dv;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              const float2 z = __bfloat1622float2(g2[e]);
-              const float2 w = *reinterpret_cast<const float2*>(nw + col + v + 2 * e);
-              p2[e] = __floats2bfloat162_rn(o[v + 2 * e] * r * w.x / (1.0f + __expf(-z.x)),
-                                            o[v + 2 * e + 1] * r * w.y / (1.0f + __expf(-z.y)));
-            }
-            *reinterpret_cast<uint4*>(out + col + v) = pk;
+          for (int e = 0; e < 4; ++e) {
+            const float2 z = __bfloat1622float2(g2[e]);
+            const float2 w = in ? __ldg(reinterpret_cast<const float2*>(nw + col + v + 2 * e)) : make_float2(0.f, 0.f);
+            p2[e] = __floats2bfloat162_rn(__fdividef(o[v + 2 * e] * r * w.x, 1.0f + __expf(-z.x)),
+                                          __fdividef(o[v + 2 * e + 1] * r * w.y, 1.0f + __expf(-z.y)));
           }
+          if (whole) *slot = pk;
+          else if (ok && in) *reinterpret_cast<uint4*>(out + col + v) = pk;
+        }
+      }
+      if (whole) {
+        fence_proxy_async_smem();
+        named_bar_sync(1, 256);
+        if (warp == 2 && lane == 0) {
+          for (int k = 0; k < min(2, nv - 2 * sl); ++k) tma_store_3d(&tm_out, tile + k * MC_KCH, (2 * sl + k) * 64, h, start);
+          tma_store_commit();
         }
       }
     }
+    if (warp == 2 && lane == 0) tma_store_wait_read();            // shared memory may go only when the stores have read it
     // the state's running maximum after the portion (the scan reads the old one): its last chunk writes it
     if (half == 0 && t == len - 1) {
       const bool last = ch + 1 == c.n_chunks || p.row[c.c_start[ch + 1]] != p.row[start];
@@ -761,22 +798,23 @@ extern "C" int tahb_mlstm_chunks(const MlstmParams* p, const MlstmChunkParams* c
   if (p->dk % 8 || p->dv % 8 || p->dk > 128 || p->dv > 256 || p->n_seq > 65535 || p->heads > 65535 || p->ld_out % 8) return -2;
   const int nk = (p->dk + 63) / 64, nv = (p->dv + 63) / 64;
   auto base = reinterpret_cast<const __nv_bfloat16*>(p->qkvg);
-  CUtensorMap mq, mv, ms;
+  CUtensorMap mq, mv, ms, mo;
   int rc;
   if ((rc = make_head_map(&mq, base, p->dk, 2 * p->heads, n_tokens, p->ld))) return rc;
   if ((rc = make_head_map(&mv, base + (size_t)2 * p->heads * p->dk, p->dv, 2 * p->heads, n_tokens, p->ld))) return rc;
   if ((rc = make_state_map(&ms, c->s0, p->dk, p->dv, (long long)c->n_chunks * p->heads * 2))) return rc;
+  if ((rc = make_head_map(&mo, reinterpret_cast<const __nv_bfloat16*>(p->out), p->dv, p->heads, n_tokens, p->ld_out))) return rc;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(mlstm_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, McStateSmem::bytes(4)) != cudaSuccess ||
+    if (cudaFuncSetAttribute(mlstm_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, McStateSmem::BYTES) != cudaSuccess ||
         cudaFuncSetAttribute(mlstm_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, McOutSmem::BYTES) != cudaSuccess)
       return -10;
     configured = true;
   }
   const dim3 grid(c->n_chunks, p->heads);
-  mlstm_chunk_state_kernel<<<grid, 256, McStateSmem::bytes(nv), stream>>>(mq, mv, *p, *c, nv);
+  mlstm_chunk_state_kernel<<<dim3(c->n_chunks, p->heads, (nv + 1) / 2), 256, McStateSmem::BYTES, stream>>>(mq, mv, *p, *c, nv);
   const int blocks = (int)(((long long)p->dk * p->dv / 4 + 255) / 256) + 1;
   mlstm_chunk_scan_kernel<<<dim3(blocks, p->heads, p->n_seq), 256, 0, stream>>>(*p, *c);
-  mlstm_chunk_out_kernel<<<grid, MC_OUT_THREADS, McOutSmem::BYTES, stream>>>(mq, mv, ms, *p, *c, nk, nv);
+  mlstm_chunk_out_kernel<<<grid, MC_OUT_THREADS, McOutSmem::BYTES, stream>>>(mq, mv, ms, mo, *p, *c, nk, nv);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

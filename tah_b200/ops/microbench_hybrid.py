@@ -1,0 +1,143 @@
+"""Micro-benchmark cases of the hybrid decoder's kernels (windowed attention, mLSTM, fp32-residual norms); run through
+:mod:`tah_b200.ops.microbench`, whose timing rules and flags apply.
+
+FLOPs and bytes are those of the algorithm: visible (query, key) pairs for attention, for the chunkwise mLSTM one
+128-token causal block plus the state read-out and update per chunk with every product counted once.
+"""
+from __future__ import annotations
+
+import torch
+
+from tah_b200.ops import cuda as K
+
+
+def _bf(*s):
+    return torch.randn(*s, device="cuda").to(torch.bfloat16)
+
+
+def _i32(x):
+    return torch.tensor(x, dtype=torch.int32, device="cuda")
+
+
+def _paged(rows, ctx, nkv, dk, dv):
+    per = (ctx + 15) // 16
+    pool = _bf(rows * per, nkv * 16 * (dk + dv))
+    pt = torch.randperm(rows * per, device="cuda").to(torch.int32).view(rows, per)
+    return pool, pt
+
+
+def _window_kw(a):
+    far = min(a.ctx, 512)
+    return dict(nq=a.nq, nkv=a.nkv, dk=a.hd, dv=a.hd, page_size=16, scale=a.hd ** -0.5, window=a.window or 2 ** 31 - 1,
+                keep_first=a.keep if a.window else 0, bias=torch.randn(a.nq, far + 1, device="cuda"),
+                sink=torch.randn(a.nq, device="cuda"))
+
+
+def _visible(i, a):
+    return min(i + 1, a.window + min(a.keep, max(0, i + 1 - a.window))) if a.window else i + 1
+
+
+def bench_window_prefill(a):
+    B, T = a.rows, a.ctx
+    n = B * T
+    pool, pt = _paged(B, T, a.nkv, a.hd, a.hd)
+    q, out, gate = _bf(n, a.nq * a.hd), torch.empty(n, a.nq * a.hd, dtype=torch.bfloat16, device="cuda"), _bf(n, a.nq)
+    pos = torch.arange(T, device="cuda", dtype=torch.int32).repeat(B)
+    row = torch.arange(B, device="cuda", dtype=torch.int32).repeat_interleave(T)
+    q0 = [b * T + t for b in range(B) for t in range(0, T, 128)]
+    qn = [min(128, T - t) for b in range(B) for t in range(0, T, 128)]
+    q0, qn, kw = _i32(q0), _i32(qn), _window_kw(a)
+    fn = lambda i: K.window_attn_tiles(q, out, pool, pt, pos, row, q0, qn, pool.shape[0], gate=gate, **kw)
+    pairs = B * sum(_visible(i, a) for i in range(T))
+    res = {"op": "window_prefill", "seqs": B, "T": T, "window": a.window, "keep": a.keep}
+    return res, fn, 4.0 * pairs * a.nq * a.hd, n * (2 * a.nq + 2 * a.nkv) * a.hd * 2
+
+
+def bench_window_decode(a):
+    from tah_b200.engine.hybrid import decode_splits
+    B, T = a.rows, a.ctx
+    pool, pt = _paged(B, T, a.nkv, a.hd, a.hd)
+    q, out, gate = _bf(B, a.nq * a.hd), torch.empty(B, a.nq * a.hd, dtype=torch.bfloat16, device="cuda"), _bf(B, a.nq)
+    pos, row, kw = _i32([T - 1] * B), _i32(list(range(B))), _window_kw(a)
+    ws = torch.empty(B * a.nq * a.nsplit * (a.hd + 2), device="cuda")
+    fn = lambda i: K.window_attn_decode(q, out, pool, pt, pos, row, gate=gate, n_split=a.nsplit, ws=ws, **kw)
+    keys = B * _visible(T - 1, a)
+    res = {"op": "window_decode", "rows": B, "ctx": T, "window": a.window, "n_split": a.nsplit}
+    return res, fn, 4.0 * keys * a.nq * a.hd, keys * a.nkv * 2 * a.hd * 2
+
+
+def _mlstm_case(a, n, rows):
+    H, dk, dv = a.nkv, a.hd, a.dv
+    F = H * (2 * dk + 2 * dv)
+    x, z, out = _bf(n, F), torch.randn(n, 2 * H, device="cuda"), torch.empty(n, H * dv, dtype=torch.bfloat16, device="cuda")
+    z[:, H:] += 4.0
+    state = tuple(torch.zeros(rows, *s, device="cuda") for s in ((H, dk, dv), (H, dk), (H,)))
+    return x, z, torch.ones(H * dv, device="cuda"), out, state, dict(heads=H, dk=dk, dv=dv, dim=dk, vdim=dv, cap=15.0, eps=1e-6)
+
+
+def bench_mlstm_chunks(a):
+    B, T = a.rows, a.ctx
+    n, H, dk, dv = B * T, a.nkv, a.hd, a.dv
+    x, z, nw, out, state, kw = _mlstm_case(a, n, B)
+    pos = torch.arange(T, device="cuda", dtype=torch.int32).repeat(B)
+    row = torch.arange(B, device="cuda", dtype=torch.int32).repeat_interleave(T)
+    starts = [b * T + t for b in range(B) for t in range(0, T, 128)]
+    lens = [min(128, T - t) for b in range(B) for t in range(0, T, 128)]
+    per = (T + 127) // 128
+    ws = torch.empty(K.mlstm_chunk_ws_floats(len(starts), H, dk, dv), device="cuda")
+    c = dict(chunk_start=_i32(starts), chunk_len=_i32(lens), seq_chunk0=_i32([b * per for b in range(B)]), seq_chunks=_i32([per] * B))
+    fn = lambda i: K.mlstm_chunks(x, z, nw, out, state, pos, row, ws=ws, **c, **kw)
+    flops = H * sum(l * (l + 1) * (dk + dv) + 4.0 * l * dk * dv for l in lens)
+    byts = n * H * ((2 * dk + 3 * dv) * 2 + 8) + B * H * dk * dv * 8
+    return {"op": "mlstm_chunks", "seqs": B, "T": T, "heads": H, "dk": dk, "dv": dv}, fn, flops, byts
+
+
+def bench_mlstm_step(a):
+    B, H, dk, dv = a.rows, a.nkv, a.hd, a.dv
+    x, z, nw, out, state, kw = _mlstm_case(a, B, B)
+    pos, row = _i32([5] * B), _i32(list(range(B)))
+    fn = lambda i: K.mlstm_recurrent(x, z, nw, out, state, pos, row, **kw)
+    return {"op": "mlstm_step", "rows": B, "heads": H, "dk": dk, "dv": dv}, fn, 6.0 * B * H * dk * dv, B * H * (dk * dv * 8 + (2 * dk + 3 * dv) * 2)
+
+
+def bench_residual_norm(a):
+    M, W = a.m, a.k
+    y, x, h = _bf(M, W), torch.randn(M, W, device="cuda"), torch.empty(M, W, dtype=torch.bfloat16, device="cuda")
+    w = torch.full((W,), 0.5, device="cuda")
+    fn = lambda i: K.residual_norm(y, x, w, w, W, 1e-6, h)
+    return {"op": "residual_norm", "M": M, "W": W}, fn, 0.0, M * W * (2 + 8 + 2)
+
+
+def bench_qkv_post(a):
+    M = a.m
+    F = (a.nq + 2 * a.nkv) * a.hd
+    qkv, q = _bf(M, F + 64), torch.empty(M, a.nq * a.hd, dtype=torch.bfloat16, device="cuda")
+    pool = _bf((M + 15) // 16, a.nkv * 16 * 2 * a.hd)
+    slot = torch.arange(M, device="cuda", dtype=torch.int32)
+    b, w = torch.randn(F + 64, device="cuda"), torch.ones(a.hd, device="cuda")
+    fn = lambda i: K.qkv_post(qkv, b, w, w, q, pool, slot, a.nq, a.nkv, a.hd, a.hd, a.hd, 16, 1e-6)
+    return {"op": "qkv_post", "M": M}, fn, 0.0, 2 * M * F * 2
+
+
+def bench_qk_norm_rope(a):
+    """The like kernel of the Qwen3 engine."""
+    M = a.m
+    F = (a.nq + 2 * a.nkv) * a.hd
+    qkv, q = _bf(M, F), torch.empty(M, a.nq * a.hd, dtype=torch.bfloat16, device="cuda")
+    pool = torch.zeros((M + 15) // 16, 2, a.nkv, 16, a.hd, dtype=torch.bfloat16, device="cuda")
+    slot = torch.arange(M, device="cuda", dtype=torch.int32)
+    w = torch.ones(a.hd, device="cuda", dtype=torch.bfloat16)
+    fn = lambda i: K.qk_norm_rope_kv(qkv, w, w, slot, a.nq, a.nkv, a.hd, 1e-6, 1e6, q_out=q, caches=[pool], slot=slot)
+    return {"op": "qk_norm_rope", "M": M}, fn, 0.0, 2 * M * F * 2
+
+
+def bench_few_linear(a):
+    M, W, F = a.m, a.k, a.f
+    x, w, b, out = _bf(M, W), _bf(F, W), torch.randn(F, device="cuda"), torch.empty(M, F, device="cuda")
+    fn = lambda i: K.few_linear(x, w, b, out=out)
+    return {"op": "few_linear", "M": M, "K": W, "F": F}, fn, 2.0 * M * W * F, (M * W + F * W) * 2 + M * F * 4
+
+
+CASES = {"window_prefill": bench_window_prefill, "window_decode": bench_window_decode, "mlstm_chunks": bench_mlstm_chunks,
+         "mlstm_step": bench_mlstm_step, "residual_norm": bench_residual_norm, "qkv_post": bench_qkv_post,
+         "qk_norm_rope": bench_qk_norm_rope, "few_linear": bench_few_linear}

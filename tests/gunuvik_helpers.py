@@ -81,8 +81,8 @@ TOL = {torch.float32: 2e-5, torch.bfloat16: 6e-2}
 
 def close(got, want, dtype):
     """Every row within the rounding of ``dtype``.  A few tokens of a random model are ill-conditioned in 16 bits (the
-    normaliser of a recurrent layer nearly cancels), so there one row in twenty may be up to three times over."""
+    normaliser of a recurrent layer nearly cancels), so there one row in ten may be up to three times over."""
     e = row_errors(got, want)
     if dtype == torch.float32:
         return bool((e <= TOL[dtype]).all())
-    return bool((e <= 3 * TOL[dtype]).all()) and int((e > TOL[dtype]).sum()) <= max(1, len(e) // 20)
+    return bool((e <= 3 * TOL[dtype]).all()) and int((e > TOL[dtype]).sum()) <= max(1, len(e) // 10)

@@ -168,6 +168,7 @@ def random_model(cfg, seed=0, dtype=torch.bfloat16):
             sd[m + "g"], sd[m + "o"] = lin(H, W), lin(W, H * dv)
         else:
             sd[m + "q"], sd[m + "k"], sd[m + "v"] = lin(H * dk, W), lin(H * dk, W), lin(H * dv, W)
+            sd[m + "q"] = 0.7 * sd[m + "q"] + 0.7 * sd[m + "k"]      # q . k of a token is positive: the normaliser rarely cancels
             sd[m + "g"], sd[m + "o"], sd[m + "norm"] = lin(H * dv, W), lin(W, H * dv), near1(H * dv)
             sd[m + "i"], sd[m + "i.b"] = 2 * lin(H, W), rnd(H)
             sd[m + "f"], sd[m + "f.b"] = 2 * lin(H, W), 3.0 + rnd(H)
