@@ -113,15 +113,26 @@ __global__ void __launch_bounds__(MR_THREADS, 3) mlstm_recurrent_kernel(const Ml
     if (rg < nrg) {
       const float4 vv = ldf4(v + c * 4);
       float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-      for (int r = rg; r < dk; r += nrg) {
-        float4* sp = reinterpret_cast<float4*>(S + (size_t)r * dv) + c;
-        float4 a = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *sp;
-        const float kr = s_k[r], qr = s_q[r];
-        a.x = fmaf(keep, a.x, kr * vv.x); a.y = fmaf(keep, a.y, kr * vv.y);
-        a.z = fmaf(keep, a.z, kr * vv.z); a.w = fmaf(keep, a.w, kr * vv.w);
-        o.x = fmaf(a.x, qr, o.x); o.y = fmaf(a.y, qr, o.y); o.z = fmaf(a.z, qr, o.z); o.w = fmaf(a.w, qr, o.w);
-        *sp = a;
+      constexpr int U = 8;               // rows in flight: all their loads are issued before the first store
+      for (int r0 = rg; r0 < dk; r0 += U * nrg) {
+        float4 a[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int r = r0 + u * nrg;
+          a[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (!fresh && r < dk) a[u] = *(reinterpret_cast<const float4*>(S + (size_t)r * dv) + c);
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int r = r0 + u * nrg;
+          if (r < dk) {
+            const float kr = s_k[r], qr = s_q[r];
+            a[u].x = fmaf(keep, a[u].x, kr * vv.x); a[u].y = fmaf(keep, a[u].y, kr * vv.y);
+            a[u].z = fmaf(keep, a[u].z, kr * vv.z); a[u].w = fmaf(keep, a[u].w, kr * vv.w);
+            o.x = fmaf(a[u].x, qr, o.x); o.y = fmaf(a[u].y, qr, o.y); o.z = fmaf(a[u].z, qr, o.z); o.w = fmaf(a[u].w, qr, o.w);
+            *(reinterpret_cast<float4*>(S + (size_t)r * dv) + c) = a[u];
+          }
+        }
       }
       *reinterpret_cast<float4*>(s_red + (size_t)rg * dv + c * 4) = o;
     }
@@ -256,7 +267,7 @@ struct McStateSmem {
 
 __global__ void __launch_bounds__(256, 2)
 mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
-                         const MlstmParams p, const MlstmChunkParams c, const int nv_all) {
+                         const __grid_constant__ CUtensorMap tm_dS, const MlstmParams p, const MlstmChunkParams c, const int nv_all) {
   extern __shared__ __align__(1024) uint8_t mc_smem[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int ch = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * 2, nv = min(2, nv_all - v0);
@@ -354,19 +365,27 @@ mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   __syncwarp();
   tc_fence_after();
   {
+    // [128 key dims][32 columns] fp32 tiles (128-byte swizzled rows) over the operands, then one TMA store per tile
     const int d = (warp & 3) * 32 + lane;                      // row of S (key dim)
     const uint32_t trow = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
-    float* dst = c.dS + (chh * p.dk + d) * p.dv + v0 * 64;
+    __syncthreads();                                           // every thread has read the weighted keys
 #pragma unroll 1
     for (int col = (warp >> 2) * 32; col < nv * 64; col += 64) {
       float o[32];
       tmem_ld32(trow + col, o);
       tmem_ld_wait();
-      if (d < p.dk) {
+      uint8_t* tile = mc_smem + (col / 32) * MC_KCH;
 #pragma unroll
-        for (int e = 0; e < 32; e += 4)
-          if (v0 * 64 + col + e < p.dv) *reinterpret_cast<float4*>(dst + col + e) = make_float4(o[e], o[e + 1], o[e + 2], o[e + 3]);
-      }
+      for (int e = 0; e < 8; ++e)
+        *reinterpret_cast<float4*>(tile + d * 128 + ((e ^ (d & 7)) << 4)) = make_float4(o[4 * e], o[4 * e + 1], o[4 * e + 2], o[4 * e + 3]);
+    }
+    fence_proxy_async_smem();
+    __syncthreads();
+    if (tid == 0) {
+      for (int k = 0; k < nv * 2; ++k)
+        if (v0 * 64 + k * 32 < p.dv) tma_store_3d(&tm_dS, mc_smem + k * MC_KCH, v0 * 64 + k * 32, 0, (int)chh);
+      tma_store_commit();
+      tma_store_wait_read();
     }
   }
   tc_fence_before();
@@ -777,6 +796,19 @@ static int make_state_map(CUtensorMap* m, const __nv_bfloat16* base, int dk, int
   return r == CUDA_SUCCESS ? 0 : -3;
 }
 
+// [n][dk][dv] fp32, boxes of 128 rows x 32 columns (rows past dk are not written)
+static int make_dS_map(CUtensorMap* m, float* base, int dk, int dv, long long n) {
+  PfEncodeFn fn = pf_encode_fn();
+  if (fn == nullptr) return -1;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || dv % 4) return -2;
+  cuuint64_t dims[3] = {(cuuint64_t)dv, (cuuint64_t)dk, (cuuint64_t)n};
+  cuuint64_t strides[2] = {(cuuint64_t)dv * 4, (cuuint64_t)dk * dv * 4};
+  cuuint32_t box[3] = {32u, 128u, 1u}, estr[3] = {1u, 1u, 1u};
+  CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_FLOAT32, 3, base, dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                  CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -3;
+}
+
 }  // namespace tahb
 
 using namespace tahb;
@@ -798,12 +830,13 @@ extern "C" int tahb_mlstm_chunks(const MlstmParams* p, const MlstmChunkParams* c
   if (p->dk % 8 || p->dv % 8 || p->dk > 128 || p->dv > 256 || p->n_seq > 65535 || p->heads > 65535 || p->ld_out % 8) return -2;
   const int nk = (p->dk + 63) / 64, nv = (p->dv + 63) / 64;
   auto base = reinterpret_cast<const __nv_bfloat16*>(p->qkvg);
-  CUtensorMap mq, mv, ms, mo;
+  CUtensorMap mq, mv, ms, mo, md;
   int rc;
   if ((rc = make_head_map(&mq, base, p->dk, 2 * p->heads, n_tokens, p->ld))) return rc;
   if ((rc = make_head_map(&mv, base + (size_t)2 * p->heads * p->dk, p->dv, 2 * p->heads, n_tokens, p->ld))) return rc;
   if ((rc = make_state_map(&ms, c->s0, p->dk, p->dv, (long long)c->n_chunks * p->heads * 2))) return rc;
   if ((rc = make_head_map(&mo, reinterpret_cast<const __nv_bfloat16*>(p->out), p->dv, p->heads, n_tokens, p->ld_out))) return rc;
+  if ((rc = make_dS_map(&md, c->dS, p->dk, p->dv, (long long)c->n_chunks * p->heads))) return rc;
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(mlstm_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, McStateSmem::BYTES) != cudaSuccess ||
@@ -812,7 +845,7 @@ extern "C" int tahb_mlstm_chunks(const MlstmParams* p, const MlstmChunkParams* c
     configured = true;
   }
   const dim3 grid(c->n_chunks, p->heads);
-  mlstm_chunk_state_kernel<<<dim3(c->n_chunks, p->heads, (nv + 1) / 2), 256, McStateSmem::BYTES, stream>>>(mq, mv, *p, *c, nv);
+  mlstm_chunk_state_kernel<<<dim3(c->n_chunks, p->heads, (nv + 1) / 2), 256, McStateSmem::BYTES, stream>>>(mq, mv, md, *p, *c, nv);
   const int blocks = (int)(((long long)p->dk * p->dv / 4 + 255) / 256) + 1;
   mlstm_chunk_scan_kernel<<<dim3(blocks, p->heads, p->n_seq), 256, 0, stream>>>(*p, *c);
   mlstm_chunk_out_kernel<<<grid, MC_OUT_THREADS, McOutSmem::BYTES, stream>>>(mq, mv, ms, mo, *p, *c, nk, nv);
