@@ -18,7 +18,7 @@ def parse_args(argv=None):
     ap = argparse.ArgumentParser(description="TaH evaluation")
     ap.add_argument("--eval_config", required=True)
     ap.add_argument("--model_path", required=True)
-    ap.add_argument("--backend", default="tah", choices=["sglang", "hf", "tah"])
+    ap.add_argument("--backend", default="tah", choices=["sglang", "hf", "tah", "engine"])
     ap.add_argument("--dataset_name", required=True, help="registered benchmark name(s), comma separated")
     ap.add_argument("--job_nums", type=int, default=8)
     ap.add_argument("--tp_size_per_job", type=int, default=1)

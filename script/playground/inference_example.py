@@ -5,6 +5,11 @@
 
 With ``--random_init`` a tiny random model is used (no download), which is enough to see the
 engine and the colouring at work.
+
+A checkpoint directory of another registered family (``config.json`` decides, e.g. Gunuvik) is served by that family's
+engine; without a tokenizer in the directory the prompts are token ids, one ``--prompt_ids`` per request:
+
+    python script/playground/inference_example.py --model path/to/gunuvik --prompt_ids 5,17,3 --prompt_ids 8,2 --temperature 0
 """
 import argparse
 import os
@@ -20,6 +25,23 @@ from tah_b200 import TaHForCausalLM  # noqa: E402
 from tah_b200.model.utils import IterCountColors, TaHForCasualLM_generate  # noqa: E402
 
 
+def run_family_engine(a):
+    """Serve the requests with the engine of the checkpoint's family and print the generated tokens."""
+    from tah_b200.models import load_model, make_engine
+    tok = None
+    if not a.prompt_ids:
+        from transformers import AutoTokenizer
+        tok = AutoTokenizer.from_pretrained(a.model)
+    prompts = [[int(t) for t in p.split(",")] for p in a.prompt_ids] if tok is None else [tok.encode(a.prompt)]
+    eng = make_engine(load_model(a.model, getattr(torch, a.dtype), "cuda"), max_rows=max(1, min(64, len(prompts))))
+    out, stats = eng.serve([torch.tensor(p) for p in prompts], max_new_tokens=a.max_new_tokens, do_sample=a.temperature > 0,
+                           temperature=a.temperature if a.temperature > 0 else 1.0, top_p=a.top_p, top_k=a.top_k, seed=a.seed,
+                           eos_token_id=getattr(tok, "eos_token_id", None))
+    for row in out:
+        print(tok.decode(row) if tok is not None else ",".join(map(str, row)))
+    print(f"# {stats}", file=sys.stderr)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--model", default="nics-efc/TaH-plus-1.7B")
@@ -29,7 +51,14 @@ def main():
     ap.add_argument("--top_p", type=float, default=0.95)
     ap.add_argument("--top_k", type=int, default=20)
     ap.add_argument("--random_init", action="store_true")
+    ap.add_argument("--prompt_ids", action="append", default=[], help="comma-separated token ids of a request (repeatable)")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
+    ap.add_argument("--seed", type=int, default=None)
     a = ap.parse_args()
+    if not a.random_init and os.path.isfile(os.path.join(a.model, "config.json")):
+        from tah_b200.models.registry import family_of_config, read_config
+        if family_of_config(read_config(a.model)).name != "qwen3-tah":
+            return run_family_engine(a)
     dev = "cuda" if torch.cuda.is_available() else "cpu"
     if a.random_init:
         from tests.helpers import tiny_tah

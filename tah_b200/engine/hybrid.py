@@ -415,6 +415,9 @@ class HybridEngine(DecodeEngine):
         """Run the entries as one batch, from the cache and state that earlier steps left; returns the logits
         ``[wanted, vocab]`` in the order of the entries and of their ``want``."""
         toks, want, at = [], [], 0
+        entries = [e for e in entries if len(e.tokens)]
+        if not entries:
+            return torch.empty(0, self.w.vocab, dtype=self.dtype, device=self.device)
         for e in entries:
             if any(not 0 <= w < len(e.tokens) for w in e.want):
                 raise ValueError("a wanted place lies outside the entry's tokens")

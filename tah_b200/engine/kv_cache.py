@@ -116,9 +116,11 @@ class PagedKVCache:
             self.free_stack[d].copy_(torch.arange(self.n_pages[d], dtype=torch.int32, device=self.free_stack[d].device))
             self.free_count[d].fill_(self.n_pages[d])
 
-    def layer_pool(self, depth: int, layer: int) -> torch.Tensor:
-        if self.geo.layers is not None and self.geo.layers[layer].shared_with is not None:
-            layer = self.geo.layers[layer].shared_with
+    def layer_pool(self, depth: int, layer: int) -> Optional[torch.Tensor]:
+        """The pool a layer reads (its own or the one it shares); None for a layer without keys."""
+        l = self.geo.layers[layer] if self.geo.layers is not None else None
+        if l is not None and l.shared_with is not None:
+            layer = l.shared_with
         return self.pool[depth][layer]
 
     def assign_prefill(self, depth: int, counts: torch.Tensor) -> torch.Tensor:

@@ -7,6 +7,8 @@ per-sample time is the batch time divided by the batch size.
 * ``tah`` - this framework's paged-KV engine (left-padded prompts, ``do_sample = temperature > 0``).
   Unlike the reference, ``tp_size > 1`` is honoured: one tensor-parallel engine over ``tp_size`` GPUs, either the
   ranks of a ``torchrun`` job or follower processes spawned by the job (:mod:`tah_b200.evaluate.tp_group`).
+* ``engine`` - the engine of whatever registered model family the checkpoint's ``config.json`` names
+  (:mod:`tah_b200.models.registry`), with continuous batching.
 * ``hf`` - a plain HuggingFace ``generate`` on the base model (needs the checkpoint's HF weights).
 * ``sglang`` - only if the optional package is importable.
 """
@@ -121,6 +123,28 @@ def setup_tah(config: Dict, model_path: str, tokenizer, tp_size: int = 1):
     return model, infer
 
 
+def setup_engine(config: Dict, model_path: str, tokenizer, tp_size: int = 1):
+    if tp_size and tp_size > 1:
+        raise ValueError("the 'engine' backend runs on one GPU per job")
+    from tah_b200.models.registry import load_model, make_engine
+    model = load_model(model_path, _dtype(config), "cuda")
+    eng = make_engine(model, max_rows=int(config.get("batch_size", 64)))
+    temperature = float(config.get("temperature", 0.0))
+    kw = dict(max_new_tokens=int(config.get("max_new_tokens", 1024)), do_sample=temperature > 0,
+              temperature=temperature if temperature > 0 else 1.0, top_p=float(config.get("top_p", 1.0)),
+              top_k=int(config.get("top_k", 0)), min_p=float(config.get("min_p", 0.0)),
+              eos_token_id=getattr(tokenizer, "eos_token_id", None))
+
+    def serve_all(prompts: List[str], rows: int) -> List[Tuple[str, float]]:
+        ids = [torch.tensor(tokenizer.encode(p), dtype=torch.long) for p in prompts]
+        (tokens, _), secs = time_inference(eng.serve, ids, rows=int(rows), **kw)
+        return [(tokenizer.decode(t) if t else "", secs / max(1, len(prompts))) for t in tokens]
+
+    infer: InferFn = lambda prompts: serve_all(prompts, len(prompts))
+    infer.serve_all = serve_all
+    return model, infer
+
+
 def setup_hf(config: Dict, model_path: str, tokenizer, tp_size: int = 1):
     from transformers import AutoModelForCausalLM
     model = AutoModelForCausalLM.from_pretrained(model_path, torch_dtype=_dtype(config), device_map="auto")
@@ -158,7 +182,7 @@ def setup_sglang(config: Dict, model_path: str, tokenizer, tp_size: int = 1):
     return engine, infer
 
 
-_SETUP_BY_NAME = {"tah": setup_tah, "hf": setup_hf, "sglang": setup_sglang}
+_SETUP_BY_NAME = {"tah": setup_tah, "engine": setup_engine, "hf": setup_hf, "sglang": setup_sglang}
 
 
 def setup_backend(backend: str, config: Dict, model_path: str, tokenizer, tp_size: int = 1):

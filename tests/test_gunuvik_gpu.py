@@ -528,3 +528,27 @@ def test_trace_replay_program(tmp_path):
             raw = torch.frombuffer(bytearray(open(os.path.join(out, f"{step}.f32"), "rb").read()), dtype=torch.float32)
             assert H.close(raw.view(-1, cfg["vocab"]), want, getattr(torch, dtype))
             os.unlink(os.path.join(out, f"{step}.f32"))
+
+
+def test_playground_command_line_and_evaluation_backend(tmp_path):
+    from tah_b200.evaluate.backends import setup_backend
+    cfg, sd, d = H.make(tmp_path, "mixed", seed=8)
+    prompts = [H.tokens(cfg, 9, 1), H.tokens(cfg, 4, 2)]
+    cmd = [sys.executable, os.path.join(ROOT, "script", "playground", "inference_example.py"), "--model", d, "--dtype", "float32",
+           "--temperature", "0", "--max_new_tokens", "8"]
+    for p in prompts:
+        cmd += ["--prompt_ids", ",".join(map(str, p))]
+    r = subprocess.run(cmd, capture_output=True, text=True, timeout=240)
+    assert r.returncode == 0, r.stderr[-2000:]
+    rows = [[int(t) for t in l.split(",")] for l in r.stdout.split()]
+    assert len(rows) == 2 and all(_tokens_follow(cfg, sd, p, o, 1e-4) for p, o in zip(prompts, rows))
+
+    class Ids:                                             # a tokenizer whose texts are token ids
+        eos_token_id = None
+        encode = staticmethod(lambda s: [int(t) for t in s.split()])
+        decode = staticmethod(lambda ids: " ".join(map(str, ids)))
+
+    model, infer = setup_backend("engine", dict(dtype="float32", max_new_tokens=8, batch_size=4), d, Ids())
+    for rows_n in (1, 2):
+        got = infer.serve_all([Ids.decode(p) for p in prompts], rows_n)
+        assert [Ids.encode(t) for t, _ in got] == rows
