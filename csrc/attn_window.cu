@@ -336,13 +336,14 @@ __device__ __forceinline__ float finish_scale(const WindowAttnParams& p, int t, 
   return f;
 }
 
-template <int VEC, int GB>
-__global__ void __launch_bounds__(160, (VEC * GB <= 4) ? 4 : 2) window_decode_kernel(const WindowAttnParams p) {
+template <int VEC, int GB, bool EXACT>   // EXACT: dk = dv = VEC * 64, known to the compiler
+__global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) window_decode_kernel(const WindowAttnParams p) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int DPL = VEC * 8;
+  const int dk = EXACT ? VEC * 64 : p.dk, dv = EXACT ? VEC * 64 : p.dv;
   extern __shared__ __align__(128) uint8_t wd_smem[];
-  const int kblk = WD_PAGE * p.dk, vblk = WD_PAGE * p.dv;              // elements of one K / V block of a page
+  const int kblk = WD_PAGE * dk, vblk = WD_PAGE * dv;              // elements of one K / V block of a page
   const int stage_elems = WD_STAGE_PAGES * (kblk + vblk);
   __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(wd_smem);
   uint64_t* full_bar = reinterpret_cast<uint64_t*>(wd_smem + (size_t)WD_NSTAGE * stage_elems * 2);
@@ -410,37 +411,41 @@ __global__ void __launch_bounds__(160, (VEC * GB <= 4) ? 4 : 2) window_decode_ke
     for (int g = 0; g < GB; ++g) {
       const bool live = grp0 + g < G;
       const int h = kvh * G + (live ? grp0 + g : 0);
-      const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(p.q) + ((size_t)t * p.nq + h) * p.dk;
+      const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(p.q) + ((size_t)t * p.nq + h) * dk;
       bias[g] = p.bias == nullptr ? nullptr : p.bias + (size_t)h * (p.far + 1);
 #pragma unroll
       for (int v = 0; v < VEC; ++v) {
         const int c = (v * 8 + gl) * 8;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) qv[g][v * 8 + e] = live && c < p.dk ? __bfloat162float(qp[c + e]) * (p.scale * LOG2E) : 0.f;
+        for (int e = 0; e < 8; ++e) qv[g][v * 8 + e] = live && c < dk ? __bfloat162float(qp[c + e]) * (p.scale * LOG2E) : 0.f;
       }
     }
     for (int it = 0; it < n_iter; ++it) {
       const int s = it % WD_NSTAGE;
-      mbar_wait(&full_bar[s], (it / WD_NSTAGE) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
-      const __nv_bfloat16* st = stages + (size_t)s * stage_elems;
-      float sc[WD_STAGE_PAGES][GB];
+      float b[WD_STAGE_PAGES][GB];
       bool ok[WD_STAGE_PAGES];
 #pragma unroll
-      for (int u = 0; u < WD_STAGE_PAGES; ++u) {
+      for (int u = 0; u < WD_STAGE_PAGES; ++u) {          // the biases are fetched while the keys are still on their way
         const int idx = pb + it * WD_STAGE_PAGES + u;
         const int j = (idx < kp ? idx : w0 + idx - kp) * WD_PAGE + grp;
         ok[u] = idx < pe && j <= i && (j >= lo || j < p.keep_first);
-        float b[GB];
+        const int dist = min(max(i - j, 0), p.far);
 #pragma unroll
-        for (int g = 0; g < GB; ++g) b[g] = ok[u] && bias[g] != nullptr ? bias[g][min(i - j, p.far)] : 0.f;
-        const __nv_bfloat16* kq = st + (size_t)u * (kblk + vblk) + grp * p.dk;
+        for (int g = 0; g < GB; ++g) b[u][g] = bias[g] != nullptr ? __ldg(bias[g] + dist) : 0.f;
+      }
+      mbar_wait(&full_bar[s], (it / WD_NSTAGE) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
+      const __nv_bfloat16* st = stages + (size_t)s * stage_elems;
+      float sc[WD_STAGE_PAGES][GB];
+#pragma unroll
+      for (int u = 0; u < WD_STAGE_PAGES; ++u) {
+        const __nv_bfloat16* kq = st + (size_t)u * (kblk + vblk) + grp * dk;
         float se[GB], so[GB];
 #pragma unroll
         for (int g = 0; g < GB; ++g) { se[g] = 0.f; so[g] = 0.f; }
 #pragma unroll
         for (int v = 0; v < VEC; ++v) {
           const int c = (v * 8 + gl) * 8;
-          if (c < p.dk) {
+          if (c < dk) {
             const uint4 kr = *reinterpret_cast<const uint4*>(kq + c);
             const __nv_bfloat162* kh = reinterpret_cast<const __nv_bfloat162*>(&kr);
 #pragma unroll
@@ -460,7 +465,7 @@ __global__ void __launch_bounds__(160, (VEC * GB <= 4) ? 4 : 2) window_decode_ke
           d += __shfl_xor_sync(0xffffffffu, d, 1);
           d += __shfl_xor_sync(0xffffffffu, d, 2);
           d += __shfl_xor_sync(0xffffffffu, d, 4);
-          sc[u][g] = ok[u] ? d + b[g] : -INFINITY;
+          sc[u][g] = ok[u] ? d + b[u][g] : -INFINITY;
         }
       }
 #pragma unroll
@@ -477,7 +482,7 @@ __global__ void __launch_bounds__(160, (VEC * GB <= 4) ? 4 : 2) window_decode_ke
 #pragma unroll
       for (int u = 0; u < WD_STAGE_PAGES; ++u) {
         if (!ok[u]) continue;            // never touch stage memory that holds no visible key
-        const __nv_bfloat16* vq = st + (size_t)u * (kblk + vblk) + kblk + grp * p.dv;
+        const __nv_bfloat16* vq = st + (size_t)u * (kblk + vblk) + kblk + grp * dv;
         float pw[GB];
 #pragma unroll
         for (int g = 0; g < GB; ++g) {
@@ -487,7 +492,7 @@ __global__ void __launch_bounds__(160, (VEC * GB <= 4) ? 4 : 2) window_decode_ke
 #pragma unroll
         for (int v = 0; v < VEC; ++v) {
           const int c = (v * 8 + gl) * 8;
-          if (c < p.dv) {
+          if (c < dv) {
             const uint4 vr = *reinterpret_cast<const uint4*>(vq + c);
             const __nv_bfloat162* vh = reinterpret_cast<const __nv_bfloat162*>(&vr);
 #pragma unroll
@@ -522,15 +527,15 @@ __global__ void __launch_bounds__(160, (VEC * GB <= 4) ? 4 : 2) window_decode_ke
 #pragma unroll
       for (int v = 0; v < VEC; ++v) {
         const int c = (v * 8 + gl) * 8;
-        if (c < p.dv) {
+        if (c < dv) {
 #pragma unroll
-          for (int e = 0; e < 8; ++e) sm_acc[(grp * GB + g) * p.dv + c + e] = acc[g][v * 8 + e];
+          for (int e = 0; e < 8; ++e) sm_acc[(grp * GB + g) * dv + c + e] = acc[g][v * 8 + e];
         }
       }
   }
   __syncthreads();
-  for (int idx = tid; idx < GB * p.dv; idx += 160) {
-    const int g = idx / p.dv, d = idx % p.dv;
+  for (int idx = tid; idx < GB * dv; idx += 160) {
+    const int g = idx / dv, d = idx % dv;
     if (grp0 + g >= G) continue;
     float mx = -INFINITY;
 #pragma unroll
@@ -540,17 +545,17 @@ __global__ void __launch_bounds__(160, (VEC * GB <= 4) ? 4 : 2) window_decode_ke
     for (int k = 0; k < 16; ++k) {
       const float mk = sm_m[k * GB + g];
       const float w = (mk == -INFINITY) ? 0.f : exp2f(mk - mx);
-      num += w * sm_acc[(k * GB + g) * p.dv + d];
+      num += w * sm_acc[(k * GB + g) * dv + d];
       den += w * sm_l[k * GB + g];
     }
     const int h = kvh * G + grp0 + g;
     if (p.n_split == 1) {
-      reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ld_out + (size_t)h * p.dv + d] =
+      reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ld_out + (size_t)h * dv + d] =
           __float2bfloat16_rn(num * finish_scale(p, t, h, mx, den));
     } else {
-      float* w = p.ws + (((size_t)t * p.nq + h) * p.n_split + split) * (p.dv + 2);
+      float* w = p.ws + (((size_t)t * p.nq + h) * p.n_split + split) * (dv + 2);
       w[d] = num;
-      if (d == 0) { w[p.dv] = mx; w[p.dv + 1] = den; }
+      if (d == 0) { w[dv] = mx; w[dv + 1] = den; }
     }
   }
 }
@@ -859,23 +864,29 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   }
 }
 
-template <int VEC, int GB>
-static int launch_window_decode(const WindowAttnParams& p, cudaStream_t stream) {
+template <int VEC, int GB, bool EXACT>
+static int launch_window_decode_as(const WindowAttnParams& p, cudaStream_t stream) {
   const int groups = (p.nq / p.nkv + GB - 1) / GB;
   const size_t ring = (size_t)WD_NSTAGE * WD_STAGE_PAGES * WD_PAGE * (p.dk + p.dv) * 2 + 128;
   const size_t merge = (size_t)16 * GB * (p.dv + 2) * 4;
   const size_t smem = ring > merge ? ring : merge;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(window_decode_kernel<VEC, GB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
+    if (cudaFuncSetAttribute(window_decode_kernel<VEC, GB, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
       return -10;
     configured = true;
   }
   if (smem > 160 * 1024) return -11;
-  cudaError_t e = launch_chain(window_decode_kernel<VEC, GB>, dim3(p.nkv * groups, p.n, p.n_split), dim3(160), smem, stream, p);
+  cudaError_t e = launch_chain(window_decode_kernel<VEC, GB, EXACT>, dim3(p.nkv * groups, p.n, p.n_split), dim3(160), smem, stream, p);
   if (e == cudaSuccess && p.n_split > 1)
     e = launch_chain(window_decode_merge_kernel, dim3(p.n * p.nq), dim3(128), 0, stream, p);
   return e == cudaSuccess ? 0 : -3;
+}
+
+template <int VEC, int GB>
+static int launch_window_decode(const WindowAttnParams& p, cudaStream_t stream) {
+  return p.dk == VEC * 64 && p.dv == VEC * 64 ? launch_window_decode_as<VEC, GB, true>(p, stream)
+                                              : launch_window_decode_as<VEC, GB, false>(p, stream);
 }
 
 // K (or V) of a paged cache as a 4-D tensor [pages][kv heads][16 tokens][dims], read in boxes of one page's 16 tokens x 64 dims

@@ -49,7 +49,7 @@ def test_no_cluster_multicast_no_triton_no_disassembly():
 
 def test_every_device_wait_is_bounded():
     """Every spin in the kernels goes through a helper with a time limit."""
-    for name in ("gemm_tcgen05.cu", "attn_decode.cu"):
+    for name in ("gemm_tcgen05.cu", "attn_decode.cu", "attn_prefill.cu", "attn_window.cu", "mlstm.cu"):
         text = open(os.path.join(ROOT, "csrc", name)).read()
         assert "mbar_try_wait(" not in text            # only the bounded mbar_wait() may be called from kernels
         assert "while (true)" not in text and "while(1)" not in text
