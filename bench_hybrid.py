@@ -23,7 +23,7 @@ def _qwen3(gcfg, dev):
     from tah_b200.engine import TaHEngine
     from tah_b200.models import Qwen3Config, Qwen3ForCausalLM
     a = next(l.mixer for l in gcfg.layers if l.mixer.kind == "attention")
-    ff = next(l.ff for l in gcfg.layers if l.ff)
+    ff = next(l.ff for l in gcfg.layers if l.ff).ff
     cfg = Qwen3Config(vocab_size=gcfg.vocab_size, hidden_size=gcfg.hidden_size, intermediate_size=ff,
                       num_hidden_layers=len(gcfg.layers), num_attention_heads=a.heads, num_key_value_heads=a.kv_heads,
                       head_dim=a.dim, tie_word_embeddings=False)

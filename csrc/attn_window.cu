@@ -1,9 +1,12 @@
-// Paged attention with a sliding window, kept first tokens, a per-distance bias, a softmax sink and a per-head output gate.
+// Paged attention with a sliding window, kept first tokens, a query temperature, a score cap, a per-distance bias, a
+// softmax sink and a per-head output gate.
 //
 // Query at position i of a sequence sees key j when  j <= i  and  (i - j < window  or  j < keep_first).
-// score = (q . k) * scale + bias[h][min(i - j, D)]; softmax over the visible keys with exp(sink_h) added to the
-// denominator; out_h *= sigmoid(gate_h).  Every constant is a launch parameter: window = INT_MAX is plain causal
-// attention, keep_first = 0 a plain window, and the bias table, the sink and the gate may each be absent.
+// score = cap(temp(i) * (q . k) * scale) + bias[h][min(i - j, D)] with cap(s) = softcap * tanh(s / softcap) and
+// temp(i) = 1 + temp_coef * ln(floor((i + 1) / temp_every) + 1); softmax over the visible keys with exp(sink_h) added to
+// the denominator; out_h *= sigmoid(gate_h).  Every constant is a launch parameter: window = INT_MAX is plain causal
+// attention, keep_first = 0 a plain window, softcap = 0 no cap, temp_coef = 0 no temperature, and the bias table, the
+// sink and the gate may each be absent.
 //
 // Keys and values are read from the paged cache only (the tokens of the running step are written there first), so
 // portions of a prompt, single decoded tokens and layers that read another layer's cache are the same case:
@@ -182,7 +185,7 @@ __global__ void __launch_bounds__(128) qkv_post_kernel(const QkvPostParams p) {
 // What every attention kernel of this file gets.
 // ---------------------------------------------------------------------------------------------
 struct WindowAttnParams {
-  const void* q;              // [n, nq * dk]
+  const void* q;              // [n, ld_q], head h at column h * dk
   void* out;                  // [n, ld_out], head h at column h * dv
   const void* cache;          // paged cache of the layer that owns the keys
   const int* page_table;      // [rows, max_pages]
@@ -192,12 +195,28 @@ struct WindowAttnParams {
   const float* sink;          // [nq] or null
   const void* gate;           // pre-activation of head h of query t at gate[t * ld_gate + h], or null
   int n, nq, nkv, dk, dv, page_size, max_pages, window, keep_first, far;
-  long long ld_out, ld_gate;
+  long long ld_q, ld_out, ld_gate;
   float scale;
+  float softcap;              // 0 = no cap
+  float temp_coef;            // 0 = no query temperature
+  double temp_every;
   float* ws;                  // split partial results (decode kernel, n_split > 1)
   int n_split;
   int* status;
 };
+
+// scale of the scores of a query at position i
+__device__ __forceinline__ float query_scale(const WindowAttnParams& p, int i) {
+  if (p.temp_coef == 0.f) return p.scale;
+  return p.scale * (1.0f + p.temp_coef * logf((float)floor((double)(i + 1) / p.temp_every) + 1.0f));
+}
+
+// tanh on the special-function unit, 1 - 2 / (1 + exp(2 x)): absolute error ~2^-22, saturates to +-1
+__device__ __forceinline__ float tanh_sfu(float x) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + ex2_approx(x * (2.0f * 1.4426950408889634f))));
+  return fmaf(-2.0f, r, 1.0f);
+}
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 
@@ -227,7 +246,8 @@ __global__ void __launch_bounds__(128) window_attn_plain_kernel(const WindowAttn
   const int t = (int)(wg / p.nq), h = (int)(wg % p.nq), kvh = h / (p.nq / p.nkv);
   const int i = p.pos[t];
   const int* pt = p.page_table + (size_t)p.row[t] * p.max_pages;
-  const T* q = reinterpret_cast<const T*>(p.q) + ((size_t)t * p.nq + h) * p.dk;
+  const T* q = reinterpret_cast<const T*>(p.q) + (size_t)t * p.ld_q + (size_t)h * p.dk;
+  const float scale = query_scale(p, i);
   for (int d = lane; d < p.dk; d += 32) s_q[warp][d] = to_f<T>(q[d]);
   __syncwarp();
   const size_t page_elems = (size_t)p.nkv * p.page_size * (p.dk + p.dv);
@@ -254,7 +274,8 @@ __global__ void __launch_bounds__(128) window_attn_plain_kernel(const WindowAttn
 #pragma unroll
           for (int u = 0; u < 8; ++u) dot = fmaf(s_q[warp][d + u], kv[u], dot);
         }
-        s = dot * p.scale;
+        s = dot * scale;
+        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
         if (p.bias != nullptr) s += p.bias[(size_t)h * (p.far + 1) + min(i - j, p.far)];
       }
       const float mx = fmaxf(m, warp_max(s));
@@ -336,7 +357,7 @@ __device__ __forceinline__ float finish_scale(const WindowAttnParams& p, int t, 
   return f;
 }
 
-template <int VEC, int GB, bool EXACT>   // EXACT: dk = dv = VEC * 64, known to the compiler
+template <int VEC, int GB, bool EXACT, bool CAP>   // EXACT: dk = dv = VEC * 64, known to the compiler; CAP: softcap > 0
 __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) window_decode_kernel(const WindowAttnParams p) {
   pdl_launch_dependents();
   pdl_wait();
@@ -407,17 +428,19 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
   } else {
     float qv[GB][DPL];
     const float* bias[GB];
+    const float q_mul = CAP ? query_scale(p, i) / p.softcap : query_scale(p, i) * LOG2E;   // q . k becomes the tanh argument / log2 units
+    const float cap = p.softcap * LOG2E;
 #pragma unroll
     for (int g = 0; g < GB; ++g) {
       const bool live = grp0 + g < G;
       const int h = kvh * G + (live ? grp0 + g : 0);
-      const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(p.q) + ((size_t)t * p.nq + h) * dk;
+      const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)t * p.ld_q + (size_t)h * dk;
       bias[g] = p.bias == nullptr ? nullptr : p.bias + (size_t)h * (p.far + 1);
 #pragma unroll
       for (int v = 0; v < VEC; ++v) {
         const int c = (v * 8 + gl) * 8;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) qv[g][v * 8 + e] = live && c < dk ? __bfloat162float(qp[c + e]) * (p.scale * LOG2E) : 0.f;
+        for (int e = 0; e < 8; ++e) qv[g][v * 8 + e] = live && c < dk ? __bfloat162float(qp[c + e]) * q_mul : 0.f;
       }
     }
     for (int it = 0; it < n_iter; ++it) {
@@ -465,6 +488,7 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
           d += __shfl_xor_sync(0xffffffffu, d, 1);
           d += __shfl_xor_sync(0xffffffffu, d, 2);
           d += __shfl_xor_sync(0xffffffffu, d, 4);
+          if constexpr (CAP) d = cap * tanh_sfu(d);
           sc[u][g] = ok[u] ? d + b[u][g] : -INFINITY;
         }
       }
@@ -619,7 +643,50 @@ __device__ __forceinline__ void tma_load_4d(void* smem_dst, const void* tmap, in
       : "memory");
 }
 
-template <int HK, int HV>
+// cap * tanh(mul * v) of 32 scores of a thread.  The arguments of trained attention mostly lie well inside (-1, 1), where
+// x P(x^2) with a degree-5 minimax P (fitted for the absolute error, 3.3e-7 in fp32) needs no special-function unit, the
+// busiest pipe of this kernel; a warp in which some argument is larger takes the exponential form for all of them.
+__device__ __forceinline__ uint64_t pack_f32x2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul_f32x2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ void soft_cap32(float* v, float mul, float cap) {
+  float big = fabsf(v[0]);
+#pragma unroll
+  for (int c = 1; c < 32; ++c) big = fmaxf(big, fabsf(v[c]));
+  if (__all_sync(0xffffffffu, big * mul <= 1.0f)) {
+    constexpr float A[6] = {0.999996854f, -0.333240038f, 0.132535252f, -0.0509728608f, 0.016114178f, -0.00283946425f};
+    uint64_t a[6];
+#pragma unroll
+    for (int k = 0; k < 6; ++k) a[k] = pack_f32x2(A[k] * cap, A[k] * cap);
+    const uint64_t m = pack_f32x2(mul, mul);
+#pragma unroll
+    for (int c = 0; c < 32; c += 2) {
+      const uint64_t x = mul_f32x2(pack_f32x2(v[c], v[c + 1]), m), u = mul_f32x2(x, x);
+      uint64_t y = a[5];
+#pragma unroll
+      for (int k = 4; k >= 0; --k) y = fma_f32x2(y, u, a[k]);
+      y = mul_f32x2(y, x);
+      asm("mov.b64 {%0, %1}, %2;" : "=f"(v[c]), "=f"(v[c + 1]) : "l"(y));
+    }
+  } else {
+#pragma unroll
+    for (int c = 0; c < 32; ++c) v[c] = cap * tanh_sfu(v[c] * mul);
+  }
+}
+
+template <int HK, int HV, bool CAP>
 __global__ void __launch_bounds__(WP_THREADS, WpCfg<HK, HV>::MIN_CTAS)
 window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                       const __grid_constant__ CUtensorMap tm_v, const WindowAttnParams p, const WindowTiles tl) {
@@ -739,8 +806,9 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     const int row = qd * 32 + lane;
     const bool row_ok = row < qn;
     const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
-    const float sc = p.scale * LOG2E;
     const int i = i0 + row;
+    const float sc = CAP ? 1.0f : query_scale(p, i) * LOG2E;
+    const float cap_mul = CAP ? query_scale(p, i) / p.softcap : 0.f, cap = p.softcap * LOG2E;
     const int iw0 = i0 + qd * 32, iw1 = iw0 + 31;             // positions of the warp's first and last query
     const int lo = p.window > i ? 0 : i - p.window + 1;
     const int lo_w1 = p.window > iw1 ? 0 : iw1 - p.window + 1;
@@ -755,7 +823,9 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       tmem_ld32(tmem_s + lane_off + half * 32, sv);
       tmem_ld_wait();
       const int dmin = iw0 - (j0 + 31), dmax = iw1 - j0;                 // distances inside the warp's 32 x 32 patch
-      if (bias == nullptr || dmin >= p.far) {
+      if constexpr (CAP) soft_cap32(sv, cap_mul, cap);
+      if (CAP && bias == nullptr) {
+      } else if (bias == nullptr || dmin >= p.far) {
 #pragma unroll
         for (int c = 0; c < 32; ++c) sv[c] = fmaf(sv[c], sc, far_bias);
       } else if (dmin >= 0 && dmax <= p.far) {
@@ -864,7 +934,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   }
 }
 
-template <int VEC, int GB, bool EXACT>
+template <int VEC, int GB, bool EXACT, bool CAP>
 static int launch_window_decode_as(const WindowAttnParams& p, cudaStream_t stream) {
   const int groups = (p.nq / p.nkv + GB - 1) / GB;
   const size_t ring = (size_t)WD_NSTAGE * WD_STAGE_PAGES * WD_PAGE * (p.dk + p.dv) * 2 + 128;
@@ -872,12 +942,12 @@ static int launch_window_decode_as(const WindowAttnParams& p, cudaStream_t strea
   const size_t smem = ring > merge ? ring : merge;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(window_decode_kernel<VEC, GB, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
+    if (cudaFuncSetAttribute(window_decode_kernel<VEC, GB, EXACT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
       return -10;
     configured = true;
   }
   if (smem > 160 * 1024) return -11;
-  cudaError_t e = launch_chain(window_decode_kernel<VEC, GB, EXACT>, dim3(p.nkv * groups, p.n, p.n_split), dim3(160), smem, stream, p);
+  cudaError_t e = launch_chain(window_decode_kernel<VEC, GB, EXACT, CAP>, dim3(p.nkv * groups, p.n, p.n_split), dim3(160), smem, stream, p);
   if (e == cudaSuccess && p.n_split > 1)
     e = launch_chain(window_decode_merge_kernel, dim3(p.n * p.nq), dim3(128), 0, stream, p);
   return e == cudaSuccess ? 0 : -3;
@@ -885,8 +955,10 @@ static int launch_window_decode_as(const WindowAttnParams& p, cudaStream_t strea
 
 template <int VEC, int GB>
 static int launch_window_decode(const WindowAttnParams& p, cudaStream_t stream) {
-  return p.dk == VEC * 64 && p.dv == VEC * 64 ? launch_window_decode_as<VEC, GB, true>(p, stream)
-                                              : launch_window_decode_as<VEC, GB, false>(p, stream);
+  const bool exact = p.dk == VEC * 64 && p.dv == VEC * 64;
+  if (p.softcap > 0.f)
+    return exact ? launch_window_decode_as<VEC, GB, true, true>(p, stream) : launch_window_decode_as<VEC, GB, false, true>(p, stream);
+  return exact ? launch_window_decode_as<VEC, GB, true, false>(p, stream) : launch_window_decode_as<VEC, GB, false, false>(p, stream);
 }
 
 // K (or V) of a paged cache as a 4-D tensor [pages][kv heads][16 tokens][dims], read in boxes of one page's 16 tokens x 64 dims
@@ -903,18 +975,39 @@ static int make_page_map(CUtensorMap* m, const void* base, int d, int nkv, int n
   return r == CUDA_SUCCESS ? 0 : -3;
 }
 
-template <int HK, int HV>
-static int launch_window_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
+template <int HK, int HV, bool CAP>
+static int launch_window_prefill_as(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
                                  const WindowAttnParams& p, const WindowTiles& tl, int n_tiles, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(window_prefill_kernel<HK, HV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(window_prefill_kernel<HK, HV, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              WpCfg<HK, HV>::SMEM_BYTES) != cudaSuccess)
       return -10;
     configured = true;
   }
-  window_prefill_kernel<HK, HV><<<dim3(n_tiles, p.nq), WP_THREADS, WpCfg<HK, HV>::SMEM_BYTES, stream>>>(mq, mk, mv, p, tl);
+  window_prefill_kernel<HK, HV, CAP><<<dim3(n_tiles, p.nq), WP_THREADS, WpCfg<HK, HV>::SMEM_BYTES, stream>>>(mq, mk, mv, p, tl);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+template <int HK, int HV>
+static int launch_window_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
+                                 const WindowAttnParams& p, const WindowTiles& tl, int n_tiles, cudaStream_t stream) {
+  return p.softcap > 0.f ? launch_window_prefill_as<HK, HV, true>(mq, mk, mv, p, tl, n_tiles, stream)
+                         : launch_window_prefill_as<HK, HV, false>(mq, mk, mv, p, tl, n_tiles, stream);
+}
+
+// queries as a [n, cols] matrix of row pitch ld, read in boxes of 128 tokens x 64 columns
+static int make_query_map(CUtensorMap* m, const void* base, int n, long long cols, long long ld) {
+  PfEncodeFn fn = pf_encode_fn();
+  if (fn == nullptr) return -1;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || ld % 8) return -2;
+  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)n};
+  cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
+  cuuint32_t box[2] = {64u, 128u}, estr[2] = {1u, 1u};
+  CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -3;
 }
 
 }  // namespace tahb
@@ -946,21 +1039,21 @@ extern "C" int tahb_qkv_post(const void* qkv, long long ld, const float* bias, c
   return e == cudaSuccess ? 0 : -3;
 }
 
+static int check_window_attn(const WindowAttnParams* p) {
+  return p->nkv <= 0 || p->nq % p->nkv || p->dk > 256 || p->dv > 256 || p->dk % 8 || p->dv % 8 || p->window < 1 || p->far < 0 ||
+         p->keep_first < 0 || p->ld_q < (long long)p->nq * p->dk || p->softcap < 0.f ||
+         (p->temp_coef != 0.f && !(p->temp_every > 0.0)) ? -2 : 0;
+}
+
 // Host-side description of one attention launch (same fields as WindowAttnParams).
 extern "C" int tahb_window_attn_plain(const WindowAttnParams* p, int f32, cudaStream_t stream) {
   if (p->n <= 0) return 0;
-  if (p->nkv <= 0 || p->nq % p->nkv || p->dk > 256 || p->dv > 256 || p->dk % 8 || p->dv % 8 || p->window < 1 || p->far < 0)
-    return -2;
+  if (check_window_attn(p)) return -2;
   const long long warps = (long long)p->n * p->nq;
   const dim3 grid((unsigned)((warps + 3) / 4));
   cudaError_t e = f32 ? launch_chain(window_attn_plain_kernel<float>, grid, dim3(128), 0, stream, *p)
                       : launch_chain(window_attn_plain_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, *p);
   return e == cudaSuccess ? 0 : -3;
-}
-
-static int check_window_attn(const WindowAttnParams* p) {
-  return p->nkv <= 0 || p->nq % p->nkv || p->dk > 256 || p->dv > 256 || p->dk % 8 || p->dv % 8 || p->window < 1 || p->far < 0 ||
-         p->keep_first < 0 ? -2 : 0;
 }
 
 // One query per entry (decode).  bias and sink in log2 units; ws: n * nq * n_split * (dv + 2) floats when n_split > 1.
@@ -988,7 +1081,7 @@ extern "C" int tahb_window_attn_tiles(const WindowAttnParams* p, const int* q0, 
   const size_t page_elems = (size_t)p->nkv * WD_PAGE * (p->dk + p->dv);
   CUtensorMap mq, mk, mv;
   int rc;
-  if ((rc = pf_make_map(&mq, p->q, p->n, (long long)p->nq * p->dk, 128u))) return rc;
+  if ((rc = make_query_map(&mq, p->q, p->n, (long long)p->nq * p->dk, p->ld_q))) return rc;
   if ((rc = make_page_map(&mk, p->cache, p->dk, p->nkv, n_pages, page_elems))) return rc;
   if ((rc = make_page_map(&mv, reinterpret_cast<const __nv_bfloat16*>(p->cache) + (size_t)p->nkv * WD_PAGE * p->dk, p->dv,
                           p->nkv, n_pages, page_elems))) return rc;

@@ -1,11 +1,15 @@
 // Kernels of decoders that keep the residual stream in fp32 (independent of the activation type T, bf16 or fp32):
 //
-//   embed_norm      x = scale * E[token];                     h = T(rms(x) * w)
-//   residual_norm   x += rms(y) * w_out;                      h = T(rms(x) * w_next)
+//   embed_norm           x = scale * E[token] (+ sinusoid(position));    h = T(rms_g(x) * w)
+//   residual_norm        x += rms(y) * w_out;                            h = T(rms(x) * w_next)
+//   residual_add_norm    x += mult * (y + sum of expert outputs);        h = T(rms_g(x) * w_next)
 //
-// with rms(v) = v / sqrt(mean(v^2) + eps).  residual_norm is the whole seam between two sublayers of a layer with a norm
-// before and after each sublayer: y is the sublayer's output projection, w_out the product of the output norm's weight
-// and the layer scale, w_next the weight of the norm that feeds the next projection.
+// with rms(v) = v / sqrt(mean(v^2) + eps), and rms_g the same over each of `groups` equal consecutive parts of the vector.
+// residual_norm is the whole seam between two sublayers of a layer with a norm before and after each sublayer: y is the
+// sublayer's output projection, w_out the product of the output norm's weight and the layer scale, w_next the weight of the
+// norm that feeds the next projection.  residual_add_norm is the seam between two layers whose mixer and feed-forward run
+// in parallel from one norm: y holds the sum of their output projections, and the outputs of a mixture of experts are
+// gathered from the experts' token lists on the way.
 //
 // Rows are padded: `ld` columns (a multiple of 64) of which the first `width` are real; padding columns of every operand
 // are zero, so only the mean knows the difference.
@@ -49,36 +53,172 @@ __device__ __forceinline__ float block_sum_128(float v, float* red) {
 
 __device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 
+// Inverse root mean squares of the `groups` parts of a row whose vectors c = threadIdx.x + i * RN_THREADS sit in v[i]; r[i]
+// receives the factor of each element of vector i (0 in the padding).  Parts of whole 128-element warp blocks (real model
+// sizes, one group included) are summed by warp shuffles, any other size through the row in shared memory.
+// sm: 64 + groups floats, and ld more when the part size is not a multiple of 128.
+template <int VPT>
+__device__ __forceinline__ void group_inv_rms(const float4* v, int width, int groups, int ld, float eps, float* sm, float4* r) {
+  const int gs = width / groups, nvec = ld / 4, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* inv = sm + 64;
+  if (gs % 128 == 0) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const float s = warp_sum(threadIdx.x + i * RN_THREADS < nvec ? sq4(v[i]) : 0.f);
+      if (lane == 0) sm[i * 4 + warp] = s;                  // elements 128 (4 i + warp) ..
+    }
+    __syncthreads();
+    const int per = gs / 128;
+    for (int g = threadIdx.x; g < groups; g += RN_THREADS) {
+      float s = 0.f;
+      for (int k = 0; k < per; ++k) s += sm[g * per + k];
+      inv[g] = 1.0f / sqrtf(s / (float)gs + eps);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int g = (i * 4 + warp) / per;
+      const float f = g < groups ? inv[g] : 0.f;
+      r[i] = make_float4(f, f, f, f);
+    }
+    return;
+  }
+  float* row = inv + groups;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) {
+      row[4 * c] = v[i].x; row[4 * c + 1] = v[i].y; row[4 * c + 2] = v[i].z; row[4 * c + 3] = v[i].w;
+    }
+  }
+  __syncthreads();
+  for (int g = warp; g < groups; g += RN_THREADS / 32) {
+    float s = 0.f;
+    for (int k = lane; k < gs; k += 32) s = fmaf(row[g * gs + k], row[g * gs + k], s);
+    s = warp_sum(s);
+    if (lane == 0) inv[g] = 1.0f / sqrtf(s / (float)gs + eps);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = 4 * (threadIdx.x + i * RN_THREADS);
+    auto at = [&](int e) { return e < width ? inv[e / gs] : 0.f; };
+    r[i] = make_float4(at(c), at(c + 1), at(c + 2), at(c + 3));
+  }
+}
+
+static size_t group_rms_smem(int width, int groups, int ld) {
+  return (64 + (size_t)groups + ((width / groups) % 128 ? ld : 0)) * 4;
+}
+
+// Sine and cosine of p * f for the pair of entries (2 i, 2 i + 1); f = hi + lo keeps the angle's rounding error out of the
+// result at large positions.
+__device__ __forceinline__ float2 sin_cos_pair(float p, float hi, float lo) {
+  const float a = p * hi, e = fmaf(p, lo, fmaf(p, hi, -a));
+  float s, c;
+  sincosf(a, &s, &c);
+  return make_float2(fmaf(e, c, s), fmaf(-e, s, c));
+}
+
+// pos / freq: position of every token and [2, (width + 1) / 2] frequencies (high parts, then low parts), or null
 template <typename T, int VPT>
 __global__ void __launch_bounds__(RN_THREADS) embed_norm_kernel(const T* __restrict__ E, const int* __restrict__ tok,
-                                                                float scale, float* __restrict__ x,
+                                                                float scale, const int* __restrict__ pos,
+                                                                const float* __restrict__ freq, float* __restrict__ x,
                                                                 const float* __restrict__ w, T* __restrict__ h, int vocab,
-                                                                int width, int ld, float eps) {
+                                                                int width, int groups, int ld, float eps) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float red[4];
+  extern __shared__ float gsm[];
   const size_t row = blockIdx.x;
   const int id = min(max(tok[row], 0), vocab - 1);
   const int nvec = ld / 4;
-  float4 v[VPT];
-  float ss = 0.f;
+  float4 v[VPT], r[VPT];
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * RN_THREADS;
     if (c < nvec) {
       v[i] = Vec4<T>::load(E + (size_t)id * ld + c * 4);
       v[i].x *= scale; v[i].y *= scale; v[i].z *= scale; v[i].w *= scale;
-      ss += sq4(v[i]);
+      if (freq != nullptr) {
+        const float p = (float)pos[row];
+        const float* lo = freq + (width + 1) / 2;
+        if (4 * c < width) {
+          const float2 a = sin_cos_pair(p, freq[2 * c], lo[2 * c]);
+          v[i].x += a.x;
+          if (4 * c + 1 < width) v[i].y += a.y;
+        }
+        if (4 * c + 2 < width) {
+          const float2 a = sin_cos_pair(p, freq[2 * c + 1], lo[2 * c + 1]);
+          v[i].z += a.x;
+          if (4 * c + 3 < width) v[i].w += a.y;
+        }
+      }
       Vec4<float>::store(x + row * ld + c * 4, v[i]);
     }
   }
-  const float r = 1.0f / sqrtf(block_sum_128(ss, red) / (float)width + eps);
+  group_inv_rms<VPT>(v, width, groups, ld, eps, gsm, r);
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * RN_THREADS;
     if (c < nvec) {
       const float4 g = Vec4<float>::load(w + c * 4);
-      Vec4<T>::store(h + row * ld + c * 4, make_float4(v[i].x * r * g.x, v[i].y * r * g.y, v[i].z * r * g.z, v[i].w * r * g.w));
+      Vec4<T>::store(h + row * ld + c * 4,
+                     make_float4(v[i].x * r[i].x * g.x, v[i].y * r[i].y * g.y, v[i].z * r[i].z * g.z, v[i].w * r[i].w * g.w));
+    }
+  }
+}
+
+// y_ex / slot: expert outputs [list rows, ld] and the list rows slot[row * top ..] of this token, or null
+template <typename T, int VPT>
+__global__ void __launch_bounds__(RN_THREADS) residual_add_norm_kernel(const T* __restrict__ y, long long ldy,
+                                                                       const T* __restrict__ y_ex,
+                                                                       const int* __restrict__ slot, int top, float mult,
+                                                                       float* __restrict__ x, const float* __restrict__ w_next,
+                                                                       T* __restrict__ h, int width, int groups, int ld,
+                                                                       float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float gsm[];
+  const size_t row = blockIdx.x;
+  const int nvec = ld / 4;
+  float4 v[VPT], r[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) r[i] = Vec4<T>::load(y + row * ldy + c * 4);
+  }
+  if (y_ex != nullptr) {
+    for (int j = 0; j < top; ++j) {
+      const T* src = y_ex + (size_t)slot[row * top + j] * ld;
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + i * RN_THREADS;
+        if (c < nvec) {
+          const float4 e = Vec4<T>::load(src + c * 4);
+          r[i].x += e.x; r[i].y += e.y; r[i].z += e.z; r[i].w += e.w;
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) {
+      v[i] = Vec4<float>::load(x + row * ld + c * 4);
+      v[i].x = fmaf(mult, r[i].x, v[i].x); v[i].y = fmaf(mult, r[i].y, v[i].y);
+      v[i].z = fmaf(mult, r[i].z, v[i].z); v[i].w = fmaf(mult, r[i].w, v[i].w);
+      Vec4<float>::store(x + row * ld + c * 4, v[i]);
+    }
+  }
+  group_inv_rms<VPT>(v, width, groups, ld, eps, gsm, r);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) {
+      const float4 g = Vec4<float>::load(w_next + c * 4);
+      Vec4<T>::store(h + row * ld + c * 4,
+                     make_float4(v[i].x * r[i].x * g.x, v[i].y * r[i].y * g.y, v[i].z * r[i].z * g.z, v[i].w * r[i].w * g.w));
     }
   }
 }
@@ -281,13 +421,15 @@ __global__ void swiglu_f32_kernel(const float* __restrict__ gu, float* __restric
 }
 
 template <typename T>
-static int embed_norm_launch(const void* E, const int* tok, float scale, float* x, const float* w, void* h, int M,
-                             int vocab, int width, int ld, float eps, cudaStream_t stream) {
+static int embed_norm_launch(const void* E, const int* tok, float scale, const int* pos, const float* freq, float* x,
+                             const float* w, void* h, int M, int vocab, int width, int groups, int ld, float eps,
+                             cudaStream_t stream) {
+  const size_t smem = group_rms_smem(width, groups, ld);
   const int need = (ld / 4 + RN_THREADS - 1) / RN_THREADS;
   auto e = reinterpret_cast<const T*>(E);
   auto o = reinterpret_cast<T*>(h);
   cudaError_t rc;
-#define TAHB_EN(V_) rc = launch_chain(embed_norm_kernel<T, V_>, dim3(M), dim3(RN_THREADS), 0, stream, e, tok, scale, x, w, o, vocab, width, ld, eps)
+#define TAHB_EN(V_) rc = launch_chain(embed_norm_kernel<T, V_>, dim3(M), dim3(RN_THREADS), smem, stream, e, tok, scale, pos, freq, x, w, o, vocab, width, groups, ld, eps)
   if (need <= 1) TAHB_EN(1);
   else if (need <= 2) TAHB_EN(2);
   else if (need <= 4) TAHB_EN(4);
@@ -316,6 +458,27 @@ static int residual_norm_launch(const void* y, long long ldy, float* x, const fl
   return rc == cudaSuccess ? 0 : -3;
 }
 
+template <typename T>
+static int residual_add_norm_launch(const void* y, long long ldy, const void* y_ex, const int* slot, int top, float mult,
+                                    float* x, const float* w_next, void* h, int M, int width, int groups, int ld, float eps,
+                                    cudaStream_t stream) {
+  const int need = (ld / 4 + RN_THREADS - 1) / RN_THREADS;
+  const size_t smem = group_rms_smem(width, groups, ld);
+  auto yy = reinterpret_cast<const T*>(y);
+  auto ye = reinterpret_cast<const T*>(y_ex);
+  auto o = reinterpret_cast<T*>(h);
+  cudaError_t rc;
+#define TAHB_RA(V_) rc = launch_chain(residual_add_norm_kernel<T, V_>, dim3(M), dim3(RN_THREADS), smem, stream, yy, ldy, ye, slot, top, mult, x, w_next, o, width, groups, ld, eps)
+  if (need <= 1) TAHB_RA(1);
+  else if (need <= 2) TAHB_RA(2);
+  else if (need <= 4) TAHB_RA(4);
+  else if (need <= 8) TAHB_RA(8);
+  else if (need <= 16) TAHB_RA(16);
+  else return -2;
+#undef TAHB_RA
+  return rc == cudaSuccess ? 0 : -3;
+}
+
 template <typename T, int TOK>
 static int few_linear_launch(const void* x, long long ldx, const void* w, const float* b, float* out, int M, int K, int F,
                              cudaStream_t stream) {
@@ -337,12 +500,25 @@ static int few_linear_launch(const void* x, long long ldx, const void* w, const 
 
 using namespace tahb;
 
-extern "C" int tahb_embed_norm(const void* E, const int* tok, float scale, float* x, const float* w, void* h, int M,
-                               int vocab, int width, int ld, float eps, int f32, cudaStream_t stream) {
+// pos / freq: sinusoidal positions (see embed_norm_kernel), or null.  groups must divide width.
+extern "C" int tahb_embed_norm(const void* E, const int* tok, float scale, const int* pos, const float* freq, float* x,
+                               const float* w, void* h, int M, int vocab, int width, int groups, int ld, float eps, int f32,
+                               cudaStream_t stream) {
   if (M <= 0) return 0;
-  if (ld % 4 || width > ld) return -1;
-  return f32 ? embed_norm_launch<float>(E, tok, scale, x, w, h, M, vocab, width, ld, eps, stream)
-             : embed_norm_launch<__nv_bfloat16>(E, tok, scale, x, w, h, M, vocab, width, ld, eps, stream);
+  if (ld % 4 || width > ld || groups < 1 || width % groups || (freq != nullptr && pos == nullptr)) return -1;
+  return f32 ? embed_norm_launch<float>(E, tok, scale, pos, freq, x, w, h, M, vocab, width, groups, ld, eps, stream)
+             : embed_norm_launch<__nv_bfloat16>(E, tok, scale, pos, freq, x, w, h, M, vocab, width, groups, ld, eps, stream);
+}
+
+// x += mult * (y + sum_j y_ex[slot[., j]]); h = rms_g(x) * w_next.  y_ex / slot null: no expert outputs.
+extern "C" int tahb_residual_add_norm(const void* y, long long ldy, const void* y_ex, const int* slot, int top, float mult,
+                                      float* x, const float* w_next, void* h, int M, int width, int groups, int ld, float eps,
+                                      int f32, cudaStream_t stream) {
+  if (M <= 0) return 0;
+  if (ld % 4 || ldy % 4 || width > ld || groups < 1 || width % groups || (y_ex != nullptr && slot == nullptr)) return -1;
+  return f32 ? residual_add_norm_launch<float>(y, ldy, y_ex, slot, top, mult, x, w_next, h, M, width, groups, ld, eps, stream)
+             : residual_add_norm_launch<__nv_bfloat16>(y, ldy, y_ex, slot, top, mult, x, w_next, h, M, width, groups, ld, eps,
+                                                       stream);
 }
 
 extern "C" int tahb_residual_norm(const void* y, long long ldy, float* x, const float* w_out, const float* w_next, void* h,

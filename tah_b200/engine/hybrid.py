@@ -1,5 +1,6 @@
-"""HybridEngine: decoders whose layers differ - windowed attention over the paged cache beside recurrent layers with a
-state per row - on an fp32 residual stream.
+"""HybridEngine: decoders that list their layers one by one - windowed attention over the paged cache, recurrent layers with
+a state per row, dense feed-forwards and mixtures of experts, sublayers one after the other or side by side - on an fp32
+residual stream.
 
 One function, :meth:`HybridEngine._layers`, runs the layers for a packed set of tokens.  It serves
 
@@ -10,8 +11,7 @@ One function, :meth:`HybridEngine._layers`, runs the layers for a packed set of 
 * the decode tick - one token of every row, captured in a CUDA graph (:class:`tah_b200.engine.base.DecodeEngine`).
 
 Rows are cache rows: a row owns pages of the KV pool and one slot of the recurrent state.  ``admit`` / ``release`` hand
-them out.  Sizes are padded once, when the weights are laid out: matrix rows and columns to multiples of 64, head sizes
-to multiples of 8, with zeros that drop out of every result.
+them out.  The weights are laid out for the kernels once, with padded sizes (:mod:`tah_b200.engine.hybrid_weights`).
 """
 from __future__ import annotations
 
@@ -23,161 +23,15 @@ import torch
 
 from tah_b200.engine.base import DecodeEngine
 from tah_b200.engine.kv_cache import CacheGeometry, LayerKV, PagedKVCache, RecurrentState
-from tah_b200.models.gunuvik import AttentionSpec, GunuvikForCausalLM, MLSTMSpec
+from tah_b200.engine.hybrid_weights import (AttentionLayer, BlockWeights, HybridWeights, MemoryLayer, MixtureLayer, PolyNormLayer,
+                                             distance_table)
+from tah_b200.models.layered import LayeredForCausalLM
 from tah_b200.ops import cuda as K
 from tah_b200.utils.observe import nvtx_range
 
 NO_WINDOW = 2 ** 31 - 1
-LOG2E = 1.4426950408889634
 TILE = 128                        # tokens of an attention query tile and of an mLSTM chunk
 MEMORY_CHUNKS = 192               # chunks per mLSTM launch (bounds the workspace)
-
-
-def _pad(n: int, m: int) -> int:
-    return (n + m - 1) // m * m
-
-
-def distance_table(rel: torch.Tensor, far: int) -> torch.Tensor:
-    """``[heads, far + 1]`` fp32 bias by distance from a bucket table ``rel [rows, heads]``: distance ``n`` below
-    ``half = rows // 2`` has a row of its own; larger ones share rows logarithmically up to ``far``, from where the last
-    row serves.  The bucket's floor is evaluated in integers (``(far / half) ** k <= (n / half) ** (rows - half)``)."""
-    rows = rel.shape[0]
-    half = rows // 2
-    if far <= half:
-        raise ValueError(f"distance bias: the far end {far} lies inside the {half} exact distances")
-    m, k, idx = rows - half, 0, []
-    for n in range(far + 1):
-        if n < half:
-            idx.append(n)
-            continue
-        while k < m and far ** (k + 1) * half ** (m - k - 1) <= n ** m:
-            k += 1
-        idx.append(min(rows - 1, half + k))
-    return rel.float()[torch.tensor(idx, device=rel.device)].t().contiguous()
-
-
-@dataclass
-class AttentionLayer:
-    spec: AttentionSpec
-    dk: int
-    dv: int
-    nkv: int                      # heads this layer writes (0: it reads another layer's cache)
-    w_in: torch.Tensor            # rows: queries, own keys, own values, gate numbers
-    b_in: torch.Tensor
-    gate_col: int
-    q_norm: torch.Tensor
-    k_norm: Optional[torch.Tensor]
-    bias: torch.Tensor            # [heads, far + 1], natural units for the plain kernel, log2 units for the others
-    sink: torch.Tensor
-    w_o: torch.Tensor
-
-
-@dataclass
-class MemoryLayer:
-    spec: MLSTMSpec
-    dk: int
-    dv: int
-    w_in: torch.Tensor            # rows: q, k, v, output gate
-    w_if: torch.Tensor            # input and forget gate rows
-    b_if: torch.Tensor
-    norm: torch.Tensor
-    w_o: torch.Tensor
-
-
-@dataclass
-class BlockWeights:
-    mixer: object
-    norm1: torch.Tensor
-    out1: torch.Tensor            # output norm weight x layer scale
-    norm2: Optional[torch.Tensor] = None
-    out2: Optional[torch.Tensor] = None
-    w_gu: Optional[torch.Tensor] = None
-    w_down: Optional[torch.Tensor] = None
-
-
-class HybridWeights:
-    """Kernel-ready layout of a Gunuvik model's weights in the activation type ``dtype``."""
-
-    def __init__(self, model: GunuvikForCausalLM, dtype: torch.dtype, plain: bool):
-        cfg = model.config
-        unit = 1.0 if plain else LOG2E
-        dev = model.device
-        self.W, self.Wp = cfg.hidden_size, _pad(cfg.hidden_size, 64)
-        self.vocab = cfg.vocab_size
-        self.vocab_shard = (0, self.vocab, _pad(self.vocab, 64))
-        T = model.tensor
-
-        def vec(t, n):                                       # fp32 vector padded to n
-            o = torch.zeros(n, dtype=torch.float32, device=dev)
-            o[:t.numel()] = t.float()
-            return o
-
-        def heads_rows(w, h, d, dp):                         # [h * d, W] -> [h * dp, Wp]
-            o = torch.zeros(h, dp, self.Wp, dtype=dtype, device=dev)
-            o[:, :d, :w.shape[1]] = w.view(h, d, -1)
-            return o.view(h * dp, self.Wp)
-
-        def heads_vec(b, h, d, dp):
-            o = torch.zeros(h, dp, dtype=torch.float32, device=dev)
-            o[:, :d] = b.float().view(h, d)
-            return o.view(-1)
-
-        def heads_cols(w, h, d, dp):                         # [W, h * d] -> [Wp, pad64(h * dp)]
-            o = torch.zeros(self.Wp, _pad(h * dp, 64), dtype=dtype, device=dev)
-            o[:w.shape[0], :h * dp].view(w.shape[0], h, dp)[:, :, :d] = w.view(w.shape[0], h, d)
-            return o
-
-        def mat(w, rows, cols):
-            o = torch.zeros(rows, cols, dtype=dtype, device=dev)
-            o[:w.shape[0], :w.shape[1]] = w
-            return o
-
-        def stack(parts):                                    # row blocks, padded to a multiple of 64 rows
-            n = sum(p.shape[0] for p in parts)
-            return mat(torch.cat(parts), _pad(n, 64), self.Wp)
-
-        self.embed = mat(T("embed"), self.vocab, self.Wp)
-        self.head = mat(T("head"), self.vocab_shard[2], self.Wp)
-        self.final_norm = vec(T("final.norm"), self.Wp)
-        self.layers: List[BlockWeights] = []
-        for i, l in enumerate(cfg.layers):
-            p, m = f"l{i}.", l.mixer
-            x = p + "mix."
-            dk, dv = _pad(m.dim, 8), _pad(m.vdim, 8)
-            w_o = heads_cols(T(x + "o"), m.heads, m.vdim, dv)
-            if isinstance(m, AttentionSpec):
-                if max(dk, dv) > 256:
-                    raise NotImplementedError("attention head sizes above 256")
-                H, G = m.heads, m.kv_heads
-                rows = [heads_rows(T(x + "q"), H, m.dim, dk)]
-                bias = [heads_vec(T(x + "q.b"), H, m.dim, dk)]
-                own = m.kv_from is None
-                if own:
-                    rows += [heads_rows(T(x + "k"), G, m.dim, dk), heads_rows(T(x + "v"), G, m.vdim, dv)]
-                    bias += [heads_vec(T(x + "k.b"), G, m.dim, dk), heads_vec(T(x + "v.b"), G, m.vdim, dv)]
-                gate_col = sum(r.shape[0] for r in rows)
-                w_in = stack(rows + [heads_rows(T(x + "g"), H, 1, 1)])
-                mixer = AttentionLayer(m, dk, dv, G if own else 0, w_in, vec(torch.cat(bias), w_in.shape[0]), gate_col,
-                                       vec(T(x + "q.norm"), dk), vec(T(x + "k.norm"), dk) if own else None,
-                                       distance_table(T(x + "rel"), m.bias_max) * unit, vec(T(x + "sink"), H) * unit, w_o)
-            else:
-                if max(dk, dv) > 1024:
-                    raise NotImplementedError("mLSTM head sizes above 1024")
-                H = m.heads
-                w_in = stack([heads_rows(T(x + "q"), H, m.dim, dk), heads_rows(T(x + "k"), H, m.dim, dk),
-                              heads_rows(T(x + "v"), H, m.vdim, dv), heads_rows(T(x + "g"), H, m.vdim, dv)])
-                w_if = mat(torch.cat([T(x + "i"), T(x + "f")]), 2 * H, self.Wp)
-                mixer = MemoryLayer(m, dk, dv, w_in, w_if, torch.cat([T(x + "i.b"), T(x + "f.b")]).float(),
-                                    heads_vec(T(x + "norm"), H, m.vdim, dv), w_o)
-            b = BlockWeights(mixer, vec(T(p + "norm1"), self.Wp), vec(T(p + "norm1b").float() * T(p + "ls1").float(), self.Wp))
-            if l.ff is not None:
-                Ip = _pad(l.ff, 64)
-                gu = torch.cat([mat(T(p + "mlp.gate"), Ip, self.Wp), mat(T(p + "mlp.up"), Ip, self.Wp)])
-                b.w_gu = K.interleave_gate_up(gu) if dtype == torch.bfloat16 else gu
-                b.w_down = mat(T(p + "mlp.down"), self.Wp, Ip)
-                b.norm2 = vec(T(p + "norm2"), self.Wp)
-                b.out2 = vec(T(p + "norm2b").float() * T(p + "ls2").float(), self.Wp)
-            self.layers.append(b)
 
 
 class _Plan:
@@ -208,10 +62,12 @@ class _Buffers:
     def __init__(self, w: HybridWeights, n: int, dtype, dev, n_dec: int, chunks: int = 0):
         e = lambda *s: torch.empty(*s, dtype=dtype, device=dev)
         mix = [b.mixer for b in w.layers]
+        moe = [b.ff for b in w.layers if isinstance(b.ff, MixtureLayer)]
         self.x = torch.empty(n, w.Wp, dtype=torch.float32, device=dev)
         self.h, self.y = e(n, w.Wp), e(n, w.Wp)
         self.proj = e(n, max(m.w_in.shape[0] for m in mix))
-        self.q = e(n, max([m.spec.heads * m.dk for m in mix if isinstance(m, AttentionLayer)] or [0]))
+        self.q = e(n, max([m.spec.heads * m.dk for m in mix if isinstance(m, AttentionLayer) and m.own_queries]
+                          or [0]))
         # columns between heads * dv and the padded width meet zero weight columns; they only have to be finite
         self.o = torch.zeros(n, max(m.w_o.shape[1] for m in mix), dtype=dtype, device=dev)
         self.gates = torch.empty(n * max([m.w_if.shape[0] for m in mix if isinstance(m, MemoryLayer)] or [0]),
@@ -222,6 +78,13 @@ class _Buffers:
         self.mem_ws = f32(max([K.mlstm_chunk_ws_floats(chunks, m.spec.heads, m.dk, m.dv) for m in mix
                                if isinstance(m, MemoryLayer)] or [0]))
         self.act = e(n, max([b.w_down.shape[1] for b in w.layers if b.w_down is not None] or [0]))
+        # experts: logits of router and shared gate, token lists, their rows, activations and outputs
+        self.router = f32(n * max([f.w_router.shape[0] for f in moe] or [0]))
+        self.lists = {k: K.ExpertLists(n, *k, dtype, dev) for k in {(f.spec.experts, f.spec.top) for f in moe}}
+        rows = lambda f: self.lists[f.spec.experts, f.spec.top].rows
+        most = max([rows(f) for f in moe] or [0])
+        self.list_x, self.list_y = e(most * w.Wp), e(most * w.Wp)
+        self.list_act = e(max([rows(f) * f.cols for f in moe] or [0]))
 
 
 @dataclass
@@ -233,7 +96,7 @@ class StepEntry:
 
 
 class HybridEngine(DecodeEngine):
-    def __init__(self, model: GunuvikForCausalLM, max_rows: int = 64, max_seq_len: int = 2048, page_size: int = 16,
+    def __init__(self, model: LayeredForCausalLM, max_rows: int = 64, max_seq_len: int = 2048, page_size: int = 16,
                  use_cuda_graph: bool = True, prefill_tokens: int = 16384):
         """``prefill_tokens``: the most prompt tokens one step runs (longer prompts are cut into portions)."""
         self.model, self.cfg = model, model.config
@@ -294,18 +157,25 @@ class HybridEngine(DecodeEngine):
     # ------------------------------------------------------------------------------------------
     # the layers
     # ------------------------------------------------------------------------------------------
-    def _attention(self, li: int, m: AttentionLayer, b: _Buffers, plan: _Plan) -> torch.Tensor:
+    def _attention(self, li: int, m: AttentionLayer, proj: torch.Tensor, b: _Buffers, plan: _Plan) -> torch.Tensor:
+        """Attention of one layer from its projection ``proj``; returns ``b.o`` with the heads in its first columns."""
         s = m.spec
         n = b.h.shape[0]
-        proj = K.linear(b.h, m.w_in, out=b.proj[:, :m.w_in.shape[0]])
-        q = b.q.view(-1)[:n * s.heads * m.dk].view(n, s.heads * m.dk)
         pool = self.kv.layer_pool(0, li)
-        K.qkv_post(proj, m.b_in, m.q_norm, m.k_norm, q, pool, plan.slot, s.heads, m.nkv, m.dk, m.dv, s.dim, self.page_size,
-                   self.cfg.rms_norm_eps)
+        post = dict(dk=m.dk, dv=m.dv, dim=s.dim, page_size=self.page_size, eps=self.cfg.rms_norm_eps)
+        if m.own_queries:
+            q = b.q.view(-1)[:n * s.heads * m.dk].view(n, s.heads * m.dk)
+            K.qkv_post(proj, m.b_in, m.q_norm, m.k_norm, q, pool, plan.slot, s.heads, m.nkv, **post)
+        else:                                      # queries as projected; only new keys and values have to move
+            q = proj[:, :s.heads * m.dk]
+            if m.nkv:
+                K.qkv_post(proj[:, m.kv_col:], None, None, None, None, pool, plan.slot, 0, m.nkv, **post)
         o = b.o[:, :m.w_o.shape[1]]
         kw = dict(nq=s.heads, nkv=s.kv_heads, dk=m.dk, dv=m.dv, page_size=self.page_size, scale=s.scale,
-                  window=NO_WINDOW if s.window is None else s.window, keep_first=s.keep_first, bias=m.bias, sink=m.sink)
-        gate, pt, nd = proj[:, m.gate_col:m.gate_col + s.heads], self.kv.page_table[0], plan.n_dec
+                  window=NO_WINDOW if s.window is None else s.window, keep_first=s.keep_first, bias=m.bias, sink=m.sink,
+                  softcap=s.softcap, q_temp=s.q_temp)
+        pt, nd = self.kv.page_table[0], plan.n_dec
+        gate = None if m.gate_col is None else proj[:, m.gate_col:m.gate_col + s.heads]
         if self.plain:
             K.window_attn_plain(q, o, pool, pt, plan.pos, plan.row, gate=gate, **kw)
             return o
@@ -316,10 +186,9 @@ class HybridEngine(DecodeEngine):
             K.window_attn_tiles(q, o, pool, pt, plan.pos, plan.row, plan.tile_q0, plan.tile_qn, self.kv.n_pages[0], gate=gate, **kw)
         return o
 
-    def _memory(self, li: int, m: MemoryLayer, b: _Buffers, plan: _Plan) -> torch.Tensor:
+    def _memory(self, li: int, m: MemoryLayer, proj: torch.Tensor, b: _Buffers, plan: _Plan) -> torch.Tensor:
         s = m.spec
         n, nd = b.h.shape[0], plan.n_dec
-        proj = K.linear(b.h, m.w_in, out=b.proj[:, :m.w_in.shape[0]])
         gates = K.few_linear(b.h, m.w_if, m.b_if, out=b.gates[:n * m.w_if.shape[0]].view(n, -1))
         o = b.o[:, :m.w_o.shape[1]]
         kw = dict(heads=s.heads, dk=m.dk, dv=m.dv, dim=s.dim, vdim=s.vdim, cap=s.gate_cap, eps=self.cfg.rms_norm_eps)
@@ -335,23 +204,63 @@ class HybridEngine(DecodeEngine):
                                chunk_len=plan.tile_qn[ta:tb], seq_chunk0=chunk0, seq_chunks=chunks, ws=b.mem_ws, **kw)
         return o
 
+    def _mixture(self, f: MixtureLayer, proj: torch.Tensor, b: _Buffers):
+        """Routed experts of the tokens in ``b.h``: ``(outputs by list row, list rows of every token)``; the shared
+        expert's activation goes to its columns of ``b.o``."""
+        s, n = f.spec, b.h.shape[0]
+        L = b.lists[s.experts, s.top]
+        z = K.few_linear(b.h, f.w_router, None, out=b.router[:n * f.w_router.shape[0]].view(n, -1))
+        K.moe_route(z, L)
+        view = lambda t, cols: t[:L.rows * cols].view(L.rows, cols)
+        x = K.moe_gather(b.h, L, view(b.list_x, b.h.shape[1]))
+        act = K.moe_glu_linear(x, f.w_gu, s.expert.limit, L, view(b.list_act, f.cols))
+        y = K.moe_linear(act, f.w_down, L, view(b.list_y, b.h.shape[1]))
+        if f.shared is not None:
+            c = f.shared
+            K.clamped_glu(proj[:, c.in_col:c.in_col + 2 * c.cols], c.limit, b.o[:, c.out_col:c.out_col + c.cols],
+                          gate=z[:, s.experts])
+        return y, L.slot
+
+    def _parallel_layer(self, li: int, L: BlockWeights, proj: torch.Tensor, w_next: torch.Tensor, b: _Buffers, plan: _Plan) -> None:
+        """Mixer and feed-forward beside each other: both read the projection of ``b.h``, one product over the columns of
+        both brings them back, and one residual step adds their sum."""
+        f, y_ex, slot = L.ff, None, None
+        if isinstance(f, PolyNormLayer):
+            K.poly_norm(proj[:, f.in_col:f.in_col + f.cols], f.act, f.n, self.cfg.rms_norm_eps,
+                        b.o[:, f.out_col:f.out_col + f.cols])
+        elif isinstance(f, MixtureLayer):
+            y_ex, slot = self._mixture(f, proj, b)
+        K.linear(self._attention(li, L.mixer, proj, b, plan), L.mixer.w_o, out=b.y)
+        K.residual_add_norm(b.y, b.x, self.cfg.residual_mult, w_next, self.w.W, self.cfg.norm_groups, self.cfg.rms_norm_eps,
+                            b.h, y_ex, slot)
+
     def _layers(self, b: _Buffers, plan: _Plan) -> torch.Tensor:
         """Run every layer on the packed tokens of ``plan`` (``b.x`` / ``b.h`` hold their embeddings and first normed
         input); returns the final-norm output."""
         w, eps = self.w, self.cfg.rms_norm_eps
         n_layers = len(w.layers)
         for li, L in enumerate(w.layers):
-            run = self._attention if isinstance(L.mixer, AttentionLayer) else self._memory
-            K.linear(run(li, L.mixer, b, plan), L.mixer.w_o, out=b.y)
             after = w.layers[li + 1].norm1 if li + 1 < n_layers else w.final_norm
-            K.residual_norm(b.y, b.x, L.out1, L.norm2 if L.w_gu is not None else after, w.W, eps, b.h)
-            if L.w_gu is not None:
-                act = K.swiglu_linear(b.h, L.w_gu, out=b.act[:, :L.w_down.shape[1]])
-                K.linear(act, L.w_down, out=b.y)
-                K.residual_norm(b.y, b.x, L.out2, after, w.W, eps, b.h)
+            proj = K.linear(b.h, L.mixer.w_in, out=b.proj[:, :L.mixer.w_in.shape[0]])
+            if L.parallel:
+                self._parallel_layer(li, L, proj, after, b, plan)
+            else:
+                run = self._attention if isinstance(L.mixer, AttentionLayer) else self._memory
+                K.linear(run(li, L.mixer, proj, b, plan), L.mixer.w_o, out=b.y)
+                K.residual_norm(b.y, b.x, L.out1, L.norm2 if L.w_gu is not None else after, w.W, eps, b.h)
+                if L.w_gu is not None:
+                    act = K.swiglu_linear(b.h, L.w_gu, out=b.act[:, :L.w_down.shape[1]])
+                    K.linear(act, L.w_down, out=b.y)
+                    K.residual_norm(b.y, b.x, L.out2, after, w.W, eps, b.h)
             if self.layer_hook is not None:
                 self.layer_hook(li, b.x[:, :w.W])
         return b.h
+
+    def _embed(self, b: _Buffers, plan: _Plan) -> None:
+        """``b.x``: the residual stream of the tokens of ``plan``; ``b.h``: the first layer's normed input."""
+        w = self.w
+        K.embed_norm(w.embed, plan.tok, self.cfg.embedding_scale, w.layers[0].norm1, w.W, self.cfg.rms_norm_eps, b.x, b.h,
+                     groups=self.cfg.norm_groups, pos=plan.pos, freq=w.freq)
 
     # ------------------------------------------------------------------------------------------
     # one step of portions and single tokens
@@ -404,8 +313,7 @@ class HybridEngine(DecodeEngine):
         plan.groups = [(t, t + k, d_first[a:z], d_tiles[a:z]) for a, z, t, k in groups]
         K.kv_append(d_rows, d_counts, d_start, self.kv, 0, plan.pos, plan.row, plan.slot)
         b = _Buffers(self.w, n, self.dtype, dev, n_dec, 0 if self.plain else max([g[3] for g in groups] or [0]))
-        K.embed_norm(self.w.embed, plan.tok, self.cfg.embedding_scale, self.w.layers[0].norm1, self.w.W,
-                     self.cfg.rms_norm_eps, b.x, b.h)
+        self._embed(b, plan)
         h = self._layers(b, plan)
         if not want:
             return torch.empty(0, self.w.vocab, dtype=self.dtype, device=dev)
@@ -506,7 +414,7 @@ class HybridEngine(DecodeEngine):
         """Enqueue one decode tick on the current stream (graph-capturable)."""
         w = self.w
         s.binding.tick_begin(None, None, None)
-        K.embed_norm(w.embed, s.tok, self.cfg.embedding_scale, w.layers[0].norm1, w.W, self.cfg.rms_norm_eps, s.buf.x, s.buf.h)
+        self._embed(s.buf, s.plan)
         K.linear(self._layers(s.buf, s.plan), w.head, out=s.logits)
         V = w.vocab
         K.logits_post(s.logits[:, :V], s.cum[:, :V], None, s.best, s.best_val)

@@ -60,8 +60,8 @@ def main(argv=None) -> int:
     family = family_of_config(read_config(a.model))
     if not torch.cuda.is_available():
         raise RuntimeError("trace replay needs a CUDA device")
-    if family.name == "gunuvik":
-        K.use_decoder_build()
+    if family.sources is not None:
+        K.use_group_build(family.sources)
     engine = make_engine(load_model(a.model, getattr(torch, a.dtype), "cuda"), max_rows=ROWS)
     if not hasattr(engine, "step"):
         raise RuntimeError(f"the engine of family {family.name!r} has no step function for token portions")

@@ -1,4 +1,5 @@
-"""Model families: the Qwen3 backbone of TaH (0.6B / 1.7B / 4B shapes and the tiny test model) and Gunuvik."""
+"""Model families: the Qwen3 backbone of TaH (0.6B / 1.7B / 4B shapes and the tiny test model), Gunuvik and Ditilix."""
+from tah_b200.models.ditilix import DitilixConfig, DitilixForCausalLM, ditilix_preset
 from tah_b200.models.gunuvik import GunuvikConfig, GunuvikForCausalLM, gunuvik_preset
 from tah_b200.models.qwen3 import (PRESETS, LoRASpec, Qwen3Config, Qwen3ForCausalLM, attach_lora,
                                    export_hf_state_dict, from_hf_model, import_hf_state_dict, preset)
@@ -6,4 +7,5 @@ from tah_b200.models.registry import load_model, make_engine, register_family
 
 __all__ = ["PRESETS", "LoRASpec", "Qwen3Config", "Qwen3ForCausalLM", "attach_lora",
            "export_hf_state_dict", "from_hf_model", "import_hf_state_dict", "preset",
+           "DitilixConfig", "DitilixForCausalLM", "ditilix_preset",
            "GunuvikConfig", "GunuvikForCausalLM", "gunuvik_preset", "load_model", "make_engine", "register_family"]

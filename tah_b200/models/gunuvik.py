@@ -15,66 +15,23 @@ all of these values as parameters:
 """
 from __future__ import annotations
 
-import json
 import math
-import os
-from dataclasses import dataclass, field
-from typing import Dict, List, Optional, Tuple
+from dataclasses import dataclass
+from typing import Dict, List, Tuple
 
 import torch
-import torch.nn as nn
+
+from tah_b200.models.layered import (AttentionSpec, LayeredConfig, LayeredForCausalLM, LayerSpec, MLSTMSpec, SwiGLUSpec,
+                                     check_attention)
+
+
+def _attention(**kw) -> AttentionSpec:
+    """An attention spec with the mechanisms every attention layer of the design has."""
+    return AttentionSpec(proj_bias=True, qk_norm=True, sink=True, head_gate=True, **kw)
 
 
 @dataclass
-class AttentionSpec:
-    heads: int
-    kv_heads: int
-    dim: int
-    vdim: int
-    scale: float
-    bias_max: int
-    window: Optional[int] = None          # None: every earlier key
-    keep_first: int = 0
-    kv_from: Optional[int] = None
-    rel_rows: int = 32                    # rows of the distance table (a checkpoint's tensor decides)
-
-    kind = "attention"
-
-
-@dataclass
-class MLSTMSpec:
-    heads: int
-    dim: int
-    vdim: int
-    gate_cap: float
-
-    kind = "mlstm"
-
-
-@dataclass
-class LayerSpec:
-    mixer: object
-    ff: Optional[int]                     # width of the dense feed-forward, None = the layer has none
-
-
-@dataclass
-class GunuvikConfig:
-    vocab_size: int
-    hidden_size: int
-    embedding_scale: float
-    rms_norm_eps: float
-    layers: List[LayerSpec]
-    torch_dtype: str = "bfloat16"
-    raw: Dict = field(default_factory=dict)
-
-    @property
-    def num_hidden_layers(self) -> int:
-        return len(self.layers)
-
-    @property
-    def dtype(self) -> torch.dtype:
-        return getattr(torch, self.torch_dtype)
-
+class GunuvikConfig(LayeredConfig):
     @classmethod
     def from_dict(cls, d: dict) -> "GunuvikConfig":
         layers: List[LayerSpec] = []
@@ -82,18 +39,12 @@ class GunuvikConfig:
             m = e["mixer"]
             if e["type"] == "attention":
                 mask = m.get("mask") or {}
-                mixer = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
-                                      vdim=int(m["vdim"]), scale=float(m["scale"]), bias_max=int(m["bias_max"]),
-                                      window=None if mask.get("size") is None else int(mask["size"]),
-                                      keep_first=int(mask.get("keep_first") or 0),
-                                      kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
-                if mixer.heads % mixer.kv_heads:
-                    raise ValueError(f"layer {i}: {mixer.heads} query heads over {mixer.kv_heads} key/value heads")
-                if mixer.kv_from is not None:
-                    src = layers[mixer.kv_from].mixer if 0 <= mixer.kv_from < i else None
-                    if not isinstance(src, AttentionSpec) or src.kv_from is not None or \
-                            (src.kv_heads, src.dim, src.vdim) != (mixer.kv_heads, mixer.dim, mixer.vdim):
-                        raise ValueError(f"layer {i} cannot use the keys of layer {mixer.kv_from}")
+                mixer = _attention(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                                   vdim=int(m["vdim"]), scale=float(m["scale"]), bias_max=int(m["bias_max"]),
+                                   window=None if mask.get("size") is None else int(mask["size"]),
+                                   keep_first=int(mask.get("keep_first") or 0),
+                                   kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
+                check_attention(i, mixer, layers)
             elif e["type"] == "mlstm":
                 mixer = MLSTMSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))
             else:
@@ -101,14 +52,9 @@ class GunuvikConfig:
             mlp = e.get("mlp")
             if mlp is not None and mlp["kind"] != "dense":
                 raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
-            layers.append(LayerSpec(mixer, None if mlp is None else int(mlp["ff"])))
+            layers.append(LayerSpec(mixer, None if mlp is None else SwiGLUSpec(int(mlp["ff"]))))
         return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), embedding_scale=float(d["embedding"]["scale"]),
                    rms_norm_eps=float(d["norm"]["eps"]), layers=layers, raw=dict(d))
-
-    @classmethod
-    def from_pretrained(cls, path: str) -> "GunuvikConfig":
-        with open(os.path.join(path, "config.json"), encoding="utf-8") as fh:
-            return cls.from_dict(json.load(fh))
 
     def to_dict(self) -> dict:
         layers = []
@@ -122,67 +68,49 @@ class GunuvikConfig:
                     mix["kv_from"] = m.kv_from
             else:
                 mix = dict(heads=m.heads, dim=m.dim, vdim=m.vdim, gate_cap=m.gate_cap)
-            layers.append(dict(type=m.kind, mixer=mix, mlp=None if l.ff is None else dict(kind="dense", ff=l.ff)))
+            layers.append(dict(type=m.kind, mixer=mix, mlp=None if l.ff is None else dict(kind="dense", ff=l.ff.ff)))
         return dict(architecture="Gunuvik", vocab=self.vocab_size, width=self.hidden_size,
                     embedding=dict(scale=self.embedding_scale), norm=dict(eps=self.rms_norm_eps), layers=layers)
 
-
-def tensor_shapes(cfg: GunuvikConfig) -> Dict[str, Tuple[int, ...]]:
-    """On-disk tensor names and shapes of a configuration."""
-    W, V = cfg.hidden_size, cfg.vocab_size
-    out: Dict[str, Tuple[int, ...]] = {"embed": (V, W)}
-    for i, l in enumerate(cfg.layers):
-        p, m = f"l{i}.", l.mixer
-        x = p + "mix."
-        out[p + "norm1"] = out[p + "norm1b"] = out[p + "ls1"] = (W,)
-        if isinstance(m, AttentionSpec):
-            own = [("q", m.heads * m.dim)]
-            if m.kv_from is None:
-                own += [("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)]
-                out[x + "k.norm"] = (m.dim,)
-            for n, rows in own:
-                out[x + n], out[x + n + ".b"] = (rows, W), (rows,)
-            out[x + "q.norm"] = (m.dim,)
-            out[x + "rel"], out[x + "sink"] = (m.rel_rows, m.heads), (m.heads,)
-            out[x + "g"], out[x + "o"] = (m.heads, W), (W, m.heads * m.vdim)
-        else:
-            for n, rows in (("q", m.heads * m.dim), ("k", m.heads * m.dim), ("v", m.heads * m.vdim),
-                            ("g", m.heads * m.vdim), ("i", m.heads), ("f", m.heads)):
-                out[x + n] = (rows, W)
-            out[x + "i.b"] = out[x + "f.b"] = (m.heads,)
-            out[x + "norm"], out[x + "o"] = (m.heads * m.vdim,), (W, m.heads * m.vdim)
-        if l.ff is not None:
-            out[p + "norm2"] = out[p + "norm2b"] = out[p + "ls2"] = (W,)
-            out[p + "mlp.gate"] = out[p + "mlp.up"] = (l.ff, W)
-            out[p + "mlp.down"] = (W, l.ff)
-    out["final.norm"], out["head"] = (W,), (V, W)
-    return out
+    def tensor_shapes(self) -> Dict[str, Tuple[int, ...]]:
+        W, V = self.hidden_size, self.vocab_size
+        out: Dict[str, Tuple[int, ...]] = {"embed": (V, W)}
+        for i, l in enumerate(self.layers):
+            p, m = f"l{i}.", l.mixer
+            x = p + "mix."
+            out[p + "norm1"] = out[p + "norm1b"] = out[p + "ls1"] = (W,)
+            if isinstance(m, AttentionSpec):
+                own = [("q", m.heads * m.dim)]
+                if m.kv_from is None:
+                    own += [("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)]
+                    out[x + "k.norm"] = (m.dim,)
+                for n, rows in own:
+                    out[x + n], out[x + n + ".b"] = (rows, W), (rows,)
+                out[x + "q.norm"] = (m.dim,)
+                out[x + "rel"], out[x + "sink"] = (m.rel_rows, m.heads), (m.heads,)
+                out[x + "g"], out[x + "o"] = (m.heads, W), (W, m.heads * m.vdim)
+            else:
+                for n, rows in (("q", m.heads * m.dim), ("k", m.heads * m.dim), ("v", m.heads * m.vdim),
+                                ("g", m.heads * m.vdim), ("i", m.heads), ("f", m.heads)):
+                    out[x + n] = (rows, W)
+                out[x + "i.b"] = out[x + "f.b"] = (m.heads,)
+                out[x + "norm"], out[x + "o"] = (m.heads * m.vdim,), (W, m.heads * m.vdim)
+            if l.ff is not None:
+                out[p + "norm2"] = out[p + "norm2b"] = out[p + "ls2"] = (W,)
+                out[p + "mlp.gate"] = out[p + "mlp.up"] = (l.ff.ff, W)
+                out[p + "mlp.down"] = (W, l.ff.ff)
+        out["final.norm"], out["head"] = (W,), (V, W)
+        return out
 
 
-class GunuvikForCausalLM(nn.Module):
-    """The weights of a Gunuvik model.  ``tensor(name)`` gives a parameter by its on-disk name."""
+class GunuvikForCausalLM(LayeredForCausalLM):
+    config_class = GunuvikConfig
 
-    def __init__(self, cfg: GunuvikConfig, dtype=None, device=None):
-        super().__init__()
-        self.config = cfg
-        self.weights = nn.ParameterDict()
-        for name, shape in tensor_shapes(cfg).items():
-            self.weights[self._key(name)] = nn.Parameter(torch.zeros(*shape, dtype=dtype or cfg.dtype, device=device))
-
-    @staticmethod
-    def _key(name: str) -> str:
-        return name.replace(".", "/")
-
-    def tensor(self, name: str) -> torch.Tensor:
-        return self.weights[self._key(name)].detach()
-
-    @property
-    def device(self):
-        return self.tensor("embed").device
-
-    @property
-    def dtype(self):
-        return self.tensor("embed").dtype
+    @classmethod
+    def _adapt(cls, cfg, tensors) -> None:
+        for i, l in enumerate(cfg.layers):
+            if isinstance(l.mixer, AttentionSpec):
+                l.mixer.rel_rows = int(tensors[f"l{i}.mix.rel"].shape[0])
 
     @torch.no_grad()
     def init_random(self, seed: int = 0) -> "GunuvikForCausalLM":
@@ -204,40 +132,12 @@ class GunuvikForCausalLM(nn.Module):
                 p.fill_(4.0)
         return self
 
-    # ---- persistence -------------------------------------------------------------------
-    @classmethod
-    def from_pretrained(cls, path: str, dtype=None, device=None) -> "GunuvikForCausalLM":
-        from tah_b200.utils.checkpoint import load_tensors
-        cfg = GunuvikConfig.from_pretrained(path)
-        tensors = load_tensors(path)
-        for i, l in enumerate(cfg.layers):
-            if isinstance(l.mixer, AttentionSpec):
-                l.mixer.rel_rows = int(tensors[f"l{i}.mix.rel"].shape[0])
-        want = tensor_shapes(cfg)
-        missing = [n for n in want if n not in tensors]
-        extra = [n for n in tensors if n not in want]
-        wrong = [n for n in want if n in tensors and tuple(tensors[n].shape) != want[n]]
-        if missing or extra or wrong:
-            raise ValueError(f"checkpoint does not fit its configuration: missing {missing[:4]}, unknown {extra[:4]}, "
-                             f"of another shape {wrong[:4]}")
-        model = cls(cfg, dtype=dtype, device=device)
-        with torch.no_grad():
-            for n, t in tensors.items():
-                model.weights[cls._key(n)].copy_(t)
-        return model
 
-    def save_pretrained(self, path: str, max_shard_bytes: int = 5 * 1024 ** 3) -> None:
-        from tah_b200.utils.checkpoint import save_tensors
-        os.makedirs(path, exist_ok=True)
-        with open(os.path.join(path, "config.json"), "w", encoding="utf-8") as fh:
-            json.dump(self.config.to_dict(), fh, indent=2)
-        save_tensors({n: self.tensor(n) for n in tensor_shapes(self.config)}, path, max_shard_bytes)
-
-
-def _rep(n: int, attn: AttentionSpec, mem: MLSTMSpec, ff: int) -> List[LayerSpec]:
+def _rep(n: int, attn: AttentionSpec, mem: MLSTMSpec, width: int) -> List[LayerSpec]:
     """``n`` groups of four layers: an attention layer with keys of its own, a recurrent one, and two attention layers of
     which the second reads the keys of the first."""
     out: List[LayerSpec] = []
+    ff = SwiGLUSpec(width)
     for _ in range(n):
         base = len(out)
         own = AttentionSpec(**{**attn.__dict__})
@@ -249,12 +149,12 @@ def _rep(n: int, attn: AttentionSpec, mem: MLSTMSpec, ff: int) -> List[LayerSpec
 def gunuvik_preset(name: str) -> GunuvikConfig:
     """Configurations for benchmarks: ``gunuvik-1.7b`` has the layer sizes of the Qwen3-1.7B backbone."""
     if name == "gunuvik-1.7b":
-        attn = AttentionSpec(heads=16, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, bias_max=512, window=1024, keep_first=4)
+        attn = _attention(heads=16, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, bias_max=512, window=1024, keep_first=4)
         return GunuvikConfig(151936, 2048, 1.0, 1e-6, _rep(7, attn, MLSTMSpec(heads=8, dim=128, vdim=256, gate_cap=15.0), 6144))
     if name == "gunuvik-0.6b":
-        attn = AttentionSpec(heads=16, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, bias_max=256, window=512, keep_first=4)
+        attn = _attention(heads=16, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, bias_max=256, window=512, keep_first=4)
         return GunuvikConfig(151936, 1024, 1.0, 1e-6, _rep(7, attn, MLSTMSpec(heads=4, dim=128, vdim=256, gate_cap=15.0), 3072))
     if name == "gunuvik-tiny":
-        attn = AttentionSpec(heads=6, kv_heads=2, dim=40, vdim=24, scale=0.2, bias_max=50, window=21, keep_first=3, rel_rows=14)
+        attn = _attention(heads=6, kv_heads=2, dim=40, vdim=24, scale=0.2, bias_max=50, window=21, keep_first=3, rel_rows=14)
         return GunuvikConfig(300, 160, 3.0, 1e-5, _rep(1, attn, MLSTMSpec(heads=3, dim=24, vdim=40, gate_cap=8.0), 208))
     raise KeyError(name)

@@ -8,7 +8,7 @@ from __future__ import annotations
 import json
 import os
 from dataclasses import dataclass
-from typing import Callable, List
+from typing import Callable, List, Optional
 
 import torch
 
@@ -20,6 +20,7 @@ class Family:
     load: Callable[..., object]                   # (path, dtype, device) -> model
     owns: Callable[[object], bool]                # model instance -> is it this family?
     engine: Callable[..., object]                 # (model, **engine options) -> engine
+    sources: Optional[str] = None                 # kernel source group that suffices to serve it, None = all
 
 
 _FAMILIES: List[Family] = []
@@ -89,14 +90,22 @@ def _gunuvik_load(path, dtype, device):
     return GunuvikForCausalLM.from_pretrained(path, dtype=dtype, device=device)
 
 
-def _gunuvik_owns(model) -> bool:
-    return type(model).__name__ == "GunuvikForCausalLM"
+def _ditilix_load(path, dtype, device):
+    from tah_b200.models.ditilix import DitilixForCausalLM
+    return DitilixForCausalLM.from_pretrained(path, dtype=dtype, device=device)
 
 
-def _gunuvik_engine(model, **kw):
+def _is(class_name: str) -> Callable[[object], bool]:
+    return lambda model: type(model).__name__ == class_name
+
+
+def _hybrid_engine(model, **kw):
     from tah_b200.engine.hybrid import HybridEngine
     return HybridEngine(model, **kw)
 
 
 register_family(Family("qwen3-tah", _qwen3_matches, _qwen3_load, _qwen3_owns, _qwen3_engine))
-register_family(Family("gunuvik", lambda c: c.get("architecture") == "Gunuvik", _gunuvik_load, _gunuvik_owns, _gunuvik_engine))
+register_family(Family("gunuvik", lambda c: c.get("architecture") == "Gunuvik", _gunuvik_load, _is("GunuvikForCausalLM"),
+                       _hybrid_engine, "gunuvik"))
+register_family(Family("ditilix", lambda c: c.get("architecture") == "Ditilix", _ditilix_load, _is("DitilixForCausalLM"),
+                       _hybrid_engine, "ditilix"))

@@ -26,7 +26,8 @@ FLAGS.remove("--use_fast_math")
 
 
 # sources of the smaller libraries that a process may build instead of the whole one
-GROUPS = {"decoder": ("gemm_tcgen05", "elementwise", "sampling", "residual_norm", "attn_window", "mlstm")}
+_DECODER = ("gemm_tcgen05", "elementwise", "sampling", "residual_norm", "attn_window")
+GROUPS = {"gunuvik": _DECODER + ("mlstm",), "ditilix": _DECODER + ("feed_forward",)}
 
 
 def _sources(group=None):

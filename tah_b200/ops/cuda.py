@@ -39,18 +39,18 @@ def lib():
             from tah_b200.ops.build import build
             build()
         _LIB = ctypes.CDLL(_LIB_PATH)
-        if hasattr(_LIB, "tahb_decode_attn_ws_floats"):      # absent from the decoder-only build
+        if hasattr(_LIB, "tahb_decode_attn_ws_floats"):      # absent from the group builds
             _LIB.tahb_decode_attn_ws_floats.restype = c_ll
     return _LIB
 
 
-def use_decoder_build() -> None:
-    """Load the library from the sources that serving a :class:`HybridEngine` needs, compiling only those when the full
-    library is not there (a process that replays a trace or serves such a model; nothing may have been loaded yet)."""
+def use_group_build(group: str) -> None:
+    """Load the library of a source group (:data:`tah_b200.ops.build.GROUPS`), compiling only its sources when the full
+    library is not there (a process that replays a trace of one model; nothing may have been loaded yet)."""
     global _LIB_PATH
     if _LIB is None and not os.path.exists(_LIB_PATH):
         from tah_b200.ops.build import build
-        _LIB_PATH = build(group="decoder")
+        _LIB_PATH = build(group=group)
 
 
 def available() -> bool:
@@ -593,12 +593,33 @@ def swiglu_linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] 
     return out
 
 
-def embed_norm(E, tok, scale: float, w, width: int, eps: float, x, h):
+def embed_norm(E, tok, scale: float, w, width: int, eps: float, x, h, groups: int = 1, pos=None, freq=None):
     """``x = scale * E[tok]`` (fp32 residual stream) and ``h = rms(x) * w`` in the activation type of ``E``.  Rows are
-    padded to ``E.shape[1]`` columns, ``width`` of them real."""
+    padded to ``E.shape[1]`` columns, ``width`` of them real.  ``groups``: parts of the row with a root mean square of
+    their own; ``pos`` / ``freq``: token positions and :func:`sinusoid_frequencies`, adds sinusoidal positions to ``x``."""
     f32 = _act_f32(E, h)
-    _rc(lib().tahb_embed_norm(_p(E), _p(tok), c_float(scale), _p(x), _p(w), _p(h), c_int(tok.shape[0]), c_int(E.shape[0]),
-                              c_int(width), c_int(E.shape[1]), c_float(eps), c_int(f32), _stream()), "tahb_embed_norm")
+    _rc(lib().tahb_embed_norm(_p(E), _p(tok), c_float(scale), _p(pos if freq is not None else None), _p(freq), _p(x), _p(w),
+                              _p(h), c_int(tok.shape[0]), c_int(E.shape[0]), c_int(width), c_int(groups), c_int(E.shape[1]),
+                              c_float(eps), c_int(f32), _stream()), "tahb_embed_norm")
+
+
+def sinusoid_frequencies(width: int, base: float = 10000.0, device=None) -> torch.Tensor:
+    """``[2, (width + 1) // 2]`` fp32: the frequency ``base ** (-2 i / width)`` of the entry pair ``(2 i, 2 i + 1)`` as a
+    high and a low part, so that the kernel can form angles beyond fp32 rounding."""
+    i = torch.arange((width + 1) // 2, dtype=torch.float64)
+    f = base ** (-2.0 * i / width)
+    hi = f.float()
+    return torch.stack([hi, (f - hi.double()).float()]).contiguous().to(device)
+
+
+def residual_add_norm(y, x, mult: float, w_next, width: int, groups: int, eps: float, h, y_ex=None, slot=None):
+    """``x += mult * y`` (fp32, in place) and ``h = rms(x) * w_next`` with ``groups`` parts per row: the seam behind a
+    layer whose mixer and feed-forward run in parallel.  ``y_ex [list rows, ld]`` / ``slot [M, top]``: expert outputs that
+    are gathered and added to ``y``."""
+    f32 = _act_f32(y, h)
+    _rc(lib().tahb_residual_add_norm(_p(y), c_ll(y.stride(0)), _p(y_ex), _p(slot), c_int(0 if slot is None else slot.shape[1]),
+                                     c_float(mult), _p(x), _p(w_next), _p(h), c_int(y.shape[0]), c_int(width), c_int(groups),
+                                     c_int(x.shape[1]), c_float(eps), c_int(f32), _stream()), "tahb_residual_add_norm")
 
 
 def residual_norm(y, x, w_out, w_next, width: int, eps: float, h):
@@ -635,31 +656,36 @@ def kv_append(rows, counts, starts, cache, depth: int, pos, row_of, slot):
 def qkv_post(qkv, bias, q_w, k_w, q_out, cache, slot, nq: int, nkv: int, dk: int, dv: int, dim: int, page_size: int,
              eps: float):
     """Projection bias, per-head RMS norm of q / k, q to ``q_out``, k / v into the paged cache.  ``nkv = 0``: queries
-    only (a layer that reads another layer's keys)."""
+    only (a layer that reads another layer's keys); ``nq = 0``: keys and values only (``qkv`` starts at the keys)."""
     _rc(lib().tahb_qkv_post(_p(qkv), c_ll(qkv.stride(0)), _p(bias), _p(q_w), _p(k_w), _p(q_out), _p(cache), _p(slot),
                             c_int(qkv.shape[0]), c_int(nq), c_int(nkv), c_int(dk), c_int(dv), c_int(dim), c_int(page_size),
-                            c_float(eps), c_int(_act_f32(qkv, q_out)), _stream()), "tahb_qkv_post")
+                            c_float(eps), c_int(_act_f32(qkv, qkv if q_out is None else q_out)), _stream()), "tahb_qkv_post")
 
 
 class _WindowAttn(ctypes.Structure):
     _fields_ = [("q", c_void_p), ("out", c_void_p), ("cache", c_void_p), ("page_table", c_void_p), ("pos", c_void_p),
                 ("row", c_void_p), ("bias", c_void_p), ("sink", c_void_p), ("gate", c_void_p)] + \
                [(n, c_int) for n in ("n", "nq", "nkv", "dk", "dv", "page_size", "max_pages", "window", "keep_first", "far")] + \
-               [("ld_out", c_ll), ("ld_gate", c_ll), ("scale", c_float), ("ws", c_void_p), ("n_split", c_int),
+               [("ld_q", c_ll), ("ld_out", c_ll), ("ld_gate", c_ll), ("scale", c_float), ("softcap", c_float),
+                ("temp_coef", c_float), ("temp_every", ctypes.c_double), ("ws", c_void_p), ("n_split", c_int),
                 ("status", c_void_p)]
 
 
 def window_attn_args(q, out, pool, page_table, pos, row, *, nq: int, nkv: int, dk: int, dv: int, page_size: int,
-                     scale: float, window: int, keep_first: int, bias=None, sink=None, gate=None, n_split: int = 1, ws=None):
-    """Arguments of one windowed attention launch: queries ``q [n, nq * dk]`` at positions ``pos`` of cache rows ``row``
-    over the paged ``pool`` of the layer that owns the keys; see ``csrc/attn_window.cu`` for the rule."""
+                     scale: float, window: int, keep_first: int, bias=None, sink=None, gate=None, softcap=None, q_temp=None,
+                     n_split: int = 1, ws=None):
+    """Arguments of one windowed attention launch: queries ``q [n, nq * dk]`` (any row pitch) at positions ``pos`` of cache
+    rows ``row`` over the paged ``pool`` of the layer that owns the keys; ``softcap``: score cap, ``q_temp = (coef,
+    every)``: query temperature; see ``csrc/attn_window.cu`` for the rule."""
     a = _WindowAttn()
     ptr = lambda t: 0 if t is None else t.data_ptr()
     a.q, a.out, a.cache, a.page_table, a.pos, a.row = (ptr(t) for t in (q, out, pool, page_table, pos, row))
     a.bias, a.sink, a.gate = ptr(bias), ptr(sink), ptr(gate)
     a.n, a.nq, a.nkv, a.dk, a.dv, a.page_size, a.max_pages = q.shape[0], nq, nkv, dk, dv, page_size, page_table.shape[1]
     a.window, a.keep_first, a.far = window, keep_first, 0 if bias is None else bias.shape[1] - 1
-    a.ld_out, a.ld_gate = out.stride(0), 0 if gate is None else gate.stride(0)
+    a.softcap = 0.0 if softcap is None else softcap
+    a.temp_coef, a.temp_every = (0.0, 1.0) if q_temp is None else q_temp
+    a.ld_q, a.ld_out, a.ld_gate = q.stride(0), out.stride(0), 0 if gate is None else gate.stride(0)
     a.scale, a.ws, a.n_split, a.status = scale, ptr(ws), n_split, status_word(q.device).data_ptr()
     return a
 
@@ -685,6 +711,104 @@ def window_attn_tiles(q, out, pool, page_table, pos, row, tile_q0, tile_qn, n_pa
     a = window_attn_args(q, out, pool, page_table, pos, row, **kw)
     _rc(lib().tahb_window_attn_tiles(ctypes.byref(a), _p(tile_q0), _p(tile_qn), c_int(tile_q0.numel()), c_int(n_pages),
                                      _stream()), "tahb_window_attn_tiles")
+    return out
+
+
+# -------------------------------------------------------------------------------------------
+# feed-forward mechanisms (csrc/feed_forward.cu)
+# -------------------------------------------------------------------------------------------
+def poly_norm(z, act, n: int, eps: float, out):
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` of every row, ``act = (a, b, c, e)`` fp32 on the device, ``N`` the division by
+    the root mean square over the first ``n`` columns (the rest is padding)."""
+    _rc(lib().tahb_poly_norm(_p(z), c_ll(z.stride(0)), _p(act), _p(out), c_ll(out.stride(0)), c_int(z.shape[0]), c_int(n),
+                             c_int(z.shape[1]), c_float(eps), c_int(_act_f32(z, out)), _stream()), "tahb_poly_norm")
+    return out
+
+
+def clamped_glu(gu, limit: float, out, in_scale=None, gate=None, lists=None):
+    """``g sigmoid(1.702 g) (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)`` of interleaved columns
+    ``gate_0, up_0, gate_1, ...``.  ``in_scale``: factor of both per row; ``gate``: fp32 column whose sigmoid multiplies
+    the row's result; ``lists``: :class:`ExpertLists` that the rows are those of."""
+    _rc(lib().tahb_clamped_glu(_p(gu), c_ll(gu.stride(0)), _p(out), c_ll(out.stride(0)), c_int(gu.shape[0]), c_int(out.shape[1]),
+                               c_float(limit), _p(in_scale), _p(gate), c_ll(0 if gate is None else gate.stride(0)),
+                               _p(None if lists is None else lists.n_blocks), c_int(0 if lists is None else lists.bn),
+                               c_int(_act_f32(gu, out)), _stream()), "tahb_clamped_glu")
+    return out
+
+
+def expert_block(pairs: int, experts: int, dtype: torch.dtype) -> int:
+    """Rows of a block of the expert lists for ``pairs`` (token, expert) pairs: the token tile of the grouped product."""
+    if dtype == torch.float32:
+        return 64
+    avg = pairs / experts
+    return 16 if avg <= 10 else 32 if avg <= 21 else 64 if avg <= 42 else 128 if avg <= 256 else 256
+
+
+class ExpertLists:
+    """Buffers of a routed pass over ``M`` tokens: the tokens' experts and weights, and the experts' token lists in blocks
+    of ``bn`` rows (``rows`` of them at most, however the router decides)."""
+
+    def __init__(self, M: int, experts: int, top: int, dtype: torch.dtype, device, bn: Optional[int] = None):
+        i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=device)
+        self.M, self.experts, self.top = M, experts, top
+        self.bn = bn or expert_block(M * top, experts, dtype)
+        self.max_blocks = M * top // self.bn + min(experts, M * top)
+        self.rows = self.max_blocks * self.bn
+        self.expert, self.rank, self.slot = i32(M, top), i32(M, top), i32(M, top)
+        self.weight = torch.empty(M, top, dtype=torch.float32, device=device)
+        self.count = torch.zeros(experts + 1, dtype=torch.int32, device=device)
+        self.seg, self.blk_expert, self.n_blocks = i32(experts), i32(self.max_blocks), i32(1)
+        self.row_weight = torch.empty(self.rows, dtype=torch.float32, device=device)
+
+
+def moe_route(z, lists: ExpertLists):
+    """Choose ``lists.top`` experts per row of router logits ``z [M, >= experts]`` (fp32) and build the experts' lists."""
+    L = lists
+    if z.dtype != torch.float32 or z.shape[0] != L.M or z.shape[1] < L.experts:
+        raise ValueError(f"moe_route: logits {z.dtype} {tuple(z.shape)} for {L.M} tokens and {L.experts} experts")
+    _rc(lib().tahb_moe_route(_p(z), c_ll(z.stride(0)), c_int(L.M), c_int(L.experts), c_int(L.top), c_int(L.bn), _p(L.expert),
+                             _p(L.rank), _p(L.weight), _p(L.count), _p(L.seg), _p(L.blk_expert), _p(L.n_blocks),
+                             c_int(L.max_blocks), _p(status_word(z.device)), _stream()), "tahb_moe_route")
+
+
+def moe_gather(h, lists: ExpertLists, out):
+    """Copy the rows of ``h`` into the experts' lists ``out [lists.rows, width]``."""
+    L, es = lists, h.element_size()
+    if out.shape != (L.rows, h.shape[1]) or not out.is_contiguous():
+        raise ValueError(f"moe_gather: list buffer {tuple(out.shape)}, need {(L.rows, h.shape[1])}")
+    _rc(lib().tahb_moe_gather(_p(h), c_int(h.shape[1] * es), c_ll(h.stride(0) * es), c_int(L.M), c_int(L.top), _p(L.expert),
+                              _p(L.rank), _p(L.weight), _p(L.seg), _p(out), _p(L.row_weight), _p(L.slot), c_int(L.rows),
+                              _p(status_word(h.device)), _stream()), "tahb_moe_gather")
+    return out
+
+
+def moe_linear(x, w, lists: ExpertLists, out):
+    """``out[r] = x[r] @ w[expert of r]^T`` for the rows of the experts' lists; ``w [experts, F, K]``."""
+    E, F, Kd = w.shape
+    if not (x.is_contiguous() and w.is_contiguous() and out.is_contiguous()) or x.shape != (lists.rows, Kd) or out.shape != (lists.rows, F):
+        raise ValueError(f"moe_linear: x {tuple(x.shape)} w {tuple(w.shape)} out {tuple(out.shape)}")
+    if _act_f32(x, w, out):
+        _rc(lib().tahb_moe_gemm_f32(_p(w), _p(x), _p(out), c_int(F), c_int(Kd), c_int(lists.rows), _p(lists.blk_expert),
+                                    _p(lists.n_blocks), _stream()), "tahb_moe_gemm_f32")
+    else:
+        _rc(lib().tahb_moe_gemm(_p(w), _p(x), _p(out), c_int(E), c_int(F), c_int(Kd), c_int(lists.rows), c_int(lists.bn),
+                                _p(lists.blk_expert), _p(lists.n_blocks), c_int(0), _p(None), c_float(0.0),
+                                _p(status_word(x.device)), _stream()), "tahb_moe_gemm")
+    return out
+
+
+def moe_glu_linear(x, w, limit: float, lists: ExpertLists, out):
+    """:func:`clamped_glu` of :func:`moe_linear` with interleaved gate / up rows in ``w [experts, 2 F, K]``; every list row's
+    weight multiplies gate and up (the projection of the weighted input).  bf16: one kernel."""
+    E, F2, Kd = w.shape
+    if not (x.is_contiguous() and w.is_contiguous() and out.is_contiguous()) or x.shape != (lists.rows, Kd) or out.shape != (lists.rows, F2 // 2):
+        raise ValueError(f"moe_glu_linear: x {tuple(x.shape)} w {tuple(w.shape)} out {tuple(out.shape)}")
+    if _act_f32(x, w, out):
+        gu = moe_linear(x, w, lists, torch.empty(lists.rows, F2, dtype=torch.float32, device=x.device))
+        return clamped_glu(gu, limit, out, in_scale=lists.row_weight, lists=lists)
+    _rc(lib().tahb_moe_gemm(_p(w), _p(x), _p(out), c_int(E), c_int(F2), c_int(Kd), c_int(lists.rows), c_int(lists.bn),
+                            _p(lists.blk_expert), _p(lists.n_blocks), c_int(1), _p(lists.row_weight), c_float(limit),
+                            _p(status_word(x.device)), _stream()), "tahb_moe_gemm")
     return out
 
 

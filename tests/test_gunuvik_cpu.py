@@ -11,14 +11,14 @@ from tests.oracle import gunuvik_oracle as O
 
 
 def test_config_round_trip_and_shapes(tmp_path):
-    from tah_b200.models.gunuvik import GunuvikConfig, GunuvikForCausalLM, tensor_shapes
+    from tah_b200.models.gunuvik import GunuvikConfig, GunuvikForCausalLM
     for name in H.CONFIGS:
         cfg, sd, d = H.make(os.path.join(str(tmp_path), name), name)
         c = GunuvikConfig.from_pretrained(d)
         for l in c.layers:
             if l.mixer.kind == "attention":
                 l.mixer.rel_rows = cfg["_rel_rows"]
-        assert {k: tuple(v.shape) for k, v in sd.items()} == tensor_shapes(c)
+        assert {k: tuple(v.shape) for k, v in sd.items()} == c.tensor_shapes()
         again = GunuvikConfig.from_dict(c.to_dict())
         for l in again.layers:
             if l.mixer.kind == "attention":
