@@ -1,11 +1,13 @@
-"""Prefill and decode throughput of the hybrid decoder beside the Qwen3 backbone of equal layer sizes, on one GPU.
+"""Prefill and decode throughput of the layered decoders beside the framework's other models of equal layer sizes, on one GPU.
 
     python bench.py --family gunuvik [--model gunuvik-1.7b] [--steps K] [--warmup W]
+    python bench.py --family ditilix [--model ditilix-1.7b|ditilix-moe]
 
-Random weights, random token ids, bf16.  Both models go through their own engines: ``prefill`` on whole prompts and
-decode ticks (CUDA graph) at a given context, reached with ``fast_forward``.  The comparison model is the plain Qwen3
-backbone (one pass per token, no adapter) with the same width, heads, feed-forward and vocabulary; ``*_per_layer``
-divides by the number of layers, because a recurrent layer has no feed-forward of its own.  Device time from CUDA
+Random weights, random token ids, bf16.  All models go through their own engines: ``prefill`` on whole prompts and
+decode ticks (CUDA graph) at a given context, reached with ``fast_forward``.  Comparison models: the plain Qwen3
+backbone (one pass per token, no adapter) with the same width, heads and vocabulary and a feed-forward of 6144, and for
+Ditilix also Gunuvik of that size; ``*_per_layer`` divides by the number of layers, because a recurrent layer has no
+feed-forward of its own.  Device time from CUDA
 events around K calls after W warm-up calls; every call reads the weights (GBs), far more than the 126 MB L2.
 """
 from __future__ import annotations
@@ -17,11 +19,12 @@ PREFILL = ((64, 1024), (8, 8192), (1, 8192))           # prompts x tokens
 DECODE = ((256, 1024), (256, 2304), (32, 2304), (1, 2304))     # rows x context
 
 
-def _qwen3(gcfg, dev):
+def _qwen3(dev):
     import torch
     from tah_b200 import TaHConfig, TaHForCausalLM
     from tah_b200.engine import TaHEngine
-    from tah_b200.models import Qwen3Config, Qwen3ForCausalLM
+    from tah_b200.models import Qwen3Config, Qwen3ForCausalLM, gunuvik_preset
+    gcfg = gunuvik_preset("gunuvik-1.7b")
     a = next(l.mixer for l in gcfg.layers if l.mixer.kind == "attention")
     ff = next(l.ff for l in gcfg.layers if l.ff).ff
     cfg = Qwen3Config(vocab_size=gcfg.vocab_size, hidden_size=gcfg.hidden_size, intermediate_size=ff,
@@ -31,15 +34,16 @@ def _qwen3(gcfg, dev):
         base = Qwen3ForCausalLM(cfg, dtype=torch.bfloat16)
     model = TaHForCausalLM(base, TaHConfig(max_iter=1, iter_decider="IterLabelDecider", adapter_kwargs=dict(r=0),
                                            train_loss="NextTokenPredLoss")).to(dev).eval()
-    return lambda rows: TaHEngine(model, max_rows=rows), model
+    return lambda rows: TaHEngine(model, max_rows=rows), model, cfg
 
 
-def _gunuvik(gcfg, dev):
+def _layered(name, dev):
     import torch
     from tah_b200.engine import HybridEngine
-    from tah_b200.models import GunuvikForCausalLM
-    model = GunuvikForCausalLM(gcfg, dtype=torch.bfloat16, device=dev).init_random()
-    return lambda rows: HybridEngine(model, max_rows=rows), model
+    from tah_b200.models import DitilixForCausalLM, GunuvikForCausalLM, ditilix_preset, gunuvik_preset
+    cls, preset = (DitilixForCausalLM, ditilix_preset) if name.startswith("ditilix") else (GunuvikForCausalLM, gunuvik_preset)
+    model = cls(preset(name), dtype=torch.bfloat16, device=dev).init_random()
+    return lambda rows: HybridEngine(model, max_rows=rows), model, model.config
 
 
 def _prefill_ms(eng, ids, steps, warmup):
@@ -78,21 +82,24 @@ def _tick_ms(eng, rows, ctx, vocab, steps, warmup, dev):
 def run(args):
     import torch
     from bench_clocks import ClockSampler
-    from tah_b200.models import gunuvik_preset
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
-    name = args.model if args.model.startswith("gunuvik") else "gunuvik-1.7b"
-    gcfg = gunuvik_preset(name)
-    V, L = gcfg.vocab_size, len(gcfg.layers)
+    names = [args.model] if args.model.startswith(args.family) else \
+        ["gunuvik-1.7b"] if args.family == "gunuvik" else ["ditilix-1.7b", "ditilix-moe"]
+    builds = [(n, lambda d, n=n: _layered(n, d)) for n in names]
+    if args.family == "ditilix":
+        builds.append(("gunuvik-1.7b", lambda d: _layered("gunuvik-1.7b", d)))
+    builds.append(("qwen3 of the same sizes", _qwen3))
     steps, warmup = max(3, args.steps), max(3, args.warmup)
     sampler = ClockSampler(0)
     sampler.start()
-    out = {"metric": "hybrid decoder prefill / decode, device-timed", "unit": "tokens/s", "n_gpus": 1, "steps": steps,
-           "warmup": warmup, "dtype": "bf16", "data": "synthetic", "impl": "ours", "config": {"model": name, "layers": L},
+    out = {"metric": "layered decoder prefill / decode, device-timed", "unit": "tokens/s", "n_gpus": 1, "steps": steps,
+           "warmup": warmup, "dtype": "bf16", "data": "synthetic", "impl": "ours", "config": {"models": names},
            "models": {}}
-    for label, build in ((name, _gunuvik), ("qwen3 of the same sizes", _qwen3)):
+    for label, build in builds:
         torch.manual_seed(0)
-        make, model = build(gcfg, dev)
+        make, model, cfg = build(dev)
+        V, L = cfg.vocab_size, cfg.num_hidden_layers
         rec = {"parameters": sum(p.numel() for p in model.parameters()), "prefill": {}, "decode": {}}
         for B, T in PREFILL:
             eng = make(B)

@@ -22,12 +22,16 @@
 
 namespace tahb {
 
-// 8 consecutive elements as floats
+// 8 consecutive elements: as they lie in memory (Raw, 16-byte units) and as floats
 template <typename T> struct Vec8;
 template <> struct Vec8<float> {
-  static __device__ __forceinline__ void load(const float* p, float* o) {
-    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-    o[0] = a.x; o[1] = a.y; o[2] = a.z; o[3] = a.w; o[4] = b.x; o[5] = b.y; o[6] = b.z; o[7] = b.w;
+  struct Raw { float4 a, b; };
+  static __device__ __forceinline__ void renew(Raw&) {}
+  static __device__ __forceinline__ Raw raw(const float* p) {
+    return {reinterpret_cast<const float4*>(p)[0], reinterpret_cast<const float4*>(p)[1]};
+  }
+  static __device__ __forceinline__ void unpack(const Raw& r, float* o) {
+    o[0] = r.a.x; o[1] = r.a.y; o[2] = r.a.z; o[3] = r.a.w; o[4] = r.b.x; o[5] = r.b.y; o[6] = r.b.z; o[7] = r.b.w;
   }
   static __device__ __forceinline__ void store(float* p, const float* v) {
     reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
@@ -35,9 +39,12 @@ template <> struct Vec8<float> {
   }
 };
 template <> struct Vec8<__nv_bfloat16> {
-  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* o) {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
-    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+  typedef uint4 Raw;
+  // keeps the compiler from holding the unpacked floats (twice the registers) across the use in between
+  static __device__ __forceinline__ void renew(Raw& r) { asm volatile("" : "+r"(r.x), "+r"(r.y), "+r"(r.z), "+r"(r.w)); }
+  static __device__ __forceinline__ Raw raw(const __nv_bfloat16* p) { return *reinterpret_cast<const uint4*>(p); }
+  static __device__ __forceinline__ void unpack(const Raw& r, float* o) {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&r);
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const float2 f = __bfloat1622float2(h[j]);
@@ -70,16 +77,22 @@ __global__ void __launch_bounds__(PN_THREADS) poly_norm_kernel(const T* __restri
   __shared__ float red[3][PN_THREADS / 32];
   const size_t row = blockIdx.x;
   const int nvec = np / 8;
-  float v[VPT][8];
+  typename Vec8<T>::Raw raw[VPT];
   float s2 = 0.f, s4 = 0.f, s6 = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * PN_THREADS;
+    if (c < nvec) raw[i] = Vec8<T>::raw(z + row * ldz + c * 8);
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * PN_THREADS;
     if (c < nvec) {
-      Vec8<T>::load(z + row * ldz + c * 8, v[i]);
+      float v[8];
+      Vec8<T>::unpack(raw[i], v);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
-        const float q = v[i][e] * v[i][e], q2 = q * q;
+        const float q = v[e] * v[e], q2 = q * q;
         s2 += q;
         s4 += q2;
         s6 = fmaf(q2, q, s6);
@@ -104,9 +117,12 @@ __global__ void __launch_bounds__(PN_THREADS) poly_norm_kernel(const T* __restri
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * PN_THREADS;
     if (c < nvec) {
+      float v[8];
+      Vec8<T>::renew(raw[i]);
+      Vec8<T>::unpack(raw[i], v);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) v[i][e] = fmaf(v[i][e], fmaf(v[i][e], fmaf(v[i][e], k[2], k[1]), k[0]), e0);
-      Vec8<T>::store(out + row * ldo + c * 8, v[i]);
+      for (int e = 0; e < 8; ++e) v[e] = fmaf(v[e], fmaf(v[e], fmaf(v[e], k[2], k[1]), k[0]), e0);
+      Vec8<T>::store(out + row * ldo + c * 8, v);
     }
   }
 }
@@ -131,22 +147,23 @@ template <typename T>
 __global__ void __launch_bounds__(256) clamped_glu_kernel(const GluParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const long long rows = p.n_blocks != nullptr ? min((long long)p.rows, (long long)*p.n_blocks * p.bn) : p.rows;
-  const int nv = p.width / 8;
-  const long long n = rows * nv;
-  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
-    const long long r = i / nv;
+  const unsigned rows = p.n_blocks != nullptr ? min((long long)p.rows, (long long)*p.n_blocks * p.bn) : p.rows;
+  const unsigned nv = p.width / 8, n = rows * nv;              // the host checks that rows * nv fits
+  for (unsigned i = blockIdx.x * 256u + threadIdx.x; i < n; i += gridDim.x * 256u) {
+    const size_t r = i / nv;
     const int c = (int)(i % nv) * 8;
     float v[16], o[8];
     const T* src = reinterpret_cast<const T*>(p.in) + r * p.ld_in + 2 * c;
-    Vec8<T>::load(src, v);
-    Vec8<T>::load(src + 8, v + 8);
+    const typename Vec8<T>::Raw lo = Vec8<T>::raw(src), hi = Vec8<T>::raw(src + 8);
+    Vec8<T>::unpack(lo, v);
+    Vec8<T>::unpack(hi, v + 8);
     const float w = p.in_scale != nullptr ? p.in_scale[r] : 1.0f;
     const float f = p.gate != nullptr ? 1.0f / (1.0f + expf(-p.gate[r * p.ld_gate])) : 1.0f;
+    constexpr bool fast = sizeof(T) == 2;       // the result is rounded to 16 bits: approximate exponential and division do
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       const float g = fminf(w * v[2 * e], p.limit), u = fminf(fmaxf(w * v[2 * e + 1], -p.limit), p.limit);
-      o[e] = g / (1.0f + expf(-1.702f * g)) * (u + 1.0f) * f;
+      o[e] = (fast ? __fdividef(g, 1.0f + __expf(-1.702f * g)) : g / (1.0f + expf(-1.702f * g))) * (u + 1.0f) * f;
     }
     Vec8<T>::store(reinterpret_cast<T*>(p.out) + r * p.ld_out + c, o);
   }
@@ -573,9 +590,10 @@ extern "C" int tahb_clamped_glu(const void* in, long long ld_in, void* out, long
                                 int f32, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (width % 8 || ld_in % 8 || ld_out % 8 || ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) & 15)) return -1;
+  if ((long long)rows * (width / 8) > 0x7fffffffll) return -2;
   GluParams p{in, out, ld_in, ld_out, rows, width, limit, in_scale, gate, ld_gate, n_blocks, bn};
   long long blocks = ((long long)rows * (width / 8) + 255) / 256;
-  if (blocks > 148 * 16) blocks = 148 * 16;
+  if (blocks > 148 * 32) blocks = 148 * 32;
   const cudaError_t e = f32 ? launch_chain(clamped_glu_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, p)
                             : launch_chain(clamped_glu_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream, p);
   return e == cudaSuccess ? 0 : -3;

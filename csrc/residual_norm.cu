@@ -111,13 +111,13 @@ static size_t group_rms_smem(int width, int groups, int ld) {
   return (64 + (size_t)groups + ((width / groups) % 128 ? ld : 0)) * 4;
 }
 
-// Sine and cosine of p * f for the pair of entries (2 i, 2 i + 1); f = hi + lo keeps the angle's rounding error out of the
-// result at large positions.
+// Sine and cosine of p * f for the pair of entries (2 i, 2 i + 1); f = hi + lo, and the rounding error e of the angle (4e-3 at
+// position 70,000) goes into the result by the Taylor terms up to e^2.
 __device__ __forceinline__ float2 sin_cos_pair(float p, float hi, float lo) {
   const float a = p * hi, e = fmaf(p, lo, fmaf(p, hi, -a));
   float s, c;
   sincosf(a, &s, &c);
-  return make_float2(fmaf(e, c, s), fmaf(-e, s, c));
+  return make_float2(fmaf(e, fmaf(-0.5f * e, s, c), s), fmaf(-e, fmaf(0.5f * e, c, s), c));
 }
 
 // pos / freq: position of every token and [2, (width + 1) / 2] frequencies (high parts, then low parts), or null

@@ -741,7 +741,7 @@ def expert_block(pairs: int, experts: int, dtype: torch.dtype) -> int:
     if dtype == torch.float32:
         return 64
     avg = pairs / experts
-    return 16 if avg <= 10 else 32 if avg <= 21 else 64 if avg <= 42 else 128 if avg <= 256 else 256
+    return 16 if avg <= 10 else 32 if avg <= 21 else 64 if avg <= 42 else 128 if avg <= 192 else 256
 
 
 class ExpertLists:

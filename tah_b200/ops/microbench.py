@@ -421,6 +421,9 @@ def main(argv=None):
     ap.add_argument("--dv", type=int, default=256, help="mLSTM value size (heads: --nkv, q/k size: --hd)")
     ap.add_argument("--window", type=int, default=1024, help="windowed attention: window (0 = plain causal)")
     ap.add_argument("--keep", type=int, default=4, help="windowed attention: kept first tokens")
+    ap.add_argument("--softcap", type=float, default=0.0, help="windowed attention: score cap and query temperature instead of "
+                                                               "bias, sink and gate")
+    ap.add_argument("--experts", type=int, default=0, help="routed experts (--topk per token, --f wide, hidden size --k)")
     ap.add_argument("--v", type=int, default=151936)
     ap.add_argument("--topk", type=int, default=100)
     ap.add_argument("--iters", type=int, default=20)

@@ -1,5 +1,5 @@
-"""Micro-benchmark cases of the hybrid decoder's kernels (windowed attention, mLSTM, fp32-residual norms); run through
-:mod:`tah_b200.ops.microbench`, whose timing rules and flags apply.
+"""Micro-benchmark cases of the layered decoders' kernels (windowed attention, mLSTM, fp32-residual norms, PolyNorm, routed
+experts); run through :mod:`tah_b200.ops.microbench`, whose timing rules and flags apply.
 
 FLOPs and bytes are those of the algorithm: visible (query, key) pairs for attention, for the chunkwise mLSTM one
 128-token causal block plus the state read-out and update per chunk with every product counted once.
@@ -28,9 +28,11 @@ def _paged(rows, ctx, nkv, dk, dv):
 
 def _window_kw(a):
     far = min(a.ctx, 512)
-    return dict(nq=a.nq, nkv=a.nkv, dk=a.hd, dv=a.hd, page_size=16, scale=a.hd ** -0.5, window=a.window or 2 ** 31 - 1,
-                keep_first=a.keep if a.window else 0, bias=torch.randn(a.nq, far + 1, device="cuda"),
-                sink=torch.randn(a.nq, device="cuda"))
+    kw = dict(nq=a.nq, nkv=a.nkv, dk=a.hd, dv=a.hd, page_size=16, scale=a.hd ** -0.5, window=a.window or 2 ** 31 - 1,
+              keep_first=a.keep if a.window else 0)
+    if a.softcap:
+        return dict(kw, softcap=a.softcap, q_temp=(0.1, 2048))
+    return dict(kw, bias=torch.randn(a.nq, far + 1, device="cuda"), sink=torch.randn(a.nq, device="cuda"))
 
 
 def _visible(i, a):
@@ -41,7 +43,7 @@ def bench_window_prefill(a):
     B, T = a.rows, a.ctx
     n = B * T
     pool, pt = _paged(B, T, a.nkv, a.hd, a.hd)
-    q, out, gate = _bf(n, a.nq * a.hd), torch.empty(n, a.nq * a.hd, dtype=torch.bfloat16, device="cuda"), _bf(n, a.nq)
+    q, out, gate = _bf(n, a.nq * a.hd), torch.empty(n, a.nq * a.hd, dtype=torch.bfloat16, device="cuda"), None if a.softcap else _bf(n, a.nq)
     pos = torch.arange(T, device="cuda", dtype=torch.int32).repeat(B)
     row = torch.arange(B, device="cuda", dtype=torch.int32).repeat_interleave(T)
     q0 = [b * T + t for b in range(B) for t in range(0, T, 128)]
@@ -57,7 +59,7 @@ def bench_window_decode(a):
     from tah_b200.engine.hybrid import decode_splits
     B, T = a.rows, a.ctx
     pool, pt = _paged(B, T, a.nkv, a.hd, a.hd)
-    q, out, gate = _bf(B, a.nq * a.hd), torch.empty(B, a.nq * a.hd, dtype=torch.bfloat16, device="cuda"), _bf(B, a.nq)
+    q, out, gate = _bf(B, a.nq * a.hd), torch.empty(B, a.nq * a.hd, dtype=torch.bfloat16, device="cuda"), None if a.softcap else _bf(B, a.nq)
     pos, row, kw = _i32([T - 1] * B), _i32(list(range(B))), _window_kw(a)
     ws = torch.empty(B * a.nq * a.nsplit * (a.hd + 2), device="cuda")
     fn = lambda i: K.window_attn_decode(q, out, pool, pt, pos, row, gate=gate, n_split=a.nsplit, ws=ws, **kw)
@@ -138,6 +140,80 @@ def bench_few_linear(a):
     return {"op": "few_linear", "M": M, "K": W, "F": F}, fn, 2.0 * M * W * F, (M * W + F * W) * 2 + M * F * 4
 
 
+def bench_residual_add_norm(a):
+    """``--topk`` expert rows per token when ``--experts`` is given."""
+    M, W, top = a.m, a.k, a.topk if a.experts else 0
+    y, x, h = _bf(M, W), torch.randn(M, W, device="cuda"), torch.empty(M, W, dtype=torch.bfloat16, device="cuda")
+    w = torch.full((W,), 0.5, device="cuda")
+    ex = _bf(M * top, W) if top else None
+    slot = torch.randperm(M * top, device="cuda").to(torch.int32).view(M, top) if top else None
+    fn = lambda i: K.residual_add_norm(y, x, 0.5, w, W, 4, 1e-6, h, ex, slot)
+    return {"op": "residual_add_norm", "M": M, "W": W, "experts": top}, fn, 0.0, M * W * (2 + 8 + 2 + 2 * top)
+
+
+def bench_poly_norm(a):
+    M, F = a.m, a.f
+    z, out, act = _bf(M, F), torch.empty(M, F, dtype=torch.bfloat16, device="cuda"), torch.tensor([0.6, -0.4, 0.3, 0.1], device="cuda")
+    fn = lambda i: K.poly_norm(z, act, F, 1e-6, out)
+    return {"op": "poly_norm", "M": M, "F": F}, fn, 0.0, M * F * 4
+
+
+def bench_swiglu(a):
+    """The like kernel of the training path: an activation over rows in a launch of its own."""
+    M, F = a.m, a.f
+    z, out = _bf(M, 2 * F), torch.empty(M, F, dtype=torch.bfloat16, device="cuda")
+    return {"op": "swiglu", "M": M, "F": F}, lambda i: K.swiglu(z, out=out), 0.0, M * F * 6
+
+
+def bench_clamped_glu(a):
+    M, F = a.m, a.f
+    z, out, gate = _bf(M, 2 * F), torch.empty(M, F, dtype=torch.bfloat16, device="cuda"), torch.randn(M, 8, device="cuda")
+    fn = lambda i: K.clamped_glu(z, 7.0, out, gate=gate[:, 3])
+    return {"op": "clamped_glu", "M": M, "F": F}, fn, 0.0, M * F * 6
+
+
+def _lists(a):
+    L = K.ExpertLists(a.m, a.experts, a.topk, torch.bfloat16, "cuda", bn=a.bn or None)
+    z = torch.randn(a.m, a.experts + 1, device="cuda")
+    K.moe_route(z, L)
+    return L, z
+
+
+def bench_moe_route(a):
+    L, z = _lists(a)
+    return {"op": "moe_route", "M": a.m, "experts": a.experts, "top": a.topk}, lambda i: K.moe_route(z, L), 0.0, \
+        a.m * (4 * a.experts + 12 * a.topk)
+
+
+def bench_moe_gather(a):
+    L, _ = _lists(a)
+    h, x = _bf(a.m, a.k), torch.empty(L.rows, a.k, dtype=torch.bfloat16, device="cuda")
+    return {"op": "moe_gather", "M": a.m, "top": a.topk}, lambda i: K.moe_gather(h, L, x), 0.0, a.m * a.k * 2 * (1 + a.topk)
+
+
+def _moe(a, glu):
+    """FLOPs of the (token, expert) pairs; bytes: weights of the experts in use, list rows in and out."""
+    L, _ = _lists(a)
+    K.moe_gather(_bf(a.m, 64), L, torch.empty(L.rows, 64, dtype=torch.bfloat16, device="cuda"))
+    Kd, F = (a.k, 2 * a.f) if glu else (a.f, a.k)
+    x, w = _bf(L.rows, Kd), _bf(a.experts, F, Kd)
+    out = torch.empty(L.rows, a.f if glu else a.k, dtype=torch.bfloat16, device="cuda")
+    fn = (lambda i: K.moe_glu_linear(x, w, 7.0, L, out)) if glu else (lambda i: K.moe_linear(x, w, L, out))
+    pairs, used = a.m * a.topk, int(L.expert.unique().numel())
+    return {"op": "moe_glu" if glu else "moe_down", "M": a.m, "experts": a.experts, "top": a.topk, "bn": L.bn,
+            "rows": int(L.n_blocks) * L.bn}, fn, 2.0 * pairs * F * Kd, used * F * Kd * 2 + pairs * (Kd + out.shape[1]) * 2
+
+
+def bench_moe_glu(a):
+    return _moe(a, True)
+
+
+def bench_moe_down(a):
+    return _moe(a, False)
+
+
 CASES = {"window_prefill": bench_window_prefill, "window_decode": bench_window_decode, "mlstm_chunks": bench_mlstm_chunks,
          "mlstm_step": bench_mlstm_step, "residual_norm": bench_residual_norm, "qkv_post": bench_qkv_post,
-         "qk_norm_rope": bench_qk_norm_rope, "few_linear": bench_few_linear}
+         "qk_norm_rope": bench_qk_norm_rope, "few_linear": bench_few_linear, "residual_add_norm": bench_residual_add_norm,
+         "poly_norm": bench_poly_norm, "clamped_glu": bench_clamped_glu, "swiglu": bench_swiglu, "moe_route": bench_moe_route,
+         "moe_gather": bench_moe_gather, "moe_glu": bench_moe_glu, "moe_down": bench_moe_down}

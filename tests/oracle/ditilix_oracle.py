@@ -127,19 +127,37 @@ def forward(cfg, sd, tokens, dtype=torch.float64, layers_out=None):
 
 
 def random_model(cfg, seed=0, dtype=torch.bfloat16):
-    """Random weights under the on-disk names and shapes for ``cfg``, spread so that leaving a mechanism out shows."""
+    """Random weights under the on-disk names and shapes for ``cfg``, spread so that leaving a mechanism out shows.
+
+    Routing has no close calls: the first ``experts`` coordinates of an embedding are flags, ``top`` of them high, that no
+    layer writes to; a router row reads one flag (which one differs by layer) and a little of everything else.  The mixtures
+    of a model must therefore agree on ``experts`` and ``top``."""
     g = torch.Generator().manual_seed(seed)
     rnd = lambda *s: torch.randn(*s, generator=g, dtype=torch.float64)
     W, V = cfg["width"], cfg["vocab"]
     lin = lambda o, i, f=1.0: f * rnd(o, i) / math.sqrt(i)
     near1 = lambda *s: 1.0 + 0.2 * rnd(*s)
-    sd = {"embed": rnd(V, W), "final.norm": near1(W), "head": lin(V, W)}
+    moe = [l["mlp"] for l in cfg["layers"] if l["mlp"] is not None and l["mlp"]["kind"] == "moe"]
+    E, top = (moe[0]["router"]["experts"], moe[0]["router"]["top"]) if moe else (0, 0)
+    if any((m["router"]["experts"], m["router"]["top"]) != (E, top) for m in moe):
+        raise ValueError("mixtures of different router sizes")
+
+    def back(cols, f=1.0):                       # a projection back to the residual stream
+        w = lin(W, cols, f)
+        w[:E] = 0.0
+        return w
+
+    embed = rnd(V, W)
+    for t in range(V):
+        embed[t, :E] = -4.0
+        embed[t, torch.randperm(E, generator=g)[:top]] = 4.0
+    sd = {"embed": embed, "final.norm": near1(W), "head": lin(V, W)}
     for li, layer in enumerate(cfg["layers"]):
         p, mix, mlp = f"l{li}.", layer["mixer"], layer["mlp"]
         H, G, dk, dv = mix["heads"], mix["kv_heads"], mix["dim"], mix["vdim"]
         sd[p + "norm1"] = near1(W)
         m = p + "mix."
-        sd[m + "q"], sd[m + "o"] = lin(H * dk, W, 1.5), lin(W, H * dv)
+        sd[m + "q"], sd[m + "o"] = lin(H * dk, W, 1.5), back(H * dv, 2.0)
         if mix.get("kv_from") is None:
             sd[m + "k"], sd[m + "v"] = lin(G * dk, W, 1.5), lin(G * dv, W)
         if mlp is None:
@@ -147,14 +165,35 @@ def random_model(cfg, seed=0, dtype=torch.bfloat16):
         m = p + "mlp."
         if mlp["kind"] == "dense":
             F = mlp["ff"]
-            sd[m + "up"], sd[m + "down"] = lin(F, W), lin(W, F)
+            sd[m + "up"], sd[m + "down"] = lin(F, W), back(F)
             sd[m + "act"] = torch.tensor([0.6, -0.5, 0.4, 0.1], dtype=torch.float64) * near1(4)
             continue
-        ex = [(f"{m}e{i}.", mlp["expert"]["ff"]) for i in range(mlp["router"]["experts"])]
+        ex = [(f"{m}e{i}.", mlp["expert"]["ff"]) for i in range(E)]
         if mlp.get("shared"):
             ex.append((m + "shared.", mlp["shared"]["ff"]))
             sd[m + "shared.sg"] = lin(1, W)
         for e, F in ex:
-            sd[e + "gate"], sd[e + "up"], sd[e + "down"] = lin(F, W, 1.5), lin(F, W, 1.5), lin(W, F)
-        sd[m + "router"] = lin(mlp["router"]["experts"], W, 1.5)
+            sd[e + "gate"], sd[e + "up"], sd[e + "down"] = lin(F, W, 1.5), lin(F, W, 1.5), back(F)
+        sd[p + "norm1"][:E] = 1.0
+        router = lin(E, W, 0.2)
+        router[:, :E] = 0.5 * torch.eye(E, dtype=torch.float64)[torch.randperm(E, generator=g)]
+        sd[m + "router"] = router
     return {k: v.to(dtype) for k, v in sd.items()}
+
+
+def router_margin(cfg, sd, tokens):
+    """Smallest distance in router logits between a chosen and a passed-over expert, over all tokens and mixtures."""
+    low = [math.inf]
+    keep = globals()["route"]
+
+    def watch(h, router, top):
+        z = (h @ router.T).sort(-1, descending=True).values
+        if z.shape[1] > top:
+            low[0] = min(low[0], float((z[:, top - 1] - z[:, top]).min()))
+        return keep(h, router, top)
+    globals()["route"] = watch
+    try:
+        forward(cfg, sd, tokens)
+    finally:
+        globals()["route"] = keep
+    return low[0]
