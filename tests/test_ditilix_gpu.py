@@ -252,6 +252,16 @@ def test_router_and_expert_lists(M, E, top, skew):
     check_ok()
 
 
+@pytest.mark.parametrize("M,F", [(5, 65), (2048, 65), (3001, 130), (2500, 33)])
+def test_router_logits(M, F):
+    from tah_b200.ops import cuda as K
+    g = torch.Generator().manual_seed(0)
+    x, w = torch.randn(M, 192, generator=g).to(BF16), torch.randn(F, 192, generator=g).to(BF16)
+    got = K.few_linear(x.cuda(), w.cuda(), None).cpu().double()
+    assert float((got - x.double() @ w.double().T).abs().max()) < 1e-4
+    check_ok()
+
+
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("M,E,top,width,ff,bn", [(3, 5, 2, 128, 64, 16), (40, 3, 1, 192, 128, 32), (150, 9, 2, 64, 192, 64), (700, 4, 2, 320, 64, 128),
                                                  (900, 2, 1, 128, 320, 256), (2500, 7, 3, 256, 128, None), (1, 300, 4, 64, 64, None)])
