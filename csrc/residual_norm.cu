@@ -309,65 +309,55 @@ __global__ void __launch_bounds__(FL_THREADS) few_linear_kernel(const T* __restr
   }
 }
 
-// bf16 operands: far too few features for a tcgen05 tile, so warp-level m16n8k16 products with fp32 sums.  A CTA owns 16 MT
-// tokens and up to 8 NT features; its 8 warps split K.  A lane fetches 8 consecutive k of its rows with one 16-byte load:
-// which k sit in which register slot does not matter as long as x and w agree.  Every CTA reads the weights of its features,
-// so more tokens per CTA pay off for wider outputs (a router's).
-template <int MT, int NT>
+// bf16 operands: far too few features for a tcgen05 tile, so warp-level m16n8k16 products with fp32 sums.  A CTA owns 16
+// tokens and up to 32 features; its 8 warps split K.  A lane fetches 8 consecutive k of its rows with one 16-byte load:
+// which k sit in which register slot does not matter as long as x and w agree.
+constexpr int FLM_NT = 4;                  // feature tiles of 8 per CTA
 __global__ void __launch_bounds__(FL_THREADS) few_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, long long ldx,
                                                                     const __nv_bfloat16* __restrict__ w,
                                                                     const float* __restrict__ b, float* __restrict__ out,
                                                                     int M, int K, int F) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float part[FL_THREADS / 32][16 * MT][NT * 8 + 1];
+  __shared__ float part[FL_THREADS / 32][16][FLM_NT * 8 + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
-  const int t0 = blockIdx.x * 16 * MT, f0 = blockIdx.y * NT * 8;
-  const int nt = min(NT, (F - f0 + 7) / 8);
-  const __nv_bfloat16* xr[2 * MT];
+  const int t0 = blockIdx.x * 16, f0 = blockIdx.y * FLM_NT * 8;
+  const int nt = min(FLM_NT, (F - f0 + 7) / 8);
+  const __nv_bfloat16* x0 = x + (size_t)min(t0 + g, M - 1) * ldx + q * 8;
+  const __nv_bfloat16* x1 = x + (size_t)min(t0 + g + 8, M - 1) * ldx + q * 8;
+  const __nv_bfloat16* wr[FLM_NT];
+  float acc[FLM_NT][4];
 #pragma unroll
-  for (int i = 0; i < 2 * MT; ++i) xr[i] = x + (size_t)min(t0 + g + 8 * i, M - 1) * ldx + q * 8;
-  const __nv_bfloat16* wr[NT];
-  float acc[MT][NT][4];
-#pragma unroll
-  for (int j = 0; j < NT; ++j) {
+  for (int j = 0; j < FLM_NT; ++j) {
     wr[j] = w + (size_t)min(f0 + j * 8 + g, F - 1) * K + q * 8;
 #pragma unroll
-    for (int i = 0; i < MT; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
+    for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
   }
-#pragma unroll (MT == 1 ? 4 : 2)
+#pragma unroll 4
   for (int k = warp * 32; k < K; k += FL_THREADS) {
-    uint4 a[2 * MT];
+    const uint4 a = *reinterpret_cast<const uint4*>(x0 + k), c = *reinterpret_cast<const uint4*>(x1 + k);
 #pragma unroll
-    for (int i = 0; i < 2 * MT; ++i) a[i] = *reinterpret_cast<const uint4*>(xr[i] + k);
-#pragma unroll
-    for (int j = 0; j < NT; ++j) {
+    for (int j = 0; j < FLM_NT; ++j) {
       if (j < nt) {
         const uint4 v = *reinterpret_cast<const uint4*>(wr[j] + k);
-#pragma unroll
-        for (int i = 0; i < MT; ++i) {
-          float* d = acc[i][j];
-          const uint4 lo = a[2 * i], hi = a[2 * i + 1];
-          asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                       : "r"(lo.x), "r"(hi.x), "r"(lo.y), "r"(hi.y), "r"(v.x), "r"(v.y));
-          asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                       : "r"(lo.z), "r"(hi.z), "r"(lo.w), "r"(hi.w), "r"(v.z), "r"(v.w));
-        }
+        asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                     : "+f"(acc[j][0]), "+f"(acc[j][1]), "+f"(acc[j][2]), "+f"(acc[j][3])
+                     : "r"(a.x), "r"(c.x), "r"(a.y), "r"(c.y), "r"(v.x), "r"(v.y));
+        asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                     : "+f"(acc[j][0]), "+f"(acc[j][1]), "+f"(acc[j][2]), "+f"(acc[j][3])
+                     : "r"(a.z), "r"(c.z), "r"(a.w), "r"(c.w), "r"(v.z), "r"(v.w));
       }
     }
   }
 #pragma unroll
-  for (int i = 0; i < MT; ++i)
-#pragma unroll
-    for (int j = 0; j < NT; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) part[warp][16 * i + g + 8 * (e >> 1)][j * 8 + q * 2 + (e & 1)] = acc[i][j][e];
+  for (int j = 0; j < FLM_NT; ++j) {
+    part[warp][g][j * 8 + q * 2] = acc[j][0];
+    part[warp][g][j * 8 + q * 2 + 1] = acc[j][1];
+    part[warp][g + 8][j * 8 + q * 2] = acc[j][2];
+    part[warp][g + 8][j * 8 + q * 2 + 1] = acc[j][3];
+  }
   __syncthreads();
-  for (int i = threadIdx.x; i < 16 * MT * nt * 8; i += FL_THREADS) {
+  for (int i = threadIdx.x; i < 16 * nt * 8; i += FL_THREADS) {
     const int r = i / (nt * 8), f = i % (nt * 8);
     float s = 0.f;
 #pragma unroll
@@ -548,12 +538,9 @@ extern "C" int tahb_few_linear(const void* x, long long ldx, const void* w, cons
     return one ? few_linear_launch<float, 1>(x, ldx, w, b, out, M, K, F, stream)
                : few_linear_launch<float, 4>(x, ldx, w, b, out, M, K, F, stream);
   if (K % 32 || ldx % 8) return -1;
-  auto xb = reinterpret_cast<const __nv_bfloat16*>(x);
-  auto wb = reinterpret_cast<const __nv_bfloat16*>(w);
-  const bool wide = F > 32 && M >= 2048;
-  const dim3 grid(wide ? (M + 31) / 32 : (M + 15) / 16, wide ? (F + 39) / 40 : (F + 31) / 32);
-  cudaError_t rc = wide ? launch_chain(few_linear_mma_kernel<2, 5>, grid, dim3(FL_THREADS), 0, stream, xb, ldx, wb, b, out, M, K, F)
-                        : launch_chain(few_linear_mma_kernel<1, 4>, grid, dim3(FL_THREADS), 0, stream, xb, ldx, wb, b, out, M, K, F);
+  const dim3 grid((M + 15) / 16, (F + FLM_NT * 8 - 1) / (FLM_NT * 8));
+  cudaError_t rc = launch_chain(few_linear_mma_kernel, grid, dim3(FL_THREADS), 0, stream, reinterpret_cast<const __nv_bfloat16*>(x),
+                                ldx, reinterpret_cast<const __nv_bfloat16*>(w), b, out, M, K, F);
   return rc == cudaSuccess ? 0 : -3;
 }
 
