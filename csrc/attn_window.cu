@@ -1,5 +1,5 @@
 // Paged attention with a sliding window, kept first tokens, a query temperature, a score cap, a per-distance bias, a
-// softmax sink and a per-head output gate.
+// softmax sink and an output gate per head (or, for portions, per element).
 //
 // Query at position i of a sequence sees key j when  j <= i  and  (i - j < window  or  j < keep_first).
 // score = cap(temp(i) * (q . k) * scale) + bias[h][min(i - j, D)] with cap(s) = softcap * tanh(s / softcap) and
@@ -101,8 +101,11 @@ __global__ void __launch_bounds__(256) kv_append_kernel(const int* __restrict__ 
 }
 
 // ---------------------------------------------------------------------------------------------
-// After the fused projection [q | k | v | ...]: bias, per-head RMS norm of q and k, q to its own matrix, k and v to the
-// paged cache.  One warp per (token, head); a lane owns dim pairs 2 * lane, 2 * lane + 64, ...
+// After the fused projection [q | k | v | ...]: bias, per-head RMS norm of q and k, rotation of their first `rot` dims, values
+// mixed with those of an earlier layer, q to its own matrix, k and v to the paged cache.  One warp per (token, head); a lane
+// owns dim pairs 2 * lane, 2 * lane + 64, ...
+//   rotation: entries (a, b) of the pair i become (a cos - b sin, b cos + a sin), pairs (i, i + rot / 2) or (2 i, 2 i + 1)
+//   values:   v <- (1 - lambda) v + lambda v_first; without v_first the values are copied to v_keep, for the layers that mix
 // ---------------------------------------------------------------------------------------------
 struct QkvPostParams {
   const void* qkv;            // [M, ld]: nq heads of dk, then nkv heads of dk, then nkv heads of dv
@@ -115,6 +118,11 @@ struct QkvPostParams {
   int M, nq, nkv, dk, dv, dim, page_size;     // dim = real (unpadded) size of a q / k head
   long long ld;
   float eps;
+  const float2* rope;         // [M, rot / 2] (cos, sin), or null
+  int rot, interleaved;
+  const void* v_first;        // [M, nkv * dv] or null
+  const float* lambda;        // [1], with v_first
+  void* v_keep;               // [M, nkv * dv] or null
 };
 
 template <typename T>
@@ -148,14 +156,63 @@ __global__ void __launch_bounds__(128) qkv_post_kernel(const QkvPostParams p) {
     }
   }
   const float* w = is_q ? p.q_w : is_k ? p.k_w : nullptr;
+  float r = 1.0f;
   if (w != nullptr) {
-    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+    r = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
 #pragma unroll
     for (int i = 0; i < MAXP; ++i) {
       const int c = 2 * lane + 64 * i;
       if (c < d) {
         x[2 * i] *= r * w[c];
         x[2 * i + 1] *= r * w[c + 1];
+      }
+    }
+  }
+  if (p.rope != nullptr && (is_q || is_k)) {
+    const float2* tab = p.rope + (size_t)t * (p.rot / 2);
+    const int half = p.rot / 2;
+    auto entry = [&](int c) {                   // entry c of the head behind bias and norm (held by another lane)
+      float v = to_f<T>(src[c]);
+      if (p.bias != nullptr) v += p.bias[col + c];
+      return w != nullptr ? v * r * w[c] : v;
+    };
+#pragma unroll
+    for (int i = 0; i < MAXP; ++i) {
+      const int c = 2 * lane + 64 * i;
+      if (c >= p.rot) continue;
+      if (p.interleaved) {                      // rot is even: the pair lies in this lane
+        const float2 f = tab[c / 2];
+        const float a = x[2 * i], b = x[2 * i + 1];
+        x[2 * i] = a * f.x - b * f.y;
+        x[2 * i + 1] = b * f.x + a * f.y;
+      } else {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int d0 = c + e;                 // d0 < rot, as rot is even
+          const bool low = d0 < half;
+          const float2 f = tab[low ? d0 : d0 - half];
+          const float other = entry(low ? d0 + half : d0 - half);
+          x[2 * i + e] = low ? x[2 * i + e] * f.x - other * f.y : x[2 * i + e] * f.x + other * f.y;
+        }
+      }
+    }
+  }
+  if (!is_q && !is_k && (p.v_first != nullptr || p.v_keep != nullptr)) {
+    const size_t at = (size_t)t * p.nkv * p.dv + (size_t)(h - p.nq - p.nkv) * p.dv;
+    const float lam = p.v_first != nullptr ? p.lambda[0] : 0.f;
+#pragma unroll
+    for (int i = 0; i < MAXP; ++i) {
+      const int c = 2 * lane + 64 * i;
+      if (c < d) {
+        if (p.v_first != nullptr) {
+          const T* f = reinterpret_cast<const T*>(p.v_first) + at + c;
+          x[2 * i] = (1.0f - lam) * x[2 * i] + lam * to_f<T>(f[0]);
+          x[2 * i + 1] = (1.0f - lam) * x[2 * i + 1] + lam * to_f<T>(f[1]);
+        } else {
+          T* f = reinterpret_cast<T*>(p.v_keep) + at + c;
+          f[0] = from_f<T>(x[2 * i]);
+          f[1] = from_f<T>(x[2 * i + 1]);
+        }
       }
     }
   }
@@ -194,6 +251,7 @@ struct WindowAttnParams {
   const float* bias;          // [nq, far + 1] bias by distance (the last entry serves every larger distance), or null
   const float* sink;          // [nq] or null
   const void* gate;           // pre-activation of head h of query t at gate[t * ld_gate + h], or null
+  const void* wide_gate;      // pre-activation of every output element, gate[t * ld_gate + h * dv + d] (portion kernel), or null
   int n, nq, nkv, dk, dv, page_size, max_pages, window, keep_first, far;
   long long ld_q, ld_out, ld_gate;
   float scale;
@@ -619,6 +677,8 @@ struct WindowTiles {
   const int* q0;              // [n_tiles] first packed query
   const int* qn;              // [n_tiles] queries (<= 128)
   int n_pages;                // pages of the pool (an index past it reads zeros)
+  long long kv_ld;            // 0: paged cache; else the keys and values are rows [nkv * dk | nkv * dv] of this pitch, one per
+                              // token, and a page is 16 consecutive rows
 };
 
 template <int HK, int HV>
@@ -918,6 +978,12 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
           if (c + v * 8 < p.dv) {
             uint4 pk;
             __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&pk);
+            if (p.wide_gate != nullptr) {
+              float z[8];
+              load8(reinterpret_cast<const __nv_bfloat16*>(p.wide_gate) + (size_t)(q0 + row) * p.ld_gate + (size_t)head * p.dv + c + v * 8, z);
+#pragma unroll
+              for (int e = 0; e < 8; ++e) o[v * 8 + e] = __fdividef(o[v * 8 + e], 1.0f + __expf(-z[e]));
+            }
 #pragma unroll
             for (int e = 0; e < 4; ++e) p2[e] = __floats2bfloat162_rn(o[v * 8 + 2 * e] * inv, o[v * 8 + 2 * e + 1] * inv);
             *reinterpret_cast<uint4*>(dst + c + v * 8) = pk;
@@ -961,13 +1027,14 @@ static int launch_window_decode(const WindowAttnParams& p, cudaStream_t stream) 
   return exact ? launch_window_decode_as<VEC, GB, true, false>(p, stream) : launch_window_decode_as<VEC, GB, false, false>(p, stream);
 }
 
-// K (or V) of a paged cache as a 4-D tensor [pages][kv heads][16 tokens][dims], read in boxes of one page's 16 tokens x 64 dims
-static int make_page_map(CUtensorMap* m, const void* base, int d, int nkv, int n_pages, size_t page_elems) {
+// K (or V) of a paged cache as a 4-D tensor [pages][kv heads][16 tokens][dims], read in boxes of one page's 16 tokens x 64 dims;
+// tok / head / page: strides in elements
+static int make_page_map(CUtensorMap* m, const void* base, int d, int nkv, int n_pages, size_t tok, size_t head, size_t page) {
   PfEncodeFn fn = pf_encode_fn();
   if (fn == nullptr) return -1;
-  if ((reinterpret_cast<uintptr_t>(base) & 15) || d % 8 || page_elems % 8) return -2;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || d % 8 || tok % 8 || head % 8 || page % 8) return -2;
   cuuint64_t dims[4] = {(cuuint64_t)d, WD_PAGE, (cuuint64_t)nkv, (cuuint64_t)n_pages};
-  cuuint64_t strides[3] = {(cuuint64_t)d * 2, (cuuint64_t)d * WD_PAGE * 2, (cuuint64_t)page_elems * 2};
+  cuuint64_t strides[3] = {(cuuint64_t)tok * 2, (cuuint64_t)head * 2, (cuuint64_t)page * 2};
   cuuint32_t box[4] = {64u, WD_PAGE, 1u, 1u}, estr[4] = {1u, 1u, 1u, 1u};
   CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr,
                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
@@ -1024,15 +1091,14 @@ extern "C" int tahb_kv_append(const int* row, const int* count, const int* start
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
-extern "C" int tahb_qkv_post(const void* qkv, long long ld, const float* bias, const float* q_w, const float* k_w,
-                             void* q_out, void* cache, const int* slot, int M, int nq, int nkv, int dk, int dv, int dim,
-                             int page_size, float eps, int f32, cudaStream_t stream) {
-  if (M <= 0) return 0;
-  if (dk > 256 || dv > 256 || dk % 8 || dv % 8 || dim > dk) return -2;
-  QkvPostParams p;
-  p.qkv = qkv; p.bias = bias; p.q_w = q_w; p.k_w = k_w; p.q_out = q_out; p.cache = cache; p.slot = slot;
-  p.M = M; p.nq = nq; p.nkv = nkv; p.dk = dk; p.dv = dv; p.dim = dim; p.page_size = page_size; p.ld = ld; p.eps = eps;
-  const long long warps = (long long)M * (nq + 2 * nkv);
+// Host-side description of one launch (same fields as QkvPostParams).
+extern "C" int tahb_qkv_post(const QkvPostParams* q, int f32, cudaStream_t stream) {
+  const QkvPostParams& p = *q;
+  if (p.M <= 0) return 0;
+  if (p.dk > 256 || p.dv > 256 || p.dk % 8 || p.dv % 8 || p.dim > p.dk) return -2;
+  if (p.rope != nullptr && (p.rot % 2 || p.rot < 2 || p.rot > p.dim)) return -2;
+  if (p.v_first != nullptr && p.lambda == nullptr) return -2;
+  const long long warps = (long long)p.M * (p.nq + 2 * p.nkv);
   const dim3 grid((unsigned)((warps + 3) / 4));
   cudaError_t e = f32 ? launch_chain(qkv_post_kernel<float>, grid, dim3(128), 0, stream, p)
                       : launch_chain(qkv_post_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, p);
@@ -1072,20 +1138,28 @@ extern "C" int tahb_window_attn_decode(const WindowAttnParams* p, cudaStream_t s
   return -2;
 }
 
-// Query tiles of portions; n_pages = pages of the layer's pool.  bias and sink in log2 units.
+// Query tiles of portions; n_pages = pages of the layer's pool; kv_ld: see WindowTiles.  bias and sink in log2 units.
 extern "C" int tahb_window_attn_tiles(const WindowAttnParams* p, const int* q0, const int* qn, int n_tiles, int n_pages,
-                                      cudaStream_t stream) {
+                                      long long kv_ld, cudaStream_t stream) {
   if (p->n <= 0 || n_tiles <= 0) return 0;
-  if (check_window_attn(p) || p->ld_out % 8) return -2;
+  if (check_window_attn(p) || p->ld_out % 8 || (p->wide_gate != nullptr && (p->ld_gate % 8 || (reinterpret_cast<uintptr_t>(p->wide_gate) & 15))))
+    return -2;
+  if (kv_ld != 0 && kv_ld < (long long)p->nkv * (p->dk + p->dv)) return -2;
   if (p->page_size != WD_PAGE) return -5;
   const size_t page_elems = (size_t)p->nkv * WD_PAGE * (p->dk + p->dv);
   CUtensorMap mq, mk, mv;
   int rc;
   if ((rc = make_query_map(&mq, p->q, p->n, (long long)p->nq * p->dk, p->ld_q))) return rc;
-  if ((rc = make_page_map(&mk, p->cache, p->dk, p->nkv, n_pages, page_elems))) return rc;
-  if ((rc = make_page_map(&mv, reinterpret_cast<const __nv_bfloat16*>(p->cache) + (size_t)p->nkv * WD_PAGE * p->dk, p->dv,
-                          p->nkv, n_pages, page_elems))) return rc;
-  WindowTiles tl{q0, qn, n_pages};
+  auto kv = reinterpret_cast<const __nv_bfloat16*>(p->cache);
+  if (kv_ld) {
+    if ((rc = make_page_map(&mk, kv, p->dk, p->nkv, n_pages, kv_ld, p->dk, WD_PAGE * kv_ld))) return rc;
+    if ((rc = make_page_map(&mv, kv + (size_t)p->nkv * p->dk, p->dv, p->nkv, n_pages, kv_ld, p->dv, WD_PAGE * kv_ld))) return rc;
+  } else {
+    if ((rc = make_page_map(&mk, kv, p->dk, p->nkv, n_pages, p->dk, (size_t)WD_PAGE * p->dk, page_elems))) return rc;
+    if ((rc = make_page_map(&mv, kv + (size_t)p->nkv * WD_PAGE * p->dk, p->dv, p->nkv, n_pages, p->dv, (size_t)WD_PAGE * p->dv,
+                            page_elems))) return rc;
+  }
+  WindowTiles tl{q0, qn, n_pages, kv_ld};
   const int hk = p->dk <= 64 ? 1 : p->dk <= 128 ? 2 : 4, hv = p->dv <= 64 ? 1 : p->dv <= 128 ? 2 : 4;
   if (hk == 4 || hv == 4) return launch_window_prefill<4, 4>(mq, mk, mv, *p, tl, n_tiles, stream);
   if (hk == 2) return hv == 2 ? launch_window_prefill<2, 2>(mq, mk, mv, *p, tl, n_tiles, stream)

@@ -2,10 +2,10 @@
 //
 //   poly_norm       act(z) = a N(z) + b N(z^2) + c N(z^3) + e with powers element by element and N(v) = v / sqrt(mean(v^2) +
 //                   eps) over the token's vector
-//   clamped_glu     y = g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit), of interleaved
+//   clamped_glu     y = g sigmoid(slope g) (u + offset), g = min(gate, limit), u = clamp(up, -limit, limit), of interleaved
 //                   gate / up columns, optionally with a factor per row in front (a routed token's weight) or behind (a
-//                   shared expert's gate)
-//   moe_route       sigmoid scores, the `top` largest per token, and the experts' token lists in blocks of `bn` rows
+//                   shared expert's gate).  SwiGLU is slope 1, offset 0, limit infinity
+//   moe_route       sigmoid or softmax scores, the `top` largest per token, and the experts' token lists in blocks of `bn` rows
 //   moe_gather      the tokens' rows copied into the lists
 //   moe_gemm        grouped product over the lists, one weight matrix per expert (tcgen05, persistent CTAs, two accumulators
 //                   in tensor memory so that the epilogue of a tile runs under the main loop of the next); plain, or with
@@ -130,12 +130,16 @@ __global__ void __launch_bounds__(PN_THREADS) poly_norm_kernel(const T* __restri
 // ---------------------------------------------------------------------------------------------
 // clamped_glu as a kernel of its own: 8 outputs (16 interleaved inputs) per thread and step.
 // ---------------------------------------------------------------------------------------------
+struct GluShape {
+  float limit, slope, offset;
+};
+
 struct GluParams {
   const void* in;             // [rows, ld_in] gate_0, up_0, gate_1, up_1, ...
   void* out;                  // [rows, ld_out]
   long long ld_in, ld_out;
   int rows, width;            // width = outputs per row (a multiple of 8)
-  float limit;
+  GluShape a;
   const float* in_scale;      // [rows] factor of gate and up, or null
   const float* gate;          // row r of the result times sigmoid(gate[r * ld_gate]), or null
   long long ld_gate;
@@ -162,15 +166,16 @@ __global__ void __launch_bounds__(256) clamped_glu_kernel(const GluParams p) {
     constexpr bool fast = sizeof(T) == 2;       // the result is rounded to 16 bits: approximate exponential and division do
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
-      const float g = fminf(w * v[2 * e], p.limit), u = fminf(fmaxf(w * v[2 * e + 1], -p.limit), p.limit);
-      o[e] = (fast ? __fdividef(g, 1.0f + __expf(-1.702f * g)) : g / (1.0f + expf(-1.702f * g))) * (u + 1.0f) * f;
+      const float g = fminf(w * v[2 * e], p.a.limit), u = fminf(fmaxf(w * v[2 * e + 1], -p.a.limit), p.a.limit);
+      o[e] = (fast ? __fdividef(g, 1.0f + __expf(-p.a.slope * g)) : g / (1.0f + expf(-p.a.slope * g))) * (u + p.a.offset) * f;
     }
     Vec8<T>::store(reinterpret_cast<T*>(p.out) + r * p.ld_out + c, o);
   }
 }
 
 // ---------------------------------------------------------------------------------------------
-// moe_route: one warp per token picks the `top` largest scores (lower index on a tie); ranks inside an expert's list come
+// moe_route: one warp per token picks the `top` largest scores (lower index on a tie; softmax scores are over all experts
+// and stay as they are); ranks inside an expert's list come
 // from counters (shared per CTA, one global addition per CTA and expert).  The CTA that finishes last turns the counts
 // into list starts and the block table and clears the counters for the next launch.
 // ---------------------------------------------------------------------------------------------
@@ -178,6 +183,7 @@ struct RouteParams {
   const float* z;             // [M, ldz] router logits, experts in columns 0 .. E - 1
   long long ldz;
   int M, E, top, bn, tok;     // tok = tokens per CTA
+  int softmax;
   int* expert;                // [M * top]
   int* rank;                  // [M * top] place in the expert's list
   float* weight;              // [M * top] score
@@ -207,10 +213,29 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_kernel(const RoutePar
   __syncthreads();
   for (int t = warp; t < nt; t += ROUTE_THREADS / 32) {
     float s[NV];
+    if (p.softmax) {
+      float mx = -INFINITY, sum = 0.f;
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      const int e = lane + 32 * i;
-      s[i] = e < p.E ? 1.0f / (1.0f + expf(-p.z[(size_t)(t0 + t) * p.ldz + e])) : -1.0f;
+      for (int i = 0; i < NV; ++i) {
+        const int e = lane + 32 * i;
+        s[i] = e < p.E ? p.z[(size_t)(t0 + t) * p.ldz + e] : -INFINITY;
+        mx = fmaxf(mx, s[i]);
+      }
+      mx = warp_max(mx);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        s[i] = lane + 32 * i < p.E ? expf(s[i] - mx) : 0.f;
+        sum += s[i];
+      }
+      sum = warp_sum(sum);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) s[i] = lane + 32 * i < p.E ? s[i] / sum : -1.0f;
+    } else {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int e = lane + 32 * i;
+        s[i] = e < p.E ? 1.0f / (1.0f + expf(-p.z[(size_t)(t0 + t) * p.ldz + e])) : -1.0f;
+      }
     }
     for (int j = 0; j < p.top; ++j) {
       float bv = -1.0f;
@@ -316,11 +341,11 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* __restrict
 struct MoeGemmParams {
   const int* blk_expert;
   const int* n_blocks;
-  const float* row_weight;    // GLU: factor of gate and up of every list row
+  const float* row_weight;    // GLU: factor of gate and up of every list row, or null
   int f_rows;                 // weight rows of an expert
   int f_tiles;                // 128-row tiles of them
   int kb;                     // K / 64
-  float limit;
+  GluShape a;
   int* status;
 };
 
@@ -435,9 +460,9 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         float v[C::CHUNK];
         if constexpr (C::CHUNK == 32) tmem_ld32(trow + c0, v);
         else tmem_ld16(trow + c0, v);
-        float wl = 0.f;
+        float wl = 1.0f;
         if constexpr (GLU) {
-          if (lane < C::CHUNK) wl = p.row_weight[b * BN + c0 + lane];
+          if (lane < C::CHUNK && p.row_weight != nullptr) wl = p.row_weight[b * BN + c0 + lane];
         }
         tmem_ld_wait();
         if constexpr (GLU) {
@@ -446,10 +471,10 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
           for (int j = 0; j < C::CHUNK; j += 2) {
             const float recv = __shfl_xor_sync(0xffffffffu, odd ? v[j] : v[j + 1], 1);
             const float w = __shfl_sync(0xffffffffu, wl, j + (odd ? 1 : 0));
-            const float g = fminf(w * (odd ? recv : v[j]), p.limit);
-            const float u = fminf(fmaxf(w * (odd ? v[j + 1] : recv), -p.limit), p.limit);
+            const float g = fminf(w * (odd ? recv : v[j]), p.a.limit);
+            const float u = fminf(fmaxf(w * (odd ? v[j + 1] : recv), -p.a.limit), p.a.limit);
             stg[(c0 + j + (odd ? 1 : 0)) * 64 + (row >> 1)] =
-                __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f));
+                __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-p.a.slope * g)) * (u + p.a.offset));
           }
         } else {
 #pragma unroll
@@ -586,12 +611,12 @@ extern "C" int tahb_poly_norm(const void* z, long long ldz, const float* act, vo
 }
 
 extern "C" int tahb_clamped_glu(const void* in, long long ld_in, void* out, long long ld_out, int rows, int width, float limit,
-                                const float* in_scale, const float* gate, long long ld_gate, const int* n_blocks, int bn,
+                                float slope, float offset, const float* in_scale, const float* gate, long long ld_gate, const int* n_blocks, int bn,
                                 int f32, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (width % 8 || ld_in % 8 || ld_out % 8 || ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) & 15)) return -1;
   if ((long long)rows * (width / 8) > 0x7fffffffll) return -2;
-  GluParams p{in, out, ld_in, ld_out, rows, width, limit, in_scale, gate, ld_gate, n_blocks, bn};
+  GluParams p{in, out, ld_in, ld_out, rows, width, {limit, slope, offset}, in_scale, gate, ld_gate, n_blocks, bn};
   long long blocks = ((long long)rows * (width / 8) + 255) / 256;
   if (blocks > 148 * 32) blocks = 148 * 32;
   const cudaError_t e = f32 ? launch_chain(clamped_glu_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, p)
@@ -600,12 +625,12 @@ extern "C" int tahb_clamped_glu(const void* in, long long ld_in, void* out, long
 }
 
 // Router and expert lists (see moe_route_kernel); count: E + 1 ints that are zero before the first launch.
-extern "C" int tahb_moe_route(const float* z, long long ldz, int M, int E, int top, int bn, int* expert, int* rank,
+extern "C" int tahb_moe_route(const float* z, long long ldz, int M, int E, int top, int bn, int softmax, int* expert, int* rank,
                               float* weight, int* count, int* seg, int* blk_expert, int* n_blocks, int max_blocks,
                               int* status, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (E < 1 || E > ROUTE_MAX_EXPERTS || top < 1 || top > E || top > 64 || bn < 1 || ldz < E) return -2;
-  RouteParams p{z, ldz, M, E, top, bn, M >= 4096 ? 32 : 8, expert, rank, weight, count, seg, blk_expert, n_blocks, max_blocks, status};
+  RouteParams p{z, ldz, M, E, top, bn, M >= 4096 ? 32 : 8, softmax, expert, rank, weight, count, seg, blk_expert, n_blocks, max_blocks, status};
   const dim3 grid((M + p.tok - 1) / p.tok);
   const size_t smem = (size_t)(2 * E + 2 * p.tok * top) * 4;
   const int nv = (E + 31) / 32;
@@ -634,11 +659,11 @@ extern "C" int tahb_moe_gather(const void* h, int row_bytes, long long ld_bytes,
 // list_rows is a multiple of bn.
 extern "C" int tahb_moe_gemm(const void* w, const void* x, void* out, int E, int f_rows, int K, int list_rows, int bn,
                              const int* blk_expert, const int* n_blocks, int glu, const float* row_weight, float limit,
-                             int* status, cudaStream_t stream) {
+                             float slope, float offset, int* status, cudaStream_t stream) {
   if (list_rows <= 0) return 0;
   if (K % 64 || K <= 0 || f_rows % 64 || list_rows % bn || (glu && f_rows % 128)) return -2;
   if ((long long)E * f_rows > 0x7fffffffll) return -2;
-  MoeGemmParams p{blk_expert, n_blocks, row_weight, f_rows, (f_rows + 127) / 128, K / 64, limit, status};
+  MoeGemmParams p{blk_expert, n_blocks, row_weight, f_rows, (f_rows + 127) / 128, K / 64, {limit, slope, offset}, status};
   const long long w_rows = (long long)E * f_rows;
 #define TAHB_MG(B_)                                                                                           \
   if (bn == B_) return glu ? launch_moe_gemm<B_, true>(w, x, out, w_rows, K, list_rows, f_rows / 2, p, stream) \

@@ -3,13 +3,15 @@
 //   embed_norm           x = scale * E[token] (+ sinusoid(position));    h = T(rms_g(x) * w)
 //   residual_norm        x += rms(y) * w_out;                            h = T(rms(x) * w_next)
 //   residual_add_norm    x += mult * (y + sum of expert outputs);        h = T(rms_g(x) * w_next)
+//   streams_norm         x_t <- sum_s mix[s][t] x_s + out[t] * y;        h = T(rms_g(sum_t in[t] x_t) * w_next)
 //
 // with rms(v) = v / sqrt(mean(v^2) + eps), and rms_g the same over each of `groups` equal consecutive parts of the vector.
 // residual_norm is the whole seam between two sublayers of a layer with a norm before and after each sublayer: y is the
 // sublayer's output projection, w_out the product of the output norm's weight and the layer scale, w_next the weight of the
 // norm that feeds the next projection.  residual_add_norm is the seam between two layers whose mixer and feed-forward run
 // in parallel from one norm: y holds the sum of their output projections, and the outputs of a mixture of experts are
-// gathered from the experts' token lists on the way.
+// gathered from the experts' token lists on the way.  streams_norm is the seam of hyper-connections: the residual is a small
+// number of streams that a sublayer reads through one set of weights and writes through another.
 //
 // Rows are padded: `ld` columns (a multiple of 64) of which the first `width` are real; padding columns of every operand
 // are zero, so only the mean knows the difference.
@@ -17,6 +19,7 @@
 //   few_linear      z[t, f] = x[t, :] . w[f, :] + b[f] in fp32 for a handful of features (gate pre-activations that
 //                   enter a recurrence), where a GEMM with a 16-bit output would round them
 //   gemm_f32        plain fp32 matrix product for the 32-bit mode
+//   rotary_table    cosines and sines of the rotary positions of a step
 #include "common.cuh"
 
 namespace tahb {
@@ -120,19 +123,27 @@ __device__ __forceinline__ float2 sin_cos_pair(float p, float hi, float lo) {
   return make_float2(fmaf(e, fmaf(-0.5f * e, s, c), s), fmaf(-e, fmaf(0.5f * e, c, s), c));
 }
 
-// pos / freq: position of every token and [2, (width + 1) / 2] frequencies (high parts, then low parts), or null
+// pos / freq: position of every token and [2, (width + 1) / 2] frequencies (high parts, then low parts), or null.
+// streams copies of the embedding go to x [M, streams, ld]; w_in [streams]: weights of their sum, which is what the norm
+// sees (null: one stream as it is).
 template <typename T, int VPT>
 __global__ void __launch_bounds__(RN_THREADS) embed_norm_kernel(const T* __restrict__ E, const int* __restrict__ tok,
                                                                 float scale, const int* __restrict__ pos,
-                                                                const float* __restrict__ freq, float* __restrict__ x,
-                                                                const float* __restrict__ w, T* __restrict__ h, int vocab,
-                                                                int width, int groups, int ld, float eps) {
+                                                                const float* __restrict__ freq, int streams, const float* __restrict__ w_in,
+                                                                float* __restrict__ x, const float* __restrict__ w,
+                                                                T* __restrict__ h, int vocab, int width, int groups, int ld,
+                                                                float eps) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float gsm[];
   const size_t row = blockIdx.x;
   const int id = min(max(tok[row], 0), vocab - 1);
   const int nvec = ld / 4;
+  float sum_in = 1.0f;
+  if (w_in != nullptr) {
+    sum_in = 0.f;
+    for (int s = 0; s < streams; ++s) sum_in += w_in[s];
+  }
   float4 v[VPT], r[VPT];
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
@@ -154,7 +165,8 @@ __global__ void __launch_bounds__(RN_THREADS) embed_norm_kernel(const T* __restr
           if (4 * c + 3 < width) v[i].w += a.y;
         }
       }
-      Vec4<float>::store(x + row * ld + c * 4, v[i]);
+      for (int s = 0; s < streams; ++s) Vec4<float>::store(x + (row * streams + s) * ld + c * 4, v[i]);
+      v[i].x *= sum_in; v[i].y *= sum_in; v[i].z *= sum_in; v[i].w *= sum_in;
     }
   }
   group_inv_rms<VPT>(v, width, groups, ld, eps, gsm, r);
@@ -220,6 +232,114 @@ __global__ void __launch_bounds__(RN_THREADS) residual_add_norm_kernel(const T* 
       Vec4<T>::store(h + row * ld + c * 4,
                      make_float4(v[i].x * r[i].x * g.x, v[i].y * r[i].y * g.y, v[i].z * r[i].z * g.z, v[i].w * r[i].w * g.w));
     }
+  }
+}
+
+// Hyper-connections.  hc: mix [S][S] (from, to), out [S], then the next reader's in [S].  y_bias [ld] (zero in the padding)
+// or null; y_ex / slot / y_weight: expert outputs [list rows, ld], list rows and weights [M, top], or null.  Every element of
+// the streams is read and written once.
+struct StreamsParams {
+  const void* y;
+  long long ldy;
+  const float* y_bias;
+  const void* y_ex;
+  const int* slot;
+  const float* y_weight;
+  int top;
+  float* x;                   // [M, S, ld]
+  const float* hc;
+  const float* w_next;
+  void* h;
+  int width, groups, ld;
+  float eps;
+};
+
+template <typename T, int VPT, int S>
+__global__ void __launch_bounds__(RN_THREADS) streams_norm_kernel(const StreamsParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float gsm[];
+  const size_t row = blockIdx.x;
+  const int nvec = p.ld / 4;
+  const T* y = reinterpret_cast<const T*>(p.y) + row * p.ldy;
+  float4 v[VPT], r[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    r[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < nvec && p.y != nullptr) r[i] = Vec4<T>::load(y + c * 4);
+    if (c < nvec && p.y_bias != nullptr) {
+      const float4 b = Vec4<float>::load(p.y_bias + c * 4);
+      r[i].x += b.x; r[i].y += b.y; r[i].z += b.z; r[i].w += b.w;
+    }
+  }
+  if (p.y_ex != nullptr) {
+    for (int j = 0; j < p.top; ++j) {
+      const T* src = reinterpret_cast<const T*>(p.y_ex) + (size_t)p.slot[row * p.top + j] * p.ld;
+      const float w = p.y_weight != nullptr ? p.y_weight[row * p.top + j] : 1.0f;
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + i * RN_THREADS;
+        if (c < nvec) {
+          const float4 e = Vec4<T>::load(src + c * 4);
+          r[i].x = fmaf(w, e.x, r[i].x); r[i].y = fmaf(w, e.y, r[i].y);
+          r[i].z = fmaf(w, e.z, r[i].z); r[i].w = fmaf(w, e.w, r[i].w);
+        }
+      }
+    }
+  }
+  float mix[S][S], out[S], in[S];
+#pragma unroll
+  for (int s = 0; s < S; ++s) {
+#pragma unroll
+    for (int t = 0; t < S; ++t) mix[s][t] = __ldg(p.hc + s * S + t);
+    out[s] = __ldg(p.hc + S * S + s);
+    in[s] = __ldg(p.hc + S * S + S + s);
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < nvec) {
+      float* x = p.x + row * S * p.ld + c * 4;
+      float4 old[S];
+#pragma unroll
+      for (int s = 0; s < S; ++s) old[s] = Vec4<float>::load(x + (size_t)s * p.ld);
+#pragma unroll
+      for (int t = 0; t < S; ++t) {
+        float4 n = make_float4(out[t] * r[i].x, out[t] * r[i].y, out[t] * r[i].z, out[t] * r[i].w);
+#pragma unroll
+        for (int s = 0; s < S; ++s) {
+          n.x = fmaf(mix[s][t], old[s].x, n.x); n.y = fmaf(mix[s][t], old[s].y, n.y);
+          n.z = fmaf(mix[s][t], old[s].z, n.z); n.w = fmaf(mix[s][t], old[s].w, n.w);
+        }
+        Vec4<float>::store(x + (size_t)t * p.ld, n);
+        v[i].x = fmaf(in[t], n.x, v[i].x); v[i].y = fmaf(in[t], n.y, v[i].y);
+        v[i].z = fmaf(in[t], n.z, v[i].z); v[i].w = fmaf(in[t], n.w, v[i].w);
+      }
+    }
+  }
+  group_inv_rms<VPT>(v, p.width, p.groups, p.ld, p.eps, gsm, r);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c < nvec) {
+      const float4 g = Vec4<float>::load(p.w_next + c * 4);
+      Vec4<T>::store(reinterpret_cast<T*>(p.h) + row * p.ld + c * 4,
+                     make_float4(v[i].x * r[i].x * g.x, v[i].y * r[i].y * g.y, v[i].z * r[i].z * g.z, v[i].w * r[i].w * g.w));
+    }
+  }
+}
+
+// out[t][i] = mscale * (cos, sin) of pos[t] * f_i; freq: [2, half] high parts, then low parts
+__global__ void rotary_table_kernel(const int* __restrict__ pos, const float* __restrict__ freq, float mscale,
+                                    float2* __restrict__ out, int M, int half) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int n = M * half;
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
+    const float2 a = sin_cos_pair((float)pos[i / half], freq[i % half], freq[half + i % half]);
+    out[i] = make_float2(mscale * a.y, mscale * a.x);
   }
 }
 
@@ -421,15 +541,15 @@ __global__ void swiglu_f32_kernel(const float* __restrict__ gu, float* __restric
 }
 
 template <typename T>
-static int embed_norm_launch(const void* E, const int* tok, float scale, const int* pos, const float* freq, float* x,
-                             const float* w, void* h, int M, int vocab, int width, int groups, int ld, float eps,
+static int embed_norm_launch(const void* E, const int* tok, float scale, const int* pos, const float* freq, int streams,
+                             const float* w_in, float* x, const float* w, void* h, int M, int vocab, int width, int groups, int ld, float eps,
                              cudaStream_t stream) {
   const size_t smem = group_rms_smem(width, groups, ld);
   const int need = (ld / 4 + RN_THREADS - 1) / RN_THREADS;
   auto e = reinterpret_cast<const T*>(E);
   auto o = reinterpret_cast<T*>(h);
   cudaError_t rc;
-#define TAHB_EN(V_) rc = launch_chain(embed_norm_kernel<T, V_>, dim3(M), dim3(RN_THREADS), smem, stream, e, tok, scale, pos, freq, x, w, o, vocab, width, groups, ld, eps)
+#define TAHB_EN(V_) rc = launch_chain(embed_norm_kernel<T, V_>, dim3(M), dim3(RN_THREADS), smem, stream, e, tok, scale, pos, freq, streams, w_in, x, w, o, vocab, width, groups, ld, eps)
   if (need <= 1) TAHB_EN(1);
   else if (need <= 2) TAHB_EN(2);
   else if (need <= 4) TAHB_EN(4);
@@ -437,6 +557,22 @@ static int embed_norm_launch(const void* E, const int* tok, float scale, const i
   else if (need <= 16) TAHB_EN(16);
   else return -2;
 #undef TAHB_EN
+  return rc == cudaSuccess ? 0 : -3;
+}
+
+template <typename T, int S>
+static int streams_norm_launch(const StreamsParams& p, int M, cudaStream_t stream) {
+  const int need = (p.ld / 4 + RN_THREADS - 1) / RN_THREADS;
+  const size_t smem = group_rms_smem(p.width, p.groups, p.ld);
+  cudaError_t rc;
+#define TAHB_SN(V_) rc = launch_chain(streams_norm_kernel<T, V_, S>, dim3(M), dim3(RN_THREADS), smem, stream, p)
+  if (need <= 1) TAHB_SN(1);
+  else if (need <= 2) TAHB_SN(2);
+  else if (need <= 4) TAHB_SN(4);
+  else if (need <= 8) TAHB_SN(8);
+  else if (need <= 16) TAHB_SN(16);
+  else return -2;
+#undef TAHB_SN
   return rc == cudaSuccess ? 0 : -3;
 }
 
@@ -500,14 +636,39 @@ static int few_linear_launch(const void* x, long long ldx, const void* w, const 
 
 using namespace tahb;
 
-// pos / freq: sinusoidal positions (see embed_norm_kernel), or null.  groups must divide width.
-extern "C" int tahb_embed_norm(const void* E, const int* tok, float scale, const int* pos, const float* freq, float* x,
-                               const float* w, void* h, int M, int vocab, int width, int groups, int ld, float eps, int f32,
-                               cudaStream_t stream) {
+// pos / freq: sinusoidal positions; streams / w_in: copies in x and the weights of their sum (see embed_norm_kernel).
+// groups must divide width.
+extern "C" int tahb_embed_norm(const void* E, const int* tok, float scale, const int* pos, const float* freq, int streams,
+                               const float* w_in, float* x, const float* w, void* h, int M, int vocab, int width, int groups,
+                               int ld, float eps, int f32, cudaStream_t stream) {
   if (M <= 0) return 0;
-  if (ld % 4 || width > ld || groups < 1 || width % groups || (freq != nullptr && pos == nullptr)) return -1;
-  return f32 ? embed_norm_launch<float>(E, tok, scale, pos, freq, x, w, h, M, vocab, width, groups, ld, eps, stream)
-             : embed_norm_launch<__nv_bfloat16>(E, tok, scale, pos, freq, x, w, h, M, vocab, width, groups, ld, eps, stream);
+  if (ld % 4 || width > ld || groups < 1 || width % groups || (freq != nullptr && pos == nullptr) || streams < 1) return -1;
+  return f32 ? embed_norm_launch<float>(E, tok, scale, pos, freq, streams, w_in, x, w, h, M, vocab, width, groups, ld, eps, stream)
+             : embed_norm_launch<__nv_bfloat16>(E, tok, scale, pos, freq, streams, w_in, x, w, h, M, vocab, width, groups, ld, eps,
+                                                stream);
+}
+
+// Seam of hyper-connections over `streams` (1..8) residual streams (see streams_norm_kernel).
+extern "C" int tahb_streams_norm(const StreamsParams* p, int M, int streams, int f32, cudaStream_t stream) {
+  if (M <= 0) return 0;
+  if (p->ld % 4 || p->ldy % 4 || p->width > p->ld || p->groups < 1 || p->width % p->groups ||
+      (p->y_ex != nullptr && (p->slot == nullptr || p->top < 1)))
+    return -1;
+#define TAHB_SS(S_) if (streams == S_) return f32 ? streams_norm_launch<float, S_>(*p, M, stream) : streams_norm_launch<__nv_bfloat16, S_>(*p, M, stream);
+  TAHB_SS(1) TAHB_SS(2) TAHB_SS(3) TAHB_SS(4) TAHB_SS(5) TAHB_SS(6) TAHB_SS(7) TAHB_SS(8)
+#undef TAHB_SS
+  return -2;
+}
+
+extern "C" int tahb_rotary_table(const int* pos, const float* freq, float mscale, float* out, int M, int half,
+                                 cudaStream_t stream) {
+  if (M <= 0 || half <= 0) return 0;
+  if ((long long)M * half > 0x3fffffffll) return -2;
+  int blocks = (M * half + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  const cudaError_t e = launch_chain(rotary_table_kernel, dim3(blocks), dim3(256), 0, stream, pos, freq, mscale,
+                                     reinterpret_cast<float2*>(out), M, half);
+  return e == cudaSuccess ? 0 : -3;
 }
 
 // x += mult * (y + sum_j y_ex[slot[., j]]); h = rms_g(x) * w_next.  y_ex / slot null: no expert outputs.

@@ -1,6 +1,6 @@
-"""HybridEngine: decoders that list their layers one by one - windowed attention over the paged cache, recurrent layers with
-a state per row, dense feed-forwards and mixtures of experts, sublayers one after the other or side by side - on an fp32
-residual stream.
+"""HybridEngine: decoders that list their layers one by one - windowed attention and latent attention over the paged cache,
+recurrent layers with a state per row, dense feed-forwards and mixtures of experts, sublayers one after the other or side by
+side - on one or several fp32 residual streams.
 
 One function, :meth:`HybridEngine._layers`, runs the layers for a packed set of tokens.  It serves
 
@@ -23,26 +23,30 @@ import torch
 
 from tah_b200.engine.base import DecodeEngine
 from tah_b200.engine.kv_cache import CacheGeometry, LayerKV, PagedKVCache, RecurrentState
-from tah_b200.engine.hybrid_weights import (AttentionLayer, BlockWeights, HybridWeights, MemoryLayer, MixtureLayer, PolyNormLayer,
-                                             distance_table)
+from tah_b200.engine.hybrid_weights import (AttentionLayer, BlockWeights, GLALayer, HybridWeights, LatentLayer, MemoryLayer, MixtureLayer,
+                                             PolyNormLayer, distance_table)
 from tah_b200.models.layered import LayeredForCausalLM
 from tah_b200.ops import cuda as K
 from tah_b200.utils.observe import nvtx_range
 
 NO_WINDOW = 2 ** 31 - 1
-TILE = 128                        # tokens of an attention query tile and of an mLSTM chunk
-MEMORY_CHUNKS = 192               # chunks per mLSTM launch (bounds the workspace)
+TILE = 128                        # tokens of an attention query tile and of a chunk of a recurrent layer
+MEMORY_CHUNKS = 192               # chunks per launch of a recurrent layer (bounds the workspace)
+LATENT_PAGES = 8192               # cache pages whose latents are expanded to keys and values at a time
 
 
 class _Plan:
     """Which tokens a pass runs: packed token ids, positions, cache rows and KV slots.  The first ``n_dec`` tokens are
     single tokens of a row each; behind them lie the prompt portions, portion ``e`` at ``seq_start[e]``,
-    ``seq_len[e]`` tokens long, cut into tiles of up to 128 tokens (attention query tiles and mLSTM chunks)."""
+    ``seq_len[e]`` tokens long, cut into tiles of up to 128 tokens (attention query tiles and chunks of recurrent layers)."""
     tok = pos = row = slot = None
     n_dec = 0
     seq_start = seq_len = None
     tile_q0 = tile_qn = None
-    groups = ()                   # mLSTM launches: (tiles a..b, first tile and tile count of each of their portions)
+    groups = ()                   # recurrent launches: (tiles a..b, first tile and tile count of each of their portions)
+    latent = ()                   # latent expansions: (tiles a..b, cache pages of their portions)
+    latent_pages = 0              # pages of the largest of them
+    portion_of = latent_table = None      # portion of every token, and its pages inside the expansion
 
 
 def decode_splits(m: AttentionLayer, n: int) -> int:
@@ -55,19 +59,28 @@ def decode_splits(m: AttentionLayer, n: int) -> int:
     return max(1, min(K.SM_COUNT * 4 // ctas, pages // 4, 16))
 
 
-class _Buffers:
-    """Activations of a pass over ``n`` tokens, the first ``n_dec`` of them single tokens; ``chunks``: mLSTM chunks of a
-    launch."""
+def latent_splits(m: LatentLayer, n: int) -> int:
+    """Key splits of the absorbed latent attention: the number whose CTA waves (one CTA per SM) cost least, for a context of
+    some sixteen 128-key tiles of 2.5 us and 3 us for start, end and merge of a CTA."""
+    if n == 0 or not m.on_tensor_cores:
+        return 1
+    ctas = n * (1 if m.spec.heads <= 16 else (m.spec.heads + 31) // 32)
+    return min(range(1, 17), key=lambda s: -(-ctas * s // K.SM_COUNT) * (40.0 / s + 3.0))
 
-    def __init__(self, w: HybridWeights, n: int, dtype, dev, n_dec: int, chunks: int = 0):
+
+class _Buffers:
+    """Activations of a pass over ``n`` tokens, the first ``n_dec`` of them single tokens; ``chunks``: chunks of a recurrent
+    layer's launch; ``latent_pages``: cache pages of a latent expansion."""
+
+    def __init__(self, w: HybridWeights, n: int, dtype, dev, n_dec: int, chunks: int = 0, latent_pages: int = 0):
         e = lambda *s: torch.empty(*s, dtype=dtype, device=dev)
         mix = [b.mixer for b in w.layers]
         moe = [b.ff for b in w.layers if isinstance(b.ff, MixtureLayer)]
-        self.x = torch.empty(n, w.Wp, dtype=torch.float32, device=dev)
+        self.x = torch.empty((n, w.Wp) if w.streams is None else (n, w.streams, w.Wp), dtype=torch.float32, device=dev)
         self.h, self.y = e(n, w.Wp), e(n, w.Wp)
         self.proj = e(n, max(m.w_in.shape[0] for m in mix))
-        self.q = e(n, max([m.spec.heads * m.dk for m in mix if isinstance(m, AttentionLayer) and m.own_queries]
-                          or [0]))
+        self.q = e(n, max([m.spec.heads * m.dk for m in mix if isinstance(m, AttentionLayer) and m.own_queries] +
+                          [m.w_uq.shape[0] for m in mix if isinstance(m, LatentLayer)] or [0]))
         # columns between heads * dv and the padded width meet zero weight columns; they only have to be finite
         self.o = torch.zeros(n, max(m.w_o.shape[1] for m in mix), dtype=dtype, device=dev)
         self.gates = torch.empty(n * max([m.w_if.shape[0] for m in mix if isinstance(m, MemoryLayer)] or [0]),
@@ -75,8 +88,25 @@ class _Buffers:
         f32 = lambda k: torch.empty(k, dtype=torch.float32, device=dev)
         self.attn_ws = f32(max([n_dec * m.spec.heads * decode_splits(m, n_dec) * (m.dv + 2) for m in mix
                                 if isinstance(m, AttentionLayer)] or [0]))
-        self.mem_ws = f32(max([K.mlstm_chunk_ws_floats(chunks, m.spec.heads, m.dk, m.dv) for m in mix
-                               if isinstance(m, MemoryLayer)] or [0]))
+        self.mem_ws = f32(max([K.mlstm_chunk_ws_floats(chunks, m.spec.heads, m.dk, m.dv) for m in mix if isinstance(m, MemoryLayer)] +
+                              [K.gla_chunk_ws_floats(n, chunks, m.spec.heads, m.dk, m.dv) for m in mix if chunks and isinstance(m, GLALayer)]
+                              or [0]))
+        self.low = f32(n * max([m.w_a1.shape[0] for m in mix if isinstance(m, GLALayer)] or [0]))
+        self.rope = {r: f32(n * r.dims).view(n, r.dims // 2, 2) for r in w.rotary}
+        self.v_first = e(n, max([m.nkv * m.dv for m in mix if isinstance(m, AttentionLayer) and m.spec.v_mix] or [0]))
+        # latent attention: query latents; head lists of the tokens in the absorbed form; expanded keys and values of the others
+        lat = [m for m in mix if isinstance(m, LatentLayer)]
+        listed = lambda m: n if m.w_exp is None else n_dec
+        self.head_lists = {(k, h): K.HeadLists(k, h, dtype, dev) for k, h in {(listed(m), m.spec.heads) for m in lat} if k}
+        rows = lambda m: self.head_lists[listed(m), m.spec.heads].rows if listed(m) else 0
+        most = lambda size: e(max([size(m) for m in lat] or [0]))
+        self.cq = most(lambda m: n * m.Qp)
+        self.list_q, self.list_qa = most(lambda m: rows(m) * m.w_abs.shape[2]), most(lambda m: rows(m) * m.w_abs.shape[1])
+        self.list_o, self.list_v = most(lambda m: rows(m) * m.Rp), most(lambda m: rows(m) * m.w_uv.shape[1])
+        self.latents = most(lambda m: latent_pages * 16 * m.w_abs.shape[1] if m.w_exp is not None else 0)
+        self.expanded = most(lambda m: latent_pages * 16 * m.w_exp.shape[0] if m.w_exp is not None else 0)
+        self.latent_ws = f32(max([listed(m) * m.spec.heads * latent_splits(m, listed(m)) * (m.Rp + 2) for m in lat
+                                  if latent_splits(m, listed(m)) > 1] or [0]))
         self.act = e(n, max([b.w_down.shape[1] for b in w.layers if b.w_down is not None] or [0]))
         # experts: logits of router and shared gate, token lists, their rows, activations and outputs
         self.router = f32(n * max([f.w_router.shape[0] for f in moe] or [0]))
@@ -127,6 +157,12 @@ class HybridEngine(DecodeEngine):
             if isinstance(m, AttentionLayer):
                 kv.append(LayerKV(shared_with=m.spec.kv_from) if m.nkv == 0 else LayerKV(m.nkv, m.dk, m.dv))
                 st.append(None)
+            elif isinstance(m, LatentLayer):                 # one vector per token, key and value of all heads
+                kv.append(LayerKV(1, m.Rp + m.rw, 0))
+                st.append(None)
+            elif isinstance(m, GLALayer):
+                kv.append(None)
+                st.append([(m.spec.heads, m.dk, m.dv)])
             else:
                 kv.append(None)
                 st.append([(m.spec.heads, m.dk, m.dv), (m.spec.heads, m.dk), (m.spec.heads,)])
@@ -165,6 +201,11 @@ class HybridEngine(DecodeEngine):
         post = dict(dk=m.dk, dv=m.dv, dim=s.dim, page_size=self.page_size, eps=self.cfg.rms_norm_eps)
         if m.own_queries:
             q = b.q.view(-1)[:n * s.heads * m.dk].view(n, s.heads * m.dk)
+            if s.rotary is not None:
+                post.update(rope=b.rope[s.rotary], rot=s.rotary.dims, interleaved=s.rotary.interleaved)
+            if s.v_mix:
+                v = b.v_first.view(-1)[:n * m.nkv * m.dv].view(n, m.nkv * m.dv)
+                post.update(dict(v_keep=v) if m.v_keeps else dict(v_first=v, lam=m.v_lambda))
             K.qkv_post(proj, m.b_in, m.q_norm, m.k_norm, q, pool, plan.slot, s.heads, m.nkv, **post)
         else:                                      # queries as projected; only new keys and values have to move
             q = proj[:, :s.heads * m.dk]
@@ -204,22 +245,76 @@ class HybridEngine(DecodeEngine):
                                chunk_len=plan.tile_qn[ta:tb], seq_chunk0=chunk0, seq_chunks=chunks, ws=b.mem_ws, **kw)
         return o
 
+    def _gla(self, li: int, m: GLALayer, proj: torch.Tensor, b: _Buffers, plan: _Plan) -> torch.Tensor:
+        s = m.spec
+        n, nd = b.h.shape[0], plan.n_dec
+        low = K.few_linear(b.h, m.w_a1, None, out=b.low[:n * m.w_a1.shape[0]].view(n, -1))
+        o = b.o[:, :m.w_o.shape[1]]
+        kw = dict(heads=s.heads, dk=m.dk, dv=m.dv, dim=s.dim, vdim=s.vdim, tau=s.tau, eps=self.cfg.rms_norm_eps)
+        w = (m.w_a2, m.b_a2, m.norm)
+        state = self.state.layers[li]
+        if nd:
+            K.gla_recurrent(proj[:nd], low[:nd], *w, o[:nd], state, plan.pos, plan.row, slot=plan.slot, **kw)
+        if nd < n and (self.plain or m.dk > 128 or m.dv > 256):
+            K.gla_recurrent(proj, low, *w, o, state, plan.pos, plan.row, seq_start=plan.seq_start, seq_len=plan.seq_len, **kw)
+        elif nd < n:
+            for ta, tb, chunk0, chunks in plan.groups:
+                K.gla_chunks(proj, low, *w, o, state, plan.pos, plan.row, chunk_start=plan.tile_q0[ta:tb],
+                             chunk_len=plan.tile_qn[ta:tb], seq_chunk0=chunk0, seq_chunks=chunks, ws=b.mem_ws, **kw)
+        return o
+
+    def _latent(self, li: int, m: LatentLayer, proj: torch.Tensor, b: _Buffers, plan: _Plan) -> torch.Tensor:
+        """Latent attention: single tokens (without expansion weights, all tokens) against the cached latents themselves,
+        portions against keys and values expanded from the cached latents of their rows."""
+        s, n = m.spec, b.h.shape[0]
+        H, pool, rope = s.heads, self.kv.layer_pool(0, li), b.rope[s.rotary]
+        view = lambda t, r, c: t[:r * c].view(r, c)
+        cq = view(b.cq, n, m.Qp)
+        K.latent_post(proj, m.q_norm, m.c_norm, rope, cq, pool, plan.slot, q_rank=s.q_rank, q_col=0, kv_rank=s.kv_rank, Rp=m.Rp,
+                      c_col=m.c_col, rot=s.rot_dim, rw=m.rw, r_col=m.r_col, eps=self.cfg.rms_norm_eps)
+        q = K.linear(cq, m.w_uq, out=view(b.q.view(-1), n, m.w_uq.shape[0]))
+        nl = n if m.w_exp is None else plan.n_dec
+        L = b.head_lists[nl, H] if nl else None
+        list_q = view(b.list_q, L.rows, m.w_abs.shape[2]) if nl else None
+        K.latent_query(q, rope, L, list_q, heads=H, dk=m.dk, dim=s.dim, rot=s.rot_dim)
+        o, gate = b.o[:, :m.w_o.shape[1]], proj[:, m.g_col:m.g_col + H * m.dv]
+        if nl:
+            qa = K.moe_linear(list_q, m.w_abs, L, view(b.list_qa, L.rows, m.w_abs.shape[1]))
+            oc = view(b.list_o, L.rows, m.Rp)
+            kw = dict(Rp=m.Rp, rw=m.rw, page_size=self.page_size, scale=s.scale)
+            if m.on_tensor_cores:
+                K.latent_attn_decode(qa, oc, pool, self.kv.page_table[0], plan.pos, plan.row, L, sink=m.sink_log2,
+                                     n_split=latent_splits(m, nl), ws=b.latent_ws, **kw)
+            else:
+                K.latent_attn_plain(qa, oc, pool, self.kv.page_table[0], plan.pos, plan.row, L, sink=m.sink, **kw)
+            K.latent_gate(K.moe_linear(oc, m.w_uv, L, view(b.list_v, L.rows, m.w_uv.shape[1])), L, gate[:nl], o[:nl], m.dv)
+        if nl < n:
+            for ta, tb, src in plan.latent:
+                c = K.latent_gather(pool, src, self.page_size, m.Rp + m.rw, view(b.latents, src.numel() * 16, m.w_exp.shape[1]))
+                kv = K.linear(c, m.w_exp, out=view(b.expanded, c.shape[0], m.w_exp.shape[0]))
+                K.window_attn_tiles(q, o, kv, plan.latent_table, plan.pos, plan.portion_of, plan.tile_q0[ta:tb], plan.tile_qn[ta:tb],
+                                    src.numel(), kv_ld=kv.stride(0), nq=H, nkv=H, dk=m.dk, dv=m.dv, page_size=self.page_size,
+                                    scale=s.scale, window=NO_WINDOW, keep_first=0, sink=m.sink_log2, wide_gate=gate)
+        return o
+
     def _mixture(self, f: MixtureLayer, proj: torch.Tensor, b: _Buffers):
-        """Routed experts of the tokens in ``b.h``: ``(outputs by list row, list rows of every token)``; the shared
-        expert's activation goes to its columns of ``b.o``."""
+        """Routed experts of the tokens in ``b.h``: ``(outputs by list row, list rows of every token, their weights or None
+        when the inputs were weighted)``; the shared expert's activation goes to its columns of ``b.o``."""
         s, n = f.spec, b.h.shape[0]
         L = b.lists[s.experts, s.top]
         z = K.few_linear(b.h, f.w_router, None, out=b.router[:n * f.w_router.shape[0]].view(n, -1))
-        K.moe_route(z, L)
+        K.moe_route(z, L, softmax=s.softmax)
         view = lambda t, cols: t[:L.rows * cols].view(L.rows, cols)
         x = K.moe_gather(b.h, L, view(b.list_x, b.h.shape[1]))
-        act = K.moe_glu_linear(x, f.w_gu, s.expert.limit, L, view(b.list_act, f.cols))
+        ex = s.expert
+        act = K.moe_glu_linear(x, f.w_gu, ex.limit, L, view(b.list_act, f.cols), slope=ex.slope, offset=ex.offset,
+                               weighted=not s.weight_output)
         y = K.moe_linear(act, f.w_down, L, view(b.list_y, b.h.shape[1]))
         if f.shared is not None:
             c = f.shared
             K.clamped_glu(proj[:, c.in_col:c.in_col + 2 * c.cols], c.limit, b.o[:, c.out_col:c.out_col + c.cols],
-                          gate=z[:, s.experts])
-        return y, L.slot
+                          gate=z[:, s.experts], slope=s.shared.slope, offset=s.shared.offset)
+        return y, L.slot, L.weight if s.weight_output else None
 
     def _parallel_layer(self, li: int, L: BlockWeights, proj: torch.Tensor, w_next: torch.Tensor, b: _Buffers, plan: _Plan) -> None:
         """Mixer and feed-forward beside each other: both read the projection of ``b.h``, one product over the columns of
@@ -229,7 +324,9 @@ class HybridEngine(DecodeEngine):
             K.poly_norm(proj[:, f.in_col:f.in_col + f.cols], f.act, f.n, self.cfg.rms_norm_eps,
                         b.o[:, f.out_col:f.out_col + f.cols])
         elif isinstance(f, MixtureLayer):
-            y_ex, slot = self._mixture(f, proj, b)
+            y_ex, slot, weight = self._mixture(f, proj, b)
+            if weight is not None:
+                raise NotImplementedError("weighted expert outputs beside a mixer")
         K.linear(self._attention(li, L.mixer, proj, b, plan), L.mixer.w_o, out=b.y)
         K.residual_add_norm(b.y, b.x, self.cfg.residual_mult, w_next, self.w.W, self.cfg.norm_groups, self.cfg.rms_norm_eps,
                             b.h, y_ex, slot)
@@ -239,28 +336,74 @@ class HybridEngine(DecodeEngine):
         input); returns the final-norm output."""
         w, eps = self.w, self.cfg.rms_norm_eps
         n_layers = len(w.layers)
+        run = {AttentionLayer: self._attention, LatentLayer: self._latent, GLALayer: self._gla, MemoryLayer: self._memory}
+        for r, (freq, m) in w.rotary.items():
+            K.rotary_table(plan.pos, freq, m, b.rope[r])
         for li, L in enumerate(w.layers):
             after = w.layers[li + 1].norm1 if li + 1 < n_layers else w.final_norm
             proj = K.linear(b.h, L.mixer.w_in, out=b.proj[:, :L.mixer.w_in.shape[0]])
             if L.parallel:
                 self._parallel_layer(li, L, proj, after, b, plan)
             else:
-                run = self._attention if isinstance(L.mixer, AttentionLayer) else self._memory
-                K.linear(run(li, L.mixer, proj, b, plan), L.mixer.w_o, out=b.y)
-                K.residual_norm(b.y, b.x, L.out1, L.norm2 if L.w_gu is not None else after, w.W, eps, b.h)
-                if L.w_gu is not None:
-                    act = K.swiglu_linear(b.h, L.w_gu, out=b.act[:, :L.w_down.shape[1]])
-                    K.linear(act, L.w_down, out=b.y)
-                    K.residual_norm(b.y, b.x, L.out2, after, w.W, eps, b.h)
+                K.linear(run[type(L.mixer)](li, L.mixer, proj, b, plan), L.mixer.w_o, out=b.y)
+                norm = L.norm2 if L.norm2 is not None else after
+                if w.streams is None:
+                    K.residual_norm(b.y, b.x, L.out1, norm, w.W, eps, b.h)
+                else:
+                    K.streams_norm(b.y, b.x, L.hc1, norm, w.W, self.cfg.norm_groups, eps, b.h, y_bias=getattr(L.mixer, "o_bias", None))
+                if L.norm2 is not None:
+                    self._feed_forward(L, after, b)
             if self.layer_hook is not None:
-                self.layer_hook(li, b.x[:, :w.W])
+                self.layer_hook(li, (b.x if w.streams is None else b.x.sum(1))[:, :w.W])
         return b.h
+
+    def _feed_forward(self, L: BlockWeights, w_next: torch.Tensor, b: _Buffers) -> None:
+        """The second sublayer: its output joins the residual, and ``b.h`` becomes the next layer's input."""
+        w, eps = self.w, self.cfg.rms_norm_eps
+        y, ex = b.y, {}
+        if isinstance(L.ff, MixtureLayer):
+            y, (ex["y_ex"], ex["slot"], ex["y_weight"]) = None, self._mixture(L.ff, None, b)
+        else:
+            act = K.swiglu_linear(b.h, L.w_gu, out=b.act[:, :L.w_down.shape[1]])
+            K.linear(act, L.w_down, out=y)
+        if w.streams is None:
+            K.residual_norm(y, b.x, L.out2, w_next, w.W, eps, b.h)
+        else:
+            K.streams_norm(y, b.x, L.hc2, w_next, w.W, self.cfg.norm_groups, eps, b.h, **ex)
 
     def _embed(self, b: _Buffers, plan: _Plan) -> None:
         """``b.x``: the residual stream of the tokens of ``plan``; ``b.h``: the first layer's normed input."""
         w = self.w
         K.embed_norm(w.embed, plan.tok, self.cfg.embedding_scale, w.layers[0].norm1, w.W, self.cfg.rms_norm_eps, b.x, b.h,
-                     groups=self.cfg.norm_groups, pos=plan.pos, freq=w.freq)
+                     groups=self.cfg.norm_groups, pos=plan.pos, freq=w.freq, streams=w.streams or 1, w_in=w.hc_in0)
+
+    def _latent_plan(self, plan: _Plan, rows: List[int], counts: List[int], tiles: List[int], n: int) -> None:
+        """Which cache pages the portions' latent layers expand, in launches of at most ``LATENT_PAGES`` pages (a single longer
+        row is a launch of its own).  Call when the step's tokens have their pages."""
+        dev, table = self.device, self.kv.page_table[0]
+        rows_t = torch.tensor(rows, device=dev)
+        lens = self.kv.len[0][rows_t].tolist()
+        if any(l < c for l, c in zip(lens, counts)):         # nothing was appended: the pool or a row's table is full
+            raise RuntimeError("KV pool too small for the step")
+        pages = [(l + self.page_size - 1) // self.page_size for l in lens]
+        launches, base, at = [], [], 0                       # tiles a..b, pages a..b
+        for k, t in zip(pages, tiles):
+            first = launches[-1][1] if launches else 0
+            if not launches or launches[-1][3] - launches[-1][2] + k > LATENT_PAGES:
+                launches.append([first, first, at, at])
+            base.append(at - launches[-1][2])
+            launches[-1][1] += t
+            at += k
+            launches[-1][3] = at
+        pages_t = torch.tensor(pages, device=dev)
+        which = torch.repeat_interleave(torch.arange(len(rows), device=dev), pages_t, output_size=at)
+        col = torch.arange(at, device=dev) - (torch.cumsum(pages_t, 0) - pages_t)[which]
+        src = table[rows_t[which], col].contiguous()
+        plan.latent = [(a, b, src[c:d]) for a, b, c, d in launches]
+        plan.latent_pages = max(d - c for _, _, c, d in launches)
+        plan.latent_table = (torch.tensor(base, device=dev).view(-1, 1) + torch.arange(max(pages), device=dev)).to(torch.int32)
+        e = torch.repeat_interleave(torch.arange(len(rows), device=dev), torch.tensor(counts, device=dev), output_size=sum(counts))
+        plan.portion_of = torch.nn.functional.pad(e.to(torch.int32), (n - e.numel(), 0))
 
     # ------------------------------------------------------------------------------------------
     # one step of portions and single tokens
@@ -312,7 +455,9 @@ class HybridEngine(DecodeEngine):
         plan.tile_q0, plan.tile_qn = d_q0, d_qn
         plan.groups = [(t, t + k, d_first[a:z], d_tiles[a:z]) for a, z, t, k in groups]
         K.kv_append(d_rows, d_counts, d_start, self.kv, 0, plan.pos, plan.row, plan.slot)
-        b = _Buffers(self.w, n, self.dtype, dev, n_dec, 0 if self.plain else max([g[3] for g in groups] or [0]))
+        if n_dec < n and any(isinstance(L.mixer, LatentLayer) and L.mixer.w_exp is not None for L in self.w.layers):
+            self._latent_plan(plan, rows[n_dec:], counts[n_dec:], tiles, n)
+        b = _Buffers(self.w, n, self.dtype, dev, n_dec, 0 if self.plain else max([g[3] for g in groups] or [0]), plan.latent_pages)
         self._embed(b, plan)
         h = self._layers(b, plan)
         if not want:

@@ -5,11 +5,12 @@ to multiples of 8), tables in the units of the kernels.
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import List, Optional
+from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from tah_b200.models.layered import (AttentionSpec, LayeredForCausalLM, MixtureSpec, MLSTMSpec, PolyNormSpec, SwiGLUSpec)
+from tah_b200.models.layered import (AttentionSpec, GLASpec, LatentAttentionSpec, LayeredForCausalLM, MixtureSpec, MLSTMSpec,
+                                     PolyNormSpec, RotarySpec, SwiGLUSpec)
 from tah_b200.ops import cuda as K
 
 LOG2E = 1.4426950408889634
@@ -53,11 +54,53 @@ class AttentionLayer:
     k_norm: Optional[torch.Tensor] = None
     bias: Optional[torch.Tensor] = None   # [heads, far + 1], natural units for the plain kernel, log2 units for the others
     sink: Optional[torch.Tensor] = None
+    o_bias: Optional[torch.Tensor] = None
+    v_keeps: bool = False                 # this layer's values are the ones later layers mix in
+    v_lambda: Optional[torch.Tensor] = None   # [1] weight of those values in this layer's
 
     @property
     def own_queries(self) -> bool:
-        """Queries need a step of their own between projection and attention (bias or norm)."""
-        return self.b_in is not None or self.q_norm is not None
+        """Queries need a step of their own between projection and attention (bias, norm or rotation)."""
+        return self.b_in is not None or self.q_norm is not None or self.spec.rotary is not None or self.spec.v_mix
+
+
+@dataclass
+class LatentLayer:
+    """Latent attention.  Cached row: ``[c: Rp columns | rotated part: rw]``; head lists and expansions also carry the rotated
+    part through their matrix products, by unit rows."""
+    spec: LatentAttentionSpec
+    dk: int                       # a head's query / key, dim + rot_dim padded to 8
+    dv: int
+    Qp: int                       # query latent, padded to 64
+    Rp: int
+    rw: int
+    w_in: torch.Tensor            # rows: query latent, c, rotated part, output gate
+    c_col: int
+    r_col: int
+    g_col: int
+    q_norm: torch.Tensor
+    c_norm: torch.Tensor
+    w_uq: torch.Tensor            # [heads * dk, Qp]
+    w_abs: torch.Tensor           # [heads, row of the cache padded to 64, dk padded to 64]: query -> query against cached rows
+    w_uv: torch.Tensor            # [heads, dv padded to 64, Rp]: weighted c -> value
+    w_exp: Optional[torch.Tensor]             # [heads * dk + heads * dv, row padded to 64]: cached rows -> keys and values
+    w_o: torch.Tensor
+    sink: torch.Tensor            # natural units for the plain kernel, log2 units for the others
+    sink_log2: torch.Tensor
+    on_tensor_cores: bool         # single tokens run on the tensor-core kernel
+
+
+@dataclass
+class GLALayer:
+    spec: GLASpec
+    dk: int
+    dv: int
+    w_in: torch.Tensor            # rows: q, k, v, output gate
+    w_a1: torch.Tensor            # decay features, rows padded to 4
+    w_a2: torch.Tensor            # [heads * dk, features]
+    b_a2: torch.Tensor
+    norm: torch.Tensor            # [dv], shared by the heads
+    w_o: torch.Tensor
 
 
 @dataclass
@@ -113,6 +156,8 @@ class BlockWeights:
     out2: Optional[torch.Tensor] = None
     w_gu: Optional[torch.Tensor] = None
     w_down: Optional[torch.Tensor] = None
+    hc1: Optional[torch.Tensor] = None    # hyper-connections behind the mixer: mix, out, in of the next reader
+    hc2: Optional[torch.Tensor] = None    # the same behind the feed-forward
 
 
 class HybridWeights:
@@ -167,14 +212,21 @@ class HybridWeights:
             return K.interleave_gate_up(torch.cat([mat(T(p + "gate"), n, self.Wp), mat(T(p + "up"), n, self.Wp)]))
 
         self.embed = mat(T("embed"), self.vocab, self.Wp)
-        self.head = mat(T("head"), self.vocab_shard[2], self.Wp)
-        self.final_norm = vec(T("final.norm").float() * cfg.logit_scale, self.Wp)
+        self.head = mat(T("embed" if cfg.tied_head else "head"), self.vocab_shard[2], self.Wp)
+        norm = lambda name: cfg.norm_offset + T(name).float()
+        self.final_norm = vec(norm("final.norm") * cfg.logit_scale, self.Wp)
+        self.rotary: Dict[RotarySpec, Tuple[torch.Tensor, float]] = {}       # frequencies (high, low parts), sine / cosine factor
+        for r in {r for r in (getattr(l.mixer, "rotary", None) for l in cfg.layers) if r is not None}:
+            f, m = r.frequencies()
+            f = torch.tensor(f, dtype=torch.float64)
+            self.rotary[r] = (torch.stack([f.float(), (f - f.float().double()).float()]).contiguous().to(dev), m)
         self.freq = K.sinusoid_frequencies(self.W, device=dev) if cfg.sinusoidal else None
         self.layers: List[BlockWeights] = []
         for i, l in enumerate(cfg.layers):
             p, m, f = f"l{i}.", l.mixer, l.ff
             x = p + "mix."
-            dk, dv = _pad(m.dim, 8), _pad(m.vdim, 8)
+            kd = m.dim + m.rot_dim if isinstance(m, LatentAttentionSpec) else m.dim
+            dk, dv = _pad(kd, 8), _pad(m.vdim, 8)
             w_o = heads_cols(T(x + "o"), m.heads, m.vdim, dv)
             ff, ff_rows, ff_cols = None, [], []
             if isinstance(m, AttentionSpec):
@@ -207,6 +259,24 @@ class HybridWeights:
                     mixer.bias = distance_table(T(x + "rel"), m.bias_max) * unit
                 if m.sink:
                     mixer.sink = vec(T(x + "sink"), H) * unit
+                if m.out_bias:
+                    mixer.o_bias = vec(T(x + "o.b"), self.Wp)
+                if m.v_mix:
+                    mixer.v_keeps = not any(isinstance(b.mixer, AttentionLayer) and b.mixer.spec.v_mix for b in self.layers)
+                    if not mixer.v_keeps:
+                        mixer.v_lambda = T(x + "vmix").float().reshape(1)
+            elif isinstance(m, LatentAttentionSpec):
+                mixer = self._latent(x, m, dk, dv, w_o, dtype, plain, T, mat, stack, heads_rows)
+            elif isinstance(m, GLASpec):
+                if max(dk, dv) > 1024:
+                    raise NotImplementedError("gated linear attention head sizes above 1024")
+                H, rank = m.heads, _pad(m.rank, 4)
+                w_in = stack([heads_rows(T(x + "q"), H, m.dim, dk), heads_rows(T(x + "k"), H, m.dim, dk),
+                              heads_rows(T(x + "v"), H, m.vdim, dv), heads_rows(T(x + "g"), H, m.vdim, dv)])
+                w_a2 = torch.zeros(H, dk, rank, dtype=dtype, device=dev)
+                w_a2[:, :m.dim, :m.rank] = T(x + "a2").view(H, m.dim, m.rank)
+                mixer = GLALayer(m, dk, dv, w_in, mat(T(x + "a1"), rank, self.Wp), w_a2.view(H * dk, rank),
+                                 heads_vec(T(x + "a2.b"), H, m.dim, dk), vec(T(x + "norm"), dv), w_o)
             else:
                 if max(dk, dv) > 1024:
                     raise NotImplementedError("mLSTM head sizes above 1024")
@@ -216,24 +286,83 @@ class HybridWeights:
                 w_if = mat(torch.cat([T(x + "i"), T(x + "f")]), 2 * H, self.Wp)
                 mixer = MemoryLayer(m, dk, dv, w_in, w_if, torch.cat([T(x + "i.b"), T(x + "f.b")]).float(),
                                     heads_vec(T(x + "norm"), H, m.vdim, dv), w_o)
-            b = BlockWeights(mixer, vec(T(p + "norm1"), self.Wp), l.parallel, ff)
+            b = BlockWeights(mixer, vec(norm(p + "norm1"), self.Wp), l.parallel, ff)
             if l.parallel:
                 if not isinstance(m, AttentionSpec):
                     raise NotImplementedError("a parallel layer around a recurrent mixer")
             else:
-                if cfg.norm_groups != 1:
-                    raise NotImplementedError("grouped norms in a layer with output norms")
-                b.out1 = vec(T(p + "norm1b").float() * T(p + "ls1").float(), self.Wp)
+                if cfg.streams is None:
+                    if cfg.norm_groups != 1:
+                        raise NotImplementedError("grouped norms in a layer with output norms")
+                    b.out1 = vec(T(p + "norm1b").float() * T(p + "ls1").float(), self.Wp)
                 if f is not None:
-                    if not isinstance(f, SwiGLUSpec):
-                        raise NotImplementedError(f"feed-forward {f.kind} in a layer of two sublayers")
+                    b.norm2 = vec(norm(p + "norm2"), self.Wp)
+                    if cfg.streams is None:
+                        b.out2 = vec(T(p + "norm2b").float() * T(p + "ls2").float(), self.Wp)
+                if isinstance(f, SwiGLUSpec):
                     Ip = _pad(f.ff, 64)
                     gu = torch.cat([mat(T(p + "mlp.gate"), Ip, self.Wp), mat(T(p + "mlp.up"), Ip, self.Wp)])
                     b.w_gu = K.interleave_gate_up(gu) if dtype == torch.bfloat16 else gu
                     b.w_down = mat(T(p + "mlp.down"), self.Wp, Ip)
-                    b.norm2 = vec(T(p + "norm2"), self.Wp)
-                    b.out2 = vec(T(p + "norm2b").float() * T(p + "ls2").float(), self.Wp)
+                elif isinstance(f, MixtureSpec) and f.shared is None and cfg.streams is not None:
+                    b.ff = self._mixture(p + "mlp.", f, T(p + "mlp.router"), None, T, mat, cols_of, gate_up)
+                elif f is not None:
+                    raise NotImplementedError(f"feed-forward {f.kind} in a layer of two sublayers")
             self.layers.append(b)
+
+        self.streams, self.hc_in0 = cfg.streams, None
+        if cfg.streams is not None:
+            self._streams(cfg, T)
+
+    def _streams(self, cfg, T) -> None:
+        """Hyper-connection weights of every seam: how the sublayer in front writes, how the next one (at the end: the plain
+        sum) reads."""
+        flat = lambda *names: torch.cat([T(n).float().reshape(-1) for n in names])
+        subs = [(i, q) for i, l in enumerate(cfg.layers) for q in ((1,) if l.ff is None else (1, 2))]
+        ins = [flat(f"l{i}.hc{q}.in") for i, q in subs] + [torch.ones(cfg.streams, device=self.embed.device)]
+        self.hc_in0 = ins[0]
+        for k, (i, q) in enumerate(subs):
+            w = torch.cat([flat(f"l{i}.hc{q}.mix", f"l{i}.hc{q}.out"), ins[k + 1]]).contiguous()
+            setattr(self.layers[i], f"hc{q}", w)
+
+    def _latent(self, x, m, dk, dv, w_o, dtype, plain, T, mat, stack, heads_rows) -> LatentLayer:
+        H, d, r, R = m.heads, m.dim, m.rot_dim, m.kv_rank
+        dev = self.embed.device
+        Qp, Rp, rw = _pad(m.q_rank, 64), _pad(R, 64), _pad(r, 8)
+        lp, dkv, unit = _pad(Rp + rw, 64), T(x + "dkv"), torch.arange(r, device=dev)
+        w_in = stack([mat(T(x + "dq"), Qp, self.Wp), mat(dkv[:R], Rp, self.Wp), mat(dkv[R:], rw, self.Wp),
+                      heads_rows(T(x + "g"), H, m.vdim, dv)])
+        w_uq = torch.zeros(H, dk, Qp, dtype=dtype, device=dev)
+        w_uq[:, :d + r, :m.q_rank] = T(x + "uq").view(H, d + r, m.q_rank)
+        w_uq = mat(w_uq.view(H * dk, Qp), _pad(H * dk, 64), Qp)
+        uk, uv = T(x + "uk").view(H, d, R), T(x + "uv").view(H, m.vdim, R)
+        w_abs = torch.zeros(H, lp, _pad(dk, 64), dtype=dtype, device=dev)
+        w_abs[:, :R, :d] = uk.transpose(1, 2)
+        w_abs[:, Rp + unit, d + unit] = 1.0
+        w_uv = torch.zeros(H, _pad(dv, 64), Rp, dtype=dtype, device=dev)
+        w_uv[:, :m.vdim, :R] = uv
+        w_exp = None
+        if not plain and max(dk, dv) <= 256:
+            w_exp = torch.zeros(_pad(H * (dk + dv), 64), lp, dtype=dtype, device=dev)
+            k = w_exp[:H * dk].view(H, dk, lp)
+            k[:, :d, :R] = uk
+            k[:, d + unit, Rp + unit] = 1.0
+            w_exp[H * dk:H * (dk + dv)].view(H, dv, lp)[:, :m.vdim, :R] = uv
+        vec = lambda t, n: torch.nn.functional.pad(t.float(), (0, n - t.numel())).contiguous()
+        sink = T(x + "sink").float().contiguous()
+        return LatentLayer(m, dk, dv, Qp, Rp, rw, w_in, Qp, Qp + Rp, Qp + Rp + rw, vec(T(x + "dq.norm"), Qp), vec(T(x + "dkv.norm"), Rp),
+                           w_uq, w_abs, w_uv, w_exp, w_o, sink, sink * LOG2E, not plain and K.latent_decode_fits(H, Rp, rw))
+
+    @staticmethod
+    def _mixture(p, f, router, shared, T, mat, cols_of, gate_up) -> MixtureLayer:
+        n, E = _pad(f.expert.ff, 64), f.experts
+        first = gate_up(f"{p}e0.", n)
+        w_gu = first.new_empty(E, *first.shape)
+        w_down = first.new_empty(E, first.shape[1], n)
+        for e in range(E):
+            w_gu[e] = gate_up(f"{p}e{e}.", n)
+            w_down[e] = cols_of(T(f"{p}e{e}.down"), n)
+        return MixtureLayer(f, n, mat(router, router.shape[0], first.shape[1]), w_gu, w_down, shared)
 
     @staticmethod
     def _parallel(p, f, in_col, out_col, T, mat, cols_of, gate_up):
@@ -248,17 +377,10 @@ class HybridWeights:
                     [torch.nn.functional.pad(w, (0, 0, 0, n - f.ff))], [cols_of(T(p + "down"), n)])
         if not isinstance(f, MixtureSpec):
             raise NotImplementedError(f"feed-forward {f.kind} beside a mixer")
-        n, E = _pad(f.expert.ff, 64), f.experts
         router, shared, rows, cols = T(p + "router"), None, [], []
         if f.shared is not None:
             ns = _pad(f.shared.ff, 64)
             router = torch.cat([router, T(p + "shared.sg")])
             shared = SharedExpertLayer(ns, f.shared.limit, in_col, out_col)
             rows, cols = [gate_up(p + "shared.", ns)], [cols_of(T(p + "shared.down"), ns)]
-        first = gate_up(f"{p}e0.", n)
-        w_gu = first.new_empty(E, *first.shape)
-        w_down = first.new_empty(E, first.shape[1], n)
-        for e in range(E):
-            w_gu[e] = gate_up(f"{p}e{e}.", n)
-            w_down[e] = cols_of(T(f"{p}e{e}.down"), n)
-        return MixtureLayer(f, n, mat(router, router.shape[0], first.shape[1]), w_gu, w_down, shared), rows, cols
+        return HybridWeights._mixture(p, f, router, shared, T, mat, cols_of, gate_up), rows, cols

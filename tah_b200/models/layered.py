@@ -2,12 +2,13 @@
 made of, the configuration the engine reads, and a model class that holds the weights under their on-disk names.
 
 The computation is the engine's (:mod:`tah_b200.engine.hybrid`).  A family (:mod:`tah_b200.models.gunuvik`,
-:mod:`tah_b200.models.ditilix`) reads its own ``config.json`` into these specs and says which tensors it has; every constant
+:mod:`tah_b200.models.ditilix`, :mod:`tah_b200.models.niralix`) reads its own ``config.json`` into these specs and says which tensors it has; every constant
 of a mechanism is a field here, and a mechanism that a family does not have is absent (``None`` / ``False``).
 """
 from __future__ import annotations
 
 import json
+import math
 import os
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Tuple
@@ -19,6 +20,40 @@ import torch.nn as nn
 # ------------------------------------------------------------------------------------
 # mixers
 # ------------------------------------------------------------------------------------
+@dataclass(frozen=True)
+class YarnSpec:
+    """Rotary frequencies stretched by ``factor`` for the slow pairs (fewer than ``slow`` turns within ``original`` positions),
+    unchanged for the fast ones (more than ``fast`` turns), blended linearly between."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotation of the first ``dims`` entries of a head by position; pairs ``(2 i, 2 i + 1)`` when ``interleaved``, else
+    ``(i, i + dims / 2)``."""
+    dims: int
+    base: float
+    interleaved: bool = False
+    yarn: Optional[YarnSpec] = None
+
+    def frequencies(self) -> Tuple[List[float], float]:
+        """``(frequency of every pair, factor of sine and cosine)`` in double precision."""
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        y = self.yarn
+        if y is None:
+            return f, 1.0
+
+        def pair_at(turns):                   # (real-valued) index whose frequency makes `turns` turns within y.original
+            return self.dims * math.log(y.original / (2 * math.pi * turns)) / (2 * math.log(self.base))
+
+        lo, hi = max(math.floor(pair_at(y.fast)), 0), min(math.ceil(pair_at(y.slow)), self.dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(len(f))]
+        return [a / y.factor * r + a * (1.0 - r) for a, r in zip(f, ramp)], 0.1 * math.log(y.factor) + 1.0
+
+
 @dataclass
 class AttentionSpec:
     """Causal attention over the paged cache: ``score = cap(temp(i) * (q . k) * scale) + bias[distance]``."""
@@ -38,6 +73,9 @@ class AttentionSpec:
     head_gate: bool = False               # output gate number per head
     softcap: Optional[float] = None       # cap(s) = softcap * tanh(s / softcap)
     q_temp: Optional[Tuple[float, float]] = None      # (coef, every): temp(i) = 1 + coef * ln(floor((i + 1) / every) + 1)
+    rotary: Optional[RotarySpec] = None
+    out_bias: bool = False                # bias of the output projection
+    v_mix: bool = False                   # values mixed with those of the first layer that has this flag
 
     kind = "attention"
 
@@ -52,6 +90,40 @@ class MLSTMSpec:
     kind = "mlstm"
 
 
+@dataclass
+class LatentAttentionSpec:
+    """Causal attention whose keys and values are linear in one cached latent of ``kv_rank`` and one rotated key part of
+    ``rot_dim`` per token; queries come from a latent of ``q_rank``.  Softmax with a learned sink per head, output times
+    ``sigmoid(W_g h)``."""
+    heads: int
+    dim: int                              # unrotated part of queries and keys
+    rot_dim: int                          # rotated part, keys share one
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rotary: RotarySpec
+
+    kind = "latent_attention"
+
+
+@dataclass
+class GLASpec:
+    """Gated linear attention: matrix memory with the decay ``sigmoid(z) ** (1 / tau)`` per key channel."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: int = 16                        # decay features (a checkpoint's tensor decides)
+
+    kind = "gla"
+
+
+def check_rotary(i: int, r: Optional[RotarySpec], size: int) -> None:
+    if r is not None and (r.dims < 2 or r.dims % 2 or r.dims > size or not r.base > 1.0):
+        raise ValueError(f"layer {i}: rotation of {r.dims} of {size} dims with base {r.base}")
+
+
 def check_attention(i: int, m: AttentionSpec, layers: List["LayerSpec"]) -> None:
     """Refuse head counts that do not divide and a ``kv_from`` that names no earlier layer with keys of the same shape."""
     if m.heads < 1 or m.kv_heads < 1 or m.heads % m.kv_heads:
@@ -60,6 +132,11 @@ def check_attention(i: int, m: AttentionSpec, layers: List["LayerSpec"]) -> None
         raise ValueError(f"layer {i}: score cap {m.softcap}")
     if m.q_temp is not None and not m.q_temp[1] > 0:
         raise ValueError(f"layer {i}: query temperature steps of {m.q_temp[1]} positions")
+    check_rotary(i, m.rotary, m.dim)
+    if m.v_mix:
+        first = next((l.mixer for l in layers if isinstance(l.mixer, AttentionSpec) and l.mixer.v_mix), m)
+        if m.kv_from is not None or (first.kv_heads, first.vdim) != (m.kv_heads, m.vdim):
+            raise ValueError(f"layer {i} cannot mix its values with those of the first layer that mixes")
     if m.kv_from is not None:
         src = layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
         if not isinstance(src, AttentionSpec) or src.kv_from is not None or \
@@ -87,19 +164,24 @@ class PolyNormSpec:
 
 @dataclass
 class ExpertSpec:
-    """A clamped gated unit: ``down(g sigmoid(1.702 g) (u + 1))``, ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``."""
+    """A clamped gated unit: ``down(g sigmoid(slope g) (u + offset))``, ``g = min(gate, limit)``, ``u = clamp(up, -limit,
+    limit)``.  SwiGLU: slope 1, offset 0, no limit."""
     ff: int
-    limit: float
+    limit: float = math.inf
+    slope: float = 1.702
+    offset: float = 1.0
 
 
 @dataclass
 class MixtureSpec:
-    """``top`` of ``experts`` by sigmoid score; the score multiplies the expert's input.  ``shared``: an expert of every
-    token, its output times a sigmoid gate."""
+    """``top`` of ``experts`` by score: a sigmoid, or a softmax over all experts.  The score multiplies the expert's input or
+    its output.  ``shared``: an expert of every token, its output times a sigmoid gate."""
     experts: int
     top: int
     expert: ExpertSpec
     shared: Optional[ExpertSpec] = None
+    softmax: bool = False
+    weight_output: bool = False
 
     kind = "moe"
 
@@ -126,6 +208,9 @@ class LayeredConfig:
     sinusoidal: bool = False              # sinusoidal positions added to the embedding
     residual_mult: float = 1.0            # factor of the sublayers' sum in a parallel layer
     logit_scale: float = 1.0
+    norm_offset: float = 0.0              # stored norm weights of the residual stream are this much below their value
+    streams: Optional[int] = None         # hyper-connections over that many residual streams; None: a plain residual sum
+    tied_head: bool = False               # the embedding table is the output projection
     raw: Dict = field(default_factory=dict)
 
     @property
@@ -162,7 +247,7 @@ class LayeredForCausalLM(nn.Module):
         self.config = cfg
         self.weights = nn.ParameterDict()
         for name, shape in cfg.tensor_shapes().items():
-            self.weights[self._key(name)] = nn.Parameter(torch.zeros(*shape, dtype=dtype or cfg.dtype, device=device),
+            self.weights[self._key(name)] = nn.Parameter(torch.zeros(shape, dtype=dtype or cfg.dtype, device=device),
                                                          requires_grad=False)
 
     @staticmethod

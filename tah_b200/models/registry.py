@@ -95,6 +95,11 @@ def _ditilix_load(path, dtype, device):
     return DitilixForCausalLM.from_pretrained(path, dtype=dtype, device=device)
 
 
+def _niralix_load(path, dtype, device):
+    from tah_b200.models.niralix import NiralixForCausalLM
+    return NiralixForCausalLM.from_pretrained(path, dtype=dtype, device=device)
+
+
 def _is(class_name: str) -> Callable[[object], bool]:
     return lambda model: type(model).__name__ == class_name
 
@@ -109,3 +114,5 @@ register_family(Family("gunuvik", lambda c: c.get("architecture") == "Gunuvik", 
                        _hybrid_engine, "gunuvik"))
 register_family(Family("ditilix", lambda c: c.get("architecture") == "Ditilix", _ditilix_load, _is("DitilixForCausalLM"),
                        _hybrid_engine, "ditilix"))
+register_family(Family("niralix", lambda c: c.get("architecture") == "Niralix", _niralix_load, _is("NiralixForCausalLM"),
+                       _hybrid_engine, "niralix"))

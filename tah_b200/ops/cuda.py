@@ -593,14 +593,18 @@ def swiglu_linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] 
     return out
 
 
-def embed_norm(E, tok, scale: float, w, width: int, eps: float, x, h, groups: int = 1, pos=None, freq=None):
+def embed_norm(E, tok, scale: float, w, width: int, eps: float, x, h, groups: int = 1, pos=None, freq=None, streams: int = 1,
+               w_in=None):
     """``x = scale * E[tok]`` (fp32 residual stream) and ``h = rms(x) * w`` in the activation type of ``E``.  Rows are
     padded to ``E.shape[1]`` columns, ``width`` of them real.  ``groups``: parts of the row with a root mean square of
-    their own; ``pos`` / ``freq``: token positions and :func:`sinusoid_frequencies`, adds sinusoidal positions to ``x``."""
+    their own; ``pos`` / ``freq``: token positions and :func:`sinusoid_frequencies`, adds sinusoidal positions to ``x``;
+    ``streams`` / ``w_in``: that many copies in ``x [M, streams, ld]``, and the fp32 weights of their sum (what ``h`` sees)."""
     f32 = _act_f32(E, h)
-    _rc(lib().tahb_embed_norm(_p(E), _p(tok), c_float(scale), _p(pos if freq is not None else None), _p(freq), _p(x), _p(w),
-                              _p(h), c_int(tok.shape[0]), c_int(E.shape[0]), c_int(width), c_int(groups), c_int(E.shape[1]),
-                              c_float(eps), c_int(f32), _stream()), "tahb_embed_norm")
+    if x.numel() != tok.shape[0] * streams * E.shape[1]:
+        raise ValueError(f"embed_norm: residual {tuple(x.shape)} for {streams} streams of {E.shape[1]} columns")
+    _rc(lib().tahb_embed_norm(_p(E), _p(tok), c_float(scale), _p(pos if freq is not None else None), _p(freq), c_int(streams),
+                              _p(w_in), _p(x), _p(w), _p(h), c_int(tok.shape[0]), c_int(E.shape[0]), c_int(width),
+                              c_int(groups), c_int(E.shape[1]), c_float(eps), c_int(f32), _stream()), "tahb_embed_norm")
 
 
 def sinusoid_frequencies(width: int, base: float = 10000.0, device=None) -> torch.Tensor:
@@ -610,6 +614,36 @@ def sinusoid_frequencies(width: int, base: float = 10000.0, device=None) -> torc
     f = base ** (-2.0 * i / width)
     hi = f.float()
     return torch.stack([hi, (f - hi.double()).float()]).contiguous().to(device)
+
+
+def rotary_table(pos, freq, mscale: float, out):
+    """``out [n, half, 2]``: ``mscale * (cos, sin)`` of ``pos * f``; ``freq [2, half]``: frequencies as high and low parts."""
+    _rc(lib().tahb_rotary_table(_p(pos), _p(freq), c_float(mscale), _p(out), c_int(pos.shape[0]), c_int(freq.shape[1]), _stream()),
+        "tahb_rotary_table")
+    return out
+
+
+class _Streams(ctypes.Structure):
+    _fields_ = [("y", c_void_p), ("ldy", c_ll), ("y_bias", c_void_p), ("y_ex", c_void_p), ("slot", c_void_p), ("y_weight", c_void_p),
+                ("top", c_int), ("x", c_void_p), ("hc", c_void_p), ("w_next", c_void_p), ("h", c_void_p), ("width", c_int),
+                ("groups", c_int), ("ld", c_int), ("eps", c_float)]
+
+
+def streams_norm(y, x, hc, w_next, width: int, groups: int, eps: float, h, y_bias=None, y_ex=None, slot=None, y_weight=None):
+    """The seam of hyper-connections: with ``x [M, S, ld]`` (fp32, in place) and ``hc`` = mix ``[S, S]`` (from, to), out
+    ``[S]``, in ``[S]`` back to back, ``x_t <- sum_s mix[s, t] x_s + out[t] * y`` and ``h = rms(sum_t in[t] x_t) * w_next``.
+    ``y`` may be None; ``y_bias [ld]`` is added to it; ``y_ex [list rows, ld]`` / ``slot [M, top]`` / ``y_weight [M, top]``:
+    expert outputs that are gathered and added with their weights."""
+    M, S, ld = x.shape
+    a = _Streams()
+    ptr = lambda t: 0 if t is None else t.data_ptr()
+    if hc.numel() != S * S + 2 * S or hc.dtype != torch.float32:
+        raise ValueError(f"streams_norm: {hc.numel()} weights for {S} streams")
+    a.y, a.ldy, a.y_bias, a.y_ex, a.slot, a.y_weight = ptr(y), 0 if y is None else y.stride(0), ptr(y_bias), ptr(y_ex), ptr(slot), ptr(y_weight)
+    a.top, a.x, a.hc, a.w_next, a.h = 0 if slot is None else slot.shape[1], ptr(x), ptr(hc), ptr(w_next), ptr(h)
+    a.width, a.groups, a.ld, a.eps = width, groups, ld, eps
+    f32 = _act_f32(h, *[t for t in (y, y_ex) if t is not None])
+    _rc(lib().tahb_streams_norm(ctypes.byref(a), c_int(M), c_int(S), c_int(f32), _stream()), "tahb_streams_norm")
 
 
 def residual_add_norm(y, x, mult: float, w_next, width: int, groups: int, eps: float, h, y_ex=None, slot=None):
@@ -653,18 +687,33 @@ def kv_append(rows, counts, starts, cache, depth: int, pos, row_of, slot):
         "tahb_kv_append")
 
 
+class _QkvPost(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("qkv", "bias", "q_w", "k_w", "q_out", "cache", "slot")] + \
+               [(n, c_int) for n in ("M", "nq", "nkv", "dk", "dv", "dim", "page_size")] + [("ld", c_ll), ("eps", c_float),
+                ("rope", c_void_p), ("rot", c_int), ("interleaved", c_int), ("v_first", c_void_p), ("lam", c_void_p),
+                ("v_keep", c_void_p)]
+
+
 def qkv_post(qkv, bias, q_w, k_w, q_out, cache, slot, nq: int, nkv: int, dk: int, dv: int, dim: int, page_size: int,
-             eps: float):
-    """Projection bias, per-head RMS norm of q / k, q to ``q_out``, k / v into the paged cache.  ``nkv = 0``: queries
-    only (a layer that reads another layer's keys); ``nq = 0``: keys and values only (``qkv`` starts at the keys)."""
-    _rc(lib().tahb_qkv_post(_p(qkv), c_ll(qkv.stride(0)), _p(bias), _p(q_w), _p(k_w), _p(q_out), _p(cache), _p(slot),
-                            c_int(qkv.shape[0]), c_int(nq), c_int(nkv), c_int(dk), c_int(dv), c_int(dim), c_int(page_size),
-                            c_float(eps), c_int(_act_f32(qkv, qkv if q_out is None else q_out)), _stream()), "tahb_qkv_post")
+             eps: float, rope=None, rot: int = 0, interleaved: bool = False, v_first=None, lam=None, v_keep=None):
+    """Projection bias, per-head RMS norm of q / k, rotation of their first ``rot`` dims (``rope [n, rot / 2, 2]``, see
+    :func:`rotary_table`; pairs ``(2 i, 2 i + 1)`` when ``interleaved``, else ``(i, i + rot / 2)``), q to ``q_out``, k / v into
+    the paged cache.  ``nkv = 0``: queries only (a layer that reads another layer's keys); ``nq = 0``: keys and values only
+    (``qkv`` starts at the keys).  ``v_first [n, nkv * dv]`` / ``lam [1]``: values become ``(1 - lam) v + lam v_first``;
+    ``v_keep [n, nkv * dv]`` receives the values instead."""
+    a = _QkvPost()
+    ptr = lambda t: 0 if t is None else t.data_ptr()
+    for n, t in (("qkv", qkv), ("bias", bias), ("q_w", q_w), ("k_w", k_w), ("q_out", q_out), ("cache", cache), ("slot", slot),
+                 ("rope", rope), ("v_first", v_first), ("lam", lam), ("v_keep", v_keep)):
+        setattr(a, n, ptr(t))
+    a.M, a.nq, a.nkv, a.dk, a.dv, a.dim, a.page_size = qkv.shape[0], nq, nkv, dk, dv, dim, page_size
+    a.ld, a.eps, a.rot, a.interleaved = qkv.stride(0), eps, rot, int(interleaved)
+    _rc(lib().tahb_qkv_post(ctypes.byref(a), c_int(_act_f32(qkv, qkv if q_out is None else q_out)), _stream()), "tahb_qkv_post")
 
 
 class _WindowAttn(ctypes.Structure):
     _fields_ = [("q", c_void_p), ("out", c_void_p), ("cache", c_void_p), ("page_table", c_void_p), ("pos", c_void_p),
-                ("row", c_void_p), ("bias", c_void_p), ("sink", c_void_p), ("gate", c_void_p)] + \
+                ("row", c_void_p), ("bias", c_void_p), ("sink", c_void_p), ("gate", c_void_p), ("wide_gate", c_void_p)] + \
                [(n, c_int) for n in ("n", "nq", "nkv", "dk", "dv", "page_size", "max_pages", "window", "keep_first", "far")] + \
                [("ld_q", c_ll), ("ld_out", c_ll), ("ld_gate", c_ll), ("scale", c_float), ("softcap", c_float),
                 ("temp_coef", c_float), ("temp_every", ctypes.c_double), ("ws", c_void_p), ("n_split", c_int),
@@ -673,14 +722,15 @@ class _WindowAttn(ctypes.Structure):
 
 def window_attn_args(q, out, pool, page_table, pos, row, *, nq: int, nkv: int, dk: int, dv: int, page_size: int,
                      scale: float, window: int, keep_first: int, bias=None, sink=None, gate=None, softcap=None, q_temp=None,
-                     n_split: int = 1, ws=None):
+                     n_split: int = 1, ws=None, wide_gate=None):
     """Arguments of one windowed attention launch: queries ``q [n, nq * dk]`` (any row pitch) at positions ``pos`` of cache
     rows ``row`` over the paged ``pool`` of the layer that owns the keys; ``softcap``: score cap, ``q_temp = (coef,
     every)``: query temperature; see ``csrc/attn_window.cu`` for the rule."""
     a = _WindowAttn()
     ptr = lambda t: 0 if t is None else t.data_ptr()
     a.q, a.out, a.cache, a.page_table, a.pos, a.row = (ptr(t) for t in (q, out, pool, page_table, pos, row))
-    a.bias, a.sink, a.gate = ptr(bias), ptr(sink), ptr(gate)
+    a.bias, a.sink, a.gate, a.wide_gate = ptr(bias), ptr(sink), ptr(gate), ptr(wide_gate)
+    gate = wide_gate if gate is None else gate
     a.n, a.nq, a.nkv, a.dk, a.dv, a.page_size, a.max_pages = q.shape[0], nq, nkv, dk, dv, page_size, page_table.shape[1]
     a.window, a.keep_first, a.far = window, keep_first, 0 if bias is None else bias.shape[1] - 1
     a.softcap = 0.0 if softcap is None else softcap
@@ -705,13 +755,119 @@ def window_attn_decode(q, out, pool, page_table, pos, row, **kw):
     return out
 
 
-def window_attn_tiles(q, out, pool, page_table, pos, row, tile_q0, tile_qn, n_pages: int, **kw):
+def window_attn_tiles(q, out, pool, page_table, pos, row, tile_q0, tile_qn, n_pages: int, kv_ld: int = 0, **kw):
     """Windowed attention of prompt portions on the tensor cores (bf16, pages of 16): tiles of up to 128 consecutive
-    tokens of one row.  ``bias`` and ``sink`` in log2 units."""
+    tokens of one row.  ``bias`` and ``sink`` in log2 units.  ``kv_ld``: ``pool`` is not a paged cache but a matrix of that
+    pitch whose rows ``[keys of all heads | values of all heads]`` are a token each, 16 of them a page.  ``wide_gate``: gate
+    pre-activations of every output element (``gate``: of every head)."""
     a = window_attn_args(q, out, pool, page_table, pos, row, **kw)
     _rc(lib().tahb_window_attn_tiles(ctypes.byref(a), _p(tile_q0), _p(tile_qn), c_int(tile_q0.numel()), c_int(n_pages),
-                                     _stream()), "tahb_window_attn_tiles")
+                                     c_ll(kv_ld), _stream()), "tahb_window_attn_tiles")
     return out
+
+
+# -------------------------------------------------------------------------------------------
+# latent attention (csrc/attn_latent.cu)
+# -------------------------------------------------------------------------------------------
+class _LatentPost(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("proj", "q_w", "c_w", "rope", "cq", "cache", "slot")] + \
+               [(n, c_int) for n in ("M", "q_rank", "Qp", "q_col", "kv_rank", "Rp", "c_col", "rot", "rw", "r_col")] + \
+               [("ld", c_ll), ("eps", c_float)]
+
+
+def latent_post(proj, q_w, c_w, rope, cq, cache, slot, *, q_rank: int, q_col: int, kv_rank: int, Rp: int, c_col: int, rot: int,
+                rw: int, r_col: int, eps: float):
+    """After the projection ``[query latent | c | r | ...]``: ``cq`` = RMS norm of the query latent, and the cached row
+    ``[norm of c (Rp columns) | rotated r (rw columns)]`` of every token."""
+    a = _LatentPost()
+    for n, t in (("proj", proj), ("q_w", q_w), ("c_w", c_w), ("rope", rope), ("cq", cq), ("cache", cache), ("slot", slot)):
+        setattr(a, n, t.data_ptr())
+    a.M, a.q_rank, a.Qp, a.q_col, a.kv_rank, a.Rp, a.c_col = proj.shape[0], q_rank, cq.shape[1], q_col, kv_rank, Rp, c_col
+    a.rot, a.rw, a.r_col, a.ld, a.eps = rot, rw, r_col, proj.stride(0), eps
+    _rc(lib().tahb_latent_post(ctypes.byref(a), c_int(_act_f32(proj, cq, cache)), _stream()), "tahb_latent_post")
+
+
+class _LatentQuery(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("q", "rope", "list")] + \
+               [(n, c_int) for n in ("n", "n_list", "npad", "heads", "dk", "dq", "dim", "rot")] + [("ld", c_ll)]
+
+
+class HeadLists:
+    """Block table of head lists (``heads`` runs of ``npad`` rows), in the form the grouped products take."""
+
+    def __init__(self, n: int, heads: int, dtype: torch.dtype, device):
+        self.bn = 64 if dtype == torch.float32 else 16 if n <= 16 else 32 if n <= 32 else 64 if n <= 64 else 128
+        self.n, self.heads, self.npad = n, heads, (n + self.bn - 1) // self.bn * self.bn
+        self.rows = heads * self.npad
+        self.blk_expert = torch.arange(heads, dtype=torch.int32, device=device).repeat_interleave(self.npad // self.bn)
+        self.n_blocks = torch.full((1,), self.rows // self.bn, dtype=torch.int32, device=device)
+
+
+def latent_query(q, rope, lists: Optional[HeadLists], list_out, *, heads: int, dk: int, dim: int, rot: int):
+    """Rotate the last ``rot`` dims of every head of ``q [n, heads * dk]``: the first ``lists.n`` tokens go to the head lists
+    ``list_out [lists.rows, dq]``, the others are rotated in place."""
+    a = _LatentQuery()
+    a.q, a.rope, a.list = q.data_ptr(), rope.data_ptr(), 0 if lists is None else list_out.data_ptr()
+    a.n, a.n_list, a.npad = q.shape[0], 0 if lists is None else lists.n, 0 if lists is None else lists.npad
+    a.heads, a.dk, a.dq, a.dim, a.rot, a.ld = heads, dk, dk if lists is None else list_out.shape[1], dim, rot, q.stride(0)
+    _rc(lib().tahb_latent_query(ctypes.byref(a), c_int(_act_f32(q)), _stream()), "tahb_latent_query")
+
+
+def latent_gather(pool, src_pages, page_size: int, row: int, out):
+    """Pages ``src_pages`` of a latent cache (rows of ``row`` elements) one after another as rows of ``out [pages * page_size,
+    lp]``, zeros behind the cached row."""
+    es = pool.element_size()
+    if out.shape[0] < src_pages.numel() * page_size or not out.is_contiguous():
+        raise ValueError(f"latent_gather: {tuple(out.shape)} for {src_pages.numel()} pages")
+    _rc(lib().tahb_latent_gather(_p(pool), _p(src_pages), c_int(src_pages.numel()), c_int(pool.shape[0]), c_int(page_size),
+                                 c_int(row * es), c_int(out.shape[1] * es), _p(out), _stream()), "tahb_latent_gather")
+    return out
+
+
+def latent_gate(list_v, lists: HeadLists, gate, out, dv: int):
+    """``out[t, h * dv + d] = list_v[h * npad + t, d] * sigmoid(gate[t, h * dv + d])``: back from head lists to token rows."""
+    _rc(lib().tahb_latent_gate(_p(list_v), c_int(lists.npad), c_int(list_v.shape[1]), _p(gate), c_ll(gate.stride(0)), _p(out),
+                               c_ll(out.stride(0)), c_int(lists.n), c_int(lists.heads), c_int(dv), c_int(_act_f32(list_v, gate, out)),
+                               _stream()), "tahb_latent_gate")
+    return out
+
+
+class _LatentAttn(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("q", "out", "cache", "page_table", "pos", "row", "sink")] + \
+               [(n, c_int) for n in ("n", "npad", "heads", "Rp", "rw", "lq", "page_size", "max_pages")] + \
+               [("scale", c_float), ("ws", c_void_p), ("n_split", c_int), ("n_pages", c_int), ("status", c_void_p)]
+
+
+def _latent_attn_args(q, out, pool, page_table, pos, row, lists: HeadLists, *, Rp: int, rw: int, page_size: int, scale: float,
+                      sink=None, n_split: int = 1, ws=None):
+    a = _LatentAttn()
+    ptr = lambda t: 0 if t is None else t.data_ptr()
+    a.q, a.out, a.cache, a.page_table, a.pos, a.row, a.sink = (ptr(t) for t in (q, out, pool, page_table, pos, row, sink))
+    a.n, a.npad, a.heads, a.Rp, a.rw, a.lq = lists.n, lists.npad, lists.heads, Rp, rw, q.shape[1]
+    a.page_size, a.max_pages, a.scale, a.ws, a.n_split = page_size, page_table.shape[1], scale, ptr(ws), n_split
+    a.n_pages, a.status = pool.shape[0], status_word(q.device).data_ptr()
+    if n_split > 1 and ws.numel() < lists.n * lists.heads * n_split * (Rp + 2):
+        raise ValueError("latent attention: workspace too small")
+    return a
+
+
+def latent_attn_plain(q, out, pool, page_table, pos, row, lists: HeadLists, **kw):
+    """Absorbed latent attention of the tokens of ``lists`` over the cached rows: ``q [lists.rows, lq]`` -> ``out [lists.rows,
+    Rp]``, any sizes, bf16 or fp32.  ``sink`` in natural units."""
+    a = _latent_attn_args(q, out, pool, page_table, pos, row, lists, **kw)
+    _rc(lib().tahb_latent_attn_plain(ctypes.byref(a), c_int(_act_f32(q, out, pool)), _stream()), "tahb_latent_attn_plain")
+    return out
+
+
+def latent_attn_decode(q, out, pool, page_table, pos, row, lists: HeadLists, **kw):
+    """The same on the tensor cores (bf16, pages of 16), with optional key splits.  ``sink`` in log2 units."""
+    a = _latent_attn_args(q, out, pool, page_table, pos, row, lists, **kw)
+    _rc(lib().tahb_latent_attn_decode(ctypes.byref(a), _stream()), "tahb_latent_attn_decode")
+    return out
+
+
+def latent_decode_fits(heads: int, Rp: int, rw: int) -> bool:
+    return bool(lib().tahb_latent_decode_fits(c_int(heads), c_int(Rp), c_int(rw)))
 
 
 # -------------------------------------------------------------------------------------------
@@ -725,14 +881,14 @@ def poly_norm(z, act, n: int, eps: float, out):
     return out
 
 
-def clamped_glu(gu, limit: float, out, in_scale=None, gate=None, lists=None):
-    """``g sigmoid(1.702 g) (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)`` of interleaved columns
+def clamped_glu(gu, limit: float, out, in_scale=None, gate=None, lists=None, slope: float = 1.702, offset: float = 1.0):
+    """``g sigmoid(slope g) (u + offset)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)`` of interleaved columns
     ``gate_0, up_0, gate_1, ...``.  ``in_scale``: factor of both per row; ``gate``: fp32 column whose sigmoid multiplies
     the row's result; ``lists``: :class:`ExpertLists` that the rows are those of."""
     _rc(lib().tahb_clamped_glu(_p(gu), c_ll(gu.stride(0)), _p(out), c_ll(out.stride(0)), c_int(gu.shape[0]), c_int(out.shape[1]),
-                               c_float(limit), _p(in_scale), _p(gate), c_ll(0 if gate is None else gate.stride(0)),
-                               _p(None if lists is None else lists.n_blocks), c_int(0 if lists is None else lists.bn),
-                               c_int(_act_f32(gu, out)), _stream()), "tahb_clamped_glu")
+                               c_float(limit), c_float(slope), c_float(offset), _p(in_scale), _p(gate),
+                               c_ll(0 if gate is None else gate.stride(0)), _p(None if lists is None else lists.n_blocks),
+                               c_int(0 if lists is None else lists.bn), c_int(_act_f32(gu, out)), _stream()), "tahb_clamped_glu")
     return out
 
 
@@ -761,12 +917,13 @@ class ExpertLists:
         self.row_weight = torch.empty(self.rows, dtype=torch.float32, device=device)
 
 
-def moe_route(z, lists: ExpertLists):
-    """Choose ``lists.top`` experts per row of router logits ``z [M, >= experts]`` (fp32) and build the experts' lists."""
+def moe_route(z, lists: ExpertLists, softmax: bool = False):
+    """Choose ``lists.top`` experts per row of router logits ``z [M, >= experts]`` (fp32) and build the experts' lists; the
+    weights are the chosen experts' sigmoid scores, or their softmax scores over all experts."""
     L = lists
     if z.dtype != torch.float32 or z.shape[0] != L.M or z.shape[1] < L.experts:
         raise ValueError(f"moe_route: logits {z.dtype} {tuple(z.shape)} for {L.M} tokens and {L.experts} experts")
-    _rc(lib().tahb_moe_route(_p(z), c_ll(z.stride(0)), c_int(L.M), c_int(L.experts), c_int(L.top), c_int(L.bn), _p(L.expert),
+    _rc(lib().tahb_moe_route(_p(z), c_ll(z.stride(0)), c_int(L.M), c_int(L.experts), c_int(L.top), c_int(L.bn), c_int(int(softmax)), _p(L.expert),
                              _p(L.rank), _p(L.weight), _p(L.count), _p(L.seg), _p(L.blk_expert), _p(L.n_blocks),
                              c_int(L.max_blocks), _p(status_word(z.device)), _stream()), "tahb_moe_route")
 
@@ -792,23 +949,24 @@ def moe_linear(x, w, lists: ExpertLists, out):
                                     _p(lists.n_blocks), _stream()), "tahb_moe_gemm_f32")
     else:
         _rc(lib().tahb_moe_gemm(_p(w), _p(x), _p(out), c_int(E), c_int(F), c_int(Kd), c_int(lists.rows), c_int(lists.bn),
-                                _p(lists.blk_expert), _p(lists.n_blocks), c_int(0), _p(None), c_float(0.0),
+                                _p(lists.blk_expert), _p(lists.n_blocks), c_int(0), _p(None), c_float(0.0), c_float(0.0), c_float(0.0),
                                 _p(status_word(x.device)), _stream()), "tahb_moe_gemm")
     return out
 
 
-def moe_glu_linear(x, w, limit: float, lists: ExpertLists, out):
-    """:func:`clamped_glu` of :func:`moe_linear` with interleaved gate / up rows in ``w [experts, 2 F, K]``; every list row's
-    weight multiplies gate and up (the projection of the weighted input).  bf16: one kernel."""
+def moe_glu_linear(x, w, limit: float, lists: ExpertLists, out, slope: float = 1.702, offset: float = 1.0, weighted: bool = True):
+    """:func:`clamped_glu` of :func:`moe_linear` with interleaved gate / up rows in ``w [experts, 2 F, K]``; ``weighted``: every
+    list row's weight multiplies gate and up (the projection of the weighted input).  bf16: one kernel."""
     E, F2, Kd = w.shape
     if not (x.is_contiguous() and w.is_contiguous() and out.is_contiguous()) or x.shape != (lists.rows, Kd) or out.shape != (lists.rows, F2 // 2):
         raise ValueError(f"moe_glu_linear: x {tuple(x.shape)} w {tuple(w.shape)} out {tuple(out.shape)}")
+    row_weight = lists.row_weight if weighted else None
     if _act_f32(x, w, out):
         gu = moe_linear(x, w, lists, torch.empty(lists.rows, F2, dtype=torch.float32, device=x.device))
-        return clamped_glu(gu, limit, out, in_scale=lists.row_weight, lists=lists)
+        return clamped_glu(gu, limit, out, in_scale=row_weight, lists=lists, slope=slope, offset=offset)
     _rc(lib().tahb_moe_gemm(_p(w), _p(x), _p(out), c_int(E), c_int(F2), c_int(Kd), c_int(lists.rows), c_int(lists.bn),
-                            _p(lists.blk_expert), _p(lists.n_blocks), c_int(1), _p(lists.row_weight), c_float(limit),
-                            _p(status_word(x.device)), _stream()), "tahb_moe_gemm")
+                            _p(lists.blk_expert), _p(lists.n_blocks), c_int(1), _p(row_weight), c_float(limit), c_float(slope),
+                            c_float(offset), _p(status_word(x.device)), _stream()), "tahb_moe_gemm")
     return out
 
 
@@ -867,6 +1025,65 @@ def mlstm_recurrent(qkvg, gates, norm_w, out, state, pos, row, **kw):
     """mLSTM token by token (the decode step; also any portion): updates ``state = (S, n, m)`` in place."""
     a = mlstm_args(qkvg, gates, norm_w, out, state, pos, row, **kw)
     _rc(lib().tahb_mlstm_recurrent(ctypes.byref(a), c_int(_act_f32(qkvg, out)), _stream()), "tahb_mlstm_recurrent")
+    return out
+
+
+class _Gla(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("qkvg", "low", "w2", "b2", "norm_w", "out", "S", "seq_start", "seq_len", "pos", "row",
+                                        "slot")] + \
+               [(n, c_int) for n in ("n_seq", "heads", "dk", "dv", "vdim", "rank")] + [("ld", c_ll), ("ld_out", c_ll)] + \
+               [(n, c_float) for n in ("inv_tau", "eps", "q_scale")]
+
+
+def _gla_args(qkvg, low, w2, b2, norm_w, out, state, pos, row, *, heads: int, dk: int, dv: int, dim: int, vdim: int, tau: float,
+              eps: float, seq_start=None, seq_len=None, slot=None):
+    a = _Gla()
+    ptr = lambda t: 0 if t is None else t.data_ptr()
+    for n, t in (("qkvg", qkvg), ("low", low), ("w2", w2), ("b2", b2), ("norm_w", norm_w), ("out", out), ("S", state[0]),
+                 ("seq_start", seq_start), ("seq_len", seq_len), ("pos", pos), ("row", row), ("slot", slot)):
+        setattr(a, n, ptr(t))
+    if not low.is_contiguous() or low.shape[1] != w2.shape[1] or low.dtype != torch.float32:
+        raise ValueError(f"gla: decay features {low.dtype} {tuple(low.shape)} for weights {tuple(w2.shape)}")
+    a.n_seq = qkvg.shape[0] if seq_start is None else seq_start.shape[0]
+    a.heads, a.dk, a.dv, a.vdim, a.rank, a.ld, a.ld_out = heads, dk, dv, vdim, w2.shape[1], qkvg.stride(0), out.stride(0)
+    a.inv_tau, a.eps, a.q_scale = 1.0 / tau, eps, dim ** -0.5
+    return a
+
+
+class _GlaChunks(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("c_start", "c_len", "seq_chunk0", "seq_chunks", "G", "dS", "s0")] + \
+               [("n_chunks", c_int), ("status", c_void_p)]
+
+
+def gla_chunk_ws_floats(n_tokens: int, n_chunks: int, heads: int, dk: int, dv: int) -> int:
+    """fp32 workspace of :func:`gla_chunks`: running log decays of the tokens, state sums, incoming states as bf16 pairs."""
+    return n_tokens * heads * dk + n_chunks * heads * 2 * dk * dv
+
+
+def gla_chunks(qkvg, low, w2, b2, norm_w, out, state, pos, row, *, chunk_start, chunk_len, seq_chunk0, seq_chunks, ws, **kw):
+    """Gated linear attention of prompt portions in chunks of up to 128 tokens on the tensor cores (bf16, dk <= 128, dv <=
+    256); updates ``state`` in place.  Chunks and portions as in :func:`mlstm_chunks`."""
+    a = _gla_args(qkvg, low, w2, b2, norm_w, out, state, pos, row, **kw)
+    a.n_seq = seq_chunk0.shape[0]
+    heads, dk, dv, n, T = kw["heads"], kw["dk"], kw["dv"], chunk_start.shape[0], qkvg.shape[0]
+    c = _GlaChunks()
+    c.c_start, c.c_len, c.seq_chunk0, c.seq_chunks = (t.data_ptr() for t in (chunk_start, chunk_len, seq_chunk0, seq_chunks))
+    if ws.numel() < gla_chunk_ws_floats(T, n, heads, dk, dv):
+        raise ValueError("gla_chunks: workspace too small")
+    at = ws.data_ptr()
+    for name, floats in (("dS", n * heads * dk * dv), ("s0", n * heads * dk * dv), ("G", T * heads * dk)):
+        setattr(c, name, at)
+        at += 4 * floats
+    c.n_chunks, c.status = n, status_word(qkvg.device).data_ptr()
+    _rc(lib().tahb_gla_chunks(ctypes.byref(a), ctypes.byref(c), c_int(T), _stream()), "tahb_gla_chunks")
+    return out
+
+
+def gla_recurrent(qkvg, low, w2, b2, norm_w, out, state, pos, row, **kw):
+    """Gated linear attention token by token (the decode step; also any portion): updates ``state = (S,)`` in place.
+    ``low [n, rank]`` fp32 features, decay ``exp(logsigmoid(w2 low + b2) / tau)`` per key channel."""
+    a = _gla_args(qkvg, low, w2, b2, norm_w, out, state, pos, row, **kw)
+    _rc(lib().tahb_gla_recurrent(ctypes.byref(a), c_int(_act_f32(qkvg, w2, out)), _stream()), "tahb_gla_recurrent")
     return out
 
 
