@@ -2,11 +2,12 @@
 
     python bench.py --family gunuvik [--model gunuvik-1.7b] [--steps K] [--warmup W]
     python bench.py --family ditilix [--model ditilix-1.7b|ditilix-moe]
+    python bench.py --family niralix [--model niralix-1.7b|niralix-moe]
 
 Random weights, random token ids, bf16.  All models go through their own engines: ``prefill`` on whole prompts and
 decode ticks (CUDA graph) at a given context, reached with ``fast_forward``.  Comparison models: the plain Qwen3
-backbone (one pass per token, no adapter) with the same width, heads and vocabulary and a feed-forward of 6144, and for
-Ditilix also Gunuvik of that size; ``*_per_layer`` divides by the number of layers, because a recurrent layer has no
+backbone (one pass per token, no adapter) with the same width, heads and vocabulary and a feed-forward of 6144, for
+Ditilix also Gunuvik of that size, for Niralix also Gunuvik and the routed Ditilix; ``*_per_layer`` divides by the number of layers, because a recurrent layer has no
 feed-forward of its own.  Device time from CUDA
 events around K calls after W warm-up calls; every call reads the weights (GBs), far more than the 126 MB L2.
 """
@@ -40,8 +41,10 @@ def _qwen3(dev):
 def _layered(name, dev):
     import torch
     from tah_b200.engine import HybridEngine
-    from tah_b200.models import DitilixForCausalLM, GunuvikForCausalLM, ditilix_preset, gunuvik_preset
-    cls, preset = (DitilixForCausalLM, ditilix_preset) if name.startswith("ditilix") else (GunuvikForCausalLM, gunuvik_preset)
+    from tah_b200.models import (DitilixForCausalLM, GunuvikForCausalLM, NiralixForCausalLM, ditilix_preset, gunuvik_preset,
+                                 niralix_preset)
+    cls, preset = {"ditilix": (DitilixForCausalLM, ditilix_preset), "gunuvik": (GunuvikForCausalLM, gunuvik_preset),
+                   "niralix": (NiralixForCausalLM, niralix_preset)}[name.split("-")[0]]
     model = cls(preset(name), dtype=torch.bfloat16, device=dev).init_random()
     return lambda rows: HybridEngine(model, max_rows=rows), model, model.config
 
@@ -84,11 +87,10 @@ def run(args):
     from bench_clocks import ClockSampler
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
-    names = [args.model] if args.model.startswith(args.family) else \
-        ["gunuvik-1.7b"] if args.family == "gunuvik" else ["ditilix-1.7b", "ditilix-moe"]
-    builds = [(n, lambda d, n=n: _layered(n, d)) for n in names]
-    if args.family == "ditilix":
-        builds.append(("gunuvik-1.7b", lambda d: _layered("gunuvik-1.7b", d)))
+    presets = {"gunuvik": ["gunuvik-1.7b"], "ditilix": ["ditilix-1.7b", "ditilix-moe"], "niralix": ["niralix-1.7b", "niralix-moe"]}
+    beside = {"gunuvik": [], "ditilix": ["gunuvik-1.7b"], "niralix": ["gunuvik-1.7b", "ditilix-moe"]}
+    names = [args.model] if args.model.startswith(args.family) else presets[args.family]
+    builds = [(n, lambda d, n=n: _layered(n, d)) for n in names + beside[args.family]]
     builds.append(("qwen3 of the same sizes", _qwen3))
     steps, warmup = max(3, args.steps), max(3, args.warmup)
     sampler = ClockSampler(0)

@@ -384,6 +384,7 @@ class HybridEngine(DecodeEngine):
         rows_t = torch.tensor(rows, device=dev)
         lens = self.kv.len[0][rows_t].tolist()
         if any(l < c for l, c in zip(lens, counts)):         # nothing was appended: the pool or a row's table is full
+            K.check_status(dev)
             raise RuntimeError("KV pool too small for the step")
         pages = [(l + self.page_size - 1) // self.page_size for l in lens]
         launches, base, at = [], [], 0                       # tiles a..b, pages a..b

@@ -423,6 +423,13 @@ def main(argv=None):
     ap.add_argument("--keep", type=int, default=4, help="windowed attention: kept first tokens")
     ap.add_argument("--softcap", type=float, default=0.0, help="windowed attention: score cap and query temperature instead of "
                                                                "bias, sink and gate")
+    ap.add_argument("--rank", type=int, default=512, help="latent attention: size of the cached latent")
+    ap.add_argument("--rot", type=int, default=64, help="rotated dims of a head")
+    ap.add_argument("--rotate", action="store_true", help="qkv_post: rotation and mixed values instead of the norms")
+    ap.add_argument("--lists", type=int, default=0, help="latent_query: 1 = into head lists, 0 = in place")
+    ap.add_argument("--tau", type=float, default=16.0, help="gated linear attention: decay exponent 1 / tau")
+    ap.add_argument("--streams", type=int, default=2, help="residual streams")
+    ap.add_argument("--plain-glu", action="store_true", help="routed experts: SwiGLU units and softmax scores instead of clamped units")
     ap.add_argument("--experts", type=int, default=0, help="routed experts (--topk per token, --f wide, hidden size --k)")
     ap.add_argument("--v", type=int, default=151936)
     ap.add_argument("--topk", type=int, default=100)

@@ -1,5 +1,5 @@
-"""Micro-benchmark cases of the layered decoders' kernels (windowed attention, mLSTM, fp32-residual norms, PolyNorm, routed
-experts); run through :mod:`tah_b200.ops.microbench`, whose timing rules and flags apply.
+"""Micro-benchmark cases of the layered decoders' kernels (windowed and latent attention, mLSTM, gated linear attention,
+fp32-residual norms, PolyNorm, routed experts); run through :mod:`tah_b200.ops.microbench`, whose timing rules and flags apply.
 
 FLOPs and bytes are those of the algorithm: visible (query, key) pairs for attention, for the chunkwise mLSTM one
 128-token causal block plus the state read-out and update per chunk with every product counted once.
@@ -102,6 +102,135 @@ def bench_mlstm_step(a):
     return {"op": "mlstm_step", "rows": B, "heads": H, "dk": dk, "dv": dv}, fn, 6.0 * B * H * dk * dv, B * H * (dk * dv * 8 + (2 * dk + 3 * dv) * 2)
 
 
+def _gla_case(a, n, rows):
+    H, dk, dv, rank = a.nkv, a.hd, a.dv, 16
+    x, low, out = _bf(n, H * (2 * dk + 2 * dv)), torch.randn(n, rank, device="cuda"), torch.empty(n, H * dv, dtype=torch.bfloat16, device="cuda")
+    w2, b2 = _bf(H * dk, rank) / 4, torch.full((H * dk,), 2.0, device="cuda")
+    state = (torch.zeros(rows, H, dk, dv, device="cuda"),)
+    return (x, low, w2, b2, torch.ones(dv, device="cuda"), out, state), dict(heads=H, dk=dk, dv=dv, dim=dk, vdim=dv, tau=a.tau, eps=1e-6)
+
+
+def bench_gla_chunks(a):
+    """The like of ``mlstm_chunks``; ``--tau`` 16 has no steep channels, small values do."""
+    B, T = a.rows, a.ctx
+    n, H, dk, dv = B * T, a.nkv, a.hd, a.dv
+    ops, kw = _gla_case(a, n, B)
+    pos = torch.arange(T, device="cuda", dtype=torch.int32).repeat(B)
+    row = torch.arange(B, device="cuda", dtype=torch.int32).repeat_interleave(T)
+    starts = [b * T + t for b in range(B) for t in range(0, T, 128)]
+    lens = [min(128, T - t) for b in range(B) for t in range(0, T, 128)]
+    per = (T + 127) // 128
+    ws = torch.empty(K.gla_chunk_ws_floats(n, len(starts), H, dk, dv), device="cuda")
+    c = dict(chunk_start=_i32(starts), chunk_len=_i32(lens), seq_chunk0=_i32([b * per for b in range(B)]), seq_chunks=_i32([per] * B))
+    fn = lambda i: K.gla_chunks(*ops, pos, row, ws=ws, **c, **kw)
+    flops = H * sum(l * (l + 1) * (dk + dv) + 4.0 * l * dk * dv for l in lens)
+    byts = n * (H * (2 * dk + 3 * dv) * 2 + 64) + B * H * dk * dv * 8
+    return {"op": "gla_chunks", "seqs": B, "T": T, "heads": H, "dk": dk, "dv": dv, "tau": a.tau}, fn, flops, byts
+
+
+def bench_gla_step(a):
+    B, H, dk, dv = a.rows, a.nkv, a.hd, a.dv
+    ops, kw = _gla_case(a, B, B)
+    pos, row = _i32([5] * B), _i32(list(range(B)))
+    fn = lambda i: K.gla_recurrent(*ops, pos, row, **kw)
+    return {"op": "gla_step", "rows": B, "heads": H, "dk": dk, "dv": dv}, fn, 6.0 * B * H * dk * dv, B * H * (dk * dv * 8 + (2 * dk + 3 * dv) * 2)
+
+
+def bench_latent_decode(a):
+    """``--nq`` heads over cached rows of ``--rank`` + ``--rot``; ``--nsplit`` 0: the engine's choice."""
+    B, T, H, R, rw = a.rows, a.ctx, a.nq, a.rank, a.rot
+    lq = (R + rw + 63) // 64 * 64
+    pool, pt = _paged(B, T, 1, R + rw, 0)
+    L = K.HeadLists(B, H, torch.bfloat16, "cuda")
+    q, out, sink = _bf(L.rows, lq), torch.empty(L.rows, R, dtype=torch.bfloat16, device="cuda"), torch.randn(H, device="cuda")
+    split = a.nsplit
+    if split == 0:
+        from types import SimpleNamespace
+        from tah_b200.engine.hybrid import latent_splits
+        split = latent_splits(SimpleNamespace(on_tensor_cores=True, spec=SimpleNamespace(heads=H)), B)
+    pos, row, ws = _i32([T - 1] * B), _i32(list(range(B))), torch.empty(B * H * split * (R + 2), device="cuda")
+    fn = lambda i: K.latent_attn_decode(q, out, pool, pt, pos, row, L, Rp=R, rw=rw, page_size=16, scale=0.07, sink=sink, n_split=split, ws=ws)
+    return {"op": "latent_decode", "rows": B, "ctx": T, "heads": H, "rank": R, "rot": rw, "n_split": split}, fn, \
+        2.0 * B * T * H * (2 * R + rw), B * T * (R + rw) * 2 + B * H * (2 * R + rw) * 2
+
+
+def bench_latent_prefill(a):
+    """Attention of portions over expanded keys and values: ``--nq`` heads, keys of ``--hd`` + ``--rot``, values of ``--hd``."""
+    B, T, H, dk, dv = a.rows, a.ctx, a.nq, a.hd + a.rot, a.hd
+    n, pages = B * T, B * ((T + 15) // 16)
+    kv = _bf(pages * 16, H * (dk + dv))
+    pt = torch.arange(pages, device="cuda", dtype=torch.int32).view(B, -1)
+    q, out, gate = _bf(n, H * dk), torch.empty(n, H * dv, dtype=torch.bfloat16, device="cuda"), _bf(n, H * dv)
+    pos = torch.arange(T, device="cuda", dtype=torch.int32).repeat(B)
+    row = torch.arange(B, device="cuda", dtype=torch.int32).repeat_interleave(T)
+    q0 = _i32([b * T + t for b in range(B) for t in range(0, T, 128)])
+    qn = _i32([min(128, T - t) for b in range(B) for t in range(0, T, 128)])
+    sink = torch.randn(H, device="cuda")
+    fn = lambda i: K.window_attn_tiles(q, out, kv, pt, pos, row, q0, qn, pages, kv_ld=kv.shape[1], nq=H, nkv=H, dk=dk, dv=dv, page_size=16,
+                                       scale=dk ** -0.5, window=2 ** 31 - 1, keep_first=0, sink=sink, wide_gate=gate)
+    return {"op": "latent_prefill", "seqs": B, "T": T, "heads": H, "dk": dk, "dv": dv}, fn, 1.0 * B * T * (T + 1) * H * (dk + dv), \
+        n * H * (2 * dk + 3 * dv) * 2
+
+
+def bench_latent_post(a):
+    M, Q, R, rw = a.m, a.k, a.rank, a.rot
+    proj, cq = _bf(M, Q + R + rw + 64), torch.empty(M, Q, dtype=torch.bfloat16, device="cuda")
+    pool, slot = _bf((M + 15) // 16, 16 * (R + rw)), torch.arange(M, device="cuda", dtype=torch.int32)
+    w, rope = torch.ones(max(Q, R), device="cuda"), torch.randn(M, rw // 2, 2, device="cuda")
+    fn = lambda i: K.latent_post(proj, w, w, rope, cq, pool, slot, q_rank=Q, q_col=0, kv_rank=R, Rp=R, c_col=Q, rot=rw, rw=rw, r_col=Q + R, eps=1e-6)
+    return {"op": "latent_post", "M": M, "q_rank": Q, "rank": R}, fn, 0.0, M * ((Q + R + rw) * 4 + rw * 4)
+
+
+def bench_latent_query(a):
+    """In place for portions (``--lists`` 0) or into head lists."""
+    M, H, d, r = a.m, a.nq, a.hd, a.rot
+    dk, lists = d + r, K.HeadLists(a.m, a.nq, torch.bfloat16, "cuda") if a.lists else None
+    q, rope = _bf(M, H * dk), torch.randn(M, r // 2, 2, device="cuda")
+    out = _bf(lists.rows, (dk + 63) // 64 * 64) if a.lists else None
+    fn = lambda i: K.latent_query(q, rope, lists, out, heads=H, dk=dk, dim=d, rot=r)
+    return {"op": "latent_query", "M": M, "lists": bool(a.lists)}, fn, 0.0, M * H * (dk if a.lists else r) * 4 + M * r * 4
+
+
+def bench_latent_gather(a):
+    pages, row = a.m // 16, a.rank + a.rot
+    pool, src = _bf(pages, 16 * row), torch.randperm(pages, device="cuda").to(torch.int32)
+    out = _bf(pages * 16, (row + 63) // 64 * 64)
+    return {"op": "latent_gather", "tokens": a.m}, lambda i: K.latent_gather(pool, src, 16, row, out), 0.0, a.m * (row + out.shape[1]) * 2
+
+
+def bench_latent_gate(a):
+    M, H, dv = a.m, a.nq, a.hd
+    L = K.HeadLists(M, H, torch.bfloat16, "cuda")
+    v, g, out = _bf(L.rows, dv), _bf(M, H * dv), torch.empty(M, H * dv, dtype=torch.bfloat16, device="cuda")
+    return {"op": "latent_gate", "M": M}, lambda i: K.latent_gate(v, L, g, out, dv), 0.0, M * H * dv * 6
+
+
+def bench_head_product(a):
+    """Grouped product over head lists: ``--f`` outputs of ``--k`` inputs for each of ``--nq`` heads."""
+    L = K.HeadLists(a.m, a.nq, torch.bfloat16, "cuda")
+    x, w, out = _bf(L.rows, a.k), _bf(a.nq, a.f, a.k), torch.empty(L.rows, a.f, dtype=torch.bfloat16, device="cuda")
+    return {"op": "head_product", "M": a.m, "heads": a.nq, "K": a.k, "F": a.f}, lambda i: K.moe_linear(x, w, L, out), \
+        2.0 * a.m * a.nq * a.k * a.f, (w.numel() + a.m * a.nq * (a.k + a.f)) * 2
+
+
+def bench_streams_norm(a):
+    """``--streams`` residual streams; ``--topk`` weighted expert rows per token instead of one row when ``--experts`` is given."""
+    M, W, S, top = a.m, a.k, a.streams, a.topk if a.experts else 0
+    y, x, h = _bf(M, W), torch.randn(M, S, W, device="cuda"), torch.empty(M, W, dtype=torch.bfloat16, device="cuda")
+    hc = torch.cat([0.5 * torch.eye(S).flatten(), torch.full((2 * S,), 0.5)]).cuda()
+    w = torch.full((W,), 0.5, device="cuda")
+    ex = dict(y_ex=_bf(M * top, W), slot=torch.randperm(M * top, device="cuda").to(torch.int32).view(M, top),
+              y_weight=torch.rand(M, top, device="cuda")) if top else {}
+    fn = lambda i: K.streams_norm(None if top else y, x, hc, w, W, 1, 1e-6, h, **ex)
+    return {"op": "streams_norm", "M": M, "W": W, "streams": S, "experts": top}, fn, 0.0, M * W * (2 * max(1, top) + 8 * S + 2)
+
+
+def bench_rotary_table(a):
+    M, half = a.m, a.rot // 2
+    pos, freq, out = torch.arange(M, device="cuda", dtype=torch.int32), torch.rand(2, half, device="cuda"), torch.empty(M, half, 2, device="cuda")
+    return {"op": "rotary_table", "M": M, "half": half}, lambda i: K.rotary_table(pos, freq, 1.1, out), 0.0, M * (half * 8 + 4)
+
+
 def bench_residual_norm(a):
     M, W = a.m, a.k
     y, x, h = _bf(M, W), torch.randn(M, W, device="cuda"), torch.empty(M, W, dtype=torch.bfloat16, device="cuda")
@@ -117,8 +246,12 @@ def bench_qkv_post(a):
     pool = _bf((M + 15) // 16, a.nkv * 16 * 2 * a.hd)
     slot = torch.arange(M, device="cuda", dtype=torch.int32)
     b, w = torch.randn(F + 64, device="cuda"), torch.ones(a.hd, device="cuda")
-    fn = lambda i: K.qkv_post(qkv, b, w, w, q, pool, slot, a.nq, a.nkv, a.hd, a.hd, a.hd, 16, 1e-6)
-    return {"op": "qkv_post", "M": M}, fn, 0.0, 2 * M * F * 2
+    kw, extra = {}, 0
+    if a.rotate:                              # rotation of --rot dims and mixed values instead of the norms
+        kw = dict(rope=torch.randn(M, a.rot // 2, 2, device="cuda"), rot=a.rot, v_first=_bf(M, a.nkv * a.hd), lam=torch.full((1,), 0.3, device="cuda"))
+        w, extra = None, M * (a.rot * 4 + a.nkv * a.hd * 2)
+    fn = lambda i: K.qkv_post(qkv, b, w, w, q, pool, slot, a.nq, a.nkv, a.hd, a.hd, a.hd, 16, 1e-6, **kw)
+    return {"op": "qkv_post", "M": M, "rotate": bool(a.rotate)}, fn, 0.0, 2 * M * F * 2 + extra
 
 
 def bench_qk_norm_rope(a):
@@ -181,7 +314,8 @@ def _lists(a):
 
 def bench_moe_route(a):
     L, z = _lists(a)
-    return {"op": "moe_route", "M": a.m, "experts": a.experts, "top": a.topk}, lambda i: K.moe_route(z, L), 0.0, \
+    return {"op": "moe_route", "M": a.m, "experts": a.experts, "top": a.topk, "softmax": bool(a.plain_glu)}, \
+        lambda i: K.moe_route(z, L, softmax=bool(a.plain_glu)), 0.0, \
         a.m * (4 * a.experts + 12 * a.topk)
 
 
@@ -198,7 +332,8 @@ def _moe(a, glu):
     Kd, F = (a.k, 2 * a.f) if glu else (a.f, a.k)
     x, w = _bf(L.rows, Kd), _bf(a.experts, F, Kd)
     out = torch.empty(L.rows, a.f if glu else a.k, dtype=torch.bfloat16, device="cuda")
-    fn = (lambda i: K.moe_glu_linear(x, w, 7.0, L, out)) if glu else (lambda i: K.moe_linear(x, w, L, out))
+    form = dict(slope=1.0, offset=0.0, weighted=False) if a.plain_glu else {}
+    fn = (lambda i: K.moe_glu_linear(x, w, float("inf") if a.plain_glu else 7.0, L, out, **form)) if glu else (lambda i: K.moe_linear(x, w, L, out))
     pairs, used = a.m * a.topk, int(L.expert.unique().numel())
     return {"op": "moe_glu" if glu else "moe_down", "M": a.m, "experts": a.experts, "top": a.topk, "bn": L.bn,
             "rows": int(L.n_blocks) * L.bn}, fn, 2.0 * pairs * F * Kd, used * F * Kd * 2 + pairs * (Kd + out.shape[1]) * 2
@@ -216,4 +351,7 @@ CASES = {"window_prefill": bench_window_prefill, "window_decode": bench_window_d
          "mlstm_step": bench_mlstm_step, "residual_norm": bench_residual_norm, "qkv_post": bench_qkv_post,
          "qk_norm_rope": bench_qk_norm_rope, "few_linear": bench_few_linear, "residual_add_norm": bench_residual_add_norm,
          "poly_norm": bench_poly_norm, "clamped_glu": bench_clamped_glu, "swiglu": bench_swiglu, "moe_route": bench_moe_route,
-         "moe_gather": bench_moe_gather, "moe_glu": bench_moe_glu, "moe_down": bench_moe_down}
+         "gla_chunks": bench_gla_chunks, "gla_step": bench_gla_step, "latent_decode": bench_latent_decode,
+         "latent_prefill": bench_latent_prefill, "latent_post": bench_latent_post, "latent_query": bench_latent_query,
+         "latent_gather": bench_latent_gather, "latent_gate": bench_latent_gate, "head_product": bench_head_product,
+         "streams_norm": bench_streams_norm, "rotary_table": bench_rotary_table, "moe_gather": bench_moe_gather, "moe_glu": bench_moe_glu, "moe_down": bench_moe_down}

@@ -38,12 +38,12 @@ def rotate(x, positions, rot, interleaved):
     """Rotate the first ``rot.dims`` entries of the last axis of ``x [T, heads, d]``."""
     f, m = rotary_frequencies(rot)
     out, half = x.clone(), rot["dims"] // 2
-    for t, p in enumerate(positions):
-        for i in range(half):
-            a, b = (2 * i, 2 * i + 1) if interleaved else (i, i + half)
-            c, s = m * math.cos(p * f[i]), m * math.sin(p * f[i])
-            u, v = x[t, :, a], x[t, :, b]
-            out[t, :, a], out[t, :, b] = u * c - v * s, v * c + u * s
+    pairs = [(2 * i, 2 * i + 1) if interleaved else (i, i + half) for i in range(half)]
+    for i, (a, b) in enumerate(pairs):
+        c = torch.tensor([[m * math.cos(p * f[i])] for p in positions], dtype=torch.float64).to(x.dtype)
+        s = torch.tensor([[m * math.sin(p * f[i])] for p in positions], dtype=torch.float64).to(x.dtype)
+        u, v = x[:, :, a], x[:, :, b]
+        out[:, :, a], out[:, :, b] = u * c - v * s, v * c + u * s
     return out
 
 
@@ -185,3 +185,98 @@ def forward(cfg, sd, tokens, dtype=torch.float64, layers_out=None):
         if layers_out is not None:
             layers_out.append(sum(xs))
     return rms_norm(sum(xs), 1 + sd["final.norm"], eps) @ sd["embed"].T * cfg["logit_scale"]
+
+
+def random_model(cfg, seed=0, dtype=torch.bfloat16):
+    """Random weights under the on-disk names and shapes for ``cfg``, spread so that leaving a mechanism out shows.  Every gla
+    layer has ``cfg["_rank"]`` decay features, and decay biases around ``mixer["_bias"]`` (2 when absent).
+
+    Routing has no close calls: the first ``experts`` coordinates of an embedding are flags, ``top`` of them high, that no
+    sublayer writes to and that the streams only scale; a router row reads one flag (which one differs by layer) and a little
+    of everything else.  The mixtures of a model must therefore agree on ``experts`` and ``top``."""
+    g = torch.Generator().manual_seed(seed)
+    rnd = lambda *s: torch.randn(*s, generator=g, dtype=torch.float64)
+    W, V, S = cfg["width"], cfg["vocab"], cfg["streams"]
+    lin = lambda o, i, f=1.0: f * rnd(o, i) / math.sqrt(i)
+    near1 = lambda *s: 1.0 + 0.2 * rnd(*s)
+    moe = [l["mlp"] for l in cfg["layers"] if l["mlp"] is not None and l["mlp"]["kind"] == "moe"]
+    E, top = (moe[0]["router"]["experts"], moe[0]["router"]["top"]) if moe else (0, 0)
+    if any((m["router"]["experts"], m["router"]["top"]) != (E, top) for m in moe):
+        raise ValueError("mixtures of different router sizes")
+
+    def back(cols, f=1.0):                       # a projection back to the residual streams
+        w = lin(W, cols, f)
+        w[:E] = 0.0
+        return w
+
+    def norm(n):                                 # stored around zero
+        w = 0.2 * rnd(n)
+        w[:E] = 0.0
+        return w
+
+    embed = rnd(V, W)
+    for t in range(V):
+        embed[t, :E] = -4.0
+        embed[t, torch.randperm(E, generator=g)[:top]] = 4.0
+    sd = {"embed": embed, "final.norm": norm(W)}
+    for li, layer in enumerate(cfg["layers"]):
+        p, mix, mlp = f"l{li}.", layer["mixer"], layer["mlp"]
+        for q in (1,) if mlp is None else (1, 2):
+            sd[p + f"norm{q}"] = norm(W)
+            sd[p + f"hc{q}.in"] = (0.8 + 0.5 * torch.rand(S, generator=g, dtype=torch.float64)) / S
+            sd[p + f"hc{q}.out"] = near1(S)
+            sd[p + f"hc{q}.mix"] = 0.8 * torch.eye(S, dtype=torch.float64) + 0.2 * torch.rand(S, S, generator=g, dtype=torch.float64)
+        m = p + "mix."
+        H, dv = mix["heads"], mix["vdim"]
+        if layer["type"] == "attention":
+            G, dk = mix["kv_heads"], mix["dim"]
+            for n, o, i, f in (("q", H * dk, W, 1.5), ("k", G * dk, W, 1.5), ("v", G * dv, W, 1.0)):
+                sd[m + n], sd[m + n + ".b"] = lin(o, i, f), 0.5 * rnd(o)
+            sd[m + "o"], sd[m + "o.b"] = back(H * dv, 2.0), 0.3 * rnd(W)
+            sd[m + "o.b"][:E] = 0.0
+            if mix.get("v_mix"):
+                sd[m + "vmix"] = torch.tensor(0.3, dtype=torch.float64) + 0.2 * rnd(1)[0].abs()
+        elif layer["type"] == "latent_attention":
+            d, r, Q, R = mix["dim"], mix["rot_dim"], mix["q_rank"], mix["kv_rank"]
+            sd[m + "dq"], sd[m + "dq.norm"], sd[m + "uq"] = lin(Q, W), near1(Q), lin(H * (d + r), Q, 1.5)
+            sd[m + "dkv"], sd[m + "dkv.norm"] = lin(R + r, W, 1.5), near1(R)
+            sd[m + "uk"], sd[m + "uv"] = lin(H * d, R, 1.5), lin(H * dv, R)
+            sd[m + "sink"], sd[m + "g"], sd[m + "o"] = 1.0 + rnd(H), lin(H * dv, W), back(H * dv, 3.0)
+        else:
+            dk, r = mix["dim"], cfg["_rank"]
+            for n, o in (("q", H * dk), ("k", H * dk), ("v", H * dv), ("g", H * dv)):
+                sd[m + n] = lin(o, W)
+            sd[m + "o"], sd[m + "norm"] = back(H * dv, 1.5), near1(dv)
+            sd[m + "a1"], sd[m + "a2"], sd[m + "a2.b"] = lin(r, W), lin(H * dk, r, 1.5), mix.get("_bias", 2.0) + rnd(H * dk)
+        if mlp is None:
+            continue
+        m = p + "mlp."
+        if mlp["kind"] == "dense":
+            F = mlp["ff"]
+            sd[m + "gate"], sd[m + "up"], sd[m + "down"] = lin(F, W, 1.5), lin(F, W, 1.5), back(F)
+            continue
+        for i in range(E):
+            F, e = mlp["expert"]["ff"], f"{m}e{i}."
+            sd[e + "gate"], sd[e + "up"], sd[e + "down"] = lin(F, W, 1.5), lin(F, W, 1.5), back(F, 2.0)
+        router = lin(E, W, 0.2)
+        router[:, :E] = 0.5 * torch.eye(E, dtype=torch.float64)[torch.randperm(E, generator=g)]
+        sd[m + "router"] = router
+    return {k: v.to(dtype) for k, v in sd.items()}
+
+
+def router_margin(cfg, sd, tokens):
+    """Smallest distance in router logits between a chosen and a passed-over expert, over all tokens and mixtures."""
+    low = [math.inf]
+    keep = globals()["route"]
+
+    def watch(h, router, top):
+        z = (h @ router.T).sort(-1, descending=True).values
+        if z.shape[1] > top:
+            low[0] = min(low[0], float((z[:, top - 1] - z[:, top]).min()))
+        return keep(h, router, top)
+    globals()["route"] = watch
+    try:
+        forward(cfg, sd, tokens)
+    finally:
+        globals()["route"] = keep
+    return low[0]
