@@ -1,6 +1,6 @@
 // Latent attention: keys and values of all heads are linear in one cached vector per token.
 //
-//   cached row of a token:  [c: kv_rank, padded to Rp, a multiple of 64][r: rot dims, padded to rw, a multiple of 8]
+//   cached row of a token:  [c: kv_rank, padded to Rp][r: rot dims, padded to rw], both multiples of 64
 //     c = rms(low part) * w,  r = rotated shared key part
 //   head h:  key = [Wk_h c, r], value = Wv_h c;  score = (q . key) * scale;  softmax with exp(sink_h) in the denominator;
 //   out_h *= sigmoid(gate), element by element
@@ -102,7 +102,7 @@ __global__ void __launch_bounds__(128) latent_post_kernel(const LatentPostParams
 
 // ---------------------------------------------------------------------------------------------
 // latent_query: the projected queries [n, heads * dk], head = [dim | rot], get their last rot dims rotated.  Tokens below
-// n_list go to head lists [heads * npad, dq] (zero behind dim + rot), the others stay where they are.  One warp per head.
+// n_list go to head lists [heads * npad, dq] (zero behind dim + rot), the others stay where they are.  One CTA per token.
 // ---------------------------------------------------------------------------------------------
 struct LatentQueryParams {
   void* q;
@@ -113,25 +113,31 @@ struct LatentQueryParams {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(128) latent_query_kernel(const LatentQueryParams p) {
+__global__ void __launch_bounds__(256) latent_query_kernel(const LatentQueryParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const long long wg = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
-  const int lane = threadIdx.x & 31;
-  if (wg >= (long long)p.n * p.heads) return;
-  const int t = (int)(wg / p.heads), h = (int)(wg % p.heads);
-  T* q = reinterpret_cast<T*>(p.q) + (size_t)t * p.ld + (size_t)h * p.dk;
+  const int t = blockIdx.x, half = p.rot / 2;
   const bool listed = t < p.n_list;
-  T* dst = listed ? reinterpret_cast<T*>(p.list) + ((size_t)h * p.npad + t) * p.dq : q;
-  if (listed) {
-    for (int d = lane; d < p.dim; d += 32) dst[d] = q[d];
-    for (int d = p.dim + p.rot + lane; d < p.dq; d += 32) stf(dst + d, 0.f);
+  T* src = reinterpret_cast<T*>(p.q) + (size_t)t * p.ld;
+  T* list = reinterpret_cast<T*>(p.list) + (size_t)t * p.dq;             // head h at h * npad * dq
+  const size_t head = listed ? (size_t)p.npad * p.dq : p.dk;
+  T* dst = listed ? list : src;
+  for (int i = threadIdx.x; i < p.heads * half; i += 256) {
+    const int h = i / half, k = i % half;
+    const float2 f = p.rope[(size_t)t * half + k];
+    const T* q = src + (size_t)h * p.dk + p.dim + 2 * k;
+    const float u = ldf(q), v = ldf(q + 1);
+    T* o = dst + h * head + p.dim + 2 * k;
+    stf(o, u * f.x - v * f.y);
+    stf(o + 1, v * f.x + u * f.y);
   }
-  for (int i = lane; i < p.rot / 2; i += 32) {
-    const float2 f = p.rope[(size_t)t * (p.rot / 2) + i];
-    const float u = ldf(q + p.dim + 2 * i), v = ldf(q + p.dim + 2 * i + 1);
-    stf(dst + p.dim + 2 * i, u * f.x - v * f.y);
-    stf(dst + p.dim + 2 * i + 1, v * f.x + u * f.y);
+  if (listed) {
+    const int rest = p.dq - p.rot;                                        // unrotated dims, then the zeros behind the head
+    for (int i = threadIdx.x; i < p.heads * rest; i += 256) {
+      const int h = i / rest, d = i % rest;
+      if (d < p.dim) list[h * head + d] = src[(size_t)h * p.dk + d];
+      else stf(list + h * head + d + p.rot, 0.f);
+    }
   }
 }
 
@@ -257,16 +263,20 @@ __global__ void __launch_bounds__(128) latent_attn_plain_kernel(const LatentAttn
 }
 
 // ---------------------------------------------------------------------------------------------
-// Decode kernel (bf16, pages of 16) on the tensor cores: one CTA = N query heads of one token over a run of 128-key tiles.
+// Decode kernel (bf16, pages of 16) on the tensor cores: one CTA = N query heads of one token over a run of 64-key tiles.
 // Keys lie on the lanes of the score accumulator and heads on its columns, S[key][head] = row . q', so that a few heads fill
-// a tile whose M side is 128 keys; the weighted sum is O[latent][head] += c^T P with the same shared-memory tile read
+// a product whose M side is the keys; the weighted sum is O[latent][head] += c^T P with the same shared-memory tile read
 // transposed.  Every cached row crosses HBM once per CTA for all of its heads.
-//   shared memory: q' [chunks][N][64], P [2][N][64], the rotated chunk(s) of a tile, a ring of pairs of 64-column chunks of c
-//   (128 keys x 64 columns, 16 KiB each, fetched page by page in swizzled boxes).
-// The maximum is refreshed lazily (a new one must exceed the old by 2^8 to cost a pass over O).
-// Warp roles (192 threads): warp 0 TMA, warp 1 tensor memory + MMA, warps 2..5 one thread per key.  sink in log2 units.
+//   A stage is 64 cached rows as groups of 8 keys, [group][64-column chunk][8 keys][64], one copy per group for the whole
+//   row.  Stages come in pairs: the score product of either stage of a pair runs over the 128 rows of both, so even tiles
+//   have their scores on lanes 0..63 and odd ones on 64..127 (the other half is the neighbour's, whatever it holds, and is
+//   not read), and scores and weights exist twice: the products of a tile run beside the softmax of the one before.
+// Every thread keeps the heads' reference maxima in registers; a tile whose scores stay below 2^8 times them (one vote) needs
+// no reduction, any other goes through a reduction over its keys and a pass over O.
+// Warp roles (192 threads): warp 0 TMA, warp 1 tensor memory + MMA, warps 2..5 softmax - the two warps on a tile's lanes one
+// thread per key, the other two at hand for a pass over O - and epilogue, one thread per latent.  sink in log2 units.
 // ---------------------------------------------------------------------------------------------
-constexpr int LD_PAGE = 16, LD_TILE = 128, LD_CHUNK = LD_TILE * 128, LD_THREADS = 192, LD_MAX_STAGES = 5;
+constexpr int LD_PAGE = 16, LD_TILE = 64, LD_GROUPS = LD_TILE / 8, LD_THREADS = 192, LD_MAX_STAGES = 8;
 constexpr float LD_LOG2E = 1.4426950408889634f;
 
 // Reduce N values per lane over the 32 lanes of a warp: lane x returns the result of column x / (32 / N).
@@ -297,8 +307,22 @@ __device__ __forceinline__ float warp_columns(const float* v, int lane) {
   return a[0];
 }
 
+// barrier of `nthreads` threads that also tells every one of them whether `pred` holds in any
+__device__ __forceinline__ bool named_bar_any(int id, int nthreads, bool pred) {
+  int r;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "setp.ne.b32 p, %3, 0;\n\t"
+      "barrier.cta.red.or.pred q, %1, %2, p;\n\t"
+      "selp.b32 %0, 1, 0, q;\n\t}"
+      : "=r"(r)
+      : "r"(id), "r"(nthreads), "r"((int)pred)
+      : "memory");
+  return r != 0;
+}
+
 struct LatentDecodeShape {
-  int nc, nr, pairs, stages;  // 64-column chunks of c and of r, ceil(nc / 2), ring stages (>= pairs)
+  int nc, chunks, pairs, stages;      // 64-column chunks of c, of the whole row; ceil(nc / 2); ring stages (even)
   int tmem_cols;
 };
 
@@ -307,27 +331,34 @@ __device__ __forceinline__ void tmem_ld_heads(uint32_t addr, float* v) {
   if constexpr (N == 32) tmem_ld32(addr, v);
   else tmem_ld16(addr, v);
 }
+
+// Descriptors of a stage whose 8-key groups are `group` bytes apart: keys x columns (K-major), and the same rows read as
+// columns x keys (MN-major, 64-column chunks 1024 bytes apart).  Adding n to a descriptor moves its start by 16 n bytes.
+__device__ __forceinline__ uint64_t desc_rows(uint32_t addr, uint32_t group) {
+  return (umma_desc_sw128(addr) & ~(static_cast<uint64_t>(0x3FFF) << 32)) | (static_cast<uint64_t>(group >> 4) << 32);
+}
+__device__ __forceinline__ uint64_t desc_columns(uint32_t addr, uint32_t group) {
+  return (umma_desc_mn_sw128(addr, 1024) & ~(static_cast<uint64_t>(0x3FFF) << 32)) | (static_cast<uint64_t>(group >> 4) << 32);
+}
+
 template <int N>
 __global__ void __launch_bounds__(LD_THREADS, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_c, const LatentAttnParams p,
                      const LatentDecodeShape sh) {
   extern __shared__ __align__(1024) uint8_t smem[];
-  constexpr int QCH = N * 128;                               // bytes of one 64-column chunk of q'
-  const int chunks = sh.nc + sh.nr;
+  constexpr int QCH = N * 128;                               // bytes of one 64-column chunk of q', or of the weights of a tile
+  const uint32_t group = sh.chunks * 1024, stage_bytes = LD_GROUPS * group;
   uint8_t* ring = smem;
-  uint8_t* rot_s = ring + sh.stages * 2 * LD_CHUNK;
-  uint8_t* q_s = rot_s + sh.nr * LD_CHUNK;
-  uint8_t* p_s = q_s + chunks * QCH;
-  float* s_max = reinterpret_cast<float*>(p_s + 2 * QCH);    // [4][32]
-  float* s_sum = s_max + 128;                                // [4][32]
+  uint8_t* q_s = ring + sh.stages * stage_bytes;
+  uint8_t* p_s = q_s + sh.chunks * QCH;                      // [2]
+  float* s_max = reinterpret_cast<float*>(p_s + 2 * QCH);    // [2][32]
+  float* s_sum = s_max + 64;                                 // [4][32]
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_sum + 128);
   uint64_t* q_full = bars;
-  uint64_t* rot_full = bars + 1;
-  uint64_t* rot_empty = bars + 2;
-  uint64_t* s_full = bars + 3;
-  uint64_t* p_ready = bars + 4;
-  uint64_t* pv_done = bars + 5;
-  uint64_t* full = bars + 6;                                 // [stages]
+  uint64_t* s_full = bars + 1;                               // [2]
+  uint64_t* p_ready = bars + 3;                              // [2]
+  uint64_t* pv_done = bars + 5;                              // [2]
+  uint64_t* full = bars + 7;                                 // [stages]
   uint64_t* empty = full + LD_MAX_STAGES;                    // [stages]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(empty + LD_MAX_STAGES);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
@@ -340,14 +371,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   }
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    mbar_init(rot_full, 1);
-    mbar_init(rot_empty, 1);
-    mbar_init(s_full, 1);
-    mbar_init(p_ready, 128);
-    mbar_init(pv_done, 1);
+    for (int g = 0; g < 2; ++g) { mbar_init(&s_full[g], 1); mbar_init(&p_ready[g], 128); mbar_init(&pv_done[g], 1); }
     for (int s = 0; s < sh.stages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
     *abort_flag = 0;
     mbar_fence_init();
+    prefetch_tensormap(&tm_q);
+    prefetch_tensormap(&tm_c);
   }
   if (warp == 1) {
     tmem_alloc(tmem_slot, sh.tmem_cols);
@@ -358,7 +387,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   tc_fence_after();
   pdl_launch_dependents();            // only now: a successor must not take the tensor memory first
   pdl_wait();
-  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 32;
+  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 2 * N;
   const int h0 = blockIdx.x * N, t = blockIdx.y, split = blockIdx.z;
   const int i = p.pos[t];
   const int tiles = i / LD_TILE + 1, per = (tiles + p.n_split - 1) / p.n_split;
@@ -367,163 +396,178 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   if (warp == 0) {
     // ---------------- TMA producer ----------------
     if (lane == 0 && n_tiles > 0) {
-      mbar_expect_tx(q_full, chunks * QCH);
-      for (int k = 0; k < chunks; ++k) tma_load_3d(q_s + k * QCH, &tm_q, k * 64, t, h0, q_full);
+      mbar_expect_tx(q_full, sh.chunks * QCH);
+      for (int k = 0; k < sh.chunks; ++k) tma_load_3d(q_s + k * QCH, &tm_q, k * 64, t, h0, q_full);
       const int* pt = p.page_table + (size_t)p.row[t] * p.max_pages;
       const int last_page = i / LD_PAGE;
-      int g = 0;
-      for (int n = 0; n < n_tiles && !*abort_flag; ++n) {
-        int page[8];
+      for (int n = 0; n < n_tiles; ++n) {
+        const int st = n % sh.stages;
+        int page[4];
 #pragma unroll
-        for (int u = 0; u < 8; ++u) {
-          const int a = (tb + n) * 8 + u;
-          page[u] = a <= last_page ? pt[a] : p.n_pages;      // an index past the pool reads zeros
+        for (int u = 0; u < 4; ++u) {
+          const int a = (tb + n) * 4 + u;
+          page[u] = a <= last_page ? pt[a] : p.n_pages;      // rows past the pool read as zeros
         }
-        mbar_wait(rot_empty, (n & 1) ^ 1, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
+        mbar_wait(&empty[st], ((n / sh.stages) & 1) ^ 1, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
         if (*abort_flag) break;
-        mbar_expect_tx(rot_full, sh.nr * LD_CHUNK);
-        for (int k = 0; k < sh.nr; ++k)
+        mbar_expect_tx(&full[st], stage_bytes);
 #pragma unroll
-          for (int u = 0; u < 8; ++u) tma_load_3d(rot_s + k * LD_CHUNK + u * 2048, &tm_c, p.Rp + k * 64, 0, page[u], rot_full);
-        for (int q = 0; q < sh.pairs; ++q, ++g) {
-          const int st = g % sh.stages;
-          mbar_wait(&empty[st], ((g / sh.stages) & 1) ^ 1, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
-          if (*abort_flag) break;
-          const int cols = min(2, sh.nc - 2 * q);
-          mbar_expect_tx(&full[st], cols * LD_CHUNK);
-          for (int k = 0; k < cols; ++k)
-#pragma unroll
-            for (int u = 0; u < 8; ++u)
-              tma_load_3d(ring + (st * 2 + k) * LD_CHUNK + u * 2048, &tm_c, (2 * q + k) * 64, 0, page[u], &full[st]);
-        }
+        for (int u = 0; u < LD_GROUPS; ++u)
+          tma_load_3d(ring + st * stage_bytes + u * group, &tm_c, 0, page[u / 2] * LD_PAGE + (u & 1) * 8, 0, &full[st]);
       }
     }
     __syncwarp();
   } else if (warp == 1) {
-    // ---------------- MMA issuer ----------------
+    // ---------------- MMA issuer: scores of tile n, then the weighted sum of tile n - 1 ----------------
     if (lane == 0 && n_tiles > 0) {
       constexpr uint32_t idesc_s = umma_idesc_bf16(128, N);
       constexpr uint32_t idesc_o = umma_idesc_bf16(128, N) | (1u << 15);     // A (c) read transposed
-      const uint32_t q_addr = smem_u32(q_s), p_addr = smem_u32(p_s), ring_addr = smem_u32(ring), rot_addr = smem_u32(rot_s);
+      const uint64_t rows0 = desc_rows(smem_u32(ring), group), cols0 = desc_columns(smem_u32(ring), group);
+      const uint64_t q0 = umma_desc_sw128(smem_u32(q_s)), w0 = umma_desc_sw128(smem_u32(p_s));
+      const uint32_t stage16 = stage_bytes >> 4, group16 = group >> 4;
       mbar_wait(q_full, 0, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
-      int g = 0;
-      for (int n = 0; n < n_tiles && !*abort_flag; ++n) {
-        mbar_wait(rot_full, n & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
-        tc_fence_after();
-        for (int k = 0; k < sh.nr; ++k)
-#pragma unroll
-          for (int ks = 0; ks < 4; ++ks)
-            umma_bf16(tmem_s, umma_desc_sw128(rot_addr + k * LD_CHUNK + ks * 32), umma_desc_sw128(q_addr + (sh.nc + k) * QCH + ks * 32),
-                      idesc_s, (k > 0 || ks > 0) ? 1u : 0u);
-        umma_commit(rot_empty);
-        for (int q = 0; q < sh.pairs; ++q) {
-          const int gi = g + q, st = gi % sh.stages;
-          mbar_wait(&full[st], (gi / sh.stages) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
+      for (int n = 0; n <= n_tiles && !*abort_flag; ++n) {
+        if (n < n_tiles) {
+          const int st = n % sh.stages;
+          mbar_wait(&full[st], (n / sh.stages) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
           tc_fence_after();
-          const int cols = min(2, sh.nc - 2 * q);
-          for (int k = 0; k < cols; ++k)
+          uint64_t a = rows0 + (st & ~1) * stage16, b = q0;
+          const uint32_t d = tmem_s + (n & 1) * N;
+          uint32_t acc = 0u;
+#pragma unroll 3
+          for (int k = 0; k < sh.chunks; ++k, a += 64, b += QCH / 16) {
 #pragma unroll
-            for (int ks = 0; ks < 4; ++ks)
-              umma_bf16(tmem_s, umma_desc_sw128(ring_addr + (st * 2 + k) * LD_CHUNK + ks * 32),
-                        umma_desc_sw128(q_addr + (2 * q + k) * QCH + ks * 32), idesc_s, 1u);
+            for (int ks = 0; ks < 4; ++ks) {
+              umma_bf16(d, a + 2 * ks, b + 2 * ks, idesc_s, acc);
+              acc = 1u;
+            }
+          }
+          umma_commit(&s_full[n & 1]);
         }
-        umma_commit(s_full);
-        mbar_wait(p_ready, n & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
-        tc_fence_after();
-        for (int q = 0; q < sh.pairs; ++q) {
-          const int gi = g + q, st = gi % sh.stages;
-          // the second chunk of an odd last pair holds old bytes: they only reach lanes 64.. of its block, which nobody reads
+        if (n > 0) {
+          const int m = n - 1, st = m % sh.stages;
+          mbar_wait(&p_ready[m & 1], (m >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+          tc_fence_after();
+          uint64_t a = cols0 + st * stage16;
+          const uint64_t w = w0 + (m & 1) * (QCH / 16);
+          // an odd last pair takes in the chunk behind c as well: its sums lie on lanes that nobody reads
+#pragma unroll 2
+          for (int q = 0; q < sh.pairs; ++q, a += 128) {
 #pragma unroll
-          for (int ks = 0; ks < LD_TILE / 16; ++ks)
-            umma_bf16(tmem_o + q * N, umma_desc_mn_sw128(ring_addr + st * 2 * LD_CHUNK + ks * 2048, LD_CHUNK),
-                      umma_desc_sw128(p_addr + (ks / 4) * QCH + (ks % 4) * 32), idesc_o, (n > 0 || ks > 0) ? 1u : 0u);
+            for (int ks = 0; ks < LD_TILE / 16; ++ks)
+              umma_bf16(tmem_o + q * N, a + ks * 2 * group16, w + 2 * ks, idesc_o, (m > 0 || ks > 0) ? 1u : 0u);
+          }
           umma_commit(&empty[st]);
+          umma_commit(&pv_done[m & 1]);
         }
-        umma_commit(pv_done);
-        g += sh.pairs;
       }
     }
     __syncwarp();
   } else {
-    // ---------------- softmax / epilogue: one thread per key, then one per latent ----------------
-    const int qd = warp & 3, key = qd * 32 + lane;
+    // ---------------- softmax / epilogue ----------------
+    const int qd = warp & 3, key = (qd & 1) * 32 + lane;
     const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
     const float sc = p.scale * LD_LOG2E;
-    float m_ref = -INFINITY;                                 // of head `lane` (lanes below N), the same in every warp
-    float sum[N];
+    float m[N], sum[N];                                      // reference maxima, the same in every thread; weights of its keys
 #pragma unroll
-    for (int c = 0; c < N; ++c) sum[c] = 0.f;
+    for (int c = 0; c < N; ++c) { m[c] = -INFINITY; sum[c] = 0.f; }
     for (int n = 0; n < n_tiles; ++n) {
-      const int j = (tb + n) * LD_TILE + key;
-      mbar_wait(s_full, n & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
-      __syncwarp();
-      tc_fence_after();
+      const int g = n & 1;
+      const bool active = (qd >> 1) == g;                    // this warp's lanes hold the tile's keys
       float v[N];
-      tmem_ld_heads<N>(tmem_s + lane_off, v);
-      tmem_ld_wait();
+      bool over = false;
+      if (active) {
+        mbar_wait(&s_full[g], (n >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+        __syncwarp();
+        tc_fence_after();
+        tmem_ld_heads<N>(tmem_s + g * N + lane_off, v);
+        tmem_ld_wait();
+        tc_fence_before();
+        const bool seen = (tb + n) * LD_TILE + key <= i;
 #pragma unroll
-      for (int c = 0; c < N; ++c) v[c] = j <= i ? v[c] * sc : -INFINITY;
-      const float wm = warp_columns<N, true>(v, lane);
-      s_max[(n & 1) * 128 + qd * 32 + lane] = wm;            // s_max and s_sum take turns as the exchange buffer
-      tc_fence_before();
-      named_bar_sync(1, 128);
-      float f = 1.0f;
-      if (lane < N) {
-        const float* x = s_max + (n & 1) * 128 + lane * (32 / N);
-        const float mx = fmaxf(fmaxf(x[0], x[32]), fmaxf(x[64], x[96]));
-        if (mx > m_ref + 8.0f) {
-          f = m_ref == -INFINITY ? 1.0f : exp2f(m_ref - mx);
-          m_ref = mx;
+        for (int c = 0; c < N; ++c) {
+          v[c] = seen ? v[c] * sc : -INFINITY;
+          over = over || v[c] > m[c] + 8.0f;
         }
       }
-      if (n > 0) mbar_wait(pv_done, (n - 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
-      __syncwarp();
-      tc_fence_after();
-      if (n > 0 && __any_sync(0xffffffffu, f != 1.0f)) {
-        for (int q = 0; q < sh.pairs; ++q) {
-          float o[N];
-          tmem_ld_heads<N>(tmem_o + lane_off + q * N, o);
-          tmem_ld_wait();
+      if (named_bar_any(1, 128, over)) {                     // some head's maximum grows: reduce, and rescale what is there
+        if (active) s_max[(qd & 1) * 32 + lane] = warp_columns<N, true>(v, lane);
+        named_bar_sync(1, 128);
+        float f[N];
+        bool any = false;
 #pragma unroll
-          for (int c = 0; c < N; ++c) o[c] *= __shfl_sync(0xffffffffu, f, c);
-#pragma unroll
-          for (int c = 0; c < N; ++c) tmem_st1(tmem_o + lane_off + q * N + c, o[c]);
+        for (int c = 0; c < N; ++c) {
+          const float mx = fmaxf(s_max[c * (32 / N)], s_max[32 + c * (32 / N)]);
+          const bool grow = mx > m[c] + 8.0f;
+          f[c] = grow && m[c] != -INFINITY ? exp2f(m[c] - mx) : 1.0f;
+          any = any || f[c] != 1.0f;
+          if (grow) m[c] = mx;
+          sum[c] *= f[c];
         }
-        tmem_st_wait();
+        if (n > 0 && any) {                                  // the same in all threads
+          mbar_wait(&pv_done[g ^ 1], ((n - 1) >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+          __syncwarp();
+          tc_fence_after();
+          for (int q = 0; q < sh.pairs; ++q) {
+            float o[N];
+            tmem_ld_heads<N>(tmem_o + lane_off + q * N, o);
+            tmem_ld_wait();
 #pragma unroll
-        for (int c = 0; c < N; ++c) sum[c] *= __shfl_sync(0xffffffffu, f, c);
+            for (int c = 0; c < N; ++c) tmem_st1(tmem_o + lane_off + q * N + c, o[c] * f[c]);
+          }
+          tmem_st_wait();
+          tc_fence_before();
+        }
+        named_bar_sync(1, 128);                              // s_max is read
       }
-      uint8_t* pd = p_s + (key >> 6) * QCH + (key & 7) * 2;
+      if (active) {
+        if (n > 1) mbar_wait(&pv_done[g], ((n - 2) >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);     // its weights are read
+        uint8_t* pd = p_s + g * QCH + (key & 7) * 2;
 #pragma unroll
-      for (int c = 0; c < N; ++c) {
-        const float m = __shfl_sync(0xffffffffu, m_ref, c);
-        const float w = j <= i ? ex2_approx(v[c] - m) : 0.f;
-        sum[c] += w;
-        *reinterpret_cast<__nv_bfloat16*>(pd + c * 128 + ((((key & 63) >> 3) ^ (c & 7)) << 4)) = __float2bfloat16_rn(w);
+        for (int c = 0; c < N; ++c) {
+          const float w = ex2_approx(v[c] - m[c]);           // 0 for a key that is not seen
+          sum[c] += w;
+          *reinterpret_cast<__nv_bfloat16*>(pd + c * 128 + (((key >> 3) ^ (c & 7)) << 4)) = __float2bfloat16_rn(w);
+        }
+        fence_proxy_async_smem();
       }
-      fence_proxy_async_smem();
-      tc_fence_before();
-      mbar_arrive(p_ready);
+      mbar_arrive(&p_ready[g]);
     }
     // denominators: over the keys of every warp
-    const float ws = warp_columns<N, false>(sum, lane);
+    s_sum[qd * 32 + lane] = warp_columns<N, false>(sum, lane);
     named_bar_sync(1, 128);
-    s_sum[qd * 32 + lane] = ws;
-    named_bar_sync(1, 128);
-    float den = 0.f, f = 0.f;
-    if (lane < N) {
-      const float* x = s_sum + lane * (32 / N);
-      den = x[0] + x[32] + x[64] + x[96];
-      f = den > 0.f ? 1.0f / den : 0.f;
-      if (p.n_split == 1 && p.sink != nullptr && h0 + lane < p.heads) {
-        const float sk = p.sink[h0 + lane], top = fmaxf(m_ref, sk), e = exp2f(m_ref - top);
-        f = e / (den * e + exp2f(sk - top));
-      }
+    float den[N];
+#pragma unroll
+    for (int c = 0; c < N; ++c) {
+      const float* x = s_sum + c * (32 / N);
+      den[c] = x[0] + x[32] + x[64] + x[96];
     }
-    if (n_tiles > 0) mbar_wait(pv_done, (n_tiles - 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+    if (n_tiles > 0) mbar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
     __syncwarp();
     tc_fence_after();
     const int stride = p.Rp + 2;
+    if (p.n_split > 1) {
+      if (threadIdx.x == 64) {
+#pragma unroll
+        for (int c = 0; c < N; ++c) {
+          if (h0 + c < p.heads) {
+            float* w = p.ws + (((size_t)t * p.heads + h0 + c) * p.n_split + split) * stride + p.Rp;
+            w[0] = m[c];
+            w[1] = den[c];
+          }
+        }
+      }
+    } else {
+#pragma unroll
+      for (int c = 0; c < N; ++c) {
+        float f = 1.0f / den[c];
+        if (p.sink != nullptr && h0 + c < p.heads) {
+          const float sk = p.sink[h0 + c], top = fmaxf(m[c], sk), e = exp2f(m[c] - top);
+          f = e / (den[c] * e + exp2f(sk - top));
+        }
+        den[c] = f;
+      }
+    }
     for (int q = 0; q < sh.pairs; ++q) {
       float o[N];
       if (n_tiles > 0) {
@@ -533,22 +577,17 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
 #pragma unroll
         for (int c = 0; c < N; ++c) o[c] = 0.f;
       }
-      const int d = q * 128 + key;
+      const int d = q * 128 + qd * 32 + lane;
+      if (d >= p.Rp) continue;                               // Rp is a multiple of 64: whole warps
 #pragma unroll
       for (int c = 0; c < N; ++c) {
-        const float inv = __shfl_sync(0xffffffffu, f, c);
-        if (d < p.Rp && h0 + c < p.heads) {
+        if (h0 + c < p.heads) {
           if (p.n_split == 1)
-            reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)(h0 + c) * p.npad + t) * p.Rp + d] = __float2bfloat16_rn(o[c] * inv);
+            reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)(h0 + c) * p.npad + t) * p.Rp + d] = __float2bfloat16_rn(o[c] * den[c]);
           else
             p.ws[(((size_t)t * p.heads + h0 + c) * p.n_split + split) * stride + d] = o[c];
         }
       }
-    }
-    if (p.n_split > 1 && qd == 0 && lane < N && h0 + lane < p.heads) {
-      float* w = p.ws + (((size_t)t * p.heads + h0 + lane) * p.n_split + split) * stride + p.Rp;
-      w[0] = m_ref;
-      w[1] = den;
     }
     tc_fence_before();
   }
@@ -559,31 +598,43 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   }
 }
 
-// o = sum over the splits, each against the common maximum; one CTA per (token, head)
+// o = sum over the splits, each against the common maximum: grid (token x head, ceil(Rp / 128)), one latent per thread
 __global__ void __launch_bounds__(128) latent_decode_merge_kernel(const LatentAttnParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x / p.heads, h = blockIdx.x % p.heads, stride = p.Rp + 2;
+  __shared__ float s_w[64];
+  const int h = blockIdx.x % p.heads, t = blockIdx.x / p.heads, stride = p.Rp + 2;
   const float* w = p.ws + (size_t)blockIdx.x * p.n_split * stride;
-  float mx = -INFINITY, den = 0.f;
-  for (int s = 0; s < p.n_split; ++s) mx = fmaxf(mx, w[s * stride + p.Rp]);
-  if (p.sink != nullptr) {
-    mx = fmaxf(mx, p.sink[h]);
-    den = exp2f(p.sink[h] - mx);
-  }
-  for (int s = 0; s < p.n_split; ++s) {
-    const float ms = w[s * stride + p.Rp];
-    if (ms != -INFINITY) den += exp2f(ms - mx) * w[s * stride + p.Rp + 1];
-  }
-  const float f = den > 0.f ? 1.0f / den : 0.f;
-  for (int d = threadIdx.x; d < p.Rp; d += 128) {
-    float num = 0.f;
-    for (int s = 0; s < p.n_split; ++s) {
-      const float ms = w[s * stride + p.Rp];
-      if (ms != -INFINITY) num += exp2f(ms - mx) * w[s * stride + d];
+  if (threadIdx.x < 32) {                        // up to 64 splits, two per lane
+    const int lane = threadIdx.x;
+    float m[2], l[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int s = lane + 32 * u;
+      m[u] = s < p.n_split ? w[s * stride + p.Rp] : -INFINITY;
+      l[u] = s < p.n_split ? w[s * stride + p.Rp + 1] : 0.f;
     }
-    reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)h * p.npad + t) * p.Rp + d] = __float2bfloat16_rn(num * f);
+    float mx = warp_max(fmaxf(m[0], m[1]));
+    if (p.sink != nullptr) mx = fmaxf(mx, p.sink[h]);
+    float e[2], den = 0.f;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      e[u] = m[u] != -INFINITY ? exp2f(m[u] - mx) : 0.f;
+      den += e[u] * l[u];
+    }
+    den = warp_sum(den);
+    if (p.sink != nullptr) den += exp2f(p.sink[h] - mx);
+    const float f = den > 0.f ? 1.0f / den : 0.f;
+    s_w[lane] = e[0] * f;
+    s_w[lane + 32] = e[1] * f;
   }
+  __syncthreads();
+  const int d = blockIdx.y * 128 + threadIdx.x;
+  if (d >= p.Rp) return;
+  float num = 0.f;
+#pragma unroll 8
+  for (int s = 0; s < p.n_split; ++s) num = fmaf(s_w[s], w[s * stride + d], num);      // an empty split holds zeros
+  reinterpret_cast<__nv_bfloat16*>(p.out)[((size_t)h * p.npad + t) * p.Rp + d] = __float2bfloat16_rn(num);
 }
 
 // bf16 3-D tensor, 64-element inner boxes with the 128-byte swizzle
@@ -600,22 +651,21 @@ static int map_3d(CUtensorMap* m, const void* base, cuuint64_t d0, cuuint64_t d1
   return r == CUDA_SUCCESS ? 0 : -3;
 }
 
-// Ring geometry for N heads per CTA; false when a tile does not fit.
+// Ring geometry for N heads per CTA; false when two stages do not fit.
 template <int N>
 static bool latent_decode_shape(int Rp, int rw, LatentDecodeShape* sh, size_t* smem) {
   sh->nc = Rp / 64;
-  sh->nr = (rw + 63) / 64;
+  sh->chunks = (Rp + rw) / 64;
   sh->pairs = (sh->nc + 1) / 2;
-  const size_t fixed = (size_t)sh->nr * LD_CHUNK + (size_t)(sh->nc + sh->nr + 2) * N * 128 + 2048;
-  const size_t cap = 227 * 1024;
-  if (fixed >= cap) return false;
-  sh->stages = (int)((cap - fixed) / (2 * LD_CHUNK));
+  const size_t stage = (size_t)LD_GROUPS * sh->chunks * 1024, fixed = (size_t)(sh->chunks + 2) * N * 128 + 2048, cap = 227 * 1024;
+  if (rw % 64 || fixed + 2 * stage > cap) return false;
+  sh->stages = (int)((cap - fixed) / stage) & ~1;
   if (sh->stages > LD_MAX_STAGES) sh->stages = LD_MAX_STAGES;
   int cols = 32;
-  while (cols < 32 + sh->pairs * N) cols *= 2;
+  while (cols < (2 + sh->pairs) * N) cols *= 2;
   sh->tmem_cols = cols;
-  *smem = fixed + (size_t)sh->stages * 2 * LD_CHUNK;
-  return sh->stages >= sh->pairs && cols <= 512;
+  *smem = fixed + (size_t)sh->stages * stage;
+  return cols <= 512;
 }
 
 template <int N>
@@ -632,9 +682,10 @@ static int launch_latent_decode(const LatentAttnParams& p, cudaStream_t stream) 
   CUtensorMap mq, mc;
   int rc;
   if ((rc = map_3d(&mq, p.q, p.lq, p.npad, p.heads, p.lq, (cuuint64_t)p.npad * p.lq, 1, N))) return rc;
-  if ((rc = map_3d(&mc, p.cache, len, LD_PAGE, p.n_pages, len, (cuuint64_t)LD_PAGE * len, LD_PAGE, 1))) return rc;
+  // the pool as [tokens][chunks of 64 columns], in boxes of 8 tokens x the whole row that land chunk by chunk
+  if ((rc = map_3d(&mc, p.cache, 64, (cuuint64_t)LD_PAGE * p.n_pages, sh.chunks, len, 64, 8, sh.chunks))) return rc;
   cudaError_t e = launch_chain(latent_decode_kernel<N>, dim3((p.heads + N - 1) / N, p.n, p.n_split), dim3(LD_THREADS), smem, stream, mq, mc, p, sh);
-  if (e == cudaSuccess && p.n_split > 1) e = launch_chain(latent_decode_merge_kernel, dim3(p.n * p.heads), dim3(128), 0, stream, p);
+  if (e == cudaSuccess && p.n_split > 1) e = launch_chain(latent_decode_merge_kernel, dim3(p.n * p.heads, (p.Rp + 127) / 128), dim3(128), 0, stream, p);
   return e == cudaSuccess ? 0 : -3;
 }
 
@@ -653,10 +704,8 @@ extern "C" int tahb_latent_post(const LatentPostParams* p, int f32, cudaStream_t
 extern "C" int tahb_latent_query(const LatentQueryParams* p, int f32, cudaStream_t stream) {
   if (p->n <= 0) return 0;
   if (p->rot % 2 || p->dim + p->rot > p->dk || p->dk > p->dq || p->n_list > p->npad) return -2;
-  const long long warps = (long long)p->n * p->heads;
-  const dim3 grid((unsigned)((warps + 3) / 4));
-  cudaError_t e = f32 ? launch_chain(latent_query_kernel<float>, grid, dim3(128), 0, stream, *p)
-                      : launch_chain(latent_query_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, *p);
+  cudaError_t e = f32 ? launch_chain(latent_query_kernel<float>, dim3(p->n), dim3(256), 0, stream, *p)
+                      : launch_chain(latent_query_kernel<__nv_bfloat16>, dim3(p->n), dim3(256), 0, stream, *p);
   return e == cudaSuccess ? 0 : -3;
 }
 

@@ -1161,6 +1161,9 @@ extern "C" int tahb_window_attn_tiles(const WindowAttnParams* p, const int* q0, 
   }
   WindowTiles tl{q0, qn, n_pages, kv_ld};
   const int hk = p->dk <= 64 ? 1 : p->dk <= 128 ? 2 : 4, hv = p->dv <= 64 ? 1 : p->dv <= 128 ? 2 : 4;
+  if (p->softcap == 0.f && p->dk > 128 && p->dk <= 192 && p->dv <= 128)
+    return p->dv <= 64 ? launch_window_prefill_as<3, 1, false>(mq, mk, mv, *p, tl, n_tiles, stream)
+                       : launch_window_prefill_as<3, 2, false>(mq, mk, mv, *p, tl, n_tiles, stream);
   if (hk == 4 || hv == 4) return launch_window_prefill<4, 4>(mq, mk, mv, *p, tl, n_tiles, stream);
   if (hk == 2) return hv == 2 ? launch_window_prefill<2, 2>(mq, mk, mv, *p, tl, n_tiles, stream)
                               : launch_window_prefill<2, 1>(mq, mk, mv, *p, tl, n_tiles, stream);

@@ -66,7 +66,7 @@ class AttentionLayer:
 
 @dataclass
 class LatentLayer:
-    """Latent attention.  Cached row: ``[c: Rp columns | rotated part: rw]``; head lists and expansions also carry the rotated
+    """Latent attention.  Cached row: ``[c: Rp columns | rotated part: rw]``, both multiples of 64; head lists and expansions also carry the rotated
     part through their matrix products, by unit rows."""
     spec: LatentAttentionSpec
     dk: int                       # a head's query / key, dim + rot_dim padded to 8
@@ -81,9 +81,9 @@ class LatentLayer:
     q_norm: torch.Tensor
     c_norm: torch.Tensor
     w_uq: torch.Tensor            # [heads * dk, Qp]
-    w_abs: torch.Tensor           # [heads, row of the cache padded to 64, dk padded to 64]: query -> query against cached rows
+    w_abs: torch.Tensor           # [heads, row of the cache, dk padded to 64]: query -> query against cached rows
     w_uv: torch.Tensor            # [heads, dv padded to 64, Rp]: weighted c -> value
-    w_exp: Optional[torch.Tensor]             # [heads * dk + heads * dv, row padded to 64]: cached rows -> keys and values
+    w_exp: Optional[torch.Tensor]             # [heads * dk + heads * dv, row of the cache]: cached rows -> keys and values
     w_o: torch.Tensor
     sink: torch.Tensor            # natural units for the plain kernel, log2 units for the others
     sink_log2: torch.Tensor
@@ -328,8 +328,8 @@ class HybridWeights:
     def _latent(self, x, m, dk, dv, w_o, dtype, plain, T, mat, stack, heads_rows) -> LatentLayer:
         H, d, r, R = m.heads, m.dim, m.rot_dim, m.kv_rank
         dev = self.embed.device
-        Qp, Rp, rw = _pad(m.q_rank, 64), _pad(R, 64), _pad(r, 8)
-        lp, dkv, unit = _pad(Rp + rw, 64), T(x + "dkv"), torch.arange(r, device=dev)
+        Qp, Rp, rw = _pad(m.q_rank, 64), _pad(R, 64), _pad(r, 64)
+        lp, dkv, unit = Rp + rw, T(x + "dkv"), torch.arange(r, device=dev)
         w_in = stack([mat(T(x + "dq"), Qp, self.Wp), mat(dkv[:R], Rp, self.Wp), mat(dkv[R:], rw, self.Wp),
                       heads_rows(T(x + "g"), H, m.vdim, dv)])
         w_uq = torch.zeros(H, dk, Qp, dtype=dtype, device=dev)
