@@ -263,20 +263,22 @@ __global__ void __launch_bounds__(128) latent_attn_plain_kernel(const LatentAttn
 }
 
 // ---------------------------------------------------------------------------------------------
-// Decode kernel (bf16, pages of 16) on the tensor cores: one CTA = N query heads of one token over a run of 64-key tiles.
+// Decode kernel (bf16, pages of 16) on the tensor cores: one CTA = N query heads of one token over a run of 48-key tiles.
 // Keys lie on the lanes of the score accumulator and heads on its columns, S[key][head] = row . q', so that a few heads fill
 // a product whose M side is the keys; the weighted sum is O[latent][head] += c^T P with the same shared-memory tile read
 // transposed.  Every cached row crosses HBM once per CTA for all of its heads.
-//   A stage is 64 cached rows as groups of 8 keys, [group][64-column chunk][8 keys][64], one copy per group for the whole
-//   row.  Stages come in pairs: the score product of either stage of a pair runs over the 128 rows of both, so even tiles
-//   have their scores on lanes 0..63 and odd ones on 64..127 (the other half is the neighbour's, whatever it holds, and is
-//   not read), and scores and weights exist twice: the products of a tile run beside the softmax of the one before.
+//   A stage is 48 cached rows as groups of 8 keys, [group][64-column chunk][8 keys][64], one copy per group for the whole
+//   row.  The score product has M = 64 rows, 16 on the lanes of each warp; its last 16 are whatever follows the stage and
+//   are not read.  Three stages of a 512 + 64 row fit, two of them on their way while one is at work; scores and weights
+//   exist twice, so that the score product of a tile runs beside the softmax of the one before.
+//   The products are short (few heads), so their issue rate matters: the whole MMA warp walks the loop, which keeps the
+//   descriptors in uniform registers, and one elected lane issues (42 instead of 57 cycles a product).
 // Every thread keeps the heads' reference maxima in registers; a tile whose scores stay below 2^8 times them (one vote) needs
 // no reduction, any other goes through a reduction over its keys and a pass over O.
-// Warp roles (192 threads): warp 0 TMA, warp 1 tensor memory + MMA, warps 2..5 softmax - the two warps on a tile's lanes one
-// thread per key, the other two at hand for a pass over O - and epilogue, one thread per latent.  sink in log2 units.
+// Warp roles (192 threads): warp 0 TMA, warp 1 tensor memory + MMA, warps 2..5 softmax, 16 lanes of each a key, and epilogue,
+// one thread per latent.  sink in log2 units.
 // ---------------------------------------------------------------------------------------------
-constexpr int LD_PAGE = 16, LD_TILE = 64, LD_GROUPS = LD_TILE / 8, LD_THREADS = 192, LD_MAX_STAGES = 8;
+constexpr int LD_PAGE = 16, LD_TILE = 48, LD_GROUPS = LD_TILE / 8, LD_THREADS = 192, LD_MAX_STAGES = 8;
 constexpr float LD_LOG2E = 1.4426950408889634f;
 
 // Reduce N values per lane over the 32 lanes of a warp: lane x returns the result of column x / (32 / N).
@@ -322,7 +324,7 @@ __device__ __forceinline__ bool named_bar_any(int id, int nthreads, bool pred) {
 }
 
 struct LatentDecodeShape {
-  int nc, chunks, pairs, stages;      // 64-column chunks of c, of the whole row; ceil(nc / 2); ring stages (even)
+  int nc, chunks, pairs, stages;      // 64-column chunks of c, of the whole row; ceil(nc / 2); ring stages
   int tmem_cols;
 };
 
@@ -341,6 +343,17 @@ __device__ __forceinline__ uint64_t desc_columns(uint32_t addr, uint32_t group) 
   return (umma_desc_mn_sw128(addr, 1024) & ~(static_cast<uint64_t>(0x3FFF) << 32)) | (static_cast<uint64_t>(group >> 4) << 32);
 }
 
+// As umma_bf16, by a whole warp in step: one elected lane issues.
+__device__ __forceinline__ void umma_bf16_elect(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+      ::"r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+
 template <int N>
 __global__ void __launch_bounds__(LD_THREADS, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_c, const LatentAttnParams p,
@@ -351,8 +364,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   uint8_t* ring = smem;
   uint8_t* q_s = ring + sh.stages * stage_bytes;
   uint8_t* p_s = q_s + sh.chunks * QCH;                      // [2]
-  float* s_max = reinterpret_cast<float*>(p_s + 2 * QCH);    // [2][32]
-  float* s_sum = s_max + 64;                                 // [4][32]
+  float* s_max = reinterpret_cast<float*>(p_s + 2 * QCH);    // [4][32]
+  float* s_sum = s_max + 128;                                // [4][32]
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_sum + 128);
   uint64_t* q_full = bars;
   uint64_t* s_full = bars + 1;                               // [2]
@@ -362,7 +375,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   uint64_t* empty = full + LD_MAX_STAGES;                    // [stages]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(empty + LD_MAX_STAGES);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
   if ((smem_u32(smem) & 1023u) != 0) {                       // the swizzled tiles need a 1024-byte aligned base
     pdl_launch_dependents();
     pdl_wait();
@@ -387,9 +400,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   tc_fence_after();
   pdl_launch_dependents();            // only now: a successor must not take the tensor memory first
   pdl_wait();
-  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 2 * N;
+  const uint32_t tmem_s = __shfl_sync(0xffffffffu, *tmem_slot, 0), tmem_o = tmem_s + 2 * N;
   const int h0 = blockIdx.x * N, t = blockIdx.y, split = blockIdx.z;
-  const int i = p.pos[t];
+  const int i = __shfl_sync(0xffffffffu, p.pos[t], 0);
   const int tiles = i / LD_TILE + 1, per = (tiles + p.n_split - 1) / p.n_split;
   const int tb = split * per, te = min(tiles, tb + per), n_tiles = max(0, te - tb);
 
@@ -400,72 +413,82 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       for (int k = 0; k < sh.chunks; ++k) tma_load_3d(q_s + k * QCH, &tm_q, k * 64, t, h0, q_full);
       const int* pt = p.page_table + (size_t)p.row[t] * p.max_pages;
       const int last_page = i / LD_PAGE;
+      int st = 0, ph = 1;
       for (int n = 0; n < n_tiles; ++n) {
-        const int st = n % sh.stages;
-        int page[4];
+        int page[LD_TILE / LD_PAGE];
 #pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          const int a = (tb + n) * 4 + u;
+        for (int u = 0; u < LD_TILE / LD_PAGE; ++u) {
+          const int a = (tb + n) * (LD_TILE / LD_PAGE) + u;
           page[u] = a <= last_page ? pt[a] : p.n_pages;      // rows past the pool read as zeros
         }
-        mbar_wait(&empty[st], ((n / sh.stages) & 1) ^ 1, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
+        mbar_wait(&empty[st], ph, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
         if (*abort_flag) break;
         mbar_expect_tx(&full[st], stage_bytes);
 #pragma unroll
         for (int u = 0; u < LD_GROUPS; ++u)
           tma_load_3d(ring + st * stage_bytes + u * group, &tm_c, 0, page[u / 2] * LD_PAGE + (u & 1) * 8, 0, &full[st]);
+        if (++st == sh.stages) { st = 0; ph ^= 1; }
       }
     }
     __syncwarp();
   } else if (warp == 1) {
-    // ---------------- MMA issuer: scores of tile n, then the weighted sum of tile n - 1 ----------------
-    if (lane == 0 && n_tiles > 0) {
-      constexpr uint32_t idesc_s = umma_idesc_bf16(128, N);
+    // ---------------- MMA issuer (whole warp): scores of tile n, then the weighted sum of tile n - 1 ----------------
+    if (n_tiles > 0) {
+      constexpr uint32_t idesc_s = umma_idesc_bf16(64, N);
       constexpr uint32_t idesc_o = umma_idesc_bf16(128, N) | (1u << 15);     // A (c) read transposed
       const uint64_t rows0 = desc_rows(smem_u32(ring), group), cols0 = desc_columns(smem_u32(ring), group);
       const uint64_t q0 = umma_desc_sw128(smem_u32(q_s)), w0 = umma_desc_sw128(smem_u32(p_s));
       const uint32_t stage16 = stage_bytes >> 4, group16 = group >> 4;
       mbar_wait(q_full, 0, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
-      for (int n = 0; n <= n_tiles && !*abort_flag; ++n) {
+      __syncwarp();
+      int st = 0, ph = 0, prev = 0;
+      for (int n = 0; n <= n_tiles; ++n) {                   // after an abort every wait returns at once
         if (n < n_tiles) {
-          const int st = n % sh.stages;
-          mbar_wait(&full[st], (n / sh.stages) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
+          mbar_wait(&full[st], ph, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
+          __syncwarp();
           tc_fence_after();
-          uint64_t a = rows0 + (st & ~1) * stage16, b = q0;
+          uint64_t a = rows0 + st * stage16, b = q0;
           const uint32_t d = tmem_s + (n & 1) * N;
           uint32_t acc = 0u;
 #pragma unroll 3
           for (int k = 0; k < sh.chunks; ++k, a += 64, b += QCH / 16) {
 #pragma unroll
             for (int ks = 0; ks < 4; ++ks) {
-              umma_bf16(d, a + 2 * ks, b + 2 * ks, idesc_s, acc);
+              umma_bf16_elect(d, a + 2 * ks, b + 2 * ks, idesc_s, acc);
               acc = 1u;
             }
           }
-          umma_commit(&s_full[n & 1]);
+          if (elect_one()) umma_commit(&s_full[n & 1]);
+          __syncwarp();
         }
         if (n > 0) {
-          const int m = n - 1, st = m % sh.stages;
+          const int m = n - 1;
           mbar_wait(&p_ready[m & 1], (m >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+          __syncwarp();
           tc_fence_after();
-          uint64_t a = cols0 + st * stage16;
+          uint64_t a = cols0 + prev * stage16;
           const uint64_t w = w0 + (m & 1) * (QCH / 16);
           // an odd last pair takes in the chunk behind c as well: its sums lie on lanes that nobody reads
 #pragma unroll 2
           for (int q = 0; q < sh.pairs; ++q, a += 128) {
 #pragma unroll
             for (int ks = 0; ks < LD_TILE / 16; ++ks)
-              umma_bf16(tmem_o + q * N, a + ks * 2 * group16, w + 2 * ks, idesc_o, (m > 0 || ks > 0) ? 1u : 0u);
+              umma_bf16_elect(tmem_o + q * N, a + ks * 2 * group16, w + 2 * ks, idesc_o, (m > 0 || ks > 0) ? 1u : 0u);
           }
-          umma_commit(&empty[st]);
-          umma_commit(&pv_done[m & 1]);
+          if (elect_one()) {
+            umma_commit(&empty[prev]);
+            umma_commit(&pv_done[m & 1]);
+          }
+          __syncwarp();
         }
+        prev = st;
+        if (++st == sh.stages) { st = 0; ph ^= 1; }
       }
     }
-    __syncwarp();
   } else {
     // ---------------- softmax / epilogue ----------------
-    const int qd = warp & 3, key = (qd & 1) * 32 + lane;
+    const int qd = warp & 3, key = qd * 16 + lane;           // lanes 0..15 of the first three quadrants hold the tile's keys
+    const bool mine = lane < 16 && key < LD_TILE;
     const uint32_t lane_off = static_cast<uint32_t>(qd * 32) << 16;
     const float sc = p.scale * LD_LOG2E;
     float m[N], sum[N];                                      // reference maxima, the same in every thread; weights of its keys
@@ -473,31 +496,29 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     for (int c = 0; c < N; ++c) { m[c] = -INFINITY; sum[c] = 0.f; }
     for (int n = 0; n < n_tiles; ++n) {
       const int g = n & 1;
-      const bool active = (qd >> 1) == g;                    // this warp's lanes hold the tile's keys
+      const bool seen = mine && (tb + n) * LD_TILE + key <= i;
       float v[N];
       bool over = false;
-      if (active) {
-        mbar_wait(&s_full[g], (n >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
-        __syncwarp();
-        tc_fence_after();
-        tmem_ld_heads<N>(tmem_s + g * N + lane_off, v);
-        tmem_ld_wait();
-        tc_fence_before();
-        const bool seen = (tb + n) * LD_TILE + key <= i;
+      mbar_wait(&s_full[g], (n >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
+      __syncwarp();
+      tc_fence_after();
+      tmem_ld_heads<N>(tmem_s + g * N + lane_off, v);
+      tmem_ld_wait();
+      tc_fence_before();
 #pragma unroll
-        for (int c = 0; c < N; ++c) {
-          v[c] = seen ? v[c] * sc : -INFINITY;
-          over = over || v[c] > m[c] + 8.0f;
-        }
+      for (int c = 0; c < N; ++c) {
+        v[c] = seen ? v[c] * sc : -INFINITY;
+        over = over || v[c] > m[c] + 8.0f;
       }
       if (named_bar_any(1, 128, over)) {                     // some head's maximum grows: reduce, and rescale what is there
-        if (active) s_max[(qd & 1) * 32 + lane] = warp_columns<N, true>(v, lane);
+        s_max[qd * 32 + lane] = warp_columns<N, true>(v, lane);
         named_bar_sync(1, 128);
         float f[N];
         bool any = false;
 #pragma unroll
         for (int c = 0; c < N; ++c) {
-          const float mx = fmaxf(s_max[c * (32 / N)], s_max[32 + c * (32 / N)]);
+          const float* x = s_max + c * (32 / N);
+          const float mx = fmaxf(fmaxf(x[0], x[32]), fmaxf(x[64], x[96]));
           const bool grow = mx > m[c] + 8.0f;
           f[c] = grow && m[c] != -INFINITY ? exp2f(m[c] - mx) : 1.0f;
           any = any || f[c] != 1.0f;
@@ -520,8 +541,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         }
         named_bar_sync(1, 128);                              // s_max is read
       }
-      if (active) {
-        if (n > 1) mbar_wait(&pv_done[g], ((n - 2) >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);     // its weights are read
+      if (n > 1) mbar_wait(&pv_done[g], ((n - 2) >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);     // its weights are read
+      if (mine) {
         uint8_t* pd = p_s + g * QCH + (key & 7) * 2;
 #pragma unroll
         for (int c = 0; c < N; ++c) {
@@ -651,7 +672,8 @@ static int map_3d(CUtensorMap* m, const void* base, cuuint64_t d0, cuuint64_t d1
   return r == CUDA_SUCCESS ? 0 : -3;
 }
 
-// Ring geometry for N heads per CTA; false when two stages do not fit.
+// Ring geometry for N heads per CTA; false when two stages do not fit.  The score product reads two groups of 8 rows past its
+// stage: behind the last one lie q' and the weights, which are at least as large.
 template <int N>
 static bool latent_decode_shape(int Rp, int rw, LatentDecodeShape* sh, size_t* smem) {
   sh->nc = Rp / 64;
@@ -659,7 +681,7 @@ static bool latent_decode_shape(int Rp, int rw, LatentDecodeShape* sh, size_t* s
   sh->pairs = (sh->nc + 1) / 2;
   const size_t stage = (size_t)LD_GROUPS * sh->chunks * 1024, fixed = (size_t)(sh->chunks + 2) * N * 128 + 2048, cap = 227 * 1024;
   if (rw % 64 || fixed + 2 * stage > cap) return false;
-  sh->stages = (int)((cap - fixed) / stage) & ~1;
+  sh->stages = (int)((cap - fixed) / stage);
   if (sh->stages > LD_MAX_STAGES) sh->stages = LD_MAX_STAGES;
   int cols = 32;
   while (cols < (2 + sh->pairs) * N) cols *= 2;
