@@ -619,7 +619,7 @@ def test_plain_kernels_in_bf16(tmp_path):
 
 def test_sizes_beyond_the_tensor_core_kernels(tmp_path):
     """Latents and heads that fit neither the decode kernel nor the portion kernel, recurrent heads beyond the chunk kernels."""
-    cfg = H.config([(H.latent(heads=2, dim=250, rot_dim=16, vdim=24, kv_rank=840, scale=0.06), H.dense()), (H.gla(heads=1, dim=136, vdim=24), None),
+    cfg = H.config([(H.latent(heads=2, dim=250, rot_dim=16, vdim=24, kv_rank=1300, scale=0.06), H.dense()), (H.gla(heads=1, dim=136, vdim=24), None),
                     (H.latent(heads=2, dim=40, rot_dim=8, vdim=264, kv_rank=64), None)])
     cfg, sd, d = H.make(tmp_path, cfg)
     toks = H.tokens(cfg, 140)
