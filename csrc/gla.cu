@@ -166,15 +166,30 @@ struct GlaChunkParams {
 
 constexpr float GC_RANGE = 60.0f;
 
-// grid (n_chunks, ceil(heads * dk / 64)), 256 threads: thread (segment of 32 tokens, channel)
-constexpr int GD_CH = 64;
+// The same as log_sigmoid with log1p(x) = 2 artanh(x / (2 + x)) by the series of artanh: x <= 1, so eight terms leave 1.5e-9
+// of the value, at any size of x.
+__device__ __forceinline__ float log_sigmoid_series(float z) {
+  const float x = __expf(-fabsf(z)), s = __fdividef(x, 2.0f + x), q = s * s;
+  float r = 2.0f / 15.0f;
+  r = fmaf(r, q, 2.0f / 13.0f);
+  r = fmaf(r, q, 2.0f / 11.0f);
+  r = fmaf(r, q, 2.0f / 9.0f);
+  r = fmaf(r, q, 2.0f / 7.0f);
+  r = fmaf(r, q, 2.0f / 5.0f);
+  r = fmaf(r, q, 2.0f / 3.0f);
+  r = fmaf(r, q, 2.0f);
+  return fmaf(-r, s, fminf(z, 0.f));
+}
+
+// grid (n_chunks, ceil(heads * dk / 32)), 256 threads: thread (segment of 16 tokens, channel)
+constexpr int GD_CH = 32, GD_SEG = 16;
 __global__ void __launch_bounds__(256) gla_decay_kernel(const GlaParams p, const GlaChunkParams c) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float sm[];
   float* s_low = sm;                                   // [128][rank]
-  float* s_w = s_low + 128 * p.rank;                   // [rank][64]
-  float* s_tot = s_w + GD_CH * p.rank;                 // [4][64]
+  float* s_w = s_low + 128 * p.rank;                   // [rank][GD_CH]
+  float* s_tot = s_w + GD_CH * p.rank;                 // [8][GD_CH]
   const int start = c.c_start[blockIdx.x], len = c.c_len[blockIdx.x];
   const int n_ch = p.heads * p.dk, c0 = blockIdx.y * GD_CH;
   for (int i = threadIdx.x; i < 128 * p.rank; i += 256) s_low[i] = i < len * p.rank ? p.low[(size_t)start * p.rank + i] : 0.f;
@@ -184,23 +199,23 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const GlaParams p, const
   }
   __syncthreads();
   const int ch = threadIdx.x & (GD_CH - 1), seg = threadIdx.x / GD_CH;
-  float a[32];
+  float a[GD_SEG];
   const float b = c0 + ch < n_ch ? p.b2[c0 + ch] : 0.f;
 #pragma unroll
-  for (int t = 0; t < 32; ++t) a[t] = b;
-  const float4* low = reinterpret_cast<const float4*>(s_low + seg * 32 * p.rank);
+  for (int t = 0; t < GD_SEG; ++t) a[t] = b;
+  const float4* low = reinterpret_cast<const float4*>(s_low + seg * GD_SEG * p.rank);
   for (int r = 0; r < p.rank; r += 4) {
     const float w0 = s_w[r * GD_CH + ch], w1 = s_w[(r + 1) * GD_CH + ch], w2 = s_w[(r + 2) * GD_CH + ch], w3 = s_w[(r + 3) * GD_CH + ch];
 #pragma unroll
-    for (int t = 0; t < 32; ++t) {
+    for (int t = 0; t < GD_SEG; ++t) {
       const float4 l = low[(t * p.rank + r) / 4];
       a[t] += w0 * l.x + w1 * l.y + w2 * l.z + w3 * l.w;
     }
   }
   float sum = 0.f;
 #pragma unroll
-  for (int t = 0; t < 32; ++t) {
-    sum += log_sigmoid(a[t]) * p.inv_tau;
+  for (int t = 0; t < GD_SEG; ++t) {
+    sum += log_sigmoid_series(a[t]) * p.inv_tau;
     a[t] = sum;
   }
   s_tot[seg * GD_CH + ch] = sum;
@@ -209,8 +224,8 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const GlaParams p, const
   for (int k = 0; k < seg; ++k) off += s_tot[k * GD_CH + ch];
   if (c0 + ch < n_ch) {
 #pragma unroll
-    for (int t = 0; t < 32; ++t)
-      if (seg * 32 + t < len) c.G[(size_t)(start + seg * 32 + t) * n_ch + c0 + ch] = a[t] + off;
+    for (int t = 0; t < GD_SEG; ++t)
+      if (seg * GD_SEG + t < len) c.G[(size_t)(start + seg * GD_SEG + t) * n_ch + c0 + ch] = a[t] + off;
   }
 }
 
@@ -218,8 +233,7 @@ __device__ __forceinline__ void ld8f(const float* p, float* o) {
   const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
   o[0] = a.x; o[1] = a.y; o[2] = a.z; o[3] = a.w; o[4] = b.x; o[5] = b.y; o[6] = b.z; o[7] = b.w;
 }
-__device__ __forceinline__ void ld8f(const __nv_bfloat16* p, float* o) {
-  const uint4 u = *reinterpret_cast<const uint4*>(p);
+__device__ __forceinline__ void unpack8(const uint4& u, float* o) {
   const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
@@ -284,21 +298,36 @@ gla_chunk_state_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_co
   const int n_ch = p.heads * p.dk;
   if (tid < MC_TOK) s_last[tid] = tid < p.dk ? c.G[(size_t)(start + len - 1) * n_ch + h * p.dk + tid] : 0.f;
   __syncthreads();
-  // weighted keys: 16 bytes = 8 dims of one token per step, swizzled as TMA would
-  for (int i = tid; i < MC_TOK * 16; i += 256) {
-    const int tok = i >> 4, piece = i & 15, d = piece * 8;
-    uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
-    if (tok < len && d < p.dk) {
-      float k[8], g[8];
-      ld8f(reinterpret_cast<const __nv_bfloat16*>(p.qkvg) + (size_t)(start + tok) * p.ld + (size_t)(p.heads + h) * p.dk + d, k);
-      ld8f(c.G + (size_t)(start + tok) * n_ch + h * p.dk + d, g);
+  // weighted keys: 16 bytes = 8 dims of one token per step, swizzled as TMA would; the loads of four steps go out together
+  constexpr int U = 4;
+#pragma unroll 1
+  for (int i0 = tid; i0 < MC_TOK * 16; i0 += 256 * U) {
+    uint4 raw[U];
+    float g[U][8];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) k[e] *= __expf(s_last[d + e] - g[e]);
-      split8(k, &hi, &lo);
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * 256, tok = i >> 4, d = (i & 15) * 8;
+      if (tok < len && d < p.dk) {
+        raw[u] = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.qkvg) + (size_t)(start + tok) * p.ld +
+                                                 (size_t)(p.heads + h) * p.dk + d);
+        ld8f(c.G + (size_t)(start + tok) * n_ch + h * p.dk + d, g[u]);
+      }
     }
-    const int off = (piece >> 3) * MC_KCH + tok * 128 + (((piece & 7) ^ (tok & 7)) << 4);
-    *reinterpret_cast<uint4*>(mc_smem + GcStateSmem::K_HI + off) = hi;
-    *reinterpret_cast<uint4*>(mc_smem + GcStateSmem::K_LO + off) = lo;
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * 256, tok = i >> 4, piece = i & 15, d = piece * 8;
+      uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
+      if (tok < len && d < p.dk) {
+        float k[8];
+        unpack8(raw[u], k);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) k[e] *= __expf(s_last[d + e] - g[u][e]);
+        split8(k, &hi, &lo);
+      }
+      const int off = (piece >> 3) * MC_KCH + tok * 128 + (((piece & 7) ^ (tok & 7)) << 4);
+      *reinterpret_cast<uint4*>(mc_smem + GcStateSmem::K_HI + off) = hi;
+      *reinterpret_cast<uint4*>(mc_smem + GcStateSmem::K_LO + off) = lo;
+    }
   }
   fence_proxy_async_smem();
   __syncthreads();
@@ -529,28 +558,45 @@ gla_chunk_out_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_cons
       if (lane == 0) s_count[ct >> 5] = __popc(ball);
     }
     named_bar_sync(1, 256);
-    for (int i = ct; i < MC_TOK * 16; i += 256) {
-      const int tok = i >> 4, piece = i & 15, d = piece * 8;
-      if (piece >= nk * 8) continue;
-      uint4 ah = make_uint4(0u, 0u, 0u, 0u), al = ah, bh = ah, bl = ah;
-      if (tok < len && d < p.dk) {
-        float q[8], k[8], g[8];
-        ld8f(qk + (size_t)tok * p.ld + (size_t)h * p.dk + d, q);
-        ld8f(qk + (size_t)tok * p.ld + (size_t)(p.heads + h) * p.dk + d, k);
-        ld8f(G + (size_t)tok * n_ch + d, g);
+    constexpr int U = 4;                             // steps whose loads go out together
+#pragma unroll 1
+    for (int i0 = ct; i0 < MC_TOK * 16; i0 += 256 * U) {
+      uint4 rq[U], rk[U];
+      float g[U][8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          q[e] *= p.q_scale * __expf(g[e]);
-          k[e] = s_keep[d + e] != 0.f ? k[e] * __expf(-g[e]) : 0.f;
+      for (int u = 0; u < U; ++u) {
+        const int i = i0 + u * 256, tok = i >> 4, d = (i & 15) * 8;
+        if (tok < len && d < p.dk) {
+          const __nv_bfloat16* row = qk + (size_t)tok * p.ld + d;
+          rq[u] = *reinterpret_cast<const uint4*>(row + (size_t)h * p.dk);
+          rk[u] = *reinterpret_cast<const uint4*>(row + (size_t)(p.heads + h) * p.dk);
+          ld8f(G + (size_t)tok * n_ch + d, g[u]);
         }
-        split8(q, &ah, &al);
-        split8(k, &bh, &bl);
       }
-      const int off = (piece >> 3) * MC_KCH + tok * 128 + (((piece & 7) ^ (tok & 7)) << 4);
-      *reinterpret_cast<uint4*>(mc_smem + GcOutSmem::QHI + off) = ah;
-      *reinterpret_cast<uint4*>(mc_smem + GcOutSmem::QLO + off) = al;
-      *reinterpret_cast<uint4*>(mc_smem + GcOutSmem::KHI + off) = bh;
-      *reinterpret_cast<uint4*>(mc_smem + GcOutSmem::KLO + off) = bl;
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int i = i0 + u * 256, tok = i >> 4, piece = i & 15, d = piece * 8;
+        if (piece >= nk * 8) continue;
+        uint4 ah = make_uint4(0u, 0u, 0u, 0u), al = ah, bh = ah, bl = ah;
+        if (tok < len && d < p.dk) {
+          float q[8], k[8];
+          unpack8(rq[u], q);
+          unpack8(rk[u], k);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            const float f = __expf(g[u][e]);
+            q[e] *= p.q_scale * f;
+            k[e] = s_keep[d + e] != 0.f ? __fdividef(k[e], f) : 0.f;
+          }
+          split8(q, &ah, &al);
+          split8(k, &bh, &bl);
+        }
+        const int off = (piece >> 3) * MC_KCH + tok * 128 + (((piece & 7) ^ (tok & 7)) << 4);
+        *reinterpret_cast<uint4*>(mc_smem + GcOutSmem::QHI + off) = ah;
+        *reinterpret_cast<uint4*>(mc_smem + GcOutSmem::QLO + off) = al;
+        *reinterpret_cast<uint4*>(mc_smem + GcOutSmem::KHI + off) = bh;
+        *reinterpret_cast<uint4*>(mc_smem + GcOutSmem::KLO + off) = bl;
+      }
     }
     fence_proxy_async_smem();
     mbar_arrive(qk_full);
@@ -702,7 +748,7 @@ extern "C" int tahb_gla_chunks(const GlaParams* p, const GlaChunkParams* c, int 
       return -10;
     configured = true;
   }
-  const size_t decay_smem = ((size_t)(128 + GD_CH) * p->rank + 4 * GD_CH) * 4;
+  const size_t decay_smem = ((size_t)(128 + GD_CH) * p->rank + 8 * GD_CH) * 4;
   if (decay_smem > 200 * 1024) return -2;
   cudaError_t e = launch_chain(gla_decay_kernel, dim3(c->n_chunks, (p->heads * p->dk + GD_CH - 1) / GD_CH), dim3(256), decay_smem, stream, *p, *c);
   if (e == cudaSuccess)
