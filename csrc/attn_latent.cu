@@ -102,7 +102,7 @@ __global__ void __launch_bounds__(128) latent_post_kernel(const LatentPostParams
 
 // ---------------------------------------------------------------------------------------------
 // latent_query: the projected queries [n, heads * dk], head = [dim | rot], get their last rot dims rotated.  Tokens below
-// n_list go to head lists [heads * npad, dq] (zero behind dim + rot), the others stay where they are.  One CTA per token.
+// n_list go to head lists [heads * npad, dq] (zero behind dim + rot), the others stay where they are.  Grid (n, head blocks).
 // ---------------------------------------------------------------------------------------------
 struct LatentQueryParams {
   void* q;
@@ -116,14 +116,15 @@ template <typename T>
 __global__ void __launch_bounds__(256) latent_query_kernel(const LatentQueryParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, half = p.rot / 2;
+  const int t = blockIdx.x, half = p.rot / 2, per = (p.heads + gridDim.y - 1) / gridDim.y;
+  const int h0 = blockIdx.y * per, nh = min(per, p.heads - h0);
   const bool listed = t < p.n_list;
   T* src = reinterpret_cast<T*>(p.q) + (size_t)t * p.ld;
   T* list = reinterpret_cast<T*>(p.list) + (size_t)t * p.dq;             // head h at h * npad * dq
   const size_t head = listed ? (size_t)p.npad * p.dq : p.dk;
   T* dst = listed ? list : src;
-  for (int i = threadIdx.x; i < p.heads * half; i += 256) {
-    const int h = i / half, k = i % half;
+  for (int i = threadIdx.x; i < nh * half; i += 256) {
+    const int h = h0 + i / half, k = i % half;
     const float2 f = p.rope[(size_t)t * half + k];
     const T* q = src + (size_t)h * p.dk + p.dim + 2 * k;
     const float u = ldf(q), v = ldf(q + 1);
@@ -133,8 +134,8 @@ __global__ void __launch_bounds__(256) latent_query_kernel(const LatentQueryPara
   }
   if (listed) {
     const int rest = p.dq - p.rot;                                        // unrotated dims, then the zeros behind the head
-    for (int i = threadIdx.x; i < p.heads * rest; i += 256) {
-      const int h = i / rest, d = i % rest;
+    for (int i = threadIdx.x; i < nh * rest; i += 256) {
+      const int h = h0 + i / rest, d = i % rest;
       if (d < p.dim) list[h * head + d] = src[(size_t)h * p.dk + d];
       else stf(list + h * head + d + p.rot, 0.f);
     }
@@ -726,8 +727,9 @@ extern "C" int tahb_latent_post(const LatentPostParams* p, int f32, cudaStream_t
 extern "C" int tahb_latent_query(const LatentQueryParams* p, int f32, cudaStream_t stream) {
   if (p->n <= 0) return 0;
   if (p->rot % 2 || p->dim + p->rot > p->dk || p->dk > p->dq || p->n_list > p->npad) return -2;
-  cudaError_t e = f32 ? launch_chain(latent_query_kernel<float>, dim3(p->n), dim3(256), 0, stream, *p)
-                      : launch_chain(latent_query_kernel<__nv_bfloat16>, dim3(p->n), dim3(256), 0, stream, *p);
+  const dim3 grid(p->n, p->n <= 1024 ? (p->heads + 1) / 2 : 1);           // few tokens: spread their heads over the SMs
+  cudaError_t e = f32 ? launch_chain(latent_query_kernel<float>, grid, dim3(256), 0, stream, *p)
+                      : launch_chain(latent_query_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, *p);
   return e == cudaSuccess ? 0 : -3;
 }
 
