@@ -2,8 +2,8 @@
 //
 //   cached row of a token:  [c: kv_rank, padded to Rp][r: rot dims, padded to rw], both multiples of 64
 //     c = rms(low part) * w,  r = rotated shared key part
-//   head h:  key = [Wk_h c, r], value = Wv_h c;  score = (q . key) * scale;  softmax with exp(sink_h) in the denominator;
-//   out_h *= sigmoid(gate), element by element
+//   head h:  key = [Wk_h c, r], value = Wv_h c;  score = (q . key) * scale over the last `window` tokens;  softmax with exp(sink_h)
+//   in the denominator (optional);  out_h *= sigmoid(gate), element by element (optional)
 //
 // Single tokens run in the absorbed form: q' = [Wk_h^T q_unrotated, q_rotated] against the cached rows themselves (one key
 // and one value, c, for all heads), then Wv_h on the weighted sum of c.  Prompt portions expand the row's cached latents to
@@ -156,7 +156,7 @@ __global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* __restr
   }
 }
 
-// out[t, h * dv + d] = list[h * npad + t, d] * sigmoid(gate[t, h * dv + d]), 8 elements per thread
+// out[t, h * dv + d] = list[h * npad + t, d] * sigmoid(gate[t, h * dv + d]) (gate null: no factor), 8 elements per thread
 template <typename T>
 __global__ void __launch_bounds__(256) latent_gate_kernel(const T* __restrict__ list, int npad, int ld_list, const T* __restrict__ gate,
                                                           long long ld_gate, T* __restrict__ out, long long ld_out, int n, int heads,
@@ -169,6 +169,11 @@ __global__ void __launch_bounds__(256) latent_gate_kernel(const T* __restrict__ 
   const int c = (int)(i % nv) * 8, h = (int)(i / nv % heads), t = (int)(i / nv / heads);
   float v[8], z[8];
   ld8(list + ((size_t)h * npad + t) * ld_list + c, v);
+  if (gate == nullptr) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) stf(out + (size_t)t * ld_out + (size_t)h * dv + c + e, v[e]);
+    return;
+  }
   ld8(gate + (size_t)t * ld_gate + (size_t)h * dv + c, z);
 #pragma unroll
   for (int e = 0; e < 8; ++e) stf(out + (size_t)t * ld_out + (size_t)h * dv + c + e, v[e] / (1.0f + expf(-z[e])));
@@ -191,6 +196,7 @@ struct LatentAttnParams {
   int n_split;
   int n_pages;                // pages of the pool
   int* status;
+  int window;                 // tokens that a query sees, itself the last of them
 };
 
 // Plain kernel: any sizes, bf16 or fp32.  One CTA per (head, token); 128 keys at a time, one key per thread for the scores,
@@ -215,7 +221,7 @@ __global__ void __launch_bounds__(128) latent_attn_plain_kernel(const LatentAttn
   for (int d = tid; d < p.Rp; d += 128) s_acc[d] = 0.f;
   __syncthreads();
   float m = -INFINITY, l = 0.f;
-  for (int j0 = 0; j0 <= i; j0 += 128) {
+  for (int j0 = p.window > i ? 0 : i - p.window + 1; j0 <= i; j0 += 128) {
     const int j = j0 + tid;
     float s = -INFINITY;
     int at = 0;
@@ -404,8 +410,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   const uint32_t tmem_s = __shfl_sync(0xffffffffu, *tmem_slot, 0), tmem_o = tmem_s + 2 * N;
   const int h0 = blockIdx.x * N, t = blockIdx.y, split = blockIdx.z;
   const int i = __shfl_sync(0xffffffffu, p.pos[t], 0);
-  const int tiles = i / LD_TILE + 1, per = (tiles + p.n_split - 1) / p.n_split;
-  const int tb = split * per, te = min(tiles, tb + per), n_tiles = max(0, te - tb);
+  const int lo = p.window > i ? 0 : i - p.window + 1;        // first visible key
+  const int tile0 = lo / LD_TILE, tiles = i / LD_TILE + 1, per = (tiles - tile0 + p.n_split - 1) / p.n_split;
+  const int tb = tile0 + split * per, te = min(tiles, tb + per), n_tiles = max(0, te - tb);
 
   if (warp == 0) {
     // ---------------- TMA producer ----------------
@@ -497,7 +504,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     for (int c = 0; c < N; ++c) { m[c] = -INFINITY; sum[c] = 0.f; }
     for (int n = 0; n < n_tiles; ++n) {
       const int g = n & 1;
-      const bool seen = mine && (tb + n) * LD_TILE + key <= i;
+      const int j = (tb + n) * LD_TILE + key;
+      const bool seen = mine && j <= i && j >= lo;
       float v[N];
       bool over = false;
       mbar_wait(&s_full[g], (n >> 1) & 1, abort_flag, p.status, STATUS_TIMEOUT_ACCUM);
@@ -759,7 +767,7 @@ extern "C" int tahb_latent_gate(const void* list, int npad, int ld_list, const v
 
 static int check_latent(const LatentAttnParams* p) {
   return p->Rp % 64 || p->Rp < 64 || p->rw % 8 || p->rw < 8 || p->lq < p->Rp + p->rw || p->lq % 8 || p->n > p->npad ||
-         p->heads < 1 || p->heads > 65535 ? -2 : 0;
+         p->heads < 1 || p->heads > 65535 || p->window < 1 ? -2 : 0;
 }
 
 extern "C" int tahb_latent_attn_plain(const LatentAttnParams* p, int f32, cudaStream_t stream) {

@@ -1,5 +1,5 @@
-// Paged attention with a sliding window, kept first tokens, a query temperature, a score cap, a per-distance bias, a
-// softmax sink and an output gate per head (or, for portions, per element).
+// Paged attention with a sliding window, kept first tokens or pooled blocks in front of it, a query temperature, a score cap, a
+// per-distance bias (a table or a slope), a softmax sink and an output gate per head or per element.
 //
 // Query at position i of a sequence sees key j when  j <= i  and  (i - j < window  or  j < keep_first).
 // score = cap(temp(i) * (q . k) * scale) + bias[h][min(i - j, D)] with cap(s) = softcap * tanh(s / softcap) and
@@ -8,10 +8,18 @@
 // attention, keep_first = 0 a plain window, softcap = 0 no cap, temp_coef = 0 no temperature, and the bias table, the
 // sink and the gate may each be absent.
 //
+// A slope takes slope_h * (i - j) off a score.  Pooled blocks: block b is the mean of the keys b P .. b P + P - 1 and is seen, as one
+// more key and value, when b P + P - 1 <= i - window.
+//
 // Keys and values are read from the paged cache only (the tokens of the running step are written there first), so
 // portions of a prompt, single decoded tokens and layers that read another layer's cache are the same case:
 //   page of one layer:  [K: kv_heads][page_size][dk]  then  [V: kv_heads][page_size][dv]
 // dk and dv are padded to multiples of 8; padding dims hold zeros.
+//   Values that are the keys as projected ("tied"): a page holds K only.  When the keys have a norm over all heads of a token,
+//   its weights are folded into the queries and its factor, one number per token, is a page of page_size floats beside the keys:
+//   score = factor_j * (q' . k_j), value = k_j.
+//   Pooled blocks: a pool of its own under the same page table, with S rows a page ([kv_heads][S][dk], S a power of two >= 16 / P):
+//   block b is row b % S of logical page b / S, a page that the row owns by the time the block is complete.
 #include <cuda.h>
 
 #include "attn_common.cuh"
@@ -239,6 +247,150 @@ __global__ void __launch_bounds__(128) qkv_post_kernel(const QkvPostParams p) {
 }
 
 // ---------------------------------------------------------------------------------------------
+// Keys of tied layers without norm, bias and rotation, [M, nkv * dk] of pitch ld: to the paged cache, and when a token is the
+// last of a block of P, the mean of the block to the pooled rows.  One warp per (token, head), 8 dims per lane.  The block's other
+// keys come from the projection when they are tokens of the same step (their cache writes may not have happened yet), from the
+// cache otherwise, oldest first: the sum does not depend on how a prompt was cut.
+// ---------------------------------------------------------------------------------------------
+struct TiedKeysParams {
+  const void* k;              // [M, ld]
+  void* cache;                // [pages][nkv][page_size][dk]
+  void* pooled;               // [pages][nkv][pool_rows][dk], or null
+  const int* slot;            // [M], negative = nothing to do
+  const int* pos;
+  const int* row;
+  const int* page_table;      // [rows, max_pages]
+  int M, nkv, dk, page_size, max_pages, pool, pool_rows;
+  long long ld;
+};
+
+template <typename T> struct Row8;
+template <> struct Row8<float> { using type = struct { float4 a, b; }; };
+template <> struct Row8<__nv_bfloat16> { using type = uint4; };
+
+template <typename T>
+__global__ void __launch_bounds__(128) tied_keys_kernel(const TiedKeysParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  using R = typename Row8<T>::type;
+  const long long wg = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+  const int c = (threadIdx.x & 31) * 8;
+  if (wg >= (long long)p.M * p.nkv) return;
+  const int t = (int)(wg / p.nkv), g = (int)(wg % p.nkv), sl = p.slot[t];
+  if (sl < 0 || c >= p.dk) return;
+  const T* src = reinterpret_cast<const T*>(p.k) + (size_t)t * p.ld + (size_t)g * p.dk + c;
+  T* cache = reinterpret_cast<T*>(p.cache);
+  auto at = [&](int page, int off) { return (((size_t)page * p.nkv + g) * p.page_size + off) * p.dk + c; };
+  *reinterpret_cast<R*>(cache + at(sl / p.page_size, sl % p.page_size)) = *reinterpret_cast<const R*>(src);
+  if (p.pooled == nullptr) return;
+  const int i = p.pos[t], r = p.row[t], P = p.pool;
+  if ((i + 1) % P) return;
+  const int* pt = p.page_table + (size_t)r * p.max_pages;
+  float sum[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) sum[e] = 0.f;
+#pragma unroll 4
+  for (int k = P - 1; k >= 0; --k) {
+    const bool here = t - k >= 0 && p.row[max(t - k, 0)] == r && p.pos[max(t - k, 0)] == i - k;
+    const T* q = here ? src - (size_t)k * p.ld : cache + at(pt[(i - k) / p.page_size], (i - k) % p.page_size);
+    float v[8];
+    load8(q, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sum[e] += v[e];
+  }
+  const int b = i / P;
+  T* dst = reinterpret_cast<T*>(p.pooled) + (((size_t)pt[b / p.pool_rows] * p.nkv + g) * p.pool_rows + b % p.pool_rows) * p.dk + c;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) dst[e] = from_f<T>(sum[e] / (float)P);
+}
+
+// Pooled rows one after another for the portion kernel: out[r][g * dk + d] = pooled row src[r] (page * pool_rows + row), zeros
+// where src[r] is negative.  16-byte units.
+__global__ void __launch_bounds__(128) pool_gather_kernel(const uint4* __restrict__ pooled, const int* __restrict__ src, int nkv, int units,
+                                                          int pool_rows, int n_pages, uint4* __restrict__ out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int s = src[blockIdx.x], page = s < 0 ? -1 : s / pool_rows;
+  for (int i = threadIdx.x; i < nkv * units; i += 128) {
+    const int g = i / units, c = i % units;
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (page >= 0 && page < n_pages) v = pooled[(((size_t)page * nkv + g) * pool_rows + s % pool_rows) * units + c];
+    out[(size_t)blockIdx.x * nkv * units + i] = v;
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
+// RMS norms of q and k over all heads of a token, for tied layers: q times its factor and the weights of both norms to q_out, the
+// projected k to the paged cache, k's factor to the factors beside it.  One CTA per token.
+// ---------------------------------------------------------------------------------------------
+struct NormAllParams {
+  const void* q;              // [M, ld]: nq heads of dk
+  const void* k;              // the same rows: nkv heads of dk
+  const float* w;             // [nq * dk]: weight of q's norm times that of the key head it meets (padding dims zero)
+  void* q_out;                // [M, nq * dk]
+  void* cache;                // [pages][nkv][page_size][dk]
+  float* factor;              // [pages][page_size]
+  const int* slot;            // [M], negative = no cache write
+  int M, nq, nkv, dk, dim, page_size;
+  long long ld;
+  float eps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) norm_all_kernel(const NormAllParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  using R = typename Row8<T>::type;
+  __shared__ float red[2][8];
+  const size_t t = blockIdx.x;
+  const T* q = reinterpret_cast<const T*>(p.q) + t * p.ld;
+  const T* k = reinterpret_cast<const T*>(p.k) + t * p.ld;
+  const int sl = p.slot[t], cq = p.nq * p.dk, ck = p.nkv * p.dk;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * 8; c < cq; c += 2048) {
+    float v[8];
+    load8(q + c, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sq = fmaf(v[e], v[e], sq);
+  }
+  for (int c = threadIdx.x * 8; c < ck; c += 2048) {
+    float v[8];
+    load8(k + c, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sk = fmaf(v[e], v[e], sk);
+    if (sl >= 0) {
+      const int g = c / p.dk;
+      T* dst = reinterpret_cast<T*>(p.cache) + (((size_t)(sl / p.page_size) * p.nkv + g) * p.page_size + sl % p.page_size) * p.dk + c % p.dk;
+      *reinterpret_cast<R*>(dst) = *reinterpret_cast<const R*>(k + c);
+    }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) {
+    red[0][threadIdx.x >> 5] = sq;
+    red[1][threadIdx.x >> 5] = sk;
+  }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) {
+    sq += red[0][w];
+    sk += red[1][w];
+  }
+  if (threadIdx.x == 0 && sl >= 0) p.factor[sl] = 1.0f / sqrtf(sk / (float)(p.nkv * p.dim) + p.eps);
+  const float r = 1.0f / sqrtf(sq / (float)(p.nq * p.dim) + p.eps);
+  for (int c = threadIdx.x * 8; c < cq; c += 2048) {
+    float v[8], w[8];
+    load8(q + c, v);
+    load8(p.w + c, w);
+    T o[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) o[e] = from_f<T>(v[e] * r * w[e]);
+    *reinterpret_cast<R*>(reinterpret_cast<T*>(p.q_out) + t * cq + c) = *reinterpret_cast<const R*>(o);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------
 // What every attention kernel of this file gets.
 // ---------------------------------------------------------------------------------------------
 struct WindowAttnParams {
@@ -251,7 +403,7 @@ struct WindowAttnParams {
   const float* bias;          // [nq, far + 1] bias by distance (the last entry serves every larger distance), or null
   const float* sink;          // [nq] or null
   const void* gate;           // pre-activation of head h of query t at gate[t * ld_gate + h], or null
-  const void* wide_gate;      // pre-activation of every output element, gate[t * ld_gate + h * dv + d] (portion kernel), or null
+  const void* wide_gate;      // pre-activation of every output element, gate[t * ld_gate + h * dv + d], or null
   int n, nq, nkv, dk, dv, page_size, max_pages, window, keep_first, far;
   long long ld_q, ld_out, ld_gate;
   float scale;
@@ -261,6 +413,12 @@ struct WindowAttnParams {
   float* ws;                  // split partial results (decode kernel, n_split > 1)
   int n_split;
   int* status;
+  const float* slope;         // [nq] taken off the scores per token of distance, or null
+  const float* factor;        // [pages][page_size] factor of every key's scores (tied layers), or null
+  const void* pooled;         // pooled blocks of a tied layer (plain and decode kernels: their pool; portion kernel: a matrix), or null
+  int tied;                   // the values are the keys
+  int pool, pool_rows;        // tokens of a pooled block, pooled rows of a page
+  float out_scale;            // factor of the output
 };
 
 // scale of the scores of a query at position i
@@ -285,6 +443,9 @@ __device__ __forceinline__ void visible_range(int i, int window, int keep_first,
   keep_end = min(keep_first, lo);
 }
 
+// pooled blocks that a query at position i sees
+__device__ __forceinline__ int visible_blocks(int i, int window, int pool) { return max(0, i - window + 1) / pool; }
+
 // ---------------------------------------------------------------------------------------------
 // Plain kernel: any head sizes up to 256, bf16 or fp32 cache.  One warp per (query, head); 32 keys at a time, one key
 // per lane for the scores, one dim pair per lane for the weighted values.  Used by the 32-bit mode and for head sizes
@@ -308,23 +469,27 @@ __global__ void __launch_bounds__(128) window_attn_plain_kernel(const WindowAttn
   const float scale = query_scale(p, i);
   for (int d = lane; d < p.dk; d += 32) s_q[warp][d] = to_f<T>(q[d]);
   __syncwarp();
-  const size_t page_elems = (size_t)p.nkv * p.page_size * (p.dk + p.dv);
-  const T* kc = reinterpret_cast<const T*>(p.cache) + (size_t)kvh * p.page_size * p.dk;
-  const T* vc = reinterpret_cast<const T*>(p.cache) + (size_t)p.nkv * p.page_size * p.dk + (size_t)kvh * p.page_size * p.dv;
   float m = -INFINITY, l = 0.f, acc[2 * MAXP];
 #pragma unroll
   for (int c = 0; c < 2 * MAXP; ++c) acc[c] = 0.f;
   int keep_end, lo;
   visible_range(i, p.window, p.keep_first, keep_end, lo);
+  if (p.pooled != nullptr) keep_end = visible_blocks(i, p.window, p.pool);
+  const float slope = p.slope != nullptr ? p.slope[h] : 0.f;
   for (int part = 0; part < 2; ++part) {
     const int a = part == 0 ? 0 : lo, b = part == 0 ? keep_end : i + 1;
+    const bool blocks = part == 0 && p.pooled != nullptr;
+    const int ps = blocks ? p.pool_rows : p.page_size;
+    const size_t page_elems = (size_t)p.nkv * ps * (p.tied ? p.dk : p.dk + p.dv);
+    const T* kc = reinterpret_cast<const T*>(blocks ? p.pooled : p.cache) + (size_t)kvh * ps * p.dk;
+    const T* vc = p.tied ? kc : reinterpret_cast<const T*>(p.cache) + (size_t)p.nkv * ps * p.dk + (size_t)kvh * ps * p.dv;
     for (int j0 = a; j0 < b; j0 += 32) {
       const int j = j0 + lane;
       float s = -INFINITY;
       int page = 0;
       if (j < b) {
-        page = pt[j / p.page_size];
-        const T* k = kc + (size_t)page * page_elems + (size_t)(j % p.page_size) * p.dk;
+        page = pt[j / ps];
+        const T* k = kc + (size_t)page * page_elems + (size_t)(j % ps) * p.dk;
         float dot = 0.f;
         for (int d = 0; d < p.dk; d += 8) {
           float kv[8];
@@ -333,8 +498,10 @@ __global__ void __launch_bounds__(128) window_attn_plain_kernel(const WindowAttn
           for (int u = 0; u < 8; ++u) dot = fmaf(s_q[warp][d + u], kv[u], dot);
         }
         s = dot * scale;
+        if (p.factor != nullptr) s *= p.factor[(size_t)page * ps + j % ps];
         if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
         if (p.bias != nullptr) s += p.bias[(size_t)h * (p.far + 1) + min(i - j, p.far)];
+        s -= slope * (float)(i - j);
       }
       const float mx = fmaxf(m, warp_max(s));
       const float corr = m == -INFINITY ? 0.f : expf(m - mx);
@@ -349,7 +516,7 @@ __global__ void __launch_bounds__(128) window_attn_plain_kernel(const WindowAttn
       for (int c = 0; c < 2 * MAXP; ++c) acc[c] *= corr;
       const int n_here = min(32, b - j0);
       for (int u = 0; u < n_here; ++u) {
-        const T* v = vc + (size_t)s_page[warp][u] * page_elems + (size_t)((j0 + u) % p.page_size) * p.dv;
+        const T* v = vc + (size_t)s_page[warp][u] * page_elems + (size_t)((j0 + u) % ps) * p.dv;
         const float wu = s_w[warp][u];
 #pragma unroll
         for (int c = 0; c < MAXP; ++c) {
@@ -368,13 +535,18 @@ __global__ void __launch_bounds__(128) window_attn_plain_kernel(const WindowAttn
     f = expf(m - top);
     l = l * f + expf(p.sink[h] - top);
   }
-  f = f / l;
+  f = f / l * p.out_scale;
   if (p.gate != nullptr) f *= sigmoid_f(to_f<T>(reinterpret_cast<const T*>(p.gate)[(size_t)t * p.ld_gate + h]));
   T* o = reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + (size_t)h * p.dv;
+  const T* wg_in = p.wide_gate == nullptr ? nullptr : reinterpret_cast<const T*>(p.wide_gate) + (size_t)t * p.ld_gate + (size_t)h * p.dv;
 #pragma unroll
   for (int c = 0; c < MAXP; ++c) {
     const int d = 2 * lane + 64 * c;
     if (d < p.dv) {
+      if (wg_in != nullptr) {
+        acc[2 * c] *= sigmoid_f(to_f<T>(wg_in[d]));
+        acc[2 * c + 1] *= sigmoid_f(to_f<T>(wg_in[d + 1]));
+      }
       o[d] = from_f<T>(acc[2 * c] * f);
       o[d + 1] = from_f<T>(acc[2 * c + 1] * f);
     }
@@ -409,20 +581,29 @@ __device__ __forceinline__ float finish_scale(const WindowAttnParams& p, int t, 
     f = exp2f(m - top);
     mass = mass * f + exp2f(p.sink[h] - top);
   }
-  f = mass > 0.f ? f / mass : 0.f;
+  f = mass > 0.f ? f / mass * p.out_scale : 0.f;
   if (p.gate != nullptr)
     f *= sigmoid_f(__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(size_t)t * p.ld_gate + h]));
   return f;
 }
 
-template <int VEC, int GB, bool EXACT, bool CAP>   // EXACT: dk = dv = VEC * 64, known to the compiler; CAP: softcap > 0
+// factor of output element d of head h from its own gate
+__device__ __forceinline__ float element_gate(const WindowAttnParams& p, int t, int h, int d) {
+  if (p.wide_gate == nullptr) return 1.0f;
+  const float z = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.wide_gate)[(size_t)t * p.ld_gate + (size_t)h * p.dv + d]);
+  return __fdividef(1.0f, 1.0f + __expf(-z));
+}
+
+// EXACT: dk = dv = VEC * 64, known to the compiler; CAP: softcap > 0; TIED: pages of keys only, which are the values too, then the
+// page's factors (16 floats), and pooled blocks, 16 of them as one more page, in the place of the kept part
+template <int VEC, int GB, bool EXACT, bool CAP, bool TIED>
 __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) window_decode_kernel(const WindowAttnParams p) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int DPL = VEC * 8;
   const int dk = EXACT ? VEC * 64 : p.dk, dv = EXACT ? VEC * 64 : p.dv;
   extern __shared__ __align__(128) uint8_t wd_smem[];
-  const int kblk = WD_PAGE * dk, vblk = WD_PAGE * dv;              // elements of one K / V block of a page
+  const int kblk = WD_PAGE * dk, vblk = TIED ? 2 * WD_PAGE : WD_PAGE * dv;    // elements of one K / V block of a page (tied: the factors)
   const int stage_elems = WD_STAGE_PAGES * (kblk + vblk);
   __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(wd_smem);
   uint64_t* full_bar = reinterpret_cast<uint64_t*>(wd_smem + (size_t)WD_NSTAGE * stage_elems * 2);
@@ -436,8 +617,16 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
   const int i = p.pos[t];
   const int* pt = p.page_table + (size_t)p.row[t] * p.max_pages;
   int kp, w0;
-  const int total = visible_pages(i, p.window, p.keep_first, kp, w0);
+  int total = visible_pages(i, p.window, p.keep_first, kp, w0);
   const int lo = p.window > i ? 0 : i - p.window + 1;
+  const bool pooled = TIED && p.pooled != nullptr;
+  int blocks = 0;                                                  // pooled blocks, in the first kp pages
+  if (pooled) {
+    blocks = visible_blocks(i, p.window, p.pool);
+    kp = (blocks + WD_PAGE - 1) / WD_PAGE;
+    w0 = lo / WD_PAGE;
+    total = kp + i / WD_PAGE - w0 + 1;
+  }
   const int ppc = (total + p.n_split - 1) / p.n_split;
   const int pb = split * ppc, pe = min(total, pb + ppc);
   const int n_iter = pe > pb ? (pe - pb + WD_STAGE_PAGES - 1) / WD_STAGE_PAGES : 0;
@@ -464,7 +653,37 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
   const int gl = lane & 7;
 
   if (warp == 4) {
-    if (lane == 0) {
+    if constexpr (TIED) {                                          // the lanes share a stage's copies
+      const size_t page_elems = (size_t)p.nkv * kblk;
+      const int S = p.pool_rows, chunk = S * dk;
+      for (int it = 0; it < n_iter; ++it) {
+        const int s = it % WD_NSTAGE, first = pb + it * WD_STAGE_PAGES, n_here = min(WD_STAGE_PAGES, pe - first);
+        if (lane == 0) {
+          mbar_wait(&empty_bar[s], ((it / WD_NSTAGE) & 1) ^ 1, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
+          int bytes = 0;
+          for (int u = 0; u < n_here; ++u) {
+            const int idx = first + u;
+            bytes += pooled && idx < kp ? (min(WD_PAGE, blocks - idx * WD_PAGE) + S - 1) / S * chunk * 2 : kblk * 2 + (p.factor != nullptr ? 64 : 0);
+          }
+          mbar_expect_tx(&full_bar[s], bytes);
+        }
+        __syncwarp();
+        for (int u = 0; u < n_here; ++u) {
+          const int idx = first + u;
+          __nv_bfloat16* dst = stages + (size_t)s * stage_elems + (size_t)u * (kblk + vblk);
+          if (pooled && idx < kp) {                                // S rows a copy
+            const int n = (min(WD_PAGE, blocks - idx * WD_PAGE) + S - 1) / S;
+            if (lane < n)
+              bulk_load(dst + lane * chunk, reinterpret_cast<const __nv_bfloat16*>(p.pooled) + ((size_t)pt[idx * (WD_PAGE / S) + lane] * p.nkv + kvh) * chunk,
+                        chunk * 2, &full_bar[s]);
+          } else if (lane < 2) {
+            const int page = pt[idx < kp ? idx : w0 + idx - kp];
+            if (lane == 0) bulk_load(dst, reinterpret_cast<const __nv_bfloat16*>(p.cache) + (size_t)page * page_elems + (size_t)kvh * kblk, kblk * 2, &full_bar[s]);
+            else if (p.factor != nullptr) bulk_load(dst + kblk, p.factor + (size_t)page * WD_PAGE, 64, &full_bar[s]);
+          }
+        }
+      }
+    } else if (lane == 0) {
       const size_t page_elems = (size_t)p.nkv * (kblk + vblk);
       for (int it = 0; it < n_iter; ++it) {
         const int s = it % WD_NSTAGE;
@@ -486,6 +705,7 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
   } else {
     float qv[GB][DPL];
     const float* bias[GB];
+    float slope[GB];
     const float q_mul = CAP ? query_scale(p, i) / p.softcap : query_scale(p, i) * LOG2E;   // q . k becomes the tanh argument / log2 units
     const float cap = p.softcap * LOG2E;
 #pragma unroll
@@ -494,6 +714,7 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
       const int h = kvh * G + (live ? grp0 + g : 0);
       const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)t * p.ld_q + (size_t)h * dk;
       bias[g] = p.bias == nullptr ? nullptr : p.bias + (size_t)h * (p.far + 1);
+      slope[g] = p.slope == nullptr ? 0.f : p.slope[h];
 #pragma unroll
       for (int v = 0; v < VEC; ++v) {
         const int c = (v * 8 + gl) * 8;
@@ -501,6 +722,7 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
         for (int e = 0; e < 8; ++e) qv[g][v * 8 + e] = live && c < dk ? __bfloat162float(qp[c + e]) * q_mul : 0.f;
       }
     }
+#pragma unroll 1
     for (int it = 0; it < n_iter; ++it) {
       const int s = it % WD_NSTAGE;
       float b[WD_STAGE_PAGES][GB];
@@ -509,10 +731,10 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
       for (int u = 0; u < WD_STAGE_PAGES; ++u) {          // the biases are fetched while the keys are still on their way
         const int idx = pb + it * WD_STAGE_PAGES + u;
         const int j = (idx < kp ? idx : w0 + idx - kp) * WD_PAGE + grp;
-        ok[u] = idx < pe && j <= i && (j >= lo || j < p.keep_first);
-        const int dist = min(max(i - j, 0), p.far);
+        ok[u] = idx < pe && (pooled && idx < kp ? j < blocks : j <= i && (j >= lo || j < p.keep_first));
+        const int dist = max(i - j, 0);
 #pragma unroll
-        for (int g = 0; g < GB; ++g) b[u][g] = bias[g] != nullptr ? __ldg(bias[g] + dist) : 0.f;
+        for (int g = 0; g < GB; ++g) b[u][g] = bias[g] != nullptr ? __ldg(bias[g] + min(dist, p.far)) : -slope[g] * (float)dist;
       }
       mbar_wait(&full_bar[s], (it / WD_NSTAGE) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
       const __nv_bfloat16* st = stages + (size_t)s * stage_elems;
@@ -520,6 +742,8 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
 #pragma unroll
       for (int u = 0; u < WD_STAGE_PAGES; ++u) {
         const __nv_bfloat16* kq = st + (size_t)u * (kblk + vblk) + grp * dk;
+        float fac = 1.0f;
+        if (TIED && p.factor != nullptr) fac = reinterpret_cast<const float*>(st + (size_t)u * (kblk + vblk) + kblk)[grp];
         float se[GB], so[GB];
 #pragma unroll
         for (int g = 0; g < GB; ++g) { se[g] = 0.f; so[g] = 0.f; }
@@ -546,6 +770,7 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
           d += __shfl_xor_sync(0xffffffffu, d, 1);
           d += __shfl_xor_sync(0xffffffffu, d, 2);
           d += __shfl_xor_sync(0xffffffffu, d, 4);
+          if constexpr (TIED) d *= fac;
           if constexpr (CAP) d = cap * tanh_sfu(d);
           sc[u][g] = ok[u] ? d + b[u][g] : -INFINITY;
         }
@@ -564,7 +789,8 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
 #pragma unroll
       for (int u = 0; u < WD_STAGE_PAGES; ++u) {
         if (!ok[u]) continue;            // never touch stage memory that holds no visible key
-        const __nv_bfloat16* vq = st + (size_t)u * (kblk + vblk) + kblk + grp * dv;
+        const int v_off = TIED ? p.tied - 1 : kblk;              // (0 that the compiler does not know: keys kept in registers would spill)
+        const __nv_bfloat16* vq = st + (size_t)u * (kblk + vblk) + v_off + grp * dv;
         float pw[GB];
 #pragma unroll
         for (int g = 0; g < GB; ++g) {
@@ -633,7 +859,7 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
     const int h = kvh * G + grp0 + g;
     if (p.n_split == 1) {
       reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ld_out + (size_t)h * dv + d] =
-          __float2bfloat16_rn(num * finish_scale(p, t, h, mx, den));
+          __float2bfloat16_rn(num * finish_scale(p, t, h, mx, den) * element_gate(p, t, h, d));
     } else {
       float* w = p.ws + (((size_t)t * p.nq + h) * p.n_split + split) * (dv + 2);
       w[d] = num;
@@ -660,7 +886,7 @@ __global__ void __launch_bounds__(128) window_decode_merge_kernel(const WindowAt
       const float ms = w[s * stride + p.dv];
       if (ms != -INFINITY) num += exp2f(ms - mx) * w[s * stride + d];
     }
-    reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ld_out + (size_t)h * p.dv + d] = __float2bfloat16_rn(num * f);
+    reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ld_out + (size_t)h * p.dv + d] = __float2bfloat16_rn(num * f * element_gate(p, t, h, d));
   }
 }
 
@@ -679,17 +905,21 @@ struct WindowTiles {
   int n_pages;                // pages of the pool (an index past it reads zeros)
   long long kv_ld;            // 0: paged cache; else the keys and values are rows [nkv * dk | nkv * dv] of this pitch, one per
                               // token, and a page is 16 consecutive rows
+  const int* pool_base;       // [n_tiles] first page (16 rows) of the tile's row in the matrix of pooled blocks
+  int n_pool_pages;
 };
 
-template <int HK, int HV>
+// TIED: a stage holds keys only (and their factors, 64 floats behind all stages), which the second product reads too
+template <int HK, int HV, bool TIED = false>
 struct WpCfg {
   static constexpr int BK = 64;
   static constexpr int QTILE = 128 * 64 * 2, KTILE = BK * 64 * 2;
   static constexpr int Q_BYTES = HK * QTILE, K_BYTES = HK * KTILE, V_BYTES = HV * KTILE;
   static constexpr int P_BYTES = 128 * BK * 2;
-  static constexpr int STAGE_BYTES = K_BYTES + V_BYTES;
-  static constexpr int NSTAGE = 2;
-  static constexpr int SMEM_BYTES = Q_BYTES + P_BYTES + NSTAGE * STAGE_BYTES + 128;
+  static constexpr int STAGE_BYTES = TIED ? K_BYTES : K_BYTES + V_BYTES;
+  static constexpr int NSTAGE = TIED ? 3 : 2;
+  static constexpr int FACTOR_BYTES = TIED ? NSTAGE * BK * 4 : 0;
+  static constexpr int SMEM_BYTES = Q_BYTES + P_BYTES + NSTAGE * STAGE_BYTES + FACTOR_BYTES + 128;
   static constexpr int XCOL = 64;                            // exchange columns between the two halves of a query
   static constexpr int TMEM_COLS = HV <= 2 ? 256 : 512;      // S at 0, O at 128
   static constexpr int MIN_CTAS = HK + HV <= 4 ? 2 : 1;
@@ -746,17 +976,19 @@ __device__ __forceinline__ void soft_cap32(float* v, float mul, float cap) {
   }
 }
 
-template <int HK, int HV, bool CAP>
-__global__ void __launch_bounds__(WP_THREADS, WpCfg<HK, HV>::MIN_CTAS)
+// TIED: tm_v describes the matrix of pooled blocks (or is unused), whose blocks come first
+template <int HK, int HV, bool CAP, bool TIED>
+__global__ void __launch_bounds__(WP_THREADS, WpCfg<HK, HV, TIED>::MIN_CTAS)
 window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                       const __grid_constant__ CUtensorMap tm_v, const WindowAttnParams p, const WindowTiles tl) {
-  using C = WpCfg<HK, HV>;
+  using C = WpCfg<HK, HV, TIED>;
   constexpr int BK = C::BK;
   extern __shared__ __align__(1024) uint8_t smem[];
   uint8_t* q_s = smem;
   uint8_t* p_s = q_s + C::Q_BYTES;
   uint8_t* kv_s = p_s + C::P_BYTES;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(kv_s + C::NSTAGE * C::STAGE_BYTES);
+  float* factor_s = reinterpret_cast<float*>(kv_s + C::NSTAGE * C::STAGE_BYTES);      // [NSTAGE][BK], tied
+  uint64_t* bars = reinterpret_cast<uint64_t*>(kv_s + C::NSTAGE * C::STAGE_BYTES + C::FACTOR_BYTES);
   uint64_t* q_full = bars;
   uint64_t* kv_full = bars + 1;
   uint64_t* kv_empty = kv_full + C::NSTAGE;
@@ -796,8 +1028,9 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   const int i0 = p.pos[q0], i_last = i0 + qn - 1;             // the tile's positions are consecutive
   int keep_end, lo0;
   visible_range(i0, p.window, p.keep_first, keep_end, lo0);
-  const int kb = (keep_end + BK - 1) / BK;                    // blocks of the kept part
-  const int w0 = max(lo0 / BK, kb);                           // first block of the window part
+  const bool pooled = TIED && p.pooled != nullptr;
+  const int kb = ((pooled ? visible_blocks(i_last, p.window, p.pool) : keep_end) + BK - 1) / BK;   // blocks of the kept or pooled part
+  const int w0 = pooled ? lo0 / BK : max(lo0 / BK, kb);       // first block of the window part
   const int total_blocks = kb + max(0, i_last / BK - w0 + 1);
 
   if (warp == 0) {
@@ -807,18 +1040,32 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 #pragma unroll
       for (int h = 0; h < HK; ++h) tma_load_2d(q_s + h * C::QTILE, &tm_q, head * p.dk + h * 64, q0, q_full);
       const int* pt = p.page_table + (size_t)p.row[q0] * p.max_pages;
-      const int last_page = i_last / WD_PAGE;
+      const int last_page = i_last / WD_PAGE, pool0 = pooled ? tl.pool_base[tile] : 0;
       for (int n = 0; n < total_blocks; ++n) {
         const int st = n % C::NSTAGE;
         const int b = n < kb ? n : w0 + n - kb;
+        const bool means = pooled && n < kb;
         int page[4];
 #pragma unroll
-        for (int u = 0; u < 4; ++u) page[u] = b * 4 + u <= last_page ? pt[b * 4 + u] : tl.n_pages;
+        for (int u = 0; u < 4; ++u) page[u] = means ? min(pool0 + b * 4 + u, tl.n_pool_pages) : b * 4 + u <= last_page ? pt[b * 4 + u] : tl.n_pages;
         mbar_wait(&kv_empty[st], ((n / C::NSTAGE) & 1) ^ 1, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
         if (*abort_flag) break;
-        mbar_expect_tx(&kv_full[st], C::STAGE_BYTES);
+        const bool factors = TIED && p.factor != nullptr && !means;
+        mbar_expect_tx(&kv_full[st], C::STAGE_BYTES + (factors ? BK * 4 : 0));
         uint8_t* ks = kv_s + st * C::STAGE_BYTES;
         uint8_t* vs = ks + C::K_BYTES;
+        if constexpr (TIED) {
+          if (factors) {
+#pragma unroll
+            for (int u = 0; u < 4; ++u)                       // a page past the last key: any finite numbers
+              bulk_load(factor_s + st * BK + u * WD_PAGE, p.factor + (size_t)min(page[u], tl.n_pages - 1) * WD_PAGE, WD_PAGE * 4, &kv_full[st]);
+          }
+#pragma unroll
+          for (int u = 0; u < 4; ++u)
+#pragma unroll
+            for (int h = 0; h < HK; ++h) tma_load_4d(ks + h * C::KTILE + u * 2048, means ? &tm_v : &tm_k, h * 64, 0, kvh, page[u], &kv_full[st]);
+          continue;
+        }
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
 #pragma unroll
@@ -841,7 +1088,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         mbar_wait(&kv_full[st], (n / C::NSTAGE) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
         tc_fence_after();
         const uint32_t k_addr = smem_u32(kv_s + st * C::STAGE_BYTES);
-        const uint32_t v_addr = k_addr + C::K_BYTES;
+        const uint32_t v_addr = TIED ? k_addr : k_addr + C::K_BYTES;
 #pragma unroll
         for (int ks = 0; ks < HK * 4; ++ks) {
           const uint32_t qo = (ks / 4) * C::QTILE + (ks % 4) * 32;
@@ -874,6 +1121,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     const int lo_w1 = p.window > iw1 ? 0 : iw1 - p.window + 1;
     const float* bias = p.bias == nullptr ? nullptr : p.bias + (size_t)head * (p.far + 1);
     const float far_bias = bias == nullptr ? 0.f : bias[p.far];
+    const float slope = p.slope == nullptr ? 0.f : p.slope[head];
+    const int blocks = pooled ? visible_blocks(i, p.window, p.pool) : 0;
     float m_ref = -INFINITY, l = 0.f;
     for (int n = 0; n < total_blocks; ++n) {
       const int j0 = (n < kb ? n : w0 + n - kb) * BK + half * 32;        // first key column of this thread
@@ -883,8 +1132,25 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       tmem_ld32(tmem_s + lane_off + half * 32, sv);
       tmem_ld_wait();
       const int dmin = iw0 - (j0 + 31), dmax = iw1 - j0;                 // distances inside the warp's 32 x 32 patch
+      const bool means = pooled && n < kb;
       if constexpr (CAP) soft_cap32(sv, cap_mul, cap);
-      if (CAP && bias == nullptr) {
+      if constexpr (TIED) {
+        if (p.factor != nullptr && !means) {
+          const int st = n % C::NSTAGE;
+          mbar_wait(&kv_full[st], (n / C::NSTAGE) & 1, abort_flag, p.status, STATUS_TIMEOUT_TMA_FULL);
+          const float4* f4 = reinterpret_cast<const float4*>(factor_s + st * BK + half * 32);
+#pragma unroll
+          for (int c = 0; c < 8; ++c) {
+            const float4 f = f4[c];
+            sv[4 * c] *= f.x; sv[4 * c + 1] *= f.y; sv[4 * c + 2] *= f.z; sv[4 * c + 3] *= f.w;
+          }
+        }
+      }
+      if (p.slope != nullptr) {
+        const float d0 = -slope * (float)(i - j0);
+#pragma unroll
+        for (int c = 0; c < 32; ++c) sv[c] = fmaf(sv[c], sc, fmaf(slope, (float)c, d0));
+      } else if (CAP && bias == nullptr) {
       } else if (bias == nullptr || dmin >= p.far) {
 #pragma unroll
         for (int c = 0; c < 32; ++c) sv[c] = fmaf(sv[c], sc, far_bias);
@@ -896,7 +1162,11 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 #pragma unroll
         for (int c = 0; c < 32; ++c) sv[c] = fmaf(sv[c], sc, __ldg(bias + min(max(i - j0 - c, 0), p.far)));
       }
-      if (!(dmin >= 0 && (j0 >= lo_w1 || j0 + 31 < p.keep_first))) {
+      if (means) {
+#pragma unroll
+        for (int c = 0; c < 32; ++c)
+          if (j0 + c >= blocks) sv[c] = -INFINITY;
+      } else if (!(dmin >= 0 && (j0 >= lo_w1 || j0 + 31 < p.keep_first))) {
 #pragma unroll
         for (int c = 0; c < 32; ++c) {
           const int j = j0 + c;
@@ -1000,20 +1270,20 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   }
 }
 
-template <int VEC, int GB, bool EXACT, bool CAP>
+template <int VEC, int GB, bool EXACT, bool CAP, bool TIED>
 static int launch_window_decode_as(const WindowAttnParams& p, cudaStream_t stream) {
   const int groups = (p.nq / p.nkv + GB - 1) / GB;
-  const size_t ring = (size_t)WD_NSTAGE * WD_STAGE_PAGES * WD_PAGE * (p.dk + p.dv) * 2 + 128;
+  const size_t ring = (size_t)WD_NSTAGE * WD_STAGE_PAGES * WD_PAGE * (p.dk + (TIED ? 2 : p.dv)) * 2 + 128;
   const size_t merge = (size_t)16 * GB * (p.dv + 2) * 4;
   const size_t smem = ring > merge ? ring : merge;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(window_decode_kernel<VEC, GB, EXACT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
+    if (cudaFuncSetAttribute(window_decode_kernel<VEC, GB, EXACT, CAP, TIED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
       return -10;
     configured = true;
   }
   if (smem > 160 * 1024) return -11;
-  cudaError_t e = launch_chain(window_decode_kernel<VEC, GB, EXACT, CAP>, dim3(p.nkv * groups, p.n, p.n_split), dim3(160), smem, stream, p);
+  cudaError_t e = launch_chain(window_decode_kernel<VEC, GB, EXACT, CAP, TIED>, dim3(p.nkv * groups, p.n, p.n_split), dim3(160), smem, stream, p);
   if (e == cudaSuccess && p.n_split > 1)
     e = launch_chain(window_decode_merge_kernel, dim3(p.n * p.nq), dim3(128), 0, stream, p);
   return e == cudaSuccess ? 0 : -3;
@@ -1022,9 +1292,11 @@ static int launch_window_decode_as(const WindowAttnParams& p, cudaStream_t strea
 template <int VEC, int GB>
 static int launch_window_decode(const WindowAttnParams& p, cudaStream_t stream) {
   const bool exact = p.dk == VEC * 64 && p.dv == VEC * 64;
+  if (p.tied)
+    return exact ? launch_window_decode_as<VEC, GB, true, false, true>(p, stream) : launch_window_decode_as<VEC, GB, false, false, true>(p, stream);
   if (p.softcap > 0.f)
-    return exact ? launch_window_decode_as<VEC, GB, true, true>(p, stream) : launch_window_decode_as<VEC, GB, false, true>(p, stream);
-  return exact ? launch_window_decode_as<VEC, GB, true, false>(p, stream) : launch_window_decode_as<VEC, GB, false, false>(p, stream);
+    return exact ? launch_window_decode_as<VEC, GB, true, true, false>(p, stream) : launch_window_decode_as<VEC, GB, false, true, false>(p, stream);
+  return exact ? launch_window_decode_as<VEC, GB, true, false, false>(p, stream) : launch_window_decode_as<VEC, GB, false, false, false>(p, stream);
 }
 
 // K (or V) of a paged cache as a 4-D tensor [pages][kv heads][16 tokens][dims], read in boxes of one page's 16 tokens x 64 dims;
@@ -1042,23 +1314,26 @@ static int make_page_map(CUtensorMap* m, const void* base, int d, int nkv, int n
   return r == CUDA_SUCCESS ? 0 : -3;
 }
 
-template <int HK, int HV, bool CAP>
+template <int HK, int HV, bool CAP, bool TIED = false>
 static int launch_window_prefill_as(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
                                  const WindowAttnParams& p, const WindowTiles& tl, int n_tiles, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(window_prefill_kernel<HK, HV, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             WpCfg<HK, HV>::SMEM_BYTES) != cudaSuccess)
+    if (cudaFuncSetAttribute(window_prefill_kernel<HK, HV, CAP, TIED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             WpCfg<HK, HV, TIED>::SMEM_BYTES) != cudaSuccess)
       return -10;
     configured = true;
   }
-  window_prefill_kernel<HK, HV, CAP><<<dim3(n_tiles, p.nq), WP_THREADS, WpCfg<HK, HV>::SMEM_BYTES, stream>>>(mq, mk, mv, p, tl);
+  window_prefill_kernel<HK, HV, CAP, TIED><<<dim3(n_tiles, p.nq), WP_THREADS, WpCfg<HK, HV, TIED>::SMEM_BYTES, stream>>>(mq, mk, mv, p, tl);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
 template <int HK, int HV>
 static int launch_window_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
                                  const WindowAttnParams& p, const WindowTiles& tl, int n_tiles, cudaStream_t stream) {
+  if constexpr (HK == HV) {
+    if (p.tied) return launch_window_prefill_as<HK, HV, false, true>(mq, mk, mv, p, tl, n_tiles, stream);
+  }
   return p.softcap > 0.f ? launch_window_prefill_as<HK, HV, true>(mq, mk, mv, p, tl, n_tiles, stream)
                          : launch_window_prefill_as<HK, HV, false>(mq, mk, mv, p, tl, n_tiles, stream);
 }
@@ -1106,9 +1381,49 @@ extern "C" int tahb_qkv_post(const QkvPostParams* q, int f32, cudaStream_t strea
 }
 
 static int check_window_attn(const WindowAttnParams* p) {
+  // tied layers: one size; pooled blocks are a tied layer's, in the place of kept tokens, and have no position
+  if (p->tied && (p->tied != 1 || p->dk != p->dv || p->softcap != 0.f)) return -2;
+  if (!p->tied && (p->factor != nullptr || p->pooled != nullptr)) return -2;
+  if (p->pooled != nullptr && (p->pool < 1 || p->pool_rows < 1 || p->pool_rows > 16 || (p->pool_rows & (p->pool_rows - 1)) ||
+                               p->pool_rows * p->pool < 16 || p->keep_first != 0 || p->factor != nullptr || p->slope != nullptr || p->bias != nullptr))
+    return -2;
+  if (p->slope != nullptr && p->bias != nullptr) return -2;
+  if (p->gate != nullptr && p->wide_gate != nullptr) return -2;
   return p->nkv <= 0 || p->nq % p->nkv || p->dk > 256 || p->dv > 256 || p->dk % 8 || p->dv % 8 || p->window < 1 || p->far < 0 ||
          p->keep_first < 0 || p->ld_q < (long long)p->nq * p->dk || p->softcap < 0.f ||
          (p->temp_coef != 0.f && !(p->temp_every > 0.0)) ? -2 : 0;
+}
+
+// Keys (and block means) of a tied layer without norms to the cache.
+extern "C" int tahb_tied_keys(const TiedKeysParams* p, int f32, cudaStream_t stream) {
+  if (p->M <= 0) return 0;
+  if (p->dk > 256 || p->dk % 8 || p->ld % 8 || p->nkv < 1 ||
+      (p->pooled != nullptr && (p->pool < 1 || p->pool_rows < 1 || (long long)p->pool_rows * p->pool < p->page_size)))
+    return -2;
+  const long long warps = (long long)p->M * p->nkv;
+  const dim3 grid((unsigned)((warps + 3) / 4));
+  cudaError_t e = f32 ? launch_chain(tied_keys_kernel<float>, grid, dim3(128), 0, stream, *p)
+                      : launch_chain(tied_keys_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, *p);
+  return e == cudaSuccess ? 0 : -3;
+}
+
+// n rows of nkv * row_bytes; src: pooled rows (see pool_gather_kernel)
+extern "C" int tahb_pool_gather(const void* pooled, const int* src, int n, int nkv, int row_bytes, int pool_rows, int n_pages, void* out,
+                                cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (row_bytes % 16 || nkv < 1 || pool_rows < 1) return -2;
+  cudaError_t e = launch_chain(pool_gather_kernel, dim3(n), dim3(128), 0, stream, reinterpret_cast<const uint4*>(pooled), src, nkv,
+                               row_bytes / 16, pool_rows, n_pages, reinterpret_cast<uint4*>(out));
+  return e == cudaSuccess ? 0 : -3;
+}
+
+// Norms over all heads, queries out, keys and their factors to the cache.
+extern "C" int tahb_norm_all(const NormAllParams* p, int f32, cudaStream_t stream) {
+  if (p->M <= 0) return 0;
+  if (p->dk % 8 || p->dim > p->dk || p->ld % 8 || p->nq < 1 || p->nkv < 1) return -2;
+  cudaError_t e = f32 ? launch_chain(norm_all_kernel<float>, dim3(p->M), dim3(256), 0, stream, *p)
+                      : launch_chain(norm_all_kernel<__nv_bfloat16>, dim3(p->M), dim3(256), 0, stream, *p);
+  return e == cudaSuccess ? 0 : -3;
 }
 
 // Host-side description of one attention launch (same fields as WindowAttnParams).
@@ -1139,14 +1454,17 @@ extern "C" int tahb_window_attn_decode(const WindowAttnParams* p, cudaStream_t s
 }
 
 // Query tiles of portions; n_pages = pages of the layer's pool; kv_ld: see WindowTiles.  bias and sink in log2 units.
+// Tied layers with pooled blocks: p->pooled is a matrix [16 * n_pool_pages, nkv * dk] whose page pool_base[tile] is the first of the
+// tile's row.
 extern "C" int tahb_window_attn_tiles(const WindowAttnParams* p, const int* q0, const int* qn, int n_tiles, int n_pages,
-                                      long long kv_ld, cudaStream_t stream) {
+                                      long long kv_ld, const int* pool_base, int n_pool_pages, cudaStream_t stream) {
   if (p->n <= 0 || n_tiles <= 0) return 0;
   if (check_window_attn(p) || p->ld_out % 8 || (p->wide_gate != nullptr && (p->ld_gate % 8 || (reinterpret_cast<uintptr_t>(p->wide_gate) & 15))))
     return -2;
   if (kv_ld != 0 && kv_ld < (long long)p->nkv * (p->dk + p->dv)) return -2;
+  if (p->tied && (kv_ld != 0 || n_pages < 1 || (p->pooled != nullptr && pool_base == nullptr))) return -2;
   if (p->page_size != WD_PAGE) return -5;
-  const size_t page_elems = (size_t)p->nkv * WD_PAGE * (p->dk + p->dv);
+  const size_t page_elems = (size_t)p->nkv * WD_PAGE * (p->dk + (p->tied ? 0 : p->dv));
   CUtensorMap mq, mk, mv;
   int rc;
   if ((rc = make_query_map(&mq, p->q, p->n, (long long)p->nq * p->dk, p->ld_q))) return rc;
@@ -1156,10 +1474,15 @@ extern "C" int tahb_window_attn_tiles(const WindowAttnParams* p, const int* q0, 
     if ((rc = make_page_map(&mv, kv + (size_t)p->nkv * p->dk, p->dv, p->nkv, n_pages, kv_ld, p->dv, WD_PAGE * kv_ld))) return rc;
   } else {
     if ((rc = make_page_map(&mk, kv, p->dk, p->nkv, n_pages, p->dk, (size_t)WD_PAGE * p->dk, page_elems))) return rc;
-    if ((rc = make_page_map(&mv, kv + (size_t)p->nkv * WD_PAGE * p->dk, p->dv, p->nkv, n_pages, p->dv, (size_t)WD_PAGE * p->dv,
+    mv = mk;
+    const long long pool_ld = (long long)p->nkv * p->dk;
+    if (p->pooled != nullptr && n_pool_pages > 0 &&
+        (rc = make_page_map(&mv, p->pooled, p->dk, p->nkv, n_pool_pages, pool_ld, p->dk, WD_PAGE * pool_ld)))
+      return rc;
+    if (!p->tied && (rc = make_page_map(&mv, kv + (size_t)p->nkv * WD_PAGE * p->dk, p->dv, p->nkv, n_pages, p->dv, (size_t)WD_PAGE * p->dv,
                             page_elems))) return rc;
   }
-  WindowTiles tl{q0, qn, n_pages, kv_ld};
+  WindowTiles tl{q0, qn, n_pages, kv_ld, pool_base, n_pool_pages};
   const int hk = p->dk <= 64 ? 1 : p->dk <= 128 ? 2 : 4, hv = p->dv <= 64 ? 1 : p->dv <= 128 ? 2 : 4;
   if (p->softcap == 0.f && p->dk > 128 && p->dk <= 192 && p->dv <= 128)
     return p->dv <= 64 ? launch_window_prefill_as<3, 1, false>(mq, mk, mv, *p, tl, n_tiles, stream)

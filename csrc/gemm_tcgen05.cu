@@ -51,7 +51,8 @@ struct GemmParams {
   int splits;   // cluster size along z (1 = no split-K)
   int tma_out;  // 1: stage the output tile in shared memory and write it with a TMA store
   int act;      // epilogue activation on the (non-dual) output: 0 none, 1 GELU (erf form) of the bf16-rounded value,
-                // 2 SwiGLU of interleaved gate / up rows (out has F / 2 features)
+                // 2 SwiGLU of interleaved gate / up rows (out has F / 2 features), 3 xIELU of the bf16-rounded value
+  float act_up, act_low;   // xIELU: up z^2 + z / 2 above zero, low (exp(z) - 1 - z) + z / 2 below
   // Operand majors (backward GEMMs read their operands transposed, straight from the row-major tensors):
   //   a_mn: the 128-row operand is stored [reduction, feature] (feature contiguous): dgrad reads W[F, K] as
   //         W^T, wgrad reads X[T, K] as X^T;   b_mn: the column operand is stored [reduction, column]
@@ -152,6 +153,20 @@ __device__ __noinline__ void gelu_tile(__nv_bfloat16* stg, int n_tok) {
   for (int i = e; i < n_tok * 64; i += 128) {
     const float2 f = __bfloat1622float2(v[i]);
     v[i] = __floats2bfloat162_rn(gelu_erf(f.x), gelu_erf(f.y));
+  }
+}
+
+// The same for xIELU.
+__device__ __noinline__ void xielu_tile(__nv_bfloat16* stg, int n_tok, float up, float low) {
+  __nv_bfloat162* v = reinterpret_cast<__nv_bfloat162*>(stg);
+  auto act = [&](float z) {
+    const float neg = low * (ex2_approx(z * 1.4426950408889634f) - 1.0f - z);
+    return fmaf(0.5f, z, z > 0.f ? up * z * z : neg);
+  };
+#pragma unroll 4
+  for (int i = threadIdx.x - 64; i < n_tok * 64; i += 128) {
+    const float2 f = __bfloat1622float2(v[i]);
+    v[i] = __floats2bfloat162_rn(act(f.x), act(f.y));
   }
 }
 
@@ -530,6 +545,10 @@ gemm_fl_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           push_rows(p, stg, t0, BN, f0);
           push_rows(p, stg1, t0, BN, p.up_off + f0);
         } else {
+          if (p.act == 3) {
+            named_bar_sync(1, 128);
+            xielu_tile(stg, 2 * BN, p.act_up, p.act_low);
+          }
           fence_proxy_async_smem();
           named_bar_sync(1, 128);
           if (threadIdx.x == 64) {
@@ -580,6 +599,9 @@ gemm_fl_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         if (p.act == 1) {
           named_bar_sync(1, 128);
           gelu_tile(stg, BN);
+        } else if (p.act == 3) {
+          named_bar_sync(1, 128);
+          xielu_tile(stg, BN, p.act_up, p.act_low);
         }
         fence_proxy_async_smem();
         named_bar_sync(1, 128);
@@ -689,6 +711,9 @@ gemm_fl_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         if (p.act == 1) {
           named_bar_sync(1, 128);
           gelu_tile(stg, per);
+        } else if (p.act == 3) {
+          named_bar_sync(1, 128);
+          xielu_tile(stg, per, p.act_up, p.act_low);
         }
         fence_proxy_async_smem();
         named_bar_sync(1, 128);
@@ -837,7 +862,7 @@ static int gemm_impl(const void* W, const void* X, void* out, const void* residu
                      const void* X2, int M, int F, int K, int R, long long ldw, long long ldx, long long ldo,
                      long long ldr, long long ldw2, long long ldx2, int dual, int up_off, int splits, int bn,
                      int* status, cudaStream_t stream, const GemmTpArgs& tp, const TahbQkvEpilogue* qkv = nullptr,
-                     int a_mn = 0, int b_mn = 0, int k_rows = 0) {
+                     int a_mn = 0, int b_mn = 0, int k_rows = 0, const float* xielu = nullptr) {
   if (M <= 0 || F <= 0) return 0;
   // transposed operands: W is then [K, F] (ldw = its row pitch), X is [K, M]; no LoRA extension, no dual
   if ((a_mn || b_mn) && (dual == 1 || dual == 6 || R > 0 || qkv != nullptr || tp.push_world > 0)) return -27;
@@ -852,7 +877,8 @@ static int gemm_impl(const void* W, const void* X, void* out, const void* residu
   //     tile, unsplit; 6 = pair + interleaved SwiGLU.  The pair forms halve the activation bytes per unit of work
   //     and are the fast ones at large token counts (1350-1400 vs 915-1100 TFLOP/s at 8192+ tokens).
   const bool pair = dual == 2 || dual == 6;
-  const int act = dual == 3 ? 1 : (dual == 4 || dual == 6) ? 2 : 0;
+  const int act = xielu != nullptr ? 3 : dual == 3 ? 1 : (dual == 4 || dual == 6) ? 2 : 0;
+  if (act == 3 && ((dual != 0 && dual != 2) || push || residual != nullptr || qkv != nullptr || a_mn || b_mn)) return -29;
   if (dual == 3 || dual == 4) dual = 0;
   if (act == 2 && (F % 2 || splits > 1 || push || residual != nullptr || qkv != nullptr || a_mn || b_mn)) return -29;
   const int F_full = F;
@@ -921,6 +947,8 @@ static int gemm_impl(const void* W, const void* X, void* out, const void* residu
     p.rope_cs = nullptr;
   }
   p.act = act;
+  p.act_up = xielu != nullptr ? xielu[0] : 0.f;
+  p.act_low = xielu != nullptr ? xielu[1] : 0.f;
   p.a_mn = a_mn;
   p.b_mn = b_mn;
   p.push_ld = F_full;
@@ -967,6 +995,14 @@ extern "C" int tahb_gemm(const void* W, const void* X, void* out, const void* re
                          int* status, cudaStream_t stream) {
   return gemm_impl(W, X, out, residual, W2, X2, M, F, K, R, ldw, ldx, ldo, ldr, ldw2, ldx2, dual, up_off, splits, bn,
                    status, stream, GemmTpArgs());
+}
+
+// out = xIELU(X W^T): up z^2 + z / 2 for z > 0, low (exp(z) - 1 - z) + z / 2 otherwise, z rounded to bf16.  pair: the two-tile form.
+extern "C" int tahb_gemm_xielu(const void* W, const void* X, void* out, int M, int F, int K, long long ldw, long long ldx,
+                               long long ldo, float up, float low, int pair, int splits, int bn, int* status, cudaStream_t stream) {
+  const float act[2] = {up, low};
+  return gemm_impl(W, X, out, nullptr, nullptr, nullptr, M, F, K, 0, ldw, ldx, ldo, 0, 0, 0, pair ? 2 : 0, 0, splits, bn, status, stream,
+                   GemmTpArgs(), nullptr, 0, 0, 0, act);
 }
 
 // Tensor-parallel variants of the same GEMM (see GemmParams): `push_*` turns the epilogue into a

@@ -6,6 +6,9 @@
 //   streams_norm         x_t <- sum_s mix[s][t] x_s + out[t] * y;        h = T(rms_g(sum_t in[t] x_t) * w_next)
 //
 // with rms(v) = v / sqrt(mean(v^2) + eps), and rms_g the same over each of `groups` equal consecutive parts of the vector.
+// embed_norm and residual_norm also exist with layer norms, (v - mean) / sqrt(variance + eps), in the place of rms, and both can
+// add a vector to the residual in front of the last norm; residual_norm also the scaled embedding, which makes it the seam
+// between two passes of a range of layers that runs several times.
 // residual_norm is the whole seam between two sublayers of a layer with a norm before and after each sublayer: y is the
 // sublayer's output projection, w_out the product of the output norm's weight and the layer scale, w_next the weight of the
 // norm that feeds the next projection.  residual_add_norm is the seam between two layers whose mixer and feed-forward run
@@ -110,6 +113,38 @@ __device__ __forceinline__ void group_inv_rms(const float4* v, int width, int gr
   }
 }
 
+// Mean and inverse standard deviation of a row whose vectors c = threadIdx.x + i * RN_THREADS sit in v[i]; the deviations of its
+// `width` real elements are squared after the mean is known.
+template <int VPT>
+__device__ __forceinline__ float2 row_moments(const float4* v, int width, int nvec, float eps, float* red) {
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i)
+    if (threadIdx.x + i * RN_THREADS < nvec) s += v[i].x + v[i].y + v[i].z + v[i].w;
+  const float mean = block_sum_128(s, red) / (float)width;
+  s = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = 4 * (threadIdx.x + i * RN_THREADS);
+    if (c < width) s += (v[i].x - mean) * (v[i].x - mean);
+    if (c + 1 < width) s += (v[i].y - mean) * (v[i].y - mean);
+    if (c + 2 < width) s += (v[i].z - mean) * (v[i].z - mean);
+    if (c + 3 < width) s += (v[i].w - mean) * (v[i].w - mean);
+  }
+  return make_float2(mean, 1.0f / sqrtf(block_sum_128(s, red) / (float)width + eps));
+}
+
+// (mean or 0, factor) of one of the two norms
+template <int VPT, bool CENTER>
+__device__ __forceinline__ float2 row_norm(const float4* v, int width, int nvec, float eps, float* red) {
+  if constexpr (CENTER) return row_moments<VPT>(v, width, nvec, eps, red);
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i)
+    if (threadIdx.x + i * RN_THREADS < nvec) s += sq4(v[i]);
+  return make_float2(0.f, 1.0f / sqrtf(block_sum_128(s, red) / (float)width + eps));
+}
+
 static size_t group_rms_smem(int width, int groups, int ld) {
   return (64 + (size_t)groups + ((width / groups) % 128 ? ld : 0)) * 4;
 }
@@ -125,12 +160,13 @@ __device__ __forceinline__ float2 sin_cos_pair(float p, float hi, float lo) {
 
 // pos / freq: position of every token and [2, (width + 1) / 2] frequencies (high parts, then low parts), or null.
 // streams copies of the embedding go to x [M, streams, ld]; w_in [streams]: weights of their sum, which is what the norm
-// sees (null: one stream as it is).
-template <typename T, int VPT>
+// sees (null: one stream as it is).  add [ld]: vector added to the scaled embedding (zero in the padding), or null.  CENTER: layer
+// norm (groups is 1).
+template <typename T, int VPT, bool CENTER>
 __global__ void __launch_bounds__(RN_THREADS) embed_norm_kernel(const T* __restrict__ E, const int* __restrict__ tok,
                                                                 float scale, const int* __restrict__ pos,
                                                                 const float* __restrict__ freq, int streams, const float* __restrict__ w_in,
-                                                                float* __restrict__ x, const float* __restrict__ w,
+                                                                const float* __restrict__ add, float* __restrict__ x, const float* __restrict__ w,
                                                                 T* __restrict__ h, int vocab, int width, int groups, int ld,
                                                                 float eps) {
   pdl_launch_dependents();
@@ -165,11 +201,24 @@ __global__ void __launch_bounds__(RN_THREADS) embed_norm_kernel(const T* __restr
           if (4 * c + 3 < width) v[i].w += a.y;
         }
       }
+      if (add != nullptr) {
+        const float4 a = Vec4<float>::load(add + c * 4);
+        v[i].x += a.x; v[i].y += a.y; v[i].z += a.z; v[i].w += a.w;
+      }
       for (int s = 0; s < streams; ++s) Vec4<float>::store(x + (row * streams + s) * ld + c * 4, v[i]);
       v[i].x *= sum_in; v[i].y *= sum_in; v[i].z *= sum_in; v[i].w *= sum_in;
     }
   }
-  group_inv_rms<VPT>(v, width, groups, ld, eps, gsm, r);
+  if constexpr (CENTER) {
+    const float2 n = row_moments<VPT>(v, width, nvec, eps, gsm);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      v[i].x -= n.x; v[i].y -= n.x; v[i].z -= n.x; v[i].w -= n.x;
+      r[i] = make_float4(n.y, n.y, n.y, n.y);
+    }
+  } else {
+    group_inv_rms<VPT>(v, width, groups, ld, eps, gsm, r);
+  }
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * RN_THREADS;
@@ -343,46 +392,75 @@ __global__ void rotary_table_kernel(const int* __restrict__ pos, const float* __
   }
 }
 
-template <typename T, int VPT>
-__global__ void __launch_bounds__(RN_THREADS) residual_norm_kernel(const T* __restrict__ y, long long ldy,
-                                                                   float* __restrict__ x, const float* __restrict__ w_out,
-                                                                   const float* __restrict__ w_next, T* __restrict__ h,
-                                                                   int width, int ld, float eps) {
+struct ResidualNormParams {
+  const void* y;              // [M, ldy]
+  long long ldy;
+  float* x;                   // [M, ld]
+  const float* w_out;
+  const float* w_next;
+  void* h;                    // [M, ld]
+  int width, ld;
+  float eps;
+  const float* add;           // [ld] added to the residual behind the sublayer's sum, or null
+  const void* E;              // embedding table [vocab, ld] whose rows, times scale, are added too, or null
+  const int* tok;             // [M], with E
+  int vocab;
+  float scale;
+  float* before;              // [M, ld] receives the residual as it is before these two, or null
+};
+
+// CENTER: layer norms; ENTER: add / E / before may be given
+template <typename T, int VPT, bool CENTER, bool ENTER>
+__global__ void __launch_bounds__(RN_THREADS) residual_norm_kernel(const ResidualNormParams p) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[4];
   const size_t row = blockIdx.x;
-  const int nvec = ld / 4;
+  const int nvec = p.ld / 4;
+  const T* y = reinterpret_cast<const T*>(p.y) + row * p.ldy;
+  float* x = p.x + row * p.ld;
   float4 u[VPT], v[VPT];
-  float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * RN_THREADS;
     if (c < nvec) {
-      u[i] = Vec4<T>::load(y + row * ldy + c * 4);
-      v[i] = Vec4<float>::load(x + row * ld + c * 4);
-      ss += sq4(u[i]);
+      u[i] = Vec4<T>::load(y + c * 4);
+      v[i] = Vec4<float>::load(x + c * 4);
     }
   }
-  const float ry = 1.0f / sqrtf(block_sum_128(ss, red) / (float)width + eps);
-  ss = 0.f;
+  const float2 ny = row_norm<VPT, CENTER>(u, p.width, nvec, p.eps, red);
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * RN_THREADS;
     if (c < nvec) {
-      const float4 g = Vec4<float>::load(w_out + c * 4);
-      v[i].x += u[i].x * ry * g.x; v[i].y += u[i].y * ry * g.y; v[i].z += u[i].z * ry * g.z; v[i].w += u[i].w * ry * g.w;
-      ss += sq4(v[i]);
-      Vec4<float>::store(x + row * ld + c * 4, v[i]);
+      const float4 g = Vec4<float>::load(p.w_out + c * 4);
+      if constexpr (CENTER) { u[i].x -= ny.x; u[i].y -= ny.x; u[i].z -= ny.x; u[i].w -= ny.x; }
+      v[i].x += u[i].x * ny.y * g.x; v[i].y += u[i].y * ny.y * g.y; v[i].z += u[i].z * ny.y * g.z; v[i].w += u[i].w * ny.y * g.w;
+      if constexpr (ENTER) {
+        if (p.before != nullptr) Vec4<float>::store(p.before + row * p.ld + c * 4, v[i]);
+        if (p.E != nullptr) {
+          const int id = min(max(p.tok[row], 0), p.vocab - 1);
+          const float4 e = Vec4<T>::load(reinterpret_cast<const T*>(p.E) + (size_t)id * p.ld + c * 4);
+          v[i].x = fmaf(p.scale, e.x, v[i].x); v[i].y = fmaf(p.scale, e.y, v[i].y);
+          v[i].z = fmaf(p.scale, e.z, v[i].z); v[i].w = fmaf(p.scale, e.w, v[i].w);
+        }
+        if (p.add != nullptr) {
+          const float4 a = Vec4<float>::load(p.add + c * 4);
+          v[i].x += a.x; v[i].y += a.y; v[i].z += a.z; v[i].w += a.w;
+        }
+      }
+      Vec4<float>::store(x + c * 4, v[i]);
     }
   }
-  const float rx = 1.0f / sqrtf(block_sum_128(ss, red) / (float)width + eps);
+  const float2 nx = row_norm<VPT, CENTER>(v, p.width, nvec, p.eps, red);
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * RN_THREADS;
     if (c < nvec) {
-      const float4 g = Vec4<float>::load(w_next + c * 4);
-      Vec4<T>::store(h + row * ld + c * 4, make_float4(v[i].x * rx * g.x, v[i].y * rx * g.y, v[i].z * rx * g.z, v[i].w * rx * g.w));
+      const float4 g = Vec4<float>::load(p.w_next + c * 4);
+      if constexpr (CENTER) { v[i].x -= nx.x; v[i].y -= nx.x; v[i].z -= nx.x; v[i].w -= nx.x; }
+      Vec4<T>::store(reinterpret_cast<T*>(p.h) + row * p.ld + c * 4,
+                     make_float4(v[i].x * nx.y * g.x, v[i].y * nx.y * g.y, v[i].z * nx.y * g.z, v[i].w * nx.y * g.w));
     }
   }
 }
@@ -540,16 +618,26 @@ __global__ void swiglu_f32_kernel(const float* __restrict__ gu, float* __restric
   }
 }
 
-template <typename T>
+// In place: up z^2 + z / 2 above zero, low (exp(z) - 1 - z) + z / 2 below
+__global__ void xielu_f32_kernel(float* __restrict__ x, float up, float low, int M, int I, long long ld) {
+  const long long n = (long long)M * I;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    float* q = x + i / I * ld + i % I;
+    const float z = *q;
+    *q = (z > 0.f ? up * z * z : low * (expm1f(z) - z)) + 0.5f * z;
+  }
+}
+
+template <typename T, bool CENTER>
 static int embed_norm_launch(const void* E, const int* tok, float scale, const int* pos, const float* freq, int streams,
-                             const float* w_in, float* x, const float* w, void* h, int M, int vocab, int width, int groups, int ld, float eps,
-                             cudaStream_t stream) {
+                             const float* w_in, const float* add, float* x, const float* w, void* h, int M, int vocab, int width,
+                             int groups, int ld, float eps, cudaStream_t stream) {
   const size_t smem = group_rms_smem(width, groups, ld);
   const int need = (ld / 4 + RN_THREADS - 1) / RN_THREADS;
   auto e = reinterpret_cast<const T*>(E);
   auto o = reinterpret_cast<T*>(h);
   cudaError_t rc;
-#define TAHB_EN(V_) rc = launch_chain(embed_norm_kernel<T, V_>, dim3(M), dim3(RN_THREADS), smem, stream, e, tok, scale, pos, freq, streams, w_in, x, w, o, vocab, width, groups, ld, eps)
+#define TAHB_EN(V_) rc = launch_chain(embed_norm_kernel<T, V_, CENTER>, dim3(M), dim3(RN_THREADS), smem, stream, e, tok, scale, pos, freq, streams, w_in, add, x, w, o, vocab, width, groups, ld, eps)
   if (need <= 1) TAHB_EN(1);
   else if (need <= 2) TAHB_EN(2);
   else if (need <= 4) TAHB_EN(4);
@@ -576,14 +664,11 @@ static int streams_norm_launch(const StreamsParams& p, int M, cudaStream_t strea
   return rc == cudaSuccess ? 0 : -3;
 }
 
-template <typename T>
-static int residual_norm_launch(const void* y, long long ldy, float* x, const float* w_out, const float* w_next, void* h,
-                                int M, int width, int ld, float eps, cudaStream_t stream) {
-  const int need = (ld / 4 + RN_THREADS - 1) / RN_THREADS;
-  auto yy = reinterpret_cast<const T*>(y);
-  auto o = reinterpret_cast<T*>(h);
+template <typename T, bool CENTER, bool ENTER>
+static int residual_norm_launch(const ResidualNormParams& p, int M, cudaStream_t stream) {
+  const int need = (p.ld / 4 + RN_THREADS - 1) / RN_THREADS;
   cudaError_t rc;
-#define TAHB_RN(V_) rc = launch_chain(residual_norm_kernel<T, V_>, dim3(M), dim3(RN_THREADS), 0, stream, yy, ldy, x, w_out, w_next, o, width, ld, eps)
+#define TAHB_RN(V_) rc = launch_chain(residual_norm_kernel<T, V_, CENTER, ENTER>, dim3(M), dim3(RN_THREADS), 0, stream, p)
   if (need <= 1) TAHB_RN(1);
   else if (need <= 2) TAHB_RN(2);
   else if (need <= 4) TAHB_RN(4);
@@ -636,16 +721,23 @@ static int few_linear_launch(const void* x, long long ldx, const void* w, const 
 
 using namespace tahb;
 
-// pos / freq: sinusoidal positions; streams / w_in: copies in x and the weights of their sum (see embed_norm_kernel).
-// groups must divide width.
+// pos / freq: sinusoidal positions; streams / w_in: copies in x and the weights of their sum; add: vector added to x (see
+// embed_norm_kernel).  groups must divide width; centered: layer norm, groups = 1.
 extern "C" int tahb_embed_norm(const void* E, const int* tok, float scale, const int* pos, const float* freq, int streams,
-                               const float* w_in, float* x, const float* w, void* h, int M, int vocab, int width, int groups,
-                               int ld, float eps, int f32, cudaStream_t stream) {
+                               const float* w_in, const float* add, float* x, const float* w, void* h, int M, int vocab, int width,
+                               int groups, int ld, float eps, int centered, int f32, cudaStream_t stream) {
   if (M <= 0) return 0;
-  if (ld % 4 || width > ld || groups < 1 || width % groups || (freq != nullptr && pos == nullptr) || streams < 1) return -1;
-  return f32 ? embed_norm_launch<float>(E, tok, scale, pos, freq, streams, w_in, x, w, h, M, vocab, width, groups, ld, eps, stream)
-             : embed_norm_launch<__nv_bfloat16>(E, tok, scale, pos, freq, streams, w_in, x, w, h, M, vocab, width, groups, ld, eps,
-                                                stream);
+  if (ld % 4 || width > ld || groups < 1 || width % groups || (freq != nullptr && pos == nullptr) || streams < 1 ||
+      (centered && groups != 1))
+    return -1;
+#define TAHB_EL(T_, C_) return embed_norm_launch<T_, C_>(E, tok, scale, pos, freq, streams, w_in, add, x, w, h, M, vocab, width, groups, ld, eps, stream)
+  if (centered) {
+    if (f32) TAHB_EL(float, true);
+    TAHB_EL(__nv_bfloat16, true);
+  }
+  if (f32) TAHB_EL(float, false);
+  TAHB_EL(__nv_bfloat16, false);
+#undef TAHB_EL
 }
 
 // Seam of hyper-connections over `streams` (1..8) residual streams (see streams_norm_kernel).
@@ -682,12 +774,17 @@ extern "C" int tahb_residual_add_norm(const void* y, long long ldy, const void* 
                                                        stream);
 }
 
-extern "C" int tahb_residual_norm(const void* y, long long ldy, float* x, const float* w_out, const float* w_next, void* h,
-                                  int M, int width, int ld, float eps, int f32, cudaStream_t stream) {
+// centered: layer norms in the place of the RMS norms (see residual_norm_kernel)
+extern "C" int tahb_residual_norm(const ResidualNormParams* p, int M, int centered, int f32, cudaStream_t stream) {
   if (M <= 0) return 0;
-  if (ld % 4 || ldy % 4 || width > ld) return -1;
-  return f32 ? residual_norm_launch<float>(y, ldy, x, w_out, w_next, h, M, width, ld, eps, stream)
-             : residual_norm_launch<__nv_bfloat16>(y, ldy, x, w_out, w_next, h, M, width, ld, eps, stream);
+  if (p->ld % 4 || p->ldy % 4 || p->width > p->ld || (p->E != nullptr && p->tok == nullptr)) return -1;
+  const bool enter = p->add != nullptr || p->E != nullptr || p->before != nullptr;
+#define TAHB_RL(T_) \
+  return centered ? (enter ? residual_norm_launch<T_, true, true>(*p, M, stream) : residual_norm_launch<T_, true, false>(*p, M, stream)) \
+                  : (enter ? residual_norm_launch<T_, false, true>(*p, M, stream) : residual_norm_launch<T_, false, false>(*p, M, stream))
+  if (f32) TAHB_RL(float);
+  TAHB_RL(__nv_bfloat16);
+#undef TAHB_RL
 }
 
 extern "C" int tahb_few_linear(const void* x, long long ldx, const void* w, const float* b, float* out, int M, int K, int F,
@@ -719,5 +816,13 @@ extern "C" int tahb_swiglu_f32(const float* gu, float* out, int M, int I, long l
   long long blocks = ((long long)M * I + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   swiglu_f32_kernel<<<(int)blocks, 256, 0, stream>>>(gu, out, M, I, ld_in, ld_out);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+extern "C" int tahb_xielu_f32(float* x, float up, float low, int M, int I, long long ld, cudaStream_t stream) {
+  if (M <= 0) return 0;
+  long long blocks = ((long long)M * I + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  xielu_f32_kernel<<<(int)blocks, 256, 0, stream>>>(x, up, low, M, I, ld);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

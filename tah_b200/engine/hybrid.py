@@ -1,6 +1,6 @@
 """HybridEngine: decoders that list their layers one by one - windowed attention and latent attention over the paged cache,
-recurrent layers with a state per row, dense feed-forwards and mixtures of experts, sublayers one after the other or side by
-side - on one or several fp32 residual streams.
+recurrent layers with a state per row, mixers of several branches, dense feed-forwards and mixtures of experts, sublayers one
+after the other or side by side, ranges of layers that run several times - on one or several fp32 residual streams.
 
 One function, :meth:`HybridEngine._layers`, runs the layers for a packed set of tokens.  It serves
 
@@ -23,8 +23,8 @@ import torch
 
 from tah_b200.engine.base import DecodeEngine
 from tah_b200.engine.kv_cache import CacheGeometry, LayerKV, PagedKVCache, RecurrentState
-from tah_b200.engine.hybrid_weights import (AttentionLayer, BlockWeights, GLALayer, HybridWeights, LatentLayer, MemoryLayer, MixtureLayer,
-                                             PolyNormLayer, distance_table)
+from tah_b200.engine.hybrid_weights import (AttentionLayer, BlockWeights, BranchesLayer, GLALayer, HybridWeights, LatentLayer, LayerRun,
+                                             MemoryLayer, MinGRULayer, MixtureLayer, PolyNormLayer, XIELULayer, distance_table, mixer_parts)
 from tah_b200.models.layered import LayeredForCausalLM
 from tah_b200.ops import cuda as K
 from tah_b200.utils.observe import nvtx_range
@@ -44,9 +44,12 @@ class _Plan:
     seq_start = seq_len = None
     tile_q0 = tile_qn = None
     groups = ()                   # recurrent launches: (tiles a..b, first tile and tile count of each of their portions)
-    latent = ()                   # latent expansions: (tiles a..b, cache pages of their portions)
+    latent = None                 # window -> (latent expansions: (tiles a..b, cache pages of their portions), table of their pages)
     latent_pages = 0              # pages of the largest of them
-    portion_of = latent_table = None      # portion of every token, and its pages inside the expansion
+    portion_of = None             # portion of every token
+    pooled = None                 # (window, block) -> (pooled rows that the portions see, first page of 16 of every tile)
+    pooled_rows = 0               # rows of the largest of them
+    longest = 0                   # tokens of the longest portion
 
 
 def decode_splits(m: AttentionLayer, n: int) -> int:
@@ -56,33 +59,44 @@ def decode_splits(m: AttentionLayer, n: int) -> int:
     g = m.spec.heads // m.spec.kv_heads
     ctas = n * m.spec.kv_heads * ((g + 3) // 4)
     pages = 64 if m.spec.window is None else (m.spec.window + m.spec.keep_first) // 16 + 1
+    if m.spec.pool is not None:
+        pages += 64 // m.spec.pool
     return max(1, min(K.SM_COUNT * 4 // ctas, pages // 4, 16))
 
 
 def latent_splits(m: LatentLayer, n: int) -> int:
-    """Key splits of the absorbed latent attention: the number whose CTA waves (one CTA per SM) cost least, for a context of
-    some sixteen 128-key tiles of 2.5 us and 3 us for start, end and merge of a CTA."""
+    """Key splits of the absorbed latent attention: the number whose CTA waves (one CTA per SM) cost least, at 20 ns per key and
+    3 us for start, end and merge of a CTA, for the window or a context of 2048 keys."""
     if n == 0 or not m.on_tensor_cores:
         return 1
     ctas = n * (1 if m.spec.heads <= 16 else (m.spec.heads + 31) // 32)
-    return min(range(1, 17), key=lambda s: -(-ctas * s // K.SM_COUNT) * (40.0 / s + 3.0))
+    us = 0.02 * (2048 if m.spec.window is None else min(2048, m.spec.window))
+    return min(range(1, 17), key=lambda s: -(-ctas * s // K.SM_COUNT) * (us / s + 3.0))
+
+
+def gru_splits(m: MinGRULayer, portions: int, longest: int) -> int:
+    """Segments of a portion in an elementwise recurrence: two CTAs of 64 channels per SM, segments of 256 tokens and more."""
+    ctas = portions * ((m.d + 63) // 64)
+    return max(1, min(-(-K.SM_COUNT * 2 // max(1, ctas)), longest // 256, 32))
 
 
 class _Buffers:
     """Activations of a pass over ``n`` tokens, the first ``n_dec`` of them single tokens; ``chunks``: chunks of a recurrent
-    layer's launch; ``latent_pages``: cache pages of a latent expansion."""
+    layer's launch; ``latent_pages``: cache pages of a latent expansion; ``pooled_rows``: rows of pooled blocks that portions
+    see; ``portions`` / ``longest``: number of portions and tokens of the longest."""
 
-    def __init__(self, w: HybridWeights, n: int, dtype, dev, n_dec: int, chunks: int = 0, latent_pages: int = 0):
+    def __init__(self, w: HybridWeights, n: int, dtype, dev, n_dec: int, chunks: int = 0, latent_pages: int = 0, pooled_rows: int = 0,
+                 portions: int = 0, longest: int = 0):
         e = lambda *s: torch.empty(*s, dtype=dtype, device=dev)
-        mix = [b.mixer for b in w.layers]
+        whole, mix = [b.mixer for b in w.layers], w.parts()
         moe = [b.ff for b in w.layers if isinstance(b.ff, MixtureLayer)]
         self.x = torch.empty((n, w.Wp) if w.streams is None else (n, w.streams, w.Wp), dtype=torch.float32, device=dev)
         self.h, self.y = e(n, w.Wp), e(n, w.Wp)
-        self.proj = e(n, max(m.w_in.shape[0] for m in mix))
+        self.proj = e(n, max(m.w_in.shape[0] for m in whole))
         self.q = e(n, max([m.spec.heads * m.dk for m in mix if isinstance(m, AttentionLayer) and m.own_queries] +
                           [m.w_uq.shape[0] for m in mix if isinstance(m, LatentLayer)] or [0]))
         # columns between heads * dv and the padded width meet zero weight columns; they only have to be finite
-        self.o = torch.zeros(n, max(m.w_o.shape[1] for m in mix), dtype=dtype, device=dev)
+        self.o = torch.zeros(n, max(m.w_o.shape[1] for m in whole), dtype=dtype, device=dev)
         self.gates = torch.empty(n * max([m.w_if.shape[0] for m in mix if isinstance(m, MemoryLayer)] or [0]),
                                  dtype=torch.float32, device=dev)
         f32 = lambda k: torch.empty(k, dtype=torch.float32, device=dev)
@@ -91,6 +105,8 @@ class _Buffers:
         self.mem_ws = f32(max([K.mlstm_chunk_ws_floats(chunks, m.spec.heads, m.dk, m.dv) for m in mix if isinstance(m, MemoryLayer)] +
                               [K.gla_chunk_ws_floats(n, chunks, m.spec.heads, m.dk, m.dv) for m in mix if chunks and isinstance(m, GLALayer)]
                               or [0]))
+        self.gru_ws = f32(max([portions * gru_splits(m, portions, longest) * 2 * m.d for m in mix if isinstance(m, MinGRULayer)] or [0]))
+        self.pooled = e(pooled_rows * max([m.nkv * m.dk for m in mix if isinstance(m, AttentionLayer) and m.spec.pool is not None] or [0]))
         self.low = f32(n * max([m.w_a1.shape[0] for m in mix if isinstance(m, GLALayer)] or [0]))
         self.rope = {r: f32(n * r.dims).view(n, r.dims // 2, 2) for r in w.rotary}
         self.v_first = e(n, max([m.nkv * m.dv for m in mix if isinstance(m, AttentionLayer) and m.spec.v_mix] or [0]))
@@ -152,20 +168,23 @@ class HybridEngine(DecodeEngine):
     # ------------------------------------------------------------------------------------------
     def _new_cache(self, rows: int, max_tokens: int, pool_tokens: Optional[int] = None) -> None:
         kv, st = [], []
-        for b in self.w.layers:
-            m = b.mixer
-            if isinstance(m, AttentionLayer):
-                kv.append(LayerKV(shared_with=m.spec.kv_from) if m.nkv == 0 else LayerKV(m.nkv, m.dk, m.dv))
-                st.append(None)
-            elif isinstance(m, LatentLayer):                 # one vector per token, key and value of all heads
-                kv.append(LayerKV(1, m.Rp + m.rw, 0))
-                st.append(None)
-            elif isinstance(m, GLALayer):
-                kv.append(None)
-                st.append([(m.spec.heads, m.dk, m.dv)])
-            else:
-                kv.append(None)
-                st.append([(m.spec.heads, m.dk, m.dv), (m.spec.heads, m.dk), (m.spec.heads,)])
+        for r in self.w.runs:                                # every run of a layer has a cache and a state of its own
+            cache, state = None, None
+            for m in mixer_parts(self.w.layers[r.layer].mixer):
+                if isinstance(m, AttentionLayer):
+                    s = m.spec
+                    cache = LayerKV(shared_with=s.kv_from) if m.nkv == 0 else \
+                        LayerKV(m.nkv, m.dk, 0 if s.keys_as_values else m.dv, factor=s.norm_all, block=s.pool)
+                elif isinstance(m, LatentLayer):             # one vector per token, key and value of all heads
+                    cache = LayerKV(1, m.Rp + m.rw, 0)
+                elif isinstance(m, GLALayer):
+                    state = [(m.spec.heads, m.dk, m.dv)]
+                elif isinstance(m, MinGRULayer):
+                    state = [(m.d,)]
+                else:
+                    state = [(m.spec.heads, m.dk, m.dv), (m.spec.heads, m.dk), (m.spec.heads,)]
+            kv.append(cache)
+            st.append(state)
         self.kv = self.state = None
         self._states.clear()                       # captured ticks point into the old pools
         torch.cuda.empty_cache()
@@ -194,10 +213,12 @@ class HybridEngine(DecodeEngine):
     # the layers
     # ------------------------------------------------------------------------------------------
     def _attention(self, li: int, m: AttentionLayer, proj: torch.Tensor, b: _Buffers, plan: _Plan) -> torch.Tensor:
-        """Attention of one layer from its projection ``proj``; returns ``b.o`` with the heads in its first columns."""
+        """Attention of one layer run from its projection ``proj``; returns ``b.o`` with the heads in its first columns."""
         s = m.spec
         n = b.h.shape[0]
         pool = self.kv.layer_pool(0, li)
+        if s.keys_as_values:
+            return self._attend(m, *self._tied_keys(li, m, proj, b, plan, pool), pool, proj, b, plan)
         post = dict(dk=m.dk, dv=m.dv, dim=s.dim, page_size=self.page_size, eps=self.cfg.rms_norm_eps)
         if m.own_queries:
             q = b.q.view(-1)[:n * s.heads * m.dk].view(n, s.heads * m.dk)
@@ -211,21 +232,64 @@ class HybridEngine(DecodeEngine):
             q = proj[:, :s.heads * m.dk]
             if m.nkv:
                 K.qkv_post(proj[:, m.kv_col:], None, None, None, None, pool, plan.slot, 0, m.nkv, **post)
-        o = b.o[:, :m.w_o.shape[1]]
-        kw = dict(nq=s.heads, nkv=s.kv_heads, dk=m.dk, dv=m.dv, page_size=self.page_size, scale=s.scale,
+        return self._attend(m, q, {}, pool, proj, b, plan)
+
+    def _tied_keys(self, li: int, m: AttentionLayer, proj, b: _Buffers, plan: _Plan, pool):
+        """Keys that are the values as well on their way to the cache, with the factors of their norm or the block means that they
+        complete; returns the queries and what attention has to know."""
+        s, n, pt = m.spec, b.h.shape[0], self.kv.page_table[0]
+        extra = dict(tied=True, factor=self.kv.factors[0][li], pooled=self.kv.pooled[0][li])
+        k = proj[:, m.kv_col:m.kv_col + m.nkv * m.dk]
+        if s.pool is not None:
+            extra.update(block=s.pool, pool_rows=self.kv.geo.layers[li].pool_rows(self.page_size))
+        if m.norm_w is None:
+            K.tied_keys(k, pool, plan.slot, plan.pos, plan.row, pt, m.nkv, m.dk, self.page_size, extra["pooled"],
+                        extra.get("block", 0), extra.get("pool_rows", 0))
+            return proj[:, :s.heads * m.dk], extra
+        q = b.q.view(-1)[:n * s.heads * m.dk].view(n, s.heads * m.dk)
+        K.norm_all(proj[:, :s.heads * m.dk], k, m.norm_w, q, pool, extra["factor"], plan.slot, nq=s.heads, nkv=m.nkv, dk=m.dk, dim=s.dim,
+                   page_size=self.page_size, eps=self.cfg.rms_norm_eps)
+        return q, extra
+
+    def _attend(self, m: AttentionLayer, q, extra: dict, pool, proj, b: _Buffers, plan: _Plan) -> torch.Tensor:
+        """Attention of queries ``q`` over the keys of ``pool``; ``extra``: see :meth:`_tied_keys`."""
+        s, n = m.spec, b.h.shape[0]
+        o = b.o if m.w_o is None else b.o[:, :m.w_o.shape[1]]
+        kw = dict(extra, slope=m.slope, out_scale=m.out_scale,
+                  nq=s.heads, nkv=s.kv_heads, dk=m.dk, dv=m.dv, page_size=self.page_size, scale=s.scale,
                   window=NO_WINDOW if s.window is None else s.window, keep_first=s.keep_first, bias=m.bias, sink=m.sink,
                   softcap=s.softcap, q_temp=s.q_temp)
+        if m.gate_col is not None:
+            kw["gate"] = proj[:, m.gate_col:m.gate_col + s.heads]
+        if m.wide_col is not None:
+            kw["wide_gate"] = proj[:, m.wide_col:m.wide_col + s.heads * m.dv]
         pt, nd = self.kv.page_table[0], plan.n_dec
-        gate = None if m.gate_col is None else proj[:, m.gate_col:m.gate_col + s.heads]
         if self.plain:
-            K.window_attn_plain(q, o, pool, pt, plan.pos, plan.row, gate=gate, **kw)
+            K.window_attn_plain(q, o, pool, pt, plan.pos, plan.row, **kw)
             return o
         if nd:
-            K.window_attn_decode(q[:nd], o[:nd], pool, pt, plan.pos, plan.row, gate=gate, n_split=decode_splits(m, nd),
-                                 ws=b.attn_ws, **kw)
+            K.window_attn_decode(q[:nd], o[:nd], pool, pt, plan.pos, plan.row, n_split=decode_splits(m, nd), ws=b.attn_ws, **kw)
         if nd < n:
-            K.window_attn_tiles(q, o, pool, pt, plan.pos, plan.row, plan.tile_q0, plan.tile_qn, self.kv.n_pages[0], gate=gate, **kw)
+            if s.pool is not None:                 # the block means that the portions see, as a matrix
+                src, base = plan.pooled[s.window, s.pool]
+                rows = src.numel()
+                kw["pooled"] = None if rows == 0 else K.pool_gather(kw["pooled"], src, m.nkv, m.dk, kw["pool_rows"],
+                                                                    b.pooled[:rows * m.nkv * m.dk].view(rows, m.nkv * m.dk))
+                kw["pool_base"] = base
+            K.window_attn_tiles(q, o, pool, pt, plan.pos, plan.row, plan.tile_q0, plan.tile_qn, self.kv.n_pages[0], **kw)
         return o
+
+    def _branches(self, li: int, m: BranchesLayer, proj: torch.Tensor, b: _Buffers, plan: _Plan) -> torch.Tensor:
+        """Attention and the elementwise recurrence, both scaled, side by side in ``b.o``."""
+        self._attention(li, m.left, proj, b, plan)
+        r, n, nd = m.right, b.h.shape[0], plan.n_dec
+        x, o, state = proj[:, r.in_col:], b.o[:, r.out_col:r.out_col + r.d], self.state.layers[li]
+        if nd:
+            K.min_gru_step(x[:nd], r.zb, r.xb, o[:nd], state, plan.pos, plan.row, r.out_scale, slot=plan.slot)
+        if nd < n:
+            K.min_gru_scan(x, r.zb, r.xb, o, state, plan.pos, plan.row, r.out_scale, seq_start=plan.seq_start, seq_len=plan.seq_len,
+                           n_split=gru_splits(r, plan.seq_start.numel(), plan.longest), ws=b.gru_ws)
+        return b.o[:, :m.w_o.shape[1]]
 
     def _memory(self, li: int, m: MemoryLayer, proj: torch.Tensor, b: _Buffers, plan: _Plan) -> torch.Tensor:
         s = m.spec
@@ -277,24 +341,27 @@ class HybridEngine(DecodeEngine):
         L = b.head_lists[nl, H] if nl else None
         list_q = view(b.list_q, L.rows, m.w_abs.shape[2]) if nl else None
         K.latent_query(q, rope, L, list_q, heads=H, dk=m.dk, dim=s.dim, rot=s.rot_dim)
-        o, gate = b.o[:, :m.w_o.shape[1]], proj[:, m.g_col:m.g_col + H * m.dv]
+        o, gate = b.o[:, :m.w_o.shape[1]], None if m.g_col is None else proj[:, m.g_col:m.g_col + H * m.dv]
+        window = NO_WINDOW if s.window is None else s.window
         if nl:
             qa = K.moe_linear(list_q, m.w_abs, L, view(b.list_qa, L.rows, m.w_abs.shape[1]))
             oc = view(b.list_o, L.rows, m.Rp)
-            kw = dict(Rp=m.Rp, rw=m.rw, page_size=self.page_size, scale=s.scale)
+            kw = dict(Rp=m.Rp, rw=m.rw, page_size=self.page_size, scale=s.scale, window=window)
             if m.on_tensor_cores:
                 K.latent_attn_decode(qa, oc, pool, self.kv.page_table[0], plan.pos, plan.row, L, sink=m.sink_log2,
                                      n_split=latent_splits(m, nl), ws=b.latent_ws, **kw)
             else:
                 K.latent_attn_plain(qa, oc, pool, self.kv.page_table[0], plan.pos, plan.row, L, sink=m.sink, **kw)
-            K.latent_gate(K.moe_linear(oc, m.w_uv, L, view(b.list_v, L.rows, m.w_uv.shape[1])), L, gate[:nl], o[:nl], m.dv)
+            K.latent_gate(K.moe_linear(oc, m.w_uv, L, view(b.list_v, L.rows, m.w_uv.shape[1])), L,
+                          None if gate is None else gate[:nl], o[:nl], m.dv)
         if nl < n:
-            for ta, tb, src in plan.latent:
+            launches, table = plan.latent[s.window]
+            for ta, tb, src in launches:
                 c = K.latent_gather(pool, src, self.page_size, m.Rp + m.rw, view(b.latents, src.numel() * 16, m.w_exp.shape[1]))
                 kv = K.linear(c, m.w_exp, out=view(b.expanded, c.shape[0], m.w_exp.shape[0]))
-                K.window_attn_tiles(q, o, kv, plan.latent_table, plan.pos, plan.portion_of, plan.tile_q0[ta:tb], plan.tile_qn[ta:tb],
+                K.window_attn_tiles(q, o, kv, table, plan.pos, plan.portion_of, plan.tile_q0[ta:tb], plan.tile_qn[ta:tb],
                                     src.numel(), kv_ld=kv.stride(0), nq=H, nkv=H, dk=m.dk, dv=m.dv, page_size=self.page_size,
-                                    scale=s.scale, window=NO_WINDOW, keep_first=0, sink=m.sink_log2, wide_gate=gate)
+                                    scale=s.scale, window=window, keep_first=0, sink=m.sink_log2, wide_gate=gate)
         return o
 
     def _mixture(self, f: MixtureLayer, proj: torch.Tensor, b: _Buffers):
@@ -334,59 +401,105 @@ class HybridEngine(DecodeEngine):
     def _layers(self, b: _Buffers, plan: _Plan) -> torch.Tensor:
         """Run every layer on the packed tokens of ``plan`` (``b.x`` / ``b.h`` hold their embeddings and first normed
         input); returns the final-norm output."""
-        w, eps = self.w, self.cfg.rms_norm_eps
-        n_layers = len(w.layers)
-        run = {AttentionLayer: self._attention, LatentLayer: self._latent, GLALayer: self._gla, MemoryLayer: self._memory}
+        w = self.w
+        run = {AttentionLayer: self._attention, BranchesLayer: self._branches, LatentLayer: self._latent, GLALayer: self._gla,
+               MemoryLayer: self._memory}
         for r, (freq, m) in w.rotary.items():
             K.rotary_table(plan.pos, freq, m, b.rope[r])
-        for li, L in enumerate(w.layers):
-            after = w.layers[li + 1].norm1 if li + 1 < n_layers else w.final_norm
+        for ri, r in enumerate(w.runs):
+            L, follow = w.layers[r.layer], w.runs[ri + 1] if ri + 1 < len(w.runs) else None
+            after = w.final_norm if follow is None else w.layers[follow.layer].norm1
+            b.before = None if self.layer_hook is None or follow is None or follow.add is None else torch.empty_like(b.x)
             proj = K.linear(b.h, L.mixer.w_in, out=b.proj[:, :L.mixer.w_in.shape[0]])
             if L.parallel:
-                self._parallel_layer(li, L, proj, after, b, plan)
+                self._parallel_layer(ri, L, proj, after, b, plan)
             else:
-                K.linear(run[type(L.mixer)](li, L.mixer, proj, b, plan), L.mixer.w_o, out=b.y)
-                norm = L.norm2 if L.norm2 is not None else after
-                if w.streams is None:
-                    K.residual_norm(b.y, b.x, L.out1, norm, w.W, eps, b.h)
+                K.linear(run[type(L.mixer)](ri, L.mixer, proj, b, plan), L.mixer.w_o, out=b.y)
+                if w.streams is not None:
+                    K.streams_norm(b.y, b.x, L.hc1, after if L.norm2 is None else L.norm2, w.W, self.cfg.norm_groups, self.cfg.rms_norm_eps,
+                                   b.h, y_bias=getattr(L.mixer, "o_bias", None))
+                elif L.norm2 is not None:
+                    self._seam(b.y, L.out1, L.norm2, None, b, plan)
                 else:
-                    K.streams_norm(b.y, b.x, L.hc1, norm, w.W, self.cfg.norm_groups, eps, b.h, y_bias=getattr(L.mixer, "o_bias", None))
+                    self._seam(b.y, L.out1, after, follow, b, plan)
                 if L.norm2 is not None:
-                    self._feed_forward(L, after, b)
+                    self._feed_forward(L, after, follow, b, plan)
             if self.layer_hook is not None:
-                self.layer_hook(li, (b.x if w.streams is None else b.x.sum(1))[:, :w.W])
+                x = b.x if b.before is None else b.before
+                self.layer_hook(ri, (x if w.streams is None else x.sum(1))[:, :w.W])
         return b.h
 
-    def _feed_forward(self, L: BlockWeights, w_next: torch.Tensor, b: _Buffers) -> None:
+    def _seam(self, y: torch.Tensor, w_out: torch.Tensor, w_next: torch.Tensor, follow: Optional[LayerRun], b: _Buffers, plan: _Plan) -> None:
+        """Between two sublayers with norms before and behind: output norm, residual sum, what the residual gets in front of the
+        run ``follow``, next norm."""
+        w, more = self.w, {}
+        if follow is not None and follow.add is not None:
+            more = dict(add=follow.add, before=b.before,
+                        embedding=(w.embed, plan.tok, self.cfg.embedding_scale) if follow.embedding else None)
+        K.residual_norm(y, b.x, w_out, w_next, w.W, self.cfg.rms_norm_eps, b.h, centered=self.cfg.centered, **more)
+
+    def _feed_forward(self, L: BlockWeights, w_next: torch.Tensor, follow: Optional[LayerRun], b: _Buffers, plan: _Plan) -> None:
         """The second sublayer: its output joins the residual, and ``b.h`` becomes the next layer's input."""
         w, eps = self.w, self.cfg.rms_norm_eps
         y, ex = b.y, {}
         if isinstance(L.ff, MixtureLayer):
             y, (ex["y_ex"], ex["slot"], ex["y_weight"]) = None, self._mixture(L.ff, None, b)
+        elif isinstance(L.ff, XIELULayer):
+            K.linear(K.xielu_linear(b.h, L.w_up, L.ff.up, L.ff.low, out=b.act[:, :L.w_down.shape[1]]), L.w_down, out=y)
         else:
             act = K.swiglu_linear(b.h, L.w_gu, out=b.act[:, :L.w_down.shape[1]])
             K.linear(act, L.w_down, out=y)
         if w.streams is None:
-            K.residual_norm(y, b.x, L.out2, w_next, w.W, eps, b.h)
+            self._seam(y, L.out2, w_next, follow, b, plan)
         else:
             K.streams_norm(y, b.x, L.hc2, w_next, w.W, self.cfg.norm_groups, eps, b.h, **ex)
 
     def _embed(self, b: _Buffers, plan: _Plan) -> None:
         """``b.x``: the residual stream of the tokens of ``plan``; ``b.h``: the first layer's normed input."""
-        w = self.w
-        K.embed_norm(w.embed, plan.tok, self.cfg.embedding_scale, w.layers[0].norm1, w.W, self.cfg.rms_norm_eps, b.x, b.h,
-                     groups=self.cfg.norm_groups, pos=plan.pos, freq=w.freq, streams=w.streams or 1, w_in=w.hc_in0)
+        w, first = self.w, self.w.runs[0]
+        K.embed_norm(w.embed, plan.tok, self.cfg.embedding_scale, w.layers[first.layer].norm1, w.W, self.cfg.rms_norm_eps, b.x, b.h,
+                     groups=self.cfg.norm_groups, pos=plan.pos, freq=w.freq, streams=w.streams or 1, w_in=w.hc_in0, add=first.add,
+                     centered=self.cfg.centered)
 
-    def _latent_plan(self, plan: _Plan, rows: List[int], counts: List[int], tiles: List[int], n: int) -> None:
-        """Which cache pages the portions' latent layers expand, in launches of at most ``LATENT_PAGES`` pages (a single longer
-        row is a launch of its own).  Call when the step's tokens have their pages."""
+    def _portion_plan(self, plan: _Plan, rows: List[int], counts: List[int], tiles: List[int], n: int) -> None:
+        """What the layers that do not read the paged cache directly need to know about a step's portions: the cache pages whose
+        latents are expanded, the pooled blocks that are seen.  Call when the step's tokens have their pages."""
+        lat = {m.spec.window for m in self.w.parts() if isinstance(m, LatentLayer) and m.w_exp is not None}
+        pools = {(m.spec.window, m.spec.pool) for m in self.w.parts() if isinstance(m, AttentionLayer) and m.spec.pool is not None}
+        if self.plain or not (lat or pools):
+            return
         dev, table = self.device, self.kv.page_table[0]
         rows_t = torch.tensor(rows, device=dev)
         lens = self.kv.len[0][rows_t].tolist()
         if any(l < c for l, c in zip(lens, counts)):         # nothing was appended: the pool or a row's table is full
             K.check_status(dev)
             raise RuntimeError("KV pool too small for the step")
-        pages = [(l + self.page_size - 1) // self.page_size for l in lens]
+        e = torch.repeat_interleave(torch.arange(len(rows), device=dev), torch.tensor(counts, device=dev), output_size=sum(counts))
+        plan.portion_of = torch.nn.functional.pad(e.to(torch.int32), (n - e.numel(), 0))
+        plan.latent = {w: self._latent_plan(plan, w, rows_t, lens, counts, tiles) for w in lat}
+        plan.pooled = {}
+        for window, block in pools:
+            S = LayerKV(block=block).pool_rows(self.page_size)
+            seen = [max(0, l - window) // block for l in lens]               # by the portion's last token
+            pages = torch.tensor([(k + 15) // 16 for k in seen], device=dev)
+            total = sum((k + 15) // 16 for k in seen)
+            first = torch.cumsum(pages, 0) - pages
+            which = torch.repeat_interleave(torch.arange(len(rows), device=dev), pages * 16, output_size=total * 16)
+            k = torch.arange(total * 16, device=dev) - first[which] * 16
+            live = k < torch.tensor(seen, device=dev)[which]
+            page = table[rows_t[which], torch.where(live, k // S, 0)]
+            src = torch.where(live, page * S + k % S, -1).to(torch.int32)
+            base = torch.repeat_interleave(first, torch.tensor(tiles, device=dev), output_size=sum(tiles)).to(torch.int32)
+            plan.pooled[window, block] = (src, base)
+            plan.pooled_rows = max(plan.pooled_rows, total * 16)
+
+    def _latent_plan(self, plan: _Plan, window: Optional[int], rows_t: torch.Tensor, lens: List[int], counts: List[int], tiles: List[int]):
+        """Which cache pages the portions' latent layers of a window expand, in launches of at most ``LATENT_PAGES`` pages (a single
+        longer row is a launch of its own), and where logical pages lie in them."""
+        dev, table, ps = self.device, self.kv.page_table[0], self.page_size
+        # first page that a portion's first token sees, in whole key blocks of the attention kernel
+        skip = [0 if window is None else max(0, l - c - window + 1) // 64 * 64 // ps for l, c in zip(lens, counts)]
+        pages = [(l + ps - 1) // ps - k for l, k in zip(lens, skip)]
         launches, base, at = [], [], 0                       # tiles a..b, pages a..b
         for k, t in zip(pages, tiles):
             first = launches[-1][1] if launches else 0
@@ -396,15 +509,14 @@ class HybridEngine(DecodeEngine):
             launches[-1][1] += t
             at += k
             launches[-1][3] = at
-        pages_t = torch.tensor(pages, device=dev)
-        which = torch.repeat_interleave(torch.arange(len(rows), device=dev), pages_t, output_size=at)
-        col = torch.arange(at, device=dev) - (torch.cumsum(pages_t, 0) - pages_t)[which]
+        pages_t, skip_t = torch.tensor(pages, device=dev), torch.tensor(skip, device=dev)
+        which = torch.repeat_interleave(torch.arange(len(pages), device=dev), pages_t, output_size=at)
+        col = torch.arange(at, device=dev) - (torch.cumsum(pages_t, 0) - pages_t - skip_t)[which]
         src = table[rows_t[which], col].contiguous()
-        plan.latent = [(a, b, src[c:d]) for a, b, c, d in launches]
-        plan.latent_pages = max(d - c for _, _, c, d in launches)
-        plan.latent_table = (torch.tensor(base, device=dev).view(-1, 1) + torch.arange(max(pages), device=dev)).to(torch.int32)
-        e = torch.repeat_interleave(torch.arange(len(rows), device=dev), torch.tensor(counts, device=dev), output_size=sum(counts))
-        plan.portion_of = torch.nn.functional.pad(e.to(torch.int32), (n - e.numel(), 0))
+        plan.latent_pages = max([plan.latent_pages] + [d - c for _, _, c, d in launches])
+        logical = torch.arange(max(k + f for k, f in zip(pages, skip)), device=dev)
+        where = (torch.tensor(base, device=dev) - skip_t).view(-1, 1) + logical
+        return [(a, b, src[c:d]) for a, b, c, d in launches], where.clamp(min=0).to(torch.int32)
 
     # ------------------------------------------------------------------------------------------
     # one step of portions and single tokens
@@ -456,9 +568,11 @@ class HybridEngine(DecodeEngine):
         plan.tile_q0, plan.tile_qn = d_q0, d_qn
         plan.groups = [(t, t + k, d_first[a:z], d_tiles[a:z]) for a, z, t, k in groups]
         K.kv_append(d_rows, d_counts, d_start, self.kv, 0, plan.pos, plan.row, plan.slot)
-        if n_dec < n and any(isinstance(L.mixer, LatentLayer) and L.mixer.w_exp is not None for L in self.w.layers):
-            self._latent_plan(plan, rows[n_dec:], counts[n_dec:], tiles, n)
-        b = _Buffers(self.w, n, self.dtype, dev, n_dec, 0 if self.plain else max([g[3] for g in groups] or [0]), plan.latent_pages)
+        plan.longest = max(counts)
+        if n_dec < n:
+            self._portion_plan(plan, rows[n_dec:], counts[n_dec:], tiles, n)
+        b = _Buffers(self.w, n, self.dtype, dev, n_dec, 0 if self.plain else max([g[3] for g in groups] or [0]), plan.latent_pages,
+                     plan.pooled_rows, len(counts) - n_dec, plan.longest)
         self._embed(b, plan)
         h = self._layers(b, plan)
         if not want:

@@ -9,8 +9,8 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from tah_b200.models.layered import (AttentionSpec, GLASpec, LatentAttentionSpec, LayeredForCausalLM, MixtureSpec, MLSTMSpec,
-                                     PolyNormSpec, RotarySpec, SwiGLUSpec)
+from tah_b200.models.layered import (AttentionSpec, BranchesSpec, GLASpec, LatentAttentionSpec, LayeredForCausalLM, MinGRUSpec,
+                                     MixtureSpec, MLSTMSpec, PolyNormSpec, RotarySpec, SwiGLUSpec, XIELUSpec)
 from tah_b200.ops import cuda as K
 
 LOG2E = 1.4426950408889634
@@ -45,8 +45,8 @@ class AttentionLayer:
     dk: int
     dv: int
     nkv: int                      # heads this layer writes (0: it reads another layer's cache)
-    w_in: torch.Tensor            # rows: queries, own keys, own values, gate numbers, input rows of a parallel feed-forward
-    w_o: torch.Tensor             # columns: heads, then those of a parallel feed-forward
+    w_in: Optional[torch.Tensor]  # rows: queries, own keys, own values, gates, input rows of a parallel feed-forward; None: a branch
+    w_o: Optional[torch.Tensor]   # columns: heads, then those of a parallel feed-forward; None: a branch
     kv_col: int                   # first key column of the projection
     b_in: Optional[torch.Tensor] = None
     gate_col: Optional[int] = None
@@ -57,11 +57,37 @@ class AttentionLayer:
     o_bias: Optional[torch.Tensor] = None
     v_keeps: bool = False                 # this layer's values are the ones later layers mix in
     v_lambda: Optional[torch.Tensor] = None   # [1] weight of those values in this layer's
+    wide_col: Optional[int] = None            # first column of the gate of every output element
+    slope: Optional[torch.Tensor] = None      # [heads], units as those of the bias
+    norm_w: Optional[torch.Tensor] = None     # [heads * dk] weights of the norms over all heads, those of the keys folded in
+    out_scale: float = 1.0
 
     @property
     def own_queries(self) -> bool:
         """Queries need a step of their own between projection and attention (bias, norm or rotation)."""
-        return self.b_in is not None or self.q_norm is not None or self.spec.rotary is not None or self.spec.v_mix
+        return self.b_in is not None or self.q_norm is not None or self.norm_w is not None or self.spec.rotary is not None or self.spec.v_mix
+
+
+@dataclass
+class MinGRULayer:
+    """Columns ``[z | x | g]`` of ``d`` each at ``in_col`` of the projection, output at ``out_col`` of the mixer's."""
+    spec: MinGRUSpec
+    d: int                        # width padded to 8
+    zb: torch.Tensor
+    xb: torch.Tensor
+    in_col: int
+    out_col: int
+    out_scale: float
+
+
+@dataclass
+class BranchesLayer:
+    """Two mixers from one projection whose outputs lie side by side, so that one product over both brings their sum back."""
+    spec: BranchesSpec
+    left: AttentionLayer
+    right: MinGRULayer
+    w_in: torch.Tensor
+    w_o: torch.Tensor
 
 
 @dataclass
@@ -77,7 +103,7 @@ class LatentLayer:
     w_in: torch.Tensor            # rows: query latent, c, rotated part, output gate
     c_col: int
     r_col: int
-    g_col: int
+    g_col: Optional[int]
     q_norm: torch.Tensor
     c_norm: torch.Tensor
     w_uq: torch.Tensor            # [heads * dk, Qp]
@@ -85,8 +111,8 @@ class LatentLayer:
     w_uv: torch.Tensor            # [heads, dv padded to 64, Rp]: weighted c -> value
     w_exp: Optional[torch.Tensor]             # [heads * dk + heads * dv, row of the cache]: cached rows -> keys and values
     w_o: torch.Tensor
-    sink: torch.Tensor            # natural units for the plain kernel, log2 units for the others
-    sink_log2: torch.Tensor
+    sink: Optional[torch.Tensor]  # natural units for the plain kernel, log2 units for the others
+    sink_log2: Optional[torch.Tensor]
     on_tensor_cores: bool         # single tokens run on the tensor-core kernel
 
 
@@ -127,6 +153,13 @@ class PolyNormLayer:
 
 
 @dataclass
+class XIELULayer:
+    """Numbers of the activation: ``up z^2 + z / 2`` above zero, ``low (exp(z) - 1 - z) + z / 2`` below."""
+    up: float
+    low: float
+
+
+@dataclass
 class SharedExpertLayer:
     """An expert of every token, laid out like :class:`PolyNormLayer` with interleaved gate / up rows."""
     cols: int
@@ -155,9 +188,23 @@ class BlockWeights:
     norm2: Optional[torch.Tensor] = None
     out2: Optional[torch.Tensor] = None
     w_gu: Optional[torch.Tensor] = None
+    w_up: Optional[torch.Tensor] = None
     w_down: Optional[torch.Tensor] = None
     hc1: Optional[torch.Tensor] = None    # hyper-connections behind the mixer: mix, out, in of the next reader
     hc2: Optional[torch.Tensor] = None    # the same behind the feed-forward
+
+
+@dataclass
+class LayerRun:
+    """One run of a layer.  What the residual gets in front of it: ``add`` (a vector), ``embedding`` (the embedding output)."""
+    layer: int
+    add: Optional[torch.Tensor] = None
+    embedding: bool = False
+
+
+def mixer_parts(m) -> list:
+    """A mixer, or the branches it has."""
+    return [m.left, m.right] if isinstance(m, BranchesLayer) else [m]
 
 
 class HybridWeights:
@@ -211,9 +258,55 @@ class HybridWeights:
         def gate_up(p, n):                                   # interleaved gate / up rows of a unit, padded to 2 n
             return K.interleave_gate_up(torch.cat([mat(T(p + "gate"), n, self.Wp), mat(T(p + "up"), n, self.Wp)]))
 
+        def attention(x, m):
+            """``(layer without its matrices, row blocks of the projection, their biases)`` of the tensors ``x + ...``."""
+            dk, dv, H, G, own = _pad(m.dim, 8), _pad(m.vdim, 8), m.heads, m.kv_heads, m.kv_from is None
+            if max(dk, dv) > 256:
+                raise NotImplementedError("attention head sizes above 256")
+            if m.keys_as_values and (not own or m.proj_bias or m.qk_norm or m.rotary is not None or m.v_mix or m.softcap is not None):
+                raise NotImplementedError("values that are the keys as projected beside shared keys, biases, head norms, rotation, mixed "
+                                          "values or a score cap")
+            if m.norm_all and (not m.keys_as_values or m.pool is not None) or m.pool is not None and (
+                    not m.keys_as_values or m.keep_first or m.slopes or m.bias_max is not None):
+                raise NotImplementedError("norms over all heads or pooled blocks in this combination")
+            rows = [heads_rows(T(x + "q"), H, m.dim, dk)]
+            bias = [heads_vec(T(x + "q.b"), H, m.dim, dk)] if m.proj_bias else []
+            if own:
+                rows.append(heads_rows(T(x + "k"), G, m.dim, dk))
+                if not m.keys_as_values:
+                    rows.append(heads_rows(T(x + "v"), G, m.vdim, dv))
+                if m.proj_bias:
+                    bias += [heads_vec(T(x + "k.b"), G, m.dim, dk), heads_vec(T(x + "v.b"), G, m.vdim, dv)]
+            mixer = AttentionLayer(m, dk, dv, G if own else 0, None, None, kv_col=H * dk)
+            if m.head_gate:
+                mixer.gate_col = sum(r.shape[0] for r in rows)
+                rows.append(heads_rows(T(x + "g"), H, 1, 1))
+            if m.wide_gate:
+                mixer.wide_col = sum(r.shape[0] for r in rows)
+                rows.append(heads_rows(T(x + "g"), H, m.vdim, dv))
+            if m.qk_norm:
+                mixer.q_norm, mixer.k_norm = vec(T(x + "q.norm"), dk), vec(T(x + "k.norm"), dk) if own else None
+            if m.norm_all:                                   # score = factor_j * (q * w_q * w_k) . k_j: both weights go to the queries
+                wq, wk = heads_vec(T(x + "q.norm"), H, m.dim, dk), heads_vec(T(x + "k.norm"), G, m.dim, dk)
+                mixer.norm_w = (wq.view(G, H // G, dk) * wk.view(G, 1, dk)).reshape(-1).contiguous()
+            if m.bias_max is not None:
+                mixer.bias = distance_table(T(x + "rel"), m.bias_max) * unit
+            if m.slopes:
+                mixer.slope = (torch.tensor([2.0 ** (-8.0 * (h + 1) / H) for h in range(H)], dtype=torch.float64) * unit).float().to(dev)
+            if m.sink:
+                mixer.sink = vec(T(x + "sink"), H) * unit
+            if m.out_bias:
+                mixer.o_bias = vec(T(x + "o.b"), self.Wp)
+            if m.v_mix:
+                mixer.v_keeps = not any(isinstance(b.mixer, AttentionLayer) and b.mixer.spec.v_mix for b in self.layers)
+                if not mixer.v_keeps:
+                    mixer.v_lambda = T(x + "vmix").float().reshape(1)
+            return mixer, rows, bias
+
         self.embed = mat(T("embed"), self.vocab, self.Wp)
         self.head = mat(T("embed" if cfg.tied_head else "head"), self.vocab_shard[2], self.Wp)
         norm = lambda name: cfg.norm_offset + T(name).float()
+        out_norm = lambda p, q: vec(T(f"{p}norm{q}b").float() * (T(f"{p}ls{q}").float() if cfg.layer_scale else 1.0), self.Wp)
         self.final_norm = vec(norm("final.norm") * cfg.logit_scale, self.Wp)
         self.rotary: Dict[RotarySpec, Tuple[torch.Tensor, float]] = {}       # frequencies (high, low parts), sine / cosine factor
         for r in {r for r in (getattr(l.mixer, "rotary", None) for l in cfg.layers) if r is not None}:
@@ -225,46 +318,35 @@ class HybridWeights:
         for i, l in enumerate(cfg.layers):
             p, m, f = f"l{i}.", l.mixer, l.ff
             x = p + "mix."
-            kd = m.dim + m.rot_dim if isinstance(m, LatentAttentionSpec) else m.dim
-            dk, dv = _pad(kd, 8), _pad(m.vdim, 8)
-            w_o = heads_cols(T(x + "o"), m.heads, m.vdim, dv)
             ff, ff_rows, ff_cols = None, [], []
+            if not isinstance(m, BranchesSpec):
+                kd = m.dim + m.rot_dim if isinstance(m, LatentAttentionSpec) else m.dim
+                dk, dv = _pad(kd, 8), _pad(m.vdim, 8)
+                w_o = heads_cols(T(x + "o"), m.heads, m.vdim, dv)
             if isinstance(m, AttentionSpec):
-                if max(dk, dv) > 256:
-                    raise NotImplementedError("attention head sizes above 256")
-                H, G, own = m.heads, m.kv_heads, m.kv_from is None
-                rows = [heads_rows(T(x + "q"), H, m.dim, dk)]
-                bias = [heads_vec(T(x + "q.b"), H, m.dim, dk)] if m.proj_bias else []
-                if own:
-                    rows += [heads_rows(T(x + "k"), G, m.dim, dk), heads_rows(T(x + "v"), G, m.vdim, dv)]
-                    if m.proj_bias:
-                        bias += [heads_vec(T(x + "k.b"), G, m.dim, dk), heads_vec(T(x + "v.b"), G, m.vdim, dv)]
-                gate_col = None
-                if m.head_gate:
-                    gate_col = sum(r.shape[0] for r in rows)
-                    rows.append(heads_rows(T(x + "g"), H, 1, 1))
+                mixer, rows, bias = attention(x, m)
                 if l.parallel:
                     ff, ff_rows, ff_cols = self._parallel(p + "mlp.", f, _pad(sum(r.shape[0] for r in rows), 8), w_o.shape[1],
                                                           T, mat, cols_of, gate_up)
                     fill = -sum(r.shape[0] for r in rows) % 8
                     if fill:
                         rows.append(torch.zeros(fill, self.Wp, dtype=dtype, device=dev))
-                w_in = stack(rows + ff_rows)
-                mixer = AttentionLayer(m, dk, dv, G if own else 0, w_in, torch.cat([w_o] + ff_cols, 1) if ff_cols else w_o,
-                                       kv_col=H * dk, b_in=vec(torch.cat(bias), w_in.shape[0]) if bias else None,
-                                       gate_col=gate_col)
-                if m.qk_norm:
-                    mixer.q_norm, mixer.k_norm = vec(T(x + "q.norm"), dk), vec(T(x + "k.norm"), dk) if own else None
-                if m.bias_max is not None:
-                    mixer.bias = distance_table(T(x + "rel"), m.bias_max) * unit
-                if m.sink:
-                    mixer.sink = vec(T(x + "sink"), H) * unit
-                if m.out_bias:
-                    mixer.o_bias = vec(T(x + "o.b"), self.Wp)
-                if m.v_mix:
-                    mixer.v_keeps = not any(isinstance(b.mixer, AttentionLayer) and b.mixer.spec.v_mix for b in self.layers)
-                    if not mixer.v_keeps:
-                        mixer.v_lambda = T(x + "vmix").float().reshape(1)
+                mixer.w_in, mixer.w_o = stack(rows + ff_rows), torch.cat([w_o] + ff_cols, 1) if ff_cols else w_o
+                if bias:
+                    mixer.b_in = vec(torch.cat(bias), mixer.w_in.shape[0])
+            elif isinstance(m, BranchesSpec):
+                left, rows, _ = attention(x + "left.", m.left)
+                left.out_scale = m.left_scale
+                D, D8 = m.right.width, _pad(m.right.width, 8)
+                r, in_col, heads = x + "right.", _pad(sum(t.shape[0] for t in rows), 8), m.left.heads * left.dv
+                if in_col != sum(t.shape[0] for t in rows):
+                    rows.append(torch.zeros(in_col - sum(t.shape[0] for t in rows), self.Wp, dtype=dtype, device=dev))
+                rows += [mat(T(r + n), D8, self.Wp) for n in ("z", "x", "g")]
+                w_o = torch.zeros(self.Wp, _pad(heads + D8, 64), dtype=dtype, device=dev)
+                w_o[:, :heads] = heads_cols(T(x + "left.o"), m.left.heads, m.left.vdim, left.dv)[:, :heads]
+                w_o[:self.W, heads:heads + D] = T(r + "o")
+                right = MinGRULayer(m.right, D8, vec(T(r + "z.b"), D8), vec(T(r + "x.b"), D8), in_col, heads, m.right_scale)
+                mixer = BranchesLayer(m, left, right, stack(rows), w_o)
             elif isinstance(m, LatentAttentionSpec):
                 mixer = self._latent(x, m, dk, dv, w_o, dtype, plain, T, mat, stack, heads_rows)
             elif isinstance(m, GLASpec):
@@ -294,16 +376,21 @@ class HybridWeights:
                 if cfg.streams is None:
                     if cfg.norm_groups != 1:
                         raise NotImplementedError("grouped norms in a layer with output norms")
-                    b.out1 = vec(T(p + "norm1b").float() * T(p + "ls1").float(), self.Wp)
+                    b.out1 = out_norm(p, 1)
                 if f is not None:
                     b.norm2 = vec(norm(p + "norm2"), self.Wp)
                     if cfg.streams is None:
-                        b.out2 = vec(T(p + "norm2b").float() * T(p + "ls2").float(), self.Wp)
+                        b.out2 = out_norm(p, 2)
                 if isinstance(f, SwiGLUSpec):
                     Ip = _pad(f.ff, 64)
                     gu = torch.cat([mat(T(p + "mlp.gate"), Ip, self.Wp), mat(T(p + "mlp.up"), Ip, self.Wp)])
                     b.w_gu = K.interleave_gate_up(gu) if dtype == torch.bfloat16 else gu
                     b.w_down = mat(T(p + "mlp.down"), self.Wp, Ip)
+                elif isinstance(f, XIELUSpec) and cfg.streams is None:
+                    Ip, act = _pad(f.ff, 64), T(p + "mlp.act").double()
+                    soft = torch.logaddexp(act, torch.zeros_like(act)).tolist()
+                    b.ff = XIELULayer(soft[0], 0.5 + soft[1])
+                    b.w_up, b.w_down = mat(T(p + "mlp.up"), Ip, self.Wp), mat(T(p + "mlp.down"), self.Wp, Ip)
                 elif isinstance(f, MixtureSpec) and f.shared is None and cfg.streams is not None:
                     b.ff = self._mixture(p + "mlp.", f, T(p + "mlp.router"), None, T, mat, cols_of, gate_up)
                 elif f is not None:
@@ -313,6 +400,16 @@ class HybridWeights:
         self.streams, self.hc_in0 = cfg.streams, None
         if cfg.streams is not None:
             self._streams(cfg, T)
+        if cfg.loop is not None and (cfg.streams is not None or any(l.parallel or getattr(l.mixer, "kv_from", None) is not None or
+                                                                    getattr(l.mixer, "v_mix", False) for l in cfg.layers)):
+            raise NotImplementedError("a loop over layers with residual streams, parallel feed-forwards or another layer's keys or values")
+        if cfg.centered and (cfg.streams is not None or cfg.norm_groups != 1 or any(l.parallel for l in cfg.layers)):
+            raise NotImplementedError("layer norms with residual streams, grouped norms or parallel feed-forwards")
+        self.runs = [LayerRun(i) if t is None else LayerRun(i, vec(T("loop.step")[t], self.Wp), t > 0) for i, t in cfg.layer_runs()]
+
+    def parts(self) -> list:
+        """The mixers of all layers, branches one by one."""
+        return [p for b in self.layers for p in mixer_parts(b.mixer)]
 
     def _streams(self, cfg, T) -> None:
         """Hyper-connection weights of every seam: how the sublayer in front writes, how the next one (at the end: the plain
@@ -330,8 +427,8 @@ class HybridWeights:
         dev = self.embed.device
         Qp, Rp, rw = _pad(m.q_rank, 64), _pad(R, 64), _pad(r, 64)
         lp, dkv, unit = Rp + rw, T(x + "dkv"), torch.arange(r, device=dev)
-        w_in = stack([mat(T(x + "dq"), Qp, self.Wp), mat(dkv[:R], Rp, self.Wp), mat(dkv[R:], rw, self.Wp),
-                      heads_rows(T(x + "g"), H, m.vdim, dv)])
+        w_in = stack([mat(T(x + "dq"), Qp, self.Wp), mat(dkv[:R], Rp, self.Wp), mat(dkv[R:], rw, self.Wp)] +
+                     ([heads_rows(T(x + "g"), H, m.vdim, dv)] if m.gate else []))
         w_uq = torch.zeros(H, dk, Qp, dtype=dtype, device=dev)
         w_uq[:, :d + r, :m.q_rank] = T(x + "uq").view(H, d + r, m.q_rank)
         w_uq = mat(w_uq.view(H * dk, Qp), _pad(H * dk, 64), Qp)
@@ -349,9 +446,10 @@ class HybridWeights:
             k[:, d + unit, Rp + unit] = 1.0
             w_exp[H * dk:H * (dk + dv)].view(H, dv, lp)[:, :m.vdim, :R] = uv
         vec = lambda t, n: torch.nn.functional.pad(t.float(), (0, n - t.numel())).contiguous()
-        sink = T(x + "sink").float().contiguous()
-        return LatentLayer(m, dk, dv, Qp, Rp, rw, w_in, Qp, Qp + Rp, Qp + Rp + rw, vec(T(x + "dq.norm"), Qp), vec(T(x + "dkv.norm"), Rp),
-                           w_uq, w_abs, w_uv, w_exp, w_o, sink, sink * LOG2E, not plain and K.latent_decode_fits(H, Rp, rw))
+        sink = T(x + "sink").float().contiguous() if m.sink else None
+        return LatentLayer(m, dk, dv, Qp, Rp, rw, w_in, Qp, Qp + Rp, Qp + Rp + rw if m.gate else None, vec(T(x + "dq.norm"), Qp),
+                           vec(T(x + "dkv.norm"), Rp), w_uq, w_abs, w_uv, w_exp, w_o, sink, None if sink is None else sink * LOG2E,
+                           not plain and K.latent_decode_fits(H, Rp, rw))
 
     @staticmethod
     def _mixture(p, f, router, shared, T, mat, cols_of, gate_up) -> MixtureLayer:

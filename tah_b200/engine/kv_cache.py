@@ -13,7 +13,10 @@ popped by the tick kernel), so decode never returns to the host for memory.
 A model whose layers differ gives ``CacheGeometry.layers``: one :class:`LayerKV` per layer with its own K and V sizes, or
 ``None`` for a layer without keys (a recurrent layer), or ``LayerKV(shared_with=j)`` for a layer that reads the cache of
 layer ``j``.  All layers share one page table; the pool of a layer is then a tensor of its own with the same page layout
-``[K: kv_heads, page_size, k_dim][V: kv_heads, page_size, v_dim]``.  What recurrent layers carry from token to token
+``[K: kv_heads, page_size, k_dim][V: kv_heads, page_size, v_dim]``.  Beside it a layer may have further pools under the same page
+table: ``factors``, one fp32 number per token, and ``pooled``, the means of blocks of ``block`` keys.  A page holds
+``pool_rows`` of those (a power of two, at least ``page_size / block``), so block ``b`` is row ``b % pool_rows`` of the row's
+logical page ``b // pool_rows``, which the row owns by the time the block is complete.  What recurrent layers carry from token to token
 lives beside the pages in :class:`RecurrentState`, one slot per cache row.
 """
 from __future__ import annotations
@@ -32,6 +35,15 @@ class LayerKV:
     k_dim: int = 0
     v_dim: int = 0
     shared_with: Optional[int] = None     # the layer whose pool this layer reads
+    factor: bool = False                  # one fp32 number per token beside the keys
+    block: Optional[int] = None           # keys of a pooled block; None: no pooled blocks
+
+    def pool_rows(self, page_size: int) -> int:
+        """Pooled blocks that a page has room for."""
+        n = 1
+        while self.block is not None and n * self.block < page_size:
+            n *= 2
+        return 0 if self.block is None else n
 
 
 @dataclass
@@ -66,6 +78,8 @@ class PagedKVCache:
         self.max_pages = [ppr] * n_depths
         self.n_pages: List[int] = []
         self.pool: List = []              # per depth: one tensor, or with geo.layers a list with one tensor (or None) per layer
+        self.factors: List[List[Optional[torch.Tensor]]] = []     # per depth and layer (see the module docstring)
+        self.pooled: List[List[Optional[torch.Tensor]]] = []
         self.page_table: List[torch.Tensor] = []
         self.len: List[torch.Tensor] = []
         self.free_stack: List[torch.Tensor] = []
@@ -86,6 +100,11 @@ class PagedKVCache:
                         torch.zeros(pages + self.guard_pages, l.kv_heads * geo.page_size * (l.k_dim + l.v_dim), dtype=dtype,
                                     device=device) for l in geo.layers]
             self.pool.append(pool)
+            self.factors.append([None if l is None or not l.factor else
+                                 torch.zeros(pages + self.guard_pages, geo.page_size, device=device) for l in geo.layers or []])
+            self.pooled.append([None if l is None or l.block is None else
+                                torch.zeros(pages + self.guard_pages, l.kv_heads * l.pool_rows(geo.page_size) * l.k_dim, dtype=dtype,
+                                            device=device) for l in geo.layers or []])
             if self.guard_pages:
                 for t in self._pools(d):
                     t[..., pages:, :].view(torch.int16).fill_(GUARD_PATTERN)
@@ -104,7 +123,9 @@ class PagedKVCache:
     def _pools(self, depth: int) -> List[torch.Tensor]:
         """The pool tensors of a depth as ``[..., pages, elements of a page]`` views."""
         p = self.pool[depth]
-        return [p.flatten(2)] if self.geo.layers is None else [t for t in p if t is not None]
+        if self.geo.layers is None:
+            return [p.flatten(2)]
+        return [t for t in p + self.factors[depth] + self.pooled[depth] if t is not None]
 
     def bytes(self) -> int:
         return sum(t.numel() * t.element_size() for d in range(self.n_depths) for t in self._pools(d))

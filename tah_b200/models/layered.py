@@ -2,8 +2,9 @@
 made of, the configuration the engine reads, and a model class that holds the weights under their on-disk names.
 
 The computation is the engine's (:mod:`tah_b200.engine.hybrid`).  A family (:mod:`tah_b200.models.gunuvik`,
-:mod:`tah_b200.models.ditilix`, :mod:`tah_b200.models.niralix`) reads its own ``config.json`` into these specs and says which tensors it has; every constant
-of a mechanism is a field here, and a mechanism that a family does not have is absent (``None`` / ``False``).
+:mod:`tah_b200.models.ditilix`, :mod:`tah_b200.models.niralix`, :mod:`tah_b200.models.pidenex`) reads its own ``config.json`` into
+these specs and says which tensors it has; every constant of a mechanism is a field here, and a mechanism that a family does
+not have is absent (``None`` / ``False``).
 """
 from __future__ import annotations
 
@@ -56,7 +57,7 @@ class RotarySpec:
 
 @dataclass
 class AttentionSpec:
-    """Causal attention over the paged cache: ``score = cap(temp(i) * (q . k) * scale) + bias[distance]``."""
+    """Causal attention over the paged cache: ``score = cap(temp(i) * (q . k) * scale) + bias[distance] - slope_h * distance``."""
     heads: int
     kv_heads: int
     dim: int                              # per-head size of queries and keys
@@ -76,6 +77,11 @@ class AttentionSpec:
     rotary: Optional[RotarySpec] = None
     out_bias: bool = False                # bias of the output projection
     v_mix: bool = False                   # values mixed with those of the first layer that has this flag
+    keys_as_values: bool = False          # the values are the keys as projected (in front of any norm)
+    pool: Optional[int] = None            # means of the blocks of that many keys wholly in front of the window are keys as well
+    slopes: bool = False                  # distance bias: slope_h = 2 ** (-8 (h + 1) / heads) per token
+    norm_all: bool = False                # RMS norm of q and of k over all heads at once
+    wide_gate: bool = False               # the heads' outputs times sigmoid(W_g h), element by element
 
     kind = "attention"
 
@@ -93,8 +99,7 @@ class MLSTMSpec:
 @dataclass
 class LatentAttentionSpec:
     """Causal attention whose keys and values are linear in one cached latent of ``kv_rank`` and one rotated key part of
-    ``rot_dim`` per token; queries come from a latent of ``q_rank``.  Softmax with a learned sink per head, output times
-    ``sigmoid(W_g h)``."""
+    ``rot_dim`` per token; queries come from a latent of ``q_rank``."""
     heads: int
     dim: int                              # unrotated part of queries and keys
     rot_dim: int                          # rotated part, keys share one
@@ -103,6 +108,9 @@ class LatentAttentionSpec:
     kv_rank: int
     scale: float
     rotary: RotarySpec
+    window: Optional[int] = None          # None: every earlier token
+    sink: bool = True                     # learned softmax sink per head
+    gate: bool = True                     # output times sigmoid(W_g h), element by element
 
     kind = "latent_attention"
 
@@ -119,6 +127,25 @@ class GLASpec:
     kind = "gla"
 
 
+@dataclass
+class MinGRUSpec:
+    """Elementwise gated recurrence whose gates read the current token only: ``S <- (1 - z) S + z * candidate``."""
+    width: int
+
+    kind = "min_gru"
+
+
+@dataclass
+class BranchesSpec:
+    """Attention and an elementwise recurrence from one input, ``left_scale * left + right_scale * right``."""
+    left: AttentionSpec
+    right: MinGRUSpec
+    left_scale: float
+    right_scale: float
+
+    kind = "parallel"
+
+
 def check_rotary(i: int, r: Optional[RotarySpec], size: int) -> None:
     if r is not None and (r.dims < 2 or r.dims % 2 or r.dims > size or not r.base > 1.0):
         raise ValueError(f"layer {i}: rotation of {r.dims} of {size} dims with base {r.base}")
@@ -133,6 +160,12 @@ def check_attention(i: int, m: AttentionSpec, layers: List["LayerSpec"]) -> None
     if m.q_temp is not None and not m.q_temp[1] > 0:
         raise ValueError(f"layer {i}: query temperature steps of {m.q_temp[1]} positions")
     check_rotary(i, m.rotary, m.dim)
+    if m.window is not None and m.window < 1:
+        raise ValueError(f"layer {i}: a window of {m.window} tokens")
+    if m.keys_as_values and m.dim != m.vdim:
+        raise ValueError(f"layer {i}: keys of {m.dim} cannot be values of {m.vdim}")
+    if m.pool is not None and (m.pool < 1 or m.window is None):
+        raise ValueError(f"layer {i}: blocks of {m.pool} tokens in front of a window of {m.window}")
     if m.v_mix:
         first = next((l.mixer for l in layers if isinstance(l.mixer, AttentionSpec) and l.mixer.v_mix), m)
         if m.kv_from is not None or (first.kv_heads, first.vdim) != (m.kv_heads, m.vdim):
@@ -160,6 +193,15 @@ class PolyNormSpec:
     ff: int
 
     kind = "poly_norm"
+
+
+@dataclass
+class XIELUSpec:
+    """``down(act(up(h)))``: ``softplus(p) z^2 + z / 2`` above zero, ``(1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2`` below, with
+    two learned numbers."""
+    ff: int
+
+    kind = "xielu"
 
 
 @dataclass
@@ -196,6 +238,15 @@ class LayerSpec:
 # ------------------------------------------------------------------------------------
 # configuration
 # ------------------------------------------------------------------------------------
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers ``start .. stop - 1`` run ``times`` times in a row with the same weights, each pass with caches and states of its
+    own.  A pass begins by adding a learned vector of its own to the residual, and from the second on the embedding output."""
+    start: int
+    stop: int
+    times: int
+
+
 @dataclass
 class LayeredConfig:
     vocab_size: int
@@ -211,11 +262,23 @@ class LayeredConfig:
     norm_offset: float = 0.0              # stored norm weights of the residual stream are this much below their value
     streams: Optional[int] = None         # hyper-connections over that many residual streams; None: a plain residual sum
     tied_head: bool = False               # the embedding table is the output projection
+    centered: bool = False                # layer norms (mean taken off) instead of RMS norms around the sublayers
+    layer_scale: bool = True              # norms behind the sublayers are followed by a learned factor per channel
+    loop: Optional[LoopSpec] = None
     raw: Dict = field(default_factory=dict)
 
     @property
     def num_hidden_layers(self) -> int:
         return len(self.layers)
+
+    def layer_runs(self) -> List[Tuple[int, Optional[int]]]:
+        """The layers in the order they run, as ``(layer, pass)``; the pass is given for the layer that begins one."""
+        n, l = len(self.layers), self.loop
+        if l is None:
+            return [(i, None) for i in range(n)]
+        return [(i, None) for i in range(l.start)] + \
+            [(i, t if i == l.start else None) for t in range(l.times) for i in range(l.start, l.stop)] + \
+            [(i, None) for i in range(l.stop, n)]
 
     @property
     def dtype(self) -> torch.dtype:

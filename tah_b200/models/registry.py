@@ -100,6 +100,11 @@ def _niralix_load(path, dtype, device):
     return NiralixForCausalLM.from_pretrained(path, dtype=dtype, device=device)
 
 
+def _pidenex_load(path, dtype, device):
+    from tah_b200.models.pidenex import PidenexForCausalLM
+    return PidenexForCausalLM.from_pretrained(path, dtype=dtype, device=device)
+
+
 def _is(class_name: str) -> Callable[[object], bool]:
     return lambda model: type(model).__name__ == class_name
 
@@ -116,3 +121,5 @@ register_family(Family("ditilix", lambda c: c.get("architecture") == "Ditilix", 
                        _hybrid_engine, "ditilix"))
 register_family(Family("niralix", lambda c: c.get("architecture") == "Niralix", _niralix_load, _is("NiralixForCausalLM"),
                        _hybrid_engine, "niralix"))
+register_family(Family("pidenex", lambda c: c.get("architecture") == "Pidenex", _pidenex_load, _is("PidenexForCausalLM"),
+                       _hybrid_engine, "pidenex"))

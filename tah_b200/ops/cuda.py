@@ -593,18 +593,43 @@ def swiglu_linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] 
     return out
 
 
+def xielu_linear(x: torch.Tensor, w: torch.Tensor, up: float, low: float, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """xIELU of ``x @ w^T``: ``up z^2 + z / 2`` for ``z > 0`` and ``low (exp(z) - 1 - z) + z / 2`` otherwise; in the epilogue of
+    the product for bf16 (on ``z`` rounded to bf16), a kernel behind it for fp32."""
+    M, Kd = x.shape
+    F = w.shape[0]
+    if w.shape[1] != Kd:
+        raise ValueError(f"xielu_linear: x {tuple(x.shape)} w {tuple(w.shape)}")
+    if _act_f32(x, w):
+        out = linear(x, w, out=out)
+        _rc(lib().tahb_xielu_f32(_p(out), c_float(up), c_float(low), c_int(M), c_int(F), c_ll(out.stride(0)), _stream()), "tahb_xielu_f32")
+        return out
+    if out is None:
+        out = torch.empty(M, F, dtype=torch.bfloat16, device=x.device)
+    for n, t in (("x", x), ("w", w), ("out", out)):
+        _check_bf16_2d(t, n)
+    pair = PAIR_AUTO and M >= PAIR_MIN_TOKENS and F % 256 == 0
+    bn, splits = (256, 1) if pair else plan_gemm(M, F, Kd)
+    _rc(lib().tahb_gemm_xielu(_p(w), _p(x), _p(out), c_int(M), c_int(F), c_int(Kd), c_ll(w.stride(0)), c_ll(x.stride(0)), c_ll(out.stride(0)),
+                              c_float(up), c_float(low), c_int(int(pair)), c_int(splits), c_int(bn), _p(status_word(x.device)), _stream()),
+        "tahb_gemm_xielu")
+    return out
+
+
 def embed_norm(E, tok, scale: float, w, width: int, eps: float, x, h, groups: int = 1, pos=None, freq=None, streams: int = 1,
-               w_in=None):
+               w_in=None, add=None, centered: bool = False):
     """``x = scale * E[tok]`` (fp32 residual stream) and ``h = rms(x) * w`` in the activation type of ``E``.  Rows are
     padded to ``E.shape[1]`` columns, ``width`` of them real.  ``groups``: parts of the row with a root mean square of
     their own; ``pos`` / ``freq``: token positions and :func:`sinusoid_frequencies`, adds sinusoidal positions to ``x``;
-    ``streams`` / ``w_in``: that many copies in ``x [M, streams, ld]``, and the fp32 weights of their sum (what ``h`` sees)."""
+    ``streams`` / ``w_in``: that many copies in ``x [M, streams, ld]``, and the fp32 weights of their sum (what ``h`` sees);
+    ``add``: fp32 vector added to ``x``; ``centered``: a layer norm in the place of the RMS norm."""
     f32 = _act_f32(E, h)
     if x.numel() != tok.shape[0] * streams * E.shape[1]:
         raise ValueError(f"embed_norm: residual {tuple(x.shape)} for {streams} streams of {E.shape[1]} columns")
     _rc(lib().tahb_embed_norm(_p(E), _p(tok), c_float(scale), _p(pos if freq is not None else None), _p(freq), c_int(streams),
-                              _p(w_in), _p(x), _p(w), _p(h), c_int(tok.shape[0]), c_int(E.shape[0]), c_int(width),
-                              c_int(groups), c_int(E.shape[1]), c_float(eps), c_int(f32), _stream()), "tahb_embed_norm")
+                              _p(w_in), _p(add), _p(x), _p(w), _p(h), c_int(tok.shape[0]), c_int(E.shape[0]), c_int(width),
+                              c_int(groups), c_int(E.shape[1]), c_float(eps), c_int(int(centered)), c_int(f32), _stream()),
+        "tahb_embed_norm")
 
 
 def sinusoid_frequencies(width: int, base: float = 10000.0, device=None) -> torch.Tensor:
@@ -656,12 +681,27 @@ def residual_add_norm(y, x, mult: float, w_next, width: int, groups: int, eps: f
                                      c_int(x.shape[1]), c_float(eps), c_int(f32), _stream()), "tahb_residual_add_norm")
 
 
-def residual_norm(y, x, w_out, w_next, width: int, eps: float, h):
-    """``x += rms(y) * w_out`` (fp32, in place) and ``h = rms(x) * w_next``: output norm, layer scale, residual sum and
-    the next sublayer's input norm in one launch.  ``w_out`` / ``w_next``: fp32 rows padded with zeros."""
-    f32 = _act_f32(y, h)
-    _rc(lib().tahb_residual_norm(_p(y), c_ll(y.stride(0)), _p(x), _p(w_out), _p(w_next), _p(h), c_int(y.shape[0]),
-                                 c_int(width), c_int(x.shape[1]), c_float(eps), c_int(f32), _stream()), "tahb_residual_norm")
+class _ResidualNorm(ctypes.Structure):
+    _fields_ = [("y", c_void_p), ("ldy", c_ll), ("x", c_void_p), ("w_out", c_void_p), ("w_next", c_void_p), ("h", c_void_p), ("width", c_int),
+                ("ld", c_int), ("eps", c_float), ("add", c_void_p), ("E", c_void_p), ("tok", c_void_p), ("vocab", c_int), ("scale", c_float),
+                ("before", c_void_p)]
+
+
+def residual_norm(y, x, w_out, w_next, width: int, eps: float, h, centered: bool = False, add=None, embedding=None, before=None):
+    """``x += norm(y) * w_out`` (fp32, in place) and ``h = norm(x) * w_next``: output norm, layer scale, residual sum and
+    the next sublayer's input norm in one launch.  ``w_out`` / ``w_next``: fp32 rows padded with zeros.  The norms are RMS norms,
+    or layer norms when ``centered``.  ``add`` (fp32 vector) and ``embedding = (E, tok, scale)``: what the residual gets in
+    addition behind the sublayer's sum; ``before`` receives it without."""
+    a = _ResidualNorm()
+    ptr = lambda t: 0 if t is None else t.data_ptr()
+    E, tok, scale = (None, None, 0.0) if embedding is None else embedding
+    f32 = _act_f32(y, h) if E is None else _act_f32(y, h, E)
+    if E is not None and E.shape[1] != x.shape[1] or before is not None and before.shape != x.shape:
+        raise ValueError(f"residual_norm: rows of {x.shape[1]} columns")
+    a.y, a.ldy, a.x, a.w_out, a.w_next, a.h = ptr(y), y.stride(0), ptr(x), ptr(w_out), ptr(w_next), ptr(h)
+    a.width, a.ld, a.eps, a.add, a.E, a.tok, a.before = width, x.shape[1], eps, ptr(add), ptr(E), ptr(tok), ptr(before)
+    a.vocab, a.scale = 0 if E is None else E.shape[0], scale
+    _rc(lib().tahb_residual_norm(ctypes.byref(a), c_int(y.shape[0]), c_int(int(centered)), c_int(f32), _stream()), "tahb_residual_norm")
 
 
 def few_linear(x, w, b, out=None):
@@ -717,19 +757,26 @@ class _WindowAttn(ctypes.Structure):
                [(n, c_int) for n in ("n", "nq", "nkv", "dk", "dv", "page_size", "max_pages", "window", "keep_first", "far")] + \
                [("ld_q", c_ll), ("ld_out", c_ll), ("ld_gate", c_ll), ("scale", c_float), ("softcap", c_float),
                 ("temp_coef", c_float), ("temp_every", ctypes.c_double), ("ws", c_void_p), ("n_split", c_int),
-                ("status", c_void_p)]
+                ("status", c_void_p), ("slope", c_void_p), ("factor", c_void_p), ("pooled", c_void_p), ("tied", c_int), ("pool", c_int),
+                ("pool_rows", c_int), ("out_scale", c_float)]
 
 
 def window_attn_args(q, out, pool, page_table, pos, row, *, nq: int, nkv: int, dk: int, dv: int, page_size: int,
                      scale: float, window: int, keep_first: int, bias=None, sink=None, gate=None, softcap=None, q_temp=None,
-                     n_split: int = 1, ws=None, wide_gate=None):
+                     n_split: int = 1, ws=None, wide_gate=None, slope=None, tied: bool = False, factor=None, pooled=None,
+                     block: int = 0, pool_rows: int = 0, out_scale: float = 1.0):
     """Arguments of one windowed attention launch: queries ``q [n, nq * dk]`` (any row pitch) at positions ``pos`` of cache
     rows ``row`` over the paged ``pool`` of the layer that owns the keys; ``softcap``: score cap, ``q_temp = (coef,
-    every)``: query temperature; see ``csrc/attn_window.cu`` for the rule."""
+    every)``: query temperature, ``slope [nq]``: taken off the scores per token of distance; ``tied``: the pool holds keys only,
+    which are the values, with an optional ``factor [pages, page_size]`` of every key's scores, and optional block means
+    ``pooled`` of ``block`` keys each, ``pool_rows`` of them a page; ``out_scale``: factor of the output; see
+    ``csrc/attn_window.cu`` for the rule."""
     a = _WindowAttn()
+    a.tied, a.pool, a.pool_rows, a.out_scale = int(tied), block, pool_rows, out_scale
     ptr = lambda t: 0 if t is None else t.data_ptr()
     a.q, a.out, a.cache, a.page_table, a.pos, a.row = (ptr(t) for t in (q, out, pool, page_table, pos, row))
     a.bias, a.sink, a.gate, a.wide_gate = ptr(bias), ptr(sink), ptr(gate), ptr(wide_gate)
+    a.slope, a.factor, a.pooled = ptr(slope), ptr(factor), ptr(pooled)
     gate = wide_gate if gate is None else gate
     a.n, a.nq, a.nkv, a.dk, a.dv, a.page_size, a.max_pages = q.shape[0], nq, nkv, dk, dv, page_size, page_table.shape[1]
     a.window, a.keep_first, a.far = window, keep_first, 0 if bias is None else bias.shape[1] - 1
@@ -749,20 +796,105 @@ def window_attn_plain(q, out, pool, page_table, pos, row, **kw):
 
 def window_attn_decode(q, out, pool, page_table, pos, row, **kw):
     """Windowed attention of single tokens (bf16, pages of 16): pipelined page copies, optional key splits (``n_split``,
-    ``ws`` of ``n * nq * n_split * (dv + 2)`` floats).  ``bias`` and ``sink`` in log2 units."""
+    ``ws`` of ``n * nq * n_split * (dv + 2)`` floats).  ``bias``, ``sink`` and ``slope`` in log2 units."""
     a = window_attn_args(q, out, pool, page_table, pos, row, **kw)
     _rc(lib().tahb_window_attn_decode(ctypes.byref(a), _stream()), "tahb_window_attn_decode")
     return out
 
 
-def window_attn_tiles(q, out, pool, page_table, pos, row, tile_q0, tile_qn, n_pages: int, kv_ld: int = 0, **kw):
+def window_attn_tiles(q, out, pool, page_table, pos, row, tile_q0, tile_qn, n_pages: int, kv_ld: int = 0, pool_base=None, **kw):
     """Windowed attention of prompt portions on the tensor cores (bf16, pages of 16): tiles of up to 128 consecutive
-    tokens of one row.  ``bias`` and ``sink`` in log2 units.  ``kv_ld``: ``pool`` is not a paged cache but a matrix of that
+    tokens of one row.  ``bias``, ``sink`` and ``slope`` in log2 units.  ``kv_ld``: ``pool`` is not a paged cache but a matrix of that
     pitch whose rows ``[keys of all heads | values of all heads]`` are a token each, 16 of them a page.  ``wide_gate``: gate
-    pre-activations of every output element (``gate``: of every head)."""
+    pre-activations of every output element (``gate``: of every head).  ``pooled`` is then the matrix of :func:`pool_gather`, and
+    ``pool_base`` the first of its pages of 16 rows that belongs to a tile's row."""
     a = window_attn_args(q, out, pool, page_table, pos, row, **kw)
+    pooled = kw.get("pooled")
     _rc(lib().tahb_window_attn_tiles(ctypes.byref(a), _p(tile_q0), _p(tile_qn), c_int(tile_q0.numel()), c_int(n_pages),
-                                     c_ll(kv_ld), _stream()), "tahb_window_attn_tiles")
+                                     c_ll(kv_ld), _p(pool_base), c_int(0 if pooled is None else pooled.shape[0] // 16), _stream()),
+        "tahb_window_attn_tiles")
+    return out
+
+
+class _TiedKeys(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("k", "cache", "pooled", "slot", "pos", "row", "page_table")] + \
+               [(n, c_int) for n in ("M", "nkv", "dk", "page_size", "max_pages", "pool", "pool_rows")] + [("ld", c_ll)]
+
+
+def tied_keys(k, cache, slot, pos, row, page_table, nkv: int, dk: int, page_size: int, pooled=None, block: int = 0, pool_rows: int = 0):
+    """Keys ``k [n, nkv * dk]`` (any row pitch) of a tied layer to the paged cache, and the mean of every block of ``block`` keys
+    that a token completes to its ``pooled`` row."""
+    a = _TiedKeys()
+    for n, t in (("k", k), ("cache", cache), ("pooled", pooled), ("slot", slot), ("pos", pos), ("row", row), ("page_table", page_table)):
+        setattr(a, n, 0 if t is None else t.data_ptr())
+    a.M, a.nkv, a.dk, a.page_size, a.max_pages = k.shape[0], nkv, dk, page_size, page_table.shape[1]
+    a.pool, a.pool_rows, a.ld = block, pool_rows, k.stride(0)
+    _rc(lib().tahb_tied_keys(ctypes.byref(a), c_int(_act_f32(k, cache)), _stream()), "tahb_tied_keys")
+
+
+def pool_gather(pooled, src, nkv: int, dk: int, pool_rows: int, out):
+    """Pooled rows ``src`` (page * pool_rows + row; negative: zeros) one after another: ``out [n, nkv * dk]``."""
+    if out.shape[0] < src.numel() or out.shape[1] != nkv * dk or not out.is_contiguous():
+        raise ValueError(f"pool_gather: {tuple(out.shape)} for {src.numel()} rows of {nkv} x {dk}")
+    _act_f32(pooled, out)
+    _rc(lib().tahb_pool_gather(_p(pooled), _p(src), c_int(src.numel()), c_int(nkv), c_int(dk * pooled.element_size()), c_int(pool_rows),
+                               c_int(pooled.shape[0]), _p(out), _stream()), "tahb_pool_gather")
+    return out
+
+
+class _NormAll(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("q", "k", "w", "q_out", "cache", "factor", "slot")] + \
+               [(n, c_int) for n in ("M", "nq", "nkv", "dk", "dim", "page_size")] + [("ld", c_ll), ("eps", c_float)]
+
+
+def norm_all(q, k, w, q_out, cache, factor, slot, *, nq: int, nkv: int, dk: int, dim: int, page_size: int, eps: float):
+    """RMS norms of q and k over all heads of a token, in a tied layer: ``q_out`` = ``q`` with its norm's factor and the weights
+    ``w [nq * dk]`` of both norms; ``k`` as it is to the paged cache, its norm's factor to ``factor [pages, page_size]``."""
+    a = _NormAll()
+    for n, t in (("q", q), ("k", k), ("w", w), ("q_out", q_out), ("cache", cache), ("factor", factor), ("slot", slot)):
+        setattr(a, n, t.data_ptr())
+    if q.stride(0) != k.stride(0) or not q_out.is_contiguous() or w.numel() != nq * dk:
+        raise ValueError("norm_all: queries and keys of one projection, packed output")
+    a.M, a.nq, a.nkv, a.dk, a.dim, a.page_size, a.ld, a.eps = q.shape[0], nq, nkv, dk, dim, page_size, q.stride(0), eps
+    _rc(lib().tahb_norm_all(ctypes.byref(a), c_int(_act_f32(q, k, q_out, cache)), _stream()), "tahb_norm_all")
+
+
+# -------------------------------------------------------------------------------------------
+# elementwise recurrence (csrc/min_gru.cu)
+# -------------------------------------------------------------------------------------------
+class _MinGru(ctypes.Structure):
+    _fields_ = [(n, c_void_p) for n in ("proj", "zb", "xb", "out", "S", "seq_start", "seq_len", "pos", "row", "slot", "ws")] + \
+               [(n, c_int) for n in ("n", "d", "n_split")] + [("ld", c_ll), ("ld_out", c_ll), ("out_scale", c_float)]
+
+
+def _min_gru_args(proj, zb, xb, out, state, pos, row, out_scale, seq_start=None, seq_len=None, slot=None, n_split=1, ws=None):
+    a = _MinGru()
+    for n, t in (("proj", proj), ("zb", zb), ("xb", xb), ("out", out), ("S", state[0]), ("seq_start", seq_start), ("seq_len", seq_len),
+                 ("pos", pos), ("row", row), ("slot", slot), ("ws", ws)):
+        setattr(a, n, 0 if t is None else t.data_ptr())
+    d = zb.numel()
+    if proj.shape[1] < 3 * d or out.shape[1] < d or state[0].shape[1] != d:
+        raise ValueError(f"min_gru: {d} channels in a projection of {proj.shape[1]}")
+    a.n, a.d, a.n_split, a.ld, a.ld_out, a.out_scale = proj.shape[0], d, n_split, proj.stride(0), out.stride(0), out_scale
+    return a
+
+
+def min_gru_step(proj, zb, xb, out, state, pos, row, out_scale: float, slot=None):
+    """One token per row of ``S <- (1 - z) S + z c(u)``, ``out = out_scale * S * silu(g)``, from columns ``[z | u | g]`` of ``proj``
+    (biases ``zb``, ``xb``); updates ``state = (S [rows, d],)`` in place.  Rows with a negative ``slot`` are left alone."""
+    a = _min_gru_args(proj, zb, xb, out, state, pos, row, out_scale, slot=slot)
+    _rc(lib().tahb_min_gru_step(ctypes.byref(a), c_int(_act_f32(proj, out)), _stream()), "tahb_min_gru_step")
+    return out
+
+
+def min_gru_scan(proj, zb, xb, out, state, pos, row, out_scale: float, *, seq_start, seq_len, n_split: int = 1, ws=None):
+    """The same for portions ``seq_start`` / ``seq_len``, each cut into ``n_split`` segments that run side by side (``ws``: portions
+    * n_split * 2 * d floats)."""
+    a = _min_gru_args(proj, zb, xb, out, state, pos, row, out_scale, seq_start, seq_len, None, n_split, ws)
+    n_seq = seq_start.numel()
+    if n_split > 1 and ws.numel() < n_seq * n_split * 2 * a.d:
+        raise ValueError("min_gru_scan: workspace too small")
+    _rc(lib().tahb_min_gru_scan(ctypes.byref(a), c_int(n_seq), c_int(_act_f32(proj, out)), _stream()), "tahb_min_gru_scan")
     return out
 
 
@@ -825,9 +957,10 @@ def latent_gather(pool, src_pages, page_size: int, row: int, out):
 
 
 def latent_gate(list_v, lists: HeadLists, gate, out, dv: int):
-    """``out[t, h * dv + d] = list_v[h * npad + t, d] * sigmoid(gate[t, h * dv + d])``: back from head lists to token rows."""
-    _rc(lib().tahb_latent_gate(_p(list_v), c_int(lists.npad), c_int(list_v.shape[1]), _p(gate), c_ll(gate.stride(0)), _p(out),
-                               c_ll(out.stride(0)), c_int(lists.n), c_int(lists.heads), c_int(dv), c_int(_act_f32(list_v, gate, out)),
+    """``out[t, h * dv + d] = list_v[h * npad + t, d] * sigmoid(gate[t, h * dv + d])`` (``gate`` None: no factor): back from head
+    lists to token rows."""
+    _rc(lib().tahb_latent_gate(_p(list_v), c_int(lists.npad), c_int(list_v.shape[1]), _p(gate), c_ll(0 if gate is None else gate.stride(0)),
+                               _p(out), c_ll(out.stride(0)), c_int(lists.n), c_int(lists.heads), c_int(dv), c_int(_act_f32(list_v, out)),
                                _stream()), "tahb_latent_gate")
     return out
 
@@ -835,17 +968,17 @@ def latent_gate(list_v, lists: HeadLists, gate, out, dv: int):
 class _LatentAttn(ctypes.Structure):
     _fields_ = [(n, c_void_p) for n in ("q", "out", "cache", "page_table", "pos", "row", "sink")] + \
                [(n, c_int) for n in ("n", "npad", "heads", "Rp", "rw", "lq", "page_size", "max_pages")] + \
-               [("scale", c_float), ("ws", c_void_p), ("n_split", c_int), ("n_pages", c_int), ("status", c_void_p)]
+               [("scale", c_float), ("ws", c_void_p), ("n_split", c_int), ("n_pages", c_int), ("status", c_void_p), ("window", c_int)]
 
 
 def _latent_attn_args(q, out, pool, page_table, pos, row, lists: HeadLists, *, Rp: int, rw: int, page_size: int, scale: float,
-                      sink=None, n_split: int = 1, ws=None):
+                      sink=None, n_split: int = 1, ws=None, window: int = 2 ** 31 - 1):
     a = _LatentAttn()
     ptr = lambda t: 0 if t is None else t.data_ptr()
     a.q, a.out, a.cache, a.page_table, a.pos, a.row, a.sink = (ptr(t) for t in (q, out, pool, page_table, pos, row, sink))
     a.n, a.npad, a.heads, a.Rp, a.rw, a.lq = lists.n, lists.npad, lists.heads, Rp, rw, q.shape[1]
     a.page_size, a.max_pages, a.scale, a.ws, a.n_split = page_size, page_table.shape[1], scale, ptr(ws), n_split
-    a.n_pages, a.status = pool.shape[0], status_word(q.device).data_ptr()
+    a.n_pages, a.status, a.window = pool.shape[0], status_word(q.device).data_ptr(), window
     if n_split > 1 and ws.numel() < lists.n * lists.heads * n_split * (Rp + 2):
         raise ValueError("latent attention: workspace too small")
     return a

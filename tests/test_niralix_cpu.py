@@ -187,7 +187,7 @@ def test_head_lists(n, heads):
 def test_latent_key_splits():
     from types import SimpleNamespace as NS
     from tah_b200.engine.hybrid import latent_splits
-    m = lambda h, tc=True: NS(on_tensor_cores=tc, spec=NS(heads=h))
+    m = lambda h, tc=True: NS(on_tensor_cores=tc, spec=NS(heads=h, window=None))
     assert latent_splits(m(16), 0) == 1 and latent_splits(m(16, False), 4) == 1 and latent_splits(m(16), 1) > 8
     assert all(1 <= latent_splits(m(h), n) <= 16 for h in (1, 16, 17, 128) for n in (1, 7, 64, 256, 1024))
 
@@ -196,18 +196,23 @@ def test_portions_fall_into_launches(monkeypatch):
     """Cache pages of the latent expansions: every portion's pages once, in order, launches within the limit."""
     from types import SimpleNamespace as NS
     from tah_b200.engine import hybrid
+    from tah_b200.engine.hybrid_weights import LatentLayer
     monkeypatch.setattr(hybrid, "LATENT_PAGES", 10)
     table = torch.randperm(200, generator=torch.Generator().manual_seed(0)).view(5, 40).to(torch.int32)
     lens = torch.tensor([70, 16, 161, 0, 33], dtype=torch.int32)
-    eng = NS(device="cpu", page_size=16, kv=NS(page_table=[table], len=[lens], max_pages=[40]))
+    latent = LatentLayer.__new__(LatentLayer)
+    latent.spec, latent.w_exp = NS(window=None), True
+    eng = NS(device="cpu", page_size=16, plain=False, kv=NS(page_table=[table], len=[lens], max_pages=[40]), w=NS(parts=lambda: [latent]))
+    eng._latent_plan = lambda *a: hybrid.HybridEngine._latent_plan(eng, *a)
     plan = hybrid._Plan()
     rows, counts, tiles = [4, 0, 2, 1], [2, 70, 150, 16], [1, 1, 2, 1]
-    hybrid.HybridEngine._latent_plan(eng, plan, rows, counts, tiles, 3 + sum(counts))
+    hybrid.HybridEngine._portion_plan(eng, plan, rows, counts, tiles, 3 + sum(counts))
     need = {4: 3, 0: 5, 2: 11, 1: 1}
-    assert [(a, b, len(s)) for a, b, s in plan.latent] == [(0, 2, 8), (2, 4, 11), (4, 5, 1)] and plan.latent_pages == 11
+    launches, where = plan.latent[None]
+    assert [(a, b, len(s)) for a, b, s in launches] == [(0, 2, 8), (2, 4, 11), (4, 5, 1)] and plan.latent_pages == 11
     flat = torch.cat([table[r, :need[r]] for r in rows])
-    assert torch.equal(torch.cat([s for _, _, s in plan.latent]), flat)
-    assert plan.latent_table[:, 0].tolist() == [0, 3, 0, 0] and plan.latent_table[2, :11].tolist() == list(range(11))
+    assert torch.equal(torch.cat([s for _, _, s in launches]), flat)
+    assert where[:, 0].tolist() == [0, 3, 0, 0] and where[2, :11].tolist() == list(range(11))
     assert plan.portion_of.tolist() == [0] * 3 + [0] * 2 + [1] * 70 + [2] * 150 + [3] * 16
 
 
