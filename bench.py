@@ -498,8 +498,8 @@ def main():
     ap.add_argument("--prompt", type=int, default=PROMPT)
     ap.add_argument("--new-tokens", type=int, default=NEW_TOKENS)
     ap.add_argument("--max-iter", type=int, default=2)
-    ap.add_argument("--family", default="tah", choices=["tah", "gunuvik", "ditilix", "niralix"],
-                    help="gunuvik / ditilix / niralix: prefill / decode of that decoder beside the framework's other models of equal "
+    ap.add_argument("--family", default="tah", choices=["tah", "gunuvik", "ditilix", "niralix", "pidenex"],
+                    help="gunuvik / ditilix / niralix / pidenex: prefill / decode of that decoder beside the framework's other models of equal "
                          "sizes (one GPU)")
     ap.add_argument("--hard-p", default=",".join(str(x) for x in HARD_P), help="comma-separated continue probabilities per depth")
     args = ap.parse_args()

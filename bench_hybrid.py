@@ -3,12 +3,13 @@
     python bench.py --family gunuvik [--model gunuvik-1.7b] [--steps K] [--warmup W]
     python bench.py --family ditilix [--model ditilix-1.7b|ditilix-moe]
     python bench.py --family niralix [--model niralix-1.7b|niralix-moe]
+    python bench.py --family pidenex [--model pidenex-1.7b|pidenex-flat]
 
 Random weights, random token ids, bf16.  All models go through their own engines: ``prefill`` on whole prompts and
 decode ticks (CUDA graph) at a given context, reached with ``fast_forward``.  Comparison models: the plain Qwen3
 backbone (one pass per token, no adapter) with the same width, heads and vocabulary and a feed-forward of 6144, for
-Ditilix also Gunuvik of that size, for Niralix also Gunuvik and the routed Ditilix; ``*_per_layer`` divides by the number of layers, because a recurrent layer has no
-feed-forward of its own.  Device time from CUDA
+Ditilix and Pidenex also Gunuvik of that size, for Niralix also Gunuvik and the routed Ditilix; ``*_per_layer`` divides by the
+number of layer runs, because a recurrent layer has no feed-forward of its own and a layer of a loop runs several times.  Device time from CUDA
 events around K calls after W warm-up calls; every call reads the weights (GBs), far more than the 126 MB L2.
 """
 from __future__ import annotations
@@ -41,10 +42,10 @@ def _qwen3(dev):
 def _layered(name, dev):
     import torch
     from tah_b200.engine import HybridEngine
-    from tah_b200.models import (DitilixForCausalLM, GunuvikForCausalLM, NiralixForCausalLM, ditilix_preset, gunuvik_preset,
-                                 niralix_preset)
+    from tah_b200.models import (DitilixForCausalLM, GunuvikForCausalLM, NiralixForCausalLM, PidenexForCausalLM, ditilix_preset,
+                                 gunuvik_preset, niralix_preset, pidenex_preset)
     cls, preset = {"ditilix": (DitilixForCausalLM, ditilix_preset), "gunuvik": (GunuvikForCausalLM, gunuvik_preset),
-                   "niralix": (NiralixForCausalLM, niralix_preset)}[name.split("-")[0]]
+                   "niralix": (NiralixForCausalLM, niralix_preset), "pidenex": (PidenexForCausalLM, pidenex_preset)}[name.split("-")[0]]
     model = cls(preset(name), dtype=torch.bfloat16, device=dev).init_random()
     return lambda rows: HybridEngine(model, max_rows=rows), model, model.config
 
@@ -87,8 +88,9 @@ def run(args):
     from bench_clocks import ClockSampler
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
-    presets = {"gunuvik": ["gunuvik-1.7b"], "ditilix": ["ditilix-1.7b", "ditilix-moe"], "niralix": ["niralix-1.7b", "niralix-moe"]}
-    beside = {"gunuvik": [], "ditilix": ["gunuvik-1.7b"], "niralix": ["gunuvik-1.7b", "ditilix-moe"]}
+    presets = {"gunuvik": ["gunuvik-1.7b"], "ditilix": ["ditilix-1.7b", "ditilix-moe"], "niralix": ["niralix-1.7b", "niralix-moe"],
+               "pidenex": ["pidenex-1.7b", "pidenex-flat"]}
+    beside = {"gunuvik": [], "ditilix": ["gunuvik-1.7b"], "niralix": ["gunuvik-1.7b", "ditilix-moe"], "pidenex": ["gunuvik-1.7b"]}
     names = [args.model] if args.model.startswith(args.family) else presets[args.family]
     builds = [(n, lambda d, n=n: _layered(n, d)) for n in names + beside[args.family]]
     builds.append(("qwen3 of the same sizes", _qwen3))
@@ -101,7 +103,7 @@ def run(args):
     for label, build in builds:
         torch.manual_seed(0)
         make, model, cfg = build(dev)
-        V, L = cfg.vocab_size, cfg.num_hidden_layers
+        V, L = cfg.vocab_size, len(cfg.layer_runs()) if hasattr(cfg, "layer_runs") else cfg.num_hidden_layers
         rec = {"parameters": sum(p.numel() for p in model.parameters()), "prefill": {}, "decode": {}}
         for B, T in PREFILL:
             eng = make(B)

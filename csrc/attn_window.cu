@@ -20,35 +20,9 @@
 //   score = factor_j * (q' . k_j), value = k_j.
 //   Pooled blocks: a pool of its own under the same page table, with S rows a page ([kv_heads][S][dk], S a power of two >= 16 / P):
 //   block b is row b % S of logical page b / S, a page that the row owns by the time the block is complete.
-#include <cuda.h>
-
-#include "attn_common.cuh"
-#include "common.cuh"
+#include "attn_window.cuh"
 
 namespace tahb {
-
-template <typename T> __device__ __forceinline__ float to_f(T v);
-template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-template <typename T> __device__ __forceinline__ T from_f(float v);
-template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
-
-// 8 consecutive elements as floats (16-byte loads)
-__device__ __forceinline__ void load8(const float* p, float* o) {
-  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-  o[0] = a.x; o[1] = a.y; o[2] = a.z; o[3] = a.w; o[4] = b.x; o[5] = b.y; o[6] = b.z; o[7] = b.w;
-}
-__device__ __forceinline__ void load8(const __nv_bfloat16* p, float* o) {
-  const uint4 u = *reinterpret_cast<const uint4*>(p);
-  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const float2 f = __bfloat1622float2(h[j]);
-    o[2 * j] = f.x;
-    o[2 * j + 1] = f.y;
-  }
-}
 
 // ---------------------------------------------------------------------------------------------
 // Append the tokens of a step to the paged cache.  entry e: `count[e]` further tokens of row `row[e]`, whose packed
@@ -247,206 +221,6 @@ __global__ void __launch_bounds__(128) qkv_post_kernel(const QkvPostParams p) {
 }
 
 // ---------------------------------------------------------------------------------------------
-// Keys of tied layers without norm, bias and rotation, [M, nkv * dk] of pitch ld: to the paged cache, and when a token is the
-// last of a block of P, the mean of the block to the pooled rows.  One warp per (token, head), 8 dims per lane.  The block's other
-// keys come from the projection when they are tokens of the same step (their cache writes may not have happened yet), from the
-// cache otherwise, oldest first: the sum does not depend on how a prompt was cut.
-// ---------------------------------------------------------------------------------------------
-struct TiedKeysParams {
-  const void* k;              // [M, ld]
-  void* cache;                // [pages][nkv][page_size][dk]
-  void* pooled;               // [pages][nkv][pool_rows][dk], or null
-  const int* slot;            // [M], negative = nothing to do
-  const int* pos;
-  const int* row;
-  const int* page_table;      // [rows, max_pages]
-  int M, nkv, dk, page_size, max_pages, pool, pool_rows;
-  long long ld;
-};
-
-template <typename T> struct Row8;
-template <> struct Row8<float> { using type = struct { float4 a, b; }; };
-template <> struct Row8<__nv_bfloat16> { using type = uint4; };
-
-template <typename T>
-__global__ void __launch_bounds__(128) tied_keys_kernel(const TiedKeysParams p) {
-  pdl_launch_dependents();
-  pdl_wait();
-  using R = typename Row8<T>::type;
-  const long long wg = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
-  const int c = (threadIdx.x & 31) * 8;
-  if (wg >= (long long)p.M * p.nkv) return;
-  const int t = (int)(wg / p.nkv), g = (int)(wg % p.nkv), sl = p.slot[t];
-  if (sl < 0 || c >= p.dk) return;
-  const T* src = reinterpret_cast<const T*>(p.k) + (size_t)t * p.ld + (size_t)g * p.dk + c;
-  T* cache = reinterpret_cast<T*>(p.cache);
-  auto at = [&](int page, int off) { return (((size_t)page * p.nkv + g) * p.page_size + off) * p.dk + c; };
-  *reinterpret_cast<R*>(cache + at(sl / p.page_size, sl % p.page_size)) = *reinterpret_cast<const R*>(src);
-  if (p.pooled == nullptr) return;
-  const int i = p.pos[t], r = p.row[t], P = p.pool;
-  if ((i + 1) % P) return;
-  const int* pt = p.page_table + (size_t)r * p.max_pages;
-  float sum[8];
-#pragma unroll
-  for (int e = 0; e < 8; ++e) sum[e] = 0.f;
-#pragma unroll 4
-  for (int k = P - 1; k >= 0; --k) {
-    const bool here = t - k >= 0 && p.row[max(t - k, 0)] == r && p.pos[max(t - k, 0)] == i - k;
-    const T* q = here ? src - (size_t)k * p.ld : cache + at(pt[(i - k) / p.page_size], (i - k) % p.page_size);
-    float v[8];
-    load8(q, v);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) sum[e] += v[e];
-  }
-  const int b = i / P;
-  T* dst = reinterpret_cast<T*>(p.pooled) + (((size_t)pt[b / p.pool_rows] * p.nkv + g) * p.pool_rows + b % p.pool_rows) * p.dk + c;
-#pragma unroll
-  for (int e = 0; e < 8; ++e) dst[e] = from_f<T>(sum[e] / (float)P);
-}
-
-// Pooled rows one after another for the portion kernel: out[r][g * dk + d] = pooled row src[r] (page * pool_rows + row), zeros
-// where src[r] is negative.  16-byte units.
-__global__ void __launch_bounds__(128) pool_gather_kernel(const uint4* __restrict__ pooled, const int* __restrict__ src, int nkv, int units,
-                                                          int pool_rows, int n_pages, uint4* __restrict__ out) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int s = src[blockIdx.x], page = s < 0 ? -1 : s / pool_rows;
-  for (int i = threadIdx.x; i < nkv * units; i += 128) {
-    const int g = i / units, c = i % units;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (page >= 0 && page < n_pages) v = pooled[(((size_t)page * nkv + g) * pool_rows + s % pool_rows) * units + c];
-    out[(size_t)blockIdx.x * nkv * units + i] = v;
-  }
-}
-
-// ---------------------------------------------------------------------------------------------
-// RMS norms of q and k over all heads of a token, for tied layers: q times its factor and the weights of both norms to q_out, the
-// projected k to the paged cache, k's factor to the factors beside it.  One CTA per token.
-// ---------------------------------------------------------------------------------------------
-struct NormAllParams {
-  const void* q;              // [M, ld]: nq heads of dk
-  const void* k;              // the same rows: nkv heads of dk
-  const float* w;             // [nq * dk]: weight of q's norm times that of the key head it meets (padding dims zero)
-  void* q_out;                // [M, nq * dk]
-  void* cache;                // [pages][nkv][page_size][dk]
-  float* factor;              // [pages][page_size]
-  const int* slot;            // [M], negative = no cache write
-  int M, nq, nkv, dk, dim, page_size;
-  long long ld;
-  float eps;
-};
-
-template <typename T>
-__global__ void __launch_bounds__(256) norm_all_kernel(const NormAllParams p) {
-  pdl_launch_dependents();
-  pdl_wait();
-  using R = typename Row8<T>::type;
-  __shared__ float red[2][8];
-  const size_t t = blockIdx.x;
-  const T* q = reinterpret_cast<const T*>(p.q) + t * p.ld;
-  const T* k = reinterpret_cast<const T*>(p.k) + t * p.ld;
-  const int sl = p.slot[t], cq = p.nq * p.dk, ck = p.nkv * p.dk;
-  float sq = 0.f, sk = 0.f;
-  for (int c = threadIdx.x * 8; c < cq; c += 2048) {
-    float v[8];
-    load8(q + c, v);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) sq = fmaf(v[e], v[e], sq);
-  }
-  for (int c = threadIdx.x * 8; c < ck; c += 2048) {
-    float v[8];
-    load8(k + c, v);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) sk = fmaf(v[e], v[e], sk);
-    if (sl >= 0) {
-      const int g = c / p.dk;
-      T* dst = reinterpret_cast<T*>(p.cache) + (((size_t)(sl / p.page_size) * p.nkv + g) * p.page_size + sl % p.page_size) * p.dk + c % p.dk;
-      *reinterpret_cast<R*>(dst) = *reinterpret_cast<const R*>(k + c);
-    }
-  }
-  sq = warp_sum(sq);
-  sk = warp_sum(sk);
-  if ((threadIdx.x & 31) == 0) {
-    red[0][threadIdx.x >> 5] = sq;
-    red[1][threadIdx.x >> 5] = sk;
-  }
-  __syncthreads();
-  sq = sk = 0.f;
-#pragma unroll
-  for (int w = 0; w < 8; ++w) {
-    sq += red[0][w];
-    sk += red[1][w];
-  }
-  if (threadIdx.x == 0 && sl >= 0) p.factor[sl] = 1.0f / sqrtf(sk / (float)(p.nkv * p.dim) + p.eps);
-  const float r = 1.0f / sqrtf(sq / (float)(p.nq * p.dim) + p.eps);
-  for (int c = threadIdx.x * 8; c < cq; c += 2048) {
-    float v[8], w[8];
-    load8(q + c, v);
-    load8(p.w + c, w);
-    T o[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) o[e] = from_f<T>(v[e] * r * w[e]);
-    *reinterpret_cast<R*>(reinterpret_cast<T*>(p.q_out) + t * cq + c) = *reinterpret_cast<const R*>(o);
-  }
-}
-
-// ---------------------------------------------------------------------------------------------
-// What every attention kernel of this file gets.
-// ---------------------------------------------------------------------------------------------
-struct WindowAttnParams {
-  const void* q;              // [n, ld_q], head h at column h * dk
-  void* out;                  // [n, ld_out], head h at column h * dv
-  const void* cache;          // paged cache of the layer that owns the keys
-  const int* page_table;      // [rows, max_pages]
-  const int* pos;             // [n] position of each query
-  const int* row;             // [n] cache row of each query
-  const float* bias;          // [nq, far + 1] bias by distance (the last entry serves every larger distance), or null
-  const float* sink;          // [nq] or null
-  const void* gate;           // pre-activation of head h of query t at gate[t * ld_gate + h], or null
-  const void* wide_gate;      // pre-activation of every output element, gate[t * ld_gate + h * dv + d], or null
-  int n, nq, nkv, dk, dv, page_size, max_pages, window, keep_first, far;
-  long long ld_q, ld_out, ld_gate;
-  float scale;
-  float softcap;              // 0 = no cap
-  float temp_coef;            // 0 = no query temperature
-  double temp_every;
-  float* ws;                  // split partial results (decode kernel, n_split > 1)
-  int n_split;
-  int* status;
-  const float* slope;         // [nq] taken off the scores per token of distance, or null
-  const float* factor;        // [pages][page_size] factor of every key's scores (tied layers), or null
-  const void* pooled;         // pooled blocks of a tied layer (plain and decode kernels: their pool; portion kernel: a matrix), or null
-  int tied;                   // the values are the keys
-  int pool, pool_rows;        // tokens of a pooled block, pooled rows of a page
-  float out_scale;            // factor of the output
-};
-
-// scale of the scores of a query at position i
-__device__ __forceinline__ float query_scale(const WindowAttnParams& p, int i) {
-  if (p.temp_coef == 0.f) return p.scale;
-  return p.scale * (1.0f + p.temp_coef * logf((float)floor((double)(i + 1) / p.temp_every) + 1.0f));
-}
-
-// tanh on the special-function unit, 1 - 2 / (1 + exp(2 x)): absolute error ~2^-22, saturates to +-1
-__device__ __forceinline__ float tanh_sfu(float x) {
-  float r;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + ex2_approx(x * (2.0f * 1.4426950408889634f))));
-  return fmaf(-2.0f, r, 1.0f);
-}
-
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
-
-// First key of the window part, and the end of the kept part in front of it: visible keys are [0, keep_end) and [lo, i].
-__device__ __forceinline__ void visible_range(int i, int window, int keep_first, int& keep_end, int& lo) {
-  lo = i - window + 1;
-  if (window > i) lo = 0;
-  keep_end = min(keep_first, lo);
-}
-
-// pooled blocks that a query at position i sees
-__device__ __forceinline__ int visible_blocks(int i, int window, int pool) { return max(0, i - window + 1) / pool; }
-
-// ---------------------------------------------------------------------------------------------
 // Plain kernel: any head sizes up to 256, bf16 or fp32 cache.  One warp per (query, head); 32 keys at a time, one key
 // per lane for the scores, one dim pair per lane for the weighted values.  Used by the 32-bit mode and for head sizes
 // that the tensor-core and pipelined kernels do not cover.
@@ -559,10 +333,8 @@ __global__ void __launch_bounds__(128) window_attn_plain_kernel(const WindowAttn
 // three-stage ring, warps 0..3 are 16 groups of 8 lanes, one token of a page per group.  Only pages that hold a visible
 // key are visited: the pages of the kept first tokens, then those of the window.  bias and sink are in log2 units.
 // ---------------------------------------------------------------------------------------------
-constexpr int WD_PAGE = 16;
 constexpr int WD_STAGE_PAGES = 2;
 constexpr int WD_NSTAGE = 3;
-constexpr float LOG2E = 1.4426950408889634f;
 
 // pages of a query at position i: `kp` pages of the kept part, then pages w0 .. i / 16; returns their number
 __device__ __forceinline__ int visible_pages(int i, int window, int keep_first, int& kp, int& w0) {
@@ -573,37 +345,14 @@ __device__ __forceinline__ int visible_pages(int i, int window, int keep_first, 
   return kp + max(0, i / WD_PAGE - w0 + 1);
 }
 
-// o = sum / (mass + exp2(sink - m)), times the head's gate; m, mass, sink in log2 units
-__device__ __forceinline__ float finish_scale(const WindowAttnParams& p, int t, int h, float m, float mass) {
-  float f = 1.0f;
-  if (p.sink != nullptr) {
-    const float top = fmaxf(m, p.sink[h]);
-    f = exp2f(m - top);
-    mass = mass * f + exp2f(p.sink[h] - top);
-  }
-  f = mass > 0.f ? f / mass * p.out_scale : 0.f;
-  if (p.gate != nullptr)
-    f *= sigmoid_f(__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(size_t)t * p.ld_gate + h]));
-  return f;
-}
-
-// factor of output element d of head h from its own gate
-__device__ __forceinline__ float element_gate(const WindowAttnParams& p, int t, int h, int d) {
-  if (p.wide_gate == nullptr) return 1.0f;
-  const float z = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.wide_gate)[(size_t)t * p.ld_gate + (size_t)h * p.dv + d]);
-  return __fdividef(1.0f, 1.0f + __expf(-z));
-}
-
-// EXACT: dk = dv = VEC * 64, known to the compiler; CAP: softcap > 0; TIED: pages of keys only, which are the values too, then the
-// page's factors (16 floats), and pooled blocks, 16 of them as one more page, in the place of the kept part
-template <int VEC, int GB, bool EXACT, bool CAP, bool TIED>
+template <int VEC, int GB, bool EXACT, bool CAP>   // EXACT: dk = dv = VEC * 64, known to the compiler; CAP: softcap > 0
 __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) window_decode_kernel(const WindowAttnParams p) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int DPL = VEC * 8;
   const int dk = EXACT ? VEC * 64 : p.dk, dv = EXACT ? VEC * 64 : p.dv;
   extern __shared__ __align__(128) uint8_t wd_smem[];
-  const int kblk = WD_PAGE * dk, vblk = TIED ? 2 * WD_PAGE : WD_PAGE * dv;    // elements of one K / V block of a page (tied: the factors)
+  const int kblk = WD_PAGE * dk, vblk = WD_PAGE * dv;              // elements of one K / V block of a page
   const int stage_elems = WD_STAGE_PAGES * (kblk + vblk);
   __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(wd_smem);
   uint64_t* full_bar = reinterpret_cast<uint64_t*>(wd_smem + (size_t)WD_NSTAGE * stage_elems * 2);
@@ -617,16 +366,8 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
   const int i = p.pos[t];
   const int* pt = p.page_table + (size_t)p.row[t] * p.max_pages;
   int kp, w0;
-  int total = visible_pages(i, p.window, p.keep_first, kp, w0);
+  const int total = visible_pages(i, p.window, p.keep_first, kp, w0);
   const int lo = p.window > i ? 0 : i - p.window + 1;
-  const bool pooled = TIED && p.pooled != nullptr;
-  int blocks = 0;                                                  // pooled blocks, in the first kp pages
-  if (pooled) {
-    blocks = visible_blocks(i, p.window, p.pool);
-    kp = (blocks + WD_PAGE - 1) / WD_PAGE;
-    w0 = lo / WD_PAGE;
-    total = kp + i / WD_PAGE - w0 + 1;
-  }
   const int ppc = (total + p.n_split - 1) / p.n_split;
   const int pb = split * ppc, pe = min(total, pb + ppc);
   const int n_iter = pe > pb ? (pe - pb + WD_STAGE_PAGES - 1) / WD_STAGE_PAGES : 0;
@@ -653,37 +394,7 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
   const int gl = lane & 7;
 
   if (warp == 4) {
-    if constexpr (TIED) {                                          // the lanes share a stage's copies
-      const size_t page_elems = (size_t)p.nkv * kblk;
-      const int S = p.pool_rows, chunk = S * dk;
-      for (int it = 0; it < n_iter; ++it) {
-        const int s = it % WD_NSTAGE, first = pb + it * WD_STAGE_PAGES, n_here = min(WD_STAGE_PAGES, pe - first);
-        if (lane == 0) {
-          mbar_wait(&empty_bar[s], ((it / WD_NSTAGE) & 1) ^ 1, abort_flag, p.status, STATUS_TIMEOUT_STAGE_EMPTY);
-          int bytes = 0;
-          for (int u = 0; u < n_here; ++u) {
-            const int idx = first + u;
-            bytes += pooled && idx < kp ? (min(WD_PAGE, blocks - idx * WD_PAGE) + S - 1) / S * chunk * 2 : kblk * 2 + (p.factor != nullptr ? 64 : 0);
-          }
-          mbar_expect_tx(&full_bar[s], bytes);
-        }
-        __syncwarp();
-        for (int u = 0; u < n_here; ++u) {
-          const int idx = first + u;
-          __nv_bfloat16* dst = stages + (size_t)s * stage_elems + (size_t)u * (kblk + vblk);
-          if (pooled && idx < kp) {                                // S rows a copy
-            const int n = (min(WD_PAGE, blocks - idx * WD_PAGE) + S - 1) / S;
-            if (lane < n)
-              bulk_load(dst + lane * chunk, reinterpret_cast<const __nv_bfloat16*>(p.pooled) + ((size_t)pt[idx * (WD_PAGE / S) + lane] * p.nkv + kvh) * chunk,
-                        chunk * 2, &full_bar[s]);
-          } else if (lane < 2) {
-            const int page = pt[idx < kp ? idx : w0 + idx - kp];
-            if (lane == 0) bulk_load(dst, reinterpret_cast<const __nv_bfloat16*>(p.cache) + (size_t)page * page_elems + (size_t)kvh * kblk, kblk * 2, &full_bar[s]);
-            else if (p.factor != nullptr) bulk_load(dst + kblk, p.factor + (size_t)page * WD_PAGE, 64, &full_bar[s]);
-          }
-        }
-      }
-    } else if (lane == 0) {
+    if (lane == 0) {
       const size_t page_elems = (size_t)p.nkv * (kblk + vblk);
       for (int it = 0; it < n_iter; ++it) {
         const int s = it % WD_NSTAGE;
@@ -722,7 +433,6 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
         for (int e = 0; e < 8; ++e) qv[g][v * 8 + e] = live && c < dk ? __bfloat162float(qp[c + e]) * q_mul : 0.f;
       }
     }
-#pragma unroll 1
     for (int it = 0; it < n_iter; ++it) {
       const int s = it % WD_NSTAGE;
       float b[WD_STAGE_PAGES][GB];
@@ -731,7 +441,7 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
       for (int u = 0; u < WD_STAGE_PAGES; ++u) {          // the biases are fetched while the keys are still on their way
         const int idx = pb + it * WD_STAGE_PAGES + u;
         const int j = (idx < kp ? idx : w0 + idx - kp) * WD_PAGE + grp;
-        ok[u] = idx < pe && (pooled && idx < kp ? j < blocks : j <= i && (j >= lo || j < p.keep_first));
+        ok[u] = idx < pe && j <= i && (j >= lo || j < p.keep_first);
         const int dist = max(i - j, 0);
 #pragma unroll
         for (int g = 0; g < GB; ++g) b[u][g] = bias[g] != nullptr ? __ldg(bias[g] + min(dist, p.far)) : -slope[g] * (float)dist;
@@ -742,8 +452,6 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
 #pragma unroll
       for (int u = 0; u < WD_STAGE_PAGES; ++u) {
         const __nv_bfloat16* kq = st + (size_t)u * (kblk + vblk) + grp * dk;
-        float fac = 1.0f;
-        if (TIED && p.factor != nullptr) fac = reinterpret_cast<const float*>(st + (size_t)u * (kblk + vblk) + kblk)[grp];
         float se[GB], so[GB];
 #pragma unroll
         for (int g = 0; g < GB; ++g) { se[g] = 0.f; so[g] = 0.f; }
@@ -770,7 +478,6 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
           d += __shfl_xor_sync(0xffffffffu, d, 1);
           d += __shfl_xor_sync(0xffffffffu, d, 2);
           d += __shfl_xor_sync(0xffffffffu, d, 4);
-          if constexpr (TIED) d *= fac;
           if constexpr (CAP) d = cap * tanh_sfu(d);
           sc[u][g] = ok[u] ? d + b[u][g] : -INFINITY;
         }
@@ -789,8 +496,7 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
 #pragma unroll
       for (int u = 0; u < WD_STAGE_PAGES; ++u) {
         if (!ok[u]) continue;            // never touch stage memory that holds no visible key
-        const int v_off = TIED ? p.tied - 1 : kblk;              // (0 that the compiler does not know: keys kept in registers would spill)
-        const __nv_bfloat16* vq = st + (size_t)u * (kblk + vblk) + v_off + grp * dv;
+        const __nv_bfloat16* vq = st + (size_t)u * (kblk + vblk) + kblk + grp * dv;
         float pw[GB];
 #pragma unroll
         for (int g = 0; g < GB; ++g) {
@@ -925,13 +631,6 @@ struct WpCfg {
   static constexpr int MIN_CTAS = HK + HV <= 4 ? 2 : 1;
 };
 constexpr int WP_THREADS = 320;
-
-__device__ __forceinline__ void tma_load_4d(void* smem_dst, const void* tmap, int c0, int c1, int c2, int c3, uint64_t* bar) {
-  asm volatile(
-      "cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];"
-      ::"r"(smem_u32(smem_dst)), "l"(reinterpret_cast<uint64_t>(tmap)), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2), "r"(c3)
-      : "memory");
-}
 
 // cap * tanh(mul * v) of 32 scores of a thread.  The arguments of trained attention mostly lie well inside (-1, 1), where
 // x P(x^2) with a degree-5 minimax P (fitted for the absolute error, 3.3e-7 in fp32) needs no special-function unit, the
@@ -1270,48 +969,34 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   }
 }
 
-template <int VEC, int GB, bool EXACT, bool CAP, bool TIED>
+cudaError_t launch_window_merge(const WindowAttnParams& p, cudaStream_t stream) {
+  return launch_chain(window_decode_merge_kernel, dim3(p.n * p.nq), dim3(128), 0, stream, p);
+}
+
+template <int VEC, int GB, bool EXACT, bool CAP>
 static int launch_window_decode_as(const WindowAttnParams& p, cudaStream_t stream) {
   const int groups = (p.nq / p.nkv + GB - 1) / GB;
-  const size_t ring = (size_t)WD_NSTAGE * WD_STAGE_PAGES * WD_PAGE * (p.dk + (TIED ? 2 : p.dv)) * 2 + 128;
+  const size_t ring = (size_t)WD_NSTAGE * WD_STAGE_PAGES * WD_PAGE * (p.dk + p.dv) * 2 + 128;
   const size_t merge = (size_t)16 * GB * (p.dv + 2) * 4;
   const size_t smem = ring > merge ? ring : merge;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(window_decode_kernel<VEC, GB, EXACT, CAP, TIED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
+    if (cudaFuncSetAttribute(window_decode_kernel<VEC, GB, EXACT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
       return -10;
     configured = true;
   }
   if (smem > 160 * 1024) return -11;
-  cudaError_t e = launch_chain(window_decode_kernel<VEC, GB, EXACT, CAP, TIED>, dim3(p.nkv * groups, p.n, p.n_split), dim3(160), smem, stream, p);
-  if (e == cudaSuccess && p.n_split > 1)
-    e = launch_chain(window_decode_merge_kernel, dim3(p.n * p.nq), dim3(128), 0, stream, p);
+  cudaError_t e = launch_chain(window_decode_kernel<VEC, GB, EXACT, CAP>, dim3(p.nkv * groups, p.n, p.n_split), dim3(160), smem, stream, p);
+  if (e == cudaSuccess && p.n_split > 1) e = launch_window_merge(p, stream);
   return e == cudaSuccess ? 0 : -3;
 }
 
 template <int VEC, int GB>
 static int launch_window_decode(const WindowAttnParams& p, cudaStream_t stream) {
   const bool exact = p.dk == VEC * 64 && p.dv == VEC * 64;
-  if (p.tied)
-    return exact ? launch_window_decode_as<VEC, GB, true, false, true>(p, stream) : launch_window_decode_as<VEC, GB, false, false, true>(p, stream);
   if (p.softcap > 0.f)
-    return exact ? launch_window_decode_as<VEC, GB, true, true, false>(p, stream) : launch_window_decode_as<VEC, GB, false, true, false>(p, stream);
-  return exact ? launch_window_decode_as<VEC, GB, true, false, false>(p, stream) : launch_window_decode_as<VEC, GB, false, false, false>(p, stream);
-}
-
-// K (or V) of a paged cache as a 4-D tensor [pages][kv heads][16 tokens][dims], read in boxes of one page's 16 tokens x 64 dims;
-// tok / head / page: strides in elements
-static int make_page_map(CUtensorMap* m, const void* base, int d, int nkv, int n_pages, size_t tok, size_t head, size_t page) {
-  PfEncodeFn fn = pf_encode_fn();
-  if (fn == nullptr) return -1;
-  if ((reinterpret_cast<uintptr_t>(base) & 15) || d % 8 || tok % 8 || head % 8 || page % 8) return -2;
-  cuuint64_t dims[4] = {(cuuint64_t)d, WD_PAGE, (cuuint64_t)nkv, (cuuint64_t)n_pages};
-  cuuint64_t strides[3] = {(cuuint64_t)tok * 2, (cuuint64_t)head * 2, (cuuint64_t)page * 2};
-  cuuint32_t box[4] = {64u, WD_PAGE, 1u, 1u}, estr[4] = {1u, 1u, 1u, 1u};
-  CUresult r = fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr,
-                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? 0 : -3;
+    return exact ? launch_window_decode_as<VEC, GB, true, true>(p, stream) : launch_window_decode_as<VEC, GB, false, true>(p, stream);
+  return exact ? launch_window_decode_as<VEC, GB, true, false>(p, stream) : launch_window_decode_as<VEC, GB, false, false>(p, stream);
 }
 
 template <int HK, int HV, bool CAP, bool TIED = false>
@@ -1352,6 +1037,20 @@ static int make_query_map(CUtensorMap* m, const void* base, int n, long long col
   return r == CUDA_SUCCESS ? 0 : -3;
 }
 
+int check_window_attn(const WindowAttnParams* p) {
+  // tied layers: one size; pooled blocks are a tied layer's, in the place of kept tokens, and have no position
+  if (p->tied && (p->tied != 1 || p->dk != p->dv || p->softcap != 0.f)) return -2;
+  if (!p->tied && (p->factor != nullptr || p->pooled != nullptr)) return -2;
+  if (p->pooled != nullptr && (p->pool < 1 || p->pool_rows < 1 || p->pool_rows > p->page_size || (p->pool_rows & (p->pool_rows - 1)) ||
+                               (long long)p->pool_rows * p->pool < p->page_size || p->keep_first != 0 || p->factor != nullptr || p->slope != nullptr || p->bias != nullptr))
+    return -2;
+  if (p->slope != nullptr && p->bias != nullptr) return -2;
+  if (p->gate != nullptr && p->wide_gate != nullptr) return -2;
+  return p->nkv <= 0 || p->nq % p->nkv || p->dk > 256 || p->dv > 256 || p->dk % 8 || p->dv % 8 || p->window < 1 || p->far < 0 ||
+         p->keep_first < 0 || p->ld_q < (long long)p->nq * p->dk || p->softcap < 0.f ||
+         (p->temp_coef != 0.f && !(p->temp_every > 0.0)) ? -2 : 0;
+}
+
 }  // namespace tahb
 
 using namespace tahb;
@@ -1380,52 +1079,6 @@ extern "C" int tahb_qkv_post(const QkvPostParams* q, int f32, cudaStream_t strea
   return e == cudaSuccess ? 0 : -3;
 }
 
-static int check_window_attn(const WindowAttnParams* p) {
-  // tied layers: one size; pooled blocks are a tied layer's, in the place of kept tokens, and have no position
-  if (p->tied && (p->tied != 1 || p->dk != p->dv || p->softcap != 0.f)) return -2;
-  if (!p->tied && (p->factor != nullptr || p->pooled != nullptr)) return -2;
-  if (p->pooled != nullptr && (p->pool < 1 || p->pool_rows < 1 || p->pool_rows > 16 || (p->pool_rows & (p->pool_rows - 1)) ||
-                               p->pool_rows * p->pool < 16 || p->keep_first != 0 || p->factor != nullptr || p->slope != nullptr || p->bias != nullptr))
-    return -2;
-  if (p->slope != nullptr && p->bias != nullptr) return -2;
-  if (p->gate != nullptr && p->wide_gate != nullptr) return -2;
-  return p->nkv <= 0 || p->nq % p->nkv || p->dk > 256 || p->dv > 256 || p->dk % 8 || p->dv % 8 || p->window < 1 || p->far < 0 ||
-         p->keep_first < 0 || p->ld_q < (long long)p->nq * p->dk || p->softcap < 0.f ||
-         (p->temp_coef != 0.f && !(p->temp_every > 0.0)) ? -2 : 0;
-}
-
-// Keys (and block means) of a tied layer without norms to the cache.
-extern "C" int tahb_tied_keys(const TiedKeysParams* p, int f32, cudaStream_t stream) {
-  if (p->M <= 0) return 0;
-  if (p->dk > 256 || p->dk % 8 || p->ld % 8 || p->nkv < 1 ||
-      (p->pooled != nullptr && (p->pool < 1 || p->pool_rows < 1 || (long long)p->pool_rows * p->pool < p->page_size)))
-    return -2;
-  const long long warps = (long long)p->M * p->nkv;
-  const dim3 grid((unsigned)((warps + 3) / 4));
-  cudaError_t e = f32 ? launch_chain(tied_keys_kernel<float>, grid, dim3(128), 0, stream, *p)
-                      : launch_chain(tied_keys_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, *p);
-  return e == cudaSuccess ? 0 : -3;
-}
-
-// n rows of nkv * row_bytes; src: pooled rows (see pool_gather_kernel)
-extern "C" int tahb_pool_gather(const void* pooled, const int* src, int n, int nkv, int row_bytes, int pool_rows, int n_pages, void* out,
-                                cudaStream_t stream) {
-  if (n <= 0) return 0;
-  if (row_bytes % 16 || nkv < 1 || pool_rows < 1) return -2;
-  cudaError_t e = launch_chain(pool_gather_kernel, dim3(n), dim3(128), 0, stream, reinterpret_cast<const uint4*>(pooled), src, nkv,
-                               row_bytes / 16, pool_rows, n_pages, reinterpret_cast<uint4*>(out));
-  return e == cudaSuccess ? 0 : -3;
-}
-
-// Norms over all heads, queries out, keys and their factors to the cache.
-extern "C" int tahb_norm_all(const NormAllParams* p, int f32, cudaStream_t stream) {
-  if (p->M <= 0) return 0;
-  if (p->dk % 8 || p->dim > p->dk || p->ld % 8 || p->nq < 1 || p->nkv < 1) return -2;
-  cudaError_t e = f32 ? launch_chain(norm_all_kernel<float>, dim3(p->M), dim3(256), 0, stream, *p)
-                      : launch_chain(norm_all_kernel<__nv_bfloat16>, dim3(p->M), dim3(256), 0, stream, *p);
-  return e == cudaSuccess ? 0 : -3;
-}
-
 // Host-side description of one attention launch (same fields as WindowAttnParams).
 extern "C" int tahb_window_attn_plain(const WindowAttnParams* p, int f32, cudaStream_t stream) {
   if (p->n <= 0) return 0;
@@ -1443,6 +1096,7 @@ extern "C" int tahb_window_attn_decode(const WindowAttnParams* p, cudaStream_t s
   if (check_window_attn(p) || p->n > 65535 || p->n_split < 1 || p->n_split > 64) return -2;
   if (p->page_size != WD_PAGE) return -5;
   if (p->n_split > 1 && p->ws == nullptr) return -4;
+  if (p->tied) return launch_tied_decode(*p, stream);
   const int d = p->dk > p->dv ? p->dk : p->dv, vec = d <= 64 ? 1 : d <= 128 ? 2 : 4;
   const int G = p->nq / p->nkv, gb = G == 1 ? 1 : (G == 2 || vec == 4) ? 2 : 4;
 #define TAHB_WD(V_, G_) if (vec == V_ && gb == G_) return launch_window_decode<V_, G_>(*p, stream);

@@ -137,20 +137,17 @@ __global__ void __launch_bounds__(MG_WARPS * 32) min_gru_scan_kernel(const MinGr
       carry = load2(st);
     }
   }
-  const T* x = reinterpret_cast<const T*>(p.proj) + (size_t)first * p.ld + c;
+  const T* x = reinterpret_cast<const T*>(p.proj) + (size_t)first * p.ld + (live ? c : 0);
   T* out = reinterpret_cast<T*>(p.out) + (size_t)first * p.ld_out + c;
   using Raw = typename Pair2<T>::type;
   Raw zr[MG_PER], ur[MG_PER], gr[MG_PER];        // of the next tile, while the one before is at work
-  auto fetch = [&](int t0) {
+  auto fetch = [&](int t0) {                     // unconditional loads, so that all of them are on their way together
 #pragma unroll
     for (int k = 0; k < MG_PER; ++k) {
-      const int t = t0 + warp * MG_PER + k;
-      if (live && t < t_end) {
-        const T* q = x + (size_t)t * p.ld;
-        zr[k] = *reinterpret_cast<const Raw*>(q);
-        ur[k] = *reinterpret_cast<const Raw*>(q + p.d);
-        if constexpr (!SUMMARY) gr[k] = *reinterpret_cast<const Raw*>(q + 2 * p.d);
-      }
+      const T* q = x + (size_t)min(t0 + warp * MG_PER + k, len - 1) * p.ld;
+      zr[k] = *reinterpret_cast<const Raw*>(q);
+      ur[k] = *reinterpret_cast<const Raw*>(q + p.d);
+      if constexpr (!SUMMARY) gr[k] = *reinterpret_cast<const Raw*>(q + 2 * p.d);
     }
   };
   fetch(t_begin);
@@ -160,12 +157,14 @@ __global__ void __launch_bounds__(MG_WARPS * 32) min_gru_scan_kernel(const MinGr
     float4 m = make_float4(1.f, 0.f, 1.f, 0.f);
 #pragma unroll
     for (int k = 0; k < MG_PER; ++k) {
-      if (live && t0 + warp * MG_PER + k < t_end) {
-        const float2 z = widen(zr[k]), u = widen(ur[k]), g = SUMMARY ? make_float2(0.f, 0.f) : widen(gr[k]);
-        token_map<T>(z.x + zb.x, u.x + xb.x, g.x, a[k].x, b[k].x, s[k].x);
-        token_map<T>(z.y + zb.y, u.y + xb.y, g.y, a[k].y, b[k].y, s[k].y);
-        m = make_float4(a[k].x * m.x, fmaf(a[k].x, m.y, b[k].x), a[k].y * m.z, fmaf(a[k].y, m.w, b[k].y));
+      const float2 z = widen(zr[k]), u = widen(ur[k]), g = SUMMARY ? make_float2(0.f, 0.f) : widen(gr[k]);
+      token_map<T>(z.x + zb.x, u.x + xb.x, g.x, a[k].x, b[k].x, s[k].x);
+      token_map<T>(z.y + zb.y, u.y + xb.y, g.y, a[k].y, b[k].y, s[k].y);
+      if (t0 + warp * MG_PER + k >= t_end) {     // behind the segment: S stays what it is
+        a[k] = make_float2(1.f, 1.f);
+        b[k] = make_float2(0.f, 0.f);
       }
+      m = make_float4(a[k].x * m.x, fmaf(a[k].x, m.y, b[k].x), a[k].y * m.z, fmaf(a[k].y, m.w, b[k].y));
     }
     s_map[buf][warp][lane] = m;
     if (t0 + MG_TILE < t_end) fetch(t0 + MG_TILE);

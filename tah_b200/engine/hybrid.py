@@ -70,13 +70,16 @@ def latent_splits(m: LatentLayer, n: int) -> int:
     if n == 0 or not m.on_tensor_cores:
         return 1
     ctas = n * (1 if m.spec.heads <= 16 else (m.spec.heads + 31) // 32)
-    us = 0.02 * (2048 if m.spec.window is None else min(2048, m.spec.window))
-    return min(range(1, 17), key=lambda s: -(-ctas * s // K.SM_COUNT) * (us / s + 3.0))
+    keys = 2048 if m.spec.window is None else min(2048, m.spec.window)
+    return min(range(1, 1 + max(1, min(16, keys // 96))), key=lambda s: -(-ctas * s // K.SM_COUNT) * (0.02 * keys / s + 3.0))
 
 
 def gru_splits(m: MinGRULayer, portions: int, longest: int) -> int:
-    """Segments of a portion in an elementwise recurrence: two CTAs of 64 channels per SM, segments of 256 tokens and more."""
+    """Segments of a portion in an elementwise recurrence (a CTA owns 64 channels of one): segments read the gates twice, so they
+    pay when they fill SMs that would idle; 256 tokens and more each."""
     ctas = portions * ((m.d + 63) // 64)
+    if ctas >= K.SM_COUNT:
+        return 1
     return max(1, min(-(-K.SM_COUNT * 2 // max(1, ctas)), longest // 256, 32))
 
 

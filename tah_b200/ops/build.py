@@ -26,7 +26,7 @@ FLAGS.remove("--use_fast_math")
 
 
 # sources of the smaller libraries that a process may build instead of the whole one
-_DECODER = ("gemm_tcgen05", "elementwise", "sampling", "residual_norm", "attn_window")
+_DECODER = ("gemm_tcgen05", "elementwise", "sampling", "residual_norm", "attn_window", "attn_tied")
 GROUPS = {"gunuvik": _DECODER + ("mlstm",), "ditilix": _DECODER + ("feed_forward",),
           "niralix": _DECODER + ("feed_forward", "gla", "attn_latent"),
           "pidenex": _DECODER + ("feed_forward", "attn_latent", "min_gru")}

@@ -757,7 +757,7 @@ class _WindowAttn(ctypes.Structure):
                [(n, c_int) for n in ("n", "nq", "nkv", "dk", "dv", "page_size", "max_pages", "window", "keep_first", "far")] + \
                [("ld_q", c_ll), ("ld_out", c_ll), ("ld_gate", c_ll), ("scale", c_float), ("softcap", c_float),
                 ("temp_coef", c_float), ("temp_every", ctypes.c_double), ("ws", c_void_p), ("n_split", c_int),
-                ("status", c_void_p), ("slope", c_void_p), ("factor", c_void_p), ("pooled", c_void_p), ("tied", c_int), ("pool", c_int),
+                ("status", c_void_p), ("slope", c_void_p), ("factor", c_void_p), ("pooled", c_void_p), ("tied", c_int), ("n_pages", c_int), ("pool", c_int),
                 ("pool_rows", c_int), ("out_scale", c_float)]
 
 
@@ -772,7 +772,7 @@ def window_attn_args(q, out, pool, page_table, pos, row, *, nq: int, nkv: int, d
     ``pooled`` of ``block`` keys each, ``pool_rows`` of them a page; ``out_scale``: factor of the output; see
     ``csrc/attn_window.cu`` for the rule."""
     a = _WindowAttn()
-    a.tied, a.pool, a.pool_rows, a.out_scale = int(tied), block, pool_rows, out_scale
+    a.tied, a.n_pages, a.pool, a.pool_rows, a.out_scale = int(tied), pool.shape[0], block, pool_rows, out_scale
     ptr = lambda t: 0 if t is None else t.data_ptr()
     a.q, a.out, a.cache, a.page_table, a.pos, a.row = (ptr(t) for t in (q, out, pool, page_table, pos, row))
     a.bias, a.sink, a.gate, a.wide_gate = ptr(bias), ptr(sink), ptr(gate), ptr(wide_gate)

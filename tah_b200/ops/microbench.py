@@ -428,6 +428,10 @@ def main(argv=None):
     ap.add_argument("--rotate", action="store_true", help="qkv_post: rotation and mixed values instead of the norms")
     ap.add_argument("--lists", type=int, default=0, help="latent_query: 1 = into head lists, 0 = in place")
     ap.add_argument("--tau", type=float, default=16.0, help="gated linear attention: decay exponent 1 / tau")
+    ap.add_argument("--block", type=int, default=0, help="tied attention: keys of a pooled block; 0 = key factors and slopes instead")
+    ap.add_argument("--latent-window", type=int, default=0, help="latent attention: window (0 = plain causal)")
+    ap.add_argument("--centered", action="store_true", help="residual_norm: layer norms")
+    ap.add_argument("--enter", action="store_true", help="residual_norm: embedding and a vector added on the way")
     ap.add_argument("--streams", type=int, default=2, help="residual streams")
     ap.add_argument("--plain-glu", action="store_true", help="routed experts: SwiGLU units and softmax scores instead of clamped units")
     ap.add_argument("--experts", type=int, default=0, help="routed experts (--topk per token, --f wide, hidden size --k)")

@@ -1,5 +1,5 @@
-"""Micro-benchmark cases of the layered decoders' kernels (windowed and latent attention, mLSTM, gated linear attention,
-fp32-residual norms, PolyNorm, routed experts); run through :mod:`tah_b200.ops.microbench`, whose timing rules and flags apply.
+"""Micro-benchmark cases of the layered decoders' kernels (windowed, tied and latent attention, mLSTM, gated linear attention,
+minGRU, fp32-residual norms, PolyNorm, xIELU, routed experts); run through :mod:`tah_b200.ops.microbench`, whose timing rules and flags apply.
 
 FLOPs and bytes are those of the algorithm: visible (query, key) pairs for attention, for the chunkwise mLSTM one
 128-token causal block plus the state read-out and update per chunk with every product counted once.
@@ -66,6 +66,114 @@ def bench_window_decode(a):
     keys = B * _visible(T - 1, a)
     res = {"op": "window_decode", "rows": B, "ctx": T, "window": a.window, "n_split": a.nsplit}
     return res, fn, 4.0 * keys * a.nq * a.hd, keys * a.nkv * 2 * a.hd * 2
+
+
+def _tied_kw(a, pages):
+    """Tied layers: ``--block`` P pooled blocks in front of the window, or with 0 key factors and slopes."""
+    from tah_b200.engine.kv_cache import LayerKV
+    kw = dict(nq=a.nq, nkv=a.nkv, dk=a.hd, dv=a.hd, page_size=16, scale=a.hd ** -0.5, window=a.window or 2 ** 31 - 1, keep_first=0, tied=True)
+    if not a.block:
+        return dict(kw, factor=torch.rand(pages, 16, device="cuda"), slope=torch.tensor([2.0 ** (-8 * (h + 1) / a.nq) for h in range(a.nq)], device="cuda"))
+    S = LayerKV(block=a.block).pool_rows(16)
+    return dict(kw, pooled=_bf(pages, a.nkv * S * a.hd), block=a.block, pool_rows=S)
+
+
+def _blocks(i, a):
+    return max(0, i - a.window + 1) // a.block if a.block else 0
+
+
+def bench_tied_prefill(a):
+    """The like of ``window_prefill``: values that are the keys.  FLOPs: visible keys and block means."""
+    B, T, a.keep = a.rows, a.ctx, 0
+    n = B * T
+    pool, pt = _paged(B, T, a.nkv, a.hd, 0)
+    q, out = _bf(n, a.nq * a.hd), torch.empty(n, a.nq * a.hd, dtype=torch.bfloat16, device="cuda")
+    pos = torch.arange(T, device="cuda", dtype=torch.int32).repeat(B)
+    row = torch.arange(B, device="cuda", dtype=torch.int32).repeat_interleave(T)
+    q0 = [b * T + t for b in range(B) for t in range(0, T, 128)]
+    qn = [min(128, T - t) for b in range(B) for t in range(0, T, 128)]
+    kw, per = _tied_kw(a, pool.shape[0]), (_blocks(T - 1, a) + 15) // 16
+    if a.block:
+        kw["pooled"] = _bf(B * per * 16, a.nkv * a.hd) if per else None
+        kw["pool_base"] = _i32([b * per for b in range(B) for _ in range(0, T, 128)])
+    else:
+        kw["wide_gate"] = _bf(n, a.nq * a.hd)
+    q0, qn = _i32(q0), _i32(qn)
+    fn = lambda i: K.window_attn_tiles(q, out, pool, pt, pos, row, q0, qn, pool.shape[0], **kw)
+    pairs = B * sum(_visible(i, a) + _blocks(i, a) for i in range(T))
+    res = {"op": "tied_prefill", "seqs": B, "T": T, "window": a.window, "block": a.block}
+    return res, fn, 4.0 * pairs * a.nq * a.hd, n * (2 * a.nq + a.nkv + (0 if a.block else a.nq)) * a.hd * 2
+
+
+def bench_tied_decode(a):
+    B, T, a.keep = a.rows, a.ctx, 0
+    pool, pt = _paged(B, T, a.nkv, a.hd, 0)
+    q, out, kw = _bf(B, a.nq * a.hd), torch.empty(B, a.nq * a.hd, dtype=torch.bfloat16, device="cuda"), _tied_kw(a, pool.shape[0])
+    if not a.block:
+        kw["wide_gate"] = _bf(B, a.nq * a.hd)
+    pos, row = _i32([T - 1] * B), _i32(list(range(B)))
+    ws = torch.empty(B * a.nq * a.nsplit * (a.hd + 2), device="cuda")
+    fn = lambda i: K.window_attn_decode(q, out, pool, pt, pos, row, n_split=a.nsplit, ws=ws, **kw)
+    keys = B * (_visible(T - 1, a) + _blocks(T - 1, a))
+    res = {"op": "tied_decode", "rows": B, "ctx": T, "window": a.window, "block": a.block, "n_split": a.nsplit}
+    return res, fn, 4.0 * keys * a.nq * a.hd, keys * (a.nkv * a.hd * 2 + (0 if a.block else 4)) + B * a.nq * a.hd * (4 if a.block else 6)
+
+
+def bench_tied_keys(a):
+    """``--m`` tokens of rows of ``--ctx``."""
+    from tah_b200.engine.kv_cache import LayerKV
+    M, T = a.m, min(a.ctx, a.m)
+    pages, S = M // 16, LayerKV(block=a.block or 16).pool_rows(16)
+    k, pool, means = _bf(M, a.nkv * a.hd + 2048), _bf(pages, a.nkv * 16 * a.hd), _bf(pages, a.nkv * S * a.hd)
+    slot = torch.arange(M, device="cuda", dtype=torch.int32)
+    pt, pos, row = torch.arange(pages, device="cuda", dtype=torch.int32).view(M // T, -1), slot % T, slot // T
+    fn = lambda i: K.tied_keys(k, pool, slot, pos, row, pt, a.nkv, a.hd, 16, means, a.block or 16, S)
+    return {"op": "tied_keys", "M": M, "block": a.block or 16}, fn, 0.0, M * a.nkv * a.hd * 4 * (1 + 1 / (a.block or 16))
+
+
+def bench_norm_all(a):
+    M, F = a.m, (a.nq + a.nkv) * a.hd
+    x, q = _bf(M, F + 64), torch.empty(M, a.nq * a.hd, dtype=torch.bfloat16, device="cuda")
+    pages = (M + 15) // 16
+    pool, fac, slot = _bf(pages, a.nkv * 16 * a.hd), torch.empty(pages, 16, device="cuda"), torch.arange(M, device="cuda", dtype=torch.int32)
+    w = torch.ones(a.nq * a.hd, device="cuda")
+    fn = lambda i: K.norm_all(x[:, :a.nq * a.hd], x[:, a.nq * a.hd:F], w, q, pool, fac, slot, nq=a.nq, nkv=a.nkv, dk=a.hd, dim=a.hd, page_size=16, eps=1e-6)
+    return {"op": "norm_all", "M": M}, fn, 0.0, 2 * M * F * 2
+
+
+def _gru_case(a, n, rows):
+    D = a.f
+    x, out = _bf(n, 3 * D), torch.empty(n, D, dtype=torch.bfloat16, device="cuda")
+    return (x, torch.full((D,), -2.0, device="cuda"), torch.zeros(D, device="cuda"), out, (torch.zeros(rows, D, device="cuda"),))
+
+
+def bench_min_gru_scan(a):
+    """``--f`` channels; ``--nsplit`` 0: the engine's choice."""
+    from types import SimpleNamespace
+    from tah_b200.engine.hybrid import gru_splits
+    B, T, D = a.rows, a.ctx, a.f
+    ops = _gru_case(a, B * T, B)
+    pos = torch.arange(T, device="cuda", dtype=torch.int32).repeat(B)
+    row = torch.arange(B, device="cuda", dtype=torch.int32).repeat_interleave(T)
+    split = a.nsplit or gru_splits(SimpleNamespace(d=D), B, T)
+    ws = torch.empty(B * split * 2 * D, device="cuda")
+    start, lens = _i32([b * T for b in range(B)]), _i32([T] * B)
+    fn = lambda i: K.min_gru_scan(*ops, pos, row, 0.7, seq_start=start, seq_len=lens, n_split=split, ws=ws)
+    return {"op": "min_gru_scan", "seqs": B, "T": T, "D": D, "n_split": split}, fn, 0.0, B * T * D * 8 + B * D * 8
+
+
+def bench_min_gru_step(a):
+    B, D = a.rows, a.f
+    ops, pos, row = _gru_case(a, B, B), _i32([5] * B), _i32(list(range(B)))
+    fn = lambda i: K.min_gru_step(*ops, pos, row, 0.7)
+    return {"op": "min_gru_step", "rows": B, "D": D}, fn, 0.0, B * D * 16
+
+
+def bench_xielu_product(a):
+    """The like of a plain product of the same size (``gemm``) and of the SwiGLU product."""
+    x, w, out = _bf(a.m, a.k), _bf(a.f, a.k), torch.empty(a.m, a.f, dtype=torch.bfloat16, device="cuda")
+    fn = lambda i: K.xielu_linear(x, w, 0.9, 1.2, out=out)
+    return {"op": "xielu_product", "M": a.m, "K": a.k, "F": a.f}, fn, 2.0 * a.m * a.k * a.f, (a.m * (a.k + a.f) + a.k * a.f) * 2
 
 
 def _mlstm_case(a, n, rows):
@@ -147,10 +255,12 @@ def bench_latent_decode(a):
     if split == 0:
         from types import SimpleNamespace
         from tah_b200.engine.hybrid import latent_splits
-        split = latent_splits(SimpleNamespace(on_tensor_cores=True, spec=SimpleNamespace(heads=H)), B)
+        split = latent_splits(SimpleNamespace(on_tensor_cores=True, spec=SimpleNamespace(heads=H, window=a.latent_window or None)), B)
     pos, row, ws = _i32([T - 1] * B), _i32(list(range(B))), torch.empty(B * H * split * (R + 2), device="cuda")
-    fn = lambda i: K.latent_attn_decode(q, out, pool, pt, pos, row, L, Rp=R, rw=rw, page_size=16, scale=0.07, sink=sink, n_split=split, ws=ws)
-    return {"op": "latent_decode", "rows": B, "ctx": T, "heads": H, "rank": R, "rot": rw, "n_split": split}, fn, \
+    fn = lambda i: K.latent_attn_decode(q, out, pool, pt, pos, row, L, Rp=R, rw=rw, page_size=16, scale=0.07, sink=sink, n_split=split, ws=ws,
+                                        window=a.latent_window or 2 ** 31 - 1)
+    T = min(T, a.latent_window or T)
+    return {"op": "latent_decode", "rows": B, "ctx": a.ctx, "window": a.latent_window, "heads": H, "rank": R, "rot": rw, "n_split": split}, fn, \
         2.0 * B * T * H * (2 * R + rw), B * T * (R + rw) * 2 + B * H * (2 * R + rw) * 2
 
 
@@ -235,8 +345,9 @@ def bench_residual_norm(a):
     M, W = a.m, a.k
     y, x, h = _bf(M, W), torch.randn(M, W, device="cuda"), torch.empty(M, W, dtype=torch.bfloat16, device="cuda")
     w = torch.full((W,), 0.5, device="cuda")
-    fn = lambda i: K.residual_norm(y, x, w, w, W, 1e-6, h)
-    return {"op": "residual_norm", "M": M, "W": W}, fn, 0.0, M * W * (2 + 8 + 2)
+    enter = dict(add=w, embedding=(_bf(1000, W), torch.randint(0, 1000, (M,), device="cuda").to(torch.int32), 0.5)) if a.enter else {}
+    fn = lambda i: K.residual_norm(y, x, w, w, W, 1e-6, h, centered=a.centered, **enter)
+    return {"op": "residual_norm", "M": M, "W": W, "centered": a.centered, "enter": a.enter}, fn, 0.0, M * W * (2 + 8 + 2)
 
 
 def bench_qkv_post(a):
@@ -347,7 +458,9 @@ def bench_moe_down(a):
     return _moe(a, False)
 
 
-CASES = {"window_prefill": bench_window_prefill, "window_decode": bench_window_decode, "mlstm_chunks": bench_mlstm_chunks,
+CASES = {"tied_prefill": bench_tied_prefill, "tied_decode": bench_tied_decode, "tied_keys": bench_tied_keys, "norm_all": bench_norm_all,
+         "min_gru_scan": bench_min_gru_scan, "min_gru_step": bench_min_gru_step, "xielu_product": bench_xielu_product,
+         "window_prefill": bench_window_prefill, "window_decode": bench_window_decode, "mlstm_chunks": bench_mlstm_chunks,
          "mlstm_step": bench_mlstm_step, "residual_norm": bench_residual_norm, "qkv_post": bench_qkv_post,
          "qk_norm_rope": bench_qk_norm_rope, "few_linear": bench_few_linear, "residual_add_norm": bench_residual_add_norm,
          "poly_norm": bench_poly_norm, "clamped_glu": bench_clamped_glu, "swiglu": bench_swiglu, "moe_route": bench_moe_route,
