@@ -574,25 +574,39 @@ __global__ void __launch_bounds__(160, VEC * GB > 4 ? 2 : GB == 4 ? 3 : 4) windo
   }
 }
 
+// Key splits (up to 64) of a head together, each against the common maximum: one warp weighs the splits, then a dim per thread.
 __global__ void __launch_bounds__(128) window_decode_merge_kernel(const WindowAttnParams p) {
   pdl_launch_dependents();
   pdl_wait();
+  __shared__ float s_w[64];
   const int t = blockIdx.x / p.nq, h = blockIdx.x % p.nq, stride = p.dv + 2;
   const float* w = p.ws + (size_t)blockIdx.x * p.n_split * stride;
-  float mx = -INFINITY, den = 0.f;
-  for (int s = 0; s < p.n_split; ++s) mx = fmaxf(mx, w[s * stride + p.dv]);
-  for (int s = 0; s < p.n_split; ++s) {
-    const float ms = w[s * stride + p.dv];
-    if (ms != -INFINITY) den += exp2f(ms - mx) * w[s * stride + p.dv + 1];
+  if (threadIdx.x < 32) {                        // two splits per lane
+    float m[2], e[2], mx = -INFINITY, den = 0.f;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int s = threadIdx.x + 32 * u;
+      m[u] = s < p.n_split ? w[s * stride + p.dv] : -INFINITY;
+      e[u] = s < p.n_split ? w[s * stride + p.dv + 1] : 0.f;
+      mx = fmaxf(mx, m[u]);
+    }
+    mx = warp_max(mx);
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const float f = m[u] == -INFINITY ? 0.f : exp2f(m[u] - mx);
+      den += f * e[u];
+      e[u] = f;
+    }
+    const float f = finish_scale(p, t, h, mx, warp_sum(den));
+    s_w[threadIdx.x] = e[0] * f;
+    s_w[threadIdx.x + 32] = e[1] * f;
   }
-  const float f = finish_scale(p, t, h, mx, den);
+  __syncthreads();
   for (int d = threadIdx.x; d < p.dv; d += blockDim.x) {
     float num = 0.f;
-    for (int s = 0; s < p.n_split; ++s) {
-      const float ms = w[s * stride + p.dv];
-      if (ms != -INFINITY) num += exp2f(ms - mx) * w[s * stride + d];
-    }
-    reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ld_out + (size_t)h * p.dv + d] = __float2bfloat16_rn(num * f * element_gate(p, t, h, d));
+#pragma unroll 8
+    for (int s = 0; s < p.n_split; ++s) num = fmaf(s_w[s], w[s * stride + d], num);      // an empty split holds zeros
+    reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)t * p.ld_out + (size_t)h * p.dv + d] = __float2bfloat16_rn(num * element_gate(p, t, h, d));
   }
 }
 

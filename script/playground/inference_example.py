@@ -6,7 +6,7 @@
 With ``--random_init`` a tiny random model is used (no download), which is enough to see the
 engine and the colouring at work.
 
-A checkpoint directory of another registered family (``config.json`` decides, e.g. Gunuvik, Ditilix or Niralix) is served by that family's
+A checkpoint directory of another registered family (``config.json`` decides, e.g. Gunuvik, Ditilix, Niralix or Pidenex) is served by that family's
 engine; without a tokenizer in the directory the prompts are token ids, one ``--prompt_ids`` per request:
 
     python script/playground/inference_example.py --model path/to/gunuvik --prompt_ids 5,17,3 --prompt_ids 8,2 --temperature 0

@@ -277,8 +277,9 @@ def bench_latent_prefill(a):
     qn = _i32([min(128, T - t) for b in range(B) for t in range(0, T, 128)])
     sink = torch.randn(H, device="cuda")
     fn = lambda i: K.window_attn_tiles(q, out, kv, pt, pos, row, q0, qn, pages, kv_ld=kv.shape[1], nq=H, nkv=H, dk=dk, dv=dv, page_size=16,
-                                       scale=dk ** -0.5, window=2 ** 31 - 1, keep_first=0, sink=sink, wide_gate=gate)
-    return {"op": "latent_prefill", "seqs": B, "T": T, "heads": H, "dk": dk, "dv": dv}, fn, 1.0 * B * T * (T + 1) * H * (dk + dv), \
+                                       scale=dk ** -0.5, window=a.latent_window or 2 ** 31 - 1, keep_first=0, sink=sink, wide_gate=gate)
+    seen = B * sum(min(i + 1, a.latent_window or T) for i in range(T))
+    return {"op": "latent_prefill", "seqs": B, "T": T, "window": a.latent_window, "heads": H, "dk": dk, "dv": dv}, fn, 2.0 * seen * H * (dk + dv), \
         n * H * (2 * dk + 3 * dv) * 2
 
 
