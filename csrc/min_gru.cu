@@ -57,25 +57,25 @@ __device__ __forceinline__ float rcp_approx(float x) {
   return r;
 }
 constexpr float MG_LOG2E = 1.4426950408889634f;
-// exp(-x), at most 2^40 (a sigmoid stops at 2^-40), so that the product of three of them plus one stays finite
+// exp(-x), at most 2^40 (a sigmoid stops at 2^-40), so that the product of two of them plus one stays finite
 __device__ __forceinline__ float exp_neg(float x) { return ex2_approx(fminf(-x * MG_LOG2E, 40.0f)); }
 
-// The map of a token, S -> a S + b, and the factor of its output.
+// The map of a token, S -> a S + b.
 template <typename T>
-__device__ __forceinline__ void token_map(float z, float u, float g, float& a, float& b, float& s) {
+__device__ __forceinline__ void token_map(float z, float u, float& a, float& b) {
   if constexpr (sizeof(T) == 4) {
-    const float ez = expf(-z), p = 1.0f / (1.0f + ez);
     a = 1.0f / (1.0f + expf(z));
-    b = p * (u >= 0.f ? u + 0.5f : 1.0f / (1.0f + expf(-u)));
-    s = g / (1.0f + expf(-g));
-  } else {                                       // three sigmoids with one reciprocal
-    const float ez = exp_neg(z), eu = exp_neg(u), eg = exp_neg(g);
-    const float dz = 1.0f + ez, du = 1.0f + eu, dg = 1.0f + eg;
-    const float r = rcp_approx(dz * du * dg), p = r * du * dg;
+    b = 1.0f / (1.0f + expf(-z)) * (u >= 0.f ? u + 0.5f : 1.0f / (1.0f + expf(-u)));
+  } else {                                       // two sigmoids with one reciprocal
+    const float ez = exp_neg(z), eu = exp_neg(u), dz = 1.0f + ez, du = 1.0f + eu;
+    const float r = rcp_approx(dz * du), p = r * du;
     a = ez * p;
-    b = p * (u >= 0.f ? u + 0.5f : r * dz * dg);
-    s = g * (r * dz * du);
+    b = p * (u >= 0.f ? u + 0.5f : r * dz);
   }
+}
+template <typename T>
+__device__ __forceinline__ float silu_of(float g) {
+  return sizeof(T) == 4 ? g / (1.0f + expf(-g)) : g * rcp_approx(1.0f + exp_neg(g));
 }
 
 template <typename T>
@@ -89,20 +89,20 @@ __global__ void __launch_bounds__(128) min_gru_step_kernel(const MinGruParams p)
   const float2 zb = load2(p.zb + c), xb = load2(p.xb + c);
   float* st = p.S + (size_t)p.row[t] * p.d + c;
   float2 S = p.pos[t] == 0 ? make_float2(0.f, 0.f) : load2(st);
-  float a, b, s0, s1;
-  token_map<T>(z.x + zb.x, u.x + xb.x, g.x, a, b, s0);
+  float a, b;
+  token_map<T>(z.x + zb.x, u.x + xb.x, a, b);
   S.x = fmaf(a, S.x, b);
-  token_map<T>(z.y + zb.y, u.y + xb.y, g.y, a, b, s1);
+  token_map<T>(z.y + zb.y, u.y + xb.y, a, b);
   S.y = fmaf(a, S.y, b);
   store2(st, S.x, S.y);
-  store2(reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + c, p.out_scale * S.x * s0, p.out_scale * S.y * s1);
+  store2(reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + c, p.out_scale * S.x * silu_of<T>(g.x), p.out_scale * S.y * silu_of<T>(g.y));
 }
 
 constexpr int MG_WARPS = 8, MG_PER = 8, MG_TILE = MG_WARPS * MG_PER, MG_CH = 64;
 
 // Grid (channel blocks, portions, segments).  SUMMARY: only the composition of the segment, to ws.
 template <typename T, bool SUMMARY>
-__global__ void __launch_bounds__(MG_WARPS * 32) min_gru_scan_kernel(const MinGruParams p) {
+__global__ void __launch_bounds__(MG_WARPS * 32, sizeof(T) == 2 ? 2 : 1) min_gru_scan_kernel(const MinGruParams p) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float4 s_map[2][MG_WARPS][32];      // (a, b) of two channels
@@ -141,25 +141,23 @@ __global__ void __launch_bounds__(MG_WARPS * 32) min_gru_scan_kernel(const MinGr
   T* out = reinterpret_cast<T*>(p.out) + (size_t)first * p.ld_out + c;
   using Raw = typename Pair2<T>::type;
   Raw zr[MG_PER], ur[MG_PER], gr[MG_PER];        // of the next tile, while the one before is at work
-  auto fetch = [&](int t0) {                     // unconditional loads, so that all of them are on their way together
+  auto fetch = [&](int t0, int col, Raw* r) {    // unconditional loads, so that all of them are on their way together
 #pragma unroll
-    for (int k = 0; k < MG_PER; ++k) {
-      const T* q = x + (size_t)min(t0 + warp * MG_PER + k, len - 1) * p.ld;
-      zr[k] = *reinterpret_cast<const Raw*>(q);
-      ur[k] = *reinterpret_cast<const Raw*>(q + p.d);
-      if constexpr (!SUMMARY) gr[k] = *reinterpret_cast<const Raw*>(q + 2 * p.d);
-    }
+    for (int k = 0; k < MG_PER; ++k)
+      r[k] = *reinterpret_cast<const Raw*>(x + (size_t)min(t0 + warp * MG_PER + k, len - 1) * p.ld + col);
   };
-  fetch(t_begin);
+  fetch(t_begin, 0, zr);
+  fetch(t_begin, p.d, ur);
+  if constexpr (!SUMMARY) fetch(t_begin, 2 * p.d, gr);
   int buf = 0;
   for (int t0 = t_begin; t0 < t_end; t0 += MG_TILE, buf ^= 1) {
-    float2 a[MG_PER], b[MG_PER], s[MG_PER];
+    float2 a[MG_PER], b[MG_PER];
     float4 m = make_float4(1.f, 0.f, 1.f, 0.f);
 #pragma unroll
     for (int k = 0; k < MG_PER; ++k) {
-      const float2 z = widen(zr[k]), u = widen(ur[k]), g = SUMMARY ? make_float2(0.f, 0.f) : widen(gr[k]);
-      token_map<T>(z.x + zb.x, u.x + xb.x, g.x, a[k].x, b[k].x, s[k].x);
-      token_map<T>(z.y + zb.y, u.y + xb.y, g.y, a[k].y, b[k].y, s[k].y);
+      const float2 z = widen(zr[k]), u = widen(ur[k]);
+      token_map<T>(z.x + zb.x, u.x + xb.x, a[k].x, b[k].x);
+      token_map<T>(z.y + zb.y, u.y + xb.y, a[k].y, b[k].y);
       if (t0 + warp * MG_PER + k >= t_end) {     // behind the segment: S stays what it is
         a[k] = make_float2(1.f, 1.f);
         b[k] = make_float2(0.f, 0.f);
@@ -167,7 +165,10 @@ __global__ void __launch_bounds__(MG_WARPS * 32) min_gru_scan_kernel(const MinGr
       m = make_float4(a[k].x * m.x, fmaf(a[k].x, m.y, b[k].x), a[k].y * m.z, fmaf(a[k].y, m.w, b[k].y));
     }
     s_map[buf][warp][lane] = m;
-    if (t0 + MG_TILE < t_end) fetch(t0 + MG_TILE);
+    if (t0 + MG_TILE < t_end) {
+      fetch(t0 + MG_TILE, 0, zr);
+      fetch(t0 + MG_TILE, p.d, ur);
+    }
     __syncthreads();
     float2 S = carry;
 #pragma unroll
@@ -185,12 +186,13 @@ __global__ void __launch_bounds__(MG_WARPS * 32) min_gru_scan_kernel(const MinGr
 #pragma unroll
       for (int k = 0; k < MG_PER; ++k) {
         const int t = t0 + warp * MG_PER + k;
-        if (live && t < t_end) {
-          S.x = fmaf(a[k].x, S.x, b[k].x);
-          S.y = fmaf(a[k].y, S.y, b[k].y);
-          store2(out + (size_t)t * p.ld_out, p.out_scale * S.x * s[k].x, p.out_scale * S.y * s[k].y);
-        }
+        const float2 g = widen(gr[k]);
+        S.x = fmaf(a[k].x, S.x, b[k].x);
+        S.y = fmaf(a[k].y, S.y, b[k].y);
+        if (live && t < t_end)
+          store2(out + (size_t)t * p.ld_out, p.out_scale * S.x * silu_of<T>(g.x), p.out_scale * S.y * silu_of<T>(g.y));
       }
+      if (t0 + MG_TILE < t_end) fetch(t0 + MG_TILE, 2 * p.d, gr);
     }
   }
   if (!live || warp != 0) return;
